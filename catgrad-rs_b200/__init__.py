@@ -6,6 +6,8 @@ The directory name is not a Python identifier; import it with
 * `backend`  — `CudaBackend`, the mirror of `trait Backend` over the C ABI
 * `graphs`   — the op streams of catgrad's stdlib and catgrad-llm model graphs
 * `decoder`  — the fused, KV-cached greedy runner
+* `layered`  — configurations of models with different mixers per layer (the Ralapel design)
+* `registry` — from a checkpoint folder to a decoder, by the architecture its config.json names
 * `synth`    — seeded synthetic checkpoints and prompts
 * `safetensors_io` — .safetensors checkpoint files: library-side reader, numpy writer
 * `serve`    — the LM / Tokenizer / Loader interfaces of catgrad-llm's serve.rs; `DecoderLM` with prefix reuse
@@ -18,3 +20,5 @@ from .backend import (  # noqa: F401
 )
 from . import graphs, safetensors_io, serve, synth, tp  # noqa: F401
 from .decoder import Decoder, DecoderConfig  # noqa: F401
+from .layered import LayeredConfig, LayerSpec  # noqa: F401
+from . import registry  # noqa: F401

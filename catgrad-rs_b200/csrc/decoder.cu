@@ -27,90 +27,16 @@
 //   x       [ M, H ] f32 residual stream; bf16 only where a tensor-core GEMM reads it
 
 #include <cstring>
-#include <map>
-#include <memory>
-#include <string>
 
-#include "kernels.h"
+#include "decoder.h"
 #include "nccl_dl.h"
 #include "safetensors.h"
 
 using namespace cg;
 
-namespace {
+namespace cg {
 
-struct Layer {
-  cg_tensor *w_qkv = nullptr, *w_o = nullptr, *w_gu = nullptr, *w_down = nullptr;
-  cg_tensor *ln_in = nullptr, *ln_post_attn = nullptr, *ln_pre_ffn = nullptr, *ln_post_ffn = nullptr;
-  cg_tensor *q_norm = nullptr, *k_norm = nullptr;
-  cg_tensor *k_cache = nullptr, *v_cache = nullptr;
-  // mixture-of-experts layers (qwen3.rs:64-133): router [E, H] f32, this rank's experts stacked
-  bool moe = false;
-  cg_tensor *router = nullptr, *router3 = nullptr, *we_gate = nullptr, *we_up = nullptr, *we_down = nullptr;
-};
-
-void drop(cg_tensor*& t) {
-  if (t) release(t);
-  t = nullptr;
-}
-
-}  // namespace
-
-struct cg_decoder {
-  cg_ctx* c = nullptr;
-  cg_decoder_config cfg{};
-  std::map<std::string, cg_tensor*> params;  // as handed over, until finalize
-  bool finalized = false;
-  // sharded sizes
-  int nh = 0, nkv = 0, d = 0, F = 0, Vp = 0, H = 0, qkv = 0;
-  std::vector<Layer> layers;
-  cg_tensor *embed = nullptr, *head = nullptr, *ln_f = nullptr;
-  cg_tensor *cos_t = nullptr, *sin_t = nullptr;
-  cg_tensor *cos_l = nullptr, *sin_l = nullptr;  // tables of the second rope base (gemma3.rs:154-159), or null
-  // state
-  cg_tensor* state = nullptr;     // int64[2] on device: {position, tokens generated}
-  cg_tensor* cur = nullptr;       // u32 [B]: the tokens the next step consumes
-  cg_tensor* history = nullptr;   // u32 [max_batch, max_seq]
-  cg_tensor* logits = nullptr;    // f32 [tp_world, B, Vp]
-  int64_t B = 0, pos = 0, generated = 0;
-  // workspace (sized for `cap` tokens)
-  int64_t cap = 0;
-  cg_tensor *x = nullptr, *xn = nullptr, *qkvb = nullptr, *q = nullptr, *att = nullptr, *hact = nullptr,
-            *tmp = nullptr, *xl = nullptr, *splitk = nullptr, *best = nullptr;
-  // mixture-of-experts scratch, sized for cap * top_k pairs
-  cg_tensor *m_ids = nullptr, *m_wts = nullptr, *m_pos = nullptr, *m_tiles = nullptr, *m_xg = nullptr, *m_h = nullptr,
-            *m_y = nullptr, *m_xs3 = nullptr, *m_logits = nullptr;
-  int El = 0;                    // experts on this rank
-  int EW = 1, ER = 0;            // ranks the experts are split over, and this rank's place among them
-  cg_tensor *ep_x = nullptr, *ep_y = nullptr;  // expert parallelism: every rank's rows gathered / this rank's expert sums for them
-  bool pending_reduce = false;   // x still lacks the addends pushed by the last row-parallel GEMM
-  // norm hand-over (see DecGemm): xn holds bf16(x * gain) un-normalised and ss the per-CTA sums
-  // of squares the last residual GEMM wrote; the next GEMM applies 1 / rms in its epilogue
-  bool xn_raw = false;
-  bool xn_ready = false;         // xn already holds the normalised rows the next GEMM reads (post-norm models)
-  int ss_parts = 0;
-  cg_tensor* ss = nullptr;
-  bool logits_gathered = true;   // `logits` holds every rank's slice
-  cudaGraphExec_t graph = nullptr;
-  int64_t graph_B = -1;
-  int64_t graph_gen = -1;        // option generation the graph was captured under
-  int64_t step_launches = 0;     // kernels in one decode step
-  // all steps of a decode call as one resident kernel (decode_resident.cu), when the model allows
-  ResidentPlan* rplan = nullptr;
-  int64_t rplan_B = -1, rplan_gen = -1;
-  bool resident_off = false;     // this model or device cannot take the resident kernel
-  int64_t splitk_floats = 0;
-
-  int64_t* pos_dev() { return (int64_t*)state->data(); }
-  int64_t* count_dev() { return (int64_t*)state->data() + 1; }
-};
-
-namespace {
-
-int all_reduce_f32(cg_decoder* D, float* p, int64_t n);
-bool use_push(cg_decoder* D, int64_t M, int64_t S);
-
-int get_param(cg_decoder* D, const std::string& name, cg_tensor** out, bool required = true) {
+int get_param(cg_decoder* D, const std::string& name, cg_tensor** out, bool required) {
   auto it = D->params.find(name);
   if (it == D->params.end()) {
     *out = nullptr;
@@ -119,6 +45,38 @@ int get_param(cg_decoder* D, const std::string& name, cg_tensor** out, bool requ
   *out = it->second;
   return CG_OK;
 }
+
+int norm_weight(cg_decoder* D, const std::string& name, int64_t n, cg_tensor** out, bool required) {
+  cg_tensor* p = nullptr;
+  CG_TRY(get_param(D, name, &p, required));
+  if (!p) { *out = nullptr; return CG_OK; }
+  if (p->numel() != n) return fail(D->c, CG_ERR_SHAPE, "decoder: " + name + " has an unexpected shape");
+  return as_contiguous_f32(D->c, p, out);
+}
+
+static __global__ void k_set_state(int64_t* state, int64_t pos, int64_t generated) {
+  state[0] = pos;
+  state[1] = generated;
+}
+
+// The device copy of {position, tokens generated}, set in stream order by a one-thread kernel:
+// no host buffer is involved, so nothing has to be waited for.
+int set_state(cg_decoder* D, int64_t pos, int64_t generated) {
+  k_set_state<<<1, 1, 0, D->c->core->stream>>>((int64_t*)D->state->data(), pos, generated);
+  cudaError_t e = cudaGetLastError();
+  if (e != cudaSuccess) return cuda_fail(D->c, e, "k_set_state");
+  D->c->launches++;
+  D->pos = pos;
+  D->generated = generated;
+  return CG_OK;
+}
+
+}  // namespace cg
+
+namespace {
+
+int all_reduce_f32(cg_decoder* D, float* p, int64_t n);
+bool use_push(cg_decoder* D, int64_t M, int64_t S);
 
 // bf16 copy of rows [r0, r0 + nr) x cols [c0, c0 + nc) of a 2-D parameter, into dst at row `at`
 int copy_block(cg_ctx* c, const cg_tensor* w, int64_t r0, int64_t nr, int64_t c0, int64_t nc, cg_tensor* dst, int64_t at) {
@@ -134,14 +92,6 @@ int copy_block(cg_ctx* c, const cg_tensor* w, int64_t r0, int64_t nr, int64_t c0
   CG_CUDA(c, cudaMemcpyAsync((char*)dst->data() + (size_t)at * nc * 2, cv->data(), (size_t)nr * nc * 2,
                              cudaMemcpyDeviceToDevice, c->core->stream));
   return CG_OK;
-}
-
-int norm_weight(cg_decoder* D, const std::string& name, int64_t n, cg_tensor** out, bool required = true) {
-  cg_tensor* p = nullptr;
-  CG_TRY(get_param(D, name, &p, required));
-  if (!p) { *out = nullptr; return CG_OK; }
-  if (p->numel() != n) return fail(D->c, CG_ERR_SHAPE, "decoder: " + name + " has an unexpected shape");
-  return as_contiguous_f32(D->c, p, out);
 }
 
 int ensure_workspace(cg_decoder* D, int64_t M) {
@@ -562,6 +512,7 @@ int run_head(cg_decoder* D, int64_t B, int64_t S, bool advance) {
 // One decode step for B rows reading position / count from device memory.
 int enqueue_step(cg_decoder* D, int64_t B) {
   cg_ctx* c = D->c;
+  if (D->mixed) return mixed_step(D);
   CG_TRY(k_launch_embed(c, (const uint32_t*)D->cur->data(), 1, 0, 1, D->embed->data(), D->embed->storage, D->cfg.vocab, B,
                         D->H, D->cfg.embed_scale > 0.f ? D->cfg.embed_scale : 1.f, (float*)D->x->data()));
   CG_TRY(run_layers(D, B, 1, 0, true));
@@ -654,23 +605,6 @@ int try_resident(cg_decoder* D, int steps, bool* ran) {
   return CG_OK;
 }
 
-__global__ void k_set_state(int64_t* state, int64_t pos, int64_t generated) {
-  state[0] = pos;
-  state[1] = generated;
-}
-
-// The device copy of {position, tokens generated}, set in stream order by a one-thread kernel:
-// no host buffer is involved, so nothing has to be waited for.
-int set_state(cg_decoder* D, int64_t pos, int64_t generated) {
-  k_set_state<<<1, 1, 0, D->c->core->stream>>>((int64_t*)D->state->data(), pos, generated);
-  cudaError_t e = cudaGetLastError();
-  if (e != cudaSuccess) return cuda_fail(D->c, e, "k_set_state");
-  D->c->launches++;
-  D->pos = pos;
-  D->generated = generated;
-  return CG_OK;
-}
-
 }  // namespace
 
 extern "C" {
@@ -718,9 +652,31 @@ int32_t cg_decoder_create(cg_ctx* c, const cg_decoder_config* cfg, cg_decoder** 
   return CG_OK;
 }
 
+int32_t cg_decoder_create_layers(cg_ctx* c, const cg_decoder_config* cfg, const cg_layer_config* layers, int32_t n_layers,
+                                 const cg_loop_config* loop, cg_decoder** out) {
+  if (!c || !cfg || !layers || n_layers < 1 || !out) return fail(c, CG_ERR_INVALID, "bad argument");
+  const cg_decoder_config& k = *cfg;
+  if (k.hidden <= 0 || k.vocab <= 0 || k.max_seq <= 0 || k.max_batch <= 0) return fail(c, CG_ERR_INVALID, "decoder: sizes must be positive");
+  if (k.tp_world > 1 || k.ep_world > 1)
+    return fail(c, CG_ERR_UNSUPPORTED, "decoder: models built layer by layer run on one GPU (rows can be split over GPUs)");
+  auto* D = new cg_decoder();
+  D->c = c;
+  D->cfg = k;
+  D->cfg.tp_world = 1;
+  D->cfg.tp_rank = 0;
+  D->cfg.num_layers = n_layers;
+  D->H = k.hidden;
+  D->Vp = k.vocab;
+  int st = mixed_create(D, layers, n_layers, loop);
+  if (st != CG_OK) { mixed_destroy(D); delete D; return st; }
+  *out = D;
+  return CG_OK;
+}
+
 int32_t cg_decoder_destroy(cg_decoder* D) {
   if (!D) return CG_ERR_INVALID;
   cudaStreamSynchronize(D->c->core->stream);
+  mixed_destroy(D);
   if (D->graph) cudaGraphExecDestroy(D->graph);
   if (D->rplan) decode_resident_free(D->rplan);
   for (auto& kv : D->params) release(kv.second);
@@ -801,6 +757,7 @@ int32_t cg_decoder_finalize(cg_decoder* D) {
   if (!D) return CG_ERR_INVALID;
   cg_ctx* c = D->c;
   if (D->finalized) return CG_OK;
+  if (D->mixed) return mixed_finalize(D);
   const cg_decoder_config& cfg = D->cfg;
   const int W = cfg.tp_world, R = cfg.tp_rank;
   const int64_t H = D->H, d = D->d;
@@ -972,6 +929,7 @@ int32_t cg_decoder_finalize(cg_decoder* D) {
 
 int32_t cg_decoder_reset(cg_decoder* D) {
   if (!D || !D->finalized) return CG_ERR_INVALID;
+  if (D->mixed) return mixed_reset(D);
   D->B = 0;
   return set_state(D, 0, 0);
 }
@@ -1024,6 +982,10 @@ int32_t cg_decoder_prefill(cg_decoder* D, const cg_tensor* tokens, cg_tensor** l
   CG_LAZY_EAGER_SCOPE(D ? D->c : nullptr);
   if (!D || !tokens) return CG_ERR_INVALID;
   if (!D->finalized) return fail(D->c, CG_ERR_INVALID, "decoder: finalize first");
+  if (D->mixed) {
+    CG_TRY(mixed_prefill(D, tokens, true));
+    return logits_copy(D, logits_out);
+  }
   return prefill_at(D, tokens, 0, 0, logits_out);
 }
 
@@ -1032,6 +994,10 @@ int32_t cg_decoder_append(cg_decoder* D, const cg_tensor* tokens, cg_tensor** lo
   if (!D || !tokens) return CG_ERR_INVALID;
   cg_ctx* c = D->c;
   if (!D->finalized) return fail(c, CG_ERR_INVALID, "decoder: finalize first");
+  if (D->mixed) {
+    CG_TRY(mixed_prefill(D, tokens, D->B == 0));
+    return logits_copy(D, logits_out);
+  }
   if (D->B == 0) return prefill_at(D, tokens, 0, 0, logits_out);  // nothing cached yet
   if (tokens->rank != 2 || tokens->dims[0] != D->B) return fail(c, CG_ERR_SHAPE, "decoder: append needs the cached batch size");
   return prefill_at(D, tokens, D->pos, D->generated, logits_out);
@@ -1039,6 +1005,7 @@ int32_t cg_decoder_append(cg_decoder* D, const cg_tensor* tokens, cg_tensor** lo
 
 int32_t cg_decoder_truncate(cg_decoder* D, int64_t positions) {
   if (!D || !D->finalized) return CG_ERR_INVALID;
+  if (D->mixed) return mixed_truncate(D, positions);
   if (positions < 0 || positions > D->pos) return fail(D->c, CG_ERR_INVALID, "decoder: cannot truncate to more positions than are cached");
   if (positions == 0) D->B = 0;
   return set_state(D, positions, 0);
@@ -1046,7 +1013,8 @@ int32_t cg_decoder_truncate(cg_decoder* D, int64_t positions) {
 
 int32_t cg_decoder_position(cg_decoder* D, int64_t* cached, int64_t* generated) {
   if (!D) return CG_ERR_INVALID;
-  if (cached) *cached = D->pos;
+  if (cached && D->mixed) CG_TRY(mixed_position(D, cached));
+  else if (cached) *cached = D->pos;
   if (generated) *generated = D->generated;
   return CG_OK;
 }
@@ -1055,9 +1023,11 @@ int32_t cg_decoder_decode(cg_decoder* D, int32_t steps, cg_tensor** logits_out) 
   if (!D || steps < 0) return CG_ERR_INVALID;
   cg_ctx* c = D->c;
   if (!D->finalized || D->B == 0) return fail(c, CG_ERR_INVALID, "decoder: prefill first");
-  if (D->pos + steps > D->cfg.max_seq) return fail(c, CG_ERR_SHAPE, "decoder: KV cache capacity exceeded");
+  if (!D->mixed && D->pos + steps > D->cfg.max_seq) return fail(c, CG_ERR_SHAPE, "decoder: KV cache capacity exceeded");
   if (steps == 0) return logits_copy(D, logits_out);
-  {
+  if (D->mixed) CG_TRY(mixed_begin_decode(D, steps));
+  const int asked = steps;
+  if (!D->mixed) {
     bool ran = false;
     CG_TRY(try_resident(D, steps, &ran));
     if (ran) {
@@ -1094,6 +1064,7 @@ int32_t cg_decoder_decode(cg_decoder* D, int32_t steps, cg_tensor** logits_out) 
   c->launches += (int64_t)steps * D->step_launches;  // each replay runs the captured kernels
   D->pos += steps;
   D->generated += steps;
+  if (D->mixed) mixed_advance(D, asked);
   return logits_copy(D, logits_out);
 }
 
@@ -1103,15 +1074,17 @@ int32_t cg_decoder_step_with(cg_decoder* D, const cg_tensor* tokens, cg_tensor**
   cg_ctx* c = D->c;
   if (!D->finalized || D->B == 0) return fail(c, CG_ERR_INVALID, "decoder: prefill first");
   if (tokens->tag != CG_U32 || tokens->numel() != D->B) return fail(c, CG_ERR_SHAPE, "decoder: tokens must be U32 [B]");
-  if (D->pos + 1 > D->cfg.max_seq) return fail(c, CG_ERR_SHAPE, "decoder: KV cache capacity exceeded");
+  if (!D->mixed && D->pos + 1 > D->cfg.max_seq) return fail(c, CG_ERR_SHAPE, "decoder: KV cache capacity exceeded");
   Hold tk;
   CG_TRY(as_contiguous(c, tokens, &tk.t));
+  if (D->mixed) CG_TRY(mixed_begin_decode(D, 1));
   CG_CUDA(c, cudaMemcpyAsync(D->cur->data(), tk.t->data(), (size_t)D->B * 4, cudaMemcpyDeviceToDevice, c->core->stream));
   bool ran = false;
-  CG_TRY(try_resident(D, 1, &ran));
+  if (!D->mixed) CG_TRY(try_resident(D, 1, &ran));
   if (!ran) CG_TRY(enqueue_step(D, D->B));
   D->pos += 1;
   D->generated += 1;
+  if (D->mixed) mixed_advance(D, 1);
   return logits_copy(D, logits_out);
 }
 
@@ -1119,6 +1092,7 @@ int32_t cg_decoder_time_gemms(cg_decoder* D, int32_t batch, int32_t iters, float
   if (!D || !ms_per_sweep || iters < 1) return CG_ERR_INVALID;
   cg_ctx* c = D->c;
   if (!D->finalized) return fail(c, CG_ERR_INVALID, "decoder: finalize first");
+  if (D->mixed) return fail(c, CG_ERR_UNSUPPORTED, "decoder: the GEMM sweep is for attention-only decoders");
   if (batch < 1 || batch > D->cfg.max_batch) return fail(c, CG_ERR_SHAPE, "decoder: batch out of range");
   const int64_t M = batch;
   CG_TRY(ensure_workspace(D, M));

@@ -2,6 +2,7 @@
 // elementwise maps, last-axis reductions, argmax/top-k, gathers and copies, and the f32
 // CUDA-core GEMM that serves as the exact-precision path.  Inputs are arbitrary strided
 // views (broadcast = stride 0, transpose = swapped strides); outputs are contiguous.
+#include "mixers.h"
 #include "runtime.h"
 
 #include <algorithm>
@@ -369,6 +370,7 @@ struct GemmArgs {
   int sta, stb;
   int64_t M, N, K;
   int64_t a_m, a_k, b_k, b_n;
+  int64_t c_m;  // row stride of one output matrix
   int nb;  // batch dims
   int64_t bd[CG_MAX_RANK], ba[CG_MAX_RANK], bb[CG_MAX_RANK];
 };
@@ -443,7 +445,7 @@ __global__ void __launch_bounds__(256) k_gemm_simt(GemmArgs g) {
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       int64_t n = n0 + tx * 4 + j;
-      if (n < g.N) c[m * g.N + n] = acc[i][j];
+      if (n < g.N) c[m * g.c_m + n] = acc[i][j];
     }
   }
 }
@@ -654,6 +656,7 @@ int gemm_simt(cg_ctx* c, const cg_tensor* a, const cg_tensor* b, cg_tensor* out)
   g.M = a->dims[ra - 2];
   g.K = a->dims[ra - 1];
   g.N = b->dims[rb - 1];
+  g.c_m = g.N;
   g.a_m = a->strides[ra - 2];
   g.a_k = a->strides[ra - 1];
   g.b_k = b->strides[rb - 2];
@@ -672,6 +675,21 @@ int gemm_simt(cg_ctx* c, const cg_tensor* a, const cg_tensor* b, cg_tensor* out)
   if (grid.y > 65535) return fail(c, CG_ERR_UNSUPPORTED, "matmul: M too large for the f32 kernel");
   if (a->tag == CG_F32) k_gemm_simt<float><<<grid, 256, 0, c->core->stream>>>(g);
   else k_gemm_simt<uint32_t><<<grid, 256, 0, c->core->stream>>>(g);
+  CG_LAUNCHED(c);
+  return CG_OK;
+}
+
+int gemm_nt_f32(cg_ctx* c, const float* x, int64_t ldx, const float* w, int64_t ldw, float* out, int64_t ldo, int64_t M, int64_t N,
+                int64_t K) {
+  if (M == 0 || N == 0) return CG_OK;
+  GemmArgs g{};
+  g.a = x; g.b = w; g.c = out;
+  g.sta = g.stb = ST_F32;
+  g.M = M; g.N = N; g.K = K;
+  g.a_m = ldx; g.a_k = 1; g.b_k = 1; g.b_n = ldw; g.c_m = ldo;
+  dim3 grid((unsigned)((N + 63) / 64), (unsigned)((M + 63) / 64), 1);
+  if (grid.y > 65535) return fail(c, CG_ERR_UNSUPPORTED, "matmul: M too large for the f32 kernel");
+  k_gemm_simt<float><<<grid, 256, 0, c->core->stream>>>(g);
   CG_LAUNCHED(c);
   return CG_OK;
 }

@@ -1,0 +1,189 @@
+// mixed_rows.cu — the residual stream of decoders built layer by layer: embedding, post-norm add,
+// next pre-norm and the two-part rows of a looped input in one pass; plus the f32 GEMM entry those
+// decoders use in an f32 context.
+#include <algorithm>
+
+#include "act.cuh"
+#include "mixers.h"
+
+namespace cg {
+
+namespace {
+
+__device__ __forceinline__ float warp_sum(float v) {
+#pragma unroll
+  for (int o = 16; o; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+  return v;
+}
+__device__ __forceinline__ float block_sum(float v, float* sh) {
+  const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  v = warp_sum(v);
+  __syncthreads();
+  if (lane == 0) sh[wid] = v;
+  __syncthreads();
+  v = lane < nw ? sh[lane] : 0.f;
+  return warp_sum(v);
+}
+__device__ __forceinline__ void store4(float* p, const float* v) { *(float4*)p = make_float4(v[0], v[1], v[2], v[3]); }
+__device__ __forceinline__ void store4(__nv_bfloat16* p, const float* v) {
+  const __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
+  *(uint2*)p = make_uint2(*(const uint32_t*)&lo, *(const uint32_t*)&hi);
+}
+
+constexpr int RU_VEC = 4;  // 128-bit vectors a thread keeps
+
+// One block per row; the row lives in registers (four values per vector, RU_VEC vectors per thread).
+template <class T>
+__global__ void k_row_update(RowUpdate u, int32_t* err) {
+  asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+  asm volatile("griddepcontrol.wait;" ::: "memory");
+  __shared__ float sh[32];
+  const int64_t m = blockIdx.x;
+  const int W = u.W, n4 = (W + 7) / 8 * 2;
+  const int nv = (n4 + blockDim.x - 1) / blockDim.x;
+  float v[RU_VEC][4];
+  if (u.pick) {
+    const float* row = u.x + (int64_t)u.pick[m] * u.ldx;
+#pragma unroll
+    for (int j = 0; j < RU_VEC; ++j) {
+      const int i = threadIdx.x + j * blockDim.x;
+      const float4 t = j < nv && i < n4 ? *(const float4*)(row + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f);
+      v[j][0] = t.x; v[j][1] = t.y; v[j][2] = t.z; v[j][3] = t.w;
+    }
+  } else {
+    uint32_t tok = 0;
+    if (u.tokens) {
+      tok = u.tokens[m];
+      if (tok >= u.vocab) { if (threadIdx.x == 0) *err = DEV_INDEX; tok = 0; }
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < RU_VEC; ++j) {
+      const int i = threadIdx.x + j * blockDim.x;
+      v[j][0] = v[j][1] = v[j][2] = v[j][3] = 0.f;
+      if (j < nv && i < n4) {
+        if (u.tokens) {
+          const int64_t o = (int64_t)tok * W + 4 * i;
+#pragma unroll
+          for (int e = 0; e < 4; ++e)
+            if (4 * i + e < W)
+              v[j][e] = u.table_bf16 ? __bfloat162float(((const __nv_bfloat16*)u.table)[o + e]) : ((const float*)u.table)[o + e];
+        } else {
+          const float4 t = *(const float4*)(u.y + m * u.ldy + 4 * i);
+          v[j][0] = t.x; v[j][1] = t.y; v[j][2] = t.z; v[j][3] = t.w;
+#pragma unroll
+          for (int e = 0; e < 4; ++e)
+            if (4 * i + e >= W) v[j][e] = 0.f;
+        }
+      }
+#pragma unroll
+      for (int e = 0; e < 4; ++e) ss += v[j][e] * v[j][e];
+    }
+    if (u.g1) {
+      ss = block_sum(ss, sh);
+      const float rms = sqrtf(ss / (float)W + u.eps);
+#pragma unroll
+      for (int j = 0; j < RU_VEC; ++j) {
+        const int i = threadIdx.x + j * blockDim.x;
+        if (j < nv && i < n4)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) v[j][e] = 4 * i + e < W ? v[j][e] / rms * u.g1[4 * i + e] : 0.f;
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < RU_VEC; ++j) {
+      const int i = threadIdx.x + j * blockDim.x;
+      if (j < nv && i < n4) {
+        float* xp = u.x + m * u.ldx + 4 * i;
+        if (u.add) {
+          const float4 t = *(const float4*)xp;
+          v[j][0] += t.x; v[j][1] += t.y; v[j][2] += t.z; v[j][3] += t.w;
+        }
+        store4(xp, v[j]);
+      }
+    }
+  }
+  if (u.x0)
+#pragma unroll
+    for (int j = 0; j < RU_VEC; ++j) {
+      const int i = threadIdx.x + j * blockDim.x;
+      if (j < nv && i < n4) store4((T*)u.x0 + m * u.ld0 + 4 * i, v[j]);
+    }
+  if (!u.out) return;
+  const int64_t mo = u.dst ? u.dst[m] : m;
+  if (u.g2) {
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < RU_VEC; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) ss += v[j][e] * v[j][e];
+    ss = block_sum(ss, sh);
+    const float rms = sqrtf(ss / (float)W + u.eps);
+#pragma unroll
+    for (int j = 0; j < RU_VEC; ++j) {
+      const int i = threadIdx.x + j * blockDim.x;
+      if (j < nv && i < n4)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) v[j][e] = 4 * i + e < W ? v[j][e] / rms * u.g2[4 * i + e] : 0.f;
+    }
+  }
+#pragma unroll
+  for (int j = 0; j < RU_VEC; ++j) {
+    const int i = threadIdx.x + j * blockDim.x;
+    if (j < nv && i < n4) store4((T*)u.out + mo * u.ldo + 4 * i, v[j]);
+  }
+}
+
+__global__ void k_glu_f32(const float* gu, int64_t F, int act, float* out) {
+  asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+  asm volatile("griddepcontrol.wait;" ::: "memory");
+  const int64_t m = blockIdx.y;
+  const float c = 0.7978845608028654f;  // sqrt(2 / pi)
+  for (int64_t i = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; i < F; i += (int64_t)gridDim.x * blockDim.x) {
+    const float z = gu[m * 2 * F + i];
+    const float a = act == 0 ? z / (1.f + expf(-z)) : 0.5f * z * (1.f + tanhf(c * (z + 0.044715f * z * z * z)));
+    out[m * F + i] = a * gu[m * 2 * F + F + i];
+  }
+}
+
+__global__ void k_pair_rope_tables(double base, int64_t T, int r, float* cos_t, float* sin_t) {
+  const int half = r / 2;
+  const int64_t n = T * half;
+  for (int64_t i = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; i < n; i += (int64_t)gridDim.x * blockDim.x) {
+    const int64_t p = i / half;
+    const int k = (int)(i - p * half);
+    const double a = (double)p * pow(base, -2.0 * k / r);
+    cos_t[i] = (float)cos(a);
+    sin_t[i] = (float)sin(a);
+  }
+}
+
+}  // namespace
+
+int k_launch_row_update(cg_ctx* c, const RowUpdate& u, int64_t M, int out_bf16) {
+  if (M == 0) return CG_OK;
+  const int n4 = (u.W + 7) / 8 * 2;
+  int block = (n4 + 31) / 32 * 32;
+  while (block > 256 && (n4 + block / 2 - 1) / (block / 2) <= (M > 296 ? RU_VEC : 1)) block = (block / 2 + 31) / 32 * 32;
+  block = std::min(block, 1024);
+  if ((int64_t)block * RU_VEC < n4) return fail(c, CG_ERR_UNSUPPORTED, "decoder: rows wider than 16384 are not supported");
+  if (out_bf16) CG_CUDA(c, launch_kernel(c, k_row_update<__nv_bfloat16>, dim3((unsigned)M), dim3(block), 0, 1, u, c->core->dev_err));
+  else CG_CUDA(c, launch_kernel(c, k_row_update<float>, dim3((unsigned)M), dim3(block), 0, 1, u, c->core->dev_err));
+  CG_LAUNCHED(c);
+  return CG_OK;
+}
+
+int k_launch_glu_f32(cg_ctx* c, const float* gu, int64_t M, int64_t F, int act, float* out) {
+  if (M == 0) return CG_OK;
+  CG_CUDA(c, launch_kernel(c, k_glu_f32, dim3(grid_for(F, 256, 64), (unsigned)M), dim3(256), 0, 1, gu, F, act, out));
+  CG_LAUNCHED(c);
+  return CG_OK;
+}
+
+int k_launch_pair_rope_tables(cg_ctx* c, double base, int64_t T, int r, float* cos_t, float* sin_t) {
+  k_pair_rope_tables<<<grid_for(T * (r / 2), 256), 256, 0, c->core->stream>>>(base, T, r, cos_t, sin_t);
+  CG_LAUNCHED(c);
+  return CG_OK;
+}
+
+}  // namespace cg

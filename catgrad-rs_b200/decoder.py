@@ -11,6 +11,7 @@ import ctypes as C
 import numpy as np
 
 from .backend import CudaBackend, TaggedTensor, U32, _c_vp
+from .layered import LayerStruct, LayeredConfig, LoopStruct
 
 
 class DecoderConfig(C.Structure):
@@ -33,6 +34,8 @@ class DecoderConfig(C.Structure):
 
 
 class Decoder:
+    _h = None
+
     def __init__(self, backend: CudaBackend, cfg, max_seq: int, max_batch: int, tp_rank: int = 0, tp_world: int = 1,
                  ep_rank: int = 0, ep_world: int = 1, **switches):
         self.B = backend
@@ -55,11 +58,32 @@ class Decoder:
             ("cg_decoder_tokens", [vp, out]),
             ("cg_decoder_generate", [vp, vp, i32, i32, i32, vp]),
             ("cg_decoder_time_gemms", [vp, i32, i32, C.POINTER(C.c_float), C.POINTER(i32)]),
+            ("cg_decoder_create_layers", [vp, C.POINTER(DecoderConfig), C.POINTER(LayerStruct), i32, C.POINTER(LoopStruct), out]),
+            ("cg_decoder_seq_open", [vp, C.POINTER(i32)]),
+            ("cg_decoder_seq_close", [vp, i32]),
+            ("cg_decoder_run", [vp, i32, vp, vp, vp, i32, vp, i32, out]),
+            ("cg_decoder_keep_residuals", [vp, i32]),
+            ("cg_decoder_residuals", [vp, out]),
         ]:
             fn = getattr(L, name)
             fn.argtypes = args
             fn.restype = i32
         c = DecoderConfig()
+        # a cached prefix can be shortened to any length (a recurrent state cannot go back)
+        self.keeps_prefix = not isinstance(cfg, LayeredConfig)
+        if isinstance(cfg, LayeredConfig):
+            c.num_layers, c.hidden, c.vocab = len(cfg.layers), cfg.hidden_size, cfg.vocab_size
+            c.rms_eps, c.max_seq, c.max_batch = cfg.rms_norm_eps, max_seq, max_batch
+            c.tp_rank, c.tp_world, c.ep_rank, c.ep_world = tp_rank, tp_world, ep_rank, ep_world
+            for k, v in switches.items():
+                setattr(c, k, v)
+            self.cfg = c
+            layers = (LayerStruct * len(cfg.layers))(*[s.struct() for s in cfg.layers])
+            loop = C.byref(LoopStruct(*cfg.loop)) if cfg.loop else None
+            h = vp()
+            backend._check(L.cg_decoder_create_layers(backend._ctx, C.byref(c), layers, len(layers), loop, C.byref(h)))
+            self._h = h
+            return
         c.arch = 0
         c.num_layers = cfg.num_hidden_layers
         c.hidden = cfg.hidden_size
@@ -148,7 +172,10 @@ class Decoder:
         import zlib
         gain = 0.0 if getattr(cfg, "arch", "llama") == "gemma" else 1.0
         for name, shape in synth.param_shapes(cfg).items():
-            if len(shape) == 1:
+            if isinstance(cfg, LayeredConfig):
+                mean, sd = cfg.synthetic(name)
+                t = self.B.randn(shape, (seed << 32) ^ zlib.crc32(name.encode()), std=sd, mean=mean)
+            elif len(shape) == 1:
                 t = self.B.randn(shape, 0, std=0.0, mean=gain)
             else:
                 t = self.B.randn(shape, (seed << 32) ^ zlib.crc32(name.encode()), std=std)
@@ -198,6 +225,50 @@ class Decoder:
 
     def step_with(self, tokens: TaggedTensor, want_logits=False):
         return self._maybe_logits(self.B._lib.cg_decoder_step_with, tokens._h, want_logits=want_logits)
+
+    # -- sequences of unequal length (decoders built from a LayeredConfig) ----------------
+    def open_sequence(self) -> int:
+        """A free slot, empty."""
+        s = C.c_int32()
+        self.B._check(self.B._lib.cg_decoder_seq_open(self._h, C.byref(s)))
+        return s.value
+
+    def close_sequence(self, slot: int):
+        self.B._check(self.B._lib.cg_decoder_seq_close(self._h, int(slot)))
+
+    def run(self, rows, want=(), greedy: bool = False) -> TaggedTensor | None:
+        """One batch: rows = [(slot, next tokens)], of any lengths.  `want` lists (row, place among the
+        row's new tokens) in ascending order; the logits there come back as [len(want), vocab].  With
+        greedy the rows become the current rows and `decode` continues them together."""
+        slots = np.asarray([s for s, _ in rows], dtype=np.int32)
+        lens = np.asarray([len(t) for _, t in rows], dtype=np.int32)
+        toks = np.concatenate([np.asarray(t, dtype=np.uint32).reshape(-1) for _, t in rows])
+        first = np.concatenate([[0], np.cumsum(lens)])
+        w = np.asarray([first[r] + i for r, i in want], dtype=np.int32)
+        h = _c_vp()
+        self.B._check(self.B._lib.cg_decoder_run(self._h, len(rows), slots.ctypes.data, lens.ctypes.data, toks.ctypes.data, len(w),
+                                                 w.ctypes.data if len(w) else None, int(greedy), C.byref(h)))
+        return self.B._wrap(h) if len(w) else None
+
+    def generate_batch(self, prompts, n_decode: int) -> np.ndarray:
+        """Greedy generation for prompts of unequal length as one batch: [rows, 1 + n_decode] ids."""
+        slots = [self.open_sequence() for _ in prompts]
+        try:
+            self.run([(s, p) for s, p in zip(slots, prompts)], greedy=True)
+            self.decode(n_decode)
+            return self.tokens()
+        finally:
+            for s in slots:
+                self.close_sequence(s)
+
+    def keep_residuals(self, on: bool = True):
+        self.B._check(self.B._lib.cg_decoder_keep_residuals(self._h, int(on)))
+
+    def residuals(self) -> np.ndarray:
+        """[layer runs, tokens, hidden]: the residual stream after every layer run of the last batch."""
+        h = _c_vp()
+        self.B._check(self.B._lib.cg_decoder_residuals(self._h, C.byref(h)))
+        return self.B.to_numpy(self.B._wrap(h))
 
     def tokens(self) -> np.ndarray:
         h = _c_vp()

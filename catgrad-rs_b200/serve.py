@@ -8,7 +8,8 @@ returns the greedy next token, `None` (StopIteration) at an end-of-sequence toke
 differences: the cache lives on the device inside the decoder instead of being passed in and out
 of the graph, and `set_context` keeps the longest common prefix of the old and the new context
 (the reference keeps its cache only when the new context extends the whole old one, and says so
-in a PERFORMANCE note at run.rs:296).  `Tokenizer` / `ChatTokenizer` / `Loader` are the
+in a PERFORMANCE note at run.rs:296); a decoder with recurrent layers keeps its state only when the new
+context extends the old one.  `Tokenizer` / `ChatTokenizer` / `Loader` are the
 abstract interfaces only: tokenizers are outside this library.
 """
 from __future__ import annotations
@@ -97,6 +98,8 @@ class DecoderLM(LM):
         n = longest_common_prefix(self.cached, context)
         if n == len(context) and n > 0:
             n -= 1                      # at least one token must be run to get a next token
+        if n < len(self.cached) and not self.dec.keeps_prefix:
+            n = 0                       # a recurrent state has no earlier versions
         if n < len(self.cached):
             self.dec.truncate(n)        # forget only what differs
             self.cached = self.cached[:n]

@@ -81,6 +81,8 @@ def param_shapes(cfg: ModelConfig) -> dict[str, tuple[int, ...]]:
     """Hugging Face tensor names and shapes of a checkpoint (all weights [out, in]); experts are
     already stacked [E, ...] the way the reference driver stacks them
     (catgrad-llm/examples/llama/main.rs:173-264)."""
+    if cfg.arch == "layered":
+        return cfg.param_shapes()
     H, F, d = cfg.hidden_size, cfg.intermediate_size, cfg.head_dim
     nh, nkv = cfg.num_attention_heads, cfg.num_key_value_heads
     shapes = {"model.embed_tokens.weight": (cfg.vocab_size, H), "model.norm.weight": (H,)}
@@ -128,7 +130,12 @@ def make_weights(cfg: ModelConfig, seed: int = 0, std: float = 0.02):
     shapes = param_shapes(cfg)
     for name in sorted(shapes):
         shp = shapes[name]
-        if len(shp) == 1:
+        if cfg.arch == "layered":
+            mean, sd = cfg.synthetic(name)
+            w = np.float32(mean) + rng.standard_normal(shp, dtype=np.float32) * np.float32(sd)
+            if cfg.dtype == "bf16" and len(shp) > 1:
+                w = bf16_round(w)
+        elif len(shp) == 1:
             # norm gains: an effective gain of 1 (gemma multiplies by 1 + gamma, so gamma = 0)
             w = np.zeros(shp, dtype=np.float32) if cfg.arch == "gemma" else np.ones(shp, dtype=np.float32)
         else:

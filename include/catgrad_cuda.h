@@ -384,6 +384,68 @@ int32_t cg_decoder_tokens(cg_decoder*, cg_tensor** out);
 int32_t cg_decoder_generate(cg_decoder*, const uint32_t* prompt, int32_t batch, int32_t seq,
                             int32_t n_decode, uint32_t* out);
 
+/* --- decoders built layer by layer: layers with different sequence mixers, optionally run in a loop.
+ * No counterpart in the reference, whose decoders are attention-only.  Every layer is
+ *   x <- x + norm1b(mixer(norm1(x))),  x <- x + norm2b(ff(norm2(x)))
+ * with RMS norms (the second line only where the layer has a feed-forward), a gated feed-forward
+ * down(act(gate h) * up h), a normed embedding and a norm before the head.  The residual stream,
+ * norms, positions, attention weights and everything inside a recurrence are f32.  The context's
+ * precision decides the rest: CG_PREC_BF16 runs the tensor-core kernels on bf16 weights and
+ * activations, CG_PREC_F32 runs everything in f32. */
+typedef enum cg_mixer {
+  CG_MIX_LATENT = 1, /* latent attention: keys and values are linear maps of a cached low-rank row */
+  CG_MIX_DELTA = 2,  /* gated delta rule behind short convolutions */
+  CG_MIX_SSD = 3     /* Mamba-2: scalar-decay state space with a gated group norm */
+} cg_mixer;
+typedef struct cg_layer_config {
+  int32_t mixer;     /* cg_mixer */
+  int32_t ffn;       /* width of the gated feed-forward, 0 = none */
+  int32_t act;       /* 0 silu, 1 tanh gelu */
+  int32_t heads;     /* latent: query heads; delta, ssd: value heads */
+  int32_t kv_heads;  /* delta: query/key heads, a divisor of heads */
+  int32_t dim;       /* latent: unrotated query/key size per head; delta: query/key size per head */
+  int32_t rot_dim;   /* latent: rotated query/key size, the key part shared by all heads */
+  int32_t vdim;      /* value size per head */
+  int32_t kv_rank;   /* latent: size of the cached row without its rotated part */
+  int32_t state;     /* ssd: state size (the key size of the recurrence) */
+  int32_t groups;    /* ssd: groups of heads sharing B and C */
+  int32_t norm_groups; /* ssd: equal parts of the gated norm */
+  int32_t conv;      /* delta, ssd: taps of the short convolutions */
+  double rot_base;   /* latent: base of the rotary frequencies; neighbouring components are paired */
+  double scale;      /* latent: factor on the scores */
+} cg_layer_config;
+typedef struct cg_loop_config {
+  int32_t start, stop, times; /* layers [start, stop) run `times` times in a row, each pass with its own cache or
+                                 state; before a pass x <- W [x; x0], x0 the normed embedding */
+} cg_loop_config;
+/* cfg supplies hidden, vocab, rms_eps, max_seq (capacity per sequence) and max_batch (sequences held
+ * at once).  loop may be NULL.  Parameters (cg_decoder_set_param / _load_safetensors), weights [out, in]:
+ * embed, embed.norm, final.norm, head, loop.in [hidden, 2 hidden], and per layer l<i>.norm1,
+ * .norm1b, .norm2, .norm2b, .mlp.{gate,up,down}, .mix.o and
+ *   latent  .mix.{q,dkv,dkv.norm,uk,uv}
+ *   delta   .mix.{q,k,v,b,a,g}, .mix.{q,k,v}.conv, .mix.{A_log,dt_bias,norm}
+ *   ssd     .mix.{in,conv,conv.b,dt_bias,A_log,D,norm}.
+ * The decoder then serves cg_decoder_prefill / append / decode / step_with / tokens / generate like
+ * any other (rows = slots 0 .. B-1, equal lengths), and the calls below.  cg_decoder_truncate takes
+ * 0 or the cached position only: a recurrent state has no earlier versions to go back to. */
+int32_t cg_decoder_create_layers(cg_ctx*, const cg_decoder_config* cfg, const cg_layer_config* layers, int32_t n_layers,
+                                 const cg_loop_config* loop, cg_decoder** out);
+/* Sequences of unequal length.  seq_open takes a free slot (its position is 0 and its state zero),
+ * seq_close gives it back.  run feeds rows: row r is the next lens[r] >= 1 tokens of the sequence in
+ * slots[r]; `tokens` (host) holds the rows' tokens one row after the other.  All rows are one batch.
+ * logits_out receives [n_want, vocab] for the packed token places want[0..n_want) (ascending).  With
+ * greedy != 0 the rows become the current rows and the arg-max after every row's last token its next
+ * token: cg_decoder_decode then advances all rows together, each at its own position, and
+ * cg_decoder_tokens returns what was generated. */
+int32_t cg_decoder_seq_open(cg_decoder*, int32_t* slot);
+int32_t cg_decoder_seq_close(cg_decoder*, int32_t slot);
+int32_t cg_decoder_run(cg_decoder*, int32_t rows, const int32_t* slots, const int32_t* lens, const uint32_t* tokens,
+                       int32_t n_want, const int32_t* want, int32_t greedy, cg_tensor** logits_out);
+/* Diagnostics: keep the residual stream of the next cg_decoder_run calls after every layer run, and
+ * read it back as [layer runs, tokens, hidden] F32 (the last call's tokens; one portion only). */
+int32_t cg_decoder_keep_residuals(cg_decoder*, int32_t on);
+int32_t cg_decoder_residuals(cg_decoder*, cg_tensor** out);
+
 /* Measurement hook: enqueue only the weight-streaming GEMMs of one decode step for `batch`
  * rows (every layer's qkv, o, gate/up, down projections and the LM head, on the decoder's
  * own weights) `iters` times, timed with CUDA events on the context's stream. */
