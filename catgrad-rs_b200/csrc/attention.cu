@@ -40,8 +40,10 @@ __global__ void __launch_bounds__(BQ * 2, D <= 64 ? 2 : 1) k_attn_prefill(AttnAr
   const int kvh = h / (a.nh / a.nkv);
   const int64_t q0 = (int64_t)qt * BQ;
   const __nv_bfloat16* qbase = a.q + (b * a.S) * (int64_t)a.nh * D + (int64_t)h * D;
-  const __nv_bfloat16* kbase = a.k_cache + ((b * a.nkv + kvh) * a.Tmax) * (int64_t)D;
-  const __nv_bfloat16* vbase = a.v_cache + ((b * a.nkv + kvh) * a.Tmax) * (int64_t)D;
+  const int64_t ldk = a.kv_ld > 0 ? a.kv_ld : D;  // from one key to the next
+  const int64_t kv0 = a.kv_ld > 0 ? b * a.Tmax * a.kv_ld + (int64_t)kvh * D : ((b * a.nkv + kvh) * a.Tmax) * (int64_t)D;
+  const __nv_bfloat16* kbase = a.k_cache + kv0;
+  const __nv_bfloat16* vbase = a.v_cache + kv0;
 
   // Q tile -> shared (rows past S are zero)
   constexpr int CH = D / 8;  // 16-byte chunks per row
@@ -76,7 +78,7 @@ __global__ void __launch_bounds__(BQ * 2, D <= 64 ? 2 : 1) k_attn_prefill(AttnAr
     for (int i = tid; i < BKV * CH; i += NT) {
       const int r = i / CH, ch = i - r * CH;
       const bool in = k0 + r < kv_len;
-      const int64_t off = in ? (k0 + r) * (int64_t)D + ch * 8 : 0;
+      const int64_t off = in ? (k0 + r) * ldk + ch * 8 : 0;
       const uint32_t d = (uint32_t)(((buf * BKV + r) * LD + ch * 8) * 2);
       cp_async16(sk_u + d, kbase + off, in ? 16 : 0);
       cp_async16(sv_u + d, vbase + off, in ? 16 : 0);
@@ -216,7 +218,7 @@ int launch_prefill(cg_ctx* c, const AttnArgs& a) {
     configured = true;
   }
   dim3 grid((unsigned)((a.S + BQ - 1) / BQ), (unsigned)a.nh, (unsigned)a.B);
-  const float scale = 1.0f / sqrtf((float)D);
+  const float scale = a.scale > 0.f ? a.scale : 1.0f / sqrtf((float)D);
   CG_CUDA(c, launch_kernel(c, k_attn_prefill<D, BQ, NBUF>, grid, dim3(BQ * 2), smem, 1, a, scale));
   CG_LAUNCHED(c);
   return CG_OK;

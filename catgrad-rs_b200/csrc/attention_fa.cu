@@ -37,7 +37,8 @@ struct FaArgs {
   __nv_bfloat16* out;  // [B * S, nh D]
   int64_t S, pos0, Tmax;
   int nh, nkv;
-  float scale_log2e;   // 1 / sqrt(D) * log2(e)
+  int token_major;     // keys and values lie token after token, the heads side by side
+  float scale_log2e;   // score factor (1 / sqrt(D)) * log2(e)
   int32_t* err;
 };
 
@@ -151,7 +152,8 @@ k_attn_fa(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUt
       const int qrow = (int)(b * p.S + q0);
       mbar_expect_tx(b_q_full, Q_BYTES);
       for (int s = 0; s < SUB; ++s) tma_load_2d(sq + s * BOX, &map_q, h * D + s * 64, qrow, b_q_full);
-      const int64_t kvrow0 = (b * p.nkv + kvh) * p.Tmax;
+      const int64_t kvrow0 = p.token_major ? b * p.Tmax : (b * p.nkv + kvh) * p.Tmax;
+      const int kx = p.token_major ? kvh * D : 0;
       bool ok = true;
       for (int j = 0; j < nt && ok; ++j) {
         const uint32_t buf = (uint32_t)j & 1u, ph = ((uint32_t)j >> 1) & 1u;
@@ -161,13 +163,13 @@ k_attn_fa(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUt
           if (!ok) break;
         }
         mbar_expect_tx(b_k_full + 8 * buf, KV_BYTES);
-        for (int s = 0; s < SUB; ++s) tma_load_2d(sk + buf * KV_BYTES + s * KBOX, &map_k, s * 64, row, b_k_full + 8 * buf);
+        for (int s = 0; s < SUB; ++s) tma_load_2d(sk + buf * KV_BYTES + s * KBOX, &map_k, kx + s * 64, row, b_k_full + 8 * buf);
         if (j >= 2) {
           ok = mbar_wait(b_v_empty + 8 * buf, ph ^ 1u, cta_abort, p.err);
           if (!ok) break;
         }
         mbar_expect_tx(b_v_full + 8 * buf, KV_BYTES);
-        for (int s = 0; s < SUB; ++s) tma_load_2d(sv + buf * KV_BYTES + s * KBOX, &map_v, s * 64, row, b_v_full + 8 * buf);
+        for (int s = 0; s < SUB; ++s) tma_load_2d(sv + buf * KV_BYTES + s * KBOX, &map_v, kx + s * 64, row, b_v_full + 8 * buf);
       }
     }
   } else if (warp == 1) {
@@ -364,13 +366,16 @@ int launch_fa(cg_ctx* c, const AttnArgs& a) {
   }
   CUtensorMap mq, mk, mv;
   CG_TRY(make_map(c, &mq, a.q, a.B * a.S, (int64_t)a.nh * D, (int64_t)a.nh * D, 128));
-  CG_TRY(make_map(c, &mk, a.k_cache, a.B * a.nkv * a.Tmax, D, D, FA_BK));
-  CG_TRY(make_map(c, &mv, a.v_cache, a.B * a.nkv * a.Tmax, D, D, FA_BK));
+  const bool tm = a.kv_ld > 0;
+  const int64_t kv_rows = tm ? a.B * a.Tmax : a.B * a.nkv * a.Tmax, kv_cols = tm ? (int64_t)a.nkv * D : D, kv_ld = tm ? a.kv_ld : D;
+  CG_TRY(make_map(c, &mk, a.k_cache, kv_rows, kv_cols, kv_ld, FA_BK));
+  CG_TRY(make_map(c, &mv, a.v_cache, kv_rows, kv_cols, kv_ld, FA_BK));
   FaArgs p;
   p.out = a.out;
   p.S = a.S; p.pos0 = a.pos0; p.Tmax = a.Tmax;
   p.nh = a.nh; p.nkv = a.nkv;
-  p.scale_log2e = 1.4426950408889634f / sqrtf((float)D);
+  p.token_major = tm ? 1 : 0;
+  p.scale_log2e = 1.4426950408889634f * (a.scale > 0.f ? a.scale : 1.f / sqrtf((float)D));
   p.err = c->core->dev_err;
   dim3 grid((unsigned)((a.S + FA_BQ - 1) / FA_BQ), (unsigned)a.nh, (unsigned)a.B);
   CG_CUDA(c, launch_kernel(c, k_attn_fa<D, FA_BK>, grid, dim3(192), smem, 1, mq, mk, mv, p));
@@ -383,7 +388,7 @@ int launch_fa(cg_ctx* c, const AttnArgs& a) {
 bool attn_fa_supported(const AttnArgs& a) {
   return (a.d == 64 || a.d == 128) && a.window <= 0 && a.softcap <= 0.f && !a.pos_dev && a.S >= 64 &&
          a.B * a.S < 2147483647ll && a.B * a.nkv * a.Tmax < 2147483647ll && ((uintptr_t)a.q % 16) == 0 &&
-         ((uintptr_t)a.k_cache % 16) == 0 && ((uintptr_t)a.v_cache % 16) == 0;
+         ((uintptr_t)a.k_cache % 16) == 0 && ((uintptr_t)a.v_cache % 16) == 0 && a.kv_ld % 8 == 0;
 }
 
 int k_launch_attn_fa(cg_ctx* c, const AttnArgs& a) {

@@ -4,7 +4,7 @@
 //
 // A sequence lives in a slot.  Per layer run (a looped layer counts once per pass) a slot holds
 //   latent attention   [max_seq, Lw] cached rows (normed latent, rotated key part)
-//   delta, ssd         an f32 matrix per head and the last taps - 1 inputs of the convolutions
+//   delta, ssd         an f32 matrix per head and the last inputs of the convolutions
 // Nothing is cleared when a slot is reused: a row whose first position is 0 starts from zeros.
 // Batches are rows of unequal length, packed token after token; every kernel finds a token's row,
 // slot and position through the row tables (RowsDev).  In a decode step the tables stay as they
@@ -24,6 +24,7 @@ namespace cg {
 
 namespace {
 inline int64_t up8(int64_t n) { return (n + 7) / 8 * 8; }
+inline int64_t up16(int64_t n) { return (n + 15) / 16 * 16; }
 }  // namespace
 
 struct MixedLayer {
@@ -40,7 +41,8 @@ struct MixedLayer {
   int dkv_off = 0, Dq = 0;
   // recurrences
   cg_tensor *conv_w = nullptr, *conv_b = nullptr, *a_log = nullptr, *dt_bias = nullptr, *dskip = nullptr, *norm = nullptr;
-  int H = 0, KH = 0, dk = 0, dv = 0, C = 0, gate_off = 0, small_off = 0, q_off = 0, k_off = 0, v_off = 0;
+  bool chunked = false;  // prompts run on the tensor cores, 64 tokens at a time
+  int H = 0, KH = 0, dk = 0, dv = 0, dvs = 0, C = 0, gate_off = 0, small_off = 0, q_off = 0, k_off = 0, v_off = 0;
 };
 
 struct MixedRun {
@@ -67,7 +69,9 @@ struct MixedModel {
   // workspace for `cap` tokens
   int64_t cap = 0, cap_w = 0;
   cg_tensor *x = nullptr, *xn = nullptr, *xcat = nullptr, *y = nullptr, *proj = nullptr, *cv = nullptr, *gl = nullptr, *co = nullptr,
-            *ro = nullptr, *att = nullptr, *hact = nullptr, *gu = nullptr, *q = nullptr, *cpk = nullptr, *tok = nullptr, *xw = nullptr;
+            *ro = nullptr, *att = nullptr, *hact = nullptr, *gu = nullptr, *q = nullptr, *cpk = nullptr, *tok = nullptr, *xw = nullptr,
+            *qkv = nullptr, *rn = nullptr, *tinv = nullptr, *kv = nullptr, *lat = nullptr;
+  int64_t tinv_n = 0, kv_n = 0;
   bool keep = false;
   cg_tensor* kept = nullptr;
   int64_t kept_M = 0;
@@ -118,7 +122,7 @@ int finalize_latent(cg_decoder* D, MixedLayer& L, const std::string& mx) {
   const cg_layer_config& k = L.k;
   const int64_t W = D->H, H = k.heads, d = k.dim, r = k.rot_dim, dv = k.vdim, R = k.kv_rank;
   const int st = X.act_storage();
-  L.Lw = up8(R + r);
+  L.Lw = up16(R + r);
   L.dkv_off = (int)up8(H * (d + r));
   L.Np = up8(L.dkv_off + R + r);
   // head size of the expanded keys and values that the prompt kernels work on
@@ -166,11 +170,13 @@ int finalize_recurrent(cg_decoder* D, MixedLayer& L, const std::string& mx) {
   const int st = X.act_storage();
   L.H = k.heads;
   L.dv = k.vdim;
+  L.dvs = (int)up8(L.dv);
   const int64_t inner = (int64_t)L.H * L.dv;
   L.KH = delta ? k.kv_heads : k.groups;
   L.dk = delta ? k.dim : k.state;
   const int64_t kk = (int64_t)L.KH * L.dk;
   L.C = (int)(inner + 2 * kk);
+  L.chunked = !X.f32 && chunk_supported(L.dk);
   L.gate_off = (int)up8(L.C);
   L.small_off = (int)up8(L.gate_off + inner);
   L.Np = up8(L.small_off + (delta ? 2 : 1) * L.H);
@@ -217,7 +223,7 @@ int ensure_mixed(cg_decoder* D, int64_t M) {
   if (M <= X.cap) return CG_OK;
   cg_ctx* c = D->c;
   forget_graph(D);  // it holds the old buffers
-  int64_t np = 0, cc = 0, hh = 0, inner = 0, ko = 0, fp = 0, qw = 0, lw = 0;
+  int64_t np = 0, cc = 0, hh = 0, inner = 0, ko = 0, fp = 0, qw = 0, lw = 0, qkv = 0, kh = 0;
   for (const MixedLayer& L : X.layers) {
     np = std::max(np, L.Np);
     ko = std::max(ko, L.Ko);
@@ -228,7 +234,11 @@ int ensure_mixed(cg_decoder* D, int64_t M) {
     } else {
       cc = std::max<int64_t>(cc, up8(L.C));
       hh = std::max<int64_t>(hh, L.H);
-      inner = std::max<int64_t>(inner, (int64_t)L.H * L.dv);
+      inner = std::max<int64_t>(inner, (int64_t)L.H * L.dvs);
+      if (L.chunked) {
+        qkv = std::max<int64_t>(qkv, 2 * L.KH * up16(L.dk) + (int64_t)L.H * L.dvs);
+        kh = std::max<int64_t>(kh, L.KH);
+      }
     }
   }
   const int st = X.act_storage();
@@ -247,6 +257,20 @@ int ensure_mixed(cg_decoder* D, int64_t M) {
     CG_TRY(new2(c, ST_F32, M, hh, &X.gl));
     CG_TRY(new2(c, ST_F32, M, hh, &X.co));
     CG_TRY(new2(c, ST_F32, M, inner, &X.ro));
+  }
+  if (qkv) {
+    CG_TRY(new2(c, ST_BF16, M, qkv, &X.qkv));
+    CG_TRY(new2(c, ST_F32, 2 * M, kh, &X.rn));
+  }
+  if (!X.f32) {
+    size_t lat = 0;
+    for (const MixedLayer& L : X.layers)
+      if (L.k.mixer == CG_MIX_LATENT) {
+        LatentArgs a;
+        a.H = L.k.heads; a.R = L.k.kv_rank; a.Lw = L.Lw;
+        lat = std::max(lat, latent_decode_scratch(a, std::min<int64_t>(M, LATENT_DECODE_TOKENS)));
+      }
+    if (lat) CG_TRY(new2(c, ST_F32, (int64_t)(lat + 3) / 4, 1, &X.lat));
   }
   if (qw) {
     CG_TRY(new2(c, st, M, qw, &X.q));
@@ -310,10 +334,17 @@ struct Portion {
   int max_len = 0;
 };
 
-// words of the row tables for `rows` rows and M tokens: slot, start, pos0, tok_row, pick, dst
-int64_t table_words(int64_t rows, int64_t M) { return rows + (rows + 1) + rows + M; }
+// words of the row tables: slot, start, pos0, tok_row and, for chunks of RECUR_CHUNK tokens, the first
+// chunk of every row, the chunks' first tokens and their lengths
+int64_t table_words(int64_t rows, int64_t M) {
+  return rows + (rows + 1) + rows + M + (rows + 1) + 2 * (M / RECUR_CHUNK + rows);
+}
+struct Chunks {
+  const int32_t *tok, *len, *row_chunk;
+  int n;
+};
 
-int write_tables(cg_decoder* D, const Portion& p, cg_tensor* dst, RowsDev* rd) {
+int write_tables(cg_decoder* D, const Portion& p, cg_tensor* dst, RowsDev* rd, Chunks* ch) {
   cg_ctx* c = D->c;
   const int R = (int)p.slots.size();
   std::vector<int32_t> t((size_t)table_words(R, p.M));
@@ -326,17 +357,46 @@ int write_tables(cg_decoder* D, const Portion& p, cg_tensor* dst, RowsDev* rd) {
     for (int i = 0; i < p.lens[r]; ++i) tr[at++] = r;
   }
   start[R] = at;
+  int32_t *rc = tr + p.M, *ct = rc + R + 1;
+  std::vector<int32_t> lens;
+  int nc = 0;
+  for (int r = 0; r < R; ++r) {
+    rc[r] = nc;
+    for (int i = 0; i < p.lens[r]; i += RECUR_CHUNK) {
+      ct[nc++] = start[r] + i;
+      lens.push_back(std::min(RECUR_CHUNK, p.lens[r] - i));
+    }
+  }
+  rc[R] = nc;
+  std::copy(lens.begin(), lens.end(), ct + nc);
   CG_CUDA(c, cudaMemcpyAsync(dst->data(), t.data(), t.size() * 4, cudaMemcpyHostToDevice, c->core->stream));
   const int32_t* d = (const int32_t*)dst->data();
   rd->slot = d; rd->start = d + R; rd->pos0 = d + 2 * R + 1; rd->tok_row = d + 3 * R + 1;
   rd->step = D->pos_dev();
   rd->rows = R;
   rd->M = p.M;
+  ch->row_chunk = rd->tok_row + p.M;
+  ch->tok = ch->row_chunk + R + 1;
+  ch->len = ch->tok + nc;
+  ch->n = nc;
   return CG_OK;
 }
 
+// A buffer that prompts of a new length may have to grow (never part of a captured graph).
+int grow(cg_ctx* c, int storage, int64_t n, cg_tensor** t, int64_t* have) {
+  if (n <= *have) return CG_OK;
+  CG_TRY(new2(c, storage, n, 1, t, false));
+  *have = n;
+  return CG_OK;
+}
+
+// A few new tokens: attention in the cached rows' space.  Prompts: the cached rows are expanded to
+// keys and values of Dq values per head, token after token, and run through the prompt attention.
+// f32, and sizes those kernels do not have: one block per token and head.
 int latent_layer(cg_decoder* D, const MixedLayer& L, MixedRun& run, const RowsDev& rd, const Portion* p) {
+  cg_ctx* c = D->c;
   MixedModel& X = *D->mixed;
+  CG_TRY(lin(D, X.xn->data(), X.Wp, rd.M, L.w_in, 0, L.Np, X.proj->data(), L.Np));
   LatentArgs a;
   a.proj = (const float*)X.proj->data(); a.ldp = L.Np; a.dkv_off = L.dkv_off;
   a.H = L.k.heads; a.d = L.k.dim; a.r = L.k.rot_dim; a.dv = L.k.vdim; a.R = L.k.kv_rank;
@@ -350,40 +410,125 @@ int latent_layer(cg_decoder* D, const MixedLayer& L, MixedRun& run, const RowsDe
   a.att = X.att->data(); a.ld_att = L.Ko; a.Do = L.Do;
   a.bf16 = X.f32 ? 0 : 1;
   a.rows = rd;
-  (void)p;
-  CG_TRY(k_launch_latent_prep(D->c, a));
-  return k_launch_latent_attn(D->c, a);
+  if (!X.f32 && (!p || p->max_len <= 4) && rd.M <= LATENT_DECODE_TOKENS && latent_decode_supported(a.d, a.R, a.Lw))
+    return k_launch_latent_decode(c, a, X.lat->data());
+  if (!L.w_kv || !p) {
+    CG_TRY(k_launch_latent_prep(c, a));
+    return k_launch_latent_attn(c, a);
+  }
+  const int R = rd.rows;
+  const int64_t Dp = L.Dq, kvw = 2 * a.H * Dp, es = 2;
+  bool equal = true, fresh = true;
+  int64_t ctx = 0;
+  for (int r = 0; r < R; ++r) {
+    equal = equal && p->lens[r] == p->lens[0] && p->pos0[r] == p->pos0[0];
+    fresh = fresh && p->pos0[r] == 0;
+    ctx += p->pos0[r] + p->lens[r];
+  }
+  CG_TRY(grow(c, ST_BF16, ctx * kvw, &X.kv, &X.kv_n));
+  char* kv = (char*)X.kv->data();
+  if (fresh) a.c_out = X.cpk->data();
+  CG_TRY(k_launch_latent_prep(c, a));
+  if (fresh) {
+    CG_TRY(lin(D, X.cpk->data(), L.Lw, rd.M, L.w_kv, 0, kvw, kv, kvw, true));
+  } else {
+    int64_t at = 0;
+    for (int r = 0; r < R; ++r) {
+      const int64_t n = p->pos0[r] + p->lens[r];
+      CG_TRY(lin(D, (const char*)a.cache + (size_t)p->slots[r] * a.Tmax * L.Lw * es, L.Lw, n, L.w_kv, 0, kvw, kv + (size_t)at * kvw * es, kvw,
+                 true));
+      at += n;
+    }
+  }
+  int64_t tok = 0, at = 0;
+  for (int r = 0; r < (equal ? 1 : R); ++r) {
+    AttnArgs t;
+    t.q = (const __nv_bfloat16*)a.q_out + tok * a.H * Dp;
+    t.k_cache = (const __nv_bfloat16*)kv + at * kvw;
+    t.v_cache = t.k_cache + a.H * Dp;
+    t.out = (__nv_bfloat16*)a.att + tok * L.Ko;
+    t.B = equal ? R : 1; t.S = p->lens[r]; t.pos0 = p->pos0[r]; t.Tmax = t.pos0 + t.S;
+    t.pos_dev = nullptr;
+    t.nh = t.nkv = a.H; t.d = (int)Dp;
+    t.window = 0; t.softcap = 0.f; t.scratch = nullptr;
+    t.kv_ld = kvw; t.scale = a.scale;
+    CG_TRY(k_launch_attn_prefill(c, t));
+    tok += t.S;
+    at += t.Tmax;
+  }
+  return CG_OK;
 }
 
-int recurrent_layer(cg_decoder* D, const MixedLayer& L, MixedRun& run, const RowsDev& rd, const Portion* p) {
+void recurrent_base(cg_decoder* D, const MixedLayer& L, MixedRun& run, const RowsDev& rd, RecurBase* a) {
   MixedModel& X = *D->mixed;
+  a->delta = L.k.mixer == CG_MIX_DELTA ? 1 : 0;
+  a->H = L.H; a->KH = L.KH; a->dk = L.dk; a->dv = L.dv; a->dvs = L.dvs; a->C = L.C; a->taps = L.k.conv;
+  a->q_off = L.q_off; a->k_off = L.k_off; a->v_off = L.v_off;
+  a->conv_w = (const float*)L.conv_w->data();
+  a->conv_b = L.conv_b ? (const float*)L.conv_b->data() : nullptr;
+  a->tail = (float*)run.tail->data();
+  a->a_log = (const float*)L.a_log->data(); a->dt_bias = (const float*)L.dt_bias->data();
+  a->dskip = L.dskip ? (const float*)L.dskip->data() : nullptr;
+  a->S = (float*)run.state->data();
+  a->gl = (float*)X.gl->data(); a->co = (float*)X.co->data();
+  a->o = (float*)X.ro->data();
+  a->rows = rd;
+}
+
+// One token per row: one kernel.  Prompts in a bf16 context: chunks on the tensor cores, on bf16
+// projections (the gates' projections stay f32).  Otherwise token by token.
+int recurrent_layer(cg_decoder* D, const MixedLayer& L, MixedRun& run, const RowsDev& rd, const Portion* p, const Chunks* ch) {
+  cg_ctx* c = D->c;
+  MixedModel& X = *D->mixed;
+  const int64_t M = rd.M, K = X.Wp;
+  GatedNorm n;
+  n.delta = L.k.mixer == CG_MIX_DELTA ? 1 : 0;
+  n.H = L.H; n.dv = L.dv; n.dvs = L.dvs; n.norm_groups = L.k.norm_groups;
+  n.o = (const float*)X.ro->data();
+  n.norm = (const float*)L.norm->data(); n.eps = D->cfg.rms_eps;
+  n.att = X.att->data(); n.ld_att = L.Ko; n.att_bf16 = X.f32 ? 0 : 1;
+  n.M = M;
+  if (L.chunked && p && p->max_len >= 8) {
+    ChunkArgs a;
+    recurrent_base(D, L, run, rd, &a);
+    __nv_bfloat16* pb = (__nv_bfloat16*)X.proj->data();
+    float* small = (float*)(pb + M * L.small_off);  // both fit where the f32 projection would
+    const int64_t ns = L.Np - L.small_off;
+    CG_TRY(lin(D, X.xn->data(), K, M, L.w_in, 0, L.small_off, pb, L.small_off, true));
+    CG_TRY(lin(D, X.xn->data(), K, M, L.w_in, L.small_off, ns, small, ns));
+    a.proj = pb; a.ldp = L.small_off;
+    a.small = small; a.ld_small = ns;
+    a.DKp = (int)up16(L.dk); a.dvp = L.dvs;
+    a.q = (__nv_bfloat16*)X.qkv->data();
+    a.k = a.q + M * L.KH * a.DKp;
+    a.v = a.k + M * L.KH * a.DKp;
+    a.rq = (float*)X.rn->data();
+    a.rk = a.rq + M * L.KH;
+    a.chunk_tok = ch->tok; a.chunk_len = ch->len; a.row_chunk = ch->row_chunk; a.n_chunks = ch->n;
+    a.T = nullptr;
+    if (a.delta) {
+      CG_TRY(grow(c, ST_BF16, (int64_t)ch->n * L.H * 2 * RECUR_CHUNK * RECUR_CHUNK, &X.tinv, &X.tinv_n));
+      a.T = (__nv_bfloat16*)X.tinv->data();
+    }
+    CG_TRY(k_launch_chunk_recurrence(c, a));
+    n.gate = pb + L.gate_off; n.ldg = L.small_off; n.gate_bf16 = 1;
+    return k_launch_gated_norm(c, n);
+  }
   RecurArgs a;
-  a.delta = L.k.mixer == CG_MIX_DELTA ? 1 : 0;
-  a.H = L.H; a.KH = L.KH; a.dk = L.dk; a.dv = L.dv; a.C = L.C; a.taps = L.k.conv;
-  a.q_off = L.q_off; a.k_off = L.k_off; a.v_off = L.v_off; a.gate_off = L.gate_off; a.small_off = L.small_off;
+  recurrent_base(D, L, run, rd, &a);
+  CG_TRY(lin(D, X.xn->data(), K, M, L.w_in, 0, L.Np, X.proj->data(), L.Np));
   a.proj = (const float*)X.proj->data(); a.ldp = L.Np;
-  a.conv_w = (const float*)L.conv_w->data();
-  a.conv_b = L.conv_b ? (const float*)L.conv_b->data() : nullptr;
-  a.tail = (float*)run.tail->data();
-  a.a_log = (const float*)L.a_log->data(); a.dt_bias = (const float*)L.dt_bias->data();
-  a.dskip = L.dskip ? (const float*)L.dskip->data() : nullptr;
-  a.S = (float*)run.state->data();
+  a.gate_off = L.gate_off; a.small_off = L.small_off;
   a.cv = (float*)X.cv->data(); a.ldc = up8(L.C);
-  a.gl = (float*)X.gl->data(); a.co = (float*)X.co->data();
-  a.o = (float*)X.ro->data();
-  a.norm = (const float*)L.norm->data(); a.norm_groups = L.k.norm_groups; a.eps = D->cfg.rms_eps;
-  a.att = X.att->data(); a.ld_att = L.Ko; a.bf16 = X.f32 ? 0 : 1;
-  a.rows = rd;
-  (void)p;
-  CG_TRY(k_launch_conv_heads(D->c, a));
-  CG_TRY(k_launch_conv_tail(D->c, a));
-  CG_TRY(k_launch_recur_steps(D->c, a));
-  return k_launch_gated_norm(D->c, a);
+  n.gate = a.proj + L.gate_off; n.ldg = L.Np; n.gate_bf16 = 0;
+  if ((!p || p->max_len == 1) && recur_decode_supported(L.dk, L.dv)) return k_launch_recur_decode(c, a, n);
+  CG_TRY(k_launch_recur_steps(c, a));
+  return k_launch_gated_norm(c, n);
 }
 
 // Embedding and all layer runs of one batch; x holds the residual stream afterwards.  p is null in
 // decode steps (one token per row).
-int walk(cg_decoder* D, const RowsDev& rd, const uint32_t* tokens, const Portion* p) {
+int walk(cg_decoder* D, const RowsDev& rd, const uint32_t* tokens, const Portion* p, const Chunks* ch) {
   cg_ctx* c = D->c;
   MixedModel& X = *D->mixed;
   const int64_t M = rd.M, W = D->H, Wp = X.Wp;
@@ -417,9 +562,8 @@ int walk(cg_decoder* D, const RowsDev& rd, const uint32_t* tokens, const Portion
       u.out = X.xn->data(); u.ldo = Wp; u.g2 = (const float*)L.n1->data();
       CG_TRY(k_launch_row_update(c, u, M, bf));
     }
-    CG_TRY(lin(D, X.xn->data(), Wp, M, L.w_in, 0, L.Np, X.proj->data(), L.Np));
     if (L.k.mixer == CG_MIX_LATENT) CG_TRY(latent_layer(D, L, run, rd, p));
-    else CG_TRY(recurrent_layer(D, L, run, rd, p));
+    else CG_TRY(recurrent_layer(D, L, run, rd, p, ch));
     CG_TRY(lin(D, X.att->data(), L.Ko, M, L.w_o, 0, Wp, X.y->data(), Wp));
     RowUpdate u = base;
     u.y = (const float*)X.y->data(); u.ldy = Wp; u.add = 1;
@@ -467,10 +611,9 @@ int mixed_create(cg_decoder* D, const cg_layer_config* layers, int n_layers, con
       if (k.dim < 1 || k.rot_dim < 0 || k.rot_dim % 2 || k.kv_rank < 1 || (k.rot_dim && !(k.rot_base > 0)))
         return bad_size(D, i, "latent attention sizes");
     } else if (k.mixer == CG_MIX_DELTA) {
-      if (k.dim < 1 || k.kv_heads < 1 || k.heads % k.kv_heads || k.conv < 1 || k.conv > 17) return bad_size(D, i, "delta rule sizes");
+      if (k.dim < 1 || k.kv_heads < 1 || k.heads % k.kv_heads || k.conv < 1) return bad_size(D, i, "delta rule sizes");
     } else if (k.mixer == CG_MIX_SSD) {
-      if (k.state < 1 || k.groups < 1 || k.heads % k.groups || k.norm_groups < 1 || (k.heads * k.vdim) % k.norm_groups || k.conv < 1 ||
-          k.conv > 17)
+      if (k.state < 1 || k.groups < 1 || k.heads % k.groups || k.norm_groups < 1 || (k.heads * k.vdim) % k.norm_groups || k.conv < 1)
         return bad_size(D, i, "state space sizes");
     } else return bad_size(D, i, "unknown mixer");
   }
@@ -502,7 +645,8 @@ void mixed_destroy(cg_decoder* D) {
       drop(*t);
   for (MixedRun& r : X->runs) { drop(r.cache); drop(r.state); drop(r.tail); }
   for (cg_tensor** t : {&X->embed_norm, &X->w_loop, &X->tab_run, &X->tab_dec, &X->x, &X->xn, &X->xcat, &X->y, &X->proj, &X->cv, &X->gl,
-                        &X->co, &X->ro, &X->att, &X->hact, &X->gu, &X->q, &X->cpk, &X->tok, &X->xw, &X->kept})
+                        &X->co, &X->ro, &X->att, &X->hact, &X->gu, &X->q, &X->cpk, &X->tok, &X->xw, &X->kept, &X->qkv, &X->rn,
+                        &X->tinv, &X->kv, &X->lat})
     drop(*t);
   delete X;
   D->mixed = nullptr;
@@ -543,8 +687,8 @@ int mixed_finalize(cg_decoder* D) {
     if (L.k.mixer == CG_MIX_LATENT) {
       CG_TRY(new2(c, st, slots * D->cfg.max_seq, L.Lw, &r.cache));
     } else {
-      CG_TRY(new2(c, ST_F32, slots * L.H * L.dk, L.dv, &r.state));
-      CG_TRY(new2(c, ST_F32, slots * std::max(1, L.k.conv - 1), L.C, &r.tail));
+      CG_TRY(new2(c, ST_F32, slots * L.H * L.dk, L.dvs, &r.state));
+      CG_TRY(new2(c, ST_F32, slots * L.k.conv, L.C, &r.tail));
     }
   }
   if (X.loop) {
@@ -678,8 +822,9 @@ int mixed_run(cg_decoder* D, const std::vector<int>& slots, const std::vector<in
       X.tab_run_words = n;
     }
     RowsDev rd;
-    CG_TRY(write_tables(D, p, X.tab_run, &rd));
-    CG_TRY(walk(D, rd, toks, &p));
+    Chunks ch;
+    CG_TRY(write_tables(D, p, X.tab_run, &rd, &ch));
+    CG_TRY(walk(D, rd, toks, &p, &ch));
     if (!pick.empty()) {
       int32_t* pd = (int32_t*)X.tab_run->data() + tw;
       const size_t np = pick.size();
@@ -759,7 +904,8 @@ int mixed_begin_decode(cg_decoder* D, int steps) {
   for (int s : p.slots) p.pos0.push_back(X.pos[s]);
   p.M = (int64_t)p.slots.size();
   RowsDev rd;
-  CG_TRY(write_tables(D, p, X.tab_dec, &rd));
+  Chunks ch;
+  CG_TRY(write_tables(D, p, X.tab_dec, &rd, &ch));
   CG_TRY(set_state(D, 0, D->generated));
   X.tables_current = true;
   return CG_OK;
@@ -775,7 +921,7 @@ int mixed_step(cg_decoder* D) {
   rd.step = D->pos_dev();
   rd.rows = R;
   rd.M = R;
-  CG_TRY(walk(D, rd, (const uint32_t*)D->cur->data(), nullptr));
+  CG_TRY(walk(D, rd, (const uint32_t*)D->cur->data(), nullptr, nullptr));
   RowUpdate u;
   u.x = (float*)X.x->data(); u.ldx = X.Wp; u.eps = D->cfg.rms_eps; u.W = (int)D->H;
   u.pick = rd.tok_row;  // row i of the batch is token i

@@ -79,6 +79,10 @@ struct AttnArgs {
   int64_t window;                // 0 = none
   float softcap;                 // 0 = none
   float* scratch;                // unused
+  // kv_ld > 0: keys and values lie token after token instead, key t of row b and head h at
+  // k_cache + (b * Tmax + t) * kv_ld + h * d (Tmax = tokens per row)
+  int64_t kv_ld = 0;
+  float scale = 0.f;             // factor on the scores; 0 = 1 / sqrt(d)
 };
 // Causal (optionally windowed / soft-capped) attention of S new tokens per row against cache
 // positions [0, pos0 + S).  Tensor-core flash kernel.

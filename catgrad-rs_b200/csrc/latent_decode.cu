@@ -1,0 +1,352 @@
+// latent_decode.cu — latent attention for a few new tokens per row (a decode step) in a bf16 context.
+//
+// The scores q . (Wuk c) are taken as (Wuk^T q) . c, so all heads attend over the same cached rows
+// [c, rotated key part] and the cache is read once per token instead of being expanded:
+//
+//   k_latent_absorb   one block per (head, 64 latent columns): Wuk^T q for every new token; the
+//                     last blocks norm / rotate / append the tokens' own cached rows and rotate q
+//   k_latent_dec      one block per (token, 16 heads, context slice): heads are the rows of the
+//                     MMA tile; 64 cached rows at a time through two shared-memory buffers,
+//                     online softmax, partial output in the latent space
+//   k_latent_out      one block per (head, 32 values): the slices are merged and mapped through Wuv
+#include <algorithm>
+
+#include "mixers.h"
+#include "mma.cuh"
+
+namespace cg {
+
+namespace {
+
+__device__ __forceinline__ float warp_sum(float v) {
+#pragma unroll
+  for (int o = 16; o; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+  return v;
+}
+__device__ __forceinline__ float block_sum(float v, float* sh) {
+  const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  v = warp_sum(v);
+  __syncthreads();
+  if (lane == 0) sh[wid] = v;
+  __syncthreads();
+  v = lane < nw ? sh[lane] : 0.f;
+  return warp_sum(v);
+}
+
+struct DecodeScratch {
+  __nv_bfloat16* qa;   // [M, H, Lw] queries in the cached rows' space
+  float* o;            // [M, H, splits, R] partial outputs, relative to their maximum
+  float2* ml;          // [M, H, splits] maximum, sum
+  int splits;
+};
+
+__global__ void __launch_bounds__(256) k_latent_absorb(LatentArgs a, DecodeScratch s, int col_blocks) {
+  asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+  extern __shared__ __align__(16) float sm[];
+  const int tid = threadIdx.x, M = (int)a.rows.M, D = a.d + a.r;
+  const int nb = a.H * col_blocks;
+  if ((int)blockIdx.x >= nb) {
+    // the new tokens' cached rows and the rotated parts of their queries
+    asm volatile("griddepcontrol.wait;" ::: "memory");
+    const int64_t m = blockIdx.x - nb;
+    const int row = a.rows.tok_row[m];
+    const int64_t pos = row_pos0(a.rows, row) + (m - a.rows.start[row]);
+    const float* p = a.proj + m * a.ldp;
+    const float* dk = p + a.dkv_off;
+    __nv_bfloat16* crow = (__nv_bfloat16*)a.cache + ((int64_t)a.rows.slot[row] * a.Tmax + pos) * a.Lw;
+    const int half = a.r / 2;
+    const float* ct = a.cos_t + pos * half;
+    const float* sn = a.sin_t + pos * half;
+    auto rotated = [&](const float* x, int j) {
+      const int k = j >> 1;
+      const float u = x[2 * k], w = x[2 * k + 1];
+      return (j & 1) ? w * ct[k] + u * sn[k] : u * ct[k] - w * sn[k];
+    };
+    float ss = 0.f;
+    for (int i = tid; i < a.R; i += 256) ss += dk[i] * dk[i];
+    ss = block_sum(ss, sm);
+    const float rms = sqrtf(ss / (float)a.R + a.eps);
+    for (int i = tid; i < (int)a.Lw; i += 256) {
+      const float v = i < a.R ? dk[i] / rms * a.c_gain[i] : i < a.R + a.r ? rotated(dk + a.R, i - a.R) : 0.f;
+      crow[i] = __float2bfloat16_rn(v);
+    }
+    const int w = (int)a.Lw - a.R;
+    for (int i = tid; i < a.H * w; i += 256) {
+      const int h = i / w, j = i - h * w;
+      s.qa[(m * a.H + h) * a.Lw + a.R + j] = __float2bfloat16_rn(j < a.r ? rotated(p + h * D + a.d, j) : 0.f);
+    }
+    return;
+  }
+  // Wuk^T q for 64 latent columns of one head: 64 columns x 4 slices of the head dimension
+  const int h = blockIdx.x / col_blocks, c = (blockIdx.x % col_blocks) * 64 + (tid & 63), part = tid >> 6;
+  float* q = sm;                                       // [d]
+  float* red = q + a.d;                                // [4][64]
+  __nv_bfloat16* w = (__nv_bfloat16*)(red + 256);      // [d][64]
+  const __nv_bfloat16* uk = (const __nv_bfloat16*)a.uk + (int64_t)h * a.d * a.R;
+  for (int e = part; e < a.d; e += 4) w[e * 64 + (tid & 63)] = c < a.R ? uk[(int64_t)e * a.R + c] : __float2bfloat16_rn(0.f);
+  asm volatile("griddepcontrol.wait;" ::: "memory");   // (the weights do not depend on it)
+  for (int m = 0; m < M; ++m) {
+    const float* p = a.proj + (int64_t)m * a.ldp + h * D;
+    for (int e = tid; e < a.d; e += 256) q[e] = p[e];
+    __syncthreads();
+    float v = 0.f;
+    for (int e = part; e < a.d; e += 4) v += q[e] * __bfloat162float(w[e * 64 + (tid & 63)]);
+    red[tid] = v;
+    __syncthreads();
+    if (part == 0 && c < a.R)
+      s.qa[((int64_t)m * a.H + h) * a.Lw + c] = __float2bfloat16_rn((red[tid] + red[tid + 64]) + (red[tid + 128] + red[tid + 192]));
+  }
+}
+
+constexpr int LD_KT = 64;  // cached rows per tile
+
+// NT: 8-column output tiles per warp (eight warps share the latent columns)
+template <int NT>
+__global__ void __launch_bounds__(256) k_latent_dec(LatentArgs a, DecodeScratch sc, int ldk) {
+  asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+  asm volatile("griddepcontrol.wait;" ::: "memory");
+  extern __shared__ __align__(16) uint8_t smem[];
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  __nv_bfloat16* sq = (__nv_bfloat16*)smem;            // [16][ldk]
+  __nv_bfloat16* sk = sq + 16 * ldk;                   // [2][64][ldk]
+  __nv_bfloat16* sp = sk + 2 * LD_KT * ldk;            // [16][72]
+  float* wm = (float*)(sp + 16 * 72);                  // [8][16] per-warp row maxima
+  float* wl = wm + 128;                                // [8][16] per-warp row sums
+  const int64_t m = blockIdx.x;
+  const int h0 = blockIdx.y * 16, split = blockIdx.z;
+  const int row = a.rows.tok_row[m];
+  const int64_t pos = row_pos0(a.rows, row) + (m - a.rows.start[row]);
+  const __nv_bfloat16* base = (const __nv_bfloat16*)a.cache + (int64_t)a.rows.slot[row] * a.Tmax * a.Lw;
+  const int64_t n_keys = pos + 1;
+  const int64_t per = ((n_keys + sc.splits - 1) / sc.splits + LD_KT - 1) / LD_KT * LD_KT;
+  const int64_t k_lo = split * per, k_hi = min(n_keys, k_lo + per);
+  const int CH = (int)a.Lw / 8;
+  const uint32_t sq_u = (uint32_t)__cvta_generic_to_shared(sq), sk_u = (uint32_t)__cvta_generic_to_shared(sk),
+                 sp_u = (uint32_t)__cvta_generic_to_shared(sp);
+  auto load = [&](int64_t k0, int buf) {
+    for (int i = tid; i < LD_KT * CH; i += 256) {
+      const int r = i / CH, ch = i - r * CH;
+      const bool in = k0 + r < k_hi;
+      cp_async16(sk_u + (uint32_t)((buf * LD_KT + r) * ldk + ch * 8) * 2u, base + (in ? k0 + r : k_lo) * a.Lw + ch * 8, in ? 16 : 0);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  float o[NT][4];
+#pragma unroll
+  for (int j = 0; j < NT; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
+  float mrow[2] = {-INFINITY, -INFINITY}, lrow[2] = {0.f, 0.f};
+  const int r_in = lane >> 2, cq = (lane & 3) * 2;
+  if (k_lo < k_hi) {
+    for (int i = tid; i < 16 * CH; i += 256) {
+      const int r = i / CH, ch = i - r * CH;
+      const bool in = h0 + r < a.H;
+      cp_async16(sq_u + (uint32_t)(r * ldk + ch * 8) * 2u, sc.qa + (m * a.H + (in ? h0 + r : 0)) * a.Lw + ch * 8, in ? 16 : 0);
+    }
+    load(k_lo, 0);
+    int buf = 0;
+    for (int64_t k0 = k_lo; k0 < k_hi; k0 += LD_KT, buf ^= 1) {
+      asm volatile("cp.async.wait_group 0;" ::: "memory");
+      __syncthreads();  // the tile is in place; the other buffer, sp, wm and wl are free
+      if (k0 + LD_KT < k_hi) load(k0 + LD_KT, buf ^ 1);
+      const uint32_t kb = sk_u + (uint32_t)(buf * LD_KT * ldk) * 2u;
+      // scores of this warp's eight keys
+      float s[4] = {0.f, 0.f, 0.f, 0.f};
+      for (int kk = 0; kk < (int)a.Lw; kk += 32) {
+        uint32_t q0, q1, q2, q3, p0 = 0, p1 = 0, p2 = 0, p3 = 0, b0, b1, b2, b3;
+        const bool two = kk + 16 < (int)a.Lw;
+        const int qr = (lane & 7) + 8 * ((lane >> 3) & 1), qc = 8 * (lane >> 4);
+        ldsm_x4(sq_u + (uint32_t)(qr * ldk + kk + qc) * 2u, q0, q1, q2, q3);
+        if (two) ldsm_x4(sq_u + (uint32_t)(qr * ldk + kk + 16 + qc) * 2u, p0, p1, p2, p3);
+        // four 8-column groups of the warp's keys (the last two stay inside the padded row)
+        const int kc = kk + 8 * (lane >> 3);
+        ldsm_x4(kb + (uint32_t)((warp * 8 + (lane & 7)) * ldk + (two || lane < 16 ? kc : kk)) * 2u, b0, b1, b2, b3);
+        mma_bf16(s, q0, q1, q2, q3, b0, b1);
+        if (two) mma_bf16(s, p0, p1, p2, p3, b2, b3);
+      }
+      float mx[2] = {-INFINITY, -INFINITY};
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        s[e] = k0 + warp * 8 + cq + (e & 1) < k_hi ? s[e] * a.scale : -INFINITY;
+        mx[e >> 1] = fmaxf(mx[e >> 1], s[e]);
+      }
+#pragma unroll
+      for (int x = 0; x < 2; ++x) {
+        mx[x] = fmaxf(mx[x], __shfl_xor_sync(0xffffffffu, mx[x], 1));
+        mx[x] = fmaxf(mx[x], __shfl_xor_sync(0xffffffffu, mx[x], 2));
+        if ((lane & 3) == 0) wm[warp * 16 + r_in + 8 * x] = mx[x];
+      }
+      __syncthreads();
+      float corr[2], ls[2] = {0.f, 0.f};
+#pragma unroll
+      for (int x = 0; x < 2; ++x) {
+        float t = mrow[x];
+#pragma unroll
+        for (int w = 0; w < 8; ++w) t = fmaxf(t, wm[w * 16 + r_in + 8 * x]);  // finite: the tile has a key
+        corr[x] = expf(mrow[x] - t);
+        mrow[x] = t;
+      }
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        s[e] = expf(s[e] - mrow[e >> 1]);
+        ls[e >> 1] += s[e];
+      }
+#pragma unroll
+      for (int x = 0; x < 2; ++x) {
+        ls[x] += __shfl_xor_sync(0xffffffffu, ls[x], 1);
+        ls[x] += __shfl_xor_sync(0xffffffffu, ls[x], 2);
+        if ((lane & 3) == 0) wl[warp * 16 + r_in + 8 * x] = ls[x];
+        *(uint32_t*)(sp + (r_in + 8 * x) * 72 + warp * 8 + cq) = pack_bf16(s[2 * x], s[2 * x + 1]);
+      }
+      __syncthreads();
+#pragma unroll
+      for (int x = 0; x < 2; ++x) {
+        float t = 0.f;
+#pragma unroll
+        for (int w = 0; w < 8; ++w) t += wl[w * 16 + r_in + 8 * x];
+        lrow[x] = lrow[x] * corr[x] + t;
+      }
+#pragma unroll
+      for (int j = 0; j < NT; ++j) { o[j][0] *= corr[0]; o[j][1] *= corr[0]; o[j][2] *= corr[1]; o[j][3] *= corr[1]; }
+#pragma unroll
+      for (int kk = 0; kk < LD_KT; kk += 16) {
+        uint32_t p0, p1, p2, p3;
+        ldsm_x4(sp_u + (uint32_t)(((lane & 7) + 8 * ((lane >> 3) & 1)) * 72 + kk + 8 * (lane >> 4)) * 2u, p0, p1, p2, p3);
+#pragma unroll
+        for (int j = 0; j < NT; j += 2) {
+          uint32_t b0, b1, b2, b3;
+          const int key = kk + (lane & 7) + 8 * ((lane >> 3) & 1), col = (warp * NT + j) * 8 + 8 * (lane >> 4);
+          ldsm_x4_t(kb + (uint32_t)(key * ldk + col) * 2u, b0, b1, b2, b3);
+          mma_bf16(o[j], p0, p1, p2, p3, b0, b1);
+          mma_bf16(o[j + 1], p0, p1, p2, p3, b2, b3);
+        }
+      }
+    }
+  }
+#pragma unroll
+  for (int x = 0; x < 2; ++x) {
+    const int h = h0 + r_in + 8 * x;
+    if (h >= a.H) continue;
+    const int64_t at = (m * a.H + h) * sc.splits + split;
+    if (warp == 0 && (lane & 3) == 0) sc.ml[at] = make_float2(mrow[x], lrow[x]);
+    if (k_lo >= k_hi) continue;  // nothing here: the sum says so
+#pragma unroll
+    for (int j = 0; j < NT; ++j) {
+      const int col = (warp * NT + j) * 8 + cq;
+#pragma unroll
+      for (int y = 0; y < 2; ++y)
+        if (col + y < a.R) sc.o[at * a.R + col + y] = o[j][2 * x + y];
+    }
+  }
+}
+
+// out[m, h, e] = Wuv[h, e] . (merged latent output): eight warps, four value rows each
+__global__ void __launch_bounds__(256) k_latent_out(LatentArgs a, DecodeScratch s) {
+  asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+  extern __shared__ __align__(16) float oc[];          // [R]
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int h = blockIdx.x, e0 = blockIdx.y * 32 + warp * 4;
+  const __nv_bfloat16* uv = (const __nv_bfloat16*)a.uv + (int64_t)h * a.dv * a.R;
+  asm volatile("griddepcontrol.wait;" ::: "memory");
+  for (int64_t m = blockIdx.z; m < a.rows.M; m += gridDim.z) {
+    const int64_t at = (m * a.H + h) * s.splits;
+    float mx = -INFINITY, l = 0.f;
+    for (int k = 0; k < s.splits; ++k) mx = fmaxf(mx, s.ml[at + k].x);
+    for (int k = 0; k < s.splits; ++k) {
+      const float2 v = s.ml[at + k];
+      if (v.y > 0.f) l += v.y * expf(v.x - mx);
+    }
+    const float inv = 1.f / l;
+    __syncthreads();
+    for (int i = tid; i < a.R; i += 256) {
+      float v = 0.f;
+      for (int k = 0; k < s.splits; ++k) {
+        const float2 w = s.ml[at + k];
+        if (w.y > 0.f) v += s.o[(at + k) * a.R + i] * (expf(w.x - mx) * inv);
+      }
+      oc[i] = v;
+    }
+    __syncthreads();
+    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+    for (int i = lane; i < a.R; i += 32) {
+      const float v = oc[i];
+#pragma unroll
+      for (int y = 0; y < 4; ++y)
+        if (e0 + y < a.dv) acc[y] += v * __bfloat162float(uv[(int64_t)(e0 + y) * a.R + i]);
+    }
+#pragma unroll
+    for (int y = 0; y < 4; ++y) {
+      acc[y] = warp_sum(acc[y]);
+      if (lane == 0 && e0 + y < a.dv) ((__nv_bfloat16*)a.att)[m * a.ld_att + (int64_t)h * a.Do + e0 + y] = __float2bfloat16_rn(acc[y]);
+    }
+  }
+}
+
+int pick_nt(int R) { return R <= 128 ? 2 : R <= 256 ? 4 : R <= 512 ? 8 : 0; }
+int row_pitch(const LatentArgs& a) { return std::max((int)(a.Lw + 15) / 16 * 16, pick_nt(a.R) * 64) + 8; }
+size_t dec_smem(int ldk) { return (size_t)(16 + 2 * LD_KT) * ldk * 2 + 16 * 72 * 2 + 256 * 4; }
+
+// context slices: enough blocks for every SM, at least one tile each at full context
+int pick_splits(const LatentArgs& a, int64_t M) {
+  const int64_t base = M * ((a.H + 15) / 16);
+  int s = 1;
+  while (s < 16 && base * (s * 2) <= 2 * 148 && (int64_t)s * 2 * LD_KT <= a.Tmax) s *= 2;
+  return s;
+}
+
+template <int NT>
+int launch_dec(cg_ctx* c, const LatentArgs& a, const DecodeScratch& s) {
+  const int ldk = row_pitch(a);
+  const size_t smem = dec_smem(ldk);
+  static PerDeviceSize configured_on;
+  size_t& configured = configured_on.at(c->core->device);
+  if (smem > configured) {
+    CG_CUDA(c, cudaFuncSetAttribute(k_latent_dec<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    configured = smem;
+  }
+  dim3 grid((unsigned)a.rows.M, (unsigned)((a.H + 15) / 16), (unsigned)s.splits);
+  CG_CUDA(c, launch_kernel(c, k_latent_dec<NT>, grid, dim3(256), smem, 1, a, s, ldk));
+  CG_LAUNCHED(c);
+  return CG_OK;
+}
+
+size_t up16b(size_t n) { return (n + 15) / 16 * 16; }
+
+}  // namespace
+
+bool latent_decode_supported(int d, int R, int64_t Lw) {
+  const int nt = pick_nt(R);
+  if (!nt || Lw % 16 || d > 320) return false;
+  return dec_smem(std::max((int)Lw, nt * 64) + 8) <= 227 * 1024;
+}
+
+size_t latent_decode_scratch(const LatentArgs& a, int64_t M) {
+  const size_t n = (size_t)M * a.H;
+  return up16b(n * a.Lw * 2) + up16b(n * 16 * 8) + n * 16 * a.R * 4;
+}
+
+int k_launch_latent_decode(cg_ctx* c, const LatentArgs& a, void* scratch) {
+  const int64_t M = a.rows.M;
+  if (M == 0) return CG_OK;
+  DecodeScratch s;
+  s.splits = pick_splits(a, M);
+  const size_t n = (size_t)M * a.H;
+  s.qa = (__nv_bfloat16*)scratch;
+  s.ml = (float2*)((char*)scratch + up16b(n * a.Lw * 2));
+  s.o = (float*)((char*)s.ml + up16b(n * 16 * 8));
+  const int cb = (a.R + 63) / 64;
+  const size_t sm1 = std::max<size_t>((size_t)(a.d + 256) * 4 + (size_t)a.d * 128, 128);
+  CG_CUDA(c, launch_kernel(c, k_latent_absorb, dim3((unsigned)(a.H * cb + M)), dim3(256), sm1, 1, a, s, cb));
+  CG_LAUNCHED(c);
+  switch (pick_nt(a.R)) {
+    case 2: CG_TRY(launch_dec<2>(c, a, s)); break;
+    case 4: CG_TRY(launch_dec<4>(c, a, s)); break;
+    default: CG_TRY(launch_dec<8>(c, a, s)); break;
+  }
+  const int eb = (a.dv + 31) / 32;
+  const int mz = (int)std::min<int64_t>(M, std::max<int64_t>(1, 2 * 148 / std::max(1, a.H * eb)));
+  CG_CUDA(c, launch_kernel(c, k_latent_out, dim3((unsigned)a.H, (unsigned)eb, (unsigned)mz), dim3(256), (size_t)a.R * 4, 1, a, s));
+  CG_LAUNCHED(c);
+  return CG_OK;
+}
+
+}  // namespace cg

@@ -85,12 +85,17 @@ struct LatentArgs {
   int Do;
   int bf16;                // element type of cache, q_out, c_out, uk, uv, att
   RowsDev rows;
-  // decode scratch (bf16 path)
-  float* qa = nullptr;     // [M, H, Lw] queries mapped into the cached rows' space
-  float* oc = nullptr;     // [M, H, R] attention output in that space
 };
 int k_launch_latent_prep(cg_ctx* c, const LatentArgs& a);
 int k_launch_latent_attn(cg_ctx* c, const LatentArgs& a);  // any sizes; one CTA per (token, head)
+
+// A few new tokens per row in a bf16 context: queries are mapped into the cached rows' space, so
+// that all heads attend over the same cached rows (read once), and the result is mapped back.
+// Includes what k_launch_latent_prep does, without q_out.
+constexpr int LATENT_DECODE_TOKENS = 64;
+bool latent_decode_supported(int d, int R, int64_t Lw);
+size_t latent_decode_scratch(const LatentArgs& a, int64_t M);  // bytes
+int k_launch_latent_decode(cg_ctx* c, const LatentArgs& a, void* scratch);
 
 // --------------------------------------------------------- recurrences with a matrix state ----
 // Both mixers: [conv segment | gate segment | small segment] = W_in h.  The conv segment passes a
@@ -98,35 +103,73 @@ int k_launch_latent_attn(cg_ctx* c, const LatentArgs& a);  // any sizes; one CTA
 // dk) and values (H heads of dv); head h uses query/key head h / (H / KH).
 //   delta: S <- g S;  u = b (v - S^T k);  S <- S + k u^T;  o = S^T q        (S is dk x dv)
 //   ssd:   S <- g S + dt k v^T;  o = S^T q + D v
-struct RecurArgs {
+// The convolution's last inputs are kept by position modulo taps, so that in a decode step blocks
+// may read old inputs while another block writes the new one.
+struct RecurBase {
   int delta;
-  int H, KH, dk, dv;
+  int H, KH, dk, dv, dvs;  // dvs: dv rounded up to a multiple of 8, the row length of S and o
   int C, taps;             // conv channels
   int q_off, k_off, v_off; // columns inside the conv segment
-  int gate_off, small_off; // columns inside the projection
-  const float* proj;       // [M, ldp]
-  int64_t ldp;
   const float* conv_w;     // [C, taps]
   const float* conv_b;     // [C] or null
-  float* tail;             // [slots, taps - 1, C] last inputs of the convolution
+  float* tail;             // [slots, taps, C]
   const float *a_log, *dt_bias;  // [H]
   const float* dskip;      // [H], ssd
-  float* S;                // [slots, H, dk, dv] f32
+  float* S;                // [slots, H, dk, dvs] f32
+  float *gl, *co;          // [M, H] log decay; beta (delta) or dt (ssd)
+  float* o;                // [M, H * dvs]
+  RowsDev rows;
+};
+// Token by token, any sizes and row lengths, f32.
+struct RecurArgs : RecurBase {
+  const float* proj;       // [M, ldp]
+  int64_t ldp;
+  int gate_off, small_off; // columns inside the projection
   float* cv;               // [M, ldc] conv outputs (q, k unit vectors for delta)
   int64_t ldc;
-  float *gl, *co;          // [M, H] log decay; beta (delta) or dt (ssd)
-  float* o;                // [M, H * dv]
+};
+int k_launch_recur_steps(cg_ctx* c, const RecurArgs& a);
+
+// Prompts, 64 tokens at a time on the tensor cores (bf16 context, dk <= 128).
+constexpr int RECUR_CHUNK = 64;
+struct ChunkArgs : RecurBase {
+  const __nv_bfloat16* proj;  // [M, ldp]: conv segment first
+  int64_t ldp;
+  const float* small;      // [M, ld_small]: delta beta and a, ssd dt
+  int64_t ld_small;
+  int DKp, dvp;            // dk rounded up to 16, dv rounded up to 8
+  __nv_bfloat16 *q, *k;    // [M, KH * DKp] conv outputs
+  __nv_bfloat16* v;        // [M, H * dvp]
+  float *rq, *rk;          // [M, KH] factors that make unit vectors of them
+  __nv_bfloat16* T;        // [chunks, H, 2, 64, 64] scratch (delta)
+  const int32_t *chunk_tok, *chunk_len;  // [n_chunks] first packed token, tokens
+  const int32_t* row_chunk;              // [rows + 1]
+  int n_chunks;
+};
+bool chunk_supported(int dk);
+int k_launch_chunk_recurrence(cg_ctx* c, const ChunkArgs& a);
+
+// delta: per head, rms over dv, plain weight, times silu(gate).  ssd: times silu(gate) first, then
+// rms over each of norm_groups equal parts.
+struct GatedNorm {
+  int delta;
+  int H, dv, dvs, norm_groups;
+  const float* o;          // [M, H * dvs]
+  const void* gate;        // [M, ldg], H * dv columns
+  int64_t ldg;
+  int gate_bf16;
   const float* norm;       // delta: [dv]; ssd: [H * dv]
-  int norm_groups;         // ssd
   float eps;
   void* att;               // [M, ld_att]
   int64_t ld_att;
-  int bf16;                // element type of att
-  RowsDev rows;
+  int att_bf16;
+  int64_t M;
 };
-int k_launch_conv_heads(cg_ctx* c, const RecurArgs& a);   // proj -> cv, gl, co
-int k_launch_conv_tail(cg_ctx* c, const RecurArgs& a);    // remembers the last inputs; after k_launch_conv_heads
-int k_launch_recur_steps(cg_ctx* c, const RecurArgs& a);  // cv -> o, S: token by token, any sizes
-int k_launch_gated_norm(cg_ctx* c, const RecurArgs& a);   // o -> att
+int k_launch_gated_norm(cg_ctx* c, const GatedNorm& a);
+
+// One new token per row: convolution, gates, state update, read-out and (delta) the gated norm in
+// one kernel; n gives the output.  dk, dv <= 128.
+bool recur_decode_supported(int dk, int dv);
+int k_launch_recur_decode(cg_ctx* c, const RecurArgs& a, const GatedNorm& n);
 
 }  // namespace cg

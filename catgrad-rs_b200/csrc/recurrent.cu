@@ -28,15 +28,15 @@ __device__ __forceinline__ float softplus(float x) { return x > 20.f ? x : log1p
 __device__ __forceinline__ void st(float* p, float v) { *p = v; }
 __device__ __forceinline__ void st(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
 
-// input of the convolution `back` tokens before token m of its row (i = m's place in the row)
-__device__ __forceinline__ float conv_in(const RecurArgs& a, int64_t m, int i, int back, int c, bool first, const float* tail) {
-  if (back <= i) return a.proj[(m - back) * a.ldp + c];
-  if (first) return 0.f;
-  return tail[(int64_t)(a.taps - 1 + i - back) * a.C + c];
-}
-__device__ __forceinline__ float conv_at(const RecurArgs& a, int64_t m, int i, int c, bool first, const float* tail) {
+// The convolution at channel c of token m: the row's place i, its first position p0.
+__device__ __forceinline__ float conv_at(const RecurArgs& a, int64_t m, int i, int64_t p0, int c, const float* tail) {
   float v = a.conv_b ? a.conv_b[c] : 0.f;
-  for (int j = 0; j < a.taps; ++j) v += a.conv_w[(int64_t)c * a.taps + a.taps - 1 - j] * conv_in(a, m, i, j, c, first, tail);
+  for (int j = 0; j < a.taps; ++j) {
+    float x = 0.f;
+    if (j <= i) x = a.proj[(m - j) * a.ldp + c];
+    else if (p0 + i - j >= 0) x = tail[(int64_t)((p0 + i - j) % a.taps) * a.C + c];
+    v += a.conv_w[(int64_t)c * a.taps + a.taps - 1 - j] * x;
+  }
   return silu(v);
 }
 
@@ -47,8 +47,8 @@ __global__ void __launch_bounds__(256) k_conv_heads(RecurArgs a) {
   const int64_t m = blockIdx.x;
   const int row = a.rows.tok_row[m];
   const int i = (int)(m - a.rows.start[row]);
-  const bool first = row_pos0(a.rows, row) == 0;
-  const float* tail = a.tail + (int64_t)a.rows.slot[row] * (a.taps - 1) * a.C;
+  const int64_t p0 = row_pos0(a.rows, row);
+  const float* tail = a.tail + (int64_t)a.rows.slot[row] * a.taps * a.C;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
   float* out = a.cv + m * a.ldc;
   const int norm_units = a.delta ? 2 * a.KH : 0;          // delta: q heads then k heads, contiguous from column 0
@@ -59,7 +59,7 @@ __global__ void __launch_bounds__(256) k_conv_heads(RecurArgs a) {
       const int c0 = u * a.dk;
       float ss = 0.f;
       for (int e = lane; e < a.dk; e += 32) {
-        const float v = conv_at(a, m, i, c0 + e, first, tail);
+        const float v = conv_at(a, m, i, p0, c0 + e, tail);
         out[c0 + e] = v;
         ss += v * v;
       }
@@ -69,7 +69,7 @@ __global__ void __launch_bounds__(256) k_conv_heads(RecurArgs a) {
       for (int e = lane; e < a.dk; e += 32) out[c0 + e] *= f;  // this lane's own stores
     } else {
       const int c0 = c_rest + (u - norm_units) * 128;
-      for (int e = lane; e < 128 && c0 + e < a.C; e += 32) out[c0 + e] = conv_at(a, m, i, c0 + e, first, tail);
+      for (int e = lane; e < 128 && c0 + e < a.C; e += 32) out[c0 + e] = conv_at(a, m, i, p0, c0 + e, tail);
     }
   }
   const float* sp = a.proj + m * a.ldp + a.small_off;
@@ -80,30 +80,17 @@ __global__ void __launch_bounds__(256) k_conv_heads(RecurArgs a) {
   }
 }
 
-constexpr int MAX_TAPS = 17;
-
+// the last inputs of the convolution, at their position modulo taps
 __global__ void k_conv_tail(RecurArgs a) {
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
   asm volatile("griddepcontrol.wait;" ::: "memory");
   const int row = blockIdx.y;
   const int c = blockIdx.x * blockDim.x + threadIdx.x;
   if (c >= a.C) return;
-  const int64_t s0 = a.rows.start[row];
+  const int64_t s0 = a.rows.start[row], p0 = row_pos0(a.rows, row);
   const int len = (int)(a.rows.start[row + 1] - s0);
-  const bool first = row_pos0(a.rows, row) == 0;
-  float* tail = a.tail + (int64_t)a.rows.slot[row] * (a.taps - 1) * a.C;
-  float v[MAX_TAPS - 1];
-  const int n = a.taps - 1;
-#pragma unroll
-  for (int j = 0; j < MAX_TAPS - 1; ++j) {
-    if (j < n) {
-      const int off = len - n + j;  // place in the row; negative: before it
-      v[j] = off >= 0 ? a.proj[(s0 + off) * a.ldp + c] : (first ? 0.f : tail[(int64_t)(off + n) * a.C + c]);
-    }
-  }
-#pragma unroll
-  for (int j = 0; j < MAX_TAPS - 1; ++j)
-    if (j < n) tail[(int64_t)j * a.C + c] = v[j];
+  float* tail = a.tail + (int64_t)a.rows.slot[row] * a.taps * a.C;
+  for (int i = max(0, len - a.taps + 1); i < len; ++i) tail[(int64_t)((p0 + i) % a.taps) * a.C + c] = a.proj[(s0 + i) * a.ldp + c];
 }
 
 // One block per (32 value columns, head, row), token by token.  Four threads share a column, each
@@ -122,9 +109,9 @@ __global__ void __launch_bounds__(128) k_recur_steps(RecurArgs a) {
   const bool live = e < a.dv;
   const int64_t s0 = a.rows.start[row];
   const int len = (int)(a.rows.start[row + 1] - s0);
-  float* Sg = a.S + ((int64_t)a.rows.slot[row] * a.H + h) * a.dk * a.dv;
+  float* Sg = a.S + ((int64_t)a.rows.slot[row] * a.H + h) * a.dk * a.dvs;
   const bool first = row_pos0(a.rows, row) == 0;
-  for (int i = part; i < a.dk; i += 4) S[i * 32 + col] = live && !first ? Sg[(int64_t)i * a.dv + e] : 0.f;
+  for (int i = part; i < a.dk; i += 4) S[i * 32 + col] = live && !first ? Sg[(int64_t)i * a.dvs + e] : 0.f;
   const int kh = h / (a.H / a.KH);
   for (int t = 0; t < len; ++t) {
     const int64_t m = s0 + t;
@@ -161,59 +148,262 @@ __global__ void __launch_bounds__(128) k_recur_steps(RecurArgs a) {
     if (part == 0 && live) {
       o = (red[col] + red[32 + col]) + (red[64 + col] + red[96 + col]);
       if (a.dskip) o += a.dskip[h] * v;
-      a.o[m * (int64_t)a.H * a.dv + h * a.dv + e] = o;
+      a.o[m * (int64_t)a.H * a.dvs + h * a.dvs + e] = o;
     }
   }
   if (live)
-    for (int i = part; i < a.dk; i += 4) Sg[(int64_t)i * a.dv + e] = S[i * 32 + col];
+    for (int i = part; i < a.dk; i += 4) Sg[(int64_t)i * a.dvs + e] = S[i * 32 + col];
 }
 
-// delta: per head, rms over dv, plain weight, times silu(gate).  ssd: times silu(gate) first, then
-// rms over each of norm_groups equal parts.  One block per (norm group, token).
-template <class T>
-__global__ void k_gated_norm(RecurArgs a) {
+// ------------------------------------------------------------------ one token per row ----
+// One block per (head, row).  A thread keeps four columns of up to 16 rows of the state in
+// registers from the load to the store; sums over the key dimension go through shared memory.
+constexpr int RD_ROWS = 16;
+__global__ void __launch_bounds__(256) k_recur_decode(RecurArgs a, GatedNorm n) {
+  asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+  __shared__ float sq[128], sk[128], sv[128], so[128], sg[4];
+  __shared__ __align__(16) float red[1024];
+  const int h = blockIdx.x, row = blockIdx.y, rep = a.H / a.KH, kh = h / rep;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int lpr = a.dvs / 4, rpp = 256 / lpr;         // threads per state row, rows per pass
+  const int rg = tid / lpr, cg = tid - rg * lpr;
+  const bool act = rg < rpp;
+  asm volatile("griddepcontrol.wait;" ::: "memory");
+  const int64_t m = row, pos = row_pos0(a.rows, row);
+  const int slot = a.rows.slot[row];
+  float* Sg = a.S + ((int64_t)slot * a.H + h) * a.dk * a.dvs;
+  float4 S[RD_ROWS];
+#pragma unroll
+  for (int i = 0; i < RD_ROWS; ++i) {
+    const int r = rg + i * rpp;
+    S[i] = act && r < a.dk && pos > 0 ? *(const float4*)(Sg + (int64_t)r * a.dvs + 4 * cg) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  // short convolutions of this head's channels
+  const float* p = a.proj + m * a.ldp;
+  float* tail = a.tail + (int64_t)slot * a.taps * a.C;
+  for (int x = tid; x < 2 * a.dk + a.dvs; x += 256) {
+    const int seg = x < a.dk ? 0 : x < 2 * a.dk ? 1 : 2;
+    const int e = seg == 0 ? x : seg == 1 ? x - a.dk : x - 2 * a.dk;
+    if (seg == 2 && e >= a.dv) { sv[e] = 0.f; continue; }
+    const int c = seg == 0 ? a.q_off + kh * a.dk + e : seg == 1 ? a.k_off + kh * a.dk + e : a.v_off + h * a.dv + e;
+    const float now = p[c];
+    float v = (a.conv_b ? a.conv_b[c] : 0.f) + a.conv_w[(int64_t)c * a.taps + a.taps - 1] * now;
+    for (int j = 1; j < a.taps; ++j)
+      if (pos - j >= 0) v += a.conv_w[(int64_t)c * a.taps + a.taps - 1 - j] * tail[(int64_t)((pos - j) % a.taps) * a.C + c];
+    if (seg == 2 || h % rep == 0) tail[(int64_t)(pos % a.taps) * a.C + c] = now;  // read by no block of this step
+    (seg == 0 ? sq : seg == 1 ? sk : sv)[e] = silu(v);
+  }
+  const float* sp = p + a.small_off;
+  if (tid == 64) {
+    const float dt = softplus(sp[a.delta ? a.H + h : h] + a.dt_bias[h]);
+    sg[0] = expf(-expf(a.a_log[h]) * dt);
+    sg[1] = a.delta ? 1.f / (1.f + expf(-sp[h])) : dt;
+  }
+  __syncthreads();
+  if (a.delta) {
+    if (warp < 2) {
+      float* x = warp ? sk : sq;
+      float ss = 0.f;
+      for (int e = lane; e < a.dk; e += 32) ss += x[e] * x[e];
+      ss = warp_sum(ss);
+      const float f = (warp ? 1.f : 1.f / sqrtf((float)a.dk)) / sqrtf(ss + 1e-6f);
+      for (int e = lane; e < a.dk; e += 32) x[e] *= f;
+    }
+    __syncthreads();
+  }
+  const float g = sg[0], co = sg[1];
+  auto sum_rows = [&](float4 v) {   // over all rows of the state, for this thread's columns
+    if (act) *(float4*)(red + rg * a.dvs + 4 * cg) = v;
+    __syncthreads();
+    float4 t = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (act)
+      for (int i = 0; i < rpp; ++i) {
+        const float4 r = *(const float4*)(red + i * a.dvs + 4 * cg);
+        t.x += r.x; t.y += r.y; t.z += r.z; t.w += r.w;
+      }
+    return t;
+  };
+  float4 u = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (act) u = *(const float4*)(sv + 4 * cg);
+  const float4 v4 = u;
+  if (a.delta) {
+    float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int i = 0; i < RD_ROWS; ++i) {
+      const int r = rg + i * rpp;
+      const float k = act && r < a.dk ? sk[r] : 0.f;
+      S[i].x *= g; S[i].y *= g; S[i].z *= g; S[i].w *= g;
+      s.x += S[i].x * k; s.y += S[i].y * k; s.z += S[i].z * k; s.w += S[i].w * k;
+    }
+    s = sum_rows(s);
+    u.x -= s.x; u.y -= s.y; u.z -= s.z; u.w -= s.w;
+    __syncthreads();
+  }
+  u.x *= co; u.y *= co; u.z *= co; u.w *= co;
+  float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+  for (int i = 0; i < RD_ROWS; ++i) {
+    const int r = rg + i * rpp;
+    if (act && r < a.dk) {
+      const float k = sk[r], q = sq[r];
+      if (a.delta) {
+        S[i].x += k * u.x; S[i].y += k * u.y; S[i].z += k * u.z; S[i].w += k * u.w;
+      } else {
+        S[i].x = g * S[i].x + k * u.x; S[i].y = g * S[i].y + k * u.y;
+        S[i].z = g * S[i].z + k * u.z; S[i].w = g * S[i].w + k * u.w;
+      }
+      o.x += S[i].x * q; o.y += S[i].y * q; o.z += S[i].z * q; o.w += S[i].w * q;
+      *(float4*)(Sg + (int64_t)r * a.dvs + 4 * cg) = S[i];
+    }
+  }
+  o = sum_rows(o);
+  if (!a.delta) {
+    if (rg == 0) {
+      const float d = a.dskip[h];
+      *(float4*)(a.o + m * (int64_t)a.H * a.dvs + (int64_t)h * a.dvs + 4 * cg) =
+          make_float4(o.x + d * v4.x, o.y + d * v4.y, o.z + d * v4.z, o.w + d * v4.w);
+    }
+    return;
+  }
+  if (rg == 0) *(float4*)(so + 4 * cg) = o;
+  __syncthreads();
+  const float* gate = (const float*)n.gate + m * n.ldg + (int64_t)h * a.dv;
+  const float x = tid < a.dv ? so[tid] : 0.f;
+  const float ss = block_sum(x * x, red);
+  if (tid < a.dv) {
+    const float y = x / sqrtf(ss / (float)a.dv + n.eps) * n.norm[tid] * silu(gate[tid]);
+    const int64_t at = m * n.ld_att + (int64_t)h * a.dv + tid;
+    if (n.att_bf16) ((__nv_bfloat16*)n.att)[at] = __float2bfloat16_rn(y);
+    else ((float*)n.att)[at] = y;
+  }
+}
+
+// ------------------------------------------------------------------------- gated norm ----
+__device__ __forceinline__ float ldg1(const float* p) { return *p; }
+__device__ __forceinline__ float ldg1(const __nv_bfloat16* p) { return __bfloat162float(*p); }
+__device__ __forceinline__ float4 ldg4(const float* p) { return *(const float4*)p; }
+__device__ __forceinline__ float4 ldg4(const __nv_bfloat16* p) {
+  const uint2 r = *(const uint2*)p;
+  const float2 a = __bfloat1622float2(*(const __nv_bfloat162*)&r.x), b = __bfloat1622float2(*(const __nv_bfloat162*)&r.y);
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void st4(float* p, float4 v) { *(float4*)p = v; }
+__device__ __forceinline__ void st4(__nv_bfloat16* p, float4 v) {
+  const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+  *(uint2*)p = make_uint2(*(const uint32_t*)&lo, *(const uint32_t*)&hi);
+}
+
+// One block per (norm group, token), any sizes.
+template <class TG, class T>
+__global__ void k_gated_norm(GatedNorm a) {
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
   asm volatile("griddepcontrol.wait;" ::: "memory");
   __shared__ float sh[32];
   const int64_t m = blockIdx.y;
   const int n = a.delta ? a.dv : a.H * a.dv / a.norm_groups;
   const int c0 = blockIdx.x * n;
-  const float* o = a.o + m * (int64_t)a.H * a.dv + c0;
-  const float* gate = a.proj + m * a.ldp + a.gate_off + c0;
+  const float* o = a.o + m * (int64_t)a.H * a.dvs;
+  const TG* gate = (const TG*)a.gate + m * a.ldg + c0;
   T* out = (T*)a.att + m * a.ld_att + c0;
+  auto at = [&](int i) { const int c = c0 + i, h = c / a.dv; return o[h * a.dvs + (c - h * a.dv)]; };
   float ss = 0.f;
   for (int i = threadIdx.x; i < n; i += blockDim.x) {
-    const float v = a.delta ? o[i] : o[i] * silu(gate[i]);
+    const float v = a.delta ? at(i) : at(i) * silu(ldg1(gate + i));
     ss += v * v;
   }
   ss = block_sum(ss, sh);
   const float rms = sqrtf(ss / (float)n + a.eps);
   for (int i = threadIdx.x; i < n; i += blockDim.x) {
-    const float g = silu(gate[i]);
-    const float v = a.delta ? o[i] / rms * a.norm[i] * g : o[i] * g / rms * a.norm[c0 + i];
-    st(out + i, v);
+    const float g = silu(ldg1(gate + i));
+    st(out + i, a.delta ? at(i) / rms * a.norm[i] * g : at(i) * g / rms * a.norm[c0 + i]);
   }
+}
+
+// Groups of whole 128-bit vectors, kept in registers: G threads per group (a warp, or a block).
+template <class TG, class T, int V>
+__global__ void k_gated_norm_vec(GatedNorm a, int n, int units, int threads) {
+  asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+  asm volatile("griddepcontrol.wait;" ::: "memory");
+  __shared__ float sh[32];
+  const int per = blockDim.x / threads, sub = threadIdx.x / threads, t = threadIdx.x - sub * threads;
+  const int64_t unit = blockIdx.x * (int64_t)per + sub;
+  const int64_t m = unit / units;
+  const int c0 = (int)(unit - m * units) * n;
+  const bool live = m < a.M;
+  const float* o = a.o + m * (int64_t)a.H * a.dv + c0;
+  const TG* gate = (const TG*)a.gate + m * a.ldg + c0;
+  T* out = (T*)a.att + m * a.ld_att + c0;
+  float4 x[V];
+  float ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < V; ++j) {
+    const int i = 4 * (t + j * threads);
+    x[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (live && i < n) {
+      x[j] = *(const float4*)(o + i);
+      if (!a.delta) {
+        const float4 g = ldg4(gate + i);
+        x[j].x *= silu(g.x); x[j].y *= silu(g.y); x[j].z *= silu(g.z); x[j].w *= silu(g.w);
+      }
+    }
+    ss += x[j].x * x[j].x + x[j].y * x[j].y + x[j].z * x[j].z + x[j].w * x[j].w;
+  }
+  ss = threads == 32 ? warp_sum(ss) : block_sum(ss, sh);
+  const float inv = 1.f / sqrtf(ss / (float)n + a.eps);
+#pragma unroll
+  for (int j = 0; j < V; ++j) {
+    const int i = 4 * (t + j * threads);
+    if (!live || i >= n) continue;
+    const float4 w = *(const float4*)(a.norm + (a.delta ? 0 : c0) + i);
+    float4 r = make_float4(x[j].x * inv * w.x, x[j].y * inv * w.y, x[j].z * inv * w.z, x[j].w * inv * w.w);
+    if (a.delta) {
+      const float4 g = ldg4(gate + i);
+      r.x *= silu(g.x); r.y *= silu(g.y); r.z *= silu(g.z); r.w *= silu(g.w);
+    }
+    st4(out + i, r);
+  }
+}
+
+template <class TG, class T>
+int launch_gated_norm(cg_ctx* c, const GatedNorm& a) {
+  const int units = a.delta ? a.H : a.norm_groups;
+  const int n = a.H * a.dv / units;
+  const bool vec = a.dv == a.dvs && n % 4 == 0 && a.ldg % 4 == 0 && a.ld_att % 4 == 0 && (((uintptr_t)a.gate | (uintptr_t)a.norm) & 15) == 0 && n <= 16384;
+  if (vec && n <= 512) {
+    const int64_t blocks = (a.M * units + 7) / 8;
+    if (n <= 128) CG_CUDA(c, launch_kernel(c, k_gated_norm_vec<TG, T, 1>, dim3((unsigned)blocks), dim3(256), 0, 1, a, n, units, 32));
+    else CG_CUDA(c, launch_kernel(c, k_gated_norm_vec<TG, T, 4>, dim3((unsigned)blocks), dim3(256), 0, 1, a, n, units, 32));
+  } else if (vec) {
+    const int threads = n <= 4096 ? 256 : n <= 8192 ? 512 : 1024;
+    CG_CUDA(c, launch_kernel(c, k_gated_norm_vec<TG, T, 4>, dim3((unsigned)(a.M * units)), dim3(threads), 0, 1, a, n, units, threads));
+  } else {
+    dim3 grid((unsigned)units, (unsigned)a.M);
+    if (grid.y > 65535) return fail(c, CG_ERR_UNSUPPORTED, "recurrence: too many tokens in one portion");
+    CG_CUDA(c, launch_kernel(c, k_gated_norm<TG, T>, grid, dim3(std::min(512, (n + 31) / 32 * 32)), 0, 1, a));
+  }
+  CG_LAUNCHED(c);
+  return CG_OK;
 }
 
 }  // namespace
 
-int k_launch_conv_heads(cg_ctx* c, const RecurArgs& a) {
-  if (a.rows.M == 0) return CG_OK;
-  CG_CUDA(c, launch_kernel(c, k_conv_heads, dim3((unsigned)a.rows.M), dim3(256), 0, 1, a));
-  CG_LAUNCHED(c);
-  return CG_OK;
-}
+bool recur_decode_supported(int dk, int dv) { return dk <= 128 && dv <= 128; }
 
-int k_launch_conv_tail(cg_ctx* c, const RecurArgs& a) {
-  if (a.rows.M == 0 || a.taps <= 1) return CG_OK;
-  if (a.taps > MAX_TAPS) return fail(c, CG_ERR_UNSUPPORTED, "recurrence: too many convolution taps");
-  CG_CUDA(c, launch_kernel(c, k_conv_tail, dim3((unsigned)((a.C + 127) / 128), (unsigned)a.rows.rows), dim3(128), 0, 1, a));
+int k_launch_recur_decode(cg_ctx* c, const RecurArgs& a, const GatedNorm& n) {
+  if (a.rows.rows == 0) return CG_OK;
+  CG_CUDA(c, launch_kernel(c, k_recur_decode, dim3((unsigned)a.H, (unsigned)a.rows.rows), dim3(256), 0, 1, a, n));
   CG_LAUNCHED(c);
-  return CG_OK;
+  return a.delta ? CG_OK : k_launch_gated_norm(c, n);
 }
 
 int k_launch_recur_steps(cg_ctx* c, const RecurArgs& a) {
   if (a.rows.M == 0) return CG_OK;
+  CG_CUDA(c, launch_kernel(c, k_conv_heads, dim3((unsigned)a.rows.M), dim3(256), 0, 1, a));
+  CG_LAUNCHED(c);
+  if (a.taps > 1) {
+    CG_CUDA(c, launch_kernel(c, k_conv_tail, dim3((unsigned)((a.C + 127) / 128), (unsigned)a.rows.rows), dim3(128), 0, 1, a));
+    CG_LAUNCHED(c);
+  }
   const size_t smem = (size_t)(a.dk * 34 + 128) * 4;
   static PerDeviceSize configured_on;
   size_t& configured = configured_on.at(c->core->device);
@@ -228,17 +418,10 @@ int k_launch_recur_steps(cg_ctx* c, const RecurArgs& a) {
   return CG_OK;
 }
 
-int k_launch_gated_norm(cg_ctx* c, const RecurArgs& a) {
-  if (a.rows.M == 0) return CG_OK;
-  const int parts = a.delta ? a.H : a.norm_groups;
-  const int n = a.H * a.dv / parts;
-  const int block = std::min(512, (n + 31) / 32 * 32);
-  dim3 grid((unsigned)parts, (unsigned)a.rows.M);
-  if (grid.y > 65535) return fail(c, CG_ERR_UNSUPPORTED, "recurrence: too many tokens in one portion");
-  if (a.bf16) CG_CUDA(c, launch_kernel(c, k_gated_norm<__nv_bfloat16>, grid, dim3(block), 0, 1, a));
-  else CG_CUDA(c, launch_kernel(c, k_gated_norm<float>, grid, dim3(block), 0, 1, a));
-  CG_LAUNCHED(c);
-  return CG_OK;
+int k_launch_gated_norm(cg_ctx* c, const GatedNorm& a) {
+  if (a.M == 0) return CG_OK;
+  if (a.gate_bf16) return a.att_bf16 ? launch_gated_norm<__nv_bfloat16, __nv_bfloat16>(c, a) : launch_gated_norm<__nv_bfloat16, float>(c, a);
+  return a.att_bf16 ? launch_gated_norm<float, __nv_bfloat16>(c, a) : launch_gated_norm<float, float>(c, a);
 }
 
 }  // namespace cg

@@ -1,0 +1,687 @@
+// recurrent_chunk.cu — prompts through the matrix-state recurrences, 64 tokens at a time on the
+// tensor cores.
+//
+// With G_t the running sum of the log decays inside a chunk, S0 the state before it and u_t what
+// token t writes, both recurrences read
+//   S_t = e^{G_t} S0 + sum_{s<=t} e^{G_t - G_s} k_s u_s^T,      o_t = S_t^T q_t
+// For the state space u_t = dt_t v_t.  For the delta rule u solves a unit lower triangular system:
+//   (I + A) U = R,  A_ts = b_t e^{G_t - G_s} (k_t . k_s) (s < t),  R_t = b_t (v_t - e^{G_t} S0^T k_t)
+// T = (I + A)^-1 depends on keys and gates only, so k_delta_solve makes it for all chunks at once;
+// k_chunk_scan then walks the chunks of one (row, head, 64 value columns) with S in registers.
+//
+// Precision.  The conv outputs are bf16 (and exact as such); unit norms are kept apart as f32 factors
+// per token and head, so every product of q, k, v with itself is exact in the operands.  State,
+// decays, R, U and T are f32: as a tensor-core operand each is split into a bf16 head and a bf16
+// remainder (two or three products, about 16 bits), accumulation is f32, the state itself stays in
+// f32 accumulators and is never rounded.
+#include <algorithm>
+
+#include "mixers.h"
+#include "mma.cuh"
+
+namespace cg {
+
+namespace {
+
+constexpr int CT = 64;   // tokens per chunk
+constexpr int EB = 64;   // value columns per block
+constexpr int LE = EB + 8, LT = CT + 8;
+
+__device__ __forceinline__ float silu(float x) { return x / (1.f + __expf(-x)); }
+__device__ __forceinline__ float softplus(float x) { return x > 20.f ? x : log1pf(expf(x)); }
+__device__ __forceinline__ uint32_t sm_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
+
+// v = hi + lo, both bf16
+__device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
+  const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
+  const float2 f = __bfloat1622float2(h);
+  const __nv_bfloat162 l = __floats2bfloat162_rn(a - f.x, b - f.y);
+  hi = *(const uint32_t*)&h;
+  lo = *(const uint32_t*)&l;
+}
+
+// A fragment (16 x 16) of a row-major tile at (r0, c0)
+__device__ __forceinline__ void frag_a(uint32_t base, int ld, int r0, int c0, int lane, uint32_t* a) {
+  const int r = r0 + (lane & 7) + 8 * ((lane >> 3) & 1), c = c0 + 8 * (lane >> 4);
+  ldsm_x4(base + (uint32_t)(r * ld + c) * 2u, a[0], a[1], a[2], a[3]);
+}
+// A fragment of the transpose: the tile is stored [k][m], fragment rows m0.., columns k0..
+__device__ __forceinline__ void frag_a_t(uint32_t base, int ld, int m0, int k0, int lane, uint32_t* a) {
+  const int k = k0 + (lane & 7) + 8 * (lane >> 4), m = m0 + 8 * ((lane >> 3) & 1);
+  ldsm_x4_t(base + (uint32_t)(k * ld + m) * 2u, a[0], a[1], a[2], a[3]);
+}
+// B fragments of two neighbouring 8-column tiles; the operand is stored [k][n] ...
+__device__ __forceinline__ void frag_b_kn(uint32_t base, int ld, int k0, int n0, int lane, uint32_t* b) {
+  const int k = k0 + (lane & 7) + 8 * ((lane >> 3) & 1), n = n0 + 8 * (lane >> 4);
+  ldsm_x4_t(base + (uint32_t)(k * ld + n) * 2u, b[0], b[1], b[2], b[3]);
+}
+// ... or [n][k]
+__device__ __forceinline__ void frag_b_nk(uint32_t base, int ld, int k0, int n0, int lane, uint32_t* b) {
+  const int n = n0 + (lane & 7) + 8 * (lane >> 4), k = k0 + 8 * ((lane >> 3) & 1);
+  ldsm_x4(base + (uint32_t)(n * ld + k) * 2u, b[0], b[1], b[2], b[3]);
+}
+
+// ------------------------------------------------------------- short convolutions ----
+// Any sizes: one block per token, a warp per query / key head or 128 other channels.  Queries and
+// keys are laid out with DKp values per head, values with dvp.
+__global__ void __launch_bounds__(256) k_conv_chunk_any(ChunkArgs a) {
+  asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+  asm volatile("griddepcontrol.wait;" ::: "memory");
+  const int64_t m = blockIdx.x;
+  const int row = a.rows.tok_row[m];
+  const int64_t p0 = row_pos0(a.rows, row);
+  const int i = (int)(m - a.rows.start[row]);
+  const float* tail = a.tail + (int64_t)a.rows.slot[row] * a.taps * a.C;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  auto conv = [&](int c) {
+    float v = a.conv_b ? a.conv_b[c] : 0.f;
+    for (int j = 0; j < a.taps; ++j) {
+      float x = 0.f;
+      if (j <= i) x = __bfloat162float(a.proj[(m - j) * a.ldp + c]);
+      else if (p0 + i - j >= 0) x = tail[(int64_t)((p0 + i - j) % a.taps) * a.C + c];
+      v += a.conv_w[(int64_t)c * a.taps + a.taps - 1 - j] * x;
+    }
+    return silu(v);
+  };
+  for (int u = warp; u < 2 * a.KH; u += nw) {
+    const bool isk = u >= a.KH;
+    const int h = isk ? u - a.KH : u;
+    const int c0 = (isk ? a.k_off : a.q_off) + h * a.dk;
+    __nv_bfloat16* out = (isk ? a.k : a.q) + m * (int64_t)a.KH * a.DKp + (int64_t)h * a.DKp;
+    float ss = 0.f;
+    for (int e = lane; e < a.DKp; e += 32) {
+      const __nv_bfloat16 b = __float2bfloat16_rn(e < a.dk ? conv(c0 + e) : 0.f);
+      out[e] = b;
+      const float f = __bfloat162float(b);
+      ss += f * f;
+    }
+#pragma unroll
+    for (int o = 16; o; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if (lane == 0)
+      (isk ? a.rk : a.rq)[m * a.KH + h] = a.delta ? (isk ? 1.f : rsqrtf((float)a.dk)) / sqrtf(ss + 1e-6f) : 1.f;
+  }
+  for (int x = threadIdx.x; x < a.H * a.dvp; x += blockDim.x) {
+    const int h = x / a.dvp, e = x - h * a.dvp;
+    a.v[m * (int64_t)a.H * a.dvp + x] = __float2bfloat16_rn(e < a.dv ? conv(a.v_off + h * a.dv + e) : 0.f);
+  }
+}
+
+// Sizes in multiples of 8: a thread takes 8 neighbouring channels of 16 tokens and slides over
+// them.  Same outputs.
+constexpr int CONV_TOK = 16;
+template <int TAPS>
+__global__ void __launch_bounds__(128) k_conv_chunk(ChunkArgs a) {
+  asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+  asm volatile("griddepcontrol.wait;" ::: "memory");
+  const int chunk = blockIdx.y / (CT / CONV_TOK), sub = blockIdx.y % (CT / CONV_TOK);
+  const int t_lo = sub * CONV_TOK, t_hi = min(t_lo + CONV_TOK, a.chunk_len[chunk]);
+  if (t_lo >= t_hi) return;
+  const int64_t m0 = a.chunk_tok[chunk] + t_lo;
+  const int row = a.rows.tok_row[m0];
+  const int64_t p0 = row_pos0(a.rows, row);
+  const int i0 = (int)(m0 - a.rows.start[row]);
+  const int c = (blockIdx.x * 128 + threadIdx.x) * 8;
+  const bool live = c < a.C;
+  const int cc = live ? c : 0;
+  const float* tail = a.tail + (int64_t)a.rows.slot[row] * a.taps * a.C + cc;
+  float w[TAPS][8], bias[8];
+#pragma unroll
+  for (int e = 0; e < 8; ++e) {
+    bias[e] = a.conv_b ? a.conv_b[cc + e] : 0.f;
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) w[j][e] = a.conv_w[(int64_t)(cc + e) * TAPS + TAPS - 1 - j];
+  }
+  // x[j]: the input j tokens back
+  float x[TAPS][8];
+#pragma unroll
+  for (int j = 1; j < TAPS; ++j) {
+#pragma unroll
+    for (int e = 0; e < 8; ++e) x[j][e] = 0.f;
+    if (j <= i0) {
+      const uint4 r = *(const uint4*)(a.proj + (m0 - j) * a.ldp + cc);
+      const uint32_t* p = &r.x;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const float2 f = __bfloat1622float2(*(const __nv_bfloat162*)&p[e]);
+        x[j][2 * e] = f.x; x[j][2 * e + 1] = f.y;
+      }
+    } else if (p0 + i0 - j >= 0) {
+      const float* tp = tail + (int64_t)((p0 + i0 - j) % a.taps) * a.C;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) x[j][e] = tp[e];
+    }
+  }
+  // where these channels go
+  const int qk = a.KH * a.dk;
+  __nv_bfloat16* out;
+  float* rn = nullptr;
+  int64_t ld;
+  float f = 1.f;
+  if (c >= a.v_off && c < a.v_off + a.H * a.dv) {
+    const int h = (c - a.v_off) / a.dv, e = (c - a.v_off) - h * a.dv;
+    out = a.v + (int64_t)h * a.dvp + e; ld = (int64_t)a.H * a.dvp;
+  } else {
+    const bool isk = c >= a.k_off && c < a.k_off + qk;
+    const int off = c - (isk ? a.k_off : a.q_off);
+    const int h = off / a.dk, e = off - h * a.dk;
+    out = (isk ? a.k : a.q) + (int64_t)h * a.DKp + e; ld = (int64_t)a.KH * a.DKp;
+    if (e == 0) rn = (isk ? a.rk : a.rq) + h;
+    if (!isk) f = rsqrtf((float)a.dk);
+  }
+  const int lanes = a.dk / 8;  // threads of a head: a power of two dividing the warp
+  for (int t = t_lo; t < t_hi; ++t) {
+    const int64_t m = m0 + t - t_lo;
+    const uint4 r = *(const uint4*)(a.proj + m * a.ldp + cc);
+    const uint32_t* p = &r.x;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float2 g = __bfloat1622float2(*(const __nv_bfloat162*)&p[e]);
+      x[0][2 * e] = g.x; x[0][2 * e + 1] = g.y;
+    }
+    uint32_t o[4];
+    float ss = 0.f;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      float y[2];
+#pragma unroll
+      for (int b = 0; b < 2; ++b) {
+        float v = bias[2 * e + b];
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) v += w[j][2 * e + b] * x[j][2 * e + b];
+        y[b] = silu(v);
+      }
+      const __nv_bfloat162 h2 = __floats2bfloat162_rn(y[0], y[1]);
+      o[e] = *(const uint32_t*)&h2;
+      const float2 g = __bfloat1622float2(h2);
+      ss += g.x * g.x + g.y * g.y;
+    }
+    if (live) *(uint4*)(out + m * ld) = make_uint4(o[0], o[1], o[2], o[3]);
+    if (a.delta) {
+      for (int s = lanes / 2; s; s >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, s);
+      if (live && rn) rn[m * a.KH] = f / sqrtf(ss + 1e-6f);
+    } else if (live && rn) rn[m * a.KH] = 1.f;
+#pragma unroll
+    for (int j = TAPS - 1; j > 0; --j)
+#pragma unroll
+      for (int e = 0; e < 8; ++e) x[j][e] = x[j - 1][e];
+  }
+}
+
+// log decays and write strengths
+__global__ void k_gates(ChunkArgs a) {
+  asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+  asm volatile("griddepcontrol.wait;" ::: "memory");
+  const int64_t n = a.rows.M * a.H;
+  for (int64_t i = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; i < n; i += (int64_t)gridDim.x * blockDim.x) {
+    const int64_t m = i / a.H;
+    const int h = (int)(i - m * a.H);
+    const float* sp = a.small + m * a.ld_small;
+    const float dt = softplus(sp[a.delta ? a.H + h : h] + a.dt_bias[h]);
+    a.gl[i] = -expf(a.a_log[h]) * dt;
+    a.co[i] = a.delta ? 1.f / (1.f + expf(-sp[h])) : dt;
+  }
+}
+
+// the last inputs of the convolution, at their position modulo taps
+__global__ void k_conv_tail_ring(ChunkArgs a) {
+  asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+  asm volatile("griddepcontrol.wait;" ::: "memory");
+  const int row = blockIdx.y;
+  const int c = blockIdx.x * blockDim.x + threadIdx.x;
+  if (c >= a.C) return;
+  const int64_t s0 = a.rows.start[row], p0 = row_pos0(a.rows, row);
+  const int len = (int)(a.rows.start[row + 1] - s0);
+  float* tail = a.tail + (int64_t)a.rows.slot[row] * a.taps * a.C;
+  for (int i = max(0, len - a.taps + 1); i < len; ++i)
+    tail[(int64_t)((p0 + i) % a.taps) * a.C + c] = __bfloat162float(a.proj[(s0 + i) * a.ldp + c]);
+}
+
+// ------------------------------------------------------------------ gates of a chunk ----
+struct Gates {
+  float G[CT], co[CT], rq[CT], rk[CT];
+  float last;  // sum of the chunk's log decays
+};
+// by one warp: lane l takes tokens 2 l and 2 l + 1
+__device__ __forceinline__ void load_gates(const ChunkArgs& a, int chunk, int h, int kh, Gates* g, int lane) {
+  const int len = a.chunk_len[chunk];
+  const int64_t m0 = a.chunk_tok[chunk];
+  float l[2];
+#pragma unroll
+  for (int b = 0; b < 2; ++b) {
+    const int t = 2 * lane + b;
+    const bool in = t < len;
+    l[b] = in ? a.gl[(m0 + t) * a.H + h] : 0.f;
+    g->co[t] = in ? a.co[(m0 + t) * a.H + h] : 0.f;
+    g->rq[t] = in ? a.rq[(m0 + t) * a.KH + kh] : 0.f;
+    g->rk[t] = in ? a.rk[(m0 + t) * a.KH + kh] : 0.f;
+  }
+  float sum = l[0] + l[1], inc = sum;
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const float v = __shfl_up_sync(0xffffffffu, inc, o);
+    if (lane >= o) inc += v;
+  }
+  g->G[2 * lane] = inc - sum + l[0];
+  g->G[2 * lane + 1] = inc;
+  if (lane == 31) g->last = inc;
+}
+
+// ------------------------------------------------------------------ T = (I + A)^-1 ----
+template <int DK>
+__global__ void __launch_bounds__(128) k_delta_solve(ChunkArgs a) {
+  asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+  asm volatile("griddepcontrol.wait;" ::: "memory");
+  constexpr int LK = DK + 8, LA = 68, LX = 80;
+  extern __shared__ __align__(16) uint8_t smem[];
+  float* A = (float*)smem;                       // [64][LA]
+  float* X = A + CT * LA;                        // [64][LX]
+  __nv_bfloat16* K = (__nv_bfloat16*)X;          // [64][LK], dead before X is written
+  __shared__ Gates g;
+  const int chunk = blockIdx.x, h = blockIdx.y, kh = h / (a.H / a.KH);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int len = a.chunk_len[chunk];
+  const int64_t m0 = a.chunk_tok[chunk];
+  const uint32_t ku = sm_u32(K);
+  const int ch = a.DKp / 8;
+  for (int i = tid; i < CT * (DK / 8); i += 128) {
+    const int r = i / (DK / 8), c = i - r * (DK / 8);
+    const bool in = r < len && c < ch;
+    cp_async16(ku + (uint32_t)(r * LK + c * 8) * 2u, a.k + (m0 + (in ? r : 0)) * (int64_t)a.KH * a.DKp + (int64_t)kh * a.DKp + (in ? c * 8 : 0),
+               in ? 16 : 0);
+  }
+  if (warp == 0) load_gates(a, chunk, h, kh, &g, lane);
+  cp_async_wait_all();
+  __syncthreads();
+  float acc[8][4];
+#pragma unroll
+  for (int j = 0; j < 8; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
+#pragma unroll
+  for (int kk = 0; kk < DK; kk += 16) {
+    uint32_t fa[4], fb[4];
+    frag_a(ku, LK, warp * 16, kk, lane, fa);
+#pragma unroll
+    for (int j = 0; j < 8; j += 2) {
+      frag_b_nk(ku, LK, kk, j * 8, lane, fb);
+      mma_bf16(acc[j], fa[0], fa[1], fa[2], fa[3], fb[0], fb[1]);
+      mma_bf16(acc[j + 1], fa[0], fa[1], fa[2], fa[3], fb[2], fb[3]);
+    }
+  }
+#pragma unroll
+  for (int j = 0; j < 8; ++j)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int t = warp * 16 + (lane >> 2) + 8 * (e >> 1), s = j * 8 + (lane & 3) * 2 + (e & 1);
+      A[t * LA + s] = s < t ? g.co[t] * g.rk[t] * g.rk[s] * expf(g.G[t] - g.G[s]) * acc[j][e] : 0.f;
+    }
+  __syncthreads();
+  // forward substitution, column j of the inverse by two neighbouring lanes (even and odd terms)
+  const int j = tid >> 1, half = tid & 1, s_lo = (tid >> 5) * 16;
+  for (int i = s_lo; i < CT; ++i) {
+    const float* Ai = A + i * LA;
+    float v0 = 0.f, v1 = 0.f;
+    int s = s_lo + half;
+    for (; s + 2 < i; s += 4) {
+      v0 += Ai[s] * X[s * LX + j];
+      v1 += Ai[s + 2] * X[(s + 2) * LX + j];
+    }
+    if (s < i) v0 += Ai[s] * X[s * LX + j];
+    v0 += v1;
+    v0 += __shfl_xor_sync(0xffffffffu, v0, 1);
+    if (half == 0) X[i * LX + j] = i < j ? 0.f : (i == j ? 1.f : 0.f) - v0;
+    __syncwarp();
+  }
+  __syncthreads();
+  __nv_bfloat16* out = a.T + ((int64_t)chunk * a.H + h) * 2 * CT * CT;
+  for (int i = tid; i < CT * CT / 2; i += 128) {
+    const int r = i / (CT / 2), c = (i - r * (CT / 2)) * 2;
+    const int first = c & ~15;  // rows above a column group's first were never written
+    const float x0 = r >= first ? X[r * LX + c] : 0.f, x1 = r >= first ? X[r * LX + c + 1] : 0.f;
+    uint32_t hi, lo;
+    split2(x0, x1, hi, lo);
+    *(uint32_t*)(out + r * CT + c) = hi;
+    *(uint32_t*)(out + CT * CT + r * CT + c) = lo;
+  }
+}
+
+// ------------------------------------------------------------------ the walk ----------
+template <int DK, bool DELTA>
+struct ScanSmem {
+  static constexpr int LK = DK + 8;
+  static constexpr uint32_t Q = 0, K = Q + CT * LK * 2, V = K + CT * LK * 2, T = V + CT * LE * 2;
+  static constexpr uint32_t STAGE = T + (DELTA ? 2 * CT * LT * 2 : 0);
+  static constexpr uint32_t S = 2 * STAGE;                       // [2][DK][LE]
+  static constexpr uint32_t R = S + 2 * DK * LE * 2;             // [2][64][LE]: R, then U (delta)
+  static constexpr uint32_t P = R + (DELTA ? 2 * CT * LE * 2 : 0);  // [2][64][LT]
+  static constexpr uint32_t UP = P + 2 * CT * LT * 2;            // [2][64][LE]
+  static constexpr uint32_t GATES = UP + 2 * CT * LE * 2;
+  static constexpr uint32_t BYTES = GATES + 2 * sizeof(Gates);
+};
+
+template <int DK, bool DELTA>
+__global__ void __launch_bounds__(256, 1) k_chunk_scan(ChunkArgs a) {
+  using L = ScanSmem<DK, DELTA>;
+  constexpr int LK = L::LK;
+  asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+  asm volatile("griddepcontrol.wait;" ::: "memory");
+  extern __shared__ __align__(16) uint8_t smem[];
+  const uint32_t base = sm_u32(smem);
+  Gates* gates = (Gates*)(smem + L::GATES);
+  const int e0 = blockIdx.x * EB, h = blockIdx.y, row = blockIdx.z, kh = h / (a.H / a.KH);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int wm = warp & 3, wn = warp >> 2;            // this warp's 16 tokens and 32 columns
+  const int r_in = lane >> 2, cq = (lane & 3) * 2;
+  const int c0 = a.row_chunk[row], c1 = a.row_chunk[row + 1];
+  const bool first = row_pos0(a.rows, row) == 0;
+  const int vw = min(EB, a.dvp - e0);                 // columns that exist (multiple of 8)
+
+  auto load = [&](int chunk, int stage) {
+    const int len = a.chunk_len[chunk];
+    const int64_t m0 = a.chunk_tok[chunk];
+    const uint32_t b = base + (uint32_t)stage * L::STAGE;
+    const int ch = a.DKp / 8;
+    for (int i = tid; i < CT * (DK / 8); i += 256) {
+      const int r = i / (DK / 8), c = i - r * (DK / 8);
+      const bool in = r < len && c < ch;
+      const int64_t o = (m0 + (in ? r : 0)) * (int64_t)a.KH * a.DKp + (int64_t)kh * a.DKp + (in ? c * 8 : 0);
+      const uint32_t d = (uint32_t)(r * LK + c * 8) * 2u;
+      cp_async16(b + L::Q + d, a.q + o, in ? 16 : 0);
+      cp_async16(b + L::K + d, a.k + o, in ? 16 : 0);
+    }
+    for (int i = tid; i < CT * (EB / 8); i += 256) {
+      const int r = i / (EB / 8), c = i - r * (EB / 8);
+      const bool in = r < len && c * 8 < vw;
+      cp_async16(b + L::V + (uint32_t)(r * LE + c * 8) * 2u,
+                 a.v + (m0 + (in ? r : 0)) * (int64_t)a.H * a.dvp + (int64_t)h * a.dvp + (in ? e0 + c * 8 : 0), in ? 16 : 0);
+    }
+    if (DELTA) {
+      const __nv_bfloat16* t = a.T + ((int64_t)chunk * a.H + h) * 2 * CT * CT;
+      for (int i = tid; i < 2 * CT * (CT / 8); i += 256) {
+        const int r = i / (CT / 8), c = i - r * (CT / 8);
+        cp_async16(b + L::T + (uint32_t)(r * LT + c * 8) * 2u, t + r * CT + c * 8, 16);
+      }
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  load(c0, 0);
+  if (warp == 7) load_gates(a, c0, h, kh, &gates[0], lane);
+
+  // the state: DK / 16 row tiles over the warps
+  constexpr int SN = DK == 128 ? 8 : 4;               // 8-column tiles a warp holds
+  const int sr = DK == 128 ? warp * 16 : wm * 16, sc = DK == 128 ? 0 : wn * 32;
+  float S[SN][4];
+  float* Sg = a.S + ((int64_t)a.rows.slot[row] * a.H + h) * a.dk * a.dvs;
+#pragma unroll
+  for (int j = 0; j < SN; ++j)
+#pragma unroll
+    for (int b = 0; b < 2; ++b) {
+      const int r = sr + r_in + 8 * b, c = e0 + sc + j * 8 + cq;
+      float2 v = make_float2(0.f, 0.f);
+      if (!first && r < a.dk && c < a.dvs) v = *(const float2*)(Sg + (int64_t)r * a.dvs + c);
+      S[j][2 * b] = v.x; S[j][2 * b + 1] = v.y;
+    }
+  auto publish_state = [&]() {
+#pragma unroll
+    for (int j = 0; j < SN; ++j)
+#pragma unroll
+      for (int b = 0; b < 2; ++b) {
+        uint32_t hi, lo;
+        split2(S[j][2 * b], S[j][2 * b + 1], hi, lo);
+        const uint32_t o = (uint32_t)((sr + r_in + 8 * b) * LE + sc + j * 8 + cq) * 2u;
+        *(uint32_t*)(smem + L::S + o) = hi;
+        *(uint32_t*)(smem + L::S + DK * LE * 2 + o) = lo;
+      }
+  };
+  publish_state();
+  const float dsk = a.dskip ? a.dskip[h] : 0.f;
+
+  for (int c = c0; c < c1; ++c) {
+    const int stage = (c - c0) & 1;
+    const uint32_t b = base + (uint32_t)stage * L::STAGE;
+    const uint8_t* bs = smem + (size_t)stage * L::STAGE;
+    const Gates& g = gates[stage];
+    cp_async_wait_all();
+    __syncthreads();  // tiles, gates and state of this chunk are in place; the other stage is free
+    if (c + 1 < c1) {
+      load(c + 1, stage ^ 1);
+      if (warp == 7) load_gates(a, c + 1, h, kh, &gates[stage ^ 1], lane);
+    }
+    const float glast = g.last;
+    const int t0 = wm * 16 + r_in;                    // this thread's tokens: t0 and t0 + 8
+    float qs[4][4];                                    // Q S0
+    {
+      float ks[4][4], qk[4][4];                        // K S0 (delta), Q K^T
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) qs[j][e] = ks[j][e] = qk[j][e] = 0.f;
+      const bool below = wn * 32 <= wm * 16 + 15;      // some key of this tile is visible to some token
+#pragma unroll
+      for (int kk = 0; kk < DK; kk += 16) {
+        uint32_t fq[4], fk[4], fb[4];
+        frag_a(b + L::Q, LK, wm * 16, kk, lane, fq);
+        if (DELTA) frag_a(b + L::K, LK, wm * 16, kk, lane, fk);
+#pragma unroll
+        for (int j = 0; j < 4; j += 2) {
+#pragma unroll
+          for (int part = 0; part < 2; ++part) {
+            frag_b_kn(base + L::S + (uint32_t)(part * DK * LE * 2), LE, kk, wn * 32 + j * 8, lane, fb);
+            mma_bf16(qs[j], fq[0], fq[1], fq[2], fq[3], fb[0], fb[1]);
+            mma_bf16(qs[j + 1], fq[0], fq[1], fq[2], fq[3], fb[2], fb[3]);
+            if (DELTA) {
+              mma_bf16(ks[j], fk[0], fk[1], fk[2], fk[3], fb[0], fb[1]);
+              mma_bf16(ks[j + 1], fk[0], fk[1], fk[2], fk[3], fb[2], fb[3]);
+            }
+          }
+          if (below) {
+            frag_b_nk(b + L::K, LK, kk, wn * 32 + j * 8, lane, fb);
+            mma_bf16(qk[j], fq[0], fq[1], fq[2], fq[3], fb[0], fb[1]);
+            mma_bf16(qk[j + 1], fq[0], fq[1], fq[2], fq[3], fb[2], fb[3]);
+          }
+        }
+      }
+      // P and R (or the state's addends) into shared memory, split
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+#pragma unroll
+        for (int x = 0; x < 2; ++x) {
+          const int t = t0 + 8 * x, n = wn * 32 + j * 8 + cq;
+          float p[2];
+#pragma unroll
+          for (int y = 0; y < 2; ++y) {
+            const int s = n + y;
+            p[y] = s <= t ? expf(g.G[t] - g.G[s]) * g.rq[t] * g.rk[s] * (DELTA ? 1.f : g.co[s]) * qk[j][2 * x + y] : 0.f;
+          }
+          uint32_t hi, lo;
+          split2(p[0], p[1], hi, lo);
+          const uint32_t o = (uint32_t)(t * LT + n) * 2u;
+          *(uint32_t*)(smem + L::P + o) = hi;
+          *(uint32_t*)(smem + L::P + CT * LT * 2 + o) = lo;
+          const float2 v = __bfloat1622float2(*(const __nv_bfloat162*)(bs + L::V + (uint32_t)(t * LE + n) * 2u));
+          const uint32_t oe = (uint32_t)(t * LE + n) * 2u;
+          if (DELTA) {
+            const float f = expf(g.G[t]) * g.rk[t];
+            split2(g.co[t] * (v.x - f * ks[j][2 * x]), g.co[t] * (v.y - f * ks[j][2 * x + 1]), hi, lo);
+            *(uint32_t*)(smem + L::R + oe) = hi;
+            *(uint32_t*)(smem + L::R + CT * LE * 2 + oe) = lo;
+          } else {
+            const float f = g.co[t] * expf(glast - g.G[t]) * g.rk[t];
+            split2(f * v.x, f * v.y, hi, lo);
+            *(uint32_t*)(smem + L::UP + oe) = hi;
+            *(uint32_t*)(smem + L::UP + CT * LE * 2 + oe) = lo;
+          }
+        }
+    }
+    __syncthreads();
+    if (DELTA) {
+      // U = T R
+      float u[4][4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) u[j][0] = u[j][1] = u[j][2] = u[j][3] = 0.f;
+      for (int kk = 0; kk <= wm * 16; kk += 16) {
+        uint32_t th[4], tl[4], fh[4], fl[4];
+        frag_a(b + L::T, LT, wm * 16, kk, lane, th);
+        frag_a(b + L::T + CT * LT * 2, LT, wm * 16, kk, lane, tl);
+#pragma unroll
+        for (int j = 0; j < 4; j += 2) {
+          frag_b_kn(base + L::R, LE, kk, wn * 32 + j * 8, lane, fh);
+          frag_b_kn(base + L::R + CT * LE * 2, LE, kk, wn * 32 + j * 8, lane, fl);
+#pragma unroll
+          for (int y = 0; y < 2; ++y) {
+            mma_bf16(u[j + y], th[0], th[1], th[2], th[3], fh[2 * y], fh[2 * y + 1]);
+            mma_bf16(u[j + y], th[0], th[1], th[2], th[3], fl[2 * y], fl[2 * y + 1]);
+            mma_bf16(u[j + y], tl[0], tl[1], tl[2], tl[3], fh[2 * y], fh[2 * y + 1]);
+          }
+        }
+      }
+      // U takes R's place once the four warps of these columns have read it
+      asm volatile("bar.sync %0, 128;" ::"r"(1 + wn) : "memory");
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+#pragma unroll
+        for (int x = 0; x < 2; ++x) {
+          const int t = t0 + 8 * x;
+          const uint32_t oe = (uint32_t)(t * LE + wn * 32 + j * 8 + cq) * 2u;
+          uint32_t hi, lo;
+          split2(u[j][2 * x], u[j][2 * x + 1], hi, lo);
+          *(uint32_t*)(smem + L::R + oe) = hi;
+          *(uint32_t*)(smem + L::R + CT * LE * 2 + oe) = lo;
+          const float f = expf(glast - g.G[t]) * g.rk[t];
+          split2(f * u[j][2 * x], f * u[j][2 * x + 1], hi, lo);
+          *(uint32_t*)(smem + L::UP + oe) = hi;
+          *(uint32_t*)(smem + L::UP + CT * LE * 2 + oe) = lo;
+        }
+      __syncthreads();
+    }
+    // O = e^G rq (Q S0) + P U
+    {
+#pragma unroll
+      for (int x = 0; x < 2; ++x) {
+        const float f = expf(g.G[t0 + 8 * x]) * g.rq[t0 + 8 * x];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) { qs[j][2 * x] *= f; qs[j][2 * x + 1] *= f; }
+      }
+      for (int kk = 0; kk <= wm * 16; kk += 16) {
+        uint32_t ph[4], pl[4], fh[4], fl[4];
+        frag_a(base + L::P, LT, wm * 16, kk, lane, ph);
+        frag_a(base + L::P + CT * LT * 2, LT, wm * 16, kk, lane, pl);
+#pragma unroll
+        for (int j = 0; j < 4; j += 2) {
+          frag_b_kn(DELTA ? base + L::R : b + L::V, LE, kk, wn * 32 + j * 8, lane, fh);
+          if (DELTA) frag_b_kn(base + L::R + CT * LE * 2, LE, kk, wn * 32 + j * 8, lane, fl);
+#pragma unroll
+          for (int y = 0; y < 2; ++y) {
+            mma_bf16(qs[j + y], ph[0], ph[1], ph[2], ph[3], fh[2 * y], fh[2 * y + 1]);
+            mma_bf16(qs[j + y], pl[0], pl[1], pl[2], pl[3], fh[2 * y], fh[2 * y + 1]);
+            if (DELTA) mma_bf16(qs[j + y], ph[0], ph[1], ph[2], ph[3], fl[2 * y], fl[2 * y + 1]);
+          }
+        }
+      }
+      const int len = a.chunk_len[c];
+      const int64_t m0 = a.chunk_tok[c];
+#pragma unroll
+      for (int x = 0; x < 2; ++x) {
+        const int t = t0 + 8 * x;
+        if (t >= len) continue;
+        float* o = a.o + (m0 + t) * (int64_t)a.H * a.dvs + (int64_t)h * a.dvs + e0;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const int n = wn * 32 + j * 8 + cq;
+          if (e0 + n >= a.dvs) continue;
+          float2 r = make_float2(qs[j][2 * x], qs[j][2 * x + 1]);
+          if (!DELTA) {
+            const float2 v = __bfloat1622float2(*(const __nv_bfloat162*)(bs + L::V + (uint32_t)(t * LE + n) * 2u));
+            r.x += dsk * v.x; r.y += dsk * v.y;
+          }
+          *(float2*)(o + n) = r;
+        }
+      }
+    }
+    // S = e^{G_last} S + K^T U'
+    {
+      const float f = expf(glast);
+#pragma unroll
+      for (int j = 0; j < SN; ++j) { S[j][0] *= f; S[j][1] *= f; S[j][2] *= f; S[j][3] *= f; }
+#pragma unroll
+      for (int kk = 0; kk < CT; kk += 16) {
+        uint32_t fk[4], fb[4];
+        frag_a_t(b + L::K, LK, sr, kk, lane, fk);
+#pragma unroll
+        for (int part = 0; part < 2; ++part)
+#pragma unroll
+          for (int j = 0; j < SN; j += 2) {
+            frag_b_kn(base + L::UP + (uint32_t)(part * CT * LE * 2), LE, kk, sc + j * 8, lane, fb);
+            mma_bf16(S[j], fk[0], fk[1], fk[2], fk[3], fb[0], fb[1]);
+            mma_bf16(S[j + 1], fk[0], fk[1], fk[2], fk[3], fb[2], fb[3]);
+          }
+      }
+      publish_state();  // every warp read the old one before the barrier above
+    }
+  }
+#pragma unroll
+  for (int j = 0; j < SN; ++j)
+#pragma unroll
+    for (int b = 0; b < 2; ++b) {
+      const int r = sr + r_in + 8 * b, c = e0 + sc + j * 8 + cq;
+      if (r < a.dk && c < a.dvs) *(float2*)(Sg + (int64_t)r * a.dvs + c) = make_float2(S[j][2 * b], S[j][2 * b + 1]);
+    }
+}
+
+template <int DK, bool DELTA>
+int launch_scan(cg_ctx* c, const ChunkArgs& a) {
+  using L = ScanSmem<DK, DELTA>;
+  static_assert(L::BYTES <= 227 * 1024, "shared memory");
+  static PerDeviceFlag configured_on;
+  bool& configured = configured_on.at(c->core->device);
+  if (!configured) {
+    CG_CUDA(c, cudaFuncSetAttribute(k_chunk_scan<DK, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)L::BYTES));
+    configured = true;
+  }
+  dim3 grid((unsigned)((a.dv + EB - 1) / EB), (unsigned)a.H, (unsigned)a.rows.rows);
+  CG_CUDA(c, launch_kernel(c, k_chunk_scan<DK, DELTA>, grid, dim3(256), L::BYTES, 1, a));
+  CG_LAUNCHED(c);
+  return CG_OK;
+}
+template <int DK>
+int launch_solve(cg_ctx* c, const ChunkArgs& a) {
+  constexpr size_t smem = (size_t)CT * 68 * 4 + std::max((size_t)CT * 80 * 4, (size_t)CT * (DK + 8) * 2);
+  CG_CUDA(c, launch_kernel(c, k_delta_solve<DK>, dim3((unsigned)a.n_chunks, (unsigned)a.H), dim3(128), smem, 1, a));
+  CG_LAUNCHED(c);
+  return CG_OK;
+}
+
+}  // namespace
+
+bool chunk_supported(int dk) { return dk <= 128; }
+
+int k_launch_chunk_recurrence(cg_ctx* c, const ChunkArgs& a) {
+  if (a.rows.M == 0) return CG_OK;
+  const int lanes = a.dk / 8;
+  const bool fast = a.dk % 8 == 0 && a.dv % 8 == 0 && a.DKp == a.dk && (!a.delta || (lanes & (lanes - 1)) == 0) && a.taps >= 1 && a.taps <= 4;
+  if (fast) {
+    dim3 grid((unsigned)((a.C + 1023) / 1024), (unsigned)(a.n_chunks * (CT / CONV_TOK)));
+    if (grid.y > 65535) return fail(c, CG_ERR_UNSUPPORTED, "recurrence: too many tokens in one portion");
+    switch (a.taps) {
+      case 1: CG_CUDA(c, launch_kernel(c, k_conv_chunk<1>, grid, dim3(128), 0, 1, a)); break;
+      case 2: CG_CUDA(c, launch_kernel(c, k_conv_chunk<2>, grid, dim3(128), 0, 1, a)); break;
+      case 3: CG_CUDA(c, launch_kernel(c, k_conv_chunk<3>, grid, dim3(128), 0, 1, a)); break;
+      default: CG_CUDA(c, launch_kernel(c, k_conv_chunk<4>, grid, dim3(128), 0, 1, a)); break;
+    }
+  } else {
+    CG_CUDA(c, launch_kernel(c, k_conv_chunk_any, dim3((unsigned)a.rows.M), dim3(256), 0, 1, a));
+  }
+  CG_LAUNCHED(c);
+  CG_CUDA(c, launch_kernel(c, k_gates, dim3(grid_for(a.rows.M * a.H, 256)), dim3(256), 0, 1, a));
+  CG_LAUNCHED(c);
+  if (a.taps > 1) {
+    CG_CUDA(c, launch_kernel(c, k_conv_tail_ring, dim3((unsigned)((a.C + 127) / 128), (unsigned)a.rows.rows), dim3(128), 0, 1, a));
+    CG_LAUNCHED(c);
+  }
+  const bool small = a.dk <= 64;
+  if (a.delta) {
+    CG_TRY(small ? launch_solve<64>(c, a) : launch_solve<128>(c, a));
+    return small ? launch_scan<64, true>(c, a) : launch_scan<128, true>(c, a);
+  }
+  return small ? launch_scan<64, false>(c, a) : launch_scan<128, false>(c, a);
+}
+
+}  // namespace cg
