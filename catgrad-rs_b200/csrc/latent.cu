@@ -40,6 +40,11 @@ __device__ __forceinline__ float ld(const float* p) { return *p; }
 __device__ __forceinline__ float ld(const __nv_bfloat16* p) { return __bfloat162float(*p); }
 __device__ __forceinline__ void st(float* p, float v) { *p = v; }
 __device__ __forceinline__ void st(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
+__device__ __forceinline__ void st4(float* p, float4 v) { *(float4*)p = v; }
+__device__ __forceinline__ void st4(__nv_bfloat16* p, float4 v) {
+  const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+  *(uint2*)p = make_uint2(*(const uint32_t*)&lo, *(const uint32_t*)&hi);
+}
 
 // One block per token: the latent is normed and appended with the rotated key part; the queries'
 // rotated parts are rotated and laid out head by head with Dq values each.
@@ -75,6 +80,21 @@ __global__ void __launch_bounds__(256) k_latent_prep(LatentArgs a) {
   }
   const int D = a.d + a.r, total = a.H * a.Dq;
   T* q = (T*)a.q_out + m * (int64_t)total;
+  if (((a.d | a.Dq | D) & 3) == 0 && (a.ldp & 3) == 0) {
+    // four values at a time
+    for (int i = 4 * threadIdx.x; i < total; i += 4 * blockDim.x) {
+      const int h = i / a.Dq, e = i - h * a.Dq;
+      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (e < D) v = *(const float4*)(p + h * D + e);
+      if (e >= a.d && e < D) {
+        const int k = (e - a.d) >> 1;
+        const float2 c = *(const float2*)(ct + k), s = *(const float2*)(sn + k);
+        v = make_float4(v.x * c.x - v.y * s.x, v.y * c.x + v.x * s.x, v.z * c.y - v.w * s.y, v.w * c.y + v.z * s.y);
+      }
+      st4(q + i, v);
+    }
+    return;
+  }
   for (int i = threadIdx.x; i < total; i += blockDim.x) {
     const int h = i / a.Dq, e = i - h * a.Dq;
     const float* qh = p + h * D;

@@ -77,24 +77,38 @@ __global__ void __launch_bounds__(256) k_latent_absorb(LatentArgs a, DecodeScrat
     }
     return;
   }
-  // Wuk^T q for 64 latent columns of one head: 64 columns x 4 slices of the head dimension
+  // Wuk^T q for 64 latent columns of one head, 8 tokens at a time: 64 columns x 4 slices of the head dimension
   const int h = blockIdx.x / col_blocks, c = (blockIdx.x % col_blocks) * 64 + (tid & 63), part = tid >> 6;
-  float* q = sm;                                       // [d]
-  float* red = q + a.d;                                // [4][64]
-  __nv_bfloat16* w = (__nv_bfloat16*)(red + 256);      // [d][64]
+  float* red = sm;                                     // [8][4][64]
+  float* q = red + 8 * 256;                            // [d][8]
+  __nv_bfloat16* w = (__nv_bfloat16*)(q + 8 * a.d);    // [d][64]
   const __nv_bfloat16* uk = (const __nv_bfloat16*)a.uk + (int64_t)h * a.d * a.R;
+#pragma unroll 8
   for (int e = part; e < a.d; e += 4) w[e * 64 + (tid & 63)] = c < a.R ? uk[(int64_t)e * a.R + c] : __float2bfloat16_rn(0.f);
   asm volatile("griddepcontrol.wait;" ::: "memory");   // (the weights do not depend on it)
-  for (int m = 0; m < M; ++m) {
-    const float* p = a.proj + (int64_t)m * a.ldp + h * D;
-    for (int e = tid; e < a.d; e += 256) q[e] = p[e];
+  for (int m0 = 0; m0 < M; m0 += 8) {
+    const int n = min(8, M - m0);
+    for (int i = tid; i < 8 * a.d; i += 256) {
+      const int k = i / a.d, e = i - k * a.d;
+      q[e * 8 + k] = k < n ? a.proj[(int64_t)(m0 + k) * a.ldp + h * D + e] : 0.f;
+    }
     __syncthreads();
-    float v = 0.f;
-    for (int e = part; e < a.d; e += 4) v += q[e] * __bfloat162float(w[e * 64 + (tid & 63)]);
-    red[tid] = v;
+    float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+#pragma unroll 4
+    for (int e = part; e < a.d; e += 4) {
+      const float x = __bfloat162float(w[e * 64 + (tid & 63)]);
+      const float4 q0 = *(const float4*)(q + e * 8), q1 = *(const float4*)(q + e * 8 + 4);
+      v[0] += q0.x * x; v[1] += q0.y * x; v[2] += q0.z * x; v[3] += q0.w * x;
+      v[4] += q1.x * x; v[5] += q1.y * x; v[6] += q1.z * x; v[7] += q1.w * x;
+    }
+#pragma unroll
+    for (int k = 0; k < 8; ++k) red[k * 256 + tid] = v[k];
     __syncthreads();
-    if (part == 0 && c < a.R)
-      s.qa[((int64_t)m * a.H + h) * a.Lw + c] = __float2bfloat16_rn((red[tid] + red[tid + 64]) + (red[tid + 128] + red[tid + 192]));
+    for (int k = part; k < n; k += 4) {
+      const float* r = red + k * 256 + (tid & 63);
+      if (c < a.R) s.qa[((int64_t)(m0 + k) * a.H + h) * a.Lw + c] = __float2bfloat16_rn((r[0] + r[64]) + (r[128] + r[192]));
+    }
+    // (the next round's writes to red come after its first barrier)
   }
 }
 
@@ -239,39 +253,72 @@ __global__ void __launch_bounds__(256) k_latent_dec(LatentArgs a, DecodeScratch 
   }
 }
 
-// out[m, h, e] = Wuv[h, e] . (merged latent output): eight warps, four value rows each
+// out[m, h, e] = Wuv[h, e] . (merged latent output): eight warps, four value rows each.  The rows of
+// Wuv are fetched before the dependency wait and stay in registers (R <= 512, even) for all tokens.
 __global__ void __launch_bounds__(256) k_latent_out(LatentArgs a, DecodeScratch s) {
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
-  extern __shared__ __align__(16) float oc[];          // [R]
+  extern __shared__ __align__(16) float oc[];          // [R + 1]
+  __shared__ float wt[16];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int h = blockIdx.x, e0 = blockIdx.y * 32 + warp * 4;
   const __nv_bfloat16* uv = (const __nv_bfloat16*)a.uv + (int64_t)h * a.dv * a.R;
+  const bool even = (a.R & 1) == 0;
+  __nv_bfloat162 w[4][8];
+#pragma unroll
+  for (int y = 0; y < 4; ++y)
+#pragma unroll
+    for (int k = 0; k < 8; ++k) {
+      const int i = 2 * lane + 64 * k;
+      w[y][k] = __floats2bfloat162_rn(0.f, 0.f);
+      if (e0 + y < a.dv && i < a.R) {
+        const __nv_bfloat16* p = uv + (int64_t)(e0 + y) * a.R + i;
+        if (even) w[y][k] = *(const __nv_bfloat162*)p;
+        else w[y][k] = __nv_bfloat162(p[0], i + 1 < a.R ? p[1] : __float2bfloat16_rn(0.f));
+      }
+    }
   asm volatile("griddepcontrol.wait;" ::: "memory");
   for (int64_t m = blockIdx.z; m < a.rows.M; m += gridDim.z) {
     const int64_t at = (m * a.H + h) * s.splits;
-    float mx = -INFINITY, l = 0.f;
-    for (int k = 0; k < s.splits; ++k) mx = fmaxf(mx, s.ml[at + k].x);
-    for (int k = 0; k < s.splits; ++k) {
-      const float2 v = s.ml[at + k];
-      if (v.y > 0.f) l += v.y * expf(v.x - mx);
+    // the slices' partial values, requested before their weights are known
+    float p[2][16];
+#pragma unroll
+    for (int x = 0; x < 2; ++x)
+#pragma unroll
+      for (int k = 0; k < 16; ++k) p[x][k] = k < s.splits && tid + 256 * x < a.R ? s.o[(at + k) * a.R + tid + 256 * x] : 0.f;
+    if (warp == 0) {
+      const float2 v = lane < s.splits ? s.ml[at + lane] : make_float2(-INFINITY, 0.f);
+      float mx = v.x;
+#pragma unroll
+      for (int o = 16; o; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+      const float e = v.y > 0.f ? expf(v.x - mx) : 0.f;
+      const float l = warp_sum(e * v.y);
+      if (lane < 16) wt[lane] = e / l;
     }
-    const float inv = 1.f / l;
     __syncthreads();
-    for (int i = tid; i < a.R; i += 256) {
+#pragma unroll
+    for (int x = 0; x < 2; ++x) {
       float v = 0.f;
-      for (int k = 0; k < s.splits; ++k) {
-        const float2 w = s.ml[at + k];
-        if (w.y > 0.f) v += s.o[(at + k) * a.R + i] * (expf(w.x - mx) * inv);
+#pragma unroll
+      for (int k = 0; k < 16; ++k) {
+        const float f = wt[k];
+        if (f > 0.f) v += p[x][k] * f;   // an empty slice left nothing to read
       }
-      oc[i] = v;
+      if (tid + 256 * x < a.R) oc[tid + 256 * x] = v;
     }
+    if (tid == 0) oc[a.R] = 0.f;
     __syncthreads();
     float acc[4] = {0.f, 0.f, 0.f, 0.f};
-    for (int i = lane; i < a.R; i += 32) {
-      const float v = oc[i];
 #pragma unroll
-      for (int y = 0; y < 4; ++y)
-        if (e0 + y < a.dv) acc[y] += v * __bfloat162float(uv[(int64_t)(e0 + y) * a.R + i]);
+    for (int k = 0; k < 8; ++k) {
+      const int i = 2 * lane + 64 * k;
+      if (i < a.R) {
+        const float2 v = *(const float2*)(oc + i);
+#pragma unroll
+        for (int y = 0; y < 4; ++y) {
+          const float2 f = __bfloat1622float2(w[y][k]);
+          acc[y] += v.x * f.x + v.y * f.y;
+        }
+      }
     }
 #pragma unroll
     for (int y = 0; y < 4; ++y) {
@@ -315,7 +362,7 @@ size_t up16b(size_t n) { return (n + 15) / 16 * 16; }
 
 bool latent_decode_supported(int d, int R, int64_t Lw) {
   const int nt = pick_nt(R);
-  if (!nt || Lw % 16 || d > 320) return false;
+  if (!nt || Lw % 16 || d > 224) return false;
   return dec_smem(std::max((int)Lw, nt * 64) + 8) <= 227 * 1024;
 }
 
@@ -334,7 +381,7 @@ int k_launch_latent_decode(cg_ctx* c, const LatentArgs& a, void* scratch) {
   s.ml = (float2*)((char*)scratch + up16b(n * a.Lw * 2));
   s.o = (float*)((char*)s.ml + up16b(n * 16 * 8));
   const int cb = (a.R + 63) / 64;
-  const size_t sm1 = std::max<size_t>((size_t)(a.d + 256) * 4 + (size_t)a.d * 128, 128);
+  const size_t sm1 = std::max<size_t>((size_t)(8 * 256 + 8 * a.d) * 4 + (size_t)a.d * 128, 128);
   CG_CUDA(c, launch_kernel(c, k_latent_absorb, dim3((unsigned)(a.H * cb + M)), dim3(256), sm1, 1, a, s, cb));
   CG_LAUNCHED(c);
   switch (pick_nt(a.R)) {
@@ -343,8 +390,8 @@ int k_launch_latent_decode(cg_ctx* c, const LatentArgs& a, void* scratch) {
     default: CG_TRY(launch_dec<8>(c, a, s)); break;
   }
   const int eb = (a.dv + 31) / 32;
-  const int mz = (int)std::min<int64_t>(M, std::max<int64_t>(1, 2 * 148 / std::max(1, a.H * eb)));
-  CG_CUDA(c, launch_kernel(c, k_latent_out, dim3((unsigned)a.H, (unsigned)eb, (unsigned)mz), dim3(256), (size_t)a.R * 4, 1, a, s));
+  const int mz = (int)std::min<int64_t>(M, std::max<int64_t>(1, 3 * 148 / std::max(1, a.H * eb)));
+  CG_CUDA(c, launch_kernel(c, k_latent_out, dim3((unsigned)a.H, (unsigned)eb, (unsigned)mz), dim3(256), (size_t)(a.R + 1) * 4, 1, a, s));
   CG_LAUNCHED(c);
   return CG_OK;
 }

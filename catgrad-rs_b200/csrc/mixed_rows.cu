@@ -30,10 +30,9 @@ __device__ __forceinline__ void store4(__nv_bfloat16* p, const float* v) {
   *(uint2*)p = make_uint2(*(const uint32_t*)&lo, *(const uint32_t*)&hi);
 }
 
-constexpr int RU_VEC = 4;  // 128-bit vectors a thread keeps
 
-// One block per row; the row lives in registers (four values per vector, RU_VEC vectors per thread).
-template <class T>
+// One block per row; the row lives in registers (RU_VEC 128-bit vectors per thread).
+template <class T, int RU_VEC>
 __global__ void k_row_update(RowUpdate u, int32_t* err) {
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
   asm volatile("griddepcontrol.wait;" ::: "memory");
@@ -57,9 +56,11 @@ __global__ void k_row_update(RowUpdate u, int32_t* err) {
       if (tok >= u.vocab) { if (threadIdx.x == 0) *err = DEV_INDEX; tok = 0; }
     }
     float ss = 0.f;
+    float4 old[RU_VEC];  // requested before the reduction
 #pragma unroll
     for (int j = 0; j < RU_VEC; ++j) {
       const int i = threadIdx.x + j * blockDim.x;
+      old[j] = u.add && j < nv && i < n4 ? *(const float4*)(u.x + m * u.ldx + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f);
       v[j][0] = v[j][1] = v[j][2] = v[j][3] = 0.f;
       if (j < nv && i < n4) {
         if (u.tokens) {
@@ -95,10 +96,7 @@ __global__ void k_row_update(RowUpdate u, int32_t* err) {
       const int i = threadIdx.x + j * blockDim.x;
       if (j < nv && i < n4) {
         float* xp = u.x + m * u.ldx + 4 * i;
-        if (u.add) {
-          const float4 t = *(const float4*)xp;
-          v[j][0] += t.x; v[j][1] += t.y; v[j][2] += t.z; v[j][3] += t.w;
-        }
+        v[j][0] += old[j].x; v[j][1] += old[j].y; v[j][2] += old[j].z; v[j][3] += old[j].w;
         store4(xp, v[j]);
       }
     }
@@ -163,12 +161,12 @@ __global__ void k_pair_rope_tables(double base, int64_t T, int r, float* cos_t, 
 int k_launch_row_update(cg_ctx* c, const RowUpdate& u, int64_t M, int out_bf16) {
   if (M == 0) return CG_OK;
   const int n4 = (u.W + 7) / 8 * 2;
-  int block = (n4 + 31) / 32 * 32;
-  while (block > 256 && (n4 + block / 2 - 1) / (block / 2) <= (M > 296 ? RU_VEC : 1)) block = (block / 2 + 31) / 32 * 32;
-  block = std::min(block, 1024);
-  if ((int64_t)block * RU_VEC < n4) return fail(c, CG_ERR_UNSUPPORTED, "decoder: rows wider than 16384 are not supported");
-  if (out_bf16) CG_CUDA(c, launch_kernel(c, k_row_update<__nv_bfloat16>, dim3((unsigned)M), dim3(block), 0, 1, u, c->core->dev_err));
-  else CG_CUDA(c, launch_kernel(c, k_row_update<float>, dim3((unsigned)M), dim3(block), 0, 1, u, c->core->dev_err));
+  const int vec = n4 <= 512 || (n4 <= 1024 && M <= 296) ? 1 : n4 <= 1024 ? 2 : 4;
+  const int block = ((n4 + vec - 1) / vec + 31) / 32 * 32;
+  if (block > 1024) return fail(c, CG_ERR_UNSUPPORTED, "decoder: rows wider than 16384 are not supported");
+  auto kernel = out_bf16 ? (vec == 1 ? k_row_update<__nv_bfloat16, 1> : vec == 2 ? k_row_update<__nv_bfloat16, 2> : k_row_update<__nv_bfloat16, 4>)
+                         : (vec == 1 ? k_row_update<float, 1> : vec == 2 ? k_row_update<float, 2> : k_row_update<float, 4>);
+  CG_CUDA(c, launch_kernel(c, kernel, dim3((unsigned)M), dim3(block), 0, 1, u, c->core->dev_err));
   CG_LAUNCHED(c);
   return CG_OK;
 }

@@ -333,19 +333,21 @@ __global__ void k_gated_norm_vec(GatedNorm a, int n, int units, int threads) {
   const float* o = a.o + m * (int64_t)a.H * a.dv + c0;
   const TG* gate = (const TG*)a.gate + m * a.ldg + c0;
   T* out = (T*)a.att + m * a.ld_att + c0;
-  float4 x[V];
+  float4 x[V], g[V];
   float ss = 0.f;
 #pragma unroll
   for (int j = 0; j < V; ++j) {
     const int i = 4 * (t + j * threads);
-    x[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+    x[j] = g[j] = make_float4(0.f, 0.f, 0.f, 0.f);
     if (live && i < n) {
       x[j] = *(const float4*)(o + i);
-      if (!a.delta) {
-        const float4 g = ldg4(gate + i);
-        x[j].x *= silu(g.x); x[j].y *= silu(g.y); x[j].z *= silu(g.z); x[j].w *= silu(g.w);
-      }
+      g[j] = ldg4(gate + i);
     }
+  }
+#pragma unroll
+  for (int j = 0; j < V; ++j) {
+    g[j] = make_float4(silu(g[j].x), silu(g[j].y), silu(g[j].z), silu(g[j].w));
+    if (!a.delta) { x[j].x *= g[j].x; x[j].y *= g[j].y; x[j].z *= g[j].z; x[j].w *= g[j].w; }
     ss += x[j].x * x[j].x + x[j].y * x[j].y + x[j].z * x[j].z + x[j].w * x[j].w;
   }
   ss = threads == 32 ? warp_sum(ss) : block_sum(ss, sh);
@@ -356,10 +358,7 @@ __global__ void k_gated_norm_vec(GatedNorm a, int n, int units, int threads) {
     if (!live || i >= n) continue;
     const float4 w = *(const float4*)(a.norm + (a.delta ? 0 : c0) + i);
     float4 r = make_float4(x[j].x * inv * w.x, x[j].y * inv * w.y, x[j].z * inv * w.z, x[j].w * inv * w.w);
-    if (a.delta) {
-      const float4 g = ldg4(gate + i);
-      r.x *= silu(g.x); r.y *= silu(g.y); r.z *= silu(g.z); r.w *= silu(g.w);
-    }
+    if (a.delta) { r.x *= g[j].x; r.y *= g[j].y; r.z *= g[j].z; r.w *= g[j].w; }
     st4(out + i, r);
   }
 }

@@ -7,7 +7,7 @@
 // For the state space u_t = dt_t v_t.  For the delta rule u solves a unit lower triangular system:
 //   (I + A) U = R,  A_ts = b_t e^{G_t - G_s} (k_t . k_s) (s < t),  R_t = b_t (v_t - e^{G_t} S0^T k_t)
 // T = (I + A)^-1 depends on keys and gates only, so k_delta_solve makes it for all chunks at once;
-// k_chunk_scan then walks the chunks of one (row, head, 64 value columns) with S in registers.
+// k_delta_scan / k_ssd_scan then walk the chunks of one (row, head, 64 value columns) with S in registers.
 //
 // Precision.  The conv outputs are bf16 (and exact as such); unit norms are kept apart as f32 factors
 // per token and head, so every product of q, k, v with itself is exact in the operands.  State,
@@ -27,7 +27,7 @@ constexpr int CT = 64;   // tokens per chunk
 constexpr int EB = 64;   // value columns per block
 constexpr int LE = EB + 8, LT = CT + 8;
 
-__device__ __forceinline__ float silu(float x) { return x / (1.f + __expf(-x)); }
+__device__ __forceinline__ float silu(float x) { return __fdividef(x, 1.f + __expf(-x)); }  // rounded to bf16 at once
 __device__ __forceinline__ float softplus(float x) { return x > 20.f ? x : log1pf(expf(x)); }
 __device__ __forceinline__ uint32_t sm_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 
@@ -106,9 +106,10 @@ __global__ void __launch_bounds__(256) k_conv_chunk_any(ChunkArgs a) {
   }
 }
 
-// Sizes in multiples of 8: a thread takes 8 neighbouring channels of 16 tokens and slides over
+// Sizes in multiples of 8: a thread takes 4 neighbouring channels of 16 tokens and slides over
 // them.  Same outputs.
 constexpr int CONV_TOK = 16;
+constexpr int CV = 4;  // neighbouring channels of a thread
 template <int TAPS>
 __global__ void __launch_bounds__(128) k_conv_chunk(ChunkArgs a) {
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
@@ -120,35 +121,38 @@ __global__ void __launch_bounds__(128) k_conv_chunk(ChunkArgs a) {
   const int row = a.rows.tok_row[m0];
   const int64_t p0 = row_pos0(a.rows, row);
   const int i0 = (int)(m0 - a.rows.start[row]);
-  const int c = (blockIdx.x * 128 + threadIdx.x) * 8;
+  const int c = (blockIdx.x * 128 + threadIdx.x) * CV;
   const bool live = c < a.C;
   const int cc = live ? c : 0;
   const float* tail = a.tail + (int64_t)a.rows.slot[row] * a.taps * a.C + cc;
-  float w[TAPS][8], bias[8];
+  float w[TAPS][CV], bias[CV];
 #pragma unroll
-  for (int e = 0; e < 8; ++e) {
+  for (int e = 0; e < CV; ++e) {
     bias[e] = a.conv_b ? a.conv_b[cc + e] : 0.f;
 #pragma unroll
     for (int j = 0; j < TAPS; ++j) w[j][e] = a.conv_w[(int64_t)(cc + e) * TAPS + TAPS - 1 - j];
   }
-  // x[j]: the input j tokens back
-  float x[TAPS][8];
+  // x[TAPS - 1 + i]: the input of the group's token i; x[TAPS - 1 - j]: the one j tokens before the group
+  constexpr int G = 4;
+  float x[TAPS - 1 + G][CV];
+  auto widen = [](const uint2& r, float* v) {
+    const uint32_t p[2] = {r.x, r.y};
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const float2 f = __bfloat1622float2(*(const __nv_bfloat162*)&p[e]);
+      v[2 * e] = f.x; v[2 * e + 1] = f.y;
+    }
+  };
 #pragma unroll
   for (int j = 1; j < TAPS; ++j) {
+    float* v = x[TAPS - 1 - j];
 #pragma unroll
-    for (int e = 0; e < 8; ++e) x[j][e] = 0.f;
-    if (j <= i0) {
-      const uint4 r = *(const uint4*)(a.proj + (m0 - j) * a.ldp + cc);
-      const uint32_t* p = &r.x;
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const float2 f = __bfloat1622float2(*(const __nv_bfloat162*)&p[e]);
-        x[j][2 * e] = f.x; x[j][2 * e + 1] = f.y;
-      }
-    } else if (p0 + i0 - j >= 0) {
+    for (int e = 0; e < CV; ++e) v[e] = 0.f;
+    if (j <= i0) widen(*(const uint2*)(a.proj + (m0 - j) * a.ldp + cc), v);
+    else if (p0 + i0 - j >= 0) {
       const float* tp = tail + (int64_t)((p0 + i0 - j) % a.taps) * a.C;
 #pragma unroll
-      for (int e = 0; e < 8; ++e) x[j][e] = tp[e];
+      for (int e = 0; e < CV; ++e) v[e] = tp[e];
     }
   }
   // where these channels go
@@ -168,42 +172,49 @@ __global__ void __launch_bounds__(128) k_conv_chunk(ChunkArgs a) {
     if (e == 0) rn = (isk ? a.rk : a.rq) + h;
     if (!isk) f = rsqrtf((float)a.dk);
   }
-  const int lanes = a.dk / 8;  // threads of a head: a power of two dividing the warp
-  for (int t = t_lo; t < t_hi; ++t) {
+  const int lanes = a.dk / CV;  // threads of a head: a power of two dividing the warp
+  uint2 raw[G];
+  auto fetch = [&](int t) {
+#pragma unroll
+    for (int i = 0; i < G; ++i) raw[i] = t + i < t_hi ? *(const uint2*)(a.proj + (m0 + t - t_lo + i) * a.ldp + cc) : make_uint2(0, 0);
+  };
+  fetch(t_lo);
+  for (int t = t_lo; t < t_hi; t += G) {
     const int64_t m = m0 + t - t_lo;
-    const uint4 r = *(const uint4*)(a.proj + m * a.ldp + cc);
-    const uint32_t* p = &r.x;
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const float2 g = __bfloat1622float2(*(const __nv_bfloat162*)&p[e]);
-      x[0][2 * e] = g.x; x[0][2 * e + 1] = g.y;
-    }
-    uint32_t o[4];
-    float ss = 0.f;
+    for (int i = 0; i < G; ++i) widen(raw[i], x[TAPS - 1 + i]);
+    fetch(t + G);  // the next group's inputs are on the way while this one is computed
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      float y[2];
+    for (int i = 0; i < G; ++i) {
+      uint32_t o[2];
+      float ss = 0.f;
 #pragma unroll
-      for (int b = 0; b < 2; ++b) {
-        float v = bias[2 * e + b];
+      for (int e = 0; e < 2; ++e) {
+        float y[2];
 #pragma unroll
-        for (int j = 0; j < TAPS; ++j) v += w[j][2 * e + b] * x[j][2 * e + b];
-        y[b] = silu(v);
+        for (int b = 0; b < 2; ++b) {
+          float v = bias[2 * e + b];
+#pragma unroll
+          for (int j = 0; j < TAPS; ++j) v += w[j][2 * e + b] * x[TAPS - 1 + i - j][2 * e + b];
+          y[b] = silu(v);
+        }
+        const __nv_bfloat162 h2 = __floats2bfloat162_rn(y[0], y[1]);
+        o[e] = *(const uint32_t*)&h2;
+        if (a.delta) {
+          const float2 g = __bfloat1622float2(h2);
+          ss += g.x * g.x + g.y * g.y;
+        }
       }
-      const __nv_bfloat162 h2 = __floats2bfloat162_rn(y[0], y[1]);
-      o[e] = *(const uint32_t*)&h2;
-      const float2 g = __bfloat1622float2(h2);
-      ss += g.x * g.x + g.y * g.y;
+      const bool in = live && t + i < t_hi;
+      if (in) *(uint2*)(out + (m + i) * ld) = make_uint2(o[0], o[1]);
+      if (a.delta)
+        for (int s = lanes / 2; s; s >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, s);
+      if (in && rn) rn[(m + i) * a.KH] = a.delta ? f / sqrtf(ss + 1e-6f) : 1.f;
     }
-    if (live) *(uint4*)(out + m * ld) = make_uint4(o[0], o[1], o[2], o[3]);
-    if (a.delta) {
-      for (int s = lanes / 2; s; s >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, s);
-      if (live && rn) rn[m * a.KH] = f / sqrtf(ss + 1e-6f);
-    } else if (live && rn) rn[m * a.KH] = 1.f;
 #pragma unroll
-    for (int j = TAPS - 1; j > 0; --j)
+    for (int j = 0; j < TAPS - 1; ++j)
 #pragma unroll
-      for (int e = 0; e < 8; ++e) x[j][e] = x[j - 1][e];
+      for (int e = 0; e < CV; ++e) x[j][e] = x[j + G][e];
   }
 }
 
@@ -237,33 +248,56 @@ __global__ void k_conv_tail_ring(ChunkArgs a) {
 }
 
 // ------------------------------------------------------------------ gates of a chunk ----
-struct Gates {
-  float G[CT], co[CT], rq[CT], rk[CT];
-  float last;  // sum of the chunk's log decays
+// 2^x to about 22 bits; its arguments here are at most 0
+__device__ __forceinline__ float pow2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+struct alignas(16) Gates {  // (pairs are read as 8-byte words)
+  float G[CT];           // running sum of the log decays, base 2
+  float co[CT], rk[CT];  // beta or dt; unit-norm factor of the key
+  float rq[CT];          // unit-norm factor of the query
+  float ek[CT], eq[CT];  // e^{G_t} times those factors
+  float f[CT];           // what scales token t's write in the state after the chunk: e^{G_last - G_t} rk (ssd: and dt)
+  float whole;           // e^{G_last}
 };
 // by one warp: lane l takes tokens 2 l and 2 l + 1
 __device__ __forceinline__ void load_gates(const ChunkArgs& a, int chunk, int h, int kh, Gates* g, int lane) {
   const int len = a.chunk_len[chunk];
   const int64_t m0 = a.chunk_tok[chunk];
-  float l[2];
+  float l[2], co[2], rq[2], rk[2];
 #pragma unroll
   for (int b = 0; b < 2; ++b) {
     const int t = 2 * lane + b;
     const bool in = t < len;
-    l[b] = in ? a.gl[(m0 + t) * a.H + h] : 0.f;
-    g->co[t] = in ? a.co[(m0 + t) * a.H + h] : 0.f;
-    g->rq[t] = in ? a.rq[(m0 + t) * a.KH + kh] : 0.f;
-    g->rk[t] = in ? a.rk[(m0 + t) * a.KH + kh] : 0.f;
+    l[b] = in ? a.gl[(m0 + t) * a.H + h] * 1.4426950408889634f : 0.f;
+    co[b] = in ? a.co[(m0 + t) * a.H + h] : 0.f;
+    rq[b] = in ? a.rq[(m0 + t) * a.KH + kh] : 0.f;
+    rk[b] = in ? a.rk[(m0 + t) * a.KH + kh] : 0.f;
   }
-  float sum = l[0] + l[1], inc = sum;
+  const float sum = l[0] + l[1];
+  float inc = sum;
 #pragma unroll
   for (int o = 1; o < 32; o <<= 1) {
     const float v = __shfl_up_sync(0xffffffffu, inc, o);
     if (lane >= o) inc += v;
   }
-  g->G[2 * lane] = inc - sum + l[0];
-  g->G[2 * lane + 1] = inc;
-  if (lane == 31) g->last = inc;
+  const float last = __shfl_sync(0xffffffffu, inc, 31);
+#pragma unroll
+  for (int b = 0; b < 2; ++b) {
+    const int t = 2 * lane + b;
+    const float G = b ? inc : inc - l[1];
+    g->G[t] = G;
+    g->co[t] = co[b];
+    g->rq[t] = rq[b];
+    g->rk[t] = rk[b];
+    g->eq[t] = pow2(G) * rq[b];
+    g->ek[t] = pow2(G) * rk[b];
+    g->f[t] = pow2(last - G) * rk[b] * (a.delta ? 1.f : co[b]);
+  }
+  if (lane == 0) g->whole = pow2(last);
 }
 
 // ------------------------------------------------------------------ T = (I + A)^-1 ----
@@ -271,7 +305,7 @@ template <int DK>
 __global__ void __launch_bounds__(128) k_delta_solve(ChunkArgs a) {
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
   asm volatile("griddepcontrol.wait;" ::: "memory");
-  constexpr int LK = DK + 8, LA = 68, LX = 80;
+  constexpr int LK = DK + 8, LA = 68, LX = 68;
   extern __shared__ __align__(16) uint8_t smem[];
   float* A = (float*)smem;                       // [64][LA]
   float* X = A + CT * LA;                        // [64][LX]
@@ -311,55 +345,86 @@ __global__ void __launch_bounds__(128) k_delta_solve(ChunkArgs a) {
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       const int t = warp * 16 + (lane >> 2) + 8 * (e >> 1), s = j * 8 + (lane & 3) * 2 + (e & 1);
-      A[t * LA + s] = s < t ? g.co[t] * g.rk[t] * g.rk[s] * expf(g.G[t] - g.G[s]) * acc[j][e] : 0.f;
+      A[t * LA + s] = s < t ? g.co[t] * g.rk[t] * g.rk[s] * pow2(g.G[t] - g.G[s]) * acc[j][e] : 0.f;
     }
   __syncthreads();
-  // forward substitution, column j of the inverse by two neighbouring lanes (even and odd terms)
-  const int j = tid >> 1, half = tid & 1, s_lo = (tid >> 5) * 16;
-  for (int i = s_lo; i < CT; ++i) {
-    const float* Ai = A + i * LA;
-    float v0 = 0.f, v1 = 0.f;
-    int s = s_lo + half;
-    for (; s + 2 < i; s += 4) {
-      v0 += Ai[s] * X[s * LX + j];
-      v1 += Ai[s + 2] * X[(s + 2) * LX + j];
+  // inverse by doubling blocks: four 16 x 16 diagonal blocks by substitution (one column per thread),
+  // then [T1 0; -T2 A21 T1, T2] for 32 and for 64
+  for (int i = tid; i < CT * CT; i += 128) X[(i >> 6) * LX + (i & 63)] = 0.f;
+  __syncthreads();
+  if (tid < CT) {
+    const int b0 = tid & ~15, jc = tid & 15;
+    float x[16];
+#pragma unroll
+    for (int i = 0; i < 16; ++i) {
+      float v = i == jc ? 1.f : 0.f;
+#pragma unroll
+      for (int s = 0; s < i; ++s) v -= A[(b0 + i) * LA + b0 + s] * x[s];  // x[s] = 0 above the diagonal
+      x[i] = v;
+      X[(b0 + i) * LX + tid] = v;
     }
-    if (s < i) v0 += Ai[s] * X[s * LX + j];
-    v0 += v1;
-    v0 += __shfl_xor_sync(0xffffffffu, v0, 1);
-    if (half == 0) X[i * LX + j] = i < j ? 0.f : (i == j ? 1.f : 0.f) - v0;
-    __syncwarp();
+  }
+  __syncthreads();
+  // Y[n x n] = L[n x n] Rm[n x n] (n 16 or 32): a thread takes one row and NC columns
+  auto product = [&](const float* Lm, int ldl, const float* Rm, int ldr, float* Y, int ldy, int n, float sign, int u) {
+    const int per_row = n / 8, r = u / per_row, c = (u - r * per_row) * 8;
+    float acc[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) acc[e] = 0.f;
+#pragma unroll 4
+    for (int k = 0; k < n; ++k) {
+      const float l = Lm[r * ldl + k];
+      const float4 r0 = *(const float4*)(Rm + k * ldr + c), r1 = *(const float4*)(Rm + k * ldr + c + 4);
+      acc[0] += l * r0.x; acc[1] += l * r0.y; acc[2] += l * r0.z; acc[3] += l * r0.w;
+      acc[4] += l * r1.x; acc[5] += l * r1.y; acc[6] += l * r1.z; acc[7] += l * r1.w;
+    }
+    *(float4*)(Y + r * ldy + c) = make_float4(sign * acc[0], sign * acc[1], sign * acc[2], sign * acc[3]);
+    *(float4*)(Y + r * ldy + c + 4) = make_float4(sign * acc[4], sign * acc[5], sign * acc[6], sign * acc[7]);
+  };
+  {
+    // two pairs of 16-blocks, 32 threads each; the products pass through the free upper blocks of A
+    const int pr = tid >> 5, u = tid & 31, b = pr * 32;
+    if (pr < 2) product(A + (b + 16) * LA + b, LA, X + b * LX + b, LX, A + b * LA + b + 16, LA, 16, 1.f, u);
+    __syncthreads();
+    if (pr < 2) product(X + (b + 16) * LX + b + 16, LX, A + b * LA + b + 16, LA, X + (b + 16) * LX + b, LX, 16, -1.f, u);
+    __syncthreads();
+    product(A + 32 * LA, LA, X, LX, A + 32, LA, 32, 1.f, tid);
+    __syncthreads();
+    product(X + 32 * LX + 32, LX, A + 32, LA, X + 32 * LX, LX, 32, -1.f, tid);
   }
   __syncthreads();
   __nv_bfloat16* out = a.T + ((int64_t)chunk * a.H + h) * 2 * CT * CT;
   for (int i = tid; i < CT * CT / 2; i += 128) {
     const int r = i / (CT / 2), c = (i - r * (CT / 2)) * 2;
-    const int first = c & ~15;  // rows above a column group's first were never written
-    const float x0 = r >= first ? X[r * LX + c] : 0.f, x1 = r >= first ? X[r * LX + c + 1] : 0.f;
     uint32_t hi, lo;
-    split2(x0, x1, hi, lo);
+    split2(X[r * LX + c], X[r * LX + c + 1], hi, lo);
     *(uint32_t*)(out + r * CT + c) = hi;
     *(uint32_t*)(out + CT * CT + r * CT + c) = lo;
   }
 }
 
 // ------------------------------------------------------------------ the walk ----------
-template <int DK, bool DELTA>
-struct ScanSmem {
+// Regions are reused inside a chunk so that two blocks share an SM: P takes Q's place, R and then U
+// take V's (and one more for the remainders), U' takes T's.
+template <int DK>
+struct DeltaSmem {
   static constexpr int LK = DK + 8;
-  static constexpr uint32_t Q = 0, K = Q + CT * LK * 2, V = K + CT * LK * 2, T = V + CT * LE * 2;
-  static constexpr uint32_t STAGE = T + (DELTA ? 2 * CT * LT * 2 : 0);
-  static constexpr uint32_t S = 2 * STAGE;                       // [2][DK][LE]
-  static constexpr uint32_t R = S + 2 * DK * LE * 2;             // [2][64][LE]: R, then U (delta)
-  static constexpr uint32_t P = R + (DELTA ? 2 * CT * LE * 2 : 0);  // [2][64][LT]
-  static constexpr uint32_t UP = P + 2 * CT * LT * 2;            // [2][64][LE]
-  static constexpr uint32_t GATES = UP + 2 * CT * LE * 2;
+  static constexpr uint32_t EBYTES = CT * LE * 2;
+  static constexpr uint32_t Q = 0, P = 0;                        // [64][LK] | [2][64][LT]
+  static constexpr uint32_t K = (CT * LK > 2 * CT * LT ? CT * LK : 2 * CT * LT) * 2;
+  static constexpr uint32_t V = K + CT * LK * 2;                 // [64][LE]
+  static constexpr uint32_t RL = V + EBYTES;                     // [64][LE]
+  static constexpr uint32_t T = RL + EBYTES;                     // [2][64][LT] | U' [2][64][LE]
+  static constexpr uint32_t UP = T;
+  static constexpr uint32_t S = T + 2 * EBYTES;                  // [2][DK][LE]
+  static constexpr uint32_t GATES = S + 2 * DK * LE * 2;
   static constexpr uint32_t BYTES = GATES + 2 * sizeof(Gates);
+  static_assert(LE == LT, "T and U' share a region");
 };
 
-template <int DK, bool DELTA>
-__global__ void __launch_bounds__(256, 1) k_chunk_scan(ChunkArgs a) {
-  using L = ScanSmem<DK, DELTA>;
+template <int DK>
+__global__ void __launch_bounds__(256, 2) k_delta_scan(ChunkArgs a) {
+  using L = DeltaSmem<DK>;
   constexpr int LK = L::LK;
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
   asm volatile("griddepcontrol.wait;" ::: "memory");
@@ -374,10 +439,10 @@ __global__ void __launch_bounds__(256, 1) k_chunk_scan(ChunkArgs a) {
   const bool first = row_pos0(a.rows, row) == 0;
   const int vw = min(EB, a.dvp - e0);                 // columns that exist (multiple of 8)
 
-  auto load = [&](int chunk, int stage) {
+  auto load = [&](int chunk) {
     const int len = a.chunk_len[chunk];
     const int64_t m0 = a.chunk_tok[chunk];
-    const uint32_t b = base + (uint32_t)stage * L::STAGE;
+    const uint32_t b = base;
     const int ch = a.DKp / 8;
     for (int i = tid; i < CT * (DK / 8); i += 256) {
       const int r = i / (DK / 8), c = i - r * (DK / 8);
@@ -393,7 +458,7 @@ __global__ void __launch_bounds__(256, 1) k_chunk_scan(ChunkArgs a) {
       cp_async16(b + L::V + (uint32_t)(r * LE + c * 8) * 2u,
                  a.v + (m0 + (in ? r : 0)) * (int64_t)a.H * a.dvp + (int64_t)h * a.dvp + (in ? e0 + c * 8 : 0), in ? 16 : 0);
     }
-    if (DELTA) {
+    {
       const __nv_bfloat16* t = a.T + ((int64_t)chunk * a.H + h) * 2 * CT * CT;
       for (int i = tid; i < 2 * CT * (CT / 8); i += 256) {
         const int r = i / (CT / 8), c = i - r * (CT / 8);
@@ -402,7 +467,7 @@ __global__ void __launch_bounds__(256, 1) k_chunk_scan(ChunkArgs a) {
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  load(c0, 0);
+  load(c0);
   if (warp == 7) load_gates(a, c0, h, kh, &gates[0], lane);
 
   // the state: DK / 16 row tiles over the warps
@@ -432,20 +497,14 @@ __global__ void __launch_bounds__(256, 1) k_chunk_scan(ChunkArgs a) {
       }
   };
   publish_state();
-  const float dsk = a.dskip ? a.dskip[h] : 0.f;
 
   for (int c = c0; c < c1; ++c) {
     const int stage = (c - c0) & 1;
-    const uint32_t b = base + (uint32_t)stage * L::STAGE;
-    const uint8_t* bs = smem + (size_t)stage * L::STAGE;
+    const uint32_t b = base;
     const Gates& g = gates[stage];
     cp_async_wait_all();
-    __syncthreads();  // tiles, gates and state of this chunk are in place; the other stage is free
-    if (c + 1 < c1) {
-      load(c + 1, stage ^ 1);
-      if (warp == 7) load_gates(a, c + 1, h, kh, &gates[stage ^ 1], lane);
-    }
-    const float glast = g.last;
+    __syncthreads();  // tiles, gates and state of this chunk are in place
+    if (c + 1 < c1 && warp == 7) load_gates(a, c + 1, h, kh, &gates[stage ^ 1], lane);
     const int t0 = wm * 16 + r_in;                    // this thread's tokens: t0 and t0 + 8
     float qs[4][4];                                    // Q S0
     {
@@ -459,7 +518,7 @@ __global__ void __launch_bounds__(256, 1) k_chunk_scan(ChunkArgs a) {
       for (int kk = 0; kk < DK; kk += 16) {
         uint32_t fq[4], fk[4], fb[4];
         frag_a(b + L::Q, LK, wm * 16, kk, lane, fq);
-        if (DELTA) frag_a(b + L::K, LK, wm * 16, kk, lane, fk);
+        frag_a(b + L::K, LK, wm * 16, kk, lane, fk);
 #pragma unroll
         for (int j = 0; j < 4; j += 2) {
 #pragma unroll
@@ -467,10 +526,8 @@ __global__ void __launch_bounds__(256, 1) k_chunk_scan(ChunkArgs a) {
             frag_b_kn(base + L::S + (uint32_t)(part * DK * LE * 2), LE, kk, wn * 32 + j * 8, lane, fb);
             mma_bf16(qs[j], fq[0], fq[1], fq[2], fq[3], fb[0], fb[1]);
             mma_bf16(qs[j + 1], fq[0], fq[1], fq[2], fq[3], fb[2], fb[3]);
-            if (DELTA) {
-              mma_bf16(ks[j], fk[0], fk[1], fk[2], fk[3], fb[0], fb[1]);
-              mma_bf16(ks[j + 1], fk[0], fk[1], fk[2], fk[3], fb[2], fb[3]);
-            }
+            mma_bf16(ks[j], fk[0], fk[1], fk[2], fk[3], fb[0], fb[1]);
+            mma_bf16(ks[j + 1], fk[0], fk[1], fk[2], fk[3], fb[2], fb[3]);
           }
           if (below) {
             frag_b_nk(b + L::K, LK, kk, wn * 32 + j * 8, lane, fb);
@@ -479,6 +536,7 @@ __global__ void __launch_bounds__(256, 1) k_chunk_scan(ChunkArgs a) {
           }
         }
       }
+      __syncthreads();  // Q and the old state are read
       // P and R (or the state's addends) into shared memory, split
 #pragma unroll
       for (int j = 0; j < 4; ++j)
@@ -489,30 +547,23 @@ __global__ void __launch_bounds__(256, 1) k_chunk_scan(ChunkArgs a) {
 #pragma unroll
           for (int y = 0; y < 2; ++y) {
             const int s = n + y;
-            p[y] = s <= t ? expf(g.G[t] - g.G[s]) * g.rq[t] * g.rk[s] * (DELTA ? 1.f : g.co[s]) * qk[j][2 * x + y] : 0.f;
+            p[y] = s <= t ? pow2(g.G[t] - g.G[s]) * g.rq[t] * g.rk[s] * qk[j][2 * x + y] : 0.f;
           }
           uint32_t hi, lo;
           split2(p[0], p[1], hi, lo);
           const uint32_t o = (uint32_t)(t * LT + n) * 2u;
           *(uint32_t*)(smem + L::P + o) = hi;
           *(uint32_t*)(smem + L::P + CT * LT * 2 + o) = lo;
-          const float2 v = __bfloat1622float2(*(const __nv_bfloat162*)(bs + L::V + (uint32_t)(t * LE + n) * 2u));
+          const float2 v = __bfloat1622float2(*(const __nv_bfloat162*)(smem + L::V + (uint32_t)(t * LE + n) * 2u));
           const uint32_t oe = (uint32_t)(t * LE + n) * 2u;
-          if (DELTA) {
-            const float f = expf(g.G[t]) * g.rk[t];
-            split2(g.co[t] * (v.x - f * ks[j][2 * x]), g.co[t] * (v.y - f * ks[j][2 * x + 1]), hi, lo);
-            *(uint32_t*)(smem + L::R + oe) = hi;
-            *(uint32_t*)(smem + L::R + CT * LE * 2 + oe) = lo;
-          } else {
-            const float f = g.co[t] * expf(glast - g.G[t]) * g.rk[t];
-            split2(f * v.x, f * v.y, hi, lo);
-            *(uint32_t*)(smem + L::UP + oe) = hi;
-            *(uint32_t*)(smem + L::UP + CT * LE * 2 + oe) = lo;
-          }
+          const float f = g.ek[t];
+          split2(g.co[t] * (v.x - f * ks[j][2 * x]), g.co[t] * (v.y - f * ks[j][2 * x + 1]), hi, lo);
+          *(uint32_t*)(smem + L::V + oe) = hi;  // (this thread's own value of V)
+          *(uint32_t*)(smem + L::RL + oe) = lo;
         }
     }
     __syncthreads();
-    if (DELTA) {
+    {
       // U = T R
       float u[4][4];
 #pragma unroll
@@ -523,8 +574,8 @@ __global__ void __launch_bounds__(256, 1) k_chunk_scan(ChunkArgs a) {
         frag_a(b + L::T + CT * LT * 2, LT, wm * 16, kk, lane, tl);
 #pragma unroll
         for (int j = 0; j < 4; j += 2) {
-          frag_b_kn(base + L::R, LE, kk, wn * 32 + j * 8, lane, fh);
-          frag_b_kn(base + L::R + CT * LE * 2, LE, kk, wn * 32 + j * 8, lane, fl);
+          frag_b_kn(base + L::V, LE, kk, wn * 32 + j * 8, lane, fh);
+          frag_b_kn(base + L::RL, LE, kk, wn * 32 + j * 8, lane, fl);
 #pragma unroll
           for (int y = 0; y < 2; ++y) {
             mma_bf16(u[j + y], th[0], th[1], th[2], th[3], fh[2 * y], fh[2 * y + 1]);
@@ -533,8 +584,7 @@ __global__ void __launch_bounds__(256, 1) k_chunk_scan(ChunkArgs a) {
           }
         }
       }
-      // U takes R's place once the four warps of these columns have read it
-      asm volatile("bar.sync %0, 128;" ::"r"(1 + wn) : "memory");
+      __syncthreads();  // T and R are read: U' and U take their places
 #pragma unroll
       for (int j = 0; j < 4; ++j)
 #pragma unroll
@@ -543,9 +593,9 @@ __global__ void __launch_bounds__(256, 1) k_chunk_scan(ChunkArgs a) {
           const uint32_t oe = (uint32_t)(t * LE + wn * 32 + j * 8 + cq) * 2u;
           uint32_t hi, lo;
           split2(u[j][2 * x], u[j][2 * x + 1], hi, lo);
-          *(uint32_t*)(smem + L::R + oe) = hi;
-          *(uint32_t*)(smem + L::R + CT * LE * 2 + oe) = lo;
-          const float f = expf(glast - g.G[t]) * g.rk[t];
+          *(uint32_t*)(smem + L::V + oe) = hi;
+          *(uint32_t*)(smem + L::RL + oe) = lo;
+          const float f = g.f[t];
           split2(f * u[j][2 * x], f * u[j][2 * x + 1], hi, lo);
           *(uint32_t*)(smem + L::UP + oe) = hi;
           *(uint32_t*)(smem + L::UP + CT * LE * 2 + oe) = lo;
@@ -556,7 +606,7 @@ __global__ void __launch_bounds__(256, 1) k_chunk_scan(ChunkArgs a) {
     {
 #pragma unroll
       for (int x = 0; x < 2; ++x) {
-        const float f = expf(g.G[t0 + 8 * x]) * g.rq[t0 + 8 * x];
+        const float f = g.eq[t0 + 8 * x];
 #pragma unroll
         for (int j = 0; j < 4; ++j) { qs[j][2 * x] *= f; qs[j][2 * x + 1] *= f; }
       }
@@ -566,13 +616,13 @@ __global__ void __launch_bounds__(256, 1) k_chunk_scan(ChunkArgs a) {
         frag_a(base + L::P + CT * LT * 2, LT, wm * 16, kk, lane, pl);
 #pragma unroll
         for (int j = 0; j < 4; j += 2) {
-          frag_b_kn(DELTA ? base + L::R : b + L::V, LE, kk, wn * 32 + j * 8, lane, fh);
-          if (DELTA) frag_b_kn(base + L::R + CT * LE * 2, LE, kk, wn * 32 + j * 8, lane, fl);
+          frag_b_kn(base + L::V, LE, kk, wn * 32 + j * 8, lane, fh);
+          frag_b_kn(base + L::RL, LE, kk, wn * 32 + j * 8, lane, fl);
 #pragma unroll
           for (int y = 0; y < 2; ++y) {
             mma_bf16(qs[j + y], ph[0], ph[1], ph[2], ph[3], fh[2 * y], fh[2 * y + 1]);
             mma_bf16(qs[j + y], pl[0], pl[1], pl[2], pl[3], fh[2 * y], fh[2 * y + 1]);
-            if (DELTA) mma_bf16(qs[j + y], ph[0], ph[1], ph[2], ph[3], fl[2 * y], fl[2 * y + 1]);
+            mma_bf16(qs[j + y], ph[0], ph[1], ph[2], ph[3], fl[2 * y], fl[2 * y + 1]);
           }
         }
       }
@@ -587,18 +637,14 @@ __global__ void __launch_bounds__(256, 1) k_chunk_scan(ChunkArgs a) {
         for (int j = 0; j < 4; ++j) {
           const int n = wn * 32 + j * 8 + cq;
           if (e0 + n >= a.dvs) continue;
-          float2 r = make_float2(qs[j][2 * x], qs[j][2 * x + 1]);
-          if (!DELTA) {
-            const float2 v = __bfloat1622float2(*(const __nv_bfloat162*)(bs + L::V + (uint32_t)(t * LE + n) * 2u));
-            r.x += dsk * v.x; r.y += dsk * v.y;
-          }
+          const float2 r = make_float2(qs[j][2 * x], qs[j][2 * x + 1]);
           *(float2*)(o + n) = r;
         }
       }
     }
     // S = e^{G_last} S + K^T U'
     {
-      const float f = expf(glast);
+      const float f = g.whole;
 #pragma unroll
       for (int j = 0; j < SN; ++j) { S[j][0] *= f; S[j][1] *= f; S[j][2] *= f; S[j][3] *= f; }
 #pragma unroll
@@ -614,7 +660,216 @@ __global__ void __launch_bounds__(256, 1) k_chunk_scan(ChunkArgs a) {
             mma_bf16(S[j + 1], fk[0], fk[1], fk[2], fk[3], fb[2], fb[3]);
           }
       }
-      publish_state();  // every warp read the old one before the barrier above
+    }
+    if (c + 1 < c1) {
+      __syncthreads();  // the chunk's tiles are read
+      load(c + 1);
+      publish_state();
+    }
+  }
+#pragma unroll
+  for (int j = 0; j < SN; ++j)
+#pragma unroll
+    for (int b = 0; b < 2; ++b) {
+      const int r = sr + r_in + 8 * b, c = e0 + sc + j * 8 + cq;
+      if (r < a.dk && c < a.dvs) *(float2*)(Sg + (int64_t)r * a.dvs + c) = make_float2(S[j][2 * b], S[j][2 * b + 1]);
+    }
+}
+
+// The state space needs no solve, and its values are exact as bf16: P stays in registers from the
+// score product to the value product, and the writes' scales go onto the key operand.
+template <int DK>
+struct SsdSmem {
+  static constexpr int LK = DK + 8;
+  static constexpr uint32_t Q = 0, K = CT * LK * 2, V = K + CT * LK * 2;
+  static constexpr uint32_t S = V + CT * LE * 2;                 // [2][DK][LE]
+  static constexpr uint32_t GATES = S + 2 * DK * LE * 2;
+  static constexpr uint32_t BYTES = GATES + 2 * sizeof(Gates);
+};
+
+template <int DK>
+__global__ void __launch_bounds__(256, 2) k_ssd_scan(ChunkArgs a) {
+  using L = SsdSmem<DK>;
+  constexpr int LK = L::LK;
+  asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+  asm volatile("griddepcontrol.wait;" ::: "memory");
+  extern __shared__ __align__(16) uint8_t smem[];
+  const uint32_t base = sm_u32(smem);
+  Gates* gates = (Gates*)(smem + L::GATES);
+  const int e0 = blockIdx.x * EB, h = blockIdx.y, row = blockIdx.z, kh = h / (a.H / a.KH);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int wm = warp & 3, wn = warp >> 2;            // this warp's 16 tokens and 32 columns
+  const int r_in = lane >> 2, cq = (lane & 3) * 2;
+  const int c0 = a.row_chunk[row], c1 = a.row_chunk[row + 1];
+  const bool first = row_pos0(a.rows, row) == 0;
+  const int vw = min(EB, a.dvp - e0);
+
+  auto load = [&](int chunk) {
+    const int len = a.chunk_len[chunk];
+    const int64_t m0 = a.chunk_tok[chunk];
+    const int ch = a.DKp / 8;
+    for (int i = tid; i < CT * (DK / 8); i += 256) {
+      const int r = i / (DK / 8), c = i - r * (DK / 8);
+      const bool in = r < len && c < ch;
+      const int64_t o = (m0 + (in ? r : 0)) * (int64_t)a.KH * a.DKp + (int64_t)kh * a.DKp + (in ? c * 8 : 0);
+      const uint32_t d = (uint32_t)(r * LK + c * 8) * 2u;
+      cp_async16(base + L::Q + d, a.q + o, in ? 16 : 0);
+      cp_async16(base + L::K + d, a.k + o, in ? 16 : 0);
+    }
+    for (int i = tid; i < CT * (EB / 8); i += 256) {
+      const int r = i / (EB / 8), c = i - r * (EB / 8);
+      const bool in = r < len && c * 8 < vw;
+      cp_async16(base + L::V + (uint32_t)(r * LE + c * 8) * 2u,
+                 a.v + (m0 + (in ? r : 0)) * (int64_t)a.H * a.dvp + (int64_t)h * a.dvp + (in ? e0 + c * 8 : 0), in ? 16 : 0);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  load(c0);
+  if (warp == 7) load_gates(a, c0, h, kh, &gates[0], lane);
+
+  constexpr int SN = DK == 128 ? 8 : 4;
+  const int sr = DK == 128 ? warp * 16 : wm * 16, sc = DK == 128 ? 0 : wn * 32;
+  float S[SN][4];
+  float* Sg = a.S + ((int64_t)a.rows.slot[row] * a.H + h) * a.dk * a.dvs;
+#pragma unroll
+  for (int j = 0; j < SN; ++j)
+#pragma unroll
+    for (int b = 0; b < 2; ++b) {
+      const int r = sr + r_in + 8 * b, c = e0 + sc + j * 8 + cq;
+      float2 v = make_float2(0.f, 0.f);
+      if (!first && r < a.dk && c < a.dvs) v = *(const float2*)(Sg + (int64_t)r * a.dvs + c);
+      S[j][2 * b] = v.x; S[j][2 * b + 1] = v.y;
+    }
+  auto publish_state = [&]() {
+#pragma unroll
+    for (int j = 0; j < SN; ++j)
+#pragma unroll
+      for (int b = 0; b < 2; ++b) {
+        uint32_t hi, lo;
+        split2(S[j][2 * b], S[j][2 * b + 1], hi, lo);
+        const uint32_t o = (uint32_t)((sr + r_in + 8 * b) * LE + sc + j * 8 + cq) * 2u;
+        *(uint32_t*)(smem + L::S + o) = hi;
+        *(uint32_t*)(smem + L::S + DK * LE * 2 + o) = lo;
+      }
+  };
+  publish_state();
+  const float dsk = a.dskip[h];
+  const int t0 = wm * 16 + r_in;                      // this thread's tokens: t0 and t0 + 8
+
+  for (int c = c0; c < c1; ++c) {
+    const Gates& g = gates[(c - c0) & 1];
+    cp_async_wait_all();
+    __syncthreads();  // tiles, gates and state of this chunk are in place
+    if (c + 1 < c1 && warp == 7) load_gates(a, c + 1, h, kh, &gates[(c + 1 - c0) & 1], lane);
+    float o[4][4], qk[8][4];                           // C S0, then the output; C B^T of keys 0 .. wm * 16 + 15
+#pragma unroll
+    for (int j = 0; j < 4; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) qk[j][0] = qk[j][1] = qk[j][2] = qk[j][3] = 0.f;
+#pragma unroll
+    for (int kk = 0; kk < DK; kk += 16) {
+      uint32_t fq[4], fb[4];
+      frag_a(base + L::Q, LK, wm * 16, kk, lane, fq);
+#pragma unroll
+      for (int j = 0; j < 4; j += 2)
+#pragma unroll
+        for (int part = 0; part < 2; ++part) {
+          frag_b_kn(base + L::S + (uint32_t)(part * DK * LE * 2), LE, kk, wn * 32 + j * 8, lane, fb);
+          mma_bf16(o[j], fq[0], fq[1], fq[2], fq[3], fb[0], fb[1]);
+          mma_bf16(o[j + 1], fq[0], fq[1], fq[2], fq[3], fb[2], fb[3]);
+        }
+#pragma unroll
+      for (int j = 0; j < 8; j += 2)
+        if (j <= 2 * wm) {
+          frag_b_nk(base + L::K, LK, kk, j * 8, lane, fb);
+          mma_bf16(qk[j], fq[0], fq[1], fq[2], fq[3], fb[0], fb[1]);
+          mma_bf16(qk[j + 1], fq[0], fq[1], fq[2], fq[3], fb[2], fb[3]);
+        }
+    }
+    const float G0 = g.G[t0], G1 = g.G[t0 + 8];
+    {
+      const float f0 = g.eq[t0], f1 = g.eq[t0 + 8];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) { o[j][0] *= f0; o[j][1] *= f0; o[j][2] *= f1; o[j][3] *= f1; }
+    }
+    // o += P x: the scores' accumulator layout is the operand layout of the next product
+#pragma unroll
+    for (int kt = 0; kt < 4; ++kt)
+      if (kt <= wm) {
+        uint32_t ph[4], pl[4];
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+          const int j = 2 * kt + half, s = j * 8 + cq;
+          const float2 Gs = *(const float2*)(g.G + s), cs = *(const float2*)(g.co + s);
+          float p[4] = {qk[j][0] * pow2(G0 - Gs.x) * cs.x, qk[j][1] * pow2(G0 - Gs.y) * cs.y, qk[j][2] * pow2(G1 - Gs.x) * cs.x,
+                        qk[j][3] * pow2(G1 - Gs.y) * cs.y};
+          if (kt == wm) {
+            p[0] = s <= t0 ? p[0] : 0.f;
+            p[1] = s + 1 <= t0 ? p[1] : 0.f;
+            p[2] = s <= t0 + 8 ? p[2] : 0.f;
+            p[3] = s + 1 <= t0 + 8 ? p[3] : 0.f;
+          }
+          split2(p[0], p[1], ph[2 * half], pl[2 * half]);
+          split2(p[2], p[3], ph[2 * half + 1], pl[2 * half + 1]);
+        }
+#pragma unroll
+        for (int j = 0; j < 4; j += 2) {
+          uint32_t fb[4];
+          frag_b_kn(base + L::V, LE, kt * 16, wn * 32 + j * 8, lane, fb);
+#pragma unroll
+          for (int y = 0; y < 2; ++y) {
+            mma_bf16(o[j + y], ph[0], ph[1], ph[2], ph[3], fb[2 * y], fb[2 * y + 1]);
+            mma_bf16(o[j + y], pl[0], pl[1], pl[2], pl[3], fb[2 * y], fb[2 * y + 1]);
+          }
+        }
+      }
+    {
+      const int len = a.chunk_len[c];
+      const int64_t m0 = a.chunk_tok[c];
+#pragma unroll
+      for (int x = 0; x < 2; ++x) {
+        const int t = t0 + 8 * x;
+        if (t >= len) continue;
+        float* og = a.o + (m0 + t) * (int64_t)a.H * a.dvs + (int64_t)h * a.dvs + e0;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const int n = wn * 32 + j * 8 + cq;
+          if (e0 + n >= a.dvs) continue;
+          const float2 v = __bfloat1622float2(*(const __nv_bfloat162*)(smem + L::V + (uint32_t)(t * LE + n) * 2u));
+          *(float2*)(og + n) = make_float2(o[j][2 * x] + dsk * v.x, o[j][2 * x + 1] + dsk * v.y);
+        }
+      }
+    }
+    // S = e^{G_last} S + (f B)^T x
+    {
+      const float f = g.whole;
+#pragma unroll
+      for (int j = 0; j < SN; ++j) { S[j][0] *= f; S[j][1] *= f; S[j][2] *= f; S[j][3] *= f; }
+#pragma unroll
+      for (int kk = 0; kk < CT; kk += 16) {
+        uint32_t fk[4], kh4[4], kl4[4], fb[4];
+        frag_a_t(base + L::K, LK, sr, kk, lane, fk);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const float2 w = *(const float2*)(g.f + kk + cq + 8 * (i >> 1));
+          const float2 k = __bfloat1622float2(*(const __nv_bfloat162*)&fk[i]);
+          split2(k.x * w.x, k.y * w.y, kh4[i], kl4[i]);
+        }
+#pragma unroll
+        for (int j = 0; j < SN; j += 2) {
+          frag_b_kn(base + L::V, LE, kk, sc + j * 8, lane, fb);
+#pragma unroll
+          for (int y = 0; y < 2; ++y) {
+            mma_bf16(S[j + y], kh4[0], kh4[1], kh4[2], kh4[3], fb[2 * y], fb[2 * y + 1]);
+            mma_bf16(S[j + y], kl4[0], kl4[1], kl4[2], kl4[3], fb[2 * y], fb[2 * y + 1]);
+          }
+        }
+      }
+    }
+    if (c + 1 < c1) {
+      __syncthreads();  // tiles and old state are read
+      load(c + 1);
+      publish_state();
     }
   }
 #pragma unroll
@@ -628,22 +883,23 @@ __global__ void __launch_bounds__(256, 1) k_chunk_scan(ChunkArgs a) {
 
 template <int DK, bool DELTA>
 int launch_scan(cg_ctx* c, const ChunkArgs& a) {
-  using L = ScanSmem<DK, DELTA>;
-  static_assert(L::BYTES <= 227 * 1024, "shared memory");
+  constexpr size_t smem = DELTA ? (size_t)DeltaSmem<DK>::BYTES : (size_t)SsdSmem<DK>::BYTES;
+  static_assert(smem <= 113 * 1024, "two blocks per SM");
+  auto kernel = DELTA ? k_delta_scan<DK> : k_ssd_scan<DK>;
   static PerDeviceFlag configured_on;
   bool& configured = configured_on.at(c->core->device);
   if (!configured) {
-    CG_CUDA(c, cudaFuncSetAttribute(k_chunk_scan<DK, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)L::BYTES));
+    CG_CUDA(c, cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     configured = true;
   }
   dim3 grid((unsigned)((a.dv + EB - 1) / EB), (unsigned)a.H, (unsigned)a.rows.rows);
-  CG_CUDA(c, launch_kernel(c, k_chunk_scan<DK, DELTA>, grid, dim3(256), L::BYTES, 1, a));
+  CG_CUDA(c, launch_kernel(c, kernel, grid, dim3(256), smem, 1, a));
   CG_LAUNCHED(c);
   return CG_OK;
 }
 template <int DK>
 int launch_solve(cg_ctx* c, const ChunkArgs& a) {
-  constexpr size_t smem = (size_t)CT * 68 * 4 + std::max((size_t)CT * 80 * 4, (size_t)CT * (DK + 8) * 2);
+  constexpr size_t smem = (size_t)CT * 68 * 4 + std::max((size_t)CT * 68 * 4, (size_t)CT * (DK + 8) * 2);
   CG_CUDA(c, launch_kernel(c, k_delta_solve<DK>, dim3((unsigned)a.n_chunks, (unsigned)a.H), dim3(128), smem, 1, a));
   CG_LAUNCHED(c);
   return CG_OK;
@@ -655,10 +911,10 @@ bool chunk_supported(int dk) { return dk <= 128; }
 
 int k_launch_chunk_recurrence(cg_ctx* c, const ChunkArgs& a) {
   if (a.rows.M == 0) return CG_OK;
-  const int lanes = a.dk / 8;
+  const int lanes = a.dk / CV;
   const bool fast = a.dk % 8 == 0 && a.dv % 8 == 0 && a.DKp == a.dk && (!a.delta || (lanes & (lanes - 1)) == 0) && a.taps >= 1 && a.taps <= 4;
   if (fast) {
-    dim3 grid((unsigned)((a.C + 1023) / 1024), (unsigned)(a.n_chunks * (CT / CONV_TOK)));
+    dim3 grid((unsigned)((a.C + 128 * CV - 1) / (128 * CV)), (unsigned)(a.n_chunks * (CT / CONV_TOK)));
     if (grid.y > 65535) return fail(c, CG_ERR_UNSUPPORTED, "recurrence: too many tokens in one portion");
     switch (a.taps) {
       case 1: CG_CUDA(c, launch_kernel(c, k_conv_chunk<1>, grid, dim3(128), 0, 1, a)); break;
