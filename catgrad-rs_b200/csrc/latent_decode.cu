@@ -7,12 +7,14 @@
 //                     last blocks norm / rotate / append the tokens' own cached rows and rotate q
 //   k_latent_dec      one block per (token, 16 heads, context slice): heads are the rows of the
 //                     MMA tile; 64 cached rows at a time through two shared-memory buffers,
-//                     online softmax, partial output in the latent space
-//   k_latent_out      one block per (head, 32 values): the slices are merged and mapped through Wuv
+//                     online softmax.  The slices are a thread-block cluster and merge their partial
+//                     outputs over distributed shared memory, each its share of the latent columns
+//   k_latent_out      one block per (head, 16 values): Wuv on the merged output
 #include <algorithm>
 
 #include "mixers.h"
 #include "mma.cuh"
+#include "tc_common.cuh"
 
 namespace cg {
 
@@ -35,8 +37,7 @@ __device__ __forceinline__ float block_sum(float v, float* sh) {
 
 struct DecodeScratch {
   __nv_bfloat16* qa;   // [M, H, Lw] queries in the cached rows' space
-  float* o;            // [M, H, splits, R] partial outputs, relative to their maximum
-  float2* ml;          // [M, H, splits] maximum, sum
+  float* o;            // [M, H, R] attention output in the latent space
   int splits;
 };
 
@@ -112,6 +113,7 @@ __global__ void __launch_bounds__(256) k_latent_absorb(LatentArgs a, DecodeScrat
   }
 }
 
+constexpr int MAX_SLICES = 8;  // a portable cluster
 constexpr int LD_KT = 64;  // cached rows per tile
 
 // NT: 8-column output tiles per warp (eight warps share the latent columns)
@@ -132,7 +134,7 @@ __global__ void __launch_bounds__(256) k_latent_dec(LatentArgs a, DecodeScratch 
   const int64_t pos = row_pos0(a.rows, row) + (m - a.rows.start[row]);
   const __nv_bfloat16* base = (const __nv_bfloat16*)a.cache + (int64_t)a.rows.slot[row] * a.Tmax * a.Lw;
   const int64_t n_keys = pos + 1;
-  const int64_t per = ((n_keys + sc.splits - 1) / sc.splits + LD_KT - 1) / LD_KT * LD_KT;
+  const int64_t per = ((n_keys + sc.splits - 1) / sc.splits + 15) / 16 * 16;
   const int64_t k_lo = split * per, k_hi = min(n_keys, k_lo + per);
   const int CH = (int)a.Lw / 8;
   const uint32_t sq_u = (uint32_t)__cvta_generic_to_shared(sq), sk_u = (uint32_t)__cvta_generic_to_shared(sk),
@@ -236,36 +238,73 @@ __global__ void __launch_bounds__(256) k_latent_dec(LatentArgs a, DecodeScratch 
       }
     }
   }
+  // partial outputs and {maximum, sum} per head, over the tiles (each CTA's own are read)
+  const int ldo = a.R + 4;
+  float* so = (float*)sk;                              // [16][ldo]
+  float2* sml = (float2*)wm;                           // [16]
+  __syncthreads();
 #pragma unroll
   for (int x = 0; x < 2; ++x) {
-    const int h = h0 + r_in + 8 * x;
-    if (h >= a.H) continue;
-    const int64_t at = (m * a.H + h) * sc.splits + split;
-    if (warp == 0 && (lane & 3) == 0) sc.ml[at] = make_float2(mrow[x], lrow[x]);
-    if (k_lo >= k_hi) continue;  // nothing here: the sum says so
+    if (warp == 0 && (lane & 3) == 0) sml[r_in + 8 * x] = make_float2(mrow[x], lrow[x]);
 #pragma unroll
     for (int j = 0; j < NT; ++j) {
       const int col = (warp * NT + j) * 8 + cq;
 #pragma unroll
       for (int y = 0; y < 2; ++y)
-        if (col + y < a.R) sc.o[at * a.R + col + y] = o[j][2 * x + y];
+        if (col + y < a.R) so[(r_in + 8 * x) * ldo + col + y] = o[j][2 * x + y];
     }
   }
+  const int ns = sc.splits;
+  if (ns > 1) tc::cluster_sync_all();
+  else __syncthreads();
+  float* wt = (float*)(sml + 16);                      // [ns][16] weight of each slice
+  if (tid < 16) {
+    float2 v[MAX_SLICES];
+    float mx = -INFINITY, l = 0.f;
+    const uint32_t at = tc::smem_u32(sml + tid);
+#pragma unroll
+    for (int k = 0; k < MAX_SLICES; ++k) {
+      v[k] = make_float2(-INFINITY, 0.f);
+      if (k < ns) v[k] = ns > 1 ? make_float2(tc::ld_cluster_f32(at, k), tc::ld_cluster_f32(at + 4, k)) : sml[tid];
+      mx = fmaxf(mx, v[k].x);
+    }
+#pragma unroll
+    for (int k = 0; k < MAX_SLICES; ++k) {
+      v[k].x = v[k].y > 0.f ? expf(v[k].x - mx) : 0.f;
+      l += v[k].x * v[k].y;
+    }
+#pragma unroll
+    for (int k = 0; k < MAX_SLICES; ++k)
+      if (k < ns) wt[k * 16 + tid] = v[k].x / l;
+  }
+  __syncthreads();
+  const int share = (a.R + ns - 1) / ns, c_lo = split * share, c_hi = min(a.R, c_lo + share);
+  for (int i = tid; i < 16 * share; i += 256) {
+    const int r = i / share, col = c_lo + (i - r * share);
+    if (h0 + r >= a.H || col >= c_hi) continue;
+    const uint32_t at = tc::smem_u32(so + r * ldo + col);
+    float p[MAX_SLICES], v = 0.f;
+#pragma unroll
+    for (int k = 0; k < MAX_SLICES; ++k) p[k] = k < ns ? (ns > 1 ? tc::ld_cluster_f32(at, k) : so[r * ldo + col]) : 0.f;
+#pragma unroll
+    for (int k = 0; k < MAX_SLICES; ++k)
+      if (k < ns) v += p[k] * wt[k * 16 + r];
+    sc.o[(m * a.H + h0 + r) * a.R + col] = v;
+  }
+  if (ns > 1) tc::cluster_sync_all();  // nobody leaves while another CTA may read its shared memory
 }
 
-// out[m, h, e] = Wuv[h, e] . (merged latent output): eight warps, four value rows each.  The rows of
-// Wuv are fetched before the dependency wait and stay in registers (R <= 512, even) for all tokens.
+// out[m, h, e] = Wuv[h, e] . o[m, h]: eight warps, two value rows each.  The rows of Wuv are fetched
+// before the dependency wait and stay in registers (R <= 512) for all tokens.
 __global__ void __launch_bounds__(256) k_latent_out(LatentArgs a, DecodeScratch s) {
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
-  extern __shared__ __align__(16) float oc[];          // [R + 1]
-  __shared__ float wt[16];
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int h = blockIdx.x, e0 = blockIdx.y * 32 + warp * 4;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int h = blockIdx.x, e0 = blockIdx.y * 16 + warp * 2;
   const __nv_bfloat16* uv = (const __nv_bfloat16*)a.uv + (int64_t)h * a.dv * a.R;
   const bool even = (a.R & 1) == 0;
-  __nv_bfloat162 w[4][8];
+  __nv_bfloat162 w[2][8];
 #pragma unroll
-  for (int y = 0; y < 4; ++y)
+  for (int y = 0; y < 2; ++y)
 #pragma unroll
     for (int k = 0; k < 8; ++k) {
       const int i = 2 * lane + 64 * k;
@@ -278,50 +317,27 @@ __global__ void __launch_bounds__(256) k_latent_out(LatentArgs a, DecodeScratch 
     }
   asm volatile("griddepcontrol.wait;" ::: "memory");
   for (int64_t m = blockIdx.z; m < a.rows.M; m += gridDim.z) {
-    const int64_t at = (m * a.H + h) * s.splits;
-    // the slices' partial values, requested before their weights are known
-    float p[2][16];
-#pragma unroll
-    for (int x = 0; x < 2; ++x)
-#pragma unroll
-      for (int k = 0; k < 16; ++k) p[x][k] = k < s.splits && tid + 256 * x < a.R ? s.o[(at + k) * a.R + tid + 256 * x] : 0.f;
-    if (warp == 0) {
-      const float2 v = lane < s.splits ? s.ml[at + lane] : make_float2(-INFINITY, 0.f);
-      float mx = v.x;
-#pragma unroll
-      for (int o = 16; o; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-      const float e = v.y > 0.f ? expf(v.x - mx) : 0.f;
-      const float l = warp_sum(e * v.y);
-      if (lane < 16) wt[lane] = e / l;
-    }
-    __syncthreads();
-#pragma unroll
-    for (int x = 0; x < 2; ++x) {
-      float v = 0.f;
-#pragma unroll
-      for (int k = 0; k < 16; ++k) {
-        const float f = wt[k];
-        if (f > 0.f) v += p[x][k] * f;   // an empty slice left nothing to read
-      }
-      if (tid + 256 * x < a.R) oc[tid + 256 * x] = v;
-    }
-    if (tid == 0) oc[a.R] = 0.f;
-    __syncthreads();
-    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+    const float* o = s.o + (m * a.H + h) * a.R;
+    float2 v[8];
 #pragma unroll
     for (int k = 0; k < 8; ++k) {
       const int i = 2 * lane + 64 * k;
+      v[k] = make_float2(0.f, 0.f);
       if (i < a.R) {
-        const float2 v = *(const float2*)(oc + i);
-#pragma unroll
-        for (int y = 0; y < 4; ++y) {
-          const float2 f = __bfloat1622float2(w[y][k]);
-          acc[y] += v.x * f.x + v.y * f.y;
-        }
+        if (even) v[k] = *(const float2*)(o + i);
+        else v[k] = make_float2(o[i], i + 1 < a.R ? o[i + 1] : 0.f);
       }
     }
+    float acc[2] = {0.f, 0.f};
 #pragma unroll
-    for (int y = 0; y < 4; ++y) {
+    for (int k = 0; k < 8; ++k)
+#pragma unroll
+      for (int y = 0; y < 2; ++y) {
+        const float2 f = __bfloat1622float2(w[y][k]);
+        acc[y] += v[k].x * f.x + v[k].y * f.y;
+      }
+#pragma unroll
+    for (int y = 0; y < 2; ++y) {
       acc[y] = warp_sum(acc[y]);
       if (lane == 0 && e0 + y < a.dv) ((__nv_bfloat16*)a.att)[m * a.ld_att + (int64_t)h * a.Do + e0 + y] = __float2bfloat16_rn(acc[y]);
     }
@@ -330,13 +346,13 @@ __global__ void __launch_bounds__(256) k_latent_out(LatentArgs a, DecodeScratch 
 
 int pick_nt(int R) { return R <= 128 ? 2 : R <= 256 ? 4 : R <= 512 ? 8 : 0; }
 int row_pitch(const LatentArgs& a) { return std::max((int)(a.Lw + 15) / 16 * 16, pick_nt(a.R) * 64) + 8; }
-size_t dec_smem(int ldk) { return (size_t)(16 + 2 * LD_KT) * ldk * 2 + 16 * 72 * 2 + 256 * 4; }
+size_t dec_smem(int ldk) { return (size_t)(16 + 2 * LD_KT) * ldk * 2 + 16 * 72 * 2 + 256 * 4; }  // (the merge fits over the tiles)
 
-// context slices: enough blocks for every SM, at least one tile each at full context
+// context slices: enough blocks for every SM, at most about one tile each at full context
 int pick_splits(const LatentArgs& a, int64_t M) {
   const int64_t base = M * ((a.H + 15) / 16);
   int s = 1;
-  while (s < 16 && base * (s * 2) <= 2 * 148 && (int64_t)s * 2 * LD_KT <= a.Tmax) s *= 2;
+  while (s < MAX_SLICES && base * (s * 2) <= 2 * 148 && (int64_t)s * LD_KT < a.Tmax) s *= 2;
   return s;
 }
 
@@ -351,7 +367,7 @@ int launch_dec(cg_ctx* c, const LatentArgs& a, const DecodeScratch& s) {
     configured = smem;
   }
   dim3 grid((unsigned)a.rows.M, (unsigned)((a.H + 15) / 16), (unsigned)s.splits);
-  CG_CUDA(c, launch_kernel(c, k_latent_dec<NT>, grid, dim3(256), smem, 1, a, s, ldk));
+  CG_CUDA(c, launch_kernel(c, k_latent_dec<NT>, grid, dim3(256), smem, s.splits, a, s, ldk));
   CG_LAUNCHED(c);
   return CG_OK;
 }
@@ -368,7 +384,7 @@ bool latent_decode_supported(int d, int R, int64_t Lw) {
 
 size_t latent_decode_scratch(const LatentArgs& a, int64_t M) {
   const size_t n = (size_t)M * a.H;
-  return up16b(n * a.Lw * 2) + up16b(n * 16 * 8) + n * 16 * a.R * 4;
+  return up16b(n * a.Lw * 2) + n * a.R * 4;
 }
 
 int k_launch_latent_decode(cg_ctx* c, const LatentArgs& a, void* scratch) {
@@ -378,8 +394,7 @@ int k_launch_latent_decode(cg_ctx* c, const LatentArgs& a, void* scratch) {
   s.splits = pick_splits(a, M);
   const size_t n = (size_t)M * a.H;
   s.qa = (__nv_bfloat16*)scratch;
-  s.ml = (float2*)((char*)scratch + up16b(n * a.Lw * 2));
-  s.o = (float*)((char*)s.ml + up16b(n * 16 * 8));
+  s.o = (float*)((char*)scratch + up16b(n * a.Lw * 2));
   const int cb = (a.R + 63) / 64;
   const size_t sm1 = std::max<size_t>((size_t)(8 * 256 + 8 * a.d) * 4 + (size_t)a.d * 128, 128);
   CG_CUDA(c, launch_kernel(c, k_latent_absorb, dim3((unsigned)(a.H * cb + M)), dim3(256), sm1, 1, a, s, cb));
@@ -389,9 +404,9 @@ int k_launch_latent_decode(cg_ctx* c, const LatentArgs& a, void* scratch) {
     case 4: CG_TRY(launch_dec<4>(c, a, s)); break;
     default: CG_TRY(launch_dec<8>(c, a, s)); break;
   }
-  const int eb = (a.dv + 31) / 32;
-  const int mz = (int)std::min<int64_t>(M, std::max<int64_t>(1, 3 * 148 / std::max(1, a.H * eb)));
-  CG_CUDA(c, launch_kernel(c, k_latent_out, dim3((unsigned)a.H, (unsigned)eb, (unsigned)mz), dim3(256), (size_t)(a.R + 1) * 4, 1, a, s));
+  const int eb = (a.dv + 15) / 16;
+  const int mz = (int)std::min<int64_t>(M, std::max<int64_t>(1, 4 * 148 / std::max(1, a.H * eb)));
+  CG_CUDA(c, launch_kernel(c, k_latent_out, dim3((unsigned)a.H, (unsigned)eb, (unsigned)mz), dim3(256), 0, 1, a, s));
   CG_LAUNCHED(c);
   return CG_OK;
 }

@@ -31,8 +31,21 @@ __device__ __forceinline__ void store4(__nv_bfloat16* p, const float* v) {
 }
 
 
+// v = v * inv * g for vector i of a row
+template <bool EXACT>
+__device__ __forceinline__ void gain(float* v, float inv, const float* g, int i, int W) {
+  if (EXACT) {
+    const float4 w = *(const float4*)(g + 4 * i);
+    v[0] *= inv * w.x; v[1] *= inv * w.y; v[2] *= inv * w.z; v[3] *= inv * w.w;
+  } else {
+#pragma unroll
+    for (int e = 0; e < 4; ++e) v[e] = 4 * i + e < W ? v[e] * (inv * g[4 * i + e]) : 0.f;
+  }
+}
+
 // One block per row; the row lives in registers (RU_VEC 128-bit vectors per thread).
-template <class T, int RU_VEC>
+// EXACT: W is a multiple of 8, so no column is padding and gains and table rows are read as vectors.
+template <class T, int RU_VEC, bool EXACT>
 __global__ void k_row_update(RowUpdate u, int32_t* err) {
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
   asm volatile("griddepcontrol.wait;" ::: "memory");
@@ -65,6 +78,11 @@ __global__ void k_row_update(RowUpdate u, int32_t* err) {
       if (j < nv && i < n4) {
         if (u.tokens) {
           const int64_t o = (int64_t)tok * W + 4 * i;
+          if (EXACT && u.table_bf16) {
+            const uint2 r = *(const uint2*)((const __nv_bfloat16*)u.table + o);
+            const float2 a = __bfloat1622float2(*(const __nv_bfloat162*)&r.x), b = __bfloat1622float2(*(const __nv_bfloat162*)&r.y);
+            v[j][0] = a.x; v[j][1] = a.y; v[j][2] = b.x; v[j][3] = b.y;
+          } else
 #pragma unroll
           for (int e = 0; e < 4; ++e)
             if (4 * i + e < W)
@@ -72,9 +90,10 @@ __global__ void k_row_update(RowUpdate u, int32_t* err) {
         } else {
           const float4 t = *(const float4*)(u.y + m * u.ldy + 4 * i);
           v[j][0] = t.x; v[j][1] = t.y; v[j][2] = t.z; v[j][3] = t.w;
+          if (!EXACT)
 #pragma unroll
-          for (int e = 0; e < 4; ++e)
-            if (4 * i + e >= W) v[j][e] = 0.f;
+            for (int e = 0; e < 4; ++e)
+              if (4 * i + e >= W) v[j][e] = 0.f;
         }
       }
 #pragma unroll
@@ -82,13 +101,11 @@ __global__ void k_row_update(RowUpdate u, int32_t* err) {
     }
     if (u.g1) {
       ss = block_sum(ss, sh);
-      const float rms = sqrtf(ss / (float)W + u.eps);
+      const float inv = 1.f / sqrtf(ss / (float)W + u.eps);
 #pragma unroll
       for (int j = 0; j < RU_VEC; ++j) {
         const int i = threadIdx.x + j * blockDim.x;
-        if (j < nv && i < n4)
-#pragma unroll
-          for (int e = 0; e < 4; ++e) v[j][e] = 4 * i + e < W ? v[j][e] / rms * u.g1[4 * i + e] : 0.f;
+        if (j < nv && i < n4) gain<EXACT>(v[j], inv, u.g1, i, W);
       }
     }
 #pragma unroll
@@ -116,13 +133,11 @@ __global__ void k_row_update(RowUpdate u, int32_t* err) {
 #pragma unroll
       for (int e = 0; e < 4; ++e) ss += v[j][e] * v[j][e];
     ss = block_sum(ss, sh);
-    const float rms = sqrtf(ss / (float)W + u.eps);
+    const float inv = 1.f / sqrtf(ss / (float)W + u.eps);
 #pragma unroll
     for (int j = 0; j < RU_VEC; ++j) {
       const int i = threadIdx.x + j * blockDim.x;
-      if (j < nv && i < n4)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) v[j][e] = 4 * i + e < W ? v[j][e] / rms * u.g2[4 * i + e] : 0.f;
+      if (j < nv && i < n4) gain<EXACT>(v[j], inv, u.g2, i, W);
     }
   }
 #pragma unroll
@@ -161,11 +176,16 @@ __global__ void k_pair_rope_tables(double base, int64_t T, int r, float* cos_t, 
 int k_launch_row_update(cg_ctx* c, const RowUpdate& u, int64_t M, int out_bf16) {
   if (M == 0) return CG_OK;
   const int n4 = (u.W + 7) / 8 * 2;
-  const int vec = n4 <= 512 || (n4 <= 1024 && M <= 296) ? 1 : n4 <= 1024 ? 2 : 4;
+  const bool exact = u.W % 8 == 0;
+  const int vec = M <= 296 ? (n4 <= 1024 ? 1 : 4) : n4 <= 2048 ? 2 : 4;
   const int block = ((n4 + vec - 1) / vec + 31) / 32 * 32;
   if (block > 1024) return fail(c, CG_ERR_UNSUPPORTED, "decoder: rows wider than 16384 are not supported");
-  auto kernel = out_bf16 ? (vec == 1 ? k_row_update<__nv_bfloat16, 1> : vec == 2 ? k_row_update<__nv_bfloat16, 2> : k_row_update<__nv_bfloat16, 4>)
-                         : (vec == 1 ? k_row_update<float, 1> : vec == 2 ? k_row_update<float, 2> : k_row_update<float, 4>);
+  auto pick = [&](auto t) {
+    using T = decltype(t);
+    if (exact) return vec == 1 ? k_row_update<T, 1, true> : vec == 2 ? k_row_update<T, 2, true> : k_row_update<T, 4, true>;
+    return vec == 1 ? k_row_update<T, 1, false> : vec == 2 ? k_row_update<T, 2, false> : k_row_update<T, 4, false>;
+  };
+  auto kernel = out_bf16 ? pick(__nv_bfloat16()) : pick(float());
   CG_CUDA(c, launch_kernel(c, kernel, dim3((unsigned)M), dim3(block), 0, 1, u, c->core->dev_err));
   CG_LAUNCHED(c);
   return CG_OK;

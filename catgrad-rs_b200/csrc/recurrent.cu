@@ -3,6 +3,7 @@
 // gates are f32.
 #include <algorithm>
 
+#include "act.cuh"
 #include "mixers.h"
 
 namespace cg {
@@ -346,7 +347,8 @@ __global__ void k_gated_norm_vec(GatedNorm a, int n, int units, int threads) {
   }
 #pragma unroll
   for (int j = 0; j < V; ++j) {
-    g[j] = make_float4(silu(g[j].x), silu(g[j].y), silu(g[j].z), silu(g[j].w));
+    g[j] = sizeof(TG) == 2 ? make_float4(silu_fast(g[j].x), silu_fast(g[j].y), silu_fast(g[j].z), silu_fast(g[j].w))
+                           : make_float4(silu(g[j].x), silu(g[j].y), silu(g[j].z), silu(g[j].w));
     if (!a.delta) { x[j].x *= g[j].x; x[j].y *= g[j].y; x[j].z *= g[j].z; x[j].w *= g[j].w; }
     ss += x[j].x * x[j].x + x[j].y * x[j].y + x[j].z * x[j].z + x[j].w * x[j].w;
   }

@@ -106,12 +106,50 @@ __global__ void __launch_bounds__(256) k_conv_chunk_any(ChunkArgs a) {
   }
 }
 
-// Sizes in multiples of 8: a thread takes 4 neighbouring channels of 16 tokens and slides over
+// pairs of f32 in one 64-bit register: Blackwell's packed f32 arithmetic, rounded like the scalar one
+__device__ __forceinline__ uint64_t pack2(float a, float b) {
+  uint64_t r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+  return r;
+}
+__device__ __forceinline__ float2 unpack2(uint64_t v) {
+  float2 r;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+  return r;
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+  uint64_t r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+__device__ __forceinline__ uint64_t add2(uint64_t a, uint64_t b) {
+  uint64_t r;
+  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+__device__ __forceinline__ uint64_t widen2(uint32_t v) { return pack2(__uint_as_float(v << 16), __uint_as_float(v & 0xffff0000u)); }
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float rcp(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+// Sizes in multiples of 8: a thread takes 4 neighbouring channels of 32 tokens and slides over
 // them.  Same outputs.
-constexpr int CONV_TOK = 16;
+constexpr int CONV_TOK = 32;
 constexpr int CV = 4;  // neighbouring channels of a thread
 template <int TAPS>
-__global__ void __launch_bounds__(128) k_conv_chunk(ChunkArgs a) {
+__global__ void __launch_bounds__(128, 6) k_conv_chunk(ChunkArgs a) {
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
   asm volatile("griddepcontrol.wait;" ::: "memory");
   const int chunk = blockIdx.y / (CT / CONV_TOK), sub = blockIdx.y % (CT / CONV_TOK);
@@ -125,34 +163,28 @@ __global__ void __launch_bounds__(128) k_conv_chunk(ChunkArgs a) {
   const bool live = c < a.C;
   const int cc = live ? c : 0;
   const float* tail = a.tail + (int64_t)a.rows.slot[row] * a.taps * a.C + cc;
-  float w[TAPS][CV], bias[CV];
+  uint64_t w[TAPS][CV / 2], bias[CV / 2];  // channel pairs
 #pragma unroll
-  for (int e = 0; e < CV; ++e) {
-    bias[e] = a.conv_b ? a.conv_b[cc + e] : 0.f;
+  for (int e = 0; e < CV / 2; ++e) {
+    bias[e] = a.conv_b ? pack2(a.conv_b[cc + 2 * e], a.conv_b[cc + 2 * e + 1]) : 0;
+    const float* t0 = a.conv_w + (int64_t)(cc + 2 * e) * TAPS;
 #pragma unroll
-    for (int j = 0; j < TAPS; ++j) w[j][e] = a.conv_w[(int64_t)(cc + e) * TAPS + TAPS - 1 - j];
+    for (int j = 0; j < TAPS; ++j) w[j][e] = pack2(t0[TAPS - 1 - j], t0[2 * TAPS - 1 - j]);
   }
   // x[TAPS - 1 + i]: the input of the group's token i; x[TAPS - 1 - j]: the one j tokens before the group
   constexpr int G = 4;
-  float x[TAPS - 1 + G][CV];
-  auto widen = [](const uint2& r, float* v) {
-    const uint32_t p[2] = {r.x, r.y};
-#pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      const float2 f = __bfloat1622float2(*(const __nv_bfloat162*)&p[e]);
-      v[2 * e] = f.x; v[2 * e + 1] = f.y;
-    }
-  };
+  uint64_t x[TAPS - 1 + G][CV / 2];
+  static_assert(CV == 4, "two channel pairs");
 #pragma unroll
   for (int j = 1; j < TAPS; ++j) {
-    float* v = x[TAPS - 1 - j];
-#pragma unroll
-    for (int e = 0; e < CV; ++e) v[e] = 0.f;
-    if (j <= i0) widen(*(const uint2*)(a.proj + (m0 - j) * a.ldp + cc), v);
-    else if (p0 + i0 - j >= 0) {
+    uint64_t* v = x[TAPS - 1 - j];
+    v[0] = v[1] = 0;
+    if (j <= i0) {
+      const uint2 r = *(const uint2*)(a.proj + (m0 - j) * a.ldp + cc);
+      v[0] = widen2(r.x); v[1] = widen2(r.y);
+    } else if (p0 + i0 - j >= 0) {
       const float* tp = tail + (int64_t)((p0 + i0 - j) % a.taps) * a.C;
-#pragma unroll
-      for (int e = 0; e < CV; ++e) v[e] = tp[e];
+      v[0] = pack2(tp[0], tp[1]); v[1] = pack2(tp[2], tp[3]);
     }
   }
   // where these channels go
@@ -173,48 +205,65 @@ __global__ void __launch_bounds__(128) k_conv_chunk(ChunkArgs a) {
     if (!isk) f = rsqrtf((float)a.dk);
   }
   const int lanes = a.dk / CV;  // threads of a head: a power of two dividing the warp
+  const bool normed = __any_sync(0xffffffffu, a.delta && c < a.v_off);  // this warp has query or key channels
+  const __nv_bfloat16* pin = a.proj + m0 * a.ldp + cc;
+  __nv_bfloat16* po = out + m0 * ld;
+  float* pn = rn ? rn + m0 * a.KH : nullptr;
+  const uint64_t nlog2e = pack2(-1.4426950408889634f, -1.4426950408889634f), one2 = pack2(1.f, 1.f);
+  const int n = live ? t_hi - t_lo : 0;  // tokens this thread stores
+  int t = 0;
   uint2 raw[G];
-  auto fetch = [&](int t) {
+  auto fetch = [&]() {
 #pragma unroll
-    for (int i = 0; i < G; ++i) raw[i] = t + i < t_hi ? *(const uint2*)(a.proj + (m0 + t - t_lo + i) * a.ldp + cc) : make_uint2(0, 0);
+    for (int i = 0; i < G; ++i) {
+      raw[i] = t + i < t_hi - t_lo ? *(const uint2*)pin : make_uint2(0, 0);
+      pin += a.ldp;
+    }
   };
-  fetch(t_lo);
-  for (int t = t_lo; t < t_hi; t += G) {
-    const int64_t m = m0 + t - t_lo;
+  fetch();
+  for (; t < t_hi - t_lo;) {
 #pragma unroll
-    for (int i = 0; i < G; ++i) widen(raw[i], x[TAPS - 1 + i]);
-    fetch(t + G);  // the next group's inputs are on the way while this one is computed
+    for (int i = 0; i < G; ++i) { x[TAPS - 1 + i][0] = widen2(raw[i].x); x[TAPS - 1 + i][1] = widen2(raw[i].y); }
+    t += G;
+    fetch();  // the next group's inputs are on the way while this one is computed
 #pragma unroll
     for (int i = 0; i < G; ++i) {
       uint32_t o[2];
       float ss = 0.f;
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
-        float y[2];
+        uint64_t v = bias[e];
 #pragma unroll
-        for (int b = 0; b < 2; ++b) {
-          float v = bias[2 * e + b];
-#pragma unroll
-          for (int j = 0; j < TAPS; ++j) v += w[j][2 * e + b] * x[TAPS - 1 + i - j][2 * e + b];
-          y[b] = silu(v);
-        }
-        const __nv_bfloat162 h2 = __floats2bfloat162_rn(y[0], y[1]);
+        for (int j = 0; j < TAPS; ++j) v = fma2(w[j][e], x[TAPS - 1 + i - j][e], v);
+        // silu: v / (1 + 2^(-v log2 e)), rounded to bf16 at once
+        const float2 z = unpack2(mul2(v, nlog2e));
+        const float2 d = unpack2(add2(pack2(ex2(z.x), ex2(z.y)), one2));
+        const float2 y = unpack2(mul2(v, pack2(rcp(d.x), rcp(d.y))));
+        const __nv_bfloat162 h2 = __floats2bfloat162_rn(y.x, y.y);
         o[e] = *(const uint32_t*)&h2;
-        if (a.delta) {
-          const float2 g = __bfloat1622float2(h2);
-          ss += g.x * g.x + g.y * g.y;
-        }
       }
-      const bool in = live && t + i < t_hi;
-      if (in) *(uint2*)(out + (m + i) * ld) = make_uint2(o[0], o[1]);
-      if (a.delta)
-        for (int s = lanes / 2; s; s >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, s);
-      if (in && rn) rn[(m + i) * a.KH] = a.delta ? f / sqrtf(ss + 1e-6f) : 1.f;
+      if (normed) {
+        const uint64_t a0 = widen2(o[0]), a1 = widen2(o[1]);
+        const float2 q = unpack2(fma2(a1, a1, mul2(a0, a0)));
+        ss = q.x + q.y;
+      }
+      const bool in = t - G + i < n;
+      if (in) *(uint2*)po = make_uint2(o[0], o[1]);
+      po += ld;
+      if (normed) {
+#pragma unroll
+        for (int s = 16; s; s >>= 1)
+          if (s < lanes) ss += __shfl_xor_sync(0xffffffffu, ss, s);
+      }
+      if (pn) {
+        if (in) *pn = normed ? f * rsqrtf(ss + 1e-6f) : 1.f;
+        pn += a.KH;
+      }
     }
 #pragma unroll
     for (int j = 0; j < TAPS - 1; ++j)
 #pragma unroll
-      for (int e = 0; e < CV; ++e) x[j][e] = x[j + G][e];
+      for (int e = 0; e < CV / 2; ++e) x[j][e] = x[j + G][e];
   }
 }
 
