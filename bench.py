@@ -108,6 +108,104 @@ WORKLOADS = {
 }
 
 
+# the same for models built layer by layer (catgrad-rs_b200/layered.py); measured beside an attention-only
+# decoder of equal width, feed-forward, vocabulary and number of layer runs
+LAYERED_WORKLOADS = {
+    "ralapel-w1024": ("RALAPEL_W1024", 8, 512, 128),
+    "ralapel-w2048": ("RALAPEL_W2048", 8, 512, 128),
+    "ralapel-w2048-b1": ("RALAPEL_W2048", 1, 512, 128),
+    "ralapel-w2048-long": ("RALAPEL_W2048", 4, 4096, 128),
+    "ralapel-w4096": ("RALAPEL_W4096", 8, 1024, 128),
+}
+
+
+def layered_step_bytes(cfg, batch: int, context: float) -> dict:
+    """Bytes a decode step has to move: every layer run's matrices and the head once, the f32 states
+    read and written, the cached rows read."""
+    mats, states, cache = 2 * cfg.vocab_size * cfg.hidden_size, 0, 0.0
+    shapes = cfg.param_shapes()
+    for i in cfg.layer_runs():
+        mats += sum(2 * n[0] * n[1] for k, n in shapes.items() if k.startswith(f"l{i}.") and len(n) == 2 and not k.endswith("conv"))
+        m = cfg.layers[i].sizes
+        if cfg.layers[i].mixer == "latent_attention":
+            cache += batch * context * (m["kv_rank"] + m["rot_dim"]) * 2
+        else:
+            states += 2 * 4 * batch * m["heads"] * m["vdim"] * (m["dim"] if cfg.layers[i].mixer == "delta" else m["state"])
+    if cfg.loop:
+        mats += cfg.loop[2] * 2 * shapes["loop.in"][0] * shapes["loop.in"][1]
+    return {"weights": mats, "states": states, "cached_rows": cache}
+
+
+def layered_workload(cg, C, args, local):
+    """Prefill and decode throughput of a layer-by-layer model beside the closest attention-only
+    decoder, both on random weights, same batch, prompt and decode lengths.  Prints one JSON line."""
+    import torch
+    layered = importlib.import_module("catgrad-rs_b200.layered")
+    name, B0, S0, T0 = LAYERED_WORKLOADS[args.workload]
+    cfg = getattr(layered, name)
+    B, S, T = args.batch or B0, args.prompt or S0, args.decode or T0
+    heads = max(1, cfg.hidden_size // 128)
+    closest = cg.synth.ModelConfig("llama-equal-size", cfg.hidden_size, max(L.ffn for L in cfg.layers), len(cfg.layer_runs()), heads,
+                                   max(1, heads // 4), cfg.vocab_size, head_dim=128, dtype="bf16")
+    peak, peak_kind = measured_peaks()
+
+    def timed(fn, n):
+        torch.cuda.synchronize()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record()
+        for _ in range(n):
+            fn()
+        e1.record()
+        torch.cuda.synchronize()
+        return e0.elapsed_time(e1) / n
+
+    def measure(c):
+        dec = cg.Decoder(C, c, max_seq=S + T + 1, max_batch=B)
+        dec.load_random(c, 0)
+        prompt = cg.synth.make_tokens(c, B, S, seed=1)
+        ids = C.from_numpy(prompt)
+
+        def job():
+            dec.prefill(ids)
+            dec.decode(T)
+
+        for _ in range(max(args.warmup, 3)):
+            job()
+        sampler = ClockSampler(local)
+        sampler.start()
+        n0 = C.launch_count()
+        job_ms = timed(job, args.steps)
+        launches = C.launch_count() - n0
+        dec.generate(prompt, T)
+        e2e_ms = timed(lambda: dec.generate(prompt, T), args.steps)
+        clocks = sampler.stop()
+        prefill_ms = timed(lambda: dec.prefill(ids), args.steps)
+        dec.prefill(ids)
+        dec.decode(1)
+        decode_ms = timed(lambda: dec.decode(T - 1), 1) / max(T - 1, 1)
+        dec.close()
+        if c is cfg:
+            parts = layered_step_bytes(c, B, S + T / 2)
+        else:
+            parts = {"weights": 2 * dense_params_per_step(c), "kv_cache": B * cg.synth.kv_bytes_per_token(c) * (S + T / 2)}
+        floor = sum(parts.values()) / (peak * 1e9) * 1e3
+        return {"model": c.name, "ms_per_job": job_ms, "tok_s": B * (S + T) / job_ms * 1e3, "e2e_tok_s": B * (S + T) / e2e_ms * 1e3,
+                "prefill_ms": prefill_ms, "prefill_tok_s": B * S / prefill_ms * 1e3, "decode_ms_per_step": decode_ms,
+                "decode_tok_s": B / decode_ms * 1e3, "decode_step_bytes": parts, "decode_step_hbm_floor_ms": floor,
+                "decode_step_frac_of_hbm_roofline": floor / decode_ms, "gpu_launches": launches, "clocks": clocks}
+
+    ours, other = measure(cfg), measure(closest)
+    print(json.dumps({
+        "metric": f"decode+prefill tok/s, {cfg.name}", "value": ours["tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": args.steps,
+        "warmup": max(args.warmup, 3), "ms_per_step": ours["ms_per_job"], "higher_is_better": True, "vs_baseline": None, "dtype": "bf16",
+        "data": "synthetic", "config": {"workload": f"{cfg.name} bf16, batch {B}, prompt {S}, {T} greedy decode steps", "global_batch": B,
+                                        "prompt": S, "decode": T, "layer_runs": len(cfg.layer_runs()), "parallelism": "1 GPU",
+                                        "l2": "inputs larger than L2: a decode step streams every layer run's weights"},
+        "clocks": ours["clocks"], "gpu_launches": ours["gpu_launches"],
+        "e2e": {"value": ours["e2e_tok_s"], "unit": "tok/s", "h2d_bytes_per_step": B * S * 4, "d2h_bytes_per_step": B * (T + 1) * 4},
+        "peak_gbs": peak, "peak_source": peak_kind, "this": ours, "closest_existing": other}))
+
+
 def dense_params_per_step(cfg) -> int:
     """Weights every decode step streams whatever the routing: all dense linear layers and the LM
     head (expert matrices are excluded: how many a step touches depends on the router)."""
@@ -359,9 +457,10 @@ def main():
     ap.add_argument("--steps", type=int, default=5)
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--workload", default="llama1b", choices=sorted(WORKLOADS),
+    ap.add_argument("--workload", default="llama1b", choices=sorted(WORKLOADS) + sorted(LAYERED_WORKLOADS),
                     help="llama1b is the configuration the metric is quoted on; the others are the remaining "
-                         "model shapes at their own batch / prompt / decode sizes")
+                         "model shapes at their own batch / prompt / decode sizes; ralapel-* measure a model built layer by "
+                         "layer beside an attention-only decoder of equal size (one GPU)")
     ap.add_argument("--batch", type=int, default=0)
     ap.add_argument("--prompt", type=int, default=0)
     ap.add_argument("--decode", type=int, default=0)
@@ -385,6 +484,14 @@ def main():
     cg = importlib.import_module("catgrad-rs_b200")
     synth = cg.synth
     import dataclasses
+    if args.workload in LAYERED_WORKLOADS:
+        import torch
+        if not torch.cuda.is_available():
+            raise SystemExit("bench.py needs a CUDA device (there is no CPU fallback)")
+        torch.cuda.set_device(0)
+        stream = torch.cuda.Stream()
+        torch.cuda.set_stream(stream)
+        return layered_workload(cg, cg.CudaBackend(0, cg.PREC_BF16, stream=stream.cuda_stream), args, 0)
     cfg_name, B0, S0, T0 = WORKLOADS[args.workload]
     cfg = getattr(synth, cfg_name)
     args.batch, args.prompt, args.decode = args.batch or B0, args.prompt or S0, args.decode or T0

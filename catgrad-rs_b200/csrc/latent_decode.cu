@@ -120,9 +120,22 @@ constexpr int LD_KT = 64;  // cached rows per tile
 template <int NT>
 __global__ void __launch_bounds__(256) k_latent_dec(LatentArgs a, DecodeScratch sc, int ldk) {
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
-  asm volatile("griddepcontrol.wait;" ::: "memory");
   extern __shared__ __align__(16) uint8_t smem[];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  {
+    // Before the dependency wait: this slice's cached rows are asked into L2.  The position may be a
+    // step old here and the newest row unwritten; a prefetch changes nothing but where bytes lie.
+    const int row = a.rows.tok_row[blockIdx.x];
+    int64_t n = row_pos0(a.rows, row);
+    n = n < 0 ? 0 : n > a.Tmax ? a.Tmax : n;
+    const int64_t per = ((n + sc.splits) / sc.splits + 15) / 16 * 16, lo = blockIdx.z * per;
+    const int64_t hi = min(n, lo + min(per, (int64_t)2 * LD_KT));
+    const char* p = (const char*)((const __nv_bfloat16*)a.cache + (int64_t)a.rows.slot[row] * a.Tmax * a.Lw);
+    const int64_t b_hi = hi * a.Lw * 2;
+    for (int64_t b = lo * a.Lw * 2 + tid * 128; b < b_hi; b += 256 * 128)
+      asm volatile("prefetch.global.L2 [%0];" ::"l"(p + b));
+  }
+  asm volatile("griddepcontrol.wait;" ::: "memory");
   __nv_bfloat16* sq = (__nv_bfloat16*)smem;            // [16][ldk]
   __nv_bfloat16* sk = sq + 16 * ldk;                   // [2][64][ldk]
   __nv_bfloat16* sp = sk + 2 * LD_KT * ldk;            // [16][72]
@@ -139,11 +152,17 @@ __global__ void __launch_bounds__(256) k_latent_dec(LatentArgs a, DecodeScratch 
   const int CH = (int)a.Lw / 8;
   const uint32_t sq_u = (uint32_t)__cvta_generic_to_shared(sq), sk_u = (uint32_t)__cvta_generic_to_shared(sk),
                  sp_u = (uint32_t)__cvta_generic_to_shared(sp);
+  const int row_bytes = (int)a.Lw * 2;
+  // a warp copies whole rows; rows past the slice are zeros
   auto load = [&](int64_t k0, int buf) {
-    for (int i = tid; i < LD_KT * CH; i += 256) {
-      const int r = i / CH, ch = i - r * CH;
-      const bool in = k0 + r < k_hi;
-      cp_async16(sk_u + (uint32_t)((buf * LD_KT + r) * ldk + ch * 8) * 2u, base + (in ? k0 + r : k_lo) * a.Lw + ch * 8, in ? 16 : 0);
+    const char* src = (const char*)(base + k0 * a.Lw) + lane * 16;
+    const int n = (int)min((int64_t)LD_KT, k_hi - k0);
+    uint32_t dst = sk_u + (uint32_t)((buf * LD_KT + warp) * ldk) * 2u + lane * 16;
+#pragma unroll
+    for (int r = warp; r < LD_KT; r += 8, dst += (uint32_t)(8 * ldk) * 2u) {
+      const char* p = src + (r < n ? r : 0) * row_bytes;
+      const int bytes = r < n ? 16 : 0;
+      for (int ch = lane; ch < CH; ch += 32) cp_async16(dst + (ch - lane) * 16, p + (ch - lane) * 16, bytes);
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
@@ -153,10 +172,11 @@ __global__ void __launch_bounds__(256) k_latent_dec(LatentArgs a, DecodeScratch 
   float mrow[2] = {-INFINITY, -INFINITY}, lrow[2] = {0.f, 0.f};
   const int r_in = lane >> 2, cq = (lane & 3) * 2;
   if (k_lo < k_hi) {
-    for (int i = tid; i < 16 * CH; i += 256) {
-      const int r = i / CH, ch = i - r * CH;
+#pragma unroll
+    for (int r = warp; r < 16; r += 8) {
       const bool in = h0 + r < a.H;
-      cp_async16(sq_u + (uint32_t)(r * ldk + ch * 8) * 2u, sc.qa + (m * a.H + (in ? h0 + r : 0)) * a.Lw + ch * 8, in ? 16 : 0);
+      const __nv_bfloat16* p = sc.qa + (m * a.H + (in ? h0 + r : 0)) * a.Lw;
+      for (int ch = lane; ch < CH; ch += 32) cp_async16(sq_u + (uint32_t)(r * ldk + ch * 8) * 2u, p + ch * 8, in ? 16 : 0);
     }
     load(k_lo, 0);
     int buf = 0;
@@ -166,7 +186,8 @@ __global__ void __launch_bounds__(256) k_latent_dec(LatentArgs a, DecodeScratch 
       if (k0 + LD_KT < k_hi) load(k0 + LD_KT, buf ^ 1);
       const uint32_t kb = sk_u + (uint32_t)(buf * LD_KT * ldk) * 2u;
       // scores of this warp's eight keys
-      float s[4] = {0.f, 0.f, 0.f, 0.f};
+      float s[4] = {0.f, 0.f, 0.f, 0.f}, s2[4] = {0.f, 0.f, 0.f, 0.f};  // two chains
+#pragma unroll 4
       for (int kk = 0; kk < (int)a.Lw; kk += 32) {
         uint32_t q0, q1, q2, q3, p0 = 0, p1 = 0, p2 = 0, p3 = 0, b0, b1, b2, b3;
         const bool two = kk + 16 < (int)a.Lw;
@@ -177,8 +198,10 @@ __global__ void __launch_bounds__(256) k_latent_dec(LatentArgs a, DecodeScratch 
         const int kc = kk + 8 * (lane >> 3);
         ldsm_x4(kb + (uint32_t)((warp * 8 + (lane & 7)) * ldk + (two || lane < 16 ? kc : kk)) * 2u, b0, b1, b2, b3);
         mma_bf16(s, q0, q1, q2, q3, b0, b1);
-        if (two) mma_bf16(s, p0, p1, p2, p3, b2, b3);
+        if (two) mma_bf16(s2, p0, p1, p2, p3, b2, b3);
       }
+#pragma unroll
+      for (int e = 0; e < 4; ++e) s[e] += s2[e];
       float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
@@ -239,7 +262,7 @@ __global__ void __launch_bounds__(256) k_latent_dec(LatentArgs a, DecodeScratch 
     }
   }
   // partial outputs and {maximum, sum} per head, over the tiles (each CTA's own are read)
-  const int ldo = a.R + 4;
+  const int ldo = NT * 64 + 4;                         // (columns past R are not read)
   float* so = (float*)sk;                              // [16][ldo]
   float2* sml = (float2*)wm;                           // [16]
   __syncthreads();
@@ -251,7 +274,7 @@ __global__ void __launch_bounds__(256) k_latent_dec(LatentArgs a, DecodeScratch 
       const int col = (warp * NT + j) * 8 + cq;
 #pragma unroll
       for (int y = 0; y < 2; ++y)
-        if (col + y < a.R) so[(r_in + 8 * x) * ldo + col + y] = o[j][2 * x + y];
+        if (col + y < ldo) so[(r_in + 8 * x) * ldo + col + y] = o[j][2 * x + y];
     }
   }
   const int ns = sc.splits;
@@ -279,17 +302,24 @@ __global__ void __launch_bounds__(256) k_latent_dec(LatentArgs a, DecodeScratch 
   }
   __syncthreads();
   const int share = (a.R + ns - 1) / ns, c_lo = split * share, c_hi = min(a.R, c_lo + share);
-  for (int i = tid; i < 16 * share; i += 256) {
-    const int r = i / share, col = c_lo + (i - r * share);
-    if (h0 + r >= a.H || col >= c_hi) continue;
-    const uint32_t at = tc::smem_u32(so + r * ldo + col);
-    float p[MAX_SLICES], v = 0.f;
+  // a warp takes heads `warp` and `warp + 8`: all remote loads of both are issued before the first use
+  for (int col = c_lo + lane; col < c_hi; col += 32) {
+    float p[2][MAX_SLICES];
 #pragma unroll
-    for (int k = 0; k < MAX_SLICES; ++k) p[k] = k < ns ? (ns > 1 ? tc::ld_cluster_f32(at, k) : so[r * ldo + col]) : 0.f;
+    for (int x = 0; x < 2; ++x) {
+      const uint32_t at = tc::smem_u32(so + (warp + 8 * x) * ldo + col);
 #pragma unroll
-    for (int k = 0; k < MAX_SLICES; ++k)
-      if (k < ns) v += p[k] * wt[k * 16 + r];
-    sc.o[(m * a.H + h0 + r) * a.R + col] = v;
+      for (int k = 0; k < MAX_SLICES; ++k) p[x][k] = k < ns ? (ns > 1 ? tc::ld_cluster_f32(at, k) : so[(warp + 8 * x) * ldo + col]) : 0.f;
+    }
+#pragma unroll
+    for (int x = 0; x < 2; ++x) {
+      const int r = warp + 8 * x;
+      float v = 0.f;
+#pragma unroll
+      for (int k = 0; k < MAX_SLICES; ++k)
+        if (k < ns) v += p[x][k] * wt[k * 16 + r];
+      if (h0 + r < a.H) sc.o[(m * a.H + h0 + r) * a.R + col] = v;
+    }
   }
   if (ns > 1) tc::cluster_sync_all();  // nobody leaves while another CTA may read its shared memory
 }

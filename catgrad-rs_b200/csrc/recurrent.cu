@@ -157,10 +157,10 @@ __global__ void __launch_bounds__(128) k_recur_steps(RecurArgs a) {
 }
 
 // ------------------------------------------------------------------ one token per row ----
-// One block per (head, row).  A thread keeps four columns of up to 16 rows of the state in
+// One block per (head, row).  A thread keeps four columns of up to RD_ROWS rows of the state in
 // registers from the load to the store; sums over the key dimension go through shared memory.
-constexpr int RD_ROWS = 16;
-__global__ void __launch_bounds__(256) k_recur_decode(RecurArgs a, GatedNorm n) {
+template <int RD_ROWS>
+__global__ void __launch_bounds__(256, RD_ROWS <= 8 ? 3 : 2) k_recur_decode(RecurArgs a, GatedNorm n) {
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
   __shared__ float sq[128], sk[128], sv[128], so[128], sg[4];
   __shared__ __align__(16) float red[1024];
@@ -392,7 +392,9 @@ bool recur_decode_supported(int dk, int dv) { return dk <= 128 && dv <= 128; }
 
 int k_launch_recur_decode(cg_ctx* c, const RecurArgs& a, const GatedNorm& n) {
   if (a.rows.rows == 0) return CG_OK;
-  CG_CUDA(c, launch_kernel(c, k_recur_decode, dim3((unsigned)a.H, (unsigned)a.rows.rows), dim3(256), 0, 1, a, n));
+  const int rpp = 256 / (a.dvs / 4);  // state rows per pass
+  auto kernel = (a.dk + rpp - 1) / rpp <= 8 ? k_recur_decode<8> : k_recur_decode<16>;
+  CG_CUDA(c, launch_kernel(c, kernel, dim3((unsigned)a.H, (unsigned)a.rows.rows), dim3(256), 0, 1, a, n));
   CG_LAUNCHED(c);
   return a.delta ? CG_OK : k_launch_gated_norm(c, n);
 }

@@ -1,4 +1,5 @@
 """Host-side logic of bench.py that needs no GPU: how a fixed job is spread over several GPUs."""
+import dataclasses
 import importlib
 import os
 import sys
@@ -36,3 +37,12 @@ def test_workloads_name_known_configurations():
         assert batch >= 1 and prompt >= 1 and decode >= 1
         assert cfg.num_hidden_layers >= 1 and cfg.vocab_size > 0
         assert bench.dense_params_per_step(cfg) > 0
+
+
+def test_layered_workloads_count_looped_layers():
+    layered = importlib.import_module("catgrad-rs_b200.layered")
+    for name, (cfg_name, batch, prompt, decode) in bench.LAYERED_WORKLOADS.items():
+        cfg = getattr(layered, cfg_name)
+        once = bench.layered_step_bytes(dataclasses.replace(cfg, loop=None), batch, prompt)
+        looped = bench.layered_step_bytes(cfg, batch, prompt)
+        assert all(looped[k] > once[k] > 0 for k in once)
