@@ -139,12 +139,12 @@ class LayeredConfig:
 def bench_shape(name: str, width: int, ff: int, vocab: int) -> LayeredConfig:
     """A Ralapel-shaped model at a real model's widths, for measurements: per mixer the head sizes
     larger models use (128 x 128 delta states, 128 x 64 Mamba-2 states with one group, latent rows
-    of 512 + 32), a loop over two of the layers."""
+    of 512 + 32), a loop over three of the layers."""
     ssd = LayerSpec("mamba2", {"heads": 2 * width // 64, "groups": 1, "state": 128, "vdim": 64, "norm_groups": 1, "conv": 4})
     lat = LayerSpec("latent_attention", {"heads": width // 128, "dim": 96, "rot_dim": 32, "vdim": 128, "kv_rank": 512, "scale": 128 ** -0.5,
                                          "rot": {"base": 10000.0, "dims": 32}}, ff)
     dlt = LayerSpec("delta", {"heads": width // 64, "kv_heads": width // 128, "dim": 128, "vdim": 128, "conv": 4}, ff)
-    return LayeredConfig(name, width, vocab, [ssd, lat, dlt, ssd, lat, dlt, ssd, dlt], (1, 3, 3))
+    return LayeredConfig(name, width, vocab, [ssd, lat, dlt, ssd, lat, dlt, ssd, dlt], (1, 4, 2))
 
 
 RALAPEL_W1024 = bench_shape("ralapel-w1024-shape", 1024, 4096, 32000)

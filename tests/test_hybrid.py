@@ -122,18 +122,18 @@ def everything(dec, seq, cut=None):
     return np.concatenate(out)
 
 
-MIXED = model([ssd(), with_ff(latent()), delta(), with_ff(delta(heads=2, kv_heads=1, dim=24, vdim=16, conv=2), 40)],
-              loop={"start": 1, "stop": 3, "times": 3})
+MIXED = model([delta(heads=2, kv_heads=1, dim=24, vdim=16, conv=2), ssd(), with_ff(latent()), with_ff(delta(), 40), latent(heads=2, dim=16)],
+              loop={"start": 2, "stop": 4, "times": 2})
 
 
 # ---------------------------------------------------------------------------- configuration (CPU)
 
 def test_config_reader_and_shapes():
     cfg = cg.registry.config_from_json(MIXED)
-    assert cfg.layer_runs() == [i for i, _ in oracle.layer_runs(MIXED)] == [0, 1, 2, 1, 2, 1, 2, 3]
-    assert cfg.rms_norm_eps == 1e-5 and cfg.layers[1].ffn == 88 and cfg.layers[0].ffn == 0
+    assert cfg.layer_runs() == [i for i, _ in oracle.layer_runs(MIXED)] == [0, 1, 2, 3, 2, 3, 4]
+    assert cfg.rms_norm_eps == 1e-5 and cfg.layers[2].ffn == 88 and cfg.layers[0].ffn == 0
     s = cfg.param_shapes()
-    assert s["l0.mix.in"] == (4 * 24 * 2 + 2 * 2 * 16 + 4, 72) and s["l1.mix.dkv"] == (48, 72) and s["loop.in"] == (72, 144)
+    assert s["l1.mix.in"] == (4 * 24 * 2 + 2 * 2 * 16 + 4, 72) and s["l2.mix.dkv"] == (48, 72) and s["loop.in"] == (72, 144)
     plain = cg.registry.config_from_json(model([delta()]))
     assert plain.loop is None and "loop.in" not in plain.param_shapes()
     with pytest.raises(ValueError):
@@ -185,6 +185,10 @@ ALONE = {
     "ssd_groups": [ssd(heads=6, groups=3, state=12, vdim=20, norm_groups=6, conv=5)],
     "ssd_128": [ssd(heads=4, groups=1, state=128, vdim=64, norm_groups=1)],
     "ssd_no_conv": [ssd(heads=2, groups=2, state=32, vdim=48, norm_groups=4, conv=1)],
+    # beyond what the tensor-core kernels take
+    "latent_rank_600": [latent(heads=2, dim=16, rot_dim=8, vdim=24, kv_rank=600)],
+    "delta_wide": [delta(heads=2, kv_heads=1, dim=136, vdim=144, conv=3)],
+    "ssd_wide": [ssd(heads=2, groups=1, state=144, vdim=136, norm_groups=2, conv=6)],
     "feed_forward": [with_ff(ssd(heads=1, groups=1, state=8, vdim=8, norm_groups=1), 44)],
     "narrow": [with_ff(latent(heads=1, dim=6, rot_dim=2, vdim=5, kv_rank=11), 13), delta(heads=3, kv_heads=1, dim=5, vdim=7)],
 }
@@ -475,7 +479,7 @@ def test_bad_input_is_an_error_not_a_fault(backends):
         dec.run([(s, [1]), (s, [2])])
     dec.close()
     bad = dict(W)
-    del bad["l2.mix.k.conv"]
+    del bad["l3.mix.k.conv"]
     with pytest.raises(cg.BackendPanic):
         decoder(B, MIXED, bad)
 
