@@ -1,6 +1,6 @@
 """A plain, slow restatement of the Ralapel equations in numpy float64, one function per mechanism.
 
-It is the checker of tests/test_hybrid.py and shares no code with the library: sequences are run
+tests/test_hybrid.py compares the library with it.  It shares no code with the library: sequences are run
 one at a time, recurrences one token at a time, attention one query at a time, and nothing is
 fused, chunked, absorbed or cached.  A checkpoint is a dict name -> float array, a configuration
 is the parsed config.json.
