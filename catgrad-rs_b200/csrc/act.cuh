@@ -21,4 +21,21 @@ __device__ __forceinline__ float gelu_fast(float x) {
   return 0.5f * x * (2.f * sigmoid_fast(2.f * c * (x + 0.044715f * x * x * x)));
 }
 
+// What a feed-forward applies to its projections (cg_act, include/catgrad_cuda.h).  Two projections:
+// ACT_SILU and ACT_GELU gate the second one, ACT_BOUNDED is min(g, limit) sigmoid(1.702 g) (u + 1) with
+// u kept within +-limit.  One projection: ACT_RELU2 is the square of relu.
+enum Act : int { ACT_SILU = 0, ACT_GELU = 1, ACT_BOUNDED = 2, ACT_RELU2 = 3 };
+__device__ __forceinline__ float bounded_glu(float g, float u, float limit) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return g * sigmoid_f(1.702f * g) * (u + 1.f);
+}
+__device__ __forceinline__ float glu_f(int act, float limit, float g, float u) {
+  return act == ACT_SILU ? silu_f(g) * u : act == ACT_GELU ? gelu_f(g) * u : bounded_glu(g, u, limit);
+}
+__device__ __forceinline__ float relu2_f(float x) {
+  x = fmaxf(x, 0.f);
+  return x * x;
+}
+
 }  // namespace cg

@@ -23,6 +23,13 @@ namespace {
 
 __device__ __forceinline__ float tanh_sig(float x) { return 2.f / (1.f + __expf(-2.f * x)) - 1.f; }
 
+// 1 / (l + exp(sink - m)): l sums exp(score - m), the sink is one more term without a value
+__device__ __forceinline__ float sink_scale(float m, float l, float sink) {
+  const float top = fmaxf(m, sink);
+  const float f = expf(m - top);
+  return f / (l * f + expf(sink - top));
+}
+
 // ------------------------------------------------------------------ prefill ----------
 template <int D, int BQ, int NBUF>
 __global__ void __launch_bounds__(BQ * 2, D <= 64 ? 2 : 1) k_attn_prefill(AttnArgs a, float scale) {
@@ -36,10 +43,19 @@ __global__ void __launch_bounds__(BQ * 2, D <= 64 ? 2 : 1) k_attn_prefill(AttnAr
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int qt = (int)gridDim.x - 1 - (int)blockIdx.x, h = blockIdx.y;
-  const int64_t b = blockIdx.z;
+  // the row: its first packed token, its length, the position of its first token, its place in the cache
+  int64_t b = blockIdx.z, tok0 = b * a.S, len = a.S, start_pos = a.pos0;
+  if (a.rows.rows > 0) {
+    const int row = (int)b;
+    tok0 = a.rows.start[row];
+    len = a.rows.start[row + 1] - tok0;
+    start_pos = row_pos0(a.rows, row);
+    b = a.rows.slot[row];
+  }
   const int kvh = h / (a.nh / a.nkv);
   const int64_t q0 = (int64_t)qt * BQ;
-  const __nv_bfloat16* qbase = a.q + (b * a.S) * (int64_t)a.nh * D + (int64_t)h * D;
+  if (q0 >= len) return;  // (rows of unequal length)
+  const __nv_bfloat16* qbase = a.q + tok0 * (int64_t)a.nh * D + (int64_t)h * D;
   const int64_t ldk = a.kv_ld > 0 ? a.kv_ld : D;  // from one key to the next
   const int64_t kv0 = a.kv_ld > 0 ? b * a.Tmax * a.kv_ld + (int64_t)kvh * D : ((b * a.nkv + kvh) * a.Tmax) * (int64_t)D;
   const __nv_bfloat16* kbase = a.k_cache + kv0;
@@ -50,7 +66,7 @@ __global__ void __launch_bounds__(BQ * 2, D <= 64 ? 2 : 1) k_attn_prefill(AttnAr
   for (int i = tid; i < BQ * CH; i += NT) {
     const int r = i / CH, ch = i - r * CH;
     uint4 v = make_uint4(0, 0, 0, 0);
-    if (q0 + r < a.S) v = *(const uint4*)(qbase + (q0 + r) * (int64_t)a.nh * D + ch * 8);
+    if (q0 + r < len) v = *(const uint4*)(qbase + (q0 + r) * (int64_t)a.nh * D + ch * 8);
     *(uint4*)(sq + r * LD + ch * 8) = v;
   }
 
@@ -60,11 +76,11 @@ __global__ void __launch_bounds__(BQ * 2, D <= 64 ? 2 : 1) k_attn_prefill(AttnAr
   float mrow[2] = {-INFINITY, -INFINITY}, lrow[2] = {0.f, 0.f};
 
   const int r_in = lane >> 2, cq = (lane & 3) * 2;
-  const int64_t qpos[2] = {a.pos0 + q0 + warp * 16 + r_in, a.pos0 + q0 + warp * 16 + r_in + 8};
-  const int64_t kv_len = a.pos0 + a.S;
-  const int64_t last_q = a.pos0 + std::min<int64_t>(a.S, q0 + BQ) - 1;  // last query position of this tile
+  const int64_t qpos[2] = {start_pos + q0 + warp * 16 + r_in, start_pos + q0 + warp * 16 + r_in + 8};
+  const int64_t kv_len = start_pos + len;
+  const int64_t last_q = start_pos + std::min<int64_t>(len, q0 + BQ) - 1;  // last query position of this tile
   int64_t first_k = 0;
-  if (a.window > 0) first_k = std::max<int64_t>(0, a.pos0 + q0 - a.window + 1);
+  if (a.window > 0) first_k = std::max<int64_t>(0, start_pos + q0 - a.window + 1);
   const int64_t kt0 = first_k / BKV, kt1 = last_q / BKV;  // inclusive key tile range
 
   const uint32_t sq_u = (uint32_t)__cvta_generic_to_shared(sq);
@@ -197,9 +213,10 @@ __global__ void __launch_bounds__(BQ * 2, D <= 64 ? 2 : 1) k_attn_prefill(AttnAr
 #pragma unroll
   for (int r = 0; r < 2; ++r) {
     const int64_t qi = q0 + warp * 16 + r_in + 8 * r;
-    if (qi >= a.S) continue;
-    const float inv = lrow[r] > 0.f ? 1.f / lrow[r] : 0.f;
-    __nv_bfloat16* dst = a.out + (b * a.S + qi) * (int64_t)a.nh * D + (int64_t)h * D;
+    if (qi >= len) continue;
+    float inv = lrow[r] > 0.f ? 1.f / lrow[r] : 0.f;
+    if (a.sink) inv = sink_scale(mrow[r], lrow[r], a.sink[h]);
+    __nv_bfloat16* dst = a.out + (tok0 + qi) * (int64_t)a.nh * D + (int64_t)h * D;
 #pragma unroll
     for (int j = 0; j < D / 8; ++j) {
       __nv_bfloat162 v = __floats2bfloat162_rn(o[j][2 * r] * inv, o[j][2 * r + 1] * inv);
@@ -217,7 +234,7 @@ int launch_prefill(cg_ctx* c, const AttnArgs& a) {
     CG_CUDA(c, cudaFuncSetAttribute(k_attn_prefill<D, BQ, NBUF>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     configured = true;
   }
-  dim3 grid((unsigned)((a.S + BQ - 1) / BQ), (unsigned)a.nh, (unsigned)a.B);
+  dim3 grid((unsigned)((a.S + BQ - 1) / BQ), (unsigned)a.nh, (unsigned)(a.rows.rows ? a.rows.rows : a.B));
   const float scale = a.scale > 0.f ? a.scale : 1.0f / sqrtf((float)D);
   CG_CUDA(c, launch_kernel(c, k_attn_prefill<D, BQ, NBUF>, grid, dim3(BQ * 2), smem, 1, a, scale));
   CG_LAUNCHED(c);
@@ -227,7 +244,7 @@ int launch_prefill(cg_ctx* c, const AttnArgs& a) {
 int check(cg_ctx* c, const AttnArgs& a) {
   if (a.nkv <= 0 || a.nh % a.nkv) return fail(c, CG_ERR_SHAPE, "attention: heads must be a multiple of kv heads");
   if (a.d != 64 && a.d != 128 && a.d != 256) return fail(c, CG_ERR_UNSUPPORTED, "attention: head_dim must be 64, 128 or 256");
-  if (a.pos0 + a.S > a.Tmax) return fail(c, CG_ERR_SHAPE, "attention: KV cache capacity exceeded");
+  if (!a.rows.rows && a.pos0 + a.S > a.Tmax) return fail(c, CG_ERR_SHAPE, "attention: KV cache capacity exceeded");
   if (a.B > 65535 || a.nh > 65535) return fail(c, CG_ERR_UNSUPPORTED, "attention: too many rows or heads");
   return CG_OK;
 }

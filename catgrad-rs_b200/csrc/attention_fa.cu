@@ -1,5 +1,5 @@
 // attention_fa.cu — causal prefill attention on the Blackwell tensor cores (tcgen05 + TMEM),
-// for head sizes 64 and 128 without soft-cap or window.
+// for head sizes 64 and 128 without soft-cap.
 //
 // Same mathematics as attention.cu (catgrad-llm/src/models/llama.rs:97-108 after repeat_kv,
 // catgrad-llm/src/helpers.rs:147-161, as an online-softmax pass over key tiles); what changes
@@ -39,6 +39,9 @@ struct FaArgs {
   int nh, nkv;
   int token_major;     // keys and values lie token after token, the heads side by side
   float scale_log2e;   // score factor (1 / sqrt(D)) * log2(e)
+  int64_t window;      // 0 = none
+  const float* sink;   // [nh] or null
+  RowsDev rows;        // rows of unequal length (rows.rows > 0)
   int32_t* err;
 };
 
@@ -109,11 +112,22 @@ k_attn_fa(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUt
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int qt = (int)gridDim.x - 1 - (int)blockIdx.x, h = blockIdx.y;  // longest tiles first
-  const int64_t b = blockIdx.z;
+  // the row: its first packed token, its length, the position of its first token, its place in the cache
+  int64_t b = blockIdx.z, tok0 = b * p.S, len = p.S, start_pos = p.pos0;
+  if (p.rows.rows > 0) {
+    const int row = (int)b;  // (the row tables are written in plain stream order before a prompt's kernels)
+    tok0 = p.rows.start[row];
+    len = p.rows.start[row + 1] - tok0;
+    start_pos = row_pos0(p.rows, row);
+    b = p.rows.slot[row];
+  }
   const int kvh = h / (p.nh / p.nkv);
   const int64_t q0 = (int64_t)qt * FA_BQ;
-  const int64_t last_q = p.pos0 + std::min<int64_t>(p.S, q0 + FA_BQ) - 1;
-  const int nt = (int)(last_q / FA_BK) + 1;  // key tiles 0 .. nt-1
+  if (q0 >= len) return;  // uniform over the CTA, before anything is allocated
+  const int64_t last_q = start_pos + std::min<int64_t>(len, q0 + FA_BQ) - 1;
+  // key tiles j0 .. j0 + nt - 1
+  const int j0 = p.window > 0 ? (int)(std::max<int64_t>(0, start_pos + q0 - p.window + 1) / FA_BK) : 0;
+  const int nt = (int)(last_q / FA_BK) + 1 - j0;
 
   if (tid == 0) {
     mbar_init(b_q_full, 1);
@@ -149,7 +163,7 @@ k_attn_fa(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUt
 
   if (warp == 0) {
     if (lane == 0) {
-      const int qrow = (int)(b * p.S + q0);
+      const int qrow = (int)(tok0 + q0);
       mbar_expect_tx(b_q_full, Q_BYTES);
       for (int s = 0; s < SUB; ++s) tma_load_2d(sq + s * BOX, &map_q, h * D + s * 64, qrow, b_q_full);
       const int64_t kvrow0 = p.token_major ? b * p.Tmax : (b * p.nkv + kvh) * p.Tmax;
@@ -157,7 +171,7 @@ k_attn_fa(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUt
       bool ok = true;
       for (int j = 0; j < nt && ok; ++j) {
         const uint32_t buf = (uint32_t)j & 1u, ph = ((uint32_t)j >> 1) & 1u;
-        const int row = (int)(kvrow0 + (int64_t)j * FA_BK);
+        const int row = (int)(kvrow0 + (int64_t)(j0 + j) * FA_BK);
         if (j >= 2) {
           ok = mbar_wait(b_k_empty + 8 * buf, ph ^ 1u, cta_abort, p.err);
           if (!ok) break;
@@ -223,7 +237,7 @@ k_attn_fa(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUt
     const int r = q * 32 + lane;  // query row of this thread = TMEM lane
     const uint32_t lane_base = tmem_base + ((uint32_t)(q * 32) << 16);
     const int64_t qi = q0 + r;
-    const int64_t qpos = p.pos0 + qi;
+    const int64_t qpos = start_pos + qi;
     float o[D];
 #pragma unroll
     for (int i = 0; i < D; ++i) o[i] = 0.f;
@@ -234,11 +248,17 @@ k_attn_fa(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUt
       ok = mbar_wait(b_s_full + 8 * buf, ph, cta_abort, p.err);
       if (!ok) break;
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-      const int k0 = j * FA_BK;
-      // a key column c of this tile is visible to this row iff c <= lim (causal mask)
+      const int k0 = (j0 + j) * FA_BK;
+      // a key column c of this tile is visible to this row iff low <= c <= lim (window and causal
+      // mask), tested as c - low <= lim - low without signs
       const int64_t lim64 = qpos - k0;
       const int lim = lim64 > FA_BK ? FA_BK : (lim64 < -1 ? -1 : (int)lim64);
-      const bool diag = (int64_t)k0 + FA_BK - 1 > p.pos0 + q0;  // uniform: some key may be masked for some row
+      const int64_t low64 = p.window > 0 ? lim64 - p.window + 1 : 0;
+      int low = low64 < 0 ? 0 : (low64 > 2 * FA_BK ? 2 * FA_BK : (int)low64);
+      if (lim < low) low = 2 * FA_BK;  // nothing in this tile: no column reaches it
+      const uint32_t span = lim < low ? 0u : (uint32_t)(lim - low);
+      // uniform: some key may be masked for some row
+      const bool diag = (int64_t)k0 + FA_BK - 1 > start_pos + q0 || (p.window > 0 && k0 <= last_q - p.window);
       const uint32_t s_addr = lane_base + buf * S_COLS;
       constexpr int NCH = FA_BK / 32;
       uint32_t va[32], vb[32];
@@ -256,9 +276,9 @@ k_attn_fa(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUt
 #pragma unroll
           for (int i = 0; i < 32; ++i) mx = fmaxf(mx, __uint_as_float(cur[i]));
         } else {
-          const int rel = lim - c * 32;
+          const int rel = c * 32 - low;
 #pragma unroll
-          for (int i = 0; i < 32; ++i) mx = i <= rel ? fmaxf(mx, __uint_as_float(cur[i])) : mx;
+          for (int i = 0; i < 32; ++i) mx = (uint32_t)(i + rel) <= span ? fmaxf(mx, __uint_as_float(cur[i])) : mx;
         }
         if (c + 1 < NCH) asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
       }
@@ -280,15 +300,15 @@ k_attn_fa(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUt
         uint32_t* cur = (c & 1) ? vb : va;
         uint32_t* nxt = (c & 1) ? va : vb;
         if (c + 1 < NCH) tmem_ld32(s_addr + (uint32_t)(c + 1) * 32u, nxt);
-        const int rel = lim - c * 32;
+        const int rel = c * 32 - low;
         uint32_t pk[16];
 #pragma unroll
         for (int i = 0; i < 32; i += 2) {
           float e0 = fast_exp2(fmaf(__uint_as_float(cur[i]), p.scale_log2e, -mc));
           float e1 = fast_exp2(fmaf(__uint_as_float(cur[i + 1]), p.scale_log2e, -mc));
           if (diag) {
-            e0 = i <= rel ? e0 : 0.f;
-            e1 = i + 1 <= rel ? e1 : 0.f;
+            e0 = (uint32_t)(i + rel) <= span ? e0 : 0.f;
+            e1 = (uint32_t)(i + 1 + rel) <= span ? e1 : 0.f;
           }
           ls += e0 + e1;
           const __nv_bfloat162 pr = __floats2bfloat162_rn(e0, e1);
@@ -330,9 +350,15 @@ k_attn_fa(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUt
       asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
       asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(b_o_empty) : "memory");
     }
-    if (ok && qi < p.S) {
-      const float inv = l > 0.f ? 1.f / l : 0.f;
-      __nv_bfloat16* dst = p.out + (b * p.S + qi) * (int64_t)p.nh * D + (int64_t)h * D;
+    if (ok && qi < len) {
+      float inv = l > 0.f ? 1.f / l : 0.f;
+      if (p.sink) {
+        // one more term of the denominator, without a value
+        const float mc = m * p.scale_log2e, sk = p.sink[h] * 1.4426950408889634f, top = fmaxf(mc, sk);
+        const float f = fast_exp2(mc - top);
+        inv = f / (l * f + fast_exp2(sk - top));
+      }
+      __nv_bfloat16* dst = p.out + (tok0 + qi) * (int64_t)p.nh * D + (int64_t)h * D;
 #pragma unroll
       for (int c0 = 0; c0 < D; c0 += 8) {
         uint32_t w[4];
@@ -365,7 +391,7 @@ int launch_fa(cg_ctx* c, const AttnArgs& a) {
     configured = true;
   }
   CUtensorMap mq, mk, mv;
-  CG_TRY(make_map(c, &mq, a.q, a.B * a.S, (int64_t)a.nh * D, (int64_t)a.nh * D, 128));
+  CG_TRY(make_map(c, &mq, a.q, a.rows.rows ? a.rows.M : a.B * a.S, (int64_t)a.nh * D, (int64_t)a.nh * D, 128));
   const bool tm = a.kv_ld > 0;
   const int64_t kv_rows = tm ? a.B * a.Tmax : a.B * a.nkv * a.Tmax, kv_cols = tm ? (int64_t)a.nkv * D : D, kv_ld = tm ? a.kv_ld : D;
   CG_TRY(make_map(c, &mk, a.k_cache, kv_rows, kv_cols, kv_ld, FA_BK));
@@ -376,8 +402,11 @@ int launch_fa(cg_ctx* c, const AttnArgs& a) {
   p.nh = a.nh; p.nkv = a.nkv;
   p.token_major = tm ? 1 : 0;
   p.scale_log2e = 1.4426950408889634f * (a.scale > 0.f ? a.scale : 1.f / sqrtf((float)D));
+  p.window = a.window > 0 ? a.window : 0;
+  p.sink = a.sink;
+  p.rows = a.rows;
   p.err = c->core->dev_err;
-  dim3 grid((unsigned)((a.S + FA_BQ - 1) / FA_BQ), (unsigned)a.nh, (unsigned)a.B);
+  dim3 grid((unsigned)((a.S + FA_BQ - 1) / FA_BQ), (unsigned)a.nh, (unsigned)(a.rows.rows ? a.rows.rows : a.B));
   CG_CUDA(c, launch_kernel(c, k_attn_fa<D, FA_BK>, grid, dim3(192), smem, 1, mq, mk, mv, p));
   CG_LAUNCHED(c);
   return CG_OK;
@@ -386,8 +415,8 @@ int launch_fa(cg_ctx* c, const AttnArgs& a) {
 }  // namespace
 
 bool attn_fa_supported(const AttnArgs& a) {
-  return (a.d == 64 || a.d == 128) && a.window <= 0 && a.softcap <= 0.f && !a.pos_dev && a.S >= 64 &&
-         a.B * a.S < 2147483647ll && a.B * a.nkv * a.Tmax < 2147483647ll && ((uintptr_t)a.q % 16) == 0 &&
+  return (a.d == 64 || a.d == 128) && a.softcap <= 0.f && !a.pos_dev && a.S >= 64 &&
+         (a.rows.rows ? a.rows.M : a.B * a.S) < 2147483647ll && a.B * a.nkv * a.Tmax < 2147483647ll && ((uintptr_t)a.q % 16) == 0 &&
          ((uintptr_t)a.k_cache % 16) == 0 && ((uintptr_t)a.v_cache % 16) == 0 && a.kv_ld % 8 == 0;
 }
 

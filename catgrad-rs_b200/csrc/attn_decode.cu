@@ -32,6 +32,7 @@ namespace {
 constexpr int MAX_REP = ATTN_MAX_REP;
 
 // one CTA per item; the slices of one (row, kv head) are one thread-block cluster
+template <bool ROWS>
 struct KernelEnv {
   __device__ __forceinline__ int tid() const { return threadIdx.x; }
   __device__ __forceinline__ void sync_cta() const { __syncthreads(); }
@@ -45,17 +46,19 @@ struct KernelEnv {
   __device__ __forceinline__ float* landing() const { return land; }
   // the projected row, and the position when it lives on the device, belong to the stream order
   const AttnDecArgs* args;
+  static constexpr bool kRows = ROWS;
   __device__ __forceinline__ int64_t settle(int64_t) const {
     asm volatile("griddepcontrol.wait;" ::: "memory");
+    if constexpr (ROWS) return args->rows.pos0[blockIdx.y] + *(const volatile int64_t*)args->rows.step;
     return args->pos_dev ? *(const volatile int64_t*)args->pos_dev : args->pos0;
   }
 };
 
-template <int D>
+template <int D, bool ROWS>
 __global__ void __launch_bounds__(128) k_attn_dec(AttnDecArgs a, float scale) {
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
   extern __shared__ __align__(16) uint8_t smem[];
-  KernelEnv env;
+  KernelEnv<ROWS> env;
   env.args = &a;
   env.land = (float*)(smem + attn_dec_smem_bytes<D>());
   // Before the dependency wait: the first tiles of cached keys and values can be on the way
@@ -64,12 +67,14 @@ __global__ void __launch_bounds__(128) k_attn_dec(AttnDecArgs a, float scale) {
   // own dependency wait) stores a value v only after every kernel that wrote cache rows below v
   // has completed, so whatever value is visible here, the rows below it are complete.  The value
   // may be a step old; it is re-read after the wait and a changed value repeats the request.
+  // (Row tables are copied in plain stream order before any kernel that reads them.)
   int64_t pos_early = a.pos_dev ? *(const volatile int64_t*)a.pos_dev : a.pos0;
+  if constexpr (ROWS) pos_early = a.rows.pos0[blockIdx.y] + *(const volatile int64_t*)a.rows.step;
   pos_early = pos_early < 0 ? 0 : (pos_early >= a.Tmax ? a.Tmax - 1 : pos_early);
   attn_dec_item<D>(a, scale, (int)blockIdx.x, (int64_t)blockIdx.y, (int)blockIdx.z, pos_early, smem, env);
 }
 
-template <int D>
+template <int D, bool ROWS>
 int launch(cg_ctx* c, const AttnDecArgs& args) {
   constexpr int LD = D + 8;
   constexpr int KT = D > 128 ? 16 : 32;
@@ -88,18 +93,19 @@ int launch(cg_ctx* c, const AttnDecArgs& args) {
   static PerDeviceFlag configured_on;
   bool& configured = configured_on.at(c->core->device);
   if (!configured && attn_dec_smem_bytes<D>() + attn_dec_landing_bytes() > 48 * 1024) {
-    CG_CUDA(c, cudaFuncSetAttribute(k_attn_dec<D>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    CG_CUDA(c, cudaFuncSetAttribute(k_attn_dec<D, ROWS>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                     (int)(attn_dec_smem_bytes<D>() + attn_dec_landing_bytes())));
     configured = true;
   }
   static PerDeviceFlag wide_on;
   bool& wide = wide_on.at(c->core->device);
   if (!wide && a.splits > 8) {
-    CG_CUDA(c, cudaFuncSetAttribute(k_attn_dec<D>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1));
+    CG_CUDA(c, cudaFuncSetAttribute(k_attn_dec<D, ROWS>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1));
     wide = true;
   }
   dim3 grid((unsigned)a.nkv, (unsigned)a.B, (unsigned)a.splits);
-  CG_CUDA(c, launch_kernel(c, k_attn_dec<D>, grid, dim3(128), smem, a.splits, a, 1.0f / sqrtf((float)D)));
+  const float scale = a.scale > 0.f ? a.scale : 1.0f / sqrtf((float)D);
+  CG_CUDA(c, launch_kernel(c, k_attn_dec<D, ROWS>, grid, dim3(128), smem, a.splits, a, scale));
   CG_LAUNCHED(c);
   return CG_OK;
 }
@@ -129,12 +135,19 @@ int k_launch_attn_dec(cg_ctx* c, const AttnDecArgs& a) {
     return fail(c, CG_ERR_UNSUPPORTED, "attention decode: query heads per kv head must be 1..8");
   if (a.d != 64 && a.d != 128 && a.d != 256) return fail(c, CG_ERR_UNSUPPORTED, "attention: head_dim must be 64, 128 or 256");
   if (a.B > 65535) return fail(c, CG_ERR_UNSUPPORTED, "attention: too many rows");
-  if (!a.pos_dev && a.pos0 >= a.Tmax) return fail(c, CG_ERR_SHAPE, "attention: KV cache capacity exceeded");
+  if (!a.rows.rows && !a.pos_dev && a.pos0 >= a.Tmax) return fail(c, CG_ERR_SHAPE, "attention: KV cache capacity exceeded");
   if (a.B == 0) return CG_OK;
+  if (a.rows.rows) {
+    switch (a.d) {
+      case 64: return launch<64, true>(c, a);
+      case 128: return launch<128, true>(c, a);
+      default: return launch<256, true>(c, a);
+    }
+  }
   switch (a.d) {
-    case 64: return launch<64>(c, a);
-    case 128: return launch<128>(c, a);
-    default: return launch<256>(c, a);
+    case 64: return launch<64, false>(c, a);
+    case 128: return launch<128, false>(c, a);
+    default: return launch<256, false>(c, a);
   }
 }
 

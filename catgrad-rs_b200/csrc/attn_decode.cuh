@@ -13,6 +13,8 @@
 //                    attn_dec_landing_bytes(), shared memory that nothing else uses) of the CTA that
 //                    finishes them, so one group barrier suffices and nobody waits before leaving;
 //                    otherwise the finishing CTA reads the partials where they lie (two barriers)
+//   kRows            the item is a row of AttnDecArgs::rows: its own slot and position, neighbouring pairs
+//                    rotated, norms over all heads at once, a sink
 //   settle(pos)      called once the first K/V tiles have been requested with a position that may
 //                    be one step old: waits for whatever the caller's inputs depend on and returns
 //                    the position to use (cached keys never change, so an early request is either
@@ -71,8 +73,10 @@ __device__ __forceinline__ void attn_dec_item(const AttnDecArgs& a, float scale,
   const int half = D / 2;
   // pos: position of the new token = number of cached keys.  The projected row is read with
   // L2 loads: in the resident kernel another CTA wrote it earlier in the same launch.
-  __nv_bfloat16* kbase = a.k_cache + ((b * a.nkv + kvh) * a.Tmax) * (int64_t)D;
-  __nv_bfloat16* vbase = a.v_cache + ((b * a.nkv + kvh) * a.Tmax) * (int64_t)D;
+  int64_t place = b;
+  if constexpr (Env::kRows) place = a.rows.slot[b];
+  __nv_bfloat16* kbase = a.k_cache + ((place * a.nkv + kvh) * a.Tmax) * (int64_t)D;
+  __nv_bfloat16* vbase = a.v_cache + ((place * a.nkv + kvh) * a.Tmax) * (int64_t)D;
 
   // this CTA's slice of the cached keys [lo, pos)
   int64_t pos = pos_early, t0 = 0, t1 = 0;
@@ -125,6 +129,74 @@ __device__ __forceinline__ void attn_dec_item(const AttnDecArgs& a, float scale,
   const float* qsrc = row + (int64_t)kvh * rep * D;
   const float* ksrc = row + ((int64_t)a.nh + kvh) * D;
   const float* vsrc = row + ((int64_t)a.nh + a.nkv + kvh) * D;
+  if constexpr (Env::kRows) {
+    if (a.q_gamma) {
+      // norms over all query heads and over all key heads: hsq[0], hsq[1] receive the factors
+      float ss[2] = {0.f, 0.f};
+#pragma unroll
+      for (int part = 0; part < 2; ++part) {
+        const float4* src = (const float4*)(row + (part ? (int64_t)a.nh * D : 0));
+        const int n = (part ? a.nkv : a.nh) * D / 4;
+#pragma unroll 4
+        for (int i = tid; i < n; i += 128) {
+          const float4 v = __ldcg(src + i);
+          ss[part] += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+        }
+#pragma unroll
+        for (int o = 16; o; o >>= 1) ss[part] += __shfl_xor_sync(0xffffffffu, ss[part], o);
+        if (lane == 0) red_m[part * 4 + warp] = ss[part];
+      }
+      env.sync_cta();
+      if (tid < 2) {
+        const float* r = red_m + tid * 4;
+        hsq[tid] = 1.f / sqrtf(((r[0] + r[1]) + (r[2] + r[3])) / (float)((tid ? a.nkv : a.nh) * a.norm_dim) + a.norm_eps);
+      }
+      env.sync_cta();
+    }
+    // neighbouring components (2 j, 2 j + 1) of the first rot_dims turn together
+    const int rh = a.rot_dims / 2;
+    const float* ct = a.cos_t + pos * rh;
+    const float* st = a.sin_t + pos * rh;
+    for (int i = tid; i < 16 * half; i += 128) {
+      const int h = i / half, j = i - h * half;
+      float x1 = 0.f, x2 = 0.f;
+      if (h < rep) {
+        const float2 x = __ldcg((const float2*)(qsrc + h * D) + j);
+        x1 = x.x; x2 = x.y;
+        if (a.q_gamma) {
+          const float2 g = *((const float2*)(a.q_gamma + (kvh * rep + h) * D) + j);
+          x1 *= hsq[0] * g.x; x2 *= hsq[0] * g.y;
+        }
+        if (j < rh) {
+          const float cs = ct[j], sn = st[j], t = x1;
+          x1 = cs * t - sn * x2;
+          x2 = cs * x2 + sn * t;
+        }
+      }
+      *(__nv_bfloat162*)(qt + h * LD + 2 * j) = __floats2bfloat162_rn(x1, x2);
+    }
+    for (int j = tid; j < half; j += 128) {
+      const float2 x = __ldcg((const float2*)ksrc + j), v = __ldcg((const float2*)vsrc + j);
+      float x1 = x.x, x2 = x.y;
+      if (a.q_gamma) {
+        const float2 g = *((const float2*)(a.k_gamma + kvh * D) + j);
+        x1 *= hsq[1] * g.x; x2 *= hsq[1] * g.y;
+      }
+      if (j < rh) {
+        const float cs = ct[j], sn = st[j], t = x1;
+        x1 = cs * t - sn * x2;
+        x2 = cs * x2 + sn * t;
+      }
+      const __nv_bfloat162 kk = __floats2bfloat162_rn(x1, x2), vv = __floats2bfloat162_rn(v.x, v.y);
+      knew[2 * j] = __low2float(kk); knew[2 * j + 1] = __high2float(kk);
+      vnew[2 * j] = __low2float(vv); vnew[2 * j + 1] = __high2float(vv);
+      if (split == 0) {  // append to the cache for the following steps
+        *(__nv_bfloat162*)(kbase + pos * D + 2 * j) = kk;
+        *(__nv_bfloat162*)(vbase + pos * D + 2 * j) = vv;
+      }
+    }
+    env.sync_cta();
+  } else {
   if (a.q_gamma) {
     // per-head RMSNorm over d for the rep query heads and the key head
     for (int h = warp; h <= rep; h += 4) {
@@ -178,6 +250,7 @@ __device__ __forceinline__ void attn_dec_item(const AttnDecArgs& a, float scale,
     }
   }
   env.sync_cta();
+  }
 
   // ---- 2. this warp's chunks of 32 keys: S = Q K^T, online softmax, O += P V ----
   // A thread owns head r = lane / 4 (rows 8..15 of the MMA tile are padding) and, per 8-key
@@ -310,6 +383,17 @@ __device__ __forceinline__ void attn_dec_item(const AttnDecArgs& a, float scale,
   float* part_ml = (float*)vt;                 // [MAX_REP][2]
   float* part_o = part_ml + 2 * MAX_REP;       // [MAX_REP][D]
   const int S = a.splits;
+  // the merged output oo over the merged sum ll of exp(score - mm), which the sink joins
+  auto finished = [&](int r, float mm, float ll, float oo) {
+    if constexpr (Env::kRows) {
+      if (a.sink) {
+        const float sk = a.sink[kvh * rep + r], top = fmaxf(mm, sk);
+        const float f = __expf(mm - top);
+        return oo * f / (ll * f + __expf(sk - top));
+      }
+    }
+    return ll > 0.f ? oo / ll : 0.f;
+  };
   const bool push = Env::kPush && a.push_merge && S > 1;
   // push form: output i is finished by slice (i / 128) % S, as its block number (i / 128) / S
   const int kmax = (rep * D + 128 * S - 1) / (128 * S);
@@ -375,7 +459,7 @@ __device__ __forceinline__ void attn_dec_item(const AttnDecArgs& a, float scale,
         ll += ls[s] * f;
         oo += os[s] * f;
       }
-      a.out[(b * a.nh + kvh * rep + r) * (int64_t)D + (i - r * D)] = __float2bfloat16_rn(ll > 0.f ? oo / ll : 0.f);
+      a.out[(b * a.nh + kvh * rep + r) * (int64_t)D + (i - r * D)] = __float2bfloat16_rn(finished(r, mm, ll, oo));
     }
     return;
   }
@@ -384,7 +468,7 @@ __device__ __forceinline__ void attn_dec_item(const AttnDecArgs& a, float scale,
     for (int i = tid; i < rep * D; i += 128) {
       const int r = i / D, e = i - r * D;
       const float ll = part_ml[2 * r + 1];
-      a.out[(b * a.nh + kvh * rep + r) * (int64_t)D + e] = __float2bfloat16_rn(ll > 0.f ? part_o[i] / ll : 0.f);
+      a.out[(b * a.nh + kvh * rep + r) * (int64_t)D + e] = __float2bfloat16_rn(finished(r, part_ml[2 * r], ll, part_o[i]));
     }
     env.sync_cta();  // the partials are read: the next item of a resident CTA may reuse the space
     return;
@@ -415,7 +499,7 @@ __device__ __forceinline__ void attn_dec_item(const AttnDecArgs& a, float scale,
       ll += ls[s] * f;
       oo += os[s] * f;
     }
-    a.out[(b * a.nh + kvh * rep + r) * (int64_t)D + (i - r * D)] = __float2bfloat16_rn(ll > 0.f ? oo / ll : 0.f);
+    a.out[(b * a.nh + kvh * rep + r) * (int64_t)D + (i - r * D)] = __float2bfloat16_rn(finished(r, mm, ll, oo));
   }
   // nobody leaves while a peer may still read its shared memory
   env.sync_group();

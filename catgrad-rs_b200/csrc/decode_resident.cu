@@ -206,6 +206,7 @@ struct ResidentAttnEnv {
   __device__ __forceinline__ int64_t settle(int64_t pos) const { return pos; }  // the phase barrier came first
   // items follow one another in a CTA: partials are read where they lie, behind two barriers
   static constexpr bool kPush = false;
+  static constexpr bool kRows = false;
   __device__ __forceinline__ float* landing() const { return nullptr; }
 };
 

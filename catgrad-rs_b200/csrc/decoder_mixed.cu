@@ -3,6 +3,7 @@
 // (prefill, append, decode with its captured graph, generate) are those of decoder.cu.
 //
 // A sequence lives in a slot.  Per layer run (a looped layer counts once per pass) a slot holds
+//   attention          [kv heads, max_seq, head size] keys and values
 //   latent attention   [max_seq, Lw] cached rows (normed latent, rotated key part)
 //   delta, ssd         an f32 matrix per head and the last inputs of the convolutions
 // Nothing is cleared when a slot is reused: a row whose first position is 0 starts from zeros.
@@ -12,7 +13,10 @@
 //
 // Fused steps: all projections of a mixer are one GEMM (w_in); a post-norm, the residual add and
 // the next pre-norm are one pass (k_row_update), which also writes the two-part rows a looped
-// input reads.  Matrices are padded with zeros to multiples of 8 where the tensor cores want it.
+// input reads.  Without post-norms that pass is k_stream_update: the weighted sum over a token's
+// experts, the mixing of the residual streams (a plain residual stream is one stream with unit
+// coefficients), the next sublayer's input and its norm.  Matrices are padded with zeros to multiples
+// of 8 (attention heads to the sizes of its tensor-core kernels) where the tensor cores want it.
 
 #include <algorithm>
 #include <cstring>
@@ -35,6 +39,13 @@ struct MixedLayer {
   int64_t Fp = 0;       // padded feed-forward width
   int Do = 0;           // columns a head takes in the mixer's output
   int64_t Ko = 0;       // width of the mixer's output
+  // coefficients of the streams, per sublayer
+  cg_tensor *hc_in[2] = {nullptr, nullptr}, *hc_out[2] = {nullptr, nullptr}, *hc_mix[2] = {nullptr, nullptr};
+  // experts, stacked
+  cg_tensor *router = nullptr, *correction = nullptr, *we_gate = nullptr, *we_up = nullptr, *we_down = nullptr;
+  // attention
+  cg_tensor *q_gain = nullptr, *k_gain = nullptr, *sink = nullptr;
+  int Dk = 0, Dv = 0;   // columns a key and a value head take
   // latent attention
   cg_tensor *c_gain = nullptr, *uk = nullptr, *uv = nullptr, *w_kv = nullptr, *cos_t = nullptr, *sin_t = nullptr;
   int64_t Lw = 0;       // width of a cached row
@@ -48,15 +59,20 @@ struct MixedLayer {
 struct MixedRun {
   int layer;
   bool starts_pass;
-  cg_tensor *cache = nullptr;                  // latent attention
+  cg_tensor *cache = nullptr;                  // latent attention; keys of attention
+  cg_tensor *cache_v = nullptr;                // attention
   cg_tensor *state = nullptr, *tail = nullptr;  // recurrences
 };
 
 struct MixedModel {
   std::vector<MixedLayer> layers;
   std::vector<MixedRun> runs;
-  bool loop = false;
+  bool loop = false;        // passes start from w_loop
   bool f32 = false;
+  bool sandwich = false;    // norms behind the sublayers too (k_row_update); else streams (k_stream_update)
+  bool recurrent = false;   // some layer has a state that cannot go back
+  int streams = 1;
+  float embed_scale = 1.f;
   int64_t Wp = 0;       // padded width of the residual stream
   cg_tensor *embed_norm = nullptr, *w_loop = nullptr;
   // sequences
@@ -71,6 +87,10 @@ struct MixedModel {
   cg_tensor *x = nullptr, *xn = nullptr, *xcat = nullptr, *y = nullptr, *proj = nullptr, *cv = nullptr, *gl = nullptr, *co = nullptr,
             *ro = nullptr, *att = nullptr, *hact = nullptr, *gu = nullptr, *q = nullptr, *cpk = nullptr, *tok = nullptr, *xw = nullptr,
             *qkv = nullptr, *rn = nullptr, *tinv = nullptr, *kv = nullptr, *lat = nullptr;
+  // experts: (token, expert) pairs
+  cg_tensor *m_logits = nullptr, *m_ids = nullptr, *m_wts = nullptr, *m_pos = nullptr, *m_tiles = nullptr, *m_xg = nullptr, *m_h = nullptr,
+            *m_y = nullptr;
+  int64_t m_pairs = 0;
   int64_t tinv_n = 0, kv_n = 0;
   bool keep = false;
   cg_tensor* kept = nullptr;
@@ -116,6 +136,87 @@ int f32_matrix(cg_decoder* D, const std::string& name, int64_t rows, int64_t col
   return place_all(D, name, rows, cols, *out, 0);
 }
 
+// norm gains as they are applied, after the 1 a design may add to the stored ones
+int gains(cg_decoder* D, const std::string& name, int64_t n, cg_tensor** out) {
+  if (!D->cfg.norm_plus_one) return norm_weight(D, name, n, out);
+  Hold w;
+  CG_TRY(norm_weight(D, name, n, &w.t));
+  CG_TRY(new2(D->c, ST_F32, 1, n, out, false));
+  CG_CUDA(D->c, cudaMemcpyAsync((*out)->data(), w.t->data(), (size_t)n * 4, cudaMemcpyDeviceToDevice, D->c->core->stream));
+  return k_launch_add_scalar(D->c, (float*)(*out)->data(), n, 1.f);
+}
+// n heads of d values each, spread to heads of Dp with zeros between
+int head_gains(cg_decoder* D, const std::string& name, int64_t n, int64_t d, int64_t Dp, cg_tensor** out) {
+  Hold w;
+  CG_TRY(norm_weight(D, name, n * d, &w.t));
+  CG_TRY(new2(D->c, ST_F32, n, Dp, out));
+  CG_CUDA(D->c, cudaMemcpy2DAsync((*out)->data(), (size_t)Dp * 4, w.t->data(), (size_t)d * 4, (size_t)d * 4, (size_t)n,
+                                  cudaMemcpyDeviceToDevice, D->c->core->stream));
+  return CG_OK;
+}
+// the streams' coefficients of a sublayer: all 1 for a plain residual stream
+int coefficients(cg_decoder* D, const std::string& name, int64_t n, cg_tensor** out) {
+  if (D->cfg.streams > 0) return norm_weight(D, name, n, out);
+  CG_TRY(new2(D->c, ST_F32, 1, n, out));
+  return k_launch_add_scalar(D->c, (float*)(*out)->data(), n, 1.f);
+}
+
+int rope_tables(cg_decoder* D, const MixedLayer& L, cg_tensor** cos_t, cg_tensor** sin_t) {
+  const int64_t half = std::max(L.k.rot_dim / 2, 1);
+  CG_TRY(new2(D->c, ST_F32, D->cfg.max_seq, half, cos_t));
+  CG_TRY(new2(D->c, ST_F32, D->cfg.max_seq, half, sin_t));
+  if (!L.k.rot_dim) return CG_OK;
+  return k_launch_pair_rope_tables(D->c, L.k.rot_base, D->cfg.max_seq, L.k.rot_dim, (float*)(*cos_t)->data(), (float*)(*sin_t)->data());
+}
+
+int finalize_attention(cg_decoder* D, MixedLayer& L, const std::string& mx) {
+  cg_ctx* c = D->c;
+  MixedModel& X = *D->mixed;
+  const cg_layer_config& k = L.k;
+  const int64_t W = D->H, H = k.heads, G = k.kv_heads, d = k.dim, dv = k.vdim;
+  const int st = X.act_storage();
+  // head size of the tensor-core kernels; other sizes and f32 only pad to vectors
+  const int64_t widest = std::max(d, dv);
+  const int Dp = X.f32 ? 0 : widest <= 64 ? 64 : widest <= 128 ? 128 : widest <= 256 ? 256 : 0;
+  L.Dk = Dp ? Dp : (int)up8(d);
+  L.Dv = L.Do = Dp ? Dp : (int)up8(dv);
+  L.Np = (H + G) * L.Dk + G * L.Dv;
+  L.Ko = H * L.Dv;
+  CG_TRY(new2(c, st, L.Np, X.Wp, &L.w_in));
+  for (int64_t h = 0; h < H; ++h) CG_TRY(place(D, mx + "q", H * d, W, h * d, d, 0, W, L.w_in, h * L.Dk, 0));
+  for (int64_t g = 0; g < G; ++g) {
+    CG_TRY(place(D, mx + "k", G * d, W, g * d, d, 0, W, L.w_in, (H + g) * L.Dk, 0));
+    CG_TRY(place(D, mx + "v", G * dv, W, g * dv, dv, 0, W, L.w_in, (H + G) * L.Dk + g * L.Dv, 0));
+  }
+  CG_TRY(new2(c, st, X.Wp, L.Ko, &L.w_o));
+  for (int64_t h = 0; h < H; ++h) CG_TRY(place(D, mx + "o", W, H * dv, 0, W, h * dv, dv, L.w_o, 0, h * L.Dv));
+  if (k.qk_norm) {
+    CG_TRY(head_gains(D, mx + "q.norm", H, d, L.Dk, &L.q_gain));
+    CG_TRY(head_gains(D, mx + "k.norm", G, d, L.Dk, &L.k_gain));
+  }
+  if (k.sink) CG_TRY(norm_weight(D, mx + "sink", H, &L.sink));
+  return rope_tables(D, L, &L.cos_t, &L.sin_t);
+}
+
+// [experts, rows padded to rp, cols padded to cp] from l<i>.mlp.e<j>.<name>
+int stack_experts(cg_decoder* D, const std::string& ff, const char* name, int64_t E, int64_t rows, int64_t cols, int64_t rp, int64_t cp,
+                  cg_tensor** out) {
+  CG_TRY(new2(D->c, D->mixed->act_storage(), E * rp, cp, out));
+  for (int64_t e = 0; e < E; ++e) CG_TRY(place_all(D, ff + "e" + std::to_string(e) + "." + name, rows, cols, *out, e * rp));
+  return CG_OK;
+}
+
+int finalize_experts(cg_decoder* D, MixedLayer& L, const std::string& ff) {
+  MixedModel& X = *D->mixed;
+  const int64_t W = D->H, F = L.k.ffn, E = L.k.experts;
+  CG_TRY(new2(D->c, X.act_storage(), E, X.Wp, &L.router));
+  CG_TRY(place_all(D, ff + "router", E, W, L.router, 0));
+  CG_TRY(norm_weight(D, ff + "correction", E, &L.correction));
+  CG_TRY(stack_experts(D, ff, "gate", E, F, W, L.Fp, X.Wp, &L.we_gate));
+  CG_TRY(stack_experts(D, ff, "up", E, F, W, L.Fp, X.Wp, &L.we_up));
+  return stack_experts(D, ff, "down", E, W, F, X.Wp, L.Fp, &L.we_down);
+}
+
 int finalize_latent(cg_decoder* D, MixedLayer& L, const std::string& mx) {
   cg_ctx* c = D->c;
   MixedModel& X = *D->mixed;
@@ -155,10 +256,7 @@ int finalize_latent(cg_decoder* D, MixedLayer& L, const std::string& mx) {
     }
     CG_CUDA(c, cudaStreamSynchronize(c->core->stream));
   }
-  CG_TRY(new2(c, ST_F32, D->cfg.max_seq, std::max<int64_t>(r / 2, 1), &L.cos_t));
-  CG_TRY(new2(c, ST_F32, D->cfg.max_seq, std::max<int64_t>(r / 2, 1), &L.sin_t));
-  if (r) CG_TRY(k_launch_pair_rope_tables(c, k.rot_base, D->cfg.max_seq, (int)r, (float*)L.cos_t->data(), (float*)L.sin_t->data()));
-  return CG_OK;
+  return rope_tables(D, L, &L.cos_t, &L.sin_t);
 }
 
 int finalize_recurrent(cg_decoder* D, MixedLayer& L, const std::string& mx) {
@@ -223,12 +321,20 @@ int ensure_mixed(cg_decoder* D, int64_t M) {
   if (M <= X.cap) return CG_OK;
   cg_ctx* c = D->c;
   forget_graph(D);  // it holds the old buffers
-  int64_t np = 0, cc = 0, hh = 0, inner = 0, ko = 0, fp = 0, qw = 0, lw = 0, qkv = 0, kh = 0;
+  int64_t np = 0, cc = 0, hh = 0, inner = 0, ko = 0, fp = 0, qw = 0, lw = 0, qkv = 0, kh = 0, top = 0, experts = 0, fe = 0;
   for (const MixedLayer& L : X.layers) {
     np = std::max(np, L.Np);
     ko = std::max(ko, L.Ko);
-    fp = std::max(fp, L.Fp);
-    if (L.k.mixer == CG_MIX_LATENT) {
+    if (L.k.experts) {
+      top = std::max<int64_t>(top, L.k.top_k);
+      experts = std::max<int64_t>(experts, L.k.experts);
+      fe = std::max(fe, L.Fp);
+    } else {
+      fp = std::max(fp, L.Fp);
+    }
+    if (L.k.mixer == CG_MIX_ATTENTION) {
+      qw = std::max<int64_t>(qw, (int64_t)L.k.heads * L.Dk);
+    } else if (L.k.mixer == CG_MIX_LATENT) {
       qw = std::max<int64_t>(qw, (int64_t)L.k.heads * L.Dq);
       lw = std::max(lw, L.Lw);
     } else {
@@ -242,7 +348,7 @@ int ensure_mixed(cg_decoder* D, int64_t M) {
     }
   }
   const int st = X.act_storage();
-  CG_TRY(new2(c, ST_F32, M, X.Wp, &X.x));
+  CG_TRY(new2(c, ST_F32, M * X.streams, X.Wp, &X.x));
   CG_TRY(new2(c, st, M, X.Wp, &X.xn));
   CG_TRY(new2(c, ST_F32, M, X.Wp, &X.y));
   if (X.loop) CG_TRY(new2(c, st, M, 2 * X.Wp, &X.xcat));
@@ -274,7 +380,19 @@ int ensure_mixed(cg_decoder* D, int64_t M) {
   }
   if (qw) {
     CG_TRY(new2(c, st, M, qw, &X.q));
-    CG_TRY(new2(c, st, M, lw, &X.cpk));
+    if (lw) CG_TRY(new2(c, st, M, lw, &X.cpk));
+  }
+  if (top) {
+    const int64_t P = M * top;
+    CG_TRY(new2(c, ST_F32, M, experts, &X.m_logits));
+    CG_TRY(new2(c, ST_U32, P, 1, &X.m_ids));
+    CG_TRY(new2(c, ST_F32, P, 1, &X.m_wts));
+    CG_TRY(new2(c, ST_U32, P, 1, &X.m_pos));
+    CG_TRY(new2(c, ST_U32, 3 * P + 4, 1, &X.m_tiles));
+    CG_TRY(new2(c, st, P, X.Wp, &X.m_xg));
+    CG_TRY(new2(c, st, P, fe, &X.m_h));
+    CG_TRY(new2(c, ST_F32, P, X.Wp, &X.m_y));
+    X.m_pairs = P;
   }
   drop(X.tok);
   CG_TRY(new_tensor(c, CG_U32, ST_U32, &M, 1, &X.tok));
@@ -282,9 +400,10 @@ int ensure_mixed(cg_decoder* D, int64_t M) {
   return CG_OK;
 }
 
-// out[M, N] = x[M, K] w[row0 .. row0 + N, K]^T; out_bf16 only in a bf16 context
+// out[M, N] = x[M, K] w[row0 .. row0 + N, K]^T; out_mode (of the GEMMs) 0 f32 or, only in a bf16 context,
+// 1 bf16, 4 bf16 of the square of relu
 int lin(cg_decoder* D, const void* x, int64_t ldx, int64_t M, const cg_tensor* w, int64_t row0, int64_t N, void* out, int64_t ldo,
-        bool out_bf16 = false) {
+        int out_mode = 0) {
   cg_ctx* c = D->c;
   const int64_t K = w->dims[1];
   if (D->mixed->f32)
@@ -294,14 +413,14 @@ int lin(cg_decoder* D, const void* x, int64_t ldx, int64_t M, const cg_tensor* w
   if (gemm_dec_supported(M, K)) {
     DecGemm g;
     g.x = xb; g.ldx = ldx; g.w = wb; g.ldw = K; g.w_rows = N;
-    g.out = out; g.ldo = ldo; g.residual = nullptr; g.out_mode = out_bf16 ? 1 : 0;
+    g.out = out; g.ldo = ldo; g.residual = nullptr; g.out_mode = out_mode;
     g.push = nullptr; g.dual = 0; g.act = 0;
     g.M = M; g.N = N; g.K = K;
     return gemm_dec(c, g);
   }
   const int splits = gemm_tc_pick_splits(M, N, K);
   float* ws = (int64_t)splits * M * N <= D->splitk_floats ? (float*)D->splitk->data() : nullptr;
-  return gemm_tc(c, xb, ldx, wb, K, out, ldo, nullptr, M, N, K, out_bf16 ? 1 : 0, splits, ws);
+  return gemm_tc(c, xb, ldx, wb, K, out, ldo, nullptr, M, N, K, out_mode, splits, ws);
 }
 
 // hact = act(x gate^T) * (x up^T)
@@ -324,6 +443,48 @@ int glu(cg_decoder* D, const MixedLayer& L, const void* x, int64_t M) {
     return gemm_dec(c, g);
   }
   return gemm_tc_pair(c, xb, K, w, K, (__nv_bfloat16*)X.hact->data(), F, M, F, K, L.k.act);
+}
+
+// y = the dense feed-forward of the rows xn
+int dense_ff(cg_decoder* D, const MixedLayer& L, int64_t M) {
+  MixedModel& X = *D->mixed;
+  if (L.k.act == CG_ACT_RELU2) {
+    CG_TRY(lin(D, X.xn->data(), X.Wp, M, L.w_gu, 0, L.Fp, X.hact->data(), L.Fp, X.f32 ? 0 : 4));
+    if (X.f32) CG_TRY(k_launch_relu2_f32(D->c, (float*)X.hact->data(), M * L.Fp));
+  } else {
+    CG_TRY(glu(D, L, X.xn->data(), M));
+  }
+  return lin(D, X.hact->data(), L.Fp, M, L.w_down, 0, X.Wp, X.y->data(), X.Wp);
+}
+
+// m_y[m_pos[pair]] = the chosen experts' results for the rows xn, m_wts their weights
+int experts_ff(cg_decoder* D, const MixedLayer& L, int64_t M) {
+  cg_ctx* c = D->c;
+  MixedModel& X = *D->mixed;
+  MoeArgs a;
+  a.H = (int)X.Wp; a.E = a.El = L.k.experts; a.e_lo = 0; a.k = L.k.top_k; a.Fe = (int)L.Fp;
+  a.norm_topk = 0; a.act = L.k.act; a.act_limit = (float)L.k.act_limit;
+  a.correction = (const float*)L.correction->data(); a.router_scale = (float)L.k.router_scale;
+  a.M = M;
+  a.logits = (float*)X.m_logits->data();
+  a.w.ids = (uint32_t*)X.m_ids->data();
+  a.w.wts = (float*)X.m_wts->data();
+  a.w.pos = (int32_t*)X.m_pos->data();
+  int32_t* t = (int32_t*)X.m_tiles->data();
+  a.w.tile_expert = t; a.w.tile_row0 = t + X.m_pairs; a.w.tile_rows = t + 2 * X.m_pairs; a.w.n_tiles = t + 3 * X.m_pairs;
+  a.w.xg = (__nv_bfloat16*)X.m_xg->data();
+  a.w.h = (__nv_bfloat16*)X.m_h->data();
+  a.w.y = (float*)X.m_y->data();
+  CG_TRY(lin(D, X.xn->data(), X.Wp, M, L.router, 0, a.E, a.logits, a.E));
+  CG_TRY(moe_topk(c, a));
+  if (X.f32)
+    return moe_experts_f32(c, a, (const float*)X.xn->data(), (const float*)L.we_gate->data(), (const float*)L.we_up->data(),
+                           (const float*)L.we_down->data(), (float*)X.m_h->data());
+  a.xn = (__nv_bfloat16*)X.xn->data();
+  a.w_gate = (const __nv_bfloat16*)L.we_gate->data();
+  a.w_up = (const __nv_bfloat16*)L.we_up->data();
+  a.w_down = (const __nv_bfloat16*)L.we_down->data();
+  return moe_experts(c, a);
 }
 
 // What the host knows about a portion: per row its new tokens and the position of the first.
@@ -390,6 +551,57 @@ int grow(cg_ctx* c, int storage, int64_t n, cg_tensor** t, int64_t* have) {
   return CG_OK;
 }
 
+// One token per row: norms, rotation, cache append and attention in one kernel.  Longer rows: a pass
+// that norms, rotates and appends, then the prompt attention on the tensor cores.  f32, and sizes those
+// kernels do not have: one block per token and head.
+int attention_layer(cg_decoder* D, const MixedLayer& L, MixedRun& run, const RowsDev& rd, const Portion* p) {
+  cg_ctx* c = D->c;
+  MixedModel& X = *D->mixed;
+  const cg_layer_config& k = L.k;
+  CG_TRY(lin(D, X.xn->data(), X.Wp, rd.M, L.w_in, 0, L.Np, X.proj->data(), L.Np));
+  const float* q_gain = L.q_gain ? (const float*)L.q_gain->data() : nullptr;
+  const float* k_gain = L.k_gain ? (const float*)L.k_gain->data() : nullptr;
+  const float* sink = L.sink ? (const float*)L.sink->data() : nullptr;
+  const bool tensor = !X.f32 && L.Dk == L.Dv && (L.Dk == 64 || L.Dk == 128 || L.Dk == 256);
+  if (tensor && (!p || p->max_len == 1) && k.heads / k.kv_heads <= 8) {
+    AttnDecArgs f{};
+    f.qkv = (const float*)X.proj->data();
+    f.cos_t = (const float*)L.cos_t->data(); f.sin_t = (const float*)L.sin_t->data();
+    f.q_gamma = q_gain; f.k_gamma = k_gain; f.norm_eps = D->cfg.rms_eps;
+    f.k_cache = (__nv_bfloat16*)run.cache->data(); f.v_cache = (__nv_bfloat16*)run.cache_v->data();
+    f.out = (__nv_bfloat16*)X.att->data();
+    f.Tmax = D->cfg.max_seq; f.B = rd.rows;
+    f.nh = k.heads; f.nkv = k.kv_heads; f.d = L.Dk;
+    f.window = k.window; f.rows = rd; f.rot_dims = k.rot_dim; f.norm_dim = k.dim;
+    f.scale = (float)k.scale; f.sink = sink;
+    const int64_t reach = k.window > 0 ? std::min<int64_t>(k.window, f.Tmax) : f.Tmax;
+    f.splits = attn_dec_splits(reach, f.B * f.nkv, f.d);
+    return k_launch_attn_dec(c, f);
+  }
+  RowsAttnArgs a;
+  a.proj = (const float*)X.proj->data(); a.ldp = L.Np;
+  a.H = k.heads; a.G = k.kv_heads; a.d = k.dim; a.dv = k.vdim; a.Dk = L.Dk; a.Dv = L.Dv;
+  a.q_gain = q_gain; a.k_gain = k_gain; a.eps = D->cfg.rms_eps; a.scale = (float)k.scale;
+  a.rot = k.rot_dim;
+  a.cos_t = (const float*)L.cos_t->data(); a.sin_t = (const float*)L.sin_t->data();
+  a.window = k.window; a.sink = sink;
+  a.q = X.q->data(); a.k_cache = run.cache->data(); a.v_cache = run.cache_v->data();
+  a.Tmax = D->cfg.max_seq; a.slots = D->cfg.max_batch;
+  a.att = X.att->data(); a.ld_att = L.Ko;
+  a.bf16 = X.f32 ? 0 : 1;
+  a.rows = rd;
+  CG_TRY(k_launch_rows_qkv(c, a));
+  if (!tensor || !p) return k_launch_rows_attn(c, a);
+  AttnArgs t{};
+  t.q = (const __nv_bfloat16*)a.q;
+  t.k_cache = (const __nv_bfloat16*)a.k_cache; t.v_cache = (const __nv_bfloat16*)a.v_cache;
+  t.out = (__nv_bfloat16*)a.att;
+  t.B = a.slots; t.S = p->max_len; t.Tmax = a.Tmax;
+  t.nh = a.H; t.nkv = a.G; t.d = L.Dk;
+  t.window = a.window; t.scale = a.scale; t.sink = sink; t.rows = rd;
+  return k_launch_attn_prefill(c, t);
+}
+
 // A few new tokens: attention in the cached rows' space.  Prompts: the cached rows are expanded to
 // keys and values of Dq values per head, token after token, and run through the prompt attention.
 // f32, and sizes those kernels do not have: one block per token and head.
@@ -430,13 +642,13 @@ int latent_layer(cg_decoder* D, const MixedLayer& L, MixedRun& run, const RowsDe
   if (fresh) a.c_out = X.cpk->data();
   CG_TRY(k_launch_latent_prep(c, a));
   if (fresh) {
-    CG_TRY(lin(D, X.cpk->data(), L.Lw, rd.M, L.w_kv, 0, kvw, kv, kvw, true));
+    CG_TRY(lin(D, X.cpk->data(), L.Lw, rd.M, L.w_kv, 0, kvw, kv, kvw, 1));
   } else {
     int64_t at = 0;
     for (int r = 0; r < R; ++r) {
       const int64_t n = p->pos0[r] + p->lens[r];
       CG_TRY(lin(D, (const char*)a.cache + (size_t)p->slots[r] * a.Tmax * L.Lw * es, L.Lw, n, L.w_kv, 0, kvw, kv + (size_t)at * kvw * es, kvw,
-                 true));
+                 1));
       at += n;
     }
   }
@@ -494,7 +706,7 @@ int recurrent_layer(cg_decoder* D, const MixedLayer& L, MixedRun& run, const Row
     __nv_bfloat16* pb = (__nv_bfloat16*)X.proj->data();
     float* small = (float*)(pb + M * L.small_off);  // both fit where the f32 projection would
     const int64_t ns = L.Np - L.small_off;
-    CG_TRY(lin(D, X.xn->data(), K, M, L.w_in, 0, L.small_off, pb, L.small_off, true));
+    CG_TRY(lin(D, X.xn->data(), K, M, L.w_in, 0, L.small_off, pb, L.small_off, 1));
     CG_TRY(lin(D, X.xn->data(), K, M, L.w_in, L.small_off, ns, small, ns));
     a.proj = pb; a.ldp = L.small_off;
     a.small = small; a.ld_small = ns;
@@ -526,11 +738,108 @@ int recurrent_layer(cg_decoder* D, const MixedLayer& L, MixedRun& run, const Row
   return k_launch_gated_norm(c, n);
 }
 
+int mixer(cg_decoder* D, const MixedLayer& L, MixedRun& run, const RowsDev& rd, const Portion* p, const Chunks* ch) {
+  MixedModel& X = *D->mixed;
+  if (L.k.mixer == CG_MIX_ATTENTION) CG_TRY(attention_layer(D, L, run, rd, p));
+  else if (L.k.mixer == CG_MIX_LATENT) CG_TRY(latent_layer(D, L, run, rd, p));
+  else CG_TRY(recurrent_layer(D, L, run, rd, p, ch));
+  return lin(D, X.att->data(), L.Ko, rd.M, L.w_o, 0, X.Wp, X.y->data(), X.Wp);
+}
+
+// room for the residual streams of all layer runs of M tokens
+int keep_room(cg_decoder* D, int64_t M) {
+  MixedModel& X = *D->mixed;
+  drop(X.kept);
+  int64_t d3[3] = {(int64_t)X.runs.size(), M, D->H};
+  return new_tensor(D->c, CG_F32, ST_F32, d3, 3, &X.kept);
+}
+
+// The walk of designs without post-norms: sublayer by sublayer, each update preparing the next one's
+// normed input in xn.
+int walk_streams(cg_decoder* D, const RowsDev& rd, const uint32_t* tokens, const Portion* p, const Chunks* ch) {
+  cg_ctx* c = D->c;
+  MixedModel& X = *D->mixed;
+  const int64_t M = rd.M, Wp = X.Wp;
+  const int bf = X.f32 ? 0 : 1;
+  const size_t nruns = X.runs.size();
+  StreamUpdate base;
+  base.ns = X.streams;
+  base.x = (float*)X.x->data(); base.ldx = Wp; base.eps = D->cfg.rms_eps; base.W = (int)D->H;
+  // what the update leaves for sublayer q of run i
+  auto hand_on = [&](StreamUpdate& u, size_t i, int q) {
+    if (i >= nruns) return;
+    const MixedLayer& L = X.layers[X.runs[i].layer];
+    u.in_w = (const float*)L.hc_in[q]->data();
+    u.g = (const float*)(q ? L.n2 : L.n1)->data();
+    u.out = X.xn->data(); u.ldo = Wp;
+  };
+  auto update = [&](const MixedLayer& L, int q) {
+    StreamUpdate u = base;
+    u.mix = (const float*)L.hc_mix[q]->data(); u.out_w = (const float*)L.hc_out[q]->data();
+    if (q && L.k.experts) {
+      u.y = (const float*)X.m_y->data(); u.ldy = Wp;
+      u.pos = (const int32_t*)X.m_pos->data(); u.wts = (const float*)X.m_wts->data(); u.top = L.k.top_k;
+    } else {
+      u.y = (const float*)X.y->data(); u.ldy = Wp;
+    }
+    return u;
+  };
+  {
+    StreamUpdate u = base;
+    u.tokens = tokens; u.table = D->embed->data(); u.table_bf16 = D->embed->storage == ST_BF16; u.vocab = D->cfg.vocab;
+    u.scale = X.embed_scale;
+    hand_on(u, 0, 0);
+    CG_TRY(k_launch_stream_update(c, u, M, bf));
+  }
+  for (size_t i = 0; i < nruns; ++i) {
+    MixedRun& run = X.runs[i];
+    const MixedLayer& L = X.layers[run.layer];
+    CG_TRY(mixer(D, L, run, rd, p, ch));
+    StreamUpdate u = update(L, 0);
+    if (L.k.ffn) {
+      hand_on(u, i, 1);
+      CG_TRY(k_launch_stream_update(c, u, M, bf));
+      if (L.k.experts) CG_TRY(experts_ff(D, L, M));
+      else CG_TRY(dense_ff(D, L, M));
+      u = update(L, 1);
+    }
+    hand_on(u, i + 1, 0);
+    if (X.keep && p) {
+      if (i == 0) CG_TRY(keep_room(D, M));
+      u.sum = (float*)X.kept->data() + (int64_t)i * M * D->H; u.ld_sum = D->H;
+    }
+    CG_TRY(k_launch_stream_update(c, u, M, bf));
+  }
+  return CG_OK;
+}
+
+// out[dst[i]] = the final norm of packed token pick[i]'s residual stream
+int final_rows(cg_decoder* D, const int32_t* pick, const int32_t* dst, int64_t n, void* out) {
+  MixedModel& X = *D->mixed;
+  auto fill = [&](auto& u) {
+    u.x = (float*)X.x->data(); u.ldx = X.Wp; u.eps = D->cfg.rms_eps; u.W = (int)D->H;
+    u.pick = pick; u.dst = dst;
+    u.out = out; u.ldo = X.Wp;
+  };
+  if (X.sandwich) {
+    RowUpdate u;
+    fill(u);
+    u.g2 = (const float*)D->ln_f->data();
+    return k_launch_row_update(D->c, u, n, X.f32 ? 0 : 1);
+  }
+  StreamUpdate u;
+  fill(u);
+  u.ns = X.streams;
+  u.g = (const float*)D->ln_f->data();
+  return k_launch_stream_update(D->c, u, n, X.f32 ? 0 : 1);
+}
+
 // Embedding and all layer runs of one batch; x holds the residual stream afterwards.  p is null in
 // decode steps (one token per row).
 int walk(cg_decoder* D, const RowsDev& rd, const uint32_t* tokens, const Portion* p, const Chunks* ch) {
   cg_ctx* c = D->c;
   MixedModel& X = *D->mixed;
+  if (!X.sandwich) return walk_streams(D, rd, tokens, p, ch);
   const int64_t M = rd.M, W = D->H, Wp = X.Wp;
   const int bf = X.f32 ? 0 : 1;
   char* cat_lo = X.loop ? (char*)X.xcat->data() : nullptr;
@@ -547,7 +856,7 @@ int walk(cg_decoder* D, const RowsDev& rd, const uint32_t* tokens, const Portion
   {
     RowUpdate u = base;
     u.tokens = tokens; u.table = D->embed->data(); u.table_bf16 = D->embed->storage == ST_BF16; u.vocab = D->cfg.vocab;
-    u.g1 = (const float*)X.embed_norm->data();
+    u.g1 = X.embed_norm ? (const float*)X.embed_norm->data() : nullptr;
     u.x0 = cat_hi; u.ld0 = 2 * Wp;
     hand_on(u, 0);
     CG_TRY(k_launch_row_update(c, u, M, bf));
@@ -562,28 +871,21 @@ int walk(cg_decoder* D, const RowsDev& rd, const uint32_t* tokens, const Portion
       u.out = X.xn->data(); u.ldo = Wp; u.g2 = (const float*)L.n1->data();
       CG_TRY(k_launch_row_update(c, u, M, bf));
     }
-    if (L.k.mixer == CG_MIX_LATENT) CG_TRY(latent_layer(D, L, run, rd, p));
-    else CG_TRY(recurrent_layer(D, L, run, rd, p, ch));
-    CG_TRY(lin(D, X.att->data(), L.Ko, M, L.w_o, 0, Wp, X.y->data(), Wp));
+    CG_TRY(mixer(D, L, run, rd, p, ch));
     RowUpdate u = base;
     u.y = (const float*)X.y->data(); u.ldy = Wp; u.add = 1;
     u.g1 = (const float*)L.n1b->data();
     if (L.k.ffn) {
       u.out = X.xn->data(); u.ldo = Wp; u.g2 = (const float*)L.n2->data();
       CG_TRY(k_launch_row_update(c, u, M, bf));
-      CG_TRY(glu(D, L, X.xn->data(), M));
-      CG_TRY(lin(D, X.hact->data(), L.Fp, M, L.w_down, 0, Wp, X.y->data(), Wp));
+      CG_TRY(dense_ff(D, L, M));
       u.g1 = (const float*)L.n2b->data();
       u.out = nullptr; u.g2 = nullptr;
     }
     hand_on(u, i + 1);
     CG_TRY(k_launch_row_update(c, u, M, bf));
     if (X.keep && p) {
-      if (i == 0) {
-        drop(X.kept);
-        int64_t d3[3] = {(int64_t)nruns, M, W};
-        CG_TRY(new_tensor(c, CG_F32, ST_F32, d3, 3, &X.kept));
-      }
+      if (i == 0) CG_TRY(keep_room(D, M));
       CG_CUDA(c, cudaMemcpy2DAsync((float*)X.kept->data() + (int64_t)i * M * W, (size_t)W * 4, X.x->data(), (size_t)Wp * 4, (size_t)W * 4,
                                    (size_t)M, cudaMemcpyDeviceToDevice, c->core->stream));
     }
@@ -602,12 +904,35 @@ int mixed_create(cg_decoder* D, const cg_layer_config* layers, int n_layers, con
   D->mixed = X;
   X->f32 = D->c->precision == CG_PREC_F32;
   X->Wp = up8(D->H);
+  X->sandwich = D->cfg.post_norms != 0;
+  X->streams = std::max(D->cfg.streams, 1);
+  if (D->cfg.embed_scale != 0.f) X->embed_scale = D->cfg.embed_scale;
+  if (D->cfg.streams < 0 || D->cfg.streams > MAX_STREAMS) return fail(D->c, CG_ERR_UNSUPPORTED, "decoder: at most 16 streams");
+  if (X->sandwich && (D->cfg.streams || X->embed_scale != 1.f || D->cfg.norm_plus_one))
+    return fail(D->c, CG_ERR_UNSUPPORTED, "decoder: post-norms go with one stream, plain gains and an unscaled embedding");
+  if (!X->sandwich && (D->cfg.embed_norm || D->cfg.loop_input))
+    return fail(D->c, CG_ERR_UNSUPPORTED, "decoder: a normed embedding and looped inputs go with post-norms");
   X->layers.resize(n_layers);
   for (int i = 0; i < n_layers; ++i) {
     const cg_layer_config& k = layers[i];
     X->layers[i].k = k;
     if (k.heads < 1 || k.vdim < 1 || k.ffn < 0) return bad_size(D, i, "sizes must be positive");
-    if (k.mixer == CG_MIX_LATENT) {
+    if (k.ffn && k.experts) {
+      if (X->sandwich) return bad_size(D, i, "experts and post-norms do not go together");
+      if (k.experts < 0 || k.experts > 1024 || k.top_k < 1 || k.top_k > 32 || k.top_k > k.experts)
+        return bad_size(D, i, "1 to 1024 experts, at most 32 per token");
+      if (k.act < CG_ACT_SILU || k.act > CG_ACT_BOUNDED || (k.act == CG_ACT_BOUNDED && !(k.act_limit > 0)))
+        return bad_size(D, i, "activation of the experts");
+    } else if (k.ffn && k.act != CG_ACT_SILU && k.act != CG_ACT_GELU && k.act != CG_ACT_RELU2) {
+      return bad_size(D, i, "activation of the feed-forward");
+    }
+    if (!k.ffn) X->layers[i].k.experts = 0;
+    X->recurrent = X->recurrent || k.mixer == CG_MIX_DELTA || k.mixer == CG_MIX_SSD;
+    if (k.mixer == CG_MIX_ATTENTION) {
+      if (k.dim < 1 || k.kv_heads < 1 || k.heads % k.kv_heads || k.window < 0 || k.rot_dim < 0 || k.rot_dim % 2 || k.rot_dim > k.dim ||
+          (k.rot_dim && !(k.rot_base > 0)) || !(k.scale > 0))
+        return bad_size(D, i, "attention sizes");
+    } else if (k.mixer == CG_MIX_LATENT) {
       if (k.dim < 1 || k.rot_dim < 0 || k.rot_dim % 2 || k.kv_rank < 1 || (k.rot_dim && !(k.rot_base > 0)))
         return bad_size(D, i, "latent attention sizes");
     } else if (k.mixer == CG_MIX_DELTA) {
@@ -619,7 +944,7 @@ int mixed_create(cg_decoder* D, const cg_layer_config* layers, int n_layers, con
   }
   const bool looped = loop && loop->times > 0 && loop->stop > loop->start;
   if (looped && (loop->start < 0 || loop->stop > n_layers)) return fail(D->c, CG_ERR_INVALID, "decoder: loop out of range");
-  X->loop = looped;
+  X->loop = looped && D->cfg.loop_input;
   auto add = [&](int i, bool starts) {
     MixedRun r;
     r.layer = i;
@@ -629,7 +954,7 @@ int mixed_create(cg_decoder* D, const cg_layer_config* layers, int n_layers, con
   const int a = looped ? loop->start : n_layers, b = looped ? loop->stop : n_layers;
   for (int i = 0; i < a; ++i) add(i, false);
   for (int t = 0; looped && t < loop->times; ++t)
-    for (int i = a; i < b; ++i) add(i, i == a);
+    for (int i = a; i < b; ++i) add(i, X->loop && i == a);
   for (int i = b; i < n_layers; ++i) add(i, false);
   X->open.assign(D->cfg.max_batch, 0);
   X->pos.assign(D->cfg.max_batch, 0);
@@ -639,14 +964,18 @@ int mixed_create(cg_decoder* D, const cg_layer_config* layers, int n_layers, con
 void mixed_destroy(cg_decoder* D) {
   MixedModel* X = D->mixed;
   if (!X) return;
-  for (MixedLayer& L : X->layers)
+  for (MixedLayer& L : X->layers) {
     for (cg_tensor** t : {&L.n1, &L.n1b, &L.n2, &L.n2b, &L.w_in, &L.w_o, &L.w_gu, &L.w_down, &L.c_gain, &L.uk, &L.uv, &L.w_kv, &L.cos_t,
-                          &L.sin_t, &L.conv_w, &L.conv_b, &L.a_log, &L.dt_bias, &L.dskip, &L.norm})
+                          &L.sin_t, &L.conv_w, &L.conv_b, &L.a_log, &L.dt_bias, &L.dskip, &L.norm, &L.q_gain, &L.k_gain, &L.sink,
+                          &L.router, &L.correction, &L.we_gate, &L.we_up, &L.we_down})
       drop(*t);
-  for (MixedRun& r : X->runs) { drop(r.cache); drop(r.state); drop(r.tail); }
+    for (int q = 0; q < 2; ++q) { drop(L.hc_in[q]); drop(L.hc_out[q]); drop(L.hc_mix[q]); }
+  }
+  for (MixedRun& r : X->runs) { drop(r.cache); drop(r.cache_v); drop(r.state); drop(r.tail); }
   for (cg_tensor** t : {&X->embed_norm, &X->w_loop, &X->tab_run, &X->tab_dec, &X->x, &X->xn, &X->xcat, &X->y, &X->proj, &X->cv, &X->gl,
                         &X->co, &X->ro, &X->att, &X->hact, &X->gu, &X->q, &X->cpk, &X->tok, &X->xw, &X->kept, &X->qkv, &X->rn,
-                        &X->tinv, &X->kv, &X->lat})
+                        &X->tinv, &X->kv, &X->lat, &X->m_logits, &X->m_ids, &X->m_wts, &X->m_pos, &X->m_tiles, &X->m_xg, &X->m_h,
+                        &X->m_y})
     drop(*t);
   delete X;
   D->mixed = nullptr;
@@ -660,20 +989,32 @@ int mixed_finalize(cg_decoder* D) {
   for (size_t i = 0; i < X.layers.size(); ++i) {
     MixedLayer& L = X.layers[i];
     const std::string l = "l" + std::to_string(i) + ".";
-    CG_TRY(norm_weight(D, l + "norm1", W, &L.n1));
-    CG_TRY(norm_weight(D, l + "norm1b", W, &L.n1b));
-    if (L.k.mixer == CG_MIX_LATENT) CG_TRY(finalize_latent(D, L, l + "mix."));
+    CG_TRY(gains(D, l + "norm1", W, &L.n1));
+    if (X.sandwich) CG_TRY(norm_weight(D, l + "norm1b", W, &L.n1b));
+    for (int q = 0; q < (L.k.ffn ? 2 : 1) && !X.sandwich; ++q) {
+      const std::string hc = l + (q ? "hc2." : "hc1.");
+      CG_TRY(coefficients(D, hc + "in", X.streams, &L.hc_in[q]));
+      CG_TRY(coefficients(D, hc + "out", X.streams, &L.hc_out[q]));
+      CG_TRY(coefficients(D, hc + "mix", (int64_t)X.streams * X.streams, &L.hc_mix[q]));
+    }
+    if (L.k.mixer == CG_MIX_ATTENTION) CG_TRY(finalize_attention(D, L, l + "mix."));
+    else if (L.k.mixer == CG_MIX_LATENT) CG_TRY(finalize_latent(D, L, l + "mix."));
     else CG_TRY(finalize_recurrent(D, L, l + "mix."));
     if (L.k.ffn) {
       const int64_t F = L.k.ffn;
       L.Fp = up8(F);
-      CG_TRY(norm_weight(D, l + "norm2", W, &L.n2));
-      CG_TRY(norm_weight(D, l + "norm2b", W, &L.n2b));
-      CG_TRY(new2(c, st, 2 * L.Fp, X.Wp, &L.w_gu));
-      CG_TRY(place_all(D, l + "mlp.gate", F, W, L.w_gu, 0));
-      CG_TRY(place_all(D, l + "mlp.up", F, W, L.w_gu, L.Fp));
-      CG_TRY(new2(c, st, X.Wp, L.Fp, &L.w_down));
-      CG_TRY(place_all(D, l + "mlp.down", W, F, L.w_down, 0));
+      CG_TRY(gains(D, l + "norm2", W, &L.n2));
+      if (X.sandwich) CG_TRY(norm_weight(D, l + "norm2b", W, &L.n2b));
+      if (L.k.experts) {
+        CG_TRY(finalize_experts(D, L, l + "mlp."));
+      } else {
+        const bool gated = L.k.act != CG_ACT_RELU2;
+        CG_TRY(new2(c, st, (gated ? 2 : 1) * L.Fp, X.Wp, &L.w_gu));
+        if (gated) CG_TRY(place_all(D, l + "mlp.gate", F, W, L.w_gu, 0));
+        CG_TRY(place_all(D, l + "mlp.up", F, W, L.w_gu, gated ? L.Fp : 0));
+        CG_TRY(new2(c, st, X.Wp, L.Fp, &L.w_down));
+        CG_TRY(place_all(D, l + "mlp.down", W, F, L.w_down, 0));
+      }
     }
     // the originals of this layer are no longer needed
     for (auto it = D->params.begin(); it != D->params.end();) {
@@ -684,7 +1025,10 @@ int mixed_finalize(cg_decoder* D) {
   const int64_t slots = D->cfg.max_batch;
   for (MixedRun& r : X.runs) {
     const MixedLayer& L = X.layers[r.layer];
-    if (L.k.mixer == CG_MIX_LATENT) {
+    if (L.k.mixer == CG_MIX_ATTENTION) {
+      CG_TRY(new2(c, st, slots * L.k.kv_heads * D->cfg.max_seq, L.Dk, &r.cache));
+      CG_TRY(new2(c, st, slots * L.k.kv_heads * D->cfg.max_seq, L.Dv, &r.cache_v));
+    } else if (L.k.mixer == CG_MIX_LATENT) {
       CG_TRY(new2(c, st, slots * D->cfg.max_seq, L.Lw, &r.cache));
     } else {
       CG_TRY(new2(c, ST_F32, slots * L.H * L.dk, L.dvs, &r.state));
@@ -696,12 +1040,17 @@ int mixed_finalize(cg_decoder* D) {
     CG_TRY(place(D, "loop.in", W, 2 * W, 0, W, 0, W, X.w_loop, 0, 0));
     CG_TRY(place(D, "loop.in", W, 2 * W, 0, W, W, W, X.w_loop, 0, X.Wp));
   }
-  CG_TRY(norm_weight(D, "embed.norm", W, &X.embed_norm));
-  CG_TRY(norm_weight(D, "final.norm", W, &D->ln_f));
+  if (D->cfg.embed_norm) CG_TRY(norm_weight(D, "embed.norm", W, &X.embed_norm));
+  CG_TRY(gains(D, "final.norm", W, &D->ln_f));
   CG_TRY(new2(c, st, D->cfg.vocab, W, &D->embed, false));
   CG_TRY(place_all(D, "embed", D->cfg.vocab, W, D->embed, 0));
-  CG_TRY(new2(c, st, D->cfg.vocab, X.Wp, &D->head));
-  CG_TRY(place_all(D, "head", D->cfg.vocab, W, D->head, 0));
+  if (D->cfg.tie_embeddings && X.Wp == W) {
+    D->head = D->embed;
+    D->head->rc++;
+  } else {
+    CG_TRY(new2(c, st, D->cfg.vocab, X.Wp, &D->head));
+    CG_TRY(place_all(D, D->cfg.tie_embeddings ? "embed" : "head", D->cfg.vocab, W, D->head, 0));
+  }
   for (auto& kv : D->params) release(kv.second);
   D->params.clear();
 
@@ -721,7 +1070,7 @@ int mixed_finalize(cg_decoder* D) {
   CG_TRY(new2(c, st, slots, X.Wp, &D->xl));
   // split-K partials of problems of at most 64 tokens
   int64_t widest = std::max<int64_t>(X.Wp, D->Vp);
-  for (const MixedLayer& L : X.layers) widest = std::max({widest, L.Np, 2 * L.Fp});
+  for (const MixedLayer& L : X.layers) widest = std::max({widest, L.Np, 2 * L.Fp, (int64_t)L.k.experts});
   n = X.f32 ? 1 : std::max<int64_t>(8 * 64 * widest, (int64_t)300 * 128 * 256);
   CG_TRY(new_tensor(c, CG_F32, ST_F32, &n, 1, &D->splitk));
   D->splitk_floats = n;
@@ -830,11 +1179,7 @@ int mixed_run(cg_decoder* D, const std::vector<int>& slots, const std::vector<in
       const size_t np = pick.size();
       CG_CUDA(c, cudaMemcpyAsync(pd, pick.data(), np * 4, cudaMemcpyHostToDevice, c->core->stream));
       CG_CUDA(c, cudaMemcpyAsync(pd + np, dst.data(), np * 4, cudaMemcpyHostToDevice, c->core->stream));
-      RowUpdate u;
-      u.x = (float*)X.x->data(); u.ldx = X.Wp; u.eps = D->cfg.rms_eps; u.W = (int)D->H;
-      u.pick = pd; u.dst = pd + np;
-      u.out = X.xw->data(); u.ldo = X.Wp; u.g2 = (const float*)D->ln_f->data();
-      CG_TRY(k_launch_row_update(c, u, (int64_t)np, X.f32 ? 0 : 1));
+      CG_TRY(final_rows(D, pd, pd + np, (int64_t)np, X.xw->data()));
     }
   }
   for (int r = 0; r < R; ++r) X.pos[slots[r]] += lens[r];
@@ -878,9 +1223,12 @@ int mixed_prefill(cg_decoder* D, const cg_tensor* tokens, bool fresh) {
 int mixed_truncate(cg_decoder* D, int64_t positions) {
   MixedModel& X = *D->mixed;
   if (positions == 0) return mixed_reset(D);
-  for (int s : X.cur_slots)
-    if (X.pos[s] != positions)
+  for (int s : X.cur_slots) {
+    if (X.pos[s] != positions && X.recurrent)
       return fail(D->c, CG_ERR_UNSUPPORTED, "decoder: a recurrent state cannot go back to an earlier position (truncate to 0 and run again)");
+    if (positions < 0 || positions > X.pos[s]) return fail(D->c, CG_ERR_SHAPE, "decoder: cannot truncate to more than is cached");
+  }
+  for (int s : X.cur_slots) X.pos[s] = positions;
   X.tables_current = false;
   return set_state(D, 0, 0);
 }
@@ -922,11 +1270,7 @@ int mixed_step(cg_decoder* D) {
   rd.rows = R;
   rd.M = R;
   CG_TRY(walk(D, rd, (const uint32_t*)D->cur->data(), nullptr, nullptr));
-  RowUpdate u;
-  u.x = (float*)X.x->data(); u.ldx = X.Wp; u.eps = D->cfg.rms_eps; u.W = (int)D->H;
-  u.pick = rd.tok_row;  // row i of the batch is token i
-  u.out = D->xl->data(); u.ldo = X.Wp; u.g2 = (const float*)D->ln_f->data();
-  CG_TRY(k_launch_row_update(c, u, R, X.f32 ? 0 : 1));
+  CG_TRY(final_rows(D, rd.tok_row, nullptr, R, D->xl->data()));  // row i of the batch is token i
   float* lg = (float*)D->logits->data();
   CG_TRY(lin(D, D->xl->data(), X.Wp, R, D->head, 0, D->Vp, lg, D->Vp));
   return k_launch_argmax(c, lg, R, D->Vp, 1, D->cfg.final_softcap, (uint32_t*)D->cur->data(), (uint32_t*)D->history->data(),

@@ -38,11 +38,12 @@ struct TcpArgs {
   const float* residual;
   int64_t ldo;
   int M, N, K;
-  int out_mode;   // 0 f32, 1 bf16, 2 f32 + residual (residual may alias out)
+  int out_mode;   // 0 f32, 1 bf16, 2 f32 + residual (residual may alias out), 4 bf16 of the square of relu
   int kb_total;
   int m_tiles, n_tiles;
   int row2_off;   // PAIR: rows between a gate row and its up row
-  int act;        // PAIR: 0 silu, 1 tanh-gelu
+  int act;        // PAIR: 0 silu, 1 tanh-gelu; GROUPED also 2, bounded (act.cuh)
+  float limit;    // act 2
   // GROUPED (mixture-of-experts): token tiles come from a device-built list, each belonging to
   // one expert whose weights start at row expert * w_rows of the stacked matrix; rows of a tile
   // past `tile_rows` belong to other experts and are not stored
@@ -211,7 +212,8 @@ k_gemm_tcp(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CU
               const int m = m0 + c0 + j;
               if (m >= m_end) break;
               const float g = __uint_as_float(v[j]);
-              const float h = (p.act == 0 ? silu_f(g) : gelu_f(g)) * __uint_as_float(u[j]);
+              const float h = GROUPED ? glu_f(p.act, p.limit, g, __uint_as_float(u[j]))
+                                      : (p.act == 0 ? silu_f(g) : gelu_f(g)) * __uint_as_float(u[j]);
               ((__nv_bfloat16*)p.out)[(int64_t)m * p.ldo + n] = __float2bfloat16_rn(h);
             }
           }
@@ -237,7 +239,9 @@ k_gemm_tcp(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CU
                 const int m = m0 + c0 + j;
                 if (m >= m_end) break;
                 if (p.out_mode == 0) ((float*)p.out)[(int64_t)m * p.ldo + n] = __uint_as_float(v[j]);
-                else ((__nv_bfloat16*)p.out)[(int64_t)m * p.ldo + n] = __float2bfloat16_rn(__uint_as_float(v[j]));
+                else
+                  ((__nv_bfloat16*)p.out)[(int64_t)m * p.ldo + n] =
+                      __float2bfloat16_rn(p.out_mode == 4 ? relu2_f(__uint_as_float(v[j])) : __uint_as_float(v[j]));
               }
             }
           }
@@ -306,6 +310,7 @@ int gemm_tcp(cg_ctx* c, const __nv_bfloat16* x, int64_t ldx, const __nv_bfloat16
   a.n_tiles = (int)((N + BM - 1) / BM);
   a.row2_off = (int)N;
   a.act = act;
+  a.limit = 0.f;
   a.tile_expert = a.tile_row0 = a.tile_rows = a.n_list = nullptr;
   a.w_rows = 0;
   a.err = c->core->dev_err;
@@ -320,7 +325,7 @@ int gemm_tcp(cg_ctx* c, const __nv_bfloat16* x, int64_t ldx, const __nv_bfloat16
 // moe.cu.  w (and w_up when pair) are the experts' matrices stacked along the rows
 // ([experts * N, K]); x holds the grouped activation rows; out rows follow x.
 int gemm_tcp_grouped(cg_ctx* c, const __nv_bfloat16* x, int64_t x_rows, const __nv_bfloat16* w, const __nv_bfloat16* w_up,
-                     int64_t experts, void* out, int64_t N, int64_t K, int pair, int act, const int32_t* tile_expert,
+                     int64_t experts, void* out, int64_t N, int64_t K, int pair, int act, float limit, const int32_t* tile_expert,
                      const int32_t* tile_row0, const int32_t* tile_rows, const int32_t* n_list, int64_t max_list) {
   if (x_rows <= 0 || N <= 0 || experts <= 0) return CG_OK;
   if (K <= 0 || K % 8 || ((uintptr_t)x % 16) || ((uintptr_t)w % 16) || (pair && ((uintptr_t)w_up % 16)))
@@ -338,6 +343,7 @@ int gemm_tcp_grouped(cg_ctx* c, const __nv_bfloat16* x, int64_t x_rows, const __
   a.n_tiles = (int)((N + BM - 1) / BM);
   a.row2_off = 0;
   a.act = act;
+  a.limit = limit;
   a.tile_expert = tile_expert; a.tile_row0 = tile_row0; a.tile_rows = tile_rows; a.n_list = n_list;
   a.w_rows = (int)N;
   a.err = c->core->dev_err;

@@ -68,6 +68,21 @@ struct RopeStoreArgs {
 // to the cache.
 int k_launch_rope_store(cg_ctx* c, const RopeStoreArgs& a);
 
+// A batch of rows of unequal length: row r brings the next tokens of the sequence in slot[r], packed
+// row after row, so token m of the batch belongs to row tok_row[m].
+struct RowsDev {
+  const int32_t* slot = nullptr;     // [rows] where the row's cache and state live
+  const int32_t* start = nullptr;    // [rows + 1] first packed token of the row
+  const int32_t* pos0 = nullptr;     // [rows] position of its first token when *step was 0
+  const int32_t* tok_row = nullptr;  // [M]
+  const int64_t* step = nullptr;     // decode steps taken since the tables were written
+  int rows = 0;                      // 0: the caller gives equal rows by other means
+  int64_t M = 0;
+};
+#ifdef __CUDACC__
+__device__ __forceinline__ int64_t row_pos0(const RowsDev& r, int row) { return r.pos0[row] + *r.step; }
+#endif
+
 struct AttnArgs {
   const __nv_bfloat16* q;        // [B * S, nh d]
   const __nv_bfloat16* k_cache;  // [B, nkv, Tmax, d]
@@ -83,12 +98,16 @@ struct AttnArgs {
   // k_cache + (b * Tmax + t) * kv_ld + h * d (Tmax = tokens per row)
   int64_t kv_ld = 0;
   float scale = 0.f;             // factor on the scores; 0 = 1 / sqrt(d)
+  const float* sink = nullptr;   // [nh]: exp(sink[h]) joins the denominator of the softmax
+  // rows.rows > 0: rows of unequal length, at most S tokens each, of a batch of rows.M tokens; q and out
+  // are packed, the cache is [slots, nkv, Tmax, d] and B counts the slots (pos0 is unused)
+  RowsDev rows;
 };
 // Causal (optionally windowed / soft-capped) attention of S new tokens per row against cache
 // positions [0, pos0 + S).  Tensor-core flash kernel.
 int k_launch_attn_prefill(cg_ctx* c, const AttnArgs& a);
 
-// The same on tcgen05 / TMEM for head sizes 64 and 128 without soft-cap or window (attention_fa.cu);
+// The same on tcgen05 / TMEM for head sizes 64 and 128 without soft-cap (attention_fa.cu);
 // k_launch_attn_prefill routes here by itself when the context allows it.
 bool attn_fa_supported(const AttnArgs& a);
 int k_launch_attn_fa(cg_ctx* c, const AttnArgs& a);
@@ -110,6 +129,14 @@ struct AttnDecArgs {
   int64_t window;                // 0 = none
   float softcap;                 // 0 = none
   int splits;                    // grid z = cluster size: context slices per (row, kv head)
+  // rows.rows > 0: row b is one token of the sequence in a slot at its own position (B = rows.rows, pos0
+  // and pos_dev are unused), the first rot_dims components are rotated in neighbouring pairs (tables
+  // [Tmax, rot_dims / 2]), and the gains, if any, are those of norms over all query and all key heads
+  // at once ([nh d] and [nkv d] values, of which nh and nkv times norm_dim count for the mean)
+  RowsDev rows;
+  int rot_dims = 0, norm_dim = 0;
+  float scale = 0.f;             // factor on the scores; 0 = 1 / sqrt(d)
+  const float* sink = nullptr;   // [nh]: exp(sink[h]) joins the denominator of the softmax
   int push_merge;                // set by the launcher: the slices' partials are pushed to the finishing CTA
 };
 // Rope + cache append + attention + merge of one new token per row, in one launch.
@@ -167,6 +194,7 @@ struct DecGemm {
   const float* residual;
   int out_mode;             // 0: f32, 1: bf16, 2: f32 out = product + residual,
                             // 3: the product is pushed as this rank's addend of an all-reduce (out unused)
+                            // 4: bf16, the square of relu
   const PeerPush* push;     // for out_mode 3
   // Norm hand-over between consecutive GEMMs (RMSNorm(x) W^T = (x g) W^T / rms(x) row by row):
   // a residual GEMM (out_mode 2) that is followed by a norm can also write xb_out = bf16(out * g)
@@ -211,6 +239,10 @@ struct MoeArgs {
   float* logits;              // [M, E] scratch for router3
   const __nv_bfloat16 *w_gate, *w_up;  // [El, Fe, H] experts this rank owns
   const __nv_bfloat16* w_down;         // [El, H, Fe]
+  const float* correction = nullptr;  // [E]: experts are chosen by probability + correction and weighted by
+                              // probability * router_scale
+  float router_scale = 1.f;
+  float act_limit = 0.f;      // of the bounded activation
   int H, E, k, Fe, norm_topk, act;
   int e_lo, El;               // this rank owns experts [e_lo, e_lo + El)
   int add_residual;           // 1: out = x + expert sum; 0: out = this rank's expert sum only
@@ -221,6 +253,15 @@ struct MoeArgs {
   MoeWork w;
 };
 int moe_ffn(cg_ctx* c, const MoeArgs& a);
+// The parts, for callers with normed rows (a.xn) and router logits (a.logits): ids and weights; then the
+// experts' results, a.w.y[a.w.pos[pair]] (the weighted sum is the caller's).
+int moe_topk(cg_ctx* c, const MoeArgs& a);
+int moe_experts(cg_ctx* c, const MoeArgs& a);
+// The latter in f32 (h [pairs, Fe]; a.w.xg holds [pairs] words)
+int moe_experts_f32(cg_ctx* c, const MoeArgs& a, const float* x, const float* w_gate, const float* w_up, const float* w_down, float* h);
+// out[M, N] = x[M, K] w[N, K]^T in f32 (CUDA cores)
+int gemm_nt_f32(cg_ctx* c, const float* x, int64_t ldx, const float* w, int64_t ldw, float* out, int64_t ldo, int64_t M, int64_t N,
+                int64_t K);
 int moe_pick_tn(int64_t pairs, int experts);
 int64_t moe_max_tiles(int64_t pairs, int experts_local, int tn);
 

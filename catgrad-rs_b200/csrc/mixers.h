@@ -1,28 +1,12 @@
 // mixers.h — launchers of the kernels that decoders built layer by layer use beside the GEMMs
 // (decoder_mixed.cu): the residual-stream update, latent attention (latent.cu) and the linear
 // recurrences with short convolutions (recurrent.cu).
-//
-// A batch is a set of rows of unequal length: row r brings the next tokens of the sequence in
-// slot[r], packed row after row, so token m of the batch belongs to row tok_row[m].
+// Batches are rows of unequal length (RowsDev, kernels.h).
 #pragma once
 
 #include "kernels.h"
 
 namespace cg {
-
-struct RowsDev {
-  const int32_t* slot;     // [rows] where the row's cache and state live
-  const int32_t* start;    // [rows + 1] first packed token of the row
-  const int32_t* pos0;     // [rows] position of its first token when *step was 0
-  const int32_t* tok_row;  // [M]
-  const int64_t* step;     // decode steps taken since the tables were written
-  int rows;
-  int64_t M;
-};
-
-#ifdef __CUDACC__
-__device__ __forceinline__ int64_t row_pos0(const RowsDev& r, int row) { return r.pos0[row] + *r.step; }
-#endif
 
 // One pass over the residual stream, row by row:
 //   src  = table[tokens[m]]            (tokens set)
@@ -54,14 +38,78 @@ struct RowUpdate {
 };
 int k_launch_row_update(cg_ctx* c, const RowUpdate& u, int64_t M, int out_bf16);
 
-// out[M, N] = x[M, K] w[N, K]^T in f32 (CUDA cores)
-int gemm_nt_f32(cg_ctx* c, const float* x, int64_t ldx, const float* w, int64_t ldw, float* out, int64_t ldo, int64_t M, int64_t N,
-                int64_t K);
+// The same for hyper-connected models, whose residual stream is ns rows per token: x is [M, ns, ldx].
+//   y    = y[m] | sum over the token's experts i of wts[m top + i] y[pos[m top + i]]   (top > 0)
+//   x[t] = sum over s of mix[s, t] x[s] + out_w[t] y
+// or, with tokens set, every x[t] = scale * table[tokens[m]].  Then
+//   h    = sum over s of in_w[s] x[s]                (in_w null: all ones)
+//   out  = rms(h) * g                                (out set)
+//   sum[m] = sum over s of x[s]                      (sum set)
+// With pick set, x is read only: out[dst[m]] = rms(sum of x[pick[m]]) * g.
+// A plain residual stream is ns = 1 with mix = out_w = in_w = 1.
+constexpr int MAX_STREAMS = 16;
+struct StreamUpdate {
+  const uint32_t* tokens = nullptr;
+  const void* table = nullptr;
+  int table_bf16 = 0;
+  int64_t vocab = 0;
+  float scale = 1.f;
+  const float* y = nullptr;
+  int64_t ldy = 0;
+  const int32_t* pos = nullptr;
+  const float* wts = nullptr;
+  int top = 0;
+  int ns = 1;
+  const float *mix = nullptr, *out_w = nullptr, *in_w = nullptr;
+  float* x = nullptr;
+  int64_t ldx = 0;
+  const float* g = nullptr;
+  void* out = nullptr;
+  int64_t ldo = 0;
+  float* sum = nullptr;
+  int64_t ld_sum = 0;
+  const int32_t* pick = nullptr;
+  const int32_t* dst = nullptr;
+  float eps = 0.f;
+  int W = 0;  // row length; columns up to the next multiple of 8 are kept zero
+};
+int k_launch_stream_update(cg_ctx* c, const StreamUpdate& u, int64_t M, int out_bf16);
+
+// x[i] += v
+int k_launch_add_scalar(cg_ctx* c, float* x, int64_t n, float v);
+// x[i] = max(x[i], 0)^2 in f32
+int k_launch_relu2_f32(cg_ctx* c, float* x, int64_t n);
+
 // out[m, i] = act(gu[m, i]) * gu[m, F + i] in f32
 int k_launch_glu_f32(cg_ctx* c, const float* gu, int64_t M, int64_t F, int act, float* out);
 
 // Rotary tables cos, sin [T, r / 2] of angles p * base^(-2 i / r), evaluated in double precision
 int k_launch_pair_rope_tables(cg_ctx* c, double base, int64_t T, int r, float* cos_t, float* sin_t);
+
+// ------------------------------------------------------------- attention over a row batch ----
+// Grouped-query attention with per-layer sizes, window and sink on rows of unequal length.  Heads take
+// Dk (queries, keys) and Dv (values) columns in the projection, the cache and the output, of which d
+// and dv are real and the rest zero.
+struct RowsAttnArgs {
+  const float* proj;       // [M, ldp]: H query heads, G key heads, G value heads
+  int64_t ldp;
+  int H, G, d, dv, Dk, Dv;
+  const float *q_gain, *k_gain;  // [H Dk], [G Dk]: norms over all query / key heads at once; null: none
+  float eps, scale;
+  int rot;                 // rotated components, neighbouring pairs
+  const float *cos_t, *sin_t;    // [Tmax, rot / 2]
+  int64_t window;          // 0 = none
+  const float* sink;       // [H] or null
+  void* q;                 // [M, H Dk]
+  void *k_cache, *v_cache; // [slots, G, Tmax, Dk | Dv]
+  int64_t Tmax, slots;
+  void* att;               // [M, ld_att], head h at column h * Dv
+  int64_t ld_att;
+  int bf16;                // element type of q, the cache and att
+  RowsDev rows;
+};
+int k_launch_rows_qkv(cg_ctx* c, const RowsAttnArgs& a);   // norms, rotation, q, cache append
+int k_launch_rows_attn(cg_ctx* c, const RowsAttnArgs& a);  // any sizes; one CTA per (token, head)
 
 // ------------------------------------------------------------------ latent attention ----
 // A cached row is [c (R values), rotated key part (r), zeros up to Lw].  Per head the key is

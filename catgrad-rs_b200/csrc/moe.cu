@@ -187,15 +187,19 @@ __global__ void k_moe_norm_split(float* x, const float* gamma, float eps, int pl
 }
 
 // One warp per token: softmax over the router logits, top-k (ties -> lower expert id),
-// optional renormalisation.  Dynamic shared memory: E floats per warp.
-__global__ void k_moe_topk(const float* logits, int64_t M, int E, int k, int norm_topk, uint32_t* ids, float* wts) {
+// optional renormalisation.  With `correction` [E] the experts are chosen by probability + correction
+// and weighted by probability * scale.  Dynamic shared memory: E floats per warp, 2 E with correction.
+constexpr uint32_t TAKEN = 0xFFFFFFFFu;  // a chosen expert's mark (a NaN no sum here produces)
+__global__ void k_moe_topk(const float* logits, int64_t M, int E, int k, int norm_topk, const float* correction, float scale,
+                           uint32_t* ids, float* wts) {
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
   asm volatile("griddepcontrol.wait;" ::: "memory");
   extern __shared__ float sm[];
   const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5, nw = blockDim.x >> 5;
   const int64_t m = (int64_t)blockIdx.x * nw + wid;
   if (m >= M) return;
-  float* pr = sm + (size_t)wid * E;
+  float* pr = sm + (size_t)wid * E * (correction ? 2 : 1);
+  float* ch = correction ? pr + E : pr;  // what the choice goes by
   const float* lg = logits + m * E;
   float mx = -3.4028234663852886e38f;
   for (int e = lane; e < E; e += 32) {
@@ -212,32 +216,38 @@ __global__ void k_moe_topk(const float* logits, int64_t M, int E, int k, int nor
   }
   for (int o = 16; o; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
   __syncwarp();
-  for (int e = lane; e < E; e += 32) pr[e] = pr[e] / sum;
+  for (int e = lane; e < E; e += 32) {
+    pr[e] = pr[e] / sum;
+    if (correction) ch[e] = pr[e] + correction[e];
+  }
   __syncwarp();
   float chosen = 0.f, total = 0.f;
   uint32_t chosen_id = 0;
   for (int r = 0; r < k; ++r) {
     unsigned long long best = 0;
     for (int e = lane; e < E; e += 32) {
-      const float v = pr[e];
-      if (v < 0.f) continue;
-      const unsigned long long q = ((unsigned long long)__float_as_uint(v) << 32) | (uint32_t)(0xFFFFFFFFu - (uint32_t)e);
+      const uint32_t u = __float_as_uint(ch[e]);
+      if (u == TAKEN) continue;
+      // unsigned order = float order, whatever the signs
+      const uint32_t key = u & 0x80000000u ? ~u : u | 0x80000000u;
+      const unsigned long long q = ((unsigned long long)key << 32) | (uint32_t)(0xFFFFFFFFu - (uint32_t)e);
       best = q > best ? q : best;
     }
     for (int o = 16; o; o >>= 1) {
       const unsigned long long w = __shfl_xor_sync(0xffffffffu, best, o);
       best = w > best ? w : best;
     }
-    const uint32_t e = 0xFFFFFFFFu - (uint32_t)(best & 0xFFFFFFFFull);
-    const float v = __uint_as_float((uint32_t)(best >> 32));
-    if (lane == r) { chosen = v; chosen_id = e; }
-    if (lane == 0) pr[e] = -1.f;
+    const uint32_t e = min(0xFFFFFFFFu - (uint32_t)(best & 0xFFFFFFFFull), (uint32_t)E - 1u);
+    if (lane == r) { chosen = pr[e]; chosen_id = e; }
+    __syncwarp();
+    if (lane == 0) ch[e] = __uint_as_float(TAKEN);
     __syncwarp();
   }
   total = sum_in_reference_order(chosen, k);  // bit-identical to the reference's sum over the k values
   if (lane < k) {
     ids[m * k + lane] = chosen_id;
-    wts[m * k + lane] = norm_topk ? chosen / total : chosen;
+    const float w = norm_topk ? chosen / total : chosen;
+    wts[m * k + lane] = correction ? w * scale : w;
   }
 }
 
@@ -367,6 +377,7 @@ struct MoeGemmArgs {
   int w_rows;      // rows one expert occupies in the stacked weight matrix
   int kb_total;
   int act;
+  float limit;     // of the bounded activation
   int32_t* err;
 };
 
@@ -502,7 +513,7 @@ k_moe_gemm(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CU
           for (int j = 0; j < 16; ++j) {
             if (c0 + j >= rows) break;
             const float a = __uint_as_float(g[j]);
-            const float h = (p.act == 0 ? silu_f(a) : gelu_f(a)) * __uint_as_float(u[j]);
+            const float h = glu_f(p.act, p.limit, a, __uint_as_float(u[j]));
             ((__nv_bfloat16*)p.out)[(int64_t)(row0 + c0 + j) * p.ldo + n] = __float2bfloat16_rn(h);
           }
         }
@@ -525,6 +536,78 @@ k_moe_gemm(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CU
     __syncwarp();
     asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem_acc), "r"(NCOLS) : "memory");
   }
+}
+
+// ------------------------------------------------------------- f32 form (CUDA cores) ----
+constexpr int MF_ROWS = 32, MF_COLS = 64, MF_K = 32;
+
+// src[pos[p]] = p / k
+__global__ void k_moe_sources(const int32_t* pos, int64_t P, int k, int32_t* src) {
+  asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+  asm volatile("griddepcontrol.wait;" ::: "memory");
+  for (int64_t p = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; p < P; p += (int64_t)gridDim.x * blockDim.x)
+    if (pos[p] >= 0) src[pos[p]] = (int32_t)(p / k);
+}
+
+struct MoeF32Args {
+  const int32_t *tile_expert, *tile_row0, *tile_rows, *n_tiles;
+  const float* x;         // [.., K]
+  const int32_t* src;     // row of x each grouped row reads; null: the row itself
+  const float *w, *w_up;  // [experts, N, K]; w_up null: a plain product
+  float* out;             // [grouped rows, N]
+  int N, K, act;
+  float limit;
+};
+// One block per (64 output features, tile of the list); a thread holds 4 rows x 2 features.
+__global__ void __launch_bounds__(256) k_moe_gemm_f32(MoeF32Args p) {
+  asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+  asm volatile("griddepcontrol.wait;" ::: "memory");
+  const int t = blockIdx.y;
+  if (t >= *p.n_tiles) return;
+  __shared__ float xs[MF_K][MF_ROWS + 1], ws[MF_K][MF_COLS + 1], us[MF_K][MF_COLS + 1];
+  const int row0 = p.tile_row0[t], rows = p.tile_rows[t], n0 = blockIdx.x * MF_COLS;
+  const int64_t wbase = (int64_t)p.tile_expert[t] * p.N;
+  const int tc = threadIdx.x & 31, tr = threadIdx.x >> 5;
+  float g[4][2] = {}, u[4][2] = {};
+  for (int k0 = 0; k0 < p.K; k0 += MF_K) {
+    const int k = k0 + tc;
+    for (int r = tr; r < MF_ROWS; r += 8) {
+      const int64_t row = row0 + r;
+      xs[tc][r] = r < rows && k < p.K ? p.x[(p.src ? (int64_t)p.src[row] : row) * p.K + k] : 0.f;
+    }
+    for (int r = tr; r < MF_COLS; r += 8) {
+      const bool in = n0 + r < p.N && k < p.K;
+      ws[tc][r] = in ? p.w[(wbase + n0 + r) * p.K + k] : 0.f;
+      us[tc][r] = in && p.w_up ? p.w_up[(wbase + n0 + r) * p.K + k] : 0.f;
+    }
+    __syncthreads();
+    for (int kk = 0; kk < MF_K; ++kk) {
+      const float w0 = ws[kk][tc], w1 = ws[kk][tc + 32], u0 = us[kk][tc], u1 = us[kk][tc + 32];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float x = xs[kk][tr * 4 + i];
+        g[i][0] += x * w0; g[i][1] += x * w1;
+        u[i][0] += x * u0; u[i][1] += x * u1;
+      }
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      const int r = tr * 4 + i, n = n0 + tc + 32 * j;
+      if (r < rows && n < p.N) {
+        float v = g[i][j];
+        if (p.w_up) {
+          if (p.act == ACT_BOUNDED) {
+            const float gg = fminf(v, p.limit), uu = fminf(fmaxf(u[i][j], -p.limit), p.limit);
+            v = gg / (1.f + expf(-1.702f * gg)) * (uu + 1.f);
+          } else v = glu_f(p.act, 0.f, v, u[i][j]);
+        }
+        p.out[(int64_t)(row0 + r) * p.N + n] = v;
+      }
+    }
 }
 
 template <int TN, int DUAL, int STAGES, int MINB>
@@ -567,17 +650,54 @@ int64_t moe_max_tiles(int64_t pairs, int experts_local, int tn) {
   return std::max<int64_t>(1, std::min<int64_t>(pairs, pairs / tn + experts_local));
 }
 
+static int check_moe(cg_ctx* c, const MoeArgs& a) {
+  if (a.k < 1 || a.k > 32 || a.k > a.E) return fail(c, CG_ERR_UNSUPPORTED, "moe: experts per token must be in [1, 32]");
+  if (a.E > 1024 || a.H % 8 || a.Fe % 8) return fail(c, CG_ERR_UNSUPPORTED, "moe: sizes must be multiples of 8, at most 1024 experts");
+  if (a.M * a.k > 2147483647ll / 4) return fail(c, CG_ERR_UNSUPPORTED, "moe: too many (token, expert) pairs");
+  return CG_OK;
+}
+
+// logits[M, E] = x w^T with a bf16 router matrix
+static int router_logits(cg_ctx* c, const MoeArgs& a, const __nv_bfloat16* x, const __nv_bfloat16* w, int64_t K) {
+  if (gemm_dec_supported(a.M, K)) {
+    DecGemm g;
+    g.x = x; g.ldx = K; g.w = w; g.ldw = K; g.w_rows = a.E;
+    g.out = a.logits; g.ldo = a.E; g.residual = nullptr; g.out_mode = 0; g.push = nullptr; g.dual = 0; g.act = 0;
+    g.M = a.M; g.N = a.E; g.K = K;
+    return gemm_dec(c, g);
+  }
+  return gemm_tc(c, x, K, w, K, a.logits, a.E, nullptr, a.M, a.E, K, 0, 0, nullptr);
+}
+
+static int launch_topk(cg_ctx* c, const MoeArgs& a) {
+  const int warps = 4;
+  const size_t smem = (size_t)warps * a.E * (a.correction ? 8 : 4);
+  CG_CUDA(c, launch_kernel(c, k_moe_topk, dim3((unsigned)((a.M + warps - 1) / warps)), dim3(32 * warps), smem, 1,
+                           (const float*)a.logits, a.M, a.E, a.k, a.norm_topk, a.correction, a.router_scale, a.w.ids, a.w.wts));
+  CG_LAUNCHED(c);
+  return CG_OK;
+}
+
+static int launch_plan(cg_ctx* c, const MoeArgs& a, int tn) {
+  const int64_t P = a.M * a.k;
+  // one thread per local expert is the minimum; more threads only help the histogram of a long prompt
+  const unsigned threads = P > 4096 ? 1024u : (unsigned)std::max(128, (a.El + 31) / 32 * 32);
+  CG_CUDA(c, launch_kernel(c, k_moe_plan, dim3(1), dim3(threads), (size_t)a.El * 8, 1, (const uint32_t*)a.w.ids, (int)P, a.e_lo,
+                           a.El, tn, a.w.pos, a.w.tile_expert, a.w.tile_row0, a.w.tile_rows, a.w.n_tiles));
+  CG_LAUNCHED(c);
+  return CG_OK;
+}
+
+int moe_topk(cg_ctx* c, const MoeArgs& a) {
+  if (a.M == 0) return CG_OK;
+  CG_TRY(check_moe(c, a));
+  return launch_topk(c, a);
+}
+
 int moe_ffn(cg_ctx* c, const MoeArgs& a) {
   if (a.M == 0) return CG_OK;
-  if (a.k < 1 || a.k > 32 || a.k > a.E) return fail(c, CG_ERR_UNSUPPORTED, "moe: experts per token must be in [1, 32]");
+  CG_TRY(check_moe(c, a));
   if (a.push && !a.router3) return fail(c, CG_ERR_INVALID, "moe: the pushed reduction needs the bf16 router path");
-  if (a.E > 1024 || a.H % 8 || a.Fe % 8) return fail(c, CG_ERR_UNSUPPORTED, "moe: sizes must be multiples of 8, at most 1024 experts");
-  const int64_t P = a.M * a.k;
-  if (P > 2147483647ll / 4) return fail(c, CG_ERR_UNSUPPORTED, "moe: too many (token, expert) pairs");
-  const int tn = moe_pick_tn(P, a.E);
-  const int64_t max_tiles = moe_max_tiles(P, a.El, tn);
-  if (max_tiles > 65535) return fail(c, CG_ERR_UNSUPPORTED, "moe: too many tiles");
-
   if (a.router3) {
     if (a.push)
       CG_CUDA(c, launch_kernel(c, k_moe_norm_split<1>, dim3((unsigned)a.M), dim3(256), 0, 1, a.out, a.gamma, a.eps, a.plus_one, a.H,
@@ -586,20 +706,8 @@ int moe_ffn(cg_ctx* c, const MoeArgs& a) {
       CG_CUDA(c, launch_kernel(c, k_moe_norm_split<0>, dim3((unsigned)a.M), dim3(256), 0, 1, const_cast<float*>(a.x), a.gamma, a.eps,
                                a.plus_one, a.H, a.xn, a.xs3, PeerPush{}, c->core->dev_err));
     CG_LAUNCHED(c);
-    const int64_t K3 = 3 * (int64_t)a.H;
-    if (gemm_dec_supported(a.M, K3)) {
-      DecGemm g;
-      g.x = a.xs3; g.ldx = K3; g.w = a.router3; g.ldw = K3; g.w_rows = a.E;
-      g.out = a.logits; g.ldo = a.E; g.residual = nullptr; g.out_mode = 0; g.push = nullptr; g.dual = 0; g.act = 0;
-      g.M = a.M; g.N = a.E; g.K = K3;
-      CG_TRY(gemm_dec(c, g));
-    } else {
-      CG_TRY(gemm_tc(c, a.xs3, K3, a.router3, K3, a.logits, a.E, nullptr, a.M, a.E, K3, 0, 0, nullptr));
-    }
-    const int warps = 4;
-    CG_CUDA(c, launch_kernel(c, k_moe_topk, dim3((unsigned)((a.M + warps - 1) / warps)), dim3(32 * warps),
-                             (size_t)warps * a.E * 4, 1, (const float*)a.logits, a.M, a.E, a.k, a.norm_topk, a.w.ids, a.w.wts));
-    CG_LAUNCHED(c);
+    CG_TRY(router_logits(c, a, a.xs3, a.router3, 3 * (int64_t)a.H));
+    CG_TRY(launch_topk(c, a));
   } else {
     const size_t smem = (size_t)(a.H + a.E) * 4;
     static PerDeviceSize configured_on;
@@ -612,11 +720,18 @@ int moe_ffn(cg_ctx* c, const MoeArgs& a) {
                              a.H, a.E, a.k, a.norm_topk, a.xn, a.w.ids, a.w.wts));
     CG_LAUNCHED(c);
   }
-  // one thread per local expert is the minimum; more threads only help the histogram of a long prompt
-  const unsigned plan_threads = P > 4096 ? 1024u : (unsigned)std::max(128, (a.El + 31) / 32 * 32);
-  CG_CUDA(c, launch_kernel(c, k_moe_plan, dim3(1), dim3(plan_threads), (size_t)a.El * 8, 1, (const uint32_t*)a.w.ids, (int)P, a.e_lo,
-                           a.El, tn, a.w.pos, a.w.tile_expert, a.w.tile_row0, a.w.tile_rows, a.w.n_tiles));
-  CG_LAUNCHED(c);
+  CG_TRY(moe_experts(c, a));
+  return launch_combine(c, a);
+}
+
+int moe_experts(cg_ctx* c, const MoeArgs& a) {
+  if (a.M == 0) return CG_OK;
+  CG_TRY(check_moe(c, a));
+  const int64_t P = a.M * a.k;
+  const int tn = moe_pick_tn(P, a.E);
+  const int64_t max_tiles = moe_max_tiles(P, a.El, tn);
+  if (max_tiles > 65535) return fail(c, CG_ERR_UNSUPPORTED, "moe: too many tiles");
+  CG_TRY(launch_plan(c, a, tn));
   CG_CUDA(c, launch_kernel(c, k_moe_gather, dim3(grid_for(P * (a.H / 8), 256)), dim3(256), 0, 1, (const __nv_bfloat16*)a.xn,
                            (const int32_t*)a.w.pos, P, a.k, a.H, a.w.xg));
   CG_LAUNCHED(c);
@@ -627,6 +742,7 @@ int moe_ffn(cg_ctx* c, const MoeArgs& a) {
   g.tile_rows = a.w.tile_rows;
   g.n_tiles = a.w.n_tiles;
   g.act = a.act;
+  g.limit = a.act_limit;
   g.err = c->core->dev_err;
   CUtensorMap mw, mu, mx;
   // gate / up: h[P, Fe] = act(xg Wg^T) * (xg Wu^T)
@@ -637,11 +753,10 @@ int moe_ffn(cg_ctx* c, const MoeArgs& a) {
   dim3 grid((unsigned)((a.Fe + BM - 1) / BM), (unsigned)max_tiles);
   if (tn == 128 && c->opt_persistent) {
     // many rows per expert: the persistent kernel (epilogue overlapped with the next tile)
-    CG_TRY(gemm_tcp_grouped(c, a.w.xg, P, a.w_gate, a.w_up, a.El, a.w.h, a.Fe, a.H, 1, a.act, a.w.tile_expert, a.w.tile_row0,
-                            a.w.tile_rows, a.w.n_tiles, max_tiles));
-    CG_TRY(gemm_tcp_grouped(c, a.w.h, P, a.w_down, nullptr, a.El, a.w.y, a.H, a.Fe, 0, 0, a.w.tile_expert, a.w.tile_row0,
-                            a.w.tile_rows, a.w.n_tiles, max_tiles));
-    return launch_combine(c, a);
+    CG_TRY(gemm_tcp_grouped(c, a.w.xg, P, a.w_gate, a.w_up, a.El, a.w.h, a.Fe, a.H, 1, a.act, a.act_limit, a.w.tile_expert,
+                            a.w.tile_row0, a.w.tile_rows, a.w.n_tiles, max_tiles));
+    return gemm_tcp_grouped(c, a.w.h, P, a.w_down, nullptr, a.El, a.w.y, a.H, a.Fe, 0, 0, 0.f, a.w.tile_expert, a.w.tile_row0,
+                            a.w.tile_rows, a.w.n_tiles, max_tiles);
   }
   switch (tn) {
     case 16: CG_TRY((launch_moe_gemm<16, 1, 3, 2>(c, mw, mu, mx, g, grid))); break;
@@ -660,7 +775,29 @@ int moe_ffn(cg_ctx* c, const MoeArgs& a) {
     case 64: CG_TRY((launch_moe_gemm<64, 0, 4, 2>(c, mw, mw, mx, g, grid))); break;
     default: CG_TRY((launch_moe_gemm<128, 0, 6, 1>(c, mw, mw, mx, g, grid))); break;
   }
-  return launch_combine(c, a);
+  return CG_OK;
+}
+
+int moe_experts_f32(cg_ctx* c, const MoeArgs& a, const float* x, const float* w_gate, const float* w_up, const float* w_down, float* h) {
+  if (a.M == 0) return CG_OK;
+  CG_TRY(check_moe(c, a));
+  CG_TRY(launch_plan(c, a, MF_ROWS));
+  const int64_t P = a.M * a.k, tiles = moe_max_tiles(P, a.El, MF_ROWS);
+  if (tiles > 65535) return fail(c, CG_ERR_UNSUPPORTED, "moe: too many tiles");
+  // rows in grouped order: which token each reads
+  CG_CUDA(c, launch_kernel(c, k_moe_sources, dim3(grid_for(P, 256)), dim3(256), 0, 1, (const int32_t*)a.w.pos, P, a.k, (int32_t*)a.w.xg));
+  CG_LAUNCHED(c);
+  MoeF32Args g;
+  g.tile_expert = a.w.tile_expert; g.tile_row0 = a.w.tile_row0; g.tile_rows = a.w.tile_rows; g.n_tiles = a.w.n_tiles;
+  g.x = x; g.src = (const int32_t*)a.w.xg; g.w = w_gate; g.w_up = w_up; g.out = h;
+  g.N = a.Fe; g.K = a.H; g.act = a.act; g.limit = a.act_limit;
+  CG_CUDA(c, launch_kernel(c, k_moe_gemm_f32, dim3((unsigned)((g.N + MF_COLS - 1) / MF_COLS), (unsigned)tiles), dim3(256), 0, 1, g));
+  CG_LAUNCHED(c);
+  g.x = h; g.src = nullptr; g.w = w_down; g.w_up = nullptr; g.out = a.w.y;
+  g.N = a.H; g.K = a.Fe;
+  CG_CUDA(c, launch_kernel(c, k_moe_gemm_f32, dim3((unsigned)((g.N + MF_COLS - 1) / MF_COLS), (unsigned)tiles), dim3(256), 0, 1, g));
+  CG_LAUNCHED(c);
+  return CG_OK;
 }
 
 }  // namespace cg

@@ -1,0 +1,179 @@
+// rows_attn.cu — grouped-query attention on rows of unequal length: norms over all heads of the
+// queries and of the keys, rotation of neighbouring pairs and the cache append in one pass, and the
+// attention of sizes (and of the f32 form) that the tensor-core kernels do not have.  Prompts in bf16
+// take attention_fa.cu / attention.cu, decode steps attn_decode.cu.
+#include <algorithm>
+
+#include "mixers.h"
+
+namespace cg {
+
+namespace {
+
+__device__ __forceinline__ float warp_sum(float v) {
+#pragma unroll
+  for (int o = 16; o; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+  return v;
+}
+__device__ __forceinline__ float warp_max(float v) {
+#pragma unroll
+  for (int o = 16; o; o >>= 1) v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, o));
+  return v;
+}
+__device__ __forceinline__ float block_sum(float v, float* sh) {
+  const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  v = warp_sum(v);
+  __syncthreads();
+  if (lane == 0) sh[wid] = v;
+  __syncthreads();
+  v = lane < nw ? sh[lane] : 0.f;
+  return warp_sum(v);
+}
+__device__ __forceinline__ float block_max(float v, float* sh) {
+  const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  v = warp_max(v);
+  __syncthreads();
+  if (lane == 0) sh[wid] = v;
+  __syncthreads();
+  v = lane < nw ? sh[lane] : -INFINITY;
+  return warp_max(v);
+}
+__device__ __forceinline__ float ld(const float* p) { return *p; }
+__device__ __forceinline__ float ld(const __nv_bfloat16* p) { return __bfloat162float(*p); }
+__device__ __forceinline__ void st(float* p, float v) { *p = v; }
+__device__ __forceinline__ void st(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
+__device__ __forceinline__ void st4(float* p, float4 v) { *(float4*)p = v; }
+__device__ __forceinline__ void st4(__nv_bfloat16* p, float4 v) {
+  const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+  *(uint2*)p = make_uint2(*(const uint32_t*)&lo, *(const uint32_t*)&hi);
+}
+
+// One block per token; Dk and Dv are multiples of 8, so four neighbours belong to one head.
+template <class T>
+__global__ void __launch_bounds__(256) k_rows_qkv(RowsAttnArgs a) {
+  asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+  asm volatile("griddepcontrol.wait;" ::: "memory");
+  __shared__ float sh[32];
+  const int64_t m = blockIdx.x;
+  const int row = a.rows.tok_row[m];
+  const int64_t pos = row_pos0(a.rows, row) + (m - a.rows.start[row]);
+  const int64_t slot = a.rows.slot[row];
+  const float* p = a.proj + m * a.ldp;
+  const int nq = a.H * a.Dk, nk = a.G * a.Dk, n_v = a.G * a.Dv;
+  float fq = 1.f, fk = 1.f;
+  if (a.q_gain) {
+    float sq = 0.f, sk = 0.f;
+    for (int i = 4 * threadIdx.x; i < nq + nk; i += 4 * blockDim.x) {
+      const float4 v = *(const float4*)(p + i);
+      const float s = v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+      if (i < nq) sq += s;
+      else sk += s;
+    }
+    fq = 1.f / sqrtf(block_sum(sq, sh) / (float)(a.H * a.d) + a.eps);
+    fk = 1.f / sqrtf(block_sum(sk, sh) / (float)(a.G * a.d) + a.eps);
+  }
+  const int half = a.rot / 2;
+  const float* ct = a.cos_t + pos * half;
+  const float* sn = a.sin_t + pos * half;
+  for (int i = 4 * threadIdx.x; i < nq + nk + n_v; i += 4 * blockDim.x) {
+    float4 v = *(const float4*)(p + i);
+    if (i >= nq + nk) {
+      const int j = i - nq - nk, g = j / a.Dv;
+      st4((T*)a.v_cache + ((slot * a.G + g) * a.Tmax + pos) * a.Dv + (j - g * a.Dv), v);
+      continue;
+    }
+    const bool is_q = i < nq;
+    const int j = is_q ? i : i - nq, h = j / a.Dk, e = j - h * a.Dk;
+    if (a.q_gain) {
+      const float f = is_q ? fq : fk;
+      const float4 w = *(const float4*)((is_q ? a.q_gain : a.k_gain) + j);
+      v = make_float4(v.x * (f * w.x), v.y * (f * w.y), v.z * (f * w.z), v.w * (f * w.w));
+    }
+    const int k = e >> 1;
+    if (k < half) v = make_float4(v.x * ct[k] - v.y * sn[k], v.y * ct[k] + v.x * sn[k], v.z, v.w);
+    if (k + 1 < half) v = make_float4(v.x, v.y, v.z * ct[k + 1] - v.w * sn[k + 1], v.w * ct[k + 1] + v.z * sn[k + 1]);
+    if (is_q) st4((T*)a.q + m * nq + i, v);
+    else st4((T*)a.k_cache + ((slot * a.G + h) * a.Tmax + pos) * a.Dk + e, v);
+  }
+}
+
+// One block per (token, head): an online softmax over tiles of the visible keys.
+template <class T>
+__global__ void __launch_bounds__(128) k_rows_attn(RowsAttnArgs a) {
+  asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+  asm volatile("griddepcontrol.wait;" ::: "memory");
+  constexpr int KT = 64;
+  extern __shared__ float sm[];
+  float* q = sm;          // [Dk]
+  float* o = q + a.Dk;    // [Dv]
+  float* s = o + a.Dv;    // [KT]
+  float* sh = s + KT;     // [32]
+  const int64_t m = blockIdx.x;
+  const int h = blockIdx.y, g = h / (a.H / a.G);
+  const int row = a.rows.tok_row[m];
+  const int64_t pos = row_pos0(a.rows, row) + (m - a.rows.start[row]);
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, nw = blockDim.x >> 5;
+  for (int i = tid; i < a.Dk; i += blockDim.x) q[i] = ld((const T*)a.q + (m * a.H + h) * a.Dk + i);
+  for (int i = tid; i < a.Dv; i += blockDim.x) o[i] = 0.f;
+  __syncthreads();
+  const int64_t base = ((int64_t)a.rows.slot[row] * a.G + g) * a.Tmax;
+  const T* kb = (const T*)a.k_cache + base * a.Dk;
+  const T* vb = (const T*)a.v_cache + base * a.Dv;
+  const int64_t lo = a.window > 0 ? max((int64_t)0, pos - a.window + 1) : 0;
+  // the sink is a term of the sum before any key
+  float mx = a.sink ? a.sink[h] : -INFINITY, l = a.sink ? 1.f : 0.f;
+  for (int64_t k0 = lo; k0 <= pos; k0 += KT) {
+    const int n = (int)min((int64_t)KT, pos + 1 - k0);
+    for (int j = warp; j < n; j += nw) {
+      float v = 0.f;
+      for (int i = lane; i < a.d; i += 32) v += q[i] * ld(kb + (k0 + j) * a.Dk + i);
+      v = warp_sum(v);
+      if (lane == 0) s[j] = v * a.scale;
+    }
+    __syncthreads();
+    float t = -INFINITY;
+    for (int j = tid; j < n; j += blockDim.x) t = fmaxf(t, s[j]);
+    const float mn = fmaxf(mx, block_max(t, sh));
+    const float corr = mx == -INFINITY ? 0.f : expf(mx - mn);
+    float ls = 0.f;
+    for (int j = tid; j < n; j += blockDim.x) {
+      const float e = expf(s[j] - mn);
+      s[j] = e;
+      ls += e;
+    }
+    l = l * corr + block_sum(ls, sh);  // (its barriers also publish s)
+    mx = mn;
+    for (int i = tid; i < a.dv; i += blockDim.x) {
+      float v = o[i] * corr;
+      for (int j = 0; j < n; ++j) v += s[j] * ld(vb + (k0 + j) * a.Dv + i);
+      o[i] = v;
+    }
+    __syncthreads();
+  }
+  T* out = (T*)a.att + m * a.ld_att + (int64_t)h * a.Dv;
+  for (int i = tid; i < a.Dv; i += blockDim.x) st(out + i, o[i] / l);
+}
+
+}  // namespace
+
+int k_launch_rows_qkv(cg_ctx* c, const RowsAttnArgs& a) {
+  if (a.rows.M == 0) return CG_OK;
+  if (a.Dk % 8 || a.Dv % 8 || a.ldp % 4) return fail(c, CG_ERR_INVALID, "attention: head sizes must be padded to multiples of 8");
+  if (a.bf16) CG_CUDA(c, launch_kernel(c, k_rows_qkv<__nv_bfloat16>, dim3((unsigned)a.rows.M), dim3(256), 0, 1, a));
+  else CG_CUDA(c, launch_kernel(c, k_rows_qkv<float>, dim3((unsigned)a.rows.M), dim3(256), 0, 1, a));
+  CG_LAUNCHED(c);
+  return CG_OK;
+}
+
+int k_launch_rows_attn(cg_ctx* c, const RowsAttnArgs& a) {
+  if (a.rows.M == 0) return CG_OK;
+  const size_t smem = (size_t)(a.Dk + a.Dv + 64 + 32) * 4;
+  if (smem > 48 * 1024 || a.H > 65535) return fail(c, CG_ERR_UNSUPPORTED, "attention: heads too wide or too many");
+  dim3 grid((unsigned)a.rows.M, (unsigned)a.H);
+  if (a.bf16) CG_CUDA(c, launch_kernel(c, k_rows_attn<__nv_bfloat16>, grid, dim3(128), smem, 1, a));
+  else CG_CUDA(c, launch_kernel(c, k_rows_attn<float>, grid, dim3(128), smem, 1, a));
+  CG_LAUNCHED(c);
+  return CG_OK;
+}
+
+}  // namespace cg

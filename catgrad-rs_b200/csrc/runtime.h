@@ -311,7 +311,8 @@ struct LazyPause {
 // ---- entry points implemented in other translation units, used across them ----------
 
 // y[M,N] = x[M,K] w[N,K]^T on the tcgen05 pipeline.  x, w bf16 row-major (ld in elements);
-// out_mode 0: f32 store, 1: bf16 store, 2: f32 out = acc + residual (residual may alias out).
+// out_mode 0: f32 store, 1: bf16 store, 2: f32 out = acc + residual (residual may alias out),
+// 4: bf16 store of the square of relu.
 // splits <= 0 lets the launcher choose.  `workspace` must hold splits*M*N floats when
 // splits > 1 (pass nullptr to have it allocated from the context).
 int gemm_tc(cg_ctx* c, const __nv_bfloat16* x, int64_t ldx, const __nv_bfloat16* w, int64_t ldw,
@@ -330,7 +331,7 @@ int gemm_tcp(cg_ctx* c, const __nv_bfloat16* x, int64_t ldx, const __nv_bfloat16
              void* out, int64_t ldo, const float* residual, int64_t M, int64_t N, int64_t K, int out_mode,
              int pair, int act);
 int gemm_tcp_grouped(cg_ctx* c, const __nv_bfloat16* x, int64_t x_rows, const __nv_bfloat16* w, const __nv_bfloat16* w_up,
-                     int64_t experts, void* out, int64_t N, int64_t K, int pair, int act, const int32_t* tile_expert,
+                     int64_t experts, void* out, int64_t N, int64_t K, int pair, int act, float limit, const int32_t* tile_expert,
                      const int32_t* tile_row0, const int32_t* tile_rows, const int32_t* n_list, int64_t max_list);
 // Gate and up projections with the activation fused: w holds the gate rows then the up rows
 // ([2 F, K]); out[M, F] (bf16) = act(x gate^T) * (x up^T), act 0 = silu, 1 = tanh-gelu.

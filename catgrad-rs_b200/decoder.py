@@ -30,6 +30,7 @@ class DecoderConfig(C.Structure):
         ("rope_local_theta", C.c_float), ("rope_local_every", C.c_int32),
         ("n_experts", C.c_int32), ("top_k", C.c_int32), ("moe_ffn", C.c_int32), ("norm_topk", C.c_int32),
         ("tp_rank", C.c_int32), ("tp_world", C.c_int32), ("ep_rank", C.c_int32), ("ep_world", C.c_int32),
+        ("streams", C.c_int32), ("embed_norm", C.c_int32), ("loop_input", C.c_int32),
     ]
 
 
@@ -70,15 +71,18 @@ class Decoder:
             fn.restype = i32
         c = DecoderConfig()
         # a cached prefix can be shortened to any length (a recurrent state cannot go back)
-        self.keeps_prefix = not isinstance(cfg, LayeredConfig)
+        self.keeps_prefix = not isinstance(cfg, LayeredConfig) or not cfg.recurrent
         if isinstance(cfg, LayeredConfig):
             c.num_layers, c.hidden, c.vocab = len(cfg.layers), cfg.hidden_size, cfg.vocab_size
             c.rms_eps, c.max_seq, c.max_batch = cfg.rms_norm_eps, max_seq, max_batch
+            c.embed_scale, c.streams = cfg.embed_scale, cfg.streams
+            for k, v in cfg.design.switches().items():
+                setattr(c, k, v)
             c.tp_rank, c.tp_world, c.ep_rank, c.ep_world = tp_rank, tp_world, ep_rank, ep_world
             for k, v in switches.items():
                 setattr(c, k, v)
             self.cfg = c
-            layers = (LayerStruct * len(cfg.layers))(*[s.struct() for s in cfg.layers])
+            layers = (LayerStruct * len(cfg.layers))(*[s.struct(cfg.design) for s in cfg.layers])
             loop = C.byref(LoopStruct(*cfg.loop)) if cfg.loop else None
             h = vp()
             backend._check(L.cg_decoder_create_layers(backend._ctx, C.byref(c), layers, len(layers), loop, C.byref(h)))

@@ -1,5 +1,6 @@
-"""Configurations of models described layer by layer, with different sequence mixers and an optional
-loop over some of the layers (the Ralapel design), for `Decoder`.
+"""Configurations of models described layer by layer: different sequence mixers and feed-forwards, an
+optional loop over some of the layers, and what a design fixes for all of them (the Ralapel and
+Segedra designs), for `Decoder`.
 
 No counterpart in the reference, whose decoders are attention-only.  `LayeredConfig.from_json`
 reads a checkpoint's config.json; every size and constant comes from it.
@@ -9,14 +10,17 @@ from __future__ import annotations
 import ctypes as C
 from dataclasses import dataclass, field
 
-MIXERS = {"latent_attention": 1, "delta": 2, "mamba2": 3}   # cg_mixer (include/catgrad_cuda.h)
+MIXERS = {"latent_attention": 1, "delta": 2, "mamba2": 3, "attention": 4}   # cg_mixer (include/catgrad_cuda.h)
+SILU, GELU, BOUNDED, RELU2 = range(4)                                      # cg_act
 
 
 class LayerStruct(C.Structure):
     """Mirror of `cg_layer_config` (include/catgrad_cuda.h)."""
     _fields_ = [("mixer", C.c_int32), ("ffn", C.c_int32), ("act", C.c_int32), ("heads", C.c_int32), ("kv_heads", C.c_int32),
                 ("dim", C.c_int32), ("rot_dim", C.c_int32), ("vdim", C.c_int32), ("kv_rank", C.c_int32), ("state", C.c_int32),
-                ("groups", C.c_int32), ("norm_groups", C.c_int32), ("conv", C.c_int32), ("rot_base", C.c_double), ("scale", C.c_double)]
+                ("groups", C.c_int32), ("norm_groups", C.c_int32), ("conv", C.c_int32), ("window", C.c_int32), ("qk_norm", C.c_int32),
+                ("sink", C.c_int32), ("experts", C.c_int32), ("top_k", C.c_int32), ("rot_base", C.c_double), ("scale", C.c_double),
+                ("router_scale", C.c_double), ("act_limit", C.c_double)]
 
 
 class LoopStruct(C.Structure):
@@ -24,20 +28,74 @@ class LoopStruct(C.Structure):
     _fields_ = [("start", C.c_int32), ("stop", C.c_int32), ("times", C.c_int32)]
 
 
+@dataclass(frozen=True)
+class Design:
+    """What a family of layer-by-layer models fixes for all its layers."""
+    mixers: tuple[str, ...]
+    dense_act: int               # of dense feed-forwards
+    experts: bool = False        # feed-forwards may be mixtures of experts
+    post_norms: bool = False     # norms behind the sublayers too
+    embed_norm: bool = False
+    loop_input: bool = False     # a loop's passes start from W [x; normed embedding]
+    norm_plus_one: bool = False  # layer and final norms multiply by 1 + w
+    tied_head: bool = False
+    qk_norm: bool = False        # attention: norms over all query and over all key heads
+    sink: bool = False           # attention: a learned term of the softmax's denominator per head
+
+    def switches(self) -> dict[str, int]:
+        """Fields of `cg_decoder_config`."""
+        return {"post_norms": int(self.post_norms), "embed_norm": int(self.embed_norm), "loop_input": int(self.loop_input),
+                "norm_plus_one": int(self.norm_plus_one), "tie_embeddings": int(self.tied_head)}
+
+
+DESIGNS = {
+    "Ralapel": Design(("latent_attention", "delta", "mamba2"), GELU, post_norms=True, embed_norm=True, loop_input=True),
+    "Segedra": Design(("attention",), RELU2, experts=True, norm_plus_one=True, tied_head=True, qk_norm=True, sink=True),
+}
+
+
+@dataclass
+class Experts:
+    """A mixture-of-experts feed-forward: `top` of `count` experts per token, chosen by the router's
+    softmax plus a correction, weighted by the softmax times `scale`; `limit` bounds their units."""
+    count: int
+    top: int
+    scale: float
+    limit: float
+
+
 @dataclass
 class LayerSpec:
     """One layer: the mixer's name, its sizes (the keys config.json uses) and the feed-forward width
-    (0 = the layer has none)."""
+    (of one expert if there are experts; 0 = the layer has none)."""
     mixer: str
     sizes: dict
     ffn: int = 0
-    act: int = 1   # 0 silu, 1 tanh gelu
+    act: int = GELU
+    experts: Experts | None = None
 
-    def struct(self) -> LayerStruct:
+    @property
+    def window(self) -> int:
+        """Tokens an attention layer sees, itself included; 0 = all before it."""
+        return (self.sizes.get("mask") or {}).get("size") or 0
+
+    @property
+    def rotated(self) -> int:
+        """Rotated components of an attention head."""
+        return (self.sizes.get("rot") or {}).get("dims", 0)
+
+    def struct(self, design: Design) -> LayerStruct:
         s, m = LayerStruct(), self.sizes
         s.mixer, s.ffn, s.act = MIXERS[self.mixer], self.ffn, self.act
         s.heads, s.vdim = m["heads"], m["vdim"]
-        if self.mixer == "latent_attention":
+        if self.experts:
+            e = self.experts
+            s.experts, s.top_k, s.router_scale, s.act_limit = e.count, e.top, e.scale, e.limit
+        if self.mixer == "attention":
+            s.dim, s.kv_heads, s.scale, s.window = m["dim"], m["kv_heads"], m["scale"], self.window
+            s.rot_dim, s.rot_base = self.rotated, m["rot"]["base"] if self.rotated else 0.0
+            s.qk_norm, s.sink = int(design.qk_norm), int(design.sink)
+        elif self.mixer == "latent_attention":
             s.dim, s.rot_dim, s.kv_rank, s.scale = m["dim"], m["rot_dim"], m["kv_rank"], m["scale"]
             s.rot_base = m["rot"]["base"] if m["rot_dim"] else 0.0
         elif self.mixer == "delta":
@@ -57,23 +115,37 @@ class LayeredConfig:
     rms_norm_eps: float = 1e-6
     dtype: str = "bf16"
     arch: str = "layered"
+    design: Design = DESIGNS["Ralapel"]
+    streams: int = 0                           # rows of the residual stream per token; 0 = a plain one
+    embed_scale: float = 1.0
     extras: dict = field(default_factory=dict)
 
     @classmethod
     def from_json(cls, d: dict) -> "LayeredConfig":
+        name = d["architecture"]
+        design = DESIGNS[name]
         layers = []
         for i, e in enumerate(d["layers"]):
-            if e["type"] not in MIXERS:
+            if e["type"] not in design.mixers:
                 raise ValueError(f"layer {i}: unknown mixer {e['type']!r}")
             mlp = e.get("mlp")
-            if mlp and mlp["kind"] != "dense":
+            if mlp and not (mlp["kind"] == "dense" or (mlp["kind"] == "moe" and design.experts)):
                 raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
             if e["type"] == "latent_attention" and e["mixer"]["rot_dim"] and e["mixer"]["rot"]["dims"] != e["mixer"]["rot_dim"]:
                 raise ValueError(f"layer {i}: the rotated part must be rotated whole")
-            layers.append(LayerSpec(e["type"], e["mixer"], mlp["ff"] if mlp else 0))
+            if mlp and mlp["kind"] == "moe":
+                r, x = mlp["router"], mlp["expert"]
+                layers.append(LayerSpec(e["type"], e["mixer"], x["ff"], BOUNDED, Experts(r["experts"], r["top"], r["scale"], x["limit"])))
+            else:
+                layers.append(LayerSpec(e["type"], e["mixer"], mlp["ff"] if mlp else 0, design.dense_act))
         lp = d.get("loop")
-        return cls(d.get("architecture", "layered"), d["width"], d["vocab"], layers,
-                   (lp["start"], lp["stop"], lp["times"]) if lp else None, d["norm"]["eps"])
+        return cls(name, d["width"], d["vocab"], layers, (lp["start"], lp["stop"], lp["times"]) if lp else None, d["norm"]["eps"],
+                   design=design, streams=d.get("streams") or 0, embed_scale=(d.get("embedding") or {}).get("scale", 1.0))
+
+    @property
+    def recurrent(self) -> bool:
+        """Whether some layer's state cannot go back to an earlier position."""
+        return any(L.mixer in ("delta", "mamba2") for L in self.layers)
 
     def layer_runs(self) -> list[int]:
         """Layers in the order they run."""
@@ -85,21 +157,43 @@ class LayeredConfig:
 
     def param_shapes(self) -> dict[str, tuple[int, ...]]:
         """Tensor names and shapes of a checkpoint (weights [out, in])."""
-        W = self.hidden_size
-        s = {"embed": (self.vocab_size, W), "embed.norm": (W,), "final.norm": (W,), "head": (self.vocab_size, W)}
-        if self.loop:
+        W, D = self.hidden_size, self.design
+        s = {"embed": (self.vocab_size, W), "final.norm": (W,)}
+        if D.embed_norm:
+            s["embed.norm"] = (W,)
+        if not D.tied_head:
+            s["head"] = (self.vocab_size, W)
+        if self.loop and D.loop_input:
             s["loop.in"] = (W, 2 * W)
         for i, L in enumerate(self.layers):
             p, m = f"l{i}.", L.sizes
             H, dv = m["heads"], m["vdim"]
-            s[p + "norm1"] = s[p + "norm1b"] = (W,)
-            if L.ffn:
-                s[p + "norm2"] = s[p + "norm2b"] = (W,)
-                s[p + "mlp.gate"] = s[p + "mlp.up"] = (L.ffn, W)
-                s[p + "mlp.down"] = (W, L.ffn)
+            for q in (1, 2) if L.ffn else (1,):
+                s[p + f"norm{q}"] = (W,)
+                if D.post_norms:
+                    s[p + f"norm{q}b"] = (W,)
+                if self.streams:
+                    s[p + f"hc{q}.in"] = s[p + f"hc{q}.out"] = (self.streams,)
+                    s[p + f"hc{q}.mix"] = (self.streams, self.streams)
+            if L.experts:
+                s[p + "mlp.router"], s[p + "mlp.correction"] = (L.experts.count, W), (L.experts.count,)
+                for e in range(L.experts.count):
+                    s[p + f"mlp.e{e}.gate"] = s[p + f"mlp.e{e}.up"] = (L.ffn, W)
+                    s[p + f"mlp.e{e}.down"] = (W, L.ffn)
+            elif L.ffn:
+                s[p + "mlp.up"], s[p + "mlp.down"] = (L.ffn, W), (W, L.ffn)
+                if L.act != RELU2:
+                    s[p + "mlp.gate"] = (L.ffn, W)
             p += "mix."
             s[p + "o"] = (W, H * dv)
-            if L.mixer == "latent_attention":
+            if L.mixer == "attention":
+                G, d = m["kv_heads"], m["dim"]
+                s[p + "q"], s[p + "k"], s[p + "v"] = (H * d, W), (G * d, W), (G * dv, W)
+                if D.qk_norm:
+                    s[p + "q.norm"], s[p + "k.norm"] = (H * d,), (G * d,)
+                if D.sink:
+                    s[p + "sink"] = (H,)
+            elif L.mixer == "latent_attention":
                 d, r, R = m["dim"], m["rot_dim"], m["kv_rank"]
                 s[p + "q"], s[p + "dkv"], s[p + "dkv.norm"] = (H * (d + r), W), (R + r, W), (R,)
                 s[p + "uk"], s[p + "uv"] = (H * d, R), (H * dv, R)
@@ -119,9 +213,9 @@ class LayeredConfig:
                 s[p + "norm"] = (H * dv,)
         return s
 
-    @staticmethod
-    def synthetic(name: str) -> tuple[float, float]:
-        """(mean, std) a synthetic checkpoint draws a tensor with: gains 1, slow decays, wide taps."""
+    def synthetic(self, name: str) -> tuple[float, float]:
+        """(mean, std) a synthetic checkpoint draws a tensor with: gains 1, slow decays, wide taps,
+        streams that are read and written alike."""
         leaf = name.rsplit(".", 1)[-1]
         if leaf == "A_log":
             return 0.5, 0.5
@@ -132,7 +226,12 @@ class LayeredConfig:
         if name.endswith("conv.b"):
             return 0.0, 0.1
         if leaf in ("D", "norm", "norm1", "norm1b", "norm2", "norm2b"):
-            return 1.0, 0.0
+            plus_one = self.design.norm_plus_one and ".mix." not in name
+            return 0.0 if plus_one else 1.0, 0.0
+        if ".hc" in name:
+            return {"in": 1.0, "out": 1.0, "mix": 0.0}[leaf] / self.streams, 0.5 / self.streams
+        if leaf in ("correction", "sink"):
+            return 0.0, 0.01 if leaf == "correction" else 1.0
         return 0.0, 0.02
 
 

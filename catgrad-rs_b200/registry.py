@@ -45,6 +45,7 @@ ARCHITECTURES = {
     "Gemma2ForCausalLM": _hf("gemma"),
     "Gemma3ForCausalLM": _hf("gemma"),
     "Ralapel": LayeredConfig.from_json,
+    "Segedra": LayeredConfig.from_json,
 }
 
 

@@ -52,6 +52,9 @@ pub struct DecoderConfig {
     pub tp_world: i32,
     pub ep_rank: i32,
     pub ep_world: i32,
+    pub streams: i32,
+    pub embed_norm: i32,
+    pub loop_input: i32,
 }
 
 #[repr(C)]

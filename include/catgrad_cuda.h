@@ -332,6 +332,11 @@ typedef struct cg_decoder_config {
    * this moves the bytes an all-to-all dispatch / combine would.  0 or 1 = off. */
   int32_t ep_rank;
   int32_t ep_world;
+  /* decoders built layer by layer (cg_decoder_create_layers) */
+  int32_t streams;          /* hyper-connections: rows of the residual stream per token, at most 16 (0 = a plain
+                               residual stream) */
+  int32_t embed_norm;       /* an RMS norm of the embedding */
+  int32_t loop_input;       /* a loop's passes start from W [x; normed embedding] */
 } cg_decoder_config;
 
 int32_t cg_decoder_create(cg_ctx*, const cg_decoder_config* cfg, cg_decoder** out);
@@ -386,48 +391,73 @@ int32_t cg_decoder_generate(cg_decoder*, const uint32_t* prompt, int32_t batch, 
 
 /* --- decoders built layer by layer: layers with different sequence mixers, optionally run in a loop.
  * No counterpart in the reference, whose decoders are attention-only.  Every layer is
- *   x <- x + norm1b(mixer(norm1(x))),  x <- x + norm2b(ff(norm2(x)))
- * with RMS norms (the second line only where the layer has a feed-forward), a gated feed-forward
- * down(act(gate h) * up h), a normed embedding and a norm before the head.  The residual stream,
- * norms, positions, attention weights and everything inside a recurrence are f32.  The context's
+ *   x <- x + post1(mixer(norm1(x))),  x <- x + post2(ff(norm2(x)))
+ * with RMS norms (the second line only where the layer has a feed-forward; post1, post2 are norms with
+ * post_norms, else nothing) and a norm before the head.  With streams = s > 0 the residual stream is s
+ * rows x_1 .. x_s, all equal to the embedding at first, and a sublayer f with coefficients in [s],
+ * out [s], mix [s, s] takes u = sum_s in[s] x_s and leaves
+ *   x_t <- sum_s mix[s, t] x_s + out[t] f(norm(u));
+ * the final norm reads the rows' sum.  Feed-forwards are dense (act) or a mixture of experts.  The
+ * residual stream, norms, positions, attention weights, routers and everything inside a recurrence
+ * are f32.  The context's
  * precision decides the rest: CG_PREC_BF16 runs the tensor-core kernels on bf16 weights and
  * activations, CG_PREC_F32 runs everything in f32. */
 typedef enum cg_mixer {
   CG_MIX_LATENT = 1, /* latent attention: keys and values are linear maps of a cached low-rank row */
   CG_MIX_DELTA = 2,  /* gated delta rule behind short convolutions */
-  CG_MIX_SSD = 3     /* Mamba-2: scalar-decay state space with a gated group norm */
+  CG_MIX_SSD = 3,    /* Mamba-2: scalar-decay state space with a gated group norm */
+  CG_MIX_ATTENTION = 4 /* grouped-query attention: optional norms, window and sink */
 } cg_mixer;
+typedef enum cg_act {
+  CG_ACT_SILU = 0,    /* down(silu(gate h) * up h) */
+  CG_ACT_GELU = 1,    /* down(gelu(gate h) * up h), tanh form */
+  CG_ACT_BOUNDED = 2, /* experts: g = min(gate h, act_limit), u = clamp(up h, +-act_limit), down(g sigmoid(1.702 g) (u + 1)) */
+  CG_ACT_RELU2 = 3    /* dense, not gated: down(relu(up h)^2) */
+} cg_act;
 typedef struct cg_layer_config {
   int32_t mixer;     /* cg_mixer */
-  int32_t ffn;       /* width of the gated feed-forward, 0 = none */
-  int32_t act;       /* 0 silu, 1 tanh gelu */
-  int32_t heads;     /* latent: query heads; delta, ssd: value heads */
-  int32_t kv_heads;  /* delta: query/key heads, a divisor of heads */
-  int32_t dim;       /* latent: unrotated query/key size per head; delta: query/key size per head */
-  int32_t rot_dim;   /* latent: rotated query/key size, the key part shared by all heads */
+  int32_t ffn;       /* width of the feed-forward (of one expert), 0 = none */
+  int32_t act;       /* cg_act */
+  int32_t heads;     /* latent, attention: query heads; delta, ssd: value heads */
+  int32_t kv_heads;  /* delta: query/key heads, attention: key/value heads; a divisor of heads */
+  int32_t dim;       /* latent: unrotated query/key size per head; delta, attention: query/key size per head */
+  int32_t rot_dim;   /* latent: rotated query/key size, the key part shared by all heads; attention: how many
+                        components of a head are rotated, from the first */
   int32_t vdim;      /* value size per head */
   int32_t kv_rank;   /* latent: size of the cached row without its rotated part */
   int32_t state;     /* ssd: state size (the key size of the recurrence) */
   int32_t groups;    /* ssd: groups of heads sharing B and C */
   int32_t norm_groups; /* ssd: equal parts of the gated norm */
   int32_t conv;      /* delta, ssd: taps of the short convolutions */
-  double rot_base;   /* latent: base of the rotary frequencies; neighbouring components are paired */
-  double scale;      /* latent: factor on the scores */
+  int32_t window;    /* attention: a token sees itself and the window - 1 tokens before it, 0 = all */
+  int32_t qk_norm;   /* attention: 1 = RMS norm over all query heads at once, and over all key heads, before rotation */
+  int32_t sink;      /* attention: 1 = the softmax has one more term per head, exp(sink), without a value */
+  int32_t experts;   /* feed-forward: 0 = dense, else the number of experts, softmax-routed */
+  int32_t top_k;     /* experts per token: those with the largest probability + correction */
+  double rot_base;   /* latent, attention: base of the rotary frequencies; neighbouring components are paired */
+  double scale;      /* latent, attention: factor on the scores */
+  double router_scale; /* factor on the chosen experts' probabilities, which are not renormalised */
+  double act_limit;  /* CG_ACT_BOUNDED */
 } cg_layer_config;
 typedef struct cg_loop_config {
   int32_t start, stop, times; /* layers [start, stop) run `times` times in a row, each pass with its own cache or
-                                 state; before a pass x <- W [x; x0], x0 the normed embedding */
+                                 state; with loop_input, before a pass x <- W [x; x0], x0 the normed embedding */
 } cg_loop_config;
-/* cfg supplies hidden, vocab, rms_eps, max_seq (capacity per sequence) and max_batch (sequences held
- * at once).  loop may be NULL.  Parameters (cg_decoder_set_param / _load_safetensors), weights [out, in]:
- * embed, embed.norm, final.norm, head, loop.in [hidden, 2 hidden], and per layer l<i>.norm1,
- * .norm1b, .norm2, .norm2b, .mlp.{gate,up,down}, .mix.o and
+/* cfg supplies hidden, vocab, rms_eps, max_seq (capacity per sequence), max_batch (sequences held at
+ * once), embed_scale, norm_plus_one (layer and final norms), post_norms (excludes streams), tie_embeddings,
+ * streams, embed_norm and loop_input (excludes streams).  loop may be NULL.  Parameters
+ * (cg_decoder_set_param / _load_safetensors), weights [out, in]: embed, final.norm, with the options above
+ * embed.norm, loop.in [hidden, 2 hidden] and head, and per layer l<i>.norm1, .norm2, with post_norms
+ * .norm1b, .norm2b, with streams .hc1.{in,out,mix}, .hc2.{in,out,mix}, dense .mlp.{gate,up,down},
+ * experts .mlp.{router,correction} and .mlp.e<j>.{gate,up,down}, .mix.o and
+ *   attention  .mix.{q,k,v}, with qk_norm .mix.{q,k}.norm, with sink .mix.sink
  *   latent  .mix.{q,dkv,dkv.norm,uk,uv}
  *   delta   .mix.{q,k,v,b,a,g}, .mix.{q,k,v}.conv, .mix.{A_log,dt_bias,norm}
  *   ssd     .mix.{in,conv,conv.b,dt_bias,A_log,D,norm}.
  * The decoder then serves cg_decoder_prefill / append / decode / step_with / tokens / generate like
  * any other (rows = slots 0 .. B-1, equal lengths), and the calls below.  cg_decoder_truncate takes
- * 0 or the cached position only: a recurrent state has no earlier versions to go back to. */
+ * 0 or the cached position only if the model has a recurrent layer: a state has no earlier versions
+ * to go back to. */
 int32_t cg_decoder_create_layers(cg_ctx*, const cg_decoder_config* cfg, const cg_layer_config* layers, int32_t n_layers,
                                  const cg_loop_config* loop, cg_decoder** out);
 /* Sequences of unequal length.  seq_open takes a free slot (its position is 0 and its state zero),
@@ -442,7 +472,8 @@ int32_t cg_decoder_seq_close(cg_decoder*, int32_t slot);
 int32_t cg_decoder_run(cg_decoder*, int32_t rows, const int32_t* slots, const int32_t* lens, const uint32_t* tokens,
                        int32_t n_want, const int32_t* want, int32_t greedy, cg_tensor** logits_out);
 /* Diagnostics: keep the residual stream of the next cg_decoder_run calls after every layer run, and
- * read it back as [layer runs, tokens, hidden] F32 (the last call's tokens; one portion only). */
+ * read it back as [layer runs, tokens, hidden] F32 (the last call's tokens; one portion only; several
+ * streams are summed). */
 int32_t cg_decoder_keep_residuals(cg_decoder*, int32_t on);
 int32_t cg_decoder_residuals(cg_decoder*, cg_tensor** out);
 
