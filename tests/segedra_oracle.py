@@ -5,7 +5,8 @@ run one at a time, attention one query at a time, experts one token at a time, a
 batched, grouped or cached.  A checkpoint is a dict name -> array, a configuration is the parsed
 config.json.
 
-`hooks` (optional) receives (run index, sum of the streams [T, width]) after every layer run.
+`hooks` (optional) receives (run index, sum of the streams [T, width]) after every layer run; `gaps`, a
+list, receives per routed layer run how far each token's last chosen expert is ahead of the next [T].
 `faults` lets a test plant a mistake here, on the CPU, to see that its inputs would show it.
 """
 from __future__ import annotations
@@ -98,9 +99,19 @@ def route(h, router, correction, top, scale, faults=()):
     return list(zip(chosen.tolist(), w))
 
 
-def experts_mlp(h, P, m, faults=()):
+def choice_gap(h, router, correction, top):
+    """How far the last chosen expert's corrected score is ahead of the next one's."""
+    z = router @ h
+    s = np.exp(z - z.max())
+    c = np.sort(s / s.sum() + correction)[::-1]
+    return c[top - 1] - c[top] if top < len(c) else np.inf
+
+
+def experts_mlp(h, P, m, faults=(), gaps=None):
     out = np.zeros_like(h)
     r = m["router"]
+    if gaps is not None:
+        gaps.append(np.array([choice_gap(t, P("router"), P("correction"), r["top"]) for t in h]))
     for t in range(h.shape[0]):
         for e, w in route(h[t], P("router"), P("correction"), r["top"], r["scale"], faults):
             out[t] += w * expert(h[t], P(f"e{e}.gate"), P(f"e{e}.up"), P(f"e{e}.down"), m["expert"]["limit"])
@@ -127,16 +138,19 @@ def layer_runs(cfg):
     return list(range(a)) + list(range(a, b)) * lp["times"] + list(range(b, n))
 
 
-def forward(cfg, W, tokens, hooks=None, faults=()):
+def forward(cfg, W, tokens, hooks=None, faults=(), gaps=None):
     """Logits [T, vocab] of one sequence from its first token."""
     W = {k: np.asarray(v, dtype=np.float64) for k, v in W.items()}
     eps = cfg["norm"]["eps"]
     x0 = W["embed"][np.asarray(tokens)] * cfg["embedding"]["scale"]
-    x = np.stack([x0] * cfg["streams"])
+    plain = not cfg["streams"]               # no streams: a residual sum
+    x = np.stack([x0] * (cfg["streams"] or 1))
     for run, i in enumerate(layer_runs(cfg)):
         L, l = cfg["layers"][i], f"l{i}."
 
         def sublayer(x, q, f):
+            if plain:
+                return x + f(norm(x[0], W[f"{l}norm{q}"], eps))
             y = f(norm(streams_in(x, W[f"{l}hc{q}.in"]), W[f"{l}norm{q}"], eps))
             return streams_out(x, y, W[f"{l}hc{q}.mix"], W[f"{l}hc{q}.out"], faults)
 
@@ -145,7 +159,7 @@ def forward(cfg, W, tokens, hooks=None, faults=()):
         if m and m["kind"] == "dense":
             x = sublayer(x, 2, lambda h: squared_relu_mlp(h, lambda n: W[f"{l}mlp.{n}"]))
         elif m:
-            x = sublayer(x, 2, lambda h: experts_mlp(h, lambda n: W[f"{l}mlp.{n}"], m, faults))
+            x = sublayer(x, 2, lambda h: experts_mlp(h, lambda n: W[f"{l}mlp.{n}"], m, faults, gaps))
         if hooks:
             hooks(run, x.sum(0))
     return norm(x.sum(0), W["final.norm"], eps) @ W["embed"].T
