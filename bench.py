@@ -109,29 +109,47 @@ WORKLOADS = {
 
 
 # the same for models built layer by layer (catgrad-rs_b200/layered.py); measured beside an attention-only
-# decoder of equal width, feed-forward, vocabulary and number of layer runs
+# decoder of equal width, feed-forward (or experts), vocabulary and number of layer runs
 LAYERED_WORKLOADS = {
     "ralapel-w1024": ("RALAPEL_W1024", 8, 512, 128),
     "ralapel-w2048": ("RALAPEL_W2048", 8, 512, 128),
     "ralapel-w2048-b1": ("RALAPEL_W2048", 1, 512, 128),
     "ralapel-w2048-long": ("RALAPEL_W2048", 4, 4096, 128),
     "ralapel-w4096": ("RALAPEL_W4096", 8, 1024, 128),
+    "segedra-w1024": ("SEGEDRA_W1024", 8, 512, 128),
+    "segedra-w2048": ("SEGEDRA_W2048", 8, 1024, 128),
+    "segedra-w2048-b1": ("SEGEDRA_W2048", 1, 1024, 128),
+    "segedra-w2048-long": ("SEGEDRA_W2048", 4, 4096, 128),
+    "segedra-w2880": ("SEGEDRA_W2880", 8, 1024, 128),
 }
 
 
+def experts_reached(experts: int, top: int, tokens: int) -> float:
+    """How many different experts `tokens` independent uniform choices of `top` reach on average."""
+    return experts * (1.0 - (1.0 - top / experts) ** tokens)
+
+
 def layered_step_bytes(cfg, batch: int, context: float) -> dict:
-    """Bytes a decode step has to move: every layer run's matrices and the head once, the f32 states
-    read and written, the cached rows read."""
+    """Bytes a decode step has to move: every layer run's matrices and the head once (of the experts those
+    that independent choices would reach, on average), the f32 states read and written, the cached
+    rows or visible keys and values read."""
     mats, states, cache = 2 * cfg.vocab_size * cfg.hidden_size, 0, 0.0
     shapes = cfg.param_shapes()
     for i in cfg.layer_runs():
-        mats += sum(2 * n[0] * n[1] for k, n in shapes.items() if k.startswith(f"l{i}.") and len(n) == 2 and not k.endswith("conv"))
+        e = cfg.layers[i].experts
+        mats += sum(2 * n[0] * n[1] for k, n in shapes.items()
+                    if k.startswith(f"l{i}.") and len(n) == 2 and not k.endswith("conv") and ".mlp.e" not in k)
+        if e:
+            mats += 6 * cfg.hidden_size * cfg.layers[i].ffn * experts_reached(e.count, e.top, batch)
         m = cfg.layers[i].sizes
-        if cfg.layers[i].mixer == "latent_attention":
+        if cfg.layers[i].mixer == "attention":
+            seen = min(context, cfg.layers[i].window or context)
+            cache += batch * seen * m["kv_heads"] * (m["dim"] + m["vdim"]) * 2
+        elif cfg.layers[i].mixer == "latent_attention":
             cache += batch * context * (m["kv_rank"] + m["rot_dim"]) * 2
         else:
             states += 2 * 4 * batch * m["heads"] * m["vdim"] * (m["dim"] if cfg.layers[i].mixer == "delta" else m["state"])
-    if cfg.loop:
+    if cfg.loop and "loop.in" in shapes:
         mats += cfg.loop[2] * 2 * shapes["loop.in"][0] * shapes["loop.in"][1]
     return {"weights": mats, "states": states, "cached_rows": cache}
 
@@ -145,8 +163,14 @@ def layered_workload(cg, C, args, local):
     cfg = getattr(layered, name)
     B, S, T = args.batch or B0, args.prompt or S0, args.decode or T0
     heads = max(1, cfg.hidden_size // 128)
-    closest = cg.synth.ModelConfig("llama-equal-size", cfg.hidden_size, max(L.ffn for L in cfg.layers), len(cfg.layer_runs()), heads,
-                                   max(1, heads // 4), cfg.vocab_size, head_dim=128, dtype="bf16")
+    last = cfg.layers[-1]
+    if last.experts:
+        closest = cg.synth.ModelConfig("qwen3-moe-equal-size", cfg.hidden_size, last.ffn, len(cfg.layer_runs()), last.sizes["heads"],
+                                       last.sizes["kv_heads"], cfg.vocab_size, head_dim=last.sizes["dim"], dtype="bf16", arch="qwen3",
+                                       num_local_experts=last.experts.count, num_experts_per_tok=last.experts.top, moe_intermediate_size=last.ffn)
+    else:
+        closest = cg.synth.ModelConfig("llama-equal-size", cfg.hidden_size, max(L.ffn for L in cfg.layers), len(cfg.layer_runs()), heads,
+                                       max(1, heads // 4), cfg.vocab_size, head_dim=128, dtype="bf16")
     peak, peak_kind = measured_peaks()
 
     def timed(fn, n):
@@ -188,6 +212,9 @@ def layered_workload(cg, C, args, local):
             parts = layered_step_bytes(c, B, S + T / 2)
         else:
             parts = {"weights": 2 * dense_params_per_step(c), "kv_cache": B * cg.synth.kv_bytes_per_token(c) * (S + T / 2)}
+            if c.num_local_experts:
+                parts["weights"] += c.num_hidden_layers * 6 * c.hidden_size * c.moe_intermediate_size * \
+                    experts_reached(c.num_local_experts, c.num_experts_per_tok, B)
         floor = sum(parts.values()) / (peak * 1e9) * 1e3
         return {"model": c.name, "ms_per_job": job_ms, "tok_s": B * (S + T) / job_ms * 1e3, "e2e_tok_s": B * (S + T) / e2e_ms * 1e3,
                 "prefill_ms": prefill_ms, "prefill_tok_s": B * S / prefill_ms * 1e3, "decode_ms_per_step": decode_ms,
@@ -459,8 +486,8 @@ def main():
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--workload", default="llama1b", choices=sorted(WORKLOADS) + sorted(LAYERED_WORKLOADS),
                     help="llama1b is the configuration the metric is quoted on; the others are the remaining "
-                         "model shapes at their own batch / prompt / decode sizes; ralapel-* measure a model built layer by "
-                         "layer beside an attention-only decoder of equal size (one GPU)")
+                         "model shapes at their own batch / prompt / decode sizes; ralapel-* and segedra-* measure a model "
+                         "built layer by layer beside an attention-only decoder of equal size (one GPU)")
     ap.add_argument("--batch", type=int, default=0)
     ap.add_argument("--prompt", type=int, default=0)
     ap.add_argument("--decode", type=int, default=0)

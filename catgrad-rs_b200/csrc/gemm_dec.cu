@@ -410,8 +410,9 @@ static int dec_splits(int64_t tiles, int kb_total) {
   const int cap = 3 * 148;
   int splits = 1;
   while (splits < 16 && tiles * (splits * 2) <= cap && kb_total / (splits * 2) >= 2) splits *= 2;
-  const int kb_per = (kb_total + splits - 1) / splits;
-  if ((kb_total + kb_per - 1) / kb_per != splits) splits = 1;  // an empty slice would break the cluster shape
+  // an empty slice would break the cluster shape
+  auto slices = [&](int s) { const int per = (kb_total + s - 1) / s; return (kb_total + per - 1) / per; };
+  while (splits > 1 && slices(splits) != splits) splits /= 2;
   return splits;
 }
 

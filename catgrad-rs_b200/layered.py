@@ -231,7 +231,7 @@ class LayeredConfig:
         if ".hc" in name:
             return {"in": 1.0, "out": 1.0, "mix": 0.0}[leaf] / self.streams, 0.5 / self.streams
         if leaf in ("correction", "sink"):
-            return 0.0, 0.01 if leaf == "correction" else 1.0
+            return 0.0, 0.001 if leaf == "correction" else 1.0
         return 0.0, 0.02
 
 
@@ -246,6 +246,21 @@ def bench_shape(name: str, width: int, ff: int, vocab: int) -> LayeredConfig:
     return LayeredConfig(name, width, vocab, [ssd, lat, dlt, ssd, lat, dlt, ssd, dlt], (1, 4, 2))
 
 
+def segedra_shape(name: str, width: int, heads: int, kv_heads: int, dim: int, window: int, experts: Experts, ff: int, dense_ff: int,
+                  streams: int, vocab: int) -> LayeredConfig:
+    """A Segedra-shaped model at a real model's widths, for measurements: a dense layer, then layers of
+    experts, a loop over three of them, every third layer without a window."""
+    def layer(i):
+        m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "rot": {"base": 150000.0, "dims": dim},
+             "mask": None if i % 3 == 2 else {"size": window}}
+        return LayerSpec("attention", m, ff, BOUNDED, experts) if i else LayerSpec("attention", m, dense_ff, RELU2)
+    return LayeredConfig(name, width, vocab, [layer(i) for i in range(8)], (1, 4, 2), 1e-5, design=DESIGNS["Segedra"], streams=streams,
+                         embed_scale=width ** 0.5)
+
+
+SEGEDRA_W1024 = segedra_shape("segedra-w1024-shape", 1024, 16, 4, 64, 128, Experts(32, 4, 1.0, 7.0), 512, 4096, 2, 32000)
+SEGEDRA_W2048 = segedra_shape("segedra-w2048-shape", 2048, 32, 4, 128, 512, Experts(128, 8, 2.5, 7.0), 768, 8192, 4, 151936)
+SEGEDRA_W2880 = segedra_shape("segedra-w2880-shape", 2880, 64, 8, 64, 128, Experts(32, 4, 1.0, 7.0), 2880, 11520, 4, 201088)
 RALAPEL_W1024 = bench_shape("ralapel-w1024-shape", 1024, 4096, 32000)
 RALAPEL_W2048 = bench_shape("ralapel-w2048-shape", 2048, 8192, 128256)
 RALAPEL_W4096 = bench_shape("ralapel-w4096-shape", 4096, 14336, 128256)
