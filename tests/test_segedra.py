@@ -74,7 +74,7 @@ def weights(cfg, seed=0):
 
 def sure(gaps, n):
     """Tokens none of whose expert choices is a close call."""
-    return np.min(gaps, axis=0) > 0.03 if gaps else np.ones(n, bool)
+    return np.min(gaps, axis=0) > 0.02 if gaps else np.ones(n, bool)
 
 
 def expected(cfg, W, seq, **kw):
@@ -86,7 +86,7 @@ def expected(cfg, W, seq, **kw):
 
 def agrees(got, want, ok, prec):
     ok = np.asarray(ok) if prec == "bf16" else np.ones(len(want), bool)
-    assert ok.mean() > 0.4 or len(ok) < 20
+    assert ok.mean() > 0.25 or len(ok) < 20
     return not ok.any() or close(np.asarray(got)[ok], np.asarray(want)[ok], prec)
 
 
