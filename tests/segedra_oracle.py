@@ -19,7 +19,7 @@ def rms(x, eps):
 
 
 def norm(x, w, eps):
-    """Weights are stored around zero."""
+    """RMS norm with the gain 1 + w."""
     return rms(x, eps) * (1.0 + w)
 
 
