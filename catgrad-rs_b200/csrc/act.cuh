@@ -38,4 +38,7 @@ __device__ __forceinline__ float relu2_f(float x) {
   return x * x;
 }
 
+// What a GEMM stores in bf16: output mode 1 the product itself, 4 the square of its relu, 5 its silu.
+__device__ __forceinline__ float bf16_out(int mode, float v) { return mode == 4 ? relu2_f(v) : mode == 5 ? silu_fast(v) : v; }
+
 }  // namespace cg

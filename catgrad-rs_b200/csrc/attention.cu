@@ -81,16 +81,19 @@ __global__ void __launch_bounds__(BQ * 2, D <= 64 ? 2 : 1) k_attn_prefill(AttnAr
   const int64_t last_q = start_pos + std::min<int64_t>(len, q0 + BQ) - 1;  // last query position of this tile
   int64_t first_k = 0;
   if (a.window > 0) first_k = std::max<int64_t>(0, start_pos + q0 - a.window + 1);
-  const int64_t kt0 = first_k / BKV, kt1 = last_q / BKV;  // inclusive key tile range
+  // key tiles: nk of kept first tokens, then kt0 .. last_q / BKV
+  const int64_t keep = a.window > 0 ? a.keep_first : 0;
+  const int64_t kt0 = first_k / BKV, nk = std::min<int64_t>(kt0, (keep + BKV - 1) / BKV), n_it = nk + last_q / BKV + 1 - kt0;
 
   const uint32_t sq_u = (uint32_t)__cvta_generic_to_shared(sq);
   const uint32_t sk_u = (uint32_t)__cvta_generic_to_shared(sk);
   const uint32_t sv_u = (uint32_t)__cvta_generic_to_shared(sv);
   const float LOG2E = 1.4426950408889634f;
 
-  // asynchronous copy of key/value tile kt into buffer buf (rows past the context are zero)
-  auto load_kv = [&](int buf, int64_t kt) {
-    const int64_t k0 = kt * BKV;
+  // asynchronous copy of the it-th key/value tile into buffer buf (rows past the context are zero)
+  auto tile_of = [&](int64_t it) { return it < nk ? it : kt0 + it - nk; };
+  auto load_kv = [&](int buf, int64_t it) {
+    const int64_t k0 = tile_of(it) * BKV;
     for (int i = tid; i < BKV * CH; i += NT) {
       const int r = i / CH, ch = i - r * CH;
       const bool in = k0 + r < kv_len;
@@ -101,18 +104,18 @@ __global__ void __launch_bounds__(BQ * 2, D <= 64 ? 2 : 1) k_attn_prefill(AttnAr
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  if (kt0 <= kt1) load_kv(0, kt0);
+  load_kv(0, 0);
 
-  for (int64_t kt = kt0; kt <= kt1; ++kt) {
-    const int64_t k0 = kt * BKV;
-    const int buf = NBUF == 2 ? (int)((kt - kt0) & 1) : 0;
-    if (NBUF == 2 && kt < kt1) {
-      load_kv(buf ^ 1, kt + 1);  // that buffer was last read two tiles ago, before the barrier that ended the previous tile
+  for (int64_t it = 0; it < n_it; ++it) {
+    const int64_t k0 = tile_of(it) * BKV;
+    const int buf = NBUF == 2 ? (int)(it & 1) : 0;
+    if (NBUF == 2 && it + 1 < n_it) {
+      load_kv(buf ^ 1, it + 1);  // that buffer was last read two tiles ago, before the barrier that ended the previous tile
       asm volatile("cp.async.wait_group 1;" ::: "memory");
     } else {
       asm volatile("cp.async.wait_group 0;" ::: "memory");
     }
-    __syncthreads();  // tile kt (and, the first time, Q) visible to every warp
+    __syncthreads();  // this tile (and, the first time, Q) visible to every warp
     const uint32_t sk_b = sk_u + (uint32_t)(buf * BKV * LD * 2), sv_b = sv_u + (uint32_t)(buf * BKV * LD * 2);
 
     // S = Q K^T for this warp's 16 rows x 64 keys
@@ -148,7 +151,7 @@ __global__ void __launch_bounds__(BQ * 2, D <= 64 ? 2 : 1) k_attn_prefill(AttnAr
         const int64_t qp = qpos[e >> 1];
         float v = s[j][e] * scale;
         if (a.softcap > 0.f) v = a.softcap * tanh_sig(v / a.softcap);
-        const bool keep = kpos <= qp && kpos < kv_len && (a.window <= 0 || kpos > qp - a.window);
+        const bool keep = kpos <= qp && kpos < kv_len && (a.window <= 0 || kpos > qp - a.window || kpos < keep);
         v = keep ? v : -INFINITY;
         s[j][e] = v;
         mx[e >> 1] = fmaxf(mx[e >> 1], v);
@@ -206,7 +209,7 @@ __global__ void __launch_bounds__(BQ * 2, D <= 64 ? 2 : 1) k_attn_prefill(AttnAr
       }
     }
     __syncthreads();  // every warp is done with this buffer before a later copy overwrites it
-    if (NBUF == 1 && kt < kt1) load_kv(0, kt + 1);
+    if (NBUF == 1 && it + 1 < n_it) load_kv(0, it + 1);
   }
 
   // normalise and store
@@ -216,7 +219,9 @@ __global__ void __launch_bounds__(BQ * 2, D <= 64 ? 2 : 1) k_attn_prefill(AttnAr
     if (qi >= len) continue;
     float inv = lrow[r] > 0.f ? 1.f / lrow[r] : 0.f;
     if (a.sink) inv = sink_scale(mrow[r], lrow[r], a.sink[h]);
-    __nv_bfloat16* dst = a.out + (tok0 + qi) * (int64_t)a.nh * D + (int64_t)h * D;
+    inv *= a.out_scale;
+    if (a.gate) inv *= 1.f / (1.f + expf(-a.gate[(tok0 + qi) * a.ld_gate + h]));
+    __nv_bfloat16* dst = a.out + (tok0 + qi) * (a.ld_out > 0 ? a.ld_out : (int64_t)a.nh * D) + (int64_t)h * D;
 #pragma unroll
     for (int j = 0; j < D / 8; ++j) {
       __nv_bfloat162 v = __floats2bfloat162_rn(o[j][2 * r] * inv, o[j][2 * r + 1] * inv);

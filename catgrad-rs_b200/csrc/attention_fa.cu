@@ -40,7 +40,11 @@ struct FaArgs {
   int token_major;     // keys and values lie token after token, the heads side by side
   float scale_log2e;   // score factor (1 / sqrt(D)) * log2(e)
   int64_t window;      // 0 = none
+  int64_t keep;        // with a window: first positions that stay visible
   const float* sink;   // [nh] or null
+  const float* gate;   // [tokens, ld_gate] or null: sigmoid(gate) multiplies a head's output, as out_scale does
+  int64_t ld_gate, ld_out;
+  float out_scale;
   RowsDev rows;        // rows of unequal length (rows.rows > 0)
   int32_t* err;
 };
@@ -57,6 +61,9 @@ __device__ __forceinline__ uint64_t umma_desc_mn(uint32_t saddr, uint32_t chunk_
   d |= (uint64_t)2 << 61;                               // SWIZZLE_128B
   return d;
 }
+
+// the lowest n bits, n of any size
+__device__ __forceinline__ uint32_t bits_below(int n) { return n <= 0 ? 0u : n >= 32 ? 0xffffffffu : (1u << n) - 1u; }
 
 __device__ __forceinline__ float fast_exp2(float x) {
   float y;
@@ -125,9 +132,11 @@ k_attn_fa(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUt
   const int64_t q0 = (int64_t)qt * FA_BQ;
   if (q0 >= len) return;  // uniform over the CTA, before anything is allocated
   const int64_t last_q = start_pos + std::min<int64_t>(len, q0 + FA_BQ) - 1;
-  // key tiles j0 .. j0 + nt - 1
+  // key tiles: nk of kept first tokens, then from tile j0 on
   const int j0 = p.window > 0 ? (int)(std::max<int64_t>(0, start_pos + q0 - p.window + 1) / FA_BK) : 0;
-  const int nt = (int)(last_q / FA_BK) + 1 - j0;
+  const int nk = (int)std::min<int64_t>(j0, (p.keep + FA_BK - 1) / FA_BK);
+  const int nt = nk + (int)(last_q / FA_BK) + 1 - j0;
+  auto tile_of = [&](int j) { return j < nk ? j : j0 + j - nk; };
 
   if (tid == 0) {
     mbar_init(b_q_full, 1);
@@ -171,7 +180,7 @@ k_attn_fa(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUt
       bool ok = true;
       for (int j = 0; j < nt && ok; ++j) {
         const uint32_t buf = (uint32_t)j & 1u, ph = ((uint32_t)j >> 1) & 1u;
-        const int row = (int)(kvrow0 + (int64_t)(j0 + j) * FA_BK);
+        const int row = (int)(kvrow0 + (int64_t)tile_of(j) * FA_BK);
         if (j >= 2) {
           ok = mbar_wait(b_k_empty + 8 * buf, ph ^ 1u, cta_abort, p.err);
           if (!ok) break;
@@ -248,17 +257,20 @@ k_attn_fa(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUt
       ok = mbar_wait(b_s_full + 8 * buf, ph, cta_abort, p.err);
       if (!ok) break;
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-      const int k0 = (j0 + j) * FA_BK;
-      // a key column c of this tile is visible to this row iff low <= c <= lim (window and causal
-      // mask), tested as c - low <= lim - low without signs
+      const int k0 = tile_of(j) * FA_BK;
+      // a key column c of this tile is visible to this row iff low <= c <= lim (window and causal mask)
+      // or c <= lim and c < kept; a bit per column and group of 32
       const int64_t lim64 = qpos - k0;
       const int lim = lim64 > FA_BK ? FA_BK : (lim64 < -1 ? -1 : (int)lim64);
       const int64_t low64 = p.window > 0 ? lim64 - p.window + 1 : 0;
-      int low = low64 < 0 ? 0 : (low64 > 2 * FA_BK ? 2 * FA_BK : (int)low64);
-      if (lim < low) low = 2 * FA_BK;  // nothing in this tile: no column reaches it
-      const uint32_t span = lim < low ? 0u : (uint32_t)(lim - low);
+      const int low = low64 < 0 ? 0 : (low64 > FA_BK ? FA_BK : (int)low64);
+      const int64_t kept64 = p.keep - k0;
+      const int kept = kept64 < 0 ? 0 : (kept64 > FA_BK ? FA_BK : (int)kept64);
+      auto visible = [&](int c) {
+        return bits_below(lim + 1 - c * 32) & (~bits_below(low - c * 32) | bits_below(kept - c * 32));
+      };
       // uniform: some key may be masked for some row
-      const bool diag = (int64_t)k0 + FA_BK - 1 > start_pos + q0 || (p.window > 0 && k0 <= last_q - p.window);
+      const bool diag = (int64_t)k0 + FA_BK - 1 > start_pos + q0 || (p.window > 0 && k0 <= last_q - p.window && kept < FA_BK);
       const uint32_t s_addr = lane_base + buf * S_COLS;
       constexpr int NCH = FA_BK / 32;
       uint32_t va[32], vb[32];
@@ -276,9 +288,9 @@ k_attn_fa(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUt
 #pragma unroll
           for (int i = 0; i < 32; ++i) mx = fmaxf(mx, __uint_as_float(cur[i]));
         } else {
-          const int rel = c * 32 - low;
+          const uint32_t vis = visible(c);
 #pragma unroll
-          for (int i = 0; i < 32; ++i) mx = (uint32_t)(i + rel) <= span ? fmaxf(mx, __uint_as_float(cur[i])) : mx;
+          for (int i = 0; i < 32; ++i) mx = vis & (1u << i) ? fmaxf(mx, __uint_as_float(cur[i])) : mx;
         }
         if (c + 1 < NCH) asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
       }
@@ -300,15 +312,15 @@ k_attn_fa(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUt
         uint32_t* cur = (c & 1) ? vb : va;
         uint32_t* nxt = (c & 1) ? va : vb;
         if (c + 1 < NCH) tmem_ld32(s_addr + (uint32_t)(c + 1) * 32u, nxt);
-        const int rel = c * 32 - low;
+        const uint32_t vis = visible(c);
         uint32_t pk[16];
 #pragma unroll
         for (int i = 0; i < 32; i += 2) {
           float e0 = fast_exp2(fmaf(__uint_as_float(cur[i]), p.scale_log2e, -mc));
           float e1 = fast_exp2(fmaf(__uint_as_float(cur[i + 1]), p.scale_log2e, -mc));
           if (diag) {
-            e0 = (uint32_t)(i + rel) <= span ? e0 : 0.f;
-            e1 = (uint32_t)(i + 1 + rel) <= span ? e1 : 0.f;
+            e0 = vis & (1u << i) ? e0 : 0.f;
+            e1 = vis & (2u << i) ? e1 : 0.f;
           }
           ls += e0 + e1;
           const __nv_bfloat162 pr = __floats2bfloat162_rn(e0, e1);
@@ -358,7 +370,9 @@ k_attn_fa(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUt
         const float f = fast_exp2(mc - top);
         inv = f / (l * f + fast_exp2(sk - top));
       }
-      __nv_bfloat16* dst = p.out + (tok0 + qi) * (int64_t)p.nh * D + (int64_t)h * D;
+      inv *= p.out_scale;
+      if (p.gate) inv *= 1.f / (1.f + expf(-p.gate[(tok0 + qi) * p.ld_gate + h]));
+      __nv_bfloat16* dst = p.out + (tok0 + qi) * p.ld_out + (int64_t)h * D;
 #pragma unroll
       for (int c0 = 0; c0 < D; c0 += 8) {
         uint32_t w[4];
@@ -403,7 +417,10 @@ int launch_fa(cg_ctx* c, const AttnArgs& a) {
   p.token_major = tm ? 1 : 0;
   p.scale_log2e = 1.4426950408889634f * (a.scale > 0.f ? a.scale : 1.f / sqrtf((float)D));
   p.window = a.window > 0 ? a.window : 0;
+  p.keep = p.window ? std::max<int64_t>(a.keep_first, 0) : 0;
   p.sink = a.sink;
+  p.gate = a.gate; p.ld_gate = a.ld_gate; p.out_scale = a.out_scale;
+  p.ld_out = a.ld_out > 0 ? a.ld_out : (int64_t)a.nh * D;
   p.rows = a.rows;
   p.err = c->core->dev_err;
   dim3 grid((unsigned)((a.S + FA_BQ - 1) / FA_BQ), (unsigned)a.nh, (unsigned)(a.rows.rows ? a.rows.rows : a.B));
@@ -417,7 +434,7 @@ int launch_fa(cg_ctx* c, const AttnArgs& a) {
 bool attn_fa_supported(const AttnArgs& a) {
   return (a.d == 64 || a.d == 128) && a.softcap <= 0.f && !a.pos_dev && a.S >= 64 &&
          (a.rows.rows ? a.rows.M : a.B * a.S) < 2147483647ll && a.B * a.nkv * a.Tmax < 2147483647ll && ((uintptr_t)a.q % 16) == 0 &&
-         ((uintptr_t)a.k_cache % 16) == 0 && ((uintptr_t)a.v_cache % 16) == 0 && a.kv_ld % 8 == 0;
+         ((uintptr_t)a.k_cache % 16) == 0 && ((uintptr_t)a.v_cache % 16) == 0 && a.kv_ld % 8 == 0 && ((uintptr_t)a.out % 16) == 0 && a.ld_out % 8 == 0;
 }
 
 int k_launch_attn_fa(cg_ctx* c, const AttnArgs& a) {

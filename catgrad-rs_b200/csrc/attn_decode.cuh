@@ -78,16 +78,17 @@ __device__ __forceinline__ void attn_dec_item(const AttnDecArgs& a, float scale,
   __nv_bfloat16* kbase = a.k_cache + ((place * a.nkv + kvh) * a.Tmax) * (int64_t)D;
   __nv_bfloat16* vbase = a.v_cache + ((place * a.nkv + kvh) * a.Tmax) * (int64_t)D;
 
-  // this CTA's slice of the cached keys [lo, pos)
-  int64_t pos = pos_early, t0 = 0, t1 = 0;
+  // The visible cached keys are the kf kept first ones and [lo, pos); [t0, t1) is this CTA's slice of
+  // their sequence.
+  int64_t pos = pos_early, t0 = 0, t1 = 0, lo = 0, kf = 0;
   auto plan = [&]() {
-    int64_t lo = 0;
-    if (a.window > 0) lo = max((int64_t)0, pos - a.window + 1);
-    const int64_t span = pos - lo;
+    lo = a.window > 0 ? max((int64_t)0, pos - a.window + 1) : 0;
+    if constexpr (Env::kRows) kf = min(a.keep_first, lo);
+    const int64_t span = kf + pos - lo;
     int64_t per = (span + a.splits - 1) / a.splits;
     per = (per + KT - 1) / KT * KT;
-    t0 = lo + split * per;
-    t1 = min(pos, t0 + per);
+    t0 = split * per;
+    t1 = min(span, t0 + per);
   };
   plan();
 
@@ -104,7 +105,8 @@ __device__ __forceinline__ void attn_dec_item(const AttnDecArgs& a, float scale,
       const int r = i / CH, ch = i - r * CH;
       const int64_t key = c0 + r;
       const bool ok = key < t1;
-      const int64_t kc = ok ? key : t0;
+      int64_t kc = ok ? key : t0;
+      if (kc >= kf) kc += lo - kf;
       cp_async16(kw_u + (uint32_t)(r * LD + ch * 8) * 2u, kbase + kc * (int64_t)D + ch * 8, ok ? 16 : 0);
       cp_async16(vw_u + (uint32_t)(r * LD + ch * 8) * 2u, vbase + kc * (int64_t)D + ch * 8, ok ? 16 : 0);
     }
@@ -125,7 +127,12 @@ __device__ __forceinline__ void attn_dec_item(const AttnDecArgs& a, float scale,
 
   // ---- 1. q, k, v of the new token ----
   const int heads = a.nh + 2 * a.nkv;
-  const float* row = a.qkv + b * (int64_t)heads * D;
+  int64_t ld_row = (int64_t)heads * D, ld_out = (int64_t)a.nh * D;
+  if constexpr (Env::kRows) {
+    if (a.ld_qkv) ld_row = a.ld_qkv;
+    if (a.ld_out) ld_out = a.ld_out;
+  }
+  const float* row = a.qkv + b * ld_row;
   const float* qsrc = row + (int64_t)kvh * rep * D;
   const float* ksrc = row + ((int64_t)a.nh + kvh) * D;
   const float* vsrc = row + ((int64_t)a.nh + a.nkv + kvh) * D;
@@ -152,6 +159,17 @@ __device__ __forceinline__ void attn_dec_item(const AttnDecArgs& a, float scale,
         hsq[tid] = 1.f / sqrtf(((r[0] + r[1]) + (r[2] + r[3])) / (float)((tid ? a.nkv : a.nh) * a.norm_dim) + a.norm_eps);
       }
       env.sync_cta();
+    } else if (a.head_norm) {
+      // norms per head: hsq[h] of the query heads, hsq[rep] of the key head
+      for (int h = warp; h <= rep; h += 4) {
+        const float* src = h < rep ? qsrc + h * D : ksrc;
+        float ss = 0.f;
+        for (int e = lane; e < D; e += 32) { const float v = __ldcg(src + e); ss += v * v; }
+#pragma unroll
+        for (int o = 16; o; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+        if (lane == 0) hsq[h] = 1.f / sqrtf(ss / (float)a.norm_dim + a.norm_eps);
+      }
+      env.sync_cta();
     }
     // neighbouring components (2 j, 2 j + 1) of the first rot_dims turn together
     const int rh = a.rot_dims / 2;
@@ -166,6 +184,8 @@ __device__ __forceinline__ void attn_dec_item(const AttnDecArgs& a, float scale,
         if (a.q_gamma) {
           const float2 g = *((const float2*)(a.q_gamma + (kvh * rep + h) * D) + j);
           x1 *= hsq[0] * g.x; x2 *= hsq[0] * g.y;
+        } else if (a.head_norm) {
+          x1 *= hsq[h]; x2 *= hsq[h];
         }
         if (j < rh) {
           const float cs = ct[j], sn = st[j], t = x1;
@@ -181,6 +201,8 @@ __device__ __forceinline__ void attn_dec_item(const AttnDecArgs& a, float scale,
       if (a.q_gamma) {
         const float2 g = *((const float2*)(a.k_gamma + kvh * D) + j);
         x1 *= hsq[1] * g.x; x2 *= hsq[1] * g.y;
+      } else if (a.head_norm) {
+        x1 *= hsq[rep]; x2 *= hsq[rep];
       }
       if (j < rh) {
         const float cs = ct[j], sn = st[j], t = x1;
@@ -383,9 +405,11 @@ __device__ __forceinline__ void attn_dec_item(const AttnDecArgs& a, float scale,
   float* part_ml = (float*)vt;                 // [MAX_REP][2]
   float* part_o = part_ml + 2 * MAX_REP;       // [MAX_REP][D]
   const int S = a.splits;
-  // the merged output oo over the merged sum ll of exp(score - mm), which the sink joins
+  // the merged output oo over the merged sum ll of exp(score - mm), which the sink joins, gated and scaled
   auto finished = [&](int r, float mm, float ll, float oo) {
     if constexpr (Env::kRows) {
+      oo *= a.out_scale;
+      if (a.gate) oo *= 1.f / (1.f + __expf(-__ldcg(a.gate + b * a.ld_gate + kvh * rep + r)));
       if (a.sink) {
         const float sk = a.sink[kvh * rep + r], top = fmaxf(mm, sk);
         const float f = __expf(mm - top);
@@ -459,7 +483,7 @@ __device__ __forceinline__ void attn_dec_item(const AttnDecArgs& a, float scale,
         ll += ls[s] * f;
         oo += os[s] * f;
       }
-      a.out[(b * a.nh + kvh * rep + r) * (int64_t)D + (i - r * D)] = __float2bfloat16_rn(finished(r, mm, ll, oo));
+      a.out[b * ld_out + (kvh * rep + r) * (int64_t)D + (i - r * D)] = __float2bfloat16_rn(finished(r, mm, ll, oo));
     }
     return;
   }
@@ -468,7 +492,7 @@ __device__ __forceinline__ void attn_dec_item(const AttnDecArgs& a, float scale,
     for (int i = tid; i < rep * D; i += 128) {
       const int r = i / D, e = i - r * D;
       const float ll = part_ml[2 * r + 1];
-      a.out[(b * a.nh + kvh * rep + r) * (int64_t)D + e] = __float2bfloat16_rn(finished(r, part_ml[2 * r], ll, part_o[i]));
+      a.out[b * ld_out + (kvh * rep + r) * (int64_t)D + e] = __float2bfloat16_rn(finished(r, part_ml[2 * r], ll, part_o[i]));
     }
     env.sync_cta();  // the partials are read: the next item of a resident CTA may reuse the space
     return;
@@ -499,7 +523,7 @@ __device__ __forceinline__ void attn_dec_item(const AttnDecArgs& a, float scale,
       ll += ls[s] * f;
       oo += os[s] * f;
     }
-    a.out[(b * a.nh + kvh * rep + r) * (int64_t)D + (i - r * D)] = __float2bfloat16_rn(finished(r, mm, ll, oo));
+    a.out[b * ld_out + (kvh * rep + r) * (int64_t)D + (i - r * D)] = __float2bfloat16_rn(finished(r, mm, ll, oo));
   }
   // nobody leaves while a peer may still read its shared memory
   env.sync_group();

@@ -2,23 +2,29 @@
 // their weights, per-sequence caches and states, and the walk over their layers.  The entry points
 // (prefill, append, decode with its captured graph, generate) are those of decoder.cu.
 //
-// A sequence lives in a slot.  Per layer run (a looped layer counts once per pass) a slot holds
+// A sequence lives in a slot.  Per layer run (a looped layer counts once per pass, a layer with another
+// one's parameters is a run of that layer) a slot holds
 //   attention          [kv heads, max_seq, head size] keys and values
 //   latent attention   [max_seq, Lw] cached rows (normed latent, rotated key part)
 //   delta, ssd         an f32 matrix per head and the last inputs of the convolutions
+//   lightning          an f32 matrix per head
+// (of two mixers side by side, both their parts).
 // Nothing is cleared when a slot is reused: a row whose first position is 0 starts from zeros.
 // Batches are rows of unequal length, packed token after token; every kernel finds a token's row,
 // slot and position through the row tables (RowsDev).  In a decode step the tables stay as they
 // are and a device counter moves all positions, so the step is one CUDA graph.
 //
-// Fused steps: all projections of a mixer are one GEMM (w_in); a post-norm, the residual add and
+// Fused steps: all projections of a mixer, or of two side by side, are one GEMM (w_in), their two output
+// projections one more with their sum (w_o); a post-norm, the residual add and
 // the next pre-norm are one pass (k_row_update), which also writes the two-part rows a looped
-// input reads.  Without post-norms that pass is k_stream_update: the weighted sum over a token's
+// input reads and takes the sum over a token's experts.  Factors on norms' results and on a mixer's
+// gains are folded into the f32 gains.  Without post-norms that pass is k_stream_update: the weighted sum over a token's
 // experts, the mixing of the residual streams (a plain residual stream is one stream with unit
 // coefficients), the next sublayer's input and its norm.  Matrices are padded with zeros to multiples
 // of 8 (attention heads to the sizes of its tensor-core kernels) where the tensor cores want it.
 
 #include <algorithm>
+#include <cmath>
 #include <cstring>
 
 #include "decoder.h"
@@ -33,7 +39,11 @@ inline int64_t up16(int64_t n) { return (n + 15) / 16 * 16; }
 
 struct MixedLayer {
   cg_layer_config k{};
+  std::vector<double> decay;            // lightning
+  std::unique_ptr<MixedLayer> beside;   // a second mixer: its mixer's members only
+  int64_t in_row = 0, out_col = 0;      // where this mixer starts in w_in (rows) and w_o (columns), which both share
   cg_tensor *n1 = nullptr, *n1b = nullptr, *n2 = nullptr, *n2b = nullptr;
+  cg_tensor *n1b_bias = nullptr, *n2b_bias = nullptr, *n1_bias = nullptr, *n2_bias = nullptr;
   cg_tensor *w_in = nullptr, *w_o = nullptr, *w_gu = nullptr, *w_down = nullptr;
   int64_t Np = 0;       // columns of the projection
   int64_t Fp = 0;       // padded feed-forward width
@@ -43,6 +53,7 @@ struct MixedLayer {
   cg_tensor *hc_in[2] = {nullptr, nullptr}, *hc_out[2] = {nullptr, nullptr}, *hc_mix[2] = {nullptr, nullptr};
   // experts, stacked
   cg_tensor *router = nullptr, *correction = nullptr, *we_gate = nullptr, *we_up = nullptr, *we_down = nullptr;
+  int64_t Fd = 0;       // padded width of w_gu: the dense feed-forward or the shared expert, 0 = neither
   // attention
   cg_tensor *q_gain = nullptr, *k_gain = nullptr, *sink = nullptr;
   int Dk = 0, Dv = 0;   // columns a key and a value head take
@@ -51,9 +62,15 @@ struct MixedLayer {
   int64_t Lw = 0;       // width of a cached row
   int dkv_off = 0, Dq = 0;
   // recurrences
-  cg_tensor *conv_w = nullptr, *conv_b = nullptr, *a_log = nullptr, *dt_bias = nullptr, *dskip = nullptr, *norm = nullptr;
+  cg_tensor *conv_w = nullptr, *conv_b = nullptr, *a_log = nullptr, *dt_bias = nullptr, *dskip = nullptr, *norm = nullptr,
+            *log_decay = nullptr;
   bool chunked = false;  // prompts run on the tensor cores, 64 tokens at a time
-  int H = 0, KH = 0, dk = 0, dv = 0, dvs = 0, C = 0, gate_off = 0, small_off = 0, q_off = 0, k_off = 0, v_off = 0;
+  int H = 0, KH = 0, dk = 0, dv = 0, dvs = 0, C = 0, gate_off = 0, small_off = 0, q_off = 0, k_off = 0, v_off = 0, qs = 0, vs = 0;
+
+  bool recurrent() const { return k.mixer == CG_MIX_DELTA || k.mixer == CG_MIX_SSD || k.mixer == CG_MIX_LIGHTNING; }
+  float out_scale() const { return k.out_scale != 0. ? (float)k.out_scale : 1.f; }
+  int64_t in_width() const { return Np + (beside ? beside->Np : 0); }
+  int64_t out_width() const { return Ko + (beside ? beside->Ko : 0); }
 };
 
 struct MixedRun {
@@ -62,6 +79,7 @@ struct MixedRun {
   cg_tensor *cache = nullptr;                  // latent attention; keys of attention
   cg_tensor *cache_v = nullptr;                // attention
   cg_tensor *state = nullptr, *tail = nullptr;  // recurrences
+  std::unique_ptr<MixedRun> beside;             // of the second mixer
 };
 
 struct MixedModel {
@@ -74,7 +92,7 @@ struct MixedModel {
   int streams = 1;
   float embed_scale = 1.f;
   int64_t Wp = 0;       // padded width of the residual stream
-  cg_tensor *embed_norm = nullptr, *w_loop = nullptr;
+  cg_tensor *embed_norm = nullptr, *w_loop = nullptr, *ln_f_bias = nullptr;
   // sequences
   std::vector<uint8_t> open;
   std::vector<int64_t> pos;     // tokens each slot holds
@@ -136,14 +154,19 @@ int f32_matrix(cg_decoder* D, const std::string& name, int64_t rows, int64_t col
   return place_all(D, name, rows, cols, *out, 0);
 }
 
-// norm gains as they are applied, after the 1 a design may add to the stored ones
-int gains(cg_decoder* D, const std::string& name, int64_t n, cg_tensor** out) {
-  if (!D->cfg.norm_plus_one) return norm_weight(D, name, n, out);
+// a vector as it is applied: times a factor, after the 1 a design may add to stored gains
+int gains(cg_decoder* D, const std::string& name, int64_t n, cg_tensor** out, float factor = 1.f, bool plus_one = false) {
+  if (!plus_one && factor == 1.f) return norm_weight(D, name, n, out);
   Hold w;
   CG_TRY(norm_weight(D, name, n, &w.t));
   CG_TRY(new2(D->c, ST_F32, 1, n, out, false));
   CG_CUDA(D->c, cudaMemcpyAsync((*out)->data(), w.t->data(), (size_t)n * 4, cudaMemcpyDeviceToDevice, D->c->core->stream));
-  return k_launch_add_scalar(D->c, (float*)(*out)->data(), n, 1.f);
+  return k_launch_affine(D->c, (float*)(*out)->data(), n, factor, plus_one ? factor : 0.f);
+}
+// gains and, of a layer norm, biases
+int norm_pair(cg_decoder* D, const std::string& name, cg_tensor** w, cg_tensor** b, float factor = 1.f) {
+  CG_TRY(gains(D, name, D->H, w, factor, D->cfg.norm_plus_one != 0));
+  return D->cfg.layer_norm ? gains(D, name + ".b", D->H, b, factor) : CG_OK;
 }
 // n heads of d values each, spread to heads of Dp with zeros between
 int head_gains(cg_decoder* D, const std::string& name, int64_t n, int64_t d, int64_t Dp, cg_tensor** out) {
@@ -158,7 +181,7 @@ int head_gains(cg_decoder* D, const std::string& name, int64_t n, int64_t d, int
 int coefficients(cg_decoder* D, const std::string& name, int64_t n, cg_tensor** out) {
   if (D->cfg.streams > 0) return norm_weight(D, name, n, out);
   CG_TRY(new2(D->c, ST_F32, 1, n, out));
-  return k_launch_add_scalar(D->c, (float*)(*out)->data(), n, 1.f);
+  return k_launch_affine(D->c, (float*)(*out)->data(), n, 1.f, 1.f);
 }
 
 int rope_tables(cg_decoder* D, const MixedLayer& L, cg_tensor** cos_t, cg_tensor** sin_t) {
@@ -166,7 +189,32 @@ int rope_tables(cg_decoder* D, const MixedLayer& L, cg_tensor** cos_t, cg_tensor
   CG_TRY(new2(D->c, ST_F32, D->cfg.max_seq, half, cos_t));
   CG_TRY(new2(D->c, ST_F32, D->cfg.max_seq, half, sin_t));
   if (!L.k.rot_dim) return CG_OK;
-  return k_launch_pair_rope_tables(D->c, L.k.rot_base, D->cfg.max_seq, L.k.rot_dim, (float*)(*cos_t)->data(), (float*)(*sin_t)->data());
+  PairRope f;
+  f.base = L.k.rot_base;
+  f.factor = L.k.rot_factor; f.low = L.k.rot_low; f.high = L.k.rot_high; f.original = L.k.rot_original;
+  return k_launch_pair_rope_tables(D->c, f, D->cfg.max_seq, L.k.rot_dim, (float*)(*cos_t)->data(), (float*)(*sin_t)->data());
+}
+
+// The rows of n heads of d queries or keys at dst's row `row`, Dp rows per head.  Kernels rotate
+// neighbouring components; where the design pairs i with i + r / 2, the rows are interleaved, which changes
+// neither scores nor norms.
+int place_heads(cg_decoder* D, const std::string& name, const cg_layer_config& k, int64_t n, int64_t d, int64_t Dp, cg_tensor* dst,
+                int64_t row) {
+  const int64_t W = D->H, half = k.rot_half ? k.rot_dim / 2 : 0;
+  cg_ctx* c = D->c;
+  for (int64_t h = 0; h < n; ++h) CG_TRY(place(D, name, n * d, W, h * d, d, 0, W, dst, row + h * Dp, 0));
+  if (half < 2) return CG_OK;
+  const size_t es = storage_bytes(dst->storage), line = (size_t)dst->dims[1] * es;
+  Hold t;
+  CG_TRY(new2(c, dst->storage, 2 * half, dst->dims[1], &t.t, false));
+  for (int64_t h = 0; h < n; ++h) {
+    char* at = (char*)dst->data() + (size_t)(row + h * Dp) * line;
+    CG_CUDA(c, cudaMemcpyAsync(t.t->data(), at, 2 * half * line, cudaMemcpyDeviceToDevice, c->core->stream));
+    for (int64_t i = 0; i < 2; ++i)
+      CG_CUDA(c, cudaMemcpy2DAsync(at + i * line, 2 * line, (char*)t.t->data() + i * half * line, line, line, (size_t)half,
+                                   cudaMemcpyDeviceToDevice, c->core->stream));
+  }
+  return CG_OK;
 }
 
 int finalize_attention(cg_decoder* D, MixedLayer& L, const std::string& mx) {
@@ -180,17 +228,17 @@ int finalize_attention(cg_decoder* D, MixedLayer& L, const std::string& mx) {
   const int Dp = X.f32 ? 0 : widest <= 64 ? 64 : widest <= 128 ? 128 : widest <= 256 ? 256 : 0;
   L.Dk = Dp ? Dp : (int)up8(d);
   L.Dv = L.Do = Dp ? Dp : (int)up8(dv);
-  L.Np = (H + G) * L.Dk + G * L.Dv;
+  L.gate_off = (int)((H + G) * L.Dk + G * L.Dv);
+  L.Np = up8(L.gate_off + (k.gate ? H : 0));
   L.Ko = H * L.Dv;
   CG_TRY(new2(c, st, L.Np, X.Wp, &L.w_in));
-  for (int64_t h = 0; h < H; ++h) CG_TRY(place(D, mx + "q", H * d, W, h * d, d, 0, W, L.w_in, h * L.Dk, 0));
-  for (int64_t g = 0; g < G; ++g) {
-    CG_TRY(place(D, mx + "k", G * d, W, g * d, d, 0, W, L.w_in, (H + g) * L.Dk, 0));
-    CG_TRY(place(D, mx + "v", G * dv, W, g * dv, dv, 0, W, L.w_in, (H + G) * L.Dk + g * L.Dv, 0));
-  }
+  CG_TRY(place_heads(D, mx + "q", k, H, d, L.Dk, L.w_in, 0));
+  CG_TRY(place_heads(D, mx + "k", k, G, d, L.Dk, L.w_in, H * L.Dk));
+  for (int64_t g = 0; g < G; ++g) CG_TRY(place(D, mx + "v", G * dv, W, g * dv, dv, 0, W, L.w_in, (H + G) * L.Dk + g * L.Dv, 0));
+  if (k.gate) CG_TRY(place_all(D, mx + "g", H, W, L.w_in, L.gate_off));
   CG_TRY(new2(c, st, X.Wp, L.Ko, &L.w_o));
   for (int64_t h = 0; h < H; ++h) CG_TRY(place(D, mx + "o", W, H * dv, 0, W, h * dv, dv, L.w_o, 0, h * L.Dv));
-  if (k.qk_norm) {
+  if (k.qk_norm == 1) {
     CG_TRY(head_gains(D, mx + "q.norm", H, d, L.Dk, &L.q_gain));
     CG_TRY(head_gains(D, mx + "k.norm", G, d, L.Dk, &L.k_gain));
   }
@@ -211,7 +259,7 @@ int finalize_experts(cg_decoder* D, MixedLayer& L, const std::string& ff) {
   const int64_t W = D->H, F = L.k.ffn, E = L.k.experts;
   CG_TRY(new2(D->c, X.act_storage(), E, X.Wp, &L.router));
   CG_TRY(place_all(D, ff + "router", E, W, L.router, 0));
-  CG_TRY(norm_weight(D, ff + "correction", E, &L.correction));
+  if (L.k.correction) CG_TRY(norm_weight(D, ff + "correction", E, &L.correction));
   CG_TRY(stack_experts(D, ff, "gate", E, F, W, L.Fp, X.Wp, &L.we_gate));
   CG_TRY(stack_experts(D, ff, "up", E, F, W, L.Fp, X.Wp, &L.we_up));
   return stack_experts(D, ff, "down", E, W, F, X.Wp, L.Fp, &L.we_down);
@@ -259,6 +307,41 @@ int finalize_latent(cg_decoder* D, MixedLayer& L, const std::string& mx) {
   return rope_tables(D, L, &L.cos_t, &L.sin_t);
 }
 
+int finalize_lightning(cg_decoder* D, MixedLayer& L, const std::string& mx) {
+  cg_ctx* c = D->c;
+  MixedModel& X = *D->mixed;
+  const cg_layer_config& k = L.k;
+  const int64_t W = D->H, H = k.heads, d = k.dim, dv = k.vdim;
+  const int st = X.act_storage();
+  L.H = L.KH = k.heads;
+  L.dk = k.dim; L.dv = k.vdim;
+  L.dvs = (int)up8(dv);
+  // heads as far apart as the chunk kernels read them, so that the projection itself is their operand
+  L.qs = (int)up16(d); L.vs = L.dvs;
+  L.q_off = 0; L.k_off = (int)(H * L.qs); L.v_off = 2 * L.k_off;
+  L.C = L.v_off + (int)(H * L.vs);
+  L.chunked = !X.f32 && chunk_supported(L.dk);
+  L.gate_off = L.small_off = L.C;
+  L.Np = up8(L.C + H * dv);
+  L.Do = L.dv;
+  L.Ko = up8(H * dv);
+  CG_TRY(new2(c, st, L.Np, X.Wp, &L.w_in));
+  for (int64_t h = 0; h < H; ++h) {
+    CG_TRY(place(D, mx + "q", H * d, W, h * d, d, 0, W, L.w_in, L.q_off + h * L.qs, 0));
+    CG_TRY(place(D, mx + "k", H * d, W, h * d, d, 0, W, L.w_in, L.k_off + h * L.qs, 0));
+    CG_TRY(place(D, mx + "v", H * dv, W, h * dv, dv, 0, W, L.w_in, L.v_off + h * L.vs, 0));
+  }
+  CG_TRY(place_all(D, mx + "g", H * dv, W, L.w_in, L.gate_off));
+  CG_TRY(gains(D, mx + "norm", H * dv, &L.norm, L.out_scale()));
+  std::vector<float> ld(H);
+  for (int64_t h = 0; h < H; ++h) ld[h] = (float)std::log(std::max(L.decay[h], 1e-80));  // (as good as 0 after one token)
+  CG_TRY(new2(c, ST_F32, 1, H, &L.log_decay, false));
+  CG_CUDA(c, cudaMemcpyAsync(L.log_decay->data(), ld.data(), (size_t)H * 4, cudaMemcpyHostToDevice, c->core->stream));
+  CG_CUDA(c, cudaStreamSynchronize(c->core->stream));
+  CG_TRY(new2(c, st, X.Wp, L.Ko, &L.w_o));
+  return place_all(D, mx + "o", W, H * dv, L.w_o, 0);
+}
+
 int finalize_recurrent(cg_decoder* D, MixedLayer& L, const std::string& mx) {
   cg_ctx* c = D->c;
   MixedModel& X = *D->mixed;
@@ -275,6 +358,7 @@ int finalize_recurrent(cg_decoder* D, MixedLayer& L, const std::string& mx) {
   const int64_t kk = (int64_t)L.KH * L.dk;
   L.C = (int)(inner + 2 * kk);
   L.chunked = !X.f32 && chunk_supported(L.dk);
+  L.qs = L.dk; L.vs = L.dv;
   L.gate_off = (int)up8(L.C);
   L.small_off = (int)up8(L.gate_off + inner);
   L.Np = up8(L.small_off + (delta ? 2 : 1) * L.H);
@@ -291,7 +375,7 @@ int finalize_recurrent(cg_decoder* D, MixedLayer& L, const std::string& mx) {
     CG_TRY(place_all(D, mx + "q.conv", kk, taps, L.conv_w, L.q_off));
     CG_TRY(place_all(D, mx + "k.conv", kk, taps, L.conv_w, L.k_off));
     CG_TRY(place_all(D, mx + "v.conv", inner, taps, L.conv_w, L.v_off));
-    CG_TRY(norm_weight(D, mx + "norm", L.dv, &L.norm));
+    CG_TRY(gains(D, mx + "norm", L.dv, &L.norm, L.out_scale()));
   } else {
     // stored [z | x | B | C | dt]; the convolved channels come first here
     L.v_off = 0; L.k_off = (int)inner; L.q_off = (int)(inner + kk);
@@ -302,7 +386,7 @@ int finalize_recurrent(cg_decoder* D, MixedLayer& L, const std::string& mx) {
     CG_TRY(place_all(D, mx + "conv", L.C, taps, L.conv_w, 0));
     CG_TRY(norm_weight(D, mx + "conv.b", L.C, &L.conv_b));
     CG_TRY(norm_weight(D, mx + "D", L.H, &L.dskip));
-    CG_TRY(norm_weight(D, mx + "norm", inner, &L.norm));
+    CG_TRY(gains(D, mx + "norm", inner, &L.norm, L.out_scale()));
   }
   CG_TRY(norm_weight(D, mx + "A_log", L.H, &L.a_log));
   CG_TRY(norm_weight(D, mx + "dt_bias", L.H, &L.dt_bias));
@@ -310,6 +394,43 @@ int finalize_recurrent(cg_decoder* D, MixedLayer& L, const std::string& mx) {
   L.Ko = up8(inner);
   CG_TRY(new2(c, st, X.Wp, L.Ko, &L.w_o));
   return place_all(D, mx + "o", W, inner, L.w_o, 0);
+}
+
+int finalize_mixer(cg_decoder* D, MixedLayer& L, const std::string& mx) {
+  switch (L.k.mixer) {
+    case CG_MIX_ATTENTION: return finalize_attention(D, L, mx);
+    case CG_MIX_LATENT: return finalize_latent(D, L, mx);
+    case CG_MIX_LIGHTNING: return finalize_lightning(D, L, mx);
+    default: return finalize_recurrent(D, L, mx);
+  }
+}
+
+// two mixers' projections become one matrix, and their output projections one whose rows span both
+int finalize_beside(cg_decoder* D, MixedLayer& L, const std::string& mx) {
+  cg_ctx* c = D->c;
+  MixedModel& X = *D->mixed;
+  MixedLayer& R = *L.beside;
+  CG_TRY(finalize_mixer(D, L, mx + "left."));
+  CG_TRY(finalize_mixer(D, R, mx + "right."));
+  R.in_row = L.Np;
+  R.out_col = L.Ko;
+  Hold in, out;
+  CG_TRY(new2(c, X.act_storage(), L.in_width(), X.Wp, &in.t));
+  CG_TRY(new2(c, X.act_storage(), X.Wp, L.out_width(), &out.t));
+  const size_t es = storage_bytes(X.act_storage());
+  for (MixedLayer* m : {&L, &R}) {
+    CG_CUDA(c, cudaMemcpyAsync((char*)in.t->data() + (size_t)(m->in_row * X.Wp) * es, m->w_in->data(), (size_t)(m->Np * X.Wp) * es,
+                               cudaMemcpyDeviceToDevice, c->core->stream));
+    CG_CUDA(c, cudaMemcpy2DAsync((char*)out.t->data() + (size_t)m->out_col * es, (size_t)L.out_width() * es, m->w_o->data(), (size_t)m->Ko * es,
+                                 (size_t)m->Ko * es, (size_t)X.Wp, cudaMemcpyDeviceToDevice, c->core->stream));
+    drop(m->w_in);
+    drop(m->w_o);
+  }
+  L.w_in = in.take();
+  L.w_o = out.take();
+  R.w_in = L.w_in;
+  R.w_in->rc++;
+  return CG_OK;
 }
 
 void forget_graph(cg_decoder* D) {
@@ -322,16 +443,7 @@ int ensure_mixed(cg_decoder* D, int64_t M) {
   cg_ctx* c = D->c;
   forget_graph(D);  // it holds the old buffers
   int64_t np = 0, cc = 0, hh = 0, inner = 0, ko = 0, fp = 0, qw = 0, lw = 0, qkv = 0, kh = 0, top = 0, experts = 0, fe = 0;
-  for (const MixedLayer& L : X.layers) {
-    np = std::max(np, L.Np);
-    ko = std::max(ko, L.Ko);
-    if (L.k.experts) {
-      top = std::max<int64_t>(top, L.k.top_k);
-      experts = std::max<int64_t>(experts, L.k.experts);
-      fe = std::max(fe, L.Fp);
-    } else {
-      fp = std::max(fp, L.Fp);
-    }
+  auto count_mixer = [&](const MixedLayer& L) {
     if (L.k.mixer == CG_MIX_ATTENTION) {
       qw = std::max<int64_t>(qw, (int64_t)L.k.heads * L.Dk);
     } else if (L.k.mixer == CG_MIX_LATENT) {
@@ -346,6 +458,19 @@ int ensure_mixed(cg_decoder* D, int64_t M) {
         kh = std::max<int64_t>(kh, L.KH);
       }
     }
+  };
+  for (const MixedLayer& L : X.layers) {
+    if (!L.w_in) continue;  // another layer's parameters
+    np = std::max(np, L.in_width());
+    ko = std::max(ko, L.out_width());
+    fp = std::max(fp, L.Fd);
+    if (L.k.experts) {
+      top = std::max<int64_t>(top, L.k.top_k);
+      experts = std::max<int64_t>(experts, L.k.experts);
+      fe = std::max(fe, L.Fp);
+    }
+    count_mixer(L);
+    if (L.beside) count_mixer(*L.beside);
   }
   const int st = X.act_storage();
   CG_TRY(new2(c, ST_F32, M * X.streams, X.Wp, &X.x));
@@ -427,7 +552,7 @@ int lin(cg_decoder* D, const void* x, int64_t ldx, int64_t M, const cg_tensor* w
 int glu(cg_decoder* D, const MixedLayer& L, const void* x, int64_t M) {
   cg_ctx* c = D->c;
   MixedModel& X = *D->mixed;
-  const int64_t K = X.Wp, F = L.Fp;
+  const int64_t K = X.Wp, F = L.Fd;
   if (X.f32) {
     CG_TRY(lin(D, x, K, M, L.w_gu, 0, 2 * F, X.gu->data(), 2 * F));
     return k_launch_glu_f32(c, (const float*)X.gu->data(), M, F, L.k.act, (float*)X.hact->data());
@@ -445,26 +570,30 @@ int glu(cg_decoder* D, const MixedLayer& L, const void* x, int64_t M) {
   return gemm_tc_pair(c, xb, K, w, K, (__nv_bfloat16*)X.hact->data(), F, M, F, K, L.k.act);
 }
 
-// y = the dense feed-forward of the rows xn
+// y = the dense feed-forward or the shared expert of the rows xn
 int dense_ff(cg_decoder* D, const MixedLayer& L, int64_t M) {
   MixedModel& X = *D->mixed;
   if (L.k.act == CG_ACT_RELU2) {
-    CG_TRY(lin(D, X.xn->data(), X.Wp, M, L.w_gu, 0, L.Fp, X.hact->data(), L.Fp, X.f32 ? 0 : 4));
-    if (X.f32) CG_TRY(k_launch_relu2_f32(D->c, (float*)X.hact->data(), M * L.Fp));
+    CG_TRY(lin(D, X.xn->data(), X.Wp, M, L.w_gu, 0, L.Fd, X.hact->data(), L.Fd, X.f32 ? 0 : 4));
+    if (X.f32) CG_TRY(k_launch_relu2_f32(D->c, (float*)X.hact->data(), M * L.Fd));
   } else {
     CG_TRY(glu(D, L, X.xn->data(), M));
   }
-  return lin(D, X.hact->data(), L.Fp, M, L.w_down, 0, X.Wp, X.y->data(), X.Wp);
+  return lin(D, X.hact->data(), L.Fd, M, L.w_down, 0, X.Wp, X.y->data(), X.Wp);
 }
 
-// m_y[m_pos[pair]] = the chosen experts' results for the rows xn, m_wts their weights
+// m_y[m_pos[pair]] = the chosen experts' results for the rows xn, m_wts their weights (on the rows x itself
+// where the weights go onto the inputs)
 int experts_ff(cg_decoder* D, const MixedLayer& L, int64_t M) {
   cg_ctx* c = D->c;
   MixedModel& X = *D->mixed;
   MoeArgs a;
   a.H = (int)X.Wp; a.E = a.El = L.k.experts; a.e_lo = 0; a.k = L.k.top_k; a.Fe = (int)L.Fp;
   a.norm_topk = 0; a.act = L.k.act; a.act_limit = (float)L.k.act_limit;
-  a.correction = (const float*)L.correction->data(); a.router_scale = (float)L.k.router_scale;
+  a.correction = L.correction ? (const float*)L.correction->data() : nullptr;
+  a.router_scale = (float)L.k.router_scale;
+  a.sigmoid = L.k.scoring; a.weigh_input = L.k.weigh_input;
+  a.x = (const float*)X.x->data();
   a.M = M;
   a.logits = (float*)X.m_logits->data();
   a.w.ids = (uint32_t*)X.m_ids->data();
@@ -486,6 +615,12 @@ int experts_ff(cg_decoder* D, const MixedLayer& L, int64_t M) {
   a.w_down = (const __nv_bfloat16*)L.we_down->data();
   return moe_experts(c, a);
 }
+
+// Rows of a matrix some columns wide: where the first starts, and from one to the next.
+struct Rows {
+  void* p = nullptr;
+  int64_t ld = 0;
+};
 
 // What the host knows about a portion: per row its new tokens and the position of the first.
 struct Portion {
@@ -554,40 +689,45 @@ int grow(cg_ctx* c, int storage, int64_t n, cg_tensor** t, int64_t* have) {
 // One token per row: norms, rotation, cache append and attention in one kernel.  Longer rows: a pass
 // that norms, rotates and appends, then the prompt attention on the tensor cores.  f32, and sizes those
 // kernels do not have: one block per token and head.
-int attention_layer(cg_decoder* D, const MixedLayer& L, MixedRun& run, const RowsDev& rd, const Portion* p) {
+int attention_layer(cg_decoder* D, const MixedLayer& L, MixedRun& run, const RowsDev& rd, const Portion* p, Rows in, Rows out) {
   cg_ctx* c = D->c;
   MixedModel& X = *D->mixed;
   const cg_layer_config& k = L.k;
-  CG_TRY(lin(D, X.xn->data(), X.Wp, rd.M, L.w_in, 0, L.Np, X.proj->data(), L.Np));
+  const float* proj = (const float*)in.p;
+  const float* gate = k.gate ? proj + L.gate_off : nullptr;
   const float* q_gain = L.q_gain ? (const float*)L.q_gain->data() : nullptr;
   const float* k_gain = L.k_gain ? (const float*)L.k_gain->data() : nullptr;
   const float* sink = L.sink ? (const float*)L.sink->data() : nullptr;
   const bool tensor = !X.f32 && L.Dk == L.Dv && (L.Dk == 64 || L.Dk == 128 || L.Dk == 256);
   if (tensor && (!p || p->max_len == 1) && k.heads / k.kv_heads <= 8) {
     AttnDecArgs f{};
-    f.qkv = (const float*)X.proj->data();
+    f.qkv = proj; f.ld_qkv = in.ld;
     f.cos_t = (const float*)L.cos_t->data(); f.sin_t = (const float*)L.sin_t->data();
     f.q_gamma = q_gain; f.k_gamma = k_gain; f.norm_eps = D->cfg.rms_eps;
     f.k_cache = (__nv_bfloat16*)run.cache->data(); f.v_cache = (__nv_bfloat16*)run.cache_v->data();
-    f.out = (__nv_bfloat16*)X.att->data();
+    f.out = (__nv_bfloat16*)out.p; f.ld_out = out.ld;
+    f.head_norm = k.qk_norm == 2; f.keep_first = k.keep_first;
+    f.gate = gate; f.ld_gate = in.ld; f.out_scale = L.out_scale();
     f.Tmax = D->cfg.max_seq; f.B = rd.rows;
     f.nh = k.heads; f.nkv = k.kv_heads; f.d = L.Dk;
     f.window = k.window; f.rows = rd; f.rot_dims = k.rot_dim; f.norm_dim = k.dim;
     f.scale = (float)k.scale; f.sink = sink;
-    const int64_t reach = k.window > 0 ? std::min<int64_t>(k.window, f.Tmax) : f.Tmax;
+    const int64_t reach = k.window > 0 ? std::min<int64_t>((int64_t)k.window + k.keep_first, f.Tmax) : f.Tmax;
     f.splits = attn_dec_splits(reach, f.B * f.nkv, f.d);
     return k_launch_attn_dec(c, f);
   }
   RowsAttnArgs a;
-  a.proj = (const float*)X.proj->data(); a.ldp = L.Np;
+  a.proj = proj; a.ldp = in.ld;
   a.H = k.heads; a.G = k.kv_heads; a.d = k.dim; a.dv = k.vdim; a.Dk = L.Dk; a.Dv = L.Dv;
   a.q_gain = q_gain; a.k_gain = k_gain; a.eps = D->cfg.rms_eps; a.scale = (float)k.scale;
   a.rot = k.rot_dim;
   a.cos_t = (const float*)L.cos_t->data(); a.sin_t = (const float*)L.sin_t->data();
-  a.window = k.window; a.sink = sink;
+  a.window = k.window; a.keep_first = k.keep_first; a.sink = sink;
+  a.head_norm = k.qk_norm == 2;
+  a.gate = gate; a.out_scale = L.out_scale();
   a.q = X.q->data(); a.k_cache = run.cache->data(); a.v_cache = run.cache_v->data();
   a.Tmax = D->cfg.max_seq; a.slots = D->cfg.max_batch;
-  a.att = X.att->data(); a.ld_att = L.Ko;
+  a.att = out.p; a.ld_att = out.ld;
   a.bf16 = X.f32 ? 0 : 1;
   a.rows = rd;
   CG_TRY(k_launch_rows_qkv(c, a));
@@ -598,7 +738,8 @@ int attention_layer(cg_decoder* D, const MixedLayer& L, MixedRun& run, const Row
   t.out = (__nv_bfloat16*)a.att;
   t.B = a.slots; t.S = p->max_len; t.Tmax = a.Tmax;
   t.nh = a.H; t.nkv = a.G; t.d = L.Dk;
-  t.window = a.window; t.scale = a.scale; t.sink = sink; t.rows = rd;
+  t.window = a.window; t.keep_first = a.keep_first; t.scale = a.scale; t.sink = sink; t.rows = rd;
+  t.gate = gate; t.ld_gate = in.ld; t.out_scale = a.out_scale; t.ld_out = out.ld;
   return k_launch_attn_prefill(c, t);
 }
 
@@ -675,11 +816,13 @@ void recurrent_base(cg_decoder* D, const MixedLayer& L, MixedRun& run, const Row
   MixedModel& X = *D->mixed;
   a->delta = L.k.mixer == CG_MIX_DELTA ? 1 : 0;
   a->H = L.H; a->KH = L.KH; a->dk = L.dk; a->dv = L.dv; a->dvs = L.dvs; a->C = L.C; a->taps = L.k.conv;
-  a->q_off = L.q_off; a->k_off = L.k_off; a->v_off = L.v_off;
-  a->conv_w = (const float*)L.conv_w->data();
+  a->q_off = L.q_off; a->k_off = L.k_off; a->v_off = L.v_off; a->qs = L.qs; a->vs = L.vs;
+  a->conv_w = L.conv_w ? (const float*)L.conv_w->data() : nullptr;
   a->conv_b = L.conv_b ? (const float*)L.conv_b->data() : nullptr;
-  a->tail = (float*)run.tail->data();
-  a->a_log = (const float*)L.a_log->data(); a->dt_bias = (const float*)L.dt_bias->data();
+  a->tail = run.tail ? (float*)run.tail->data() : nullptr;
+  a->a_log = L.a_log ? (const float*)L.a_log->data() : nullptr;
+  a->dt_bias = L.dt_bias ? (const float*)L.dt_bias->data() : nullptr;
+  a->log_decay = L.log_decay ? (const float*)L.log_decay->data() : nullptr;
   a->dskip = L.dskip ? (const float*)L.dskip->data() : nullptr;
   a->S = (float*)run.state->data();
   a->gl = (float*)X.gl->data(); a->co = (float*)X.co->data();
@@ -687,37 +830,56 @@ void recurrent_base(cg_decoder* D, const MixedLayer& L, MixedRun& run, const Row
   a->rows = rd;
 }
 
-// One token per row: one kernel.  Prompts in a bf16 context: chunks on the tensor cores, on bf16
-// projections (the gates' projections stay f32).  Otherwise token by token.
-int recurrent_layer(cg_decoder* D, const MixedLayer& L, MixedRun& run, const RowsDev& rd, const Portion* p, const Chunks* ch) {
+// Prompts in a bf16 context run in chunks on the tensor cores
+bool in_chunks(const MixedLayer& L, const Portion* p) { return L.chunked && p && p->max_len >= 8; }
+
+// One token per row: one kernel.  Chunks take bf16 projections made here (the decays' and step sizes'
+// projections stay f32; lightning's queries, keys and values pass silu in the GEMM).  Otherwise token by token.
+int recurrent_layer(cg_decoder* D, const MixedLayer& L, MixedRun& run, const RowsDev& rd, const Portion* p, const Chunks* ch, Rows in,
+                    Rows out) {
   cg_ctx* c = D->c;
   MixedModel& X = *D->mixed;
   const int64_t M = rd.M, K = X.Wp;
+  const bool lightning = L.k.mixer == CG_MIX_LIGHTNING, delta = L.k.mixer == CG_MIX_DELTA;
   GatedNorm n;
-  n.delta = L.k.mixer == CG_MIX_DELTA ? 1 : 0;
-  n.H = L.H; n.dv = L.dv; n.dvs = L.dvs; n.norm_groups = L.k.norm_groups;
+  n.H = L.H; n.dv = L.dv; n.dvs = L.dvs;
+  n.groups = delta ? L.H : lightning ? 1 : L.k.norm_groups;
+  n.shared_gain = delta; n.gate_first = !delta && !lightning; n.sigmoid = lightning;
   n.o = (const float*)X.ro->data();
   n.norm = (const float*)L.norm->data(); n.eps = D->cfg.rms_eps;
-  n.att = X.att->data(); n.ld_att = L.Ko; n.att_bf16 = X.f32 ? 0 : 1;
+  n.att = out.p; n.ld_att = out.ld; n.att_bf16 = X.f32 ? 0 : 1;
   n.M = M;
-  if (L.chunked && p && p->max_len >= 8) {
+  if (in_chunks(L, p)) {
     ChunkArgs a;
     recurrent_base(D, L, run, rd, &a);
+    a.chunk_tok = ch->tok; a.chunk_len = ch->len; a.row_chunk = ch->row_chunk; a.n_chunks = ch->n;
+    a.DKp = (int)up16(L.dk); a.dvp = L.dvs;
+    a.q = (__nv_bfloat16*)X.qkv->data();
+    a.T = nullptr;
+    if (lightning) {
+      const int64_t ng = L.Np - L.C;
+      __nv_bfloat16* gate = (__nv_bfloat16*)X.proj->data();
+      CG_TRY(lin(D, X.xn->data(), K, M, L.w_in, L.in_row, L.C, a.q, L.C, 5));
+      CG_TRY(lin(D, X.xn->data(), K, M, L.w_in, L.in_row + L.C, ng, gate, ng, 1));
+      a.k = a.q + L.k_off; a.v = a.q + L.v_off;
+      a.ldq = a.ldv = L.C;
+      a.proj = nullptr; a.ldp = 0; a.small = nullptr; a.ld_small = 0; a.rq = a.rk = nullptr;
+      CG_TRY(k_launch_chunk_recurrence(c, a));
+      n.gate = gate; n.ldg = ng; n.gate_bf16 = 1;
+      return k_launch_gated_norm(c, n);
+    }
     __nv_bfloat16* pb = (__nv_bfloat16*)X.proj->data();
     float* small = (float*)(pb + M * L.small_off);  // both fit where the f32 projection would
     const int64_t ns = L.Np - L.small_off;
-    CG_TRY(lin(D, X.xn->data(), K, M, L.w_in, 0, L.small_off, pb, L.small_off, 1));
-    CG_TRY(lin(D, X.xn->data(), K, M, L.w_in, L.small_off, ns, small, ns));
+    CG_TRY(lin(D, X.xn->data(), K, M, L.w_in, L.in_row, L.small_off, pb, L.small_off, 1));
+    CG_TRY(lin(D, X.xn->data(), K, M, L.w_in, L.in_row + L.small_off, ns, small, ns));
     a.proj = pb; a.ldp = L.small_off;
     a.small = small; a.ld_small = ns;
-    a.DKp = (int)up16(L.dk); a.dvp = L.dvs;
-    a.q = (__nv_bfloat16*)X.qkv->data();
     a.k = a.q + M * L.KH * a.DKp;
     a.v = a.k + M * L.KH * a.DKp;
+    a.ldq = (int64_t)L.KH * a.DKp; a.ldv = (int64_t)L.H * a.dvp;
     a.rq = (float*)X.rn->data();
     a.rk = a.rq + M * L.KH;
-    a.chunk_tok = ch->tok; a.chunk_len = ch->len; a.row_chunk = ch->row_chunk; a.n_chunks = ch->n;
-    a.T = nullptr;
     if (a.delta) {
       CG_TRY(grow(c, ST_BF16, (int64_t)ch->n * L.H * 2 * RECUR_CHUNK * RECUR_CHUNK, &X.tinv, &X.tinv_n));
       a.T = (__nv_bfloat16*)X.tinv->data();
@@ -728,22 +890,44 @@ int recurrent_layer(cg_decoder* D, const MixedLayer& L, MixedRun& run, const Row
   }
   RecurArgs a;
   recurrent_base(D, L, run, rd, &a);
-  CG_TRY(lin(D, X.xn->data(), K, M, L.w_in, 0, L.Np, X.proj->data(), L.Np));
-  a.proj = (const float*)X.proj->data(); a.ldp = L.Np;
+  a.proj = (const float*)in.p; a.ldp = in.ld;
   a.gate_off = L.gate_off; a.small_off = L.small_off;
   a.cv = (float*)X.cv->data(); a.ldc = up8(L.C);
-  n.gate = a.proj + L.gate_off; n.ldg = L.Np; n.gate_bf16 = 0;
+  n.gate = a.proj + L.gate_off; n.ldg = in.ld; n.gate_bf16 = 0;
   if ((!p || p->max_len == 1) && recur_decode_supported(L.dk, L.dv)) return k_launch_recur_decode(c, a, n);
   CG_TRY(k_launch_recur_steps(c, a));
   return k_launch_gated_norm(c, n);
 }
 
+// y = the layer's mixer, or the sum of its two, of the rows xn.  The f32 projections of both are one GEMM
+// unless one of them makes its own.
 int mixer(cg_decoder* D, const MixedLayer& L, MixedRun& run, const RowsDev& rd, const Portion* p, const Chunks* ch) {
   MixedModel& X = *D->mixed;
-  if (L.k.mixer == CG_MIX_ATTENTION) CG_TRY(attention_layer(D, L, run, rd, p));
-  else if (L.k.mixer == CG_MIX_LATENT) CG_TRY(latent_layer(D, L, run, rd, p));
-  else CG_TRY(recurrent_layer(D, L, run, rd, p, ch));
-  return lin(D, X.att->data(), L.Ko, rd.M, L.w_o, 0, X.Wp, X.y->data(), X.Wp);
+  const int64_t M = rd.M, Ko = L.out_width();
+  if (L.k.mixer == CG_MIX_LATENT) {
+    CG_TRY(latent_layer(D, L, run, rd, p));
+  } else {
+    const size_t es = storage_bytes(X.act_storage());
+    const bool joint = L.beside && !in_chunks(L, p) && !in_chunks(*L.beside, p);
+    for (int side = 0; side < (L.beside ? 2 : 1); ++side) {
+      const MixedLayer& m = side ? *L.beside : L;
+      MixedRun& r = side ? *run.beside : run;
+      Rows in, out;
+      out.p = (char*)X.att->data() + (size_t)m.out_col * es; out.ld = Ko;
+      if (joint) {
+        in.ld = L.in_width();
+        in.p = (float*)X.proj->data() + m.in_row;
+        if (!side) CG_TRY(lin(D, X.xn->data(), X.Wp, M, L.w_in, 0, in.ld, X.proj->data(), in.ld));
+      } else if (!in_chunks(m, p)) {
+        in.ld = m.Np;
+        in.p = X.proj->data();
+        CG_TRY(lin(D, X.xn->data(), X.Wp, M, L.w_in, m.in_row, m.Np, in.p, m.Np));
+      }
+      if (m.k.mixer == CG_MIX_ATTENTION) CG_TRY(attention_layer(D, m, r, rd, p, in, out));
+      else CG_TRY(recurrent_layer(D, m, r, rd, p, ch, in, out));
+    }
+  }
+  return lin(D, X.att->data(), Ko, M, L.w_o, 0, X.Wp, X.y->data(), X.Wp);
 }
 
 // room for the residual streams of all layer runs of M tokens
@@ -825,6 +1009,8 @@ int final_rows(cg_decoder* D, const int32_t* pick, const int32_t* dst, int64_t n
     RowUpdate u;
     fill(u);
     u.g2 = (const float*)D->ln_f->data();
+    u.b2 = X.ln_f_bias ? (const float*)X.ln_f_bias->data() : nullptr;
+    u.centred = D->cfg.layer_norm;
     return k_launch_row_update(D->c, u, n, X.f32 ? 0 : 1);
   }
   StreamUpdate u;
@@ -845,17 +1031,25 @@ int walk(cg_decoder* D, const RowsDev& rd, const uint32_t* tokens, const Portion
   char* cat_lo = X.loop ? (char*)X.xcat->data() : nullptr;
   char* cat_hi = X.loop ? cat_lo + (size_t)Wp * storage_bytes(X.act_storage()) : nullptr;
   const size_t nruns = X.runs.size();
-  // what the row update leaves for run i: its normed input, or the first half of a pass's input rows
+  auto data = [](const cg_tensor* t) { return t ? (const float*)t->data() : nullptr; };
+  // the next sublayer's input rows: the stream, normed if the design has norms there
+  auto input_rows = [&](RowUpdate& u, const cg_tensor* g, const cg_tensor* b) {
+    u.out = X.xn->data(); u.ldo = Wp; u.g2 = data(g); u.b2 = data(b);
+  };
+  // what the row update leaves for run i: its input, or the first half of a pass's input rows
   auto hand_on = [&](RowUpdate& u, size_t i) {
     if (i >= nruns) return;
+    const MixedLayer& L = X.layers[X.runs[i].layer];
     if (X.runs[i].starts_pass) { u.out = cat_lo; u.ldo = 2 * Wp; u.g2 = nullptr; }
-    else { u.out = X.xn->data(); u.ldo = Wp; u.g2 = (const float*)X.layers[X.runs[i].layer].n1->data(); }
+    else input_rows(u, L.n1, L.n1_bias);
   };
   RowUpdate base;
+  base.centred = D->cfg.layer_norm;
   base.x = (float*)X.x->data(); base.ldx = Wp; base.eps = D->cfg.rms_eps; base.W = (int)W;
   {
     RowUpdate u = base;
     u.tokens = tokens; u.table = D->embed->data(); u.table_bf16 = D->embed->storage == ST_BF16; u.vocab = D->cfg.vocab;
+    u.scale = X.embed_scale;
     u.g1 = X.embed_norm ? (const float*)X.embed_norm->data() : nullptr;
     u.x0 = cat_hi; u.ld0 = 2 * Wp;
     hand_on(u, 0);
@@ -868,19 +1062,26 @@ int walk(cg_decoder* D, const RowsDev& rd, const uint32_t* tokens, const Portion
       CG_TRY(lin(D, cat_lo, 2 * Wp, M, X.w_loop, 0, Wp, X.y->data(), Wp));
       RowUpdate u = base;
       u.y = (const float*)X.y->data(); u.ldy = Wp;
-      u.out = X.xn->data(); u.ldo = Wp; u.g2 = (const float*)L.n1->data();
+      input_rows(u, L.n1, L.n1_bias);
       CG_TRY(k_launch_row_update(c, u, M, bf));
     }
     CG_TRY(mixer(D, L, run, rd, p, ch));
     RowUpdate u = base;
     u.y = (const float*)X.y->data(); u.ldy = Wp; u.add = 1;
-    u.g1 = (const float*)L.n1b->data();
+    u.g1 = data(L.n1b); u.b1 = data(L.n1b_bias);
     if (L.k.ffn) {
-      u.out = X.xn->data(); u.ldo = Wp; u.g2 = (const float*)L.n2->data();
+      input_rows(u, L.n2, L.n2_bias);
       CG_TRY(k_launch_row_update(c, u, M, bf));
-      CG_TRY(dense_ff(D, L, M));
-      u.g1 = (const float*)L.n2b->data();
-      u.out = nullptr; u.g2 = nullptr;
+      if (L.k.experts) {
+        CG_TRY(experts_ff(D, L, M));
+        u.ye = (const float*)X.m_y->data(); u.ldye = Wp;
+        u.pos = (const int32_t*)X.m_pos->data(); u.top = L.k.top_k;
+        u.wts = L.k.weigh_input ? nullptr : (const float*)X.m_wts->data();
+      }
+      if (L.Fd) CG_TRY(dense_ff(D, L, M));
+      else u.y = nullptr;
+      u.g1 = data(L.n2b); u.b1 = data(L.n2b_bias);
+      u.out = nullptr; u.g2 = u.b2 = nullptr;
     }
     hand_on(u, i + 1);
     CG_TRY(k_launch_row_update(c, u, M, bf));
@@ -908,17 +1109,50 @@ int mixed_create(cg_decoder* D, const cg_layer_config* layers, int n_layers, con
   X->streams = std::max(D->cfg.streams, 1);
   if (D->cfg.embed_scale != 0.f) X->embed_scale = D->cfg.embed_scale;
   if (D->cfg.streams < 0 || D->cfg.streams > MAX_STREAMS) return fail(D->c, CG_ERR_UNSUPPORTED, "decoder: at most 16 streams");
-  if (X->sandwich && (D->cfg.streams || X->embed_scale != 1.f || D->cfg.norm_plus_one))
-    return fail(D->c, CG_ERR_UNSUPPORTED, "decoder: post-norms go with one stream, plain gains and an unscaled embedding");
-  if (!X->sandwich && (D->cfg.embed_norm || D->cfg.loop_input))
-    return fail(D->c, CG_ERR_UNSUPPORTED, "decoder: a normed embedding and looped inputs go with post-norms");
+  if (X->sandwich && (D->cfg.streams || D->cfg.norm_plus_one))
+    return fail(D->c, CG_ERR_UNSUPPORTED, "decoder: post-norms go with one stream and plain gains");
+  if (!X->sandwich && (D->cfg.embed_norm || D->cfg.loop_input || D->cfg.layer_norm || (D->cfg.residual_mult != 0.f && D->cfg.residual_mult != 1.f) ||
+                       (D->cfg.logit_scale != 0.f && D->cfg.logit_scale != 1.f)))
+    return fail(D->c, CG_ERR_UNSUPPORTED, "decoder: a normed embedding, looped inputs, layer norms, residual and logit factors go with post-norms");
   X->layers.resize(n_layers);
+  auto take_mixer = [&](int i, MixedLayer& L, bool two) -> int {
+    const cg_layer_config& k = L.k;
+    if (k.heads < 1 || k.vdim < 1) return bad_size(D, i, "sizes must be positive");
+    X->recurrent = X->recurrent || L.recurrent();
+    if (k.mixer == CG_MIX_ATTENTION) {
+      if (k.dim < 1 || k.kv_heads < 1 || k.heads % k.kv_heads || k.window < 0 || k.keep_first < 0 || k.rot_dim < 0 || k.rot_dim % 2 ||
+          k.rot_dim > k.dim || (k.rot_dim && !(k.rot_base > 0)) || !(k.scale > 0) || k.qk_norm < 0 || k.qk_norm > 2 ||
+          (k.qk_norm == 1 && k.rot_half && k.rot_dim))
+        return bad_size(D, i, "attention sizes");
+      if (!k.window) L.k.keep_first = 0;
+    } else if (k.mixer == CG_MIX_LATENT) {
+      if (k.dim < 1 || k.rot_dim < 0 || k.rot_dim % 2 || k.kv_rank < 1 || (k.rot_dim && !(k.rot_base > 0)) || two)
+        return bad_size(D, i, "latent attention sizes");
+    } else if (k.mixer == CG_MIX_DELTA) {
+      if (k.dim < 1 || k.kv_heads < 1 || k.heads % k.kv_heads || k.conv < 1) return bad_size(D, i, "delta rule sizes");
+    } else if (k.mixer == CG_MIX_SSD) {
+      if (k.state < 1 || k.groups < 1 || k.heads % k.groups || k.norm_groups < 1 || (k.heads * k.vdim) % k.norm_groups || k.conv < 1)
+        return bad_size(D, i, "state space sizes");
+    } else if (k.mixer == CG_MIX_LIGHTNING) {
+      if (k.dim < 1 || !k.decay) return bad_size(D, i, "lightning attention sizes");
+      L.k.conv = 0;
+      L.decay.assign(k.decay, k.decay + k.heads);
+      for (double x : L.decay)
+        if (!(x >= 0. && x <= 1.)) return bad_size(D, i, "decays must be in [0, 1]");
+    } else return bad_size(D, i, "unknown mixer");
+    L.k.decay = nullptr;
+    L.k.beside = nullptr;
+    return CG_OK;
+  };
   for (int i = 0; i < n_layers; ++i) {
     const cg_layer_config& k = layers[i];
     X->layers[i].k = k;
-    if (k.heads < 1 || k.vdim < 1 || k.ffn < 0) return bad_size(D, i, "sizes must be positive");
+    if (k.weights_of < 0 || k.weights_of > n_layers || k.weights_of == i + 1 || (k.weights_of && layers[k.weights_of - 1].weights_of))
+      return bad_size(D, i, "weights of no layer");
+    if (k.ffn < 0 || k.shared_ffn < 0) return bad_size(D, i, "sizes must be positive");
+    if (k.shared_ffn && (!k.experts || !X->sandwich)) return bad_size(D, i, "a shared expert goes with experts and post-norms");
+    if (k.weigh_input && !X->sandwich) return bad_size(D, i, "weighted inputs of experts go with post-norms");
     if (k.ffn && k.experts) {
-      if (X->sandwich) return bad_size(D, i, "experts and post-norms do not go together");
       if (k.experts < 0 || k.experts > 1024 || k.top_k < 1 || k.top_k > 32 || k.top_k > k.experts)
         return bad_size(D, i, "1 to 1024 experts, at most 32 per token");
       if (k.act < CG_ACT_SILU || k.act > CG_ACT_BOUNDED || (k.act == CG_ACT_BOUNDED && !(k.act_limit > 0)))
@@ -926,30 +1160,23 @@ int mixed_create(cg_decoder* D, const cg_layer_config* layers, int n_layers, con
     } else if (k.ffn && k.act != CG_ACT_SILU && k.act != CG_ACT_GELU && k.act != CG_ACT_RELU2) {
       return bad_size(D, i, "activation of the feed-forward");
     }
-    if (!k.ffn) X->layers[i].k.experts = 0;
-    X->recurrent = X->recurrent || k.mixer == CG_MIX_DELTA || k.mixer == CG_MIX_SSD;
-    if (k.mixer == CG_MIX_ATTENTION) {
-      if (k.dim < 1 || k.kv_heads < 1 || k.heads % k.kv_heads || k.window < 0 || k.rot_dim < 0 || k.rot_dim % 2 || k.rot_dim > k.dim ||
-          (k.rot_dim && !(k.rot_base > 0)) || !(k.scale > 0))
-        return bad_size(D, i, "attention sizes");
-    } else if (k.mixer == CG_MIX_LATENT) {
-      if (k.dim < 1 || k.rot_dim < 0 || k.rot_dim % 2 || k.kv_rank < 1 || (k.rot_dim && !(k.rot_base > 0)))
-        return bad_size(D, i, "latent attention sizes");
-    } else if (k.mixer == CG_MIX_DELTA) {
-      if (k.dim < 1 || k.kv_heads < 1 || k.heads % k.kv_heads || k.conv < 1) return bad_size(D, i, "delta rule sizes");
-    } else if (k.mixer == CG_MIX_SSD) {
-      if (k.state < 1 || k.groups < 1 || k.heads % k.groups || k.norm_groups < 1 || (k.heads * k.vdim) % k.norm_groups || k.conv < 1)
-        return bad_size(D, i, "state space sizes");
-    } else return bad_size(D, i, "unknown mixer");
+    if (!k.ffn) X->layers[i].k.experts = X->layers[i].k.shared_ffn = 0;
+    if (k.beside) {
+      X->layers[i].beside = std::make_unique<MixedLayer>();
+      X->layers[i].beside->k = *k.beside;
+      CG_TRY(take_mixer(i, *X->layers[i].beside, true));
+    }
+    CG_TRY(take_mixer(i, X->layers[i], k.beside != nullptr));
   }
   const bool looped = loop && loop->times > 0 && loop->stop > loop->start;
   if (looped && (loop->start < 0 || loop->stop > n_layers)) return fail(D->c, CG_ERR_INVALID, "decoder: loop out of range");
   X->loop = looped && D->cfg.loop_input;
   auto add = [&](int i, bool starts) {
     MixedRun r;
-    r.layer = i;
+    r.layer = layers[i].weights_of ? layers[i].weights_of - 1 : i;
     r.starts_pass = starts;
-    X->runs.push_back(r);
+    if (X->layers[r.layer].beside) r.beside = std::make_unique<MixedRun>();
+    X->runs.push_back(std::move(r));
   };
   const int a = looped ? loop->start : n_layers, b = looped ? loop->stop : n_layers;
   for (int i = 0; i < a; ++i) add(i, false);
@@ -964,15 +1191,23 @@ int mixed_create(cg_decoder* D, const cg_layer_config* layers, int n_layers, con
 void mixed_destroy(cg_decoder* D) {
   MixedModel* X = D->mixed;
   if (!X) return;
-  for (MixedLayer& L : X->layers) {
-    for (cg_tensor** t : {&L.n1, &L.n1b, &L.n2, &L.n2b, &L.w_in, &L.w_o, &L.w_gu, &L.w_down, &L.c_gain, &L.uk, &L.uv, &L.w_kv, &L.cos_t,
+  auto drop_layer = [](MixedLayer& L) {
+    for (cg_tensor** t : {&L.n1, &L.n1b, &L.n2, &L.n2b, &L.n1_bias, &L.n1b_bias, &L.n2_bias, &L.n2b_bias, &L.log_decay, &L.w_in, &L.w_o, &L.w_gu, &L.w_down, &L.c_gain, &L.uk, &L.uv, &L.w_kv, &L.cos_t,
                           &L.sin_t, &L.conv_w, &L.conv_b, &L.a_log, &L.dt_bias, &L.dskip, &L.norm, &L.q_gain, &L.k_gain, &L.sink,
                           &L.router, &L.correction, &L.we_gate, &L.we_up, &L.we_down})
       drop(*t);
     for (int q = 0; q < 2; ++q) { drop(L.hc_in[q]); drop(L.hc_out[q]); drop(L.hc_mix[q]); }
+  };
+  auto drop_run = [](MixedRun& r) { drop(r.cache); drop(r.cache_v); drop(r.state); drop(r.tail); };
+  for (MixedLayer& L : X->layers) {
+    if (L.beside) drop_layer(*L.beside);
+    drop_layer(L);
   }
-  for (MixedRun& r : X->runs) { drop(r.cache); drop(r.cache_v); drop(r.state); drop(r.tail); }
-  for (cg_tensor** t : {&X->embed_norm, &X->w_loop, &X->tab_run, &X->tab_dec, &X->x, &X->xn, &X->xcat, &X->y, &X->proj, &X->cv, &X->gl,
+  for (MixedRun& r : X->runs) {
+    if (r.beside) drop_run(*r.beside);
+    drop_run(r);
+  }
+  for (cg_tensor** t : {&X->embed_norm, &X->ln_f_bias, &X->w_loop, &X->tab_run, &X->tab_dec, &X->x, &X->xn, &X->xcat, &X->y, &X->proj, &X->cv, &X->gl,
                         &X->co, &X->ro, &X->att, &X->hact, &X->gu, &X->q, &X->cpk, &X->tok, &X->xw, &X->kept, &X->qkv, &X->rn,
                         &X->tinv, &X->kv, &X->lat, &X->m_logits, &X->m_ids, &X->m_wts, &X->m_pos, &X->m_tiles, &X->m_xg, &X->m_h,
                         &X->m_y})
@@ -986,34 +1221,38 @@ int mixed_finalize(cg_decoder* D) {
   MixedModel& X = *D->mixed;
   const int64_t W = D->H;
   const int st = X.act_storage();
+  const bool pre = D->cfg.post_norms != 2;
+  const float mult = D->cfg.residual_mult != 0.f ? D->cfg.residual_mult : 1.f;
   for (size_t i = 0; i < X.layers.size(); ++i) {
     MixedLayer& L = X.layers[i];
+    if (L.k.weights_of) continue;
     const std::string l = "l" + std::to_string(i) + ".";
-    CG_TRY(gains(D, l + "norm1", W, &L.n1));
-    if (X.sandwich) CG_TRY(norm_weight(D, l + "norm1b", W, &L.n1b));
+    auto norms = [&](const std::string& n, cg_tensor** w, cg_tensor** wb, cg_tensor** after, cg_tensor** after_b) -> int {
+      if (pre) CG_TRY(norm_pair(D, n, w, wb));
+      return X.sandwich ? norm_pair(D, pre ? n + "b" : n, after, after_b, mult) : CG_OK;
+    };
+    CG_TRY(norms(l + "norm1", &L.n1, &L.n1_bias, &L.n1b, &L.n1b_bias));
     for (int q = 0; q < (L.k.ffn ? 2 : 1) && !X.sandwich; ++q) {
       const std::string hc = l + (q ? "hc2." : "hc1.");
       CG_TRY(coefficients(D, hc + "in", X.streams, &L.hc_in[q]));
       CG_TRY(coefficients(D, hc + "out", X.streams, &L.hc_out[q]));
       CG_TRY(coefficients(D, hc + "mix", (int64_t)X.streams * X.streams, &L.hc_mix[q]));
     }
-    if (L.k.mixer == CG_MIX_ATTENTION) CG_TRY(finalize_attention(D, L, l + "mix."));
-    else if (L.k.mixer == CG_MIX_LATENT) CG_TRY(finalize_latent(D, L, l + "mix."));
-    else CG_TRY(finalize_recurrent(D, L, l + "mix."));
+    CG_TRY(L.beside ? finalize_beside(D, L, l + "mix.") : finalize_mixer(D, L, l + "mix."));
     if (L.k.ffn) {
-      const int64_t F = L.k.ffn;
-      L.Fp = up8(F);
-      CG_TRY(gains(D, l + "norm2", W, &L.n2));
-      if (X.sandwich) CG_TRY(norm_weight(D, l + "norm2b", W, &L.n2b));
-      if (L.k.experts) {
-        CG_TRY(finalize_experts(D, L, l + "mlp."));
-      } else {
+      L.Fp = up8(L.k.ffn);
+      CG_TRY(norms(l + "norm2", &L.n2, &L.n2_bias, &L.n2b, &L.n2b_bias));
+      if (L.k.experts) CG_TRY(finalize_experts(D, L, l + "mlp."));
+      const int64_t F = L.k.experts ? L.k.shared_ffn : L.k.ffn;
+      if (F) {
+        const std::string ff = l + (L.k.experts ? "mlp.shared." : "mlp.");
         const bool gated = L.k.act != CG_ACT_RELU2;
-        CG_TRY(new2(c, st, (gated ? 2 : 1) * L.Fp, X.Wp, &L.w_gu));
-        if (gated) CG_TRY(place_all(D, l + "mlp.gate", F, W, L.w_gu, 0));
-        CG_TRY(place_all(D, l + "mlp.up", F, W, L.w_gu, gated ? L.Fp : 0));
-        CG_TRY(new2(c, st, X.Wp, L.Fp, &L.w_down));
-        CG_TRY(place_all(D, l + "mlp.down", W, F, L.w_down, 0));
+        L.Fd = up8(F);
+        CG_TRY(new2(c, st, (gated ? 2 : 1) * L.Fd, X.Wp, &L.w_gu));
+        if (gated) CG_TRY(place_all(D, ff + "gate", F, W, L.w_gu, 0));
+        CG_TRY(place_all(D, ff + "up", F, W, L.w_gu, gated ? L.Fd : 0));
+        CG_TRY(new2(c, st, X.Wp, L.Fd, &L.w_down));
+        CG_TRY(place_all(D, ff + "down", W, F, L.w_down, 0));
       }
     }
     // the originals of this layer are no longer needed
@@ -1023,8 +1262,7 @@ int mixed_finalize(cg_decoder* D) {
     }
   }
   const int64_t slots = D->cfg.max_batch;
-  for (MixedRun& r : X.runs) {
-    const MixedLayer& L = X.layers[r.layer];
+  auto open_run = [&](MixedRun& r, const MixedLayer& L) -> int {
     if (L.k.mixer == CG_MIX_ATTENTION) {
       CG_TRY(new2(c, st, slots * L.k.kv_heads * D->cfg.max_seq, L.Dk, &r.cache));
       CG_TRY(new2(c, st, slots * L.k.kv_heads * D->cfg.max_seq, L.Dv, &r.cache_v));
@@ -1032,8 +1270,14 @@ int mixed_finalize(cg_decoder* D) {
       CG_TRY(new2(c, st, slots * D->cfg.max_seq, L.Lw, &r.cache));
     } else {
       CG_TRY(new2(c, ST_F32, slots * L.H * L.dk, L.dvs, &r.state));
-      CG_TRY(new2(c, ST_F32, slots * L.k.conv, L.C, &r.tail));
+      if (L.k.conv) CG_TRY(new2(c, ST_F32, slots * L.k.conv, L.C, &r.tail));
     }
+    return CG_OK;
+  };
+  for (MixedRun& r : X.runs) {
+    const MixedLayer& L = X.layers[r.layer];
+    CG_TRY(open_run(r, L));
+    if (r.beside) CG_TRY(open_run(*r.beside, *L.beside));
   }
   if (X.loop) {
     CG_TRY(new2(c, st, X.Wp, 2 * X.Wp, &X.w_loop));
@@ -1041,7 +1285,7 @@ int mixed_finalize(cg_decoder* D) {
     CG_TRY(place(D, "loop.in", W, 2 * W, 0, W, W, W, X.w_loop, 0, X.Wp));
   }
   if (D->cfg.embed_norm) CG_TRY(norm_weight(D, "embed.norm", W, &X.embed_norm));
-  CG_TRY(gains(D, "final.norm", W, &D->ln_f));
+  CG_TRY(norm_pair(D, "final.norm", &D->ln_f, &X.ln_f_bias, D->cfg.logit_scale != 0.f ? D->cfg.logit_scale : 1.f));
   CG_TRY(new2(c, st, D->cfg.vocab, W, &D->embed, false));
   CG_TRY(place_all(D, "embed", D->cfg.vocab, W, D->embed, 0));
   if (D->cfg.tie_embeddings && X.Wp == W) {
@@ -1070,7 +1314,7 @@ int mixed_finalize(cg_decoder* D) {
   CG_TRY(new2(c, st, slots, X.Wp, &D->xl));
   // split-K partials of problems of at most 64 tokens
   int64_t widest = std::max<int64_t>(X.Wp, D->Vp);
-  for (const MixedLayer& L : X.layers) widest = std::max({widest, L.Np, 2 * L.Fp, (int64_t)L.k.experts});
+  for (const MixedLayer& L : X.layers) widest = std::max({widest, L.in_width(), 2 * L.Fp, 2 * L.Fd, (int64_t)L.k.experts});
   n = X.f32 ? 1 : std::max<int64_t>(8 * 64 * widest, (int64_t)300 * 128 * 256);
   CG_TRY(new_tensor(c, CG_F32, ST_F32, &n, 1, &D->splitk));
   D->splitk_floats = n;

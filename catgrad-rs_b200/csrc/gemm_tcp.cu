@@ -38,7 +38,7 @@ struct TcpArgs {
   const float* residual;
   int64_t ldo;
   int M, N, K;
-  int out_mode;   // 0 f32, 1 bf16, 2 f32 + residual (residual may alias out), 4 bf16 of the square of relu
+  int out_mode;   // 0 f32, 1 bf16, 2 f32 + residual (residual may alias out), 4 bf16 of the square of relu, 5 bf16 of silu
   int kb_total;
   int m_tiles, n_tiles;
   int row2_off;   // PAIR: rows between a gate row and its up row
@@ -241,7 +241,7 @@ k_gemm_tcp(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CU
                 if (p.out_mode == 0) ((float*)p.out)[(int64_t)m * p.ldo + n] = __uint_as_float(v[j]);
                 else
                   ((__nv_bfloat16*)p.out)[(int64_t)m * p.ldo + n] =
-                      __float2bfloat16_rn(p.out_mode == 4 ? relu2_f(__uint_as_float(v[j])) : __uint_as_float(v[j]));
+                      __float2bfloat16_rn(bf16_out(p.out_mode, __uint_as_float(v[j])));
               }
             }
           }

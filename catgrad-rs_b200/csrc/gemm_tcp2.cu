@@ -54,7 +54,7 @@ struct Tcp2Args {
   const float* residual;
   int64_t ldo;
   int M, N, K;
-  int out_mode;  // 0 f32, 1 bf16, 2 f32 + residual (residual may alias out), 4 bf16 of the square of relu
+  int out_mode;  // 0 f32, 1 bf16, 2 f32 + residual (residual may alias out), 4 bf16 of the square of relu, 5 bf16 of silu
   int kb_total;
   int m_tiles, n_tiles;
   int row2_off;  // GLU: rows between a gate row and its up row
@@ -314,7 +314,7 @@ k_gemm_tcp2(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ C
               for (int j = 0; j < 32; ++j) {
                 const int m = m0 + c0 + j;
                 const float a = __uint_as_float(cur[j]);
-                if (m < m_end) ((__nv_bfloat16*)p.out)[(int64_t)m * p.ldo + n] = __float2bfloat16_rn(p.out_mode == 4 ? relu2_f(a) : a);
+                if (m < m_end) ((__nv_bfloat16*)p.out)[(int64_t)m * p.ldo + n] = __float2bfloat16_rn(bf16_out(p.out_mode, a));
               }
             }
           }

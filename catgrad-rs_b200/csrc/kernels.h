@@ -99,6 +99,12 @@ struct AttnArgs {
   int64_t kv_ld = 0;
   float scale = 0.f;             // factor on the scores; 0 = 1 / sqrt(d)
   const float* sink = nullptr;   // [nh]: exp(sink[h]) joins the denominator of the softmax
+  int64_t keep_first = 0;        // with a window: these first positions stay visible
+  // head h of token m is multiplied by out_scale and, with a gate, by sigmoid(gate[m * ld_gate + h])
+  float out_scale = 1.f;
+  const float* gate = nullptr;
+  int64_t ld_gate = 0;
+  int64_t ld_out = 0;            // from one token of out to the next; 0 = nh d
   // rows.rows > 0: rows of unequal length, at most S tokens each, of a batch of rows.M tokens; q and out
   // are packed, the cache is [slots, nkv, Tmax, d] and B counts the slots (pos0 is unused)
   RowsDev rows;
@@ -135,8 +141,14 @@ struct AttnDecArgs {
   // at once ([nh d] and [nkv d] values, of which nh and nkv times norm_dim count for the mean)
   RowsDev rows;
   int rot_dims = 0, norm_dim = 0;
+  int head_norm = 0;             // rows: norms per head, without gains, over norm_dim components
   float scale = 0.f;             // factor on the scores; 0 = 1 / sqrt(d)
   const float* sink = nullptr;   // [nh]: exp(sink[h]) joins the denominator of the softmax
+  int64_t ld_qkv = 0, ld_out = 0;  // rows: from one token to the next; 0 = (nh + 2 nkv) d, nh d
+  int64_t keep_first = 0;        // rows: with a window, these first positions stay visible
+  float out_scale = 1.f;         // rows: head h of row b is multiplied by out_scale and, with a gate, by
+  const float* gate = nullptr;   // sigmoid(gate[b * ld_gate + h])
+  int64_t ld_gate = 0;
   int push_merge;                // set by the launcher: the slices' partials are pushed to the finishing CTA
 };
 // Rope + cache append + attention + merge of one new token per row, in one launch.
@@ -194,7 +206,7 @@ struct DecGemm {
   const float* residual;
   int out_mode;             // 0: f32, 1: bf16, 2: f32 out = product + residual,
                             // 3: the product is pushed as this rank's addend of an all-reduce (out unused)
-                            // 4: bf16, the square of relu
+                            // 4: bf16, the square of relu; 5: bf16, silu
   const PeerPush* push;     // for out_mode 3
   // Norm hand-over between consecutive GEMMs (RMSNorm(x) W^T = (x g) W^T / rms(x) row by row):
   // a residual GEMM (out_mode 2) that is followed by a norm can also write xb_out = bf16(out * g)
@@ -239,9 +251,11 @@ struct MoeArgs {
   float* logits;              // [M, E] scratch for router3
   const __nv_bfloat16 *w_gate, *w_up;  // [El, Fe, H] experts this rank owns
   const __nv_bfloat16* w_down;         // [El, H, Fe]
-  const float* correction = nullptr;  // [E]: experts are chosen by probability + correction and weighted by
-                              // probability * router_scale
-  float router_scale = 1.f;
+  const float* correction = nullptr;  // [E]: experts are chosen by probability + correction
+  float router_scale = 1.f;   // factor on the weights
+  int sigmoid = 0;            // 1: an expert's probability is the sigmoid of its own logit
+  int weigh_input = 0;        // moe_experts, moe_experts_f32: the weights multiply the experts' inputs, which are the
+                              // f32 rows x here
   float act_limit = 0.f;      // of the bounded activation
   int H, E, k, Fe, norm_topk, act;
   int e_lo, El;               // this rank owns experts [e_lo, e_lo + El)
@@ -257,7 +271,7 @@ int moe_ffn(cg_ctx* c, const MoeArgs& a);
 // experts' results, a.w.y[a.w.pos[pair]] (the weighted sum is the caller's).
 int moe_topk(cg_ctx* c, const MoeArgs& a);
 int moe_experts(cg_ctx* c, const MoeArgs& a);
-// The latter in f32 (h [pairs, Fe]; a.w.xg holds [pairs] words)
+// The latter in f32 (h [pairs, Fe]; a.w.xg holds 2 [pairs] words)
 int moe_experts_f32(cg_ctx* c, const MoeArgs& a, const float* x, const float* w_gate, const float* w_up, const float* w_down, float* h);
 // out[M, N] = x[M, K] w[N, K]^T in f32 (CUDA cores)
 int gemm_nt_f32(cg_ctx* c, const float* x, int64_t ldx, const float* w, int64_t ldw, float* out, int64_t ldo, int64_t M, int64_t N,

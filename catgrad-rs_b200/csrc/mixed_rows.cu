@@ -33,15 +33,51 @@ __device__ __forceinline__ void store4(__nv_bfloat16* p, const float* v) {
 }
 
 
-// v = v * inv * g for vector i of a row
+// v = v * inv * g + b for vector i of a row, b may be null
 template <bool EXACT>
-__device__ __forceinline__ void gain(float* v, float inv, const float* g, int i, int W) {
+__device__ __forceinline__ void gain(float* v, float inv, const float* g, int i, int W, const float* b = nullptr) {
   if (EXACT) {
     const float4 w = *(const float4*)(g + 4 * i);
     v[0] *= inv * w.x; v[1] *= inv * w.y; v[2] *= inv * w.z; v[3] *= inv * w.w;
+    if (b) {
+      const float4 t = *(const float4*)(b + 4 * i);
+      v[0] += t.x; v[1] += t.y; v[2] += t.z; v[3] += t.w;
+    }
   } else {
 #pragma unroll
-    for (int e = 0; e < 4; ++e) v[e] = 4 * i + e < W ? v[e] * (inv * g[4 * i + e]) : 0.f;
+    for (int e = 0; e < 4; ++e) v[e] = 4 * i + e < W ? v[e] * (inv * g[4 * i + e]) + (b ? b[4 * i + e] : 0.f) : 0.f;
+  }
+}
+
+// The norm of a row whose vectors the block's threads hold: thread t has vectors t + j blockDim.x, the
+// columns past W are zero and stay so.
+template <int VEC, bool EXACT>
+__device__ __forceinline__ void norm_row(float (*v)[4], int centred, float eps, const float* g, const float* b, int nv, int n4, int W,
+                                         float* sh) {
+  if (centred) {
+    float s = 0.f;
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) s += (v[j][0] + v[j][1]) + (v[j][2] + v[j][3]);
+    const float mean = block_sum(s, sh) / (float)W;
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) {
+      const int i = threadIdx.x + j * blockDim.x;
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        if (j < nv && i < n4 && (EXACT || 4 * i + e < W)) v[j][e] -= mean;
+    }
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < VEC; ++j)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) ss += v[j][e] * v[j][e];
+  ss = block_sum(ss, sh);
+  const float inv = 1.f / sqrtf(ss / (float)W + eps);
+#pragma unroll
+  for (int j = 0; j < VEC; ++j) {
+    const int i = threadIdx.x + j * blockDim.x;
+    if (j < nv && i < n4) gain<EXACT>(v[j], inv, g, i, W, b);
   }
 }
 
@@ -70,7 +106,6 @@ __global__ void k_row_update(RowUpdate u, int32_t* err) {
       tok = u.tokens[m];
       if (tok >= u.vocab) { if (threadIdx.x == 0) *err = DEV_INDEX; tok = 0; }
     }
-    float ss = 0.f;
     float4 old[RU_VEC];  // requested before the reduction
 #pragma unroll
     for (int j = 0; j < RU_VEC; ++j) {
@@ -89,27 +124,28 @@ __global__ void k_row_update(RowUpdate u, int32_t* err) {
           for (int e = 0; e < 4; ++e)
             if (4 * i + e < W)
               v[j][e] = u.table_bf16 ? __bfloat162float(((const __nv_bfloat16*)u.table)[o + e]) : ((const float*)u.table)[o + e];
+#pragma unroll
+          for (int e = 0; e < 4; ++e) v[j][e] *= u.scale;
         } else {
-          const float4 t = *(const float4*)(u.y + m * u.ldy + 4 * i);
-          v[j][0] = t.x; v[j][1] = t.y; v[j][2] = t.z; v[j][3] = t.w;
+          if (u.y) {
+            const float4 t = *(const float4*)(u.y + m * u.ldy + 4 * i);
+            v[j][0] = t.x; v[j][1] = t.y; v[j][2] = t.z; v[j][3] = t.w;
+          }
+          for (int q = 0; q < u.top; ++q) {
+            const int r = u.pos[m * u.top + q];
+            if (r < 0) continue;
+            const float w = u.wts ? u.wts[m * u.top + q] : 1.f;
+            const float4 t = *(const float4*)(u.ye + (int64_t)r * u.ldye + 4 * i);
+            v[j][0] += w * t.x; v[j][1] += w * t.y; v[j][2] += w * t.z; v[j][3] += w * t.w;
+          }
           if (!EXACT)
 #pragma unroll
             for (int e = 0; e < 4; ++e)
               if (4 * i + e >= W) v[j][e] = 0.f;
         }
       }
-#pragma unroll
-      for (int e = 0; e < 4; ++e) ss += v[j][e] * v[j][e];
     }
-    if (u.g1) {
-      ss = block_sum(ss, sh);
-      const float inv = 1.f / sqrtf(ss / (float)W + u.eps);
-#pragma unroll
-      for (int j = 0; j < RU_VEC; ++j) {
-        const int i = threadIdx.x + j * blockDim.x;
-        if (j < nv && i < n4) gain<EXACT>(v[j], inv, u.g1, i, W);
-      }
-    }
+    if (u.g1) norm_row<RU_VEC, EXACT>(v, u.centred, u.eps, u.g1, u.b1, nv, n4, W, sh);
 #pragma unroll
     for (int j = 0; j < RU_VEC; ++j) {
       const int i = threadIdx.x + j * blockDim.x;
@@ -128,20 +164,7 @@ __global__ void k_row_update(RowUpdate u, int32_t* err) {
     }
   if (!u.out) return;
   const int64_t mo = u.dst ? u.dst[m] : m;
-  if (u.g2) {
-    float ss = 0.f;
-#pragma unroll
-    for (int j = 0; j < RU_VEC; ++j)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) ss += v[j][e] * v[j][e];
-    ss = block_sum(ss, sh);
-    const float inv = 1.f / sqrtf(ss / (float)W + u.eps);
-#pragma unroll
-    for (int j = 0; j < RU_VEC; ++j) {
-      const int i = threadIdx.x + j * blockDim.x;
-      if (j < nv && i < n4) gain<EXACT>(v[j], inv, u.g2, i, W);
-    }
-  }
+  if (u.g2) norm_row<RU_VEC, EXACT>(v, u.centred, u.eps, u.g2, u.b2, nv, n4, W, sh);
 #pragma unroll
   for (int j = 0; j < RU_VEC; ++j) {
     const int i = threadIdx.x + j * blockDim.x;
@@ -274,8 +297,8 @@ __global__ void k_stream_update(StreamUpdate u, int32_t* err) {
   }
 }
 
-__global__ void k_add_scalar(float* x, int64_t n, float v) {
-  for (int64_t i = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; i < n; i += (int64_t)gridDim.x * blockDim.x) x[i] += v;
+__global__ void k_affine(float* x, int64_t n, float f, float v) {
+  for (int64_t i = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; i < n; i += (int64_t)gridDim.x * blockDim.x) x[i] = x[i] * f + v;
 }
 
 __global__ void k_relu2_f32(float* x, int64_t n) {
@@ -296,13 +319,22 @@ __global__ void k_glu_f32(const float* gu, int64_t F, int act, float* out) {
   }
 }
 
-__global__ void k_pair_rope_tables(double base, int64_t T, int r, float* cos_t, float* sin_t) {
+__global__ void k_pair_rope_tables(PairRope f, int64_t T, int r, float* cos_t, float* sin_t) {
   const int half = r / 2;
   const int64_t n = T * half;
   for (int64_t i = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; i < n; i += (int64_t)gridDim.x * blockDim.x) {
     const int64_t p = i / half;
     const int k = (int)(i - p * half);
-    const double a = (double)p * pow(base, -2.0 * k / r);
+    double w = pow(f.base, -2.0 * k / r);
+    if (f.factor > 0) {
+      const double turns = f.original * w / 6.283185307179586;  // of this pair over the original context
+      if (turns < f.low) w /= f.factor;
+      else if (turns <= f.high) {
+        const double s = f.high > f.low ? (turns - f.low) / (f.high - f.low) : 1.0;
+        w = (1.0 - s) * w / f.factor + s * w;
+      }
+    }
+    const double a = (double)p * w;
     cos_t[i] = (float)cos(a);
     sin_t[i] = (float)sin(a);
   }
@@ -355,9 +387,9 @@ int k_launch_stream_update(cg_ctx* c, const StreamUpdate& u, int64_t M, int out_
   return CG_OK;
 }
 
-int k_launch_add_scalar(cg_ctx* c, float* x, int64_t n, float v) {
+int k_launch_affine(cg_ctx* c, float* x, int64_t n, float f, float v) {
   if (n == 0) return CG_OK;
-  k_add_scalar<<<grid_for(n, 256), 256, 0, c->core->stream>>>(x, n, v);
+  k_affine<<<grid_for(n, 256), 256, 0, c->core->stream>>>(x, n, f, v);
   CG_LAUNCHED(c);
   return CG_OK;
 }
@@ -376,8 +408,8 @@ int k_launch_glu_f32(cg_ctx* c, const float* gu, int64_t M, int64_t F, int act, 
   return CG_OK;
 }
 
-int k_launch_pair_rope_tables(cg_ctx* c, double base, int64_t T, int r, float* cos_t, float* sin_t) {
-  k_pair_rope_tables<<<grid_for(T * (r / 2), 256), 256, 0, c->core->stream>>>(base, T, r, cos_t, sin_t);
+int k_launch_pair_rope_tables(cg_ctx* c, const PairRope& f, int64_t T, int r, float* cos_t, float* sin_t) {
+  k_pair_rope_tables<<<grid_for(T * (r / 2), 256), 256, 0, c->core->stream>>>(f, T, r, cos_t, sin_t);
   CG_LAUNCHED(c);
   return CG_OK;
 }

@@ -9,24 +9,33 @@
 namespace cg {
 
 // One pass over the residual stream, row by row:
-//   src  = table[tokens[m]]            (tokens set)
-//        | y[m]                        (y set)
-//   x[m] = (add ? x[m] : 0) + (g1 ? rms(src) * g1 : src)
-//   out  = g2 ? rms(x) * g2 : x        (out set; f32 or bf16)
+//   src  = scale * table[tokens[m]]    (tokens set)
+//        | y[m] (y set) + sum over the token's experts i of wts[m top + i] ye[pos[m top + i]] (top > 0;
+//          wts null: ones)
+//   x[m] = (add ? x[m] : 0) + (g1 ? norm(src) * g1 + b1 : src)
+//   out  = g2 ? norm(x) * g2 + b2 : x  (out set; f32 or bf16)
 //   x0   = x                           (x0 set; a second copy in out's type)
-// With pick set, x is read only: out[dst[m]] = rms(x[pick[m]]) * g2.
+// norm divides by the root mean square, with centred after taking the mean off; biases may be null.
+// With pick set, x is read only: out[dst[m]] = norm(x[pick[m]]) * g2 + b2.
 struct RowUpdate {
   const uint32_t* tokens = nullptr;
   const void* table = nullptr;
   int table_bf16 = 0;
   int64_t vocab = 0;
+  float scale = 1.f;
   const float* y = nullptr;
   int64_t ldy = 0;
-  const float* g1 = nullptr;
+  const float* ye = nullptr;
+  int64_t ldye = 0;
+  const int32_t* pos = nullptr;
+  const float* wts = nullptr;
+  int top = 0;
+  int centred = 0;
+  const float *g1 = nullptr, *b1 = nullptr;
   int add = 0;
   float* x = nullptr;
   int64_t ldx = 0;
-  const float* g2 = nullptr;
+  const float *g2 = nullptr, *b2 = nullptr;
   void* out = nullptr;
   int64_t ldo = 0;
   void* x0 = nullptr;
@@ -75,16 +84,21 @@ struct StreamUpdate {
 };
 int k_launch_stream_update(cg_ctx* c, const StreamUpdate& u, int64_t M, int out_bf16);
 
-// x[i] += v
-int k_launch_add_scalar(cg_ctx* c, float* x, int64_t n, float v);
+// x[i] = x[i] * f + v
+int k_launch_affine(cg_ctx* c, float* x, int64_t n, float f, float v);
 // x[i] = max(x[i], 0)^2 in f32
 int k_launch_relu2_f32(cg_ctx* c, float* x, int64_t n);
 
 // out[m, i] = act(gu[m, i]) * gu[m, F + i] in f32
 int k_launch_glu_f32(cg_ctx* c, const float* gu, int64_t M, int64_t F, int act, float* out);
 
-// Rotary tables cos, sin [T, r / 2] of angles p * base^(-2 i / r), evaluated in double precision
-int k_launch_pair_rope_tables(cg_ctx* c, double base, int64_t T, int r, float* cos_t, float* sin_t);
+// Rotary tables cos, sin [T, r / 2] of angles p * f_i, f_i = base^(-2 i / r), evaluated in double precision.
+// factor > 0 stretches the slow pairs (Llama 3.1): with l = 2 pi / f, f stays where l < original / high,
+// becomes f / factor where l > original / low, and a blend of both in between.
+struct PairRope {
+  double base = 0, factor = 0, low = 0, high = 0, original = 0;
+};
+int k_launch_pair_rope_tables(cg_ctx* c, const PairRope& f, int64_t T, int r, float* cos_t, float* sin_t);
 
 // ------------------------------------------------------------- attention over a row batch ----
 // Grouped-query attention with per-layer sizes, window and sink on rows of unequal length.  Heads take
@@ -95,11 +109,15 @@ struct RowsAttnArgs {
   int64_t ldp;
   int H, G, d, dv, Dk, Dv;
   const float *q_gain, *k_gain;  // [H Dk], [G Dk]: norms over all query / key heads at once; null: none
+  int head_norm = 0;       // norms per head, without gains
   float eps, scale;
   int rot;                 // rotated components, neighbouring pairs
   const float *cos_t, *sin_t;    // [Tmax, rot / 2]
   int64_t window;          // 0 = none
+  int64_t keep_first = 0;  // with a window: these first positions stay visible
   const float* sink;       // [H] or null
+  float out_scale = 1.f;   // head h of token m is multiplied by out_scale and, with a gate, by
+  const float* gate = nullptr;  // sigmoid(gate[m * ldp + h])
   void* q;                 // [M, H Dk]
   void *k_cache, *v_cache; // [slots, G, Tmax, Dk | Dv]
   int64_t Tmax, slots;
@@ -146,23 +164,27 @@ size_t latent_decode_scratch(const LatentArgs& a, int64_t M);  // bytes
 int k_launch_latent_decode(cg_ctx* c, const LatentArgs& a, void* scratch);
 
 // --------------------------------------------------------- recurrences with a matrix state ----
-// Both mixers: [conv segment | gate segment | small segment] = W_in h.  The conv segment passes a
-// causal convolution per channel and silu and then holds, per token, queries and keys (KH heads of
-// dk) and values (H heads of dv); head h uses query/key head h / (H / KH).
-//   delta: S <- g S;  u = b (v - S^T k);  S <- S + k u^T;  o = S^T q        (S is dk x dv)
-//   ssd:   S <- g S + dt k v^T;  o = S^T q + D v
+// [conv segment | gate segment | small segment] = W_in h.  The conv segment passes a causal
+// convolution per channel (taps 0: none) and silu and then holds, per token, queries and keys (KH heads
+// of dk) and values (H heads of dv), the heads qs and vs columns apart; head h uses query/key head
+// h / (H / KH).
+//   delta:     S <- g S;  u = b (v - S^T k);  S <- S + k u^T;  o = S^T q        (S is dk x dv)
+//   ssd:       S <- g S + dt k v^T;  o = S^T q + D v
+//   lightning: S <- g S + k v^T;  o = S^T q, g a constant per head (log_decay set), no convolution
 // The convolution's last inputs are kept by position modulo taps, so that in a decode step blocks
 // may read old inputs while another block writes the new one.
 struct RecurBase {
   int delta;
   int H, KH, dk, dv, dvs;  // dvs: dv rounded up to a multiple of 8, the row length of S and o
+  int qs, vs;              // columns from one head to the next in the conv segment
   int C, taps;             // conv channels
   int q_off, k_off, v_off; // columns inside the conv segment
   const float* conv_w;     // [C, taps]
   const float* conv_b;     // [C] or null
   float* tail;             // [slots, taps, C]
   const float *a_log, *dt_bias;  // [H]
-  const float* dskip;      // [H], ssd
+  const float* log_decay = nullptr;  // [H], lightning
+  const float* dskip;      // [H], ssd; null: none
   float* S;                // [slots, H, dk, dvs] f32
   float *gl, *co;          // [M, H] log decay; beta (delta) or dt (ssd)
   float* o;                // [M, H * dvs]
@@ -186,9 +208,10 @@ struct ChunkArgs : RecurBase {
   const float* small;      // [M, ld_small]: delta beta and a, ssd dt
   int64_t ld_small;
   int DKp, dvp;            // dk rounded up to 16, dv rounded up to 8
-  __nv_bfloat16 *q, *k;    // [M, KH * DKp] conv outputs
+  __nv_bfloat16 *q, *k;    // [M, KH * DKp] conv outputs; lightning: the projections after silu
   __nv_bfloat16* v;        // [M, H * dvp]
-  float *rq, *rk;          // [M, KH] factors that make unit vectors of them
+  int64_t ldq, ldv;        // from one token to the next in q and k, and in v
+  float *rq, *rk;          // [M, KH] factors that make unit vectors of them (not lightning)
   __nv_bfloat16* T;        // [chunks, H, 2, 64, 64] scratch (delta)
   const int32_t *chunk_tok, *chunk_len;  // [n_chunks] first packed token, tokens
   const int32_t* row_chunk;              // [rows + 1]
@@ -197,16 +220,18 @@ struct ChunkArgs : RecurBase {
 bool chunk_supported(int dk);
 int k_launch_chunk_recurrence(cg_ctx* c, const ChunkArgs& a);
 
-// delta: per head, rms over dv, plain weight, times silu(gate).  ssd: times silu(gate) first, then
-// rms over each of norm_groups equal parts.
+// Over each of `groups` equal parts of the H * dv values: rms, gain and times act(gate), the gate before
+// the rms with gate_first, else after the gain.  delta: a group per head and the same gains for
+// all of them; ssd: the gate first; lightning: one group and a sigmoid.
 struct GatedNorm {
-  int delta;
-  int H, dv, dvs, norm_groups;
+  int H, dv, dvs, groups;
+  int shared_gain;         // norm holds one group's gains
+  int gate_first, sigmoid; // act is silu, or the sigmoid
   const float* o;          // [M, H * dvs]
   const void* gate;        // [M, ldg], H * dv columns
   int64_t ldg;
   int gate_bf16;
-  const float* norm;       // delta: [dv]; ssd: [H * dv]
+  const float* norm;       // [H * dv], shared_gain: [H * dv / groups]
   float eps;
   void* att;               // [M, ld_att]
   int64_t ld_att;

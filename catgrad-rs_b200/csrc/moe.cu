@@ -186,12 +186,12 @@ __global__ void k_moe_norm_split(float* x, const float* gamma, float eps, int pl
   }
 }
 
-// One warp per token: softmax over the router logits, top-k (ties -> lower expert id),
-// optional renormalisation.  With `correction` [E] the experts are chosen by probability + correction
-// and weighted by probability * scale.  Dynamic shared memory: E floats per warp, 2 E with correction.
+// One warp per token: softmax over the router logits (or the sigmoid of each), top-k (ties -> lower expert
+// id), optional renormalisation, times scale.  With `correction` [E] the experts are chosen by probability + correction
+// and weighted by probability.  Dynamic shared memory: E floats per warp, 2 E with correction.
 constexpr uint32_t TAKEN = 0xFFFFFFFFu;  // a chosen expert's mark (a NaN no sum here produces)
-__global__ void k_moe_topk(const float* logits, int64_t M, int E, int k, int norm_topk, const float* correction, float scale,
-                           uint32_t* ids, float* wts) {
+__global__ void k_moe_topk(const float* logits, int64_t M, int E, int k, int norm_topk, int sigmoid, const float* correction,
+                           float scale, uint32_t* ids, float* wts) {
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
   asm volatile("griddepcontrol.wait;" ::: "memory");
   extern __shared__ float sm[];
@@ -210,14 +210,14 @@ __global__ void k_moe_topk(const float* logits, int64_t M, int E, int k, int nor
   for (int o = 16; o; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
   float sum = 0.f;
   for (int e = lane; e < E; e += 32) {
-    const float v = expf(pr[e] - mx);
+    const float v = sigmoid ? 1.f / (1.f + expf(-pr[e])) : expf(pr[e] - mx);
     pr[e] = v;
     sum += v;
   }
   for (int o = 16; o; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
   __syncwarp();
   for (int e = lane; e < E; e += 32) {
-    pr[e] = pr[e] / sum;
+    if (!sigmoid) pr[e] = pr[e] / sum;
     if (correction) ch[e] = pr[e] + correction[e];
   }
   __syncwarp();
@@ -246,8 +246,7 @@ __global__ void k_moe_topk(const float* logits, int64_t M, int E, int k, int nor
   total = sum_in_reference_order(chosen, k);  // bit-identical to the reference's sum over the k values
   if (lane < k) {
     ids[m * k + lane] = chosen_id;
-    const float w = norm_topk ? chosen / total : chosen;
-    wts[m * k + lane] = correction ? w * scale : w;
+    wts[m * k + lane] = (norm_topk ? chosen / total : chosen) * scale;
   }
 }
 
@@ -324,6 +323,27 @@ __global__ void k_moe_gather(const __nv_bfloat16* xn, const int32_t* pos, int64_
     const int r = pos[p];
     if (r < 0) continue;
     ((uint4*)(xg + (int64_t)r * H))[j] = ((const uint4*)(xn + (p / k) * H))[j];
+  }
+}
+
+// The same where the weights multiply the experts' inputs: xg[pos[p], :] = bf16(wts[p] * x[p / k, :]) from
+// f32 rows.
+__global__ void k_moe_gather_weighted(const float* x, const float* wts, const int32_t* pos, int64_t P, int k, int H, __nv_bfloat16* xg) {
+  asm volatile("griddepcontrol.wait;" ::: "memory");
+  asm volatile("griddepcontrol.launch_dependents;" ::: "memory");  // after the wait, as in k_moe_gather
+  const int per = H / 8;
+  const int64_t total = P * per;
+  for (int64_t i = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; i < total; i += (int64_t)gridDim.x * blockDim.x) {
+    const int64_t p = i / per;
+    const int j = (int)(i - p * per);
+    const int r = pos[p];
+    if (r < 0) continue;
+    const float w = wts[p];
+    const float4* s = (const float4*)(x + (p / k) * H) + 2 * j;
+    const float4 a = s[0], b = s[1];
+    const __nv_bfloat162 v[4] = {__floats2bfloat162_rn(w * a.x, w * a.y), __floats2bfloat162_rn(w * a.z, w * a.w),
+                                 __floats2bfloat162_rn(w * b.x, w * b.y), __floats2bfloat162_rn(w * b.z, w * b.w)};
+    ((uint4*)(xg + (int64_t)r * H))[j] = make_uint4(*(const uint32_t*)&v[0], *(const uint32_t*)&v[1], *(const uint32_t*)&v[2], *(const uint32_t*)&v[3]);
   }
 }
 
@@ -541,18 +561,22 @@ k_moe_gemm(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CU
 // ------------------------------------------------------------- f32 form (CUDA cores) ----
 constexpr int MF_ROWS = 32, MF_COLS = 64, MF_K = 32;
 
-// src[pos[p]] = p / k
-__global__ void k_moe_sources(const int32_t* pos, int64_t P, int k, int32_t* src) {
+// src[pos[p]] = p / k and, with wts, in_w[pos[p]] = wts[p]
+__global__ void k_moe_sources(const int32_t* pos, int64_t P, int k, const float* wts, int32_t* src, float* in_w) {
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
   asm volatile("griddepcontrol.wait;" ::: "memory");
   for (int64_t p = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; p < P; p += (int64_t)gridDim.x * blockDim.x)
-    if (pos[p] >= 0) src[pos[p]] = (int32_t)(p / k);
+    if (pos[p] >= 0) {
+      src[pos[p]] = (int32_t)(p / k);
+      if (wts) in_w[pos[p]] = wts[p];
+    }
 }
 
 struct MoeF32Args {
   const int32_t *tile_expert, *tile_row0, *tile_rows, *n_tiles;
   const float* x;         // [.., K]
   const int32_t* src;     // row of x each grouped row reads; null: the row itself
+  const float* in_w;      // factor on it; null: 1
   const float *w, *w_up;  // [experts, N, K]; w_up null: a plain product
   float* out;             // [grouped rows, N]
   int N, K, act;
@@ -573,7 +597,9 @@ __global__ void __launch_bounds__(256) k_moe_gemm_f32(MoeF32Args p) {
     const int k = k0 + tc;
     for (int r = tr; r < MF_ROWS; r += 8) {
       const int64_t row = row0 + r;
-      xs[tc][r] = r < rows && k < p.K ? p.x[(p.src ? (int64_t)p.src[row] : row) * p.K + k] : 0.f;
+      float x = r < rows && k < p.K ? p.x[(p.src ? (int64_t)p.src[row] : row) * p.K + k] : 0.f;
+      if (p.in_w && r < rows) x *= p.in_w[row];
+      xs[tc][r] = x;
     }
     for (int r = tr; r < MF_COLS; r += 8) {
       const bool in = n0 + r < p.N && k < p.K;
@@ -673,7 +699,7 @@ static int launch_topk(cg_ctx* c, const MoeArgs& a) {
   const int warps = 4;
   const size_t smem = (size_t)warps * a.E * (a.correction ? 8 : 4);
   CG_CUDA(c, launch_kernel(c, k_moe_topk, dim3((unsigned)((a.M + warps - 1) / warps)), dim3(32 * warps), smem, 1,
-                           (const float*)a.logits, a.M, a.E, a.k, a.norm_topk, a.correction, a.router_scale, a.w.ids, a.w.wts));
+                           (const float*)a.logits, a.M, a.E, a.k, a.norm_topk, a.sigmoid, a.correction, a.router_scale, a.w.ids, a.w.wts));
   CG_LAUNCHED(c);
   return CG_OK;
 }
@@ -732,8 +758,12 @@ int moe_experts(cg_ctx* c, const MoeArgs& a) {
   const int64_t max_tiles = moe_max_tiles(P, a.El, tn);
   if (max_tiles > 65535) return fail(c, CG_ERR_UNSUPPORTED, "moe: too many tiles");
   CG_TRY(launch_plan(c, a, tn));
-  CG_CUDA(c, launch_kernel(c, k_moe_gather, dim3(grid_for(P * (a.H / 8), 256)), dim3(256), 0, 1, (const __nv_bfloat16*)a.xn,
-                           (const int32_t*)a.w.pos, P, a.k, a.H, a.w.xg));
+  if (a.weigh_input)
+    CG_CUDA(c, launch_kernel(c, k_moe_gather_weighted, dim3(grid_for(P * (a.H / 8), 256)), dim3(256), 0, 1, a.x, (const float*)a.w.wts,
+                             (const int32_t*)a.w.pos, P, a.k, a.H, a.w.xg));
+  else
+    CG_CUDA(c, launch_kernel(c, k_moe_gather, dim3(grid_for(P * (a.H / 8), 256)), dim3(256), 0, 1, (const __nv_bfloat16*)a.xn,
+                             (const int32_t*)a.w.pos, P, a.k, a.H, a.w.xg));
   CG_LAUNCHED(c);
 
   MoeGemmArgs g;
@@ -785,15 +815,17 @@ int moe_experts_f32(cg_ctx* c, const MoeArgs& a, const float* x, const float* w_
   const int64_t P = a.M * a.k, tiles = moe_max_tiles(P, a.El, MF_ROWS);
   if (tiles > 65535) return fail(c, CG_ERR_UNSUPPORTED, "moe: too many tiles");
   // rows in grouped order: which token each reads
-  CG_CUDA(c, launch_kernel(c, k_moe_sources, dim3(grid_for(P, 256)), dim3(256), 0, 1, (const int32_t*)a.w.pos, P, a.k, (int32_t*)a.w.xg));
+  float* in_w = (float*)a.w.xg + P;
+  CG_CUDA(c, launch_kernel(c, k_moe_sources, dim3(grid_for(P, 256)), dim3(256), 0, 1, (const int32_t*)a.w.pos, P, a.k,
+                           a.weigh_input ? (const float*)a.w.wts : (const float*)nullptr, (int32_t*)a.w.xg, in_w));
   CG_LAUNCHED(c);
   MoeF32Args g;
   g.tile_expert = a.w.tile_expert; g.tile_row0 = a.w.tile_row0; g.tile_rows = a.w.tile_rows; g.n_tiles = a.w.n_tiles;
-  g.x = x; g.src = (const int32_t*)a.w.xg; g.w = w_gate; g.w_up = w_up; g.out = h;
+  g.x = x; g.src = (const int32_t*)a.w.xg; g.in_w = a.weigh_input ? in_w : nullptr; g.w = w_gate; g.w_up = w_up; g.out = h;
   g.N = a.Fe; g.K = a.H; g.act = a.act; g.limit = a.act_limit;
   CG_CUDA(c, launch_kernel(c, k_moe_gemm_f32, dim3((unsigned)((g.N + MF_COLS - 1) / MF_COLS), (unsigned)tiles), dim3(256), 0, 1, g));
   CG_LAUNCHED(c);
-  g.x = h; g.src = nullptr; g.w = w_down; g.w_up = nullptr; g.out = a.w.y;
+  g.x = h; g.src = nullptr; g.in_w = nullptr; g.w = w_down; g.w_up = nullptr; g.out = a.w.y;
   g.N = a.H; g.K = a.Fe;
   CG_CUDA(c, launch_kernel(c, k_moe_gemm_f32, dim3((unsigned)((g.N + MF_COLS - 1) / MF_COLS), (unsigned)tiles), dim3(256), 0, 1, g));
   CG_LAUNCHED(c);

@@ -1,5 +1,5 @@
 // recurrent.cu — layers whose memory is a matrix per head: the gated delta rule and the Mamba-2
-// state space, both behind short causal convolutions.  State, decays, step sizes, unit norms and
+// state space, both behind short causal convolutions, and lightning attention.  State, decays, step sizes, unit norms and
 // gates are f32.
 #include <algorithm>
 
@@ -32,6 +32,7 @@ __device__ __forceinline__ void st(__nv_bfloat16* p, float v) { *p = __float2bfl
 // The convolution at channel c of token m: the row's place i, its first position p0.
 __device__ __forceinline__ float conv_at(const RecurArgs& a, int64_t m, int i, int64_t p0, int c, const float* tail) {
   float v = a.conv_b ? a.conv_b[c] : 0.f;
+  if (a.taps == 0) v = a.proj[m * a.ldp + c];
   for (int j = 0; j < a.taps; ++j) {
     float x = 0.f;
     if (j <= i) x = a.proj[(m - j) * a.ldp + c];
@@ -75,6 +76,11 @@ __global__ void __launch_bounds__(256) k_conv_heads(RecurArgs a) {
   }
   const float* sp = a.proj + m * a.ldp + a.small_off;
   for (int h = threadIdx.x; h < a.H; h += blockDim.x) {
+    if (a.log_decay) {
+      a.gl[m * a.H + h] = a.log_decay[h];
+      a.co[m * a.H + h] = 1.f;
+      continue;
+    }
     const float dt = softplus(sp[a.delta ? a.H + h : h] + a.dt_bias[h]);
     a.gl[m * a.H + h] = -expf(a.a_log[h]) * dt;
     a.co[m * a.H + h] = a.delta ? 1.f / (1.f + expf(-sp[h])) : dt;
@@ -119,10 +125,10 @@ __global__ void __launch_bounds__(128) k_recur_steps(RecurArgs a) {
     const float* cv = a.cv + m * a.ldc;
     __syncthreads();
     for (int i = tid; i < a.dk; i += 128) {
-      ks[i] = cv[a.k_off + kh * a.dk + i];
-      qs[i] = cv[a.q_off + kh * a.dk + i];
+      ks[i] = cv[a.k_off + kh * a.qs + i];
+      qs[i] = cv[a.q_off + kh * a.qs + i];
     }
-    const float v = live ? cv[a.v_off + h * a.dv + e] : 0.f;
+    const float v = live ? cv[a.v_off + h * a.vs + e] : 0.f;
     const float g = expf(a.gl[m * a.H + h]), co = a.co[m * a.H + h];
     __syncthreads();
     float u = co * v;
@@ -186,19 +192,27 @@ __global__ void __launch_bounds__(256, RD_ROWS <= 8 ? 3 : 2) k_recur_decode(Recu
     const int seg = x < a.dk ? 0 : x < 2 * a.dk ? 1 : 2;
     const int e = seg == 0 ? x : seg == 1 ? x - a.dk : x - 2 * a.dk;
     if (seg == 2 && e >= a.dv) { sv[e] = 0.f; continue; }
-    const int c = seg == 0 ? a.q_off + kh * a.dk + e : seg == 1 ? a.k_off + kh * a.dk + e : a.v_off + h * a.dv + e;
+    const int c = seg == 0 ? a.q_off + kh * a.qs + e : seg == 1 ? a.k_off + kh * a.qs + e : a.v_off + h * a.vs + e;
     const float now = p[c];
-    float v = (a.conv_b ? a.conv_b[c] : 0.f) + a.conv_w[(int64_t)c * a.taps + a.taps - 1] * now;
-    for (int j = 1; j < a.taps; ++j)
-      if (pos - j >= 0) v += a.conv_w[(int64_t)c * a.taps + a.taps - 1 - j] * tail[(int64_t)((pos - j) % a.taps) * a.C + c];
-    if (seg == 2 || h % rep == 0) tail[(int64_t)(pos % a.taps) * a.C + c] = now;  // read by no block of this step
+    float v = now;
+    if (a.taps) {
+      v = (a.conv_b ? a.conv_b[c] : 0.f) + a.conv_w[(int64_t)c * a.taps + a.taps - 1] * now;
+      for (int j = 1; j < a.taps; ++j)
+        if (pos - j >= 0) v += a.conv_w[(int64_t)c * a.taps + a.taps - 1 - j] * tail[(int64_t)((pos - j) % a.taps) * a.C + c];
+      if (seg == 2 || h % rep == 0) tail[(int64_t)(pos % a.taps) * a.C + c] = now;  // read by no block of this step
+    }
     (seg == 0 ? sq : seg == 1 ? sk : sv)[e] = silu(v);
   }
   const float* sp = p + a.small_off;
   if (tid == 64) {
-    const float dt = softplus(sp[a.delta ? a.H + h : h] + a.dt_bias[h]);
-    sg[0] = expf(-expf(a.a_log[h]) * dt);
-    sg[1] = a.delta ? 1.f / (1.f + expf(-sp[h])) : dt;
+    if (a.log_decay) {
+      sg[0] = expf(a.log_decay[h]);
+      sg[1] = 1.f;
+    } else {
+      const float dt = softplus(sp[a.delta ? a.H + h : h] + a.dt_bias[h]);
+      sg[0] = expf(-expf(a.a_log[h]) * dt);
+      sg[1] = a.delta ? 1.f / (1.f + expf(-sp[h])) : dt;
+    }
   }
   __syncthreads();
   if (a.delta) {
@@ -260,7 +274,7 @@ __global__ void __launch_bounds__(256, RD_ROWS <= 8 ? 3 : 2) k_recur_decode(Recu
   o = sum_rows(o);
   if (!a.delta) {
     if (rg == 0) {
-      const float d = a.dskip[h];
+      const float d = a.dskip ? a.dskip[h] : 0.f;
       *(float4*)(a.o + m * (int64_t)a.H * a.dvs + (int64_t)h * a.dvs + 4 * cg) =
           make_float4(o.x + d * v4.x, o.y + d * v4.y, o.z + d * v4.z, o.w + d * v4.w);
     }
@@ -294,6 +308,8 @@ __device__ __forceinline__ void st4(__nv_bfloat16* p, float4 v) {
   *(uint2*)p = make_uint2(*(const uint32_t*)&lo, *(const uint32_t*)&hi);
 }
 
+__device__ __forceinline__ float gate_act(const GatedNorm& a, float x) { return a.sigmoid ? 1.f / (1.f + expf(-x)) : silu(x); }
+
 // One block per (norm group, token), any sizes.
 template <class TG, class T>
 __global__ void k_gated_norm(GatedNorm a) {
@@ -301,7 +317,7 @@ __global__ void k_gated_norm(GatedNorm a) {
   asm volatile("griddepcontrol.wait;" ::: "memory");
   __shared__ float sh[32];
   const int64_t m = blockIdx.y;
-  const int n = a.delta ? a.dv : a.H * a.dv / a.norm_groups;
+  const int n = a.H * a.dv / a.groups;
   const int c0 = blockIdx.x * n;
   const float* o = a.o + m * (int64_t)a.H * a.dvs;
   const TG* gate = (const TG*)a.gate + m * a.ldg + c0;
@@ -309,14 +325,13 @@ __global__ void k_gated_norm(GatedNorm a) {
   auto at = [&](int i) { const int c = c0 + i, h = c / a.dv; return o[h * a.dvs + (c - h * a.dv)]; };
   float ss = 0.f;
   for (int i = threadIdx.x; i < n; i += blockDim.x) {
-    const float v = a.delta ? at(i) : at(i) * silu(ldg1(gate + i));
+    const float v = a.gate_first ? at(i) * gate_act(a, ldg1(gate + i)) : at(i);
     ss += v * v;
   }
   ss = block_sum(ss, sh);
   const float rms = sqrtf(ss / (float)n + a.eps);
   for (int i = threadIdx.x; i < n; i += blockDim.x) {
-    const float g = silu(ldg1(gate + i));
-    st(out + i, a.delta ? at(i) / rms * a.norm[i] * g : at(i) * g / rms * a.norm[c0 + i]);
+    st(out + i, at(i) * gate_act(a, ldg1(gate + i)) / rms * a.norm[a.shared_gain ? i : c0 + i]);
   }
 }
 
@@ -347,9 +362,13 @@ __global__ void k_gated_norm_vec(GatedNorm a, int n, int units, int threads) {
   }
 #pragma unroll
   for (int j = 0; j < V; ++j) {
-    g[j] = sizeof(TG) == 2 ? make_float4(silu_fast(g[j].x), silu_fast(g[j].y), silu_fast(g[j].z), silu_fast(g[j].w))
-                           : make_float4(silu(g[j].x), silu(g[j].y), silu(g[j].z), silu(g[j].w));
-    if (!a.delta) { x[j].x *= g[j].x; x[j].y *= g[j].y; x[j].z *= g[j].z; x[j].w *= g[j].w; }
+    if (a.sigmoid)
+      g[j] = sizeof(TG) == 2 ? make_float4(sigmoid_fast(g[j].x), sigmoid_fast(g[j].y), sigmoid_fast(g[j].z), sigmoid_fast(g[j].w))
+                             : make_float4(gate_act(a, g[j].x), gate_act(a, g[j].y), gate_act(a, g[j].z), gate_act(a, g[j].w));
+    else
+      g[j] = sizeof(TG) == 2 ? make_float4(silu_fast(g[j].x), silu_fast(g[j].y), silu_fast(g[j].z), silu_fast(g[j].w))
+                             : make_float4(silu(g[j].x), silu(g[j].y), silu(g[j].z), silu(g[j].w));
+    if (a.gate_first) { x[j].x *= g[j].x; x[j].y *= g[j].y; x[j].z *= g[j].z; x[j].w *= g[j].w; }
     ss += x[j].x * x[j].x + x[j].y * x[j].y + x[j].z * x[j].z + x[j].w * x[j].w;
   }
   ss = threads == 32 ? warp_sum(ss) : block_sum(ss, sh);
@@ -358,16 +377,16 @@ __global__ void k_gated_norm_vec(GatedNorm a, int n, int units, int threads) {
   for (int j = 0; j < V; ++j) {
     const int i = 4 * (t + j * threads);
     if (!live || i >= n) continue;
-    const float4 w = *(const float4*)(a.norm + (a.delta ? 0 : c0) + i);
+    const float4 w = *(const float4*)(a.norm + (a.shared_gain ? 0 : c0) + i);
     float4 r = make_float4(x[j].x * inv * w.x, x[j].y * inv * w.y, x[j].z * inv * w.z, x[j].w * inv * w.w);
-    if (a.delta) { r.x *= g[j].x; r.y *= g[j].y; r.z *= g[j].z; r.w *= g[j].w; }
+    if (!a.gate_first) { r.x *= g[j].x; r.y *= g[j].y; r.z *= g[j].z; r.w *= g[j].w; }
     st4(out + i, r);
   }
 }
 
 template <class TG, class T>
 int launch_gated_norm(cg_ctx* c, const GatedNorm& a) {
-  const int units = a.delta ? a.H : a.norm_groups;
+  const int units = a.groups;
   const int n = a.H * a.dv / units;
   const bool vec = a.dv == a.dvs && n % 4 == 0 && a.ldg % 4 == 0 && a.ld_att % 4 == 0 && (((uintptr_t)a.gate | (uintptr_t)a.norm) & 15) == 0 && n <= 16384;
   if (vec && n <= 512) {

@@ -4,7 +4,7 @@
 // With G_t the running sum of the log decays inside a chunk, S0 the state before it and u_t what
 // token t writes, both recurrences read
 //   S_t = e^{G_t} S0 + sum_{s<=t} e^{G_t - G_s} k_s u_s^T,      o_t = S_t^T q_t
-// For the state space u_t = dt_t v_t.  For the delta rule u solves a unit lower triangular system:
+// For the state space u_t = dt_t v_t, for lightning attention u_t = v_t and the decays are constants.  For the delta rule u solves a unit lower triangular system:
 //   (I + A) U = R,  A_ts = b_t e^{G_t - G_s} (k_t . k_s) (s < t),  R_t = b_t (v_t - e^{G_t} S0^T k_t)
 // T = (I + A)^-1 depends on keys and gates only, so k_delta_solve makes it for all chunks at once;
 // k_delta_scan / k_ssd_scan then walk the chunks of one (row, head, 64 value columns) with S in registers.
@@ -321,6 +321,11 @@ __device__ __forceinline__ void load_gates(const ChunkArgs& a, int chunk, int h,
   for (int b = 0; b < 2; ++b) {
     const int t = 2 * lane + b;
     const bool in = t < len;
+    if (a.log_decay) {
+      l[b] = in ? a.log_decay[h] * 1.4426950408889634f : 0.f;
+      co[b] = rq[b] = rk[b] = in ? 1.f : 0.f;
+      continue;
+    }
     l[b] = in ? a.gl[(m0 + t) * a.H + h] * 1.4426950408889634f : 0.f;
     co[b] = in ? a.co[(m0 + t) * a.H + h] : 0.f;
     rq[b] = in ? a.rq[(m0 + t) * a.KH + kh] : 0.f;
@@ -496,7 +501,7 @@ __global__ void __launch_bounds__(256, 2) k_delta_scan(ChunkArgs a) {
     for (int i = tid; i < CT * (DK / 8); i += 256) {
       const int r = i / (DK / 8), c = i - r * (DK / 8);
       const bool in = r < len && c < ch;
-      const int64_t o = (m0 + (in ? r : 0)) * (int64_t)a.KH * a.DKp + (int64_t)kh * a.DKp + (in ? c * 8 : 0);
+      const int64_t o = (m0 + (in ? r : 0)) * a.ldq + (int64_t)kh * a.DKp + (in ? c * 8 : 0);
       const uint32_t d = (uint32_t)(r * LK + c * 8) * 2u;
       cp_async16(b + L::Q + d, a.q + o, in ? 16 : 0);
       cp_async16(b + L::K + d, a.k + o, in ? 16 : 0);
@@ -505,7 +510,7 @@ __global__ void __launch_bounds__(256, 2) k_delta_scan(ChunkArgs a) {
       const int r = i / (EB / 8), c = i - r * (EB / 8);
       const bool in = r < len && c * 8 < vw;
       cp_async16(b + L::V + (uint32_t)(r * LE + c * 8) * 2u,
-                 a.v + (m0 + (in ? r : 0)) * (int64_t)a.H * a.dvp + (int64_t)h * a.dvp + (in ? e0 + c * 8 : 0), in ? 16 : 0);
+                 a.v + (m0 + (in ? r : 0)) * a.ldv + (int64_t)h * a.dvp + (in ? e0 + c * 8 : 0), in ? 16 : 0);
     }
     {
       const __nv_bfloat16* t = a.T + ((int64_t)chunk * a.H + h) * 2 * CT * CT;
@@ -760,7 +765,7 @@ __global__ void __launch_bounds__(256, 2) k_ssd_scan(ChunkArgs a) {
     for (int i = tid; i < CT * (DK / 8); i += 256) {
       const int r = i / (DK / 8), c = i - r * (DK / 8);
       const bool in = r < len && c < ch;
-      const int64_t o = (m0 + (in ? r : 0)) * (int64_t)a.KH * a.DKp + (int64_t)kh * a.DKp + (in ? c * 8 : 0);
+      const int64_t o = (m0 + (in ? r : 0)) * a.ldq + (int64_t)kh * a.DKp + (in ? c * 8 : 0);
       const uint32_t d = (uint32_t)(r * LK + c * 8) * 2u;
       cp_async16(base + L::Q + d, a.q + o, in ? 16 : 0);
       cp_async16(base + L::K + d, a.k + o, in ? 16 : 0);
@@ -769,7 +774,7 @@ __global__ void __launch_bounds__(256, 2) k_ssd_scan(ChunkArgs a) {
       const int r = i / (EB / 8), c = i - r * (EB / 8);
       const bool in = r < len && c * 8 < vw;
       cp_async16(base + L::V + (uint32_t)(r * LE + c * 8) * 2u,
-                 a.v + (m0 + (in ? r : 0)) * (int64_t)a.H * a.dvp + (int64_t)h * a.dvp + (in ? e0 + c * 8 : 0), in ? 16 : 0);
+                 a.v + (m0 + (in ? r : 0)) * a.ldv + (int64_t)h * a.dvp + (in ? e0 + c * 8 : 0), in ? 16 : 0);
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
@@ -802,7 +807,7 @@ __global__ void __launch_bounds__(256, 2) k_ssd_scan(ChunkArgs a) {
       }
   };
   publish_state();
-  const float dsk = a.dskip[h];
+  const float dsk = a.dskip ? a.dskip[h] : 0.f;
   const int t0 = wm * 16 + r_in;                      // this thread's tokens: t0 and t0 + 8
 
   for (int c = c0; c < c1; ++c) {
@@ -960,6 +965,7 @@ bool chunk_supported(int dk) { return dk <= 128; }
 
 int k_launch_chunk_recurrence(cg_ctx* c, const ChunkArgs& a) {
   if (a.rows.M == 0) return CG_OK;
+  if (a.log_decay) return a.dk <= 64 ? launch_scan<64, false>(c, a) : launch_scan<128, false>(c, a);
   const int lanes = a.dk / CV;
   const bool fast = a.dk % 8 == 0 && a.dv % 8 == 0 && a.DKp == a.dk && (!a.delta || (lanes & (lanes - 1)) == 0) && a.taps >= 1 && a.taps <= 4;
   if (fast) {

@@ -1,6 +1,6 @@
 // rows_attn.cu — grouped-query attention on rows of unequal length: norms over all heads of the
-// queries and of the keys, rotation of neighbouring pairs and the cache append in one pass, and the
-// attention of sizes (and of the f32 form) that the tensor-core kernels do not have.  Prompts in bf16
+// queries and of the keys or per head, rotation of neighbouring pairs and the cache append in one pass,
+// and the attention of sizes (and of the f32 form) that the tensor-core kernels do not have.  Prompts in bf16
 // take attention_fa.cu / attention.cu, decode steps attn_decode.cu.
 #include <algorithm>
 
@@ -54,6 +54,7 @@ __global__ void __launch_bounds__(256) k_rows_qkv(RowsAttnArgs a) {
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
   asm volatile("griddepcontrol.wait;" ::: "memory");
   __shared__ float sh[32];
+  extern __shared__ float per_head[];  // [H + G] with head_norm
   const int64_t m = blockIdx.x;
   const int row = a.rows.tok_row[m];
   const int64_t pos = row_pos0(a.rows, row) + (m - a.rows.start[row]);
@@ -72,6 +73,19 @@ __global__ void __launch_bounds__(256) k_rows_qkv(RowsAttnArgs a) {
     fq = 1.f / sqrtf(block_sum(sq, sh) / (float)(a.H * a.d) + a.eps);
     fk = 1.f / sqrtf(block_sum(sk, sh) / (float)(a.G * a.d) + a.eps);
   }
+  if (a.head_norm) {
+    const int lane = threadIdx.x & 31;
+    for (int h = threadIdx.x >> 5; h < a.H + a.G; h += blockDim.x >> 5) {
+      float ss = 0.f;
+      for (int i = 4 * lane; i < a.Dk; i += 128) {
+        const float4 v = *(const float4*)(p + h * a.Dk + i);
+        ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+      }
+      ss = warp_sum(ss);
+      if (lane == 0) per_head[h] = 1.f / sqrtf(ss / (float)a.d + a.eps);
+    }
+    __syncthreads();
+  }
   const int half = a.rot / 2;
   const float* ct = a.cos_t + pos * half;
   const float* sn = a.sin_t + pos * half;
@@ -88,6 +102,9 @@ __global__ void __launch_bounds__(256) k_rows_qkv(RowsAttnArgs a) {
       const float f = is_q ? fq : fk;
       const float4 w = *(const float4*)((is_q ? a.q_gain : a.k_gain) + j);
       v = make_float4(v.x * (f * w.x), v.y * (f * w.y), v.z * (f * w.z), v.w * (f * w.w));
+    } else if (a.head_norm) {
+      const float f = per_head[is_q ? h : a.H + h];
+      v = make_float4(v.x * f, v.y * f, v.z * f, v.w * f);
     }
     const int k = e >> 1;
     if (k < half) v = make_float4(v.x * ct[k] - v.y * sn[k], v.y * ct[k] + v.x * sn[k], v.z, v.w);
@@ -119,14 +136,17 @@ __global__ void __launch_bounds__(128) k_rows_attn(RowsAttnArgs a) {
   const int64_t base = ((int64_t)a.rows.slot[row] * a.G + g) * a.Tmax;
   const T* kb = (const T*)a.k_cache + base * a.Dk;
   const T* vb = (const T*)a.v_cache + base * a.Dv;
-  const int64_t lo = a.window > 0 ? max((int64_t)0, pos - a.window + 1) : 0;
+  // the visible keys in sequence: the kf kept first ones, then [lo, pos]
+  const int64_t lo = a.window > 0 ? max((int64_t)0, pos - a.window + 1) : 0, kf = min(a.keep_first, lo), end = kf + pos + 1 - lo;
+  auto key = [&](int64_t v) { return v < kf ? v : v - kf + lo; };
   // the sink is a term of the sum before any key
   float mx = a.sink ? a.sink[h] : -INFINITY, l = a.sink ? 1.f : 0.f;
-  for (int64_t k0 = lo; k0 <= pos; k0 += KT) {
-    const int n = (int)min((int64_t)KT, pos + 1 - k0);
+  for (int64_t k0 = 0; k0 < end; k0 += KT) {
+    const int n = (int)min((int64_t)KT, end - k0);
     for (int j = warp; j < n; j += nw) {
       float v = 0.f;
-      for (int i = lane; i < a.d; i += 32) v += q[i] * ld(kb + (k0 + j) * a.Dk + i);
+      const T* kr = kb + key(k0 + j) * a.Dk;
+      for (int i = lane; i < a.d; i += 32) v += q[i] * ld(kr + i);
       v = warp_sum(v);
       if (lane == 0) s[j] = v * a.scale;
     }
@@ -145,13 +165,15 @@ __global__ void __launch_bounds__(128) k_rows_attn(RowsAttnArgs a) {
     mx = mn;
     for (int i = tid; i < a.dv; i += blockDim.x) {
       float v = o[i] * corr;
-      for (int j = 0; j < n; ++j) v += s[j] * ld(vb + (k0 + j) * a.Dv + i);
+      for (int j = 0; j < n; ++j) v += s[j] * ld(vb + key(k0 + j) * a.Dv + i);
       o[i] = v;
     }
     __syncthreads();
   }
   T* out = (T*)a.att + m * a.ld_att + (int64_t)h * a.Dv;
-  for (int i = tid; i < a.Dv; i += blockDim.x) st(out + i, o[i] / l);
+  float f = a.out_scale;
+  if (a.gate) f *= 1.f / (1.f + expf(-a.gate[m * a.ldp + h]));
+  for (int i = tid; i < a.Dv; i += blockDim.x) st(out + i, o[i] / l * f);
 }
 
 }  // namespace
@@ -159,8 +181,10 @@ __global__ void __launch_bounds__(128) k_rows_attn(RowsAttnArgs a) {
 int k_launch_rows_qkv(cg_ctx* c, const RowsAttnArgs& a) {
   if (a.rows.M == 0) return CG_OK;
   if (a.Dk % 8 || a.Dv % 8 || a.ldp % 4) return fail(c, CG_ERR_INVALID, "attention: head sizes must be padded to multiples of 8");
-  if (a.bf16) CG_CUDA(c, launch_kernel(c, k_rows_qkv<__nv_bfloat16>, dim3((unsigned)a.rows.M), dim3(256), 0, 1, a));
-  else CG_CUDA(c, launch_kernel(c, k_rows_qkv<float>, dim3((unsigned)a.rows.M), dim3(256), 0, 1, a));
+  const size_t smem = a.head_norm ? (size_t)(a.H + a.G) * 4 : 0;
+  if (smem > 40 * 1024) return fail(c, CG_ERR_UNSUPPORTED, "attention: too many heads");
+  if (a.bf16) CG_CUDA(c, launch_kernel(c, k_rows_qkv<__nv_bfloat16>, dim3((unsigned)a.rows.M), dim3(256), smem, 1, a));
+  else CG_CUDA(c, launch_kernel(c, k_rows_qkv<float>, dim3((unsigned)a.rows.M), dim3(256), smem, 1, a));
   CG_LAUNCHED(c);
   return CG_OK;
 }

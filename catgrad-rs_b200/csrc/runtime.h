@@ -312,7 +312,7 @@ struct LazyPause {
 
 // y[M,N] = x[M,K] w[N,K]^T on the tcgen05 pipeline.  x, w bf16 row-major (ld in elements);
 // out_mode 0: f32 store, 1: bf16 store, 2: f32 out = acc + residual (residual may alias out),
-// 4: bf16 store of the square of relu.
+// 4: bf16 store of the square of relu, 5: bf16 store of silu.
 // splits <= 0 lets the launcher choose.  `workspace` must hold splits*M*N floats when
 // splits > 1 (pass nullptr to have it allocated from the context).
 int gemm_tc(cg_ctx* c, const __nv_bfloat16* x, int64_t ldx, const __nv_bfloat16* w, int64_t ldw,

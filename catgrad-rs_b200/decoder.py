@@ -31,6 +31,7 @@ class DecoderConfig(C.Structure):
         ("n_experts", C.c_int32), ("top_k", C.c_int32), ("moe_ffn", C.c_int32), ("norm_topk", C.c_int32),
         ("tp_rank", C.c_int32), ("tp_world", C.c_int32), ("ep_rank", C.c_int32), ("ep_world", C.c_int32),
         ("streams", C.c_int32), ("embed_norm", C.c_int32), ("loop_input", C.c_int32),
+        ("layer_norm", C.c_int32), ("residual_mult", C.c_float), ("logit_scale", C.c_float),
     ]
 
 
@@ -76,13 +77,15 @@ class Decoder:
             c.num_layers, c.hidden, c.vocab = len(cfg.layers), cfg.hidden_size, cfg.vocab_size
             c.rms_eps, c.max_seq, c.max_batch = cfg.rms_norm_eps, max_seq, max_batch
             c.embed_scale, c.streams = cfg.embed_scale, cfg.streams
+            c.residual_mult, c.logit_scale = cfg.residual_mult, cfg.logit_scale
             for k, v in cfg.design.switches().items():
                 setattr(c, k, v)
             c.tp_rank, c.tp_world, c.ep_rank, c.ep_world = tp_rank, tp_world, ep_rank, ep_world
             for k, v in switches.items():
                 setattr(c, k, v)
             self.cfg = c
-            layers = (LayerStruct * len(cfg.layers))(*[s.struct(cfg.design) for s in cfg.layers])
+            structs = [s.struct(cfg.design) for s in cfg.layers]  # (alive until the call returns, with what they point to)
+            layers = (LayerStruct * len(structs))(*structs)
             loop = C.byref(LoopStruct(*cfg.loop)) if cfg.loop else None
             h = vp()
             backend._check(L.cg_decoder_create_layers(backend._ctx, C.byref(c), layers, len(layers), loop, C.byref(h)))

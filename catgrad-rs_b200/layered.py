@@ -1,6 +1,6 @@
 """Configurations of models described layer by layer: different sequence mixers and feed-forwards, an
-optional loop over some of the layers, and what a design fixes for all of them (the Ralapel and
-Segedra designs), for `Decoder`.
+optional loop over some of the layers, and what a design fixes for all of them (the Ralapel, Segedra
+and Regupel designs), for `Decoder`.
 
 No counterpart in the reference, whose decoders are attention-only.  `LayeredConfig.from_json`
 reads a checkpoint's config.json; every size and constant comes from it.
@@ -10,7 +10,7 @@ from __future__ import annotations
 import ctypes as C
 from dataclasses import dataclass, field
 
-MIXERS = {"latent_attention": 1, "delta": 2, "mamba2": 3, "attention": 4}   # cg_mixer (include/catgrad_cuda.h)
+MIXERS = {"latent_attention": 1, "delta": 2, "mamba2": 3, "attention": 4, "lightning": 5}   # cg_mixer (include/catgrad_cuda.h)
 SILU, GELU, BOUNDED, RELU2 = range(4)                                      # cg_act
 
 
@@ -19,8 +19,11 @@ class LayerStruct(C.Structure):
     _fields_ = [("mixer", C.c_int32), ("ffn", C.c_int32), ("act", C.c_int32), ("heads", C.c_int32), ("kv_heads", C.c_int32),
                 ("dim", C.c_int32), ("rot_dim", C.c_int32), ("vdim", C.c_int32), ("kv_rank", C.c_int32), ("state", C.c_int32),
                 ("groups", C.c_int32), ("norm_groups", C.c_int32), ("conv", C.c_int32), ("window", C.c_int32), ("qk_norm", C.c_int32),
-                ("sink", C.c_int32), ("experts", C.c_int32), ("top_k", C.c_int32), ("rot_base", C.c_double), ("scale", C.c_double),
-                ("router_scale", C.c_double), ("act_limit", C.c_double)]
+                ("sink", C.c_int32), ("experts", C.c_int32), ("top_k", C.c_int32), ("correction", C.c_int32), ("scoring", C.c_int32),
+                ("weigh_input", C.c_int32), ("shared_ffn", C.c_int32), ("keep_first", C.c_int32), ("rot_half", C.c_int32), ("gate", C.c_int32),
+                ("weights_of", C.c_int32), ("rot_base", C.c_double), ("rot_factor", C.c_double), ("rot_low", C.c_double),
+                ("rot_high", C.c_double), ("rot_original", C.c_double), ("scale", C.c_double), ("router_scale", C.c_double),
+                ("act_limit", C.c_double), ("out_scale", C.c_double), ("decay", C.c_void_p), ("beside", C.c_void_p)]
 
 
 class LoopStruct(C.Structure):
@@ -29,50 +32,85 @@ class LoopStruct(C.Structure):
 
 
 @dataclass(frozen=True)
+class AttentionTraits:
+    """What a design's attention has besides its sizes."""
+    qk_norm: int = 0             # 1: norms over all query and over all key heads; 2: per head, without gains
+    sink: bool = False           # a learned term of the softmax's denominator per head
+    gate: bool = False           # a head's output times the sigmoid of a projection, one number per head
+    rot_half: bool = False       # component i is rotated with component i + dims / 2, not with its neighbour
+
+
+@dataclass(frozen=True)
+class Routing:
+    """How a design's experts are chosen, weighted and built."""
+    act: int
+    correction: bool = False     # a learned number per expert is added for the choice
+    sigmoid: bool = False        # scores are the sigmoids of the logits, not their softmax
+    weigh_input: bool = False    # the weights multiply the experts' inputs
+
+
+@dataclass(frozen=True)
 class Design:
     """What a family of layer-by-layer models fixes for all its layers."""
     mixers: tuple[str, ...]
-    dense_act: int               # of dense feed-forwards
-    experts: bool = False        # feed-forwards may be mixtures of experts
-    post_norms: bool = False     # norms behind the sublayers too
+    dense_act: int | None        # of dense feed-forwards; None: there are none
+    routing: Routing | None = None   # feed-forwards may be mixtures of experts
+    pre_norms: bool = True       # norms before the sublayers
+    post_norms: bool = False     # norms behind the sublayers
+    layer_norm: bool = False     # layer and final norms take the mean off and add a bias
     embed_norm: bool = False
     loop_input: bool = False     # a loop's passes start from W [x; normed embedding]
     norm_plus_one: bool = False  # layer and final norms multiply by 1 + w
     tied_head: bool = False
-    qk_norm: bool = False        # attention: norms over all query and over all key heads
-    sink: bool = False           # attention: a learned term of the softmax's denominator per head
+    attention: AttentionTraits = AttentionTraits()
+    beside: tuple[str, str] | None = None   # mixers of the "parallel" type, left and right
+    left: AttentionTraits = AttentionTraits()   # of the attention among them
 
     def switches(self) -> dict[str, int]:
         """Fields of `cg_decoder_config`."""
-        return {"post_norms": int(self.post_norms), "embed_norm": int(self.embed_norm), "loop_input": int(self.loop_input),
-                "norm_plus_one": int(self.norm_plus_one), "tie_embeddings": int(self.tied_head)}
+        return {"post_norms": 0 if not self.post_norms else 1 if self.pre_norms else 2, "layer_norm": int(self.layer_norm),
+                "embed_norm": int(self.embed_norm), "loop_input": int(self.loop_input), "norm_plus_one": int(self.norm_plus_one),
+                "tie_embeddings": int(self.tied_head)}
+
+    def norms(self, q: int) -> list[str]:
+        """Names of the norms around sublayer q of a layer."""
+        names = [f"norm{q}"] + ([f"norm{q}b"] if self.pre_norms and self.post_norms else [])
+        return [n + b for n in names for b in (("", ".b") if self.layer_norm else ("",))]
 
 
 DESIGNS = {
     "Ralapel": Design(("latent_attention", "delta", "mamba2"), GELU, post_norms=True, embed_norm=True, loop_input=True),
-    "Segedra": Design(("attention",), RELU2, experts=True, norm_plus_one=True, tied_head=True, qk_norm=True, sink=True),
+    "Segedra": Design(("attention",), RELU2, Routing(BOUNDED, correction=True), norm_plus_one=True, tied_head=True,
+                      attention=AttentionTraits(qk_norm=1, sink=True)),
+    "Regupel": Design(("attention", "parallel"), None, Routing(SILU, sigmoid=True, weigh_input=True), pre_norms=False, post_norms=True,
+                      layer_norm=True, tied_head=True, attention=AttentionTraits(qk_norm=2, sink=True, gate=True, rot_half=True),
+                      beside=("attention", "lightning"), left=AttentionTraits(qk_norm=1)),
 }
 
 
 @dataclass
 class Experts:
-    """A mixture-of-experts feed-forward: `top` of `count` experts per token, chosen by the router's
-    softmax plus a correction, weighted by the softmax times `scale`; `limit` bounds their units."""
+    """A mixture-of-experts feed-forward: `top` of `count` experts per token, their scores times `scale` the
+    weights; `limit` bounds their units where the design has that; `shared` is the width of one more
+    expert that every token runs (0: none)."""
     count: int
     top: int
-    scale: float
-    limit: float
+    scale: float = 1.0
+    limit: float = 0.0
+    shared: int = 0
 
 
 @dataclass
 class LayerSpec:
     """One layer: the mixer's name, its sizes (the keys config.json uses) and the feed-forward width
-    (of one expert if there are experts; 0 = the layer has none)."""
+    (of one expert if there are experts; 0 = the layer has none).  With `weights_of` the layer has no
+    parameters of its own but those of that layer."""
     mixer: str
     sizes: dict
     ffn: int = 0
     act: int = GELU
     experts: Experts | None = None
+    weights_of: int | None = None
 
     @property
     def window(self) -> int:
@@ -80,21 +118,55 @@ class LayerSpec:
         return (self.sizes.get("mask") or {}).get("size") or 0
 
     @property
+    def kept(self) -> int:
+        """First tokens that stay visible beyond the window."""
+        return (self.sizes.get("mask") or {}).get("keep_first") or 0
+
+    @property
     def rotated(self) -> int:
         """Rotated components of an attention head."""
         return (self.sizes.get("rot") or {}).get("dims", 0)
 
+    def parts(self, design: Design) -> list[tuple[str, "LayerSpec", AttentionTraits]]:
+        """(prefix of the tensors, single mixer, traits if it is attention)."""
+        if self.mixer != "parallel":
+            return [("", self, design.attention)]
+        return [(f"{side}.", LayerSpec(kind, self.sizes[side]), design.left) for side, kind in zip(("left", "right"), design.beside)]
+
     def struct(self, design: Design) -> LayerStruct:
-        s, m = LayerStruct(), self.sizes
-        s.mixer, s.ffn, s.act = MIXERS[self.mixer], self.ffn, self.act
-        s.heads, s.vdim = m["heads"], m["vdim"]
+        """The returned struct points into ones it keeps alive (`keep`)."""
+        if self.mixer == "parallel":
+            s, right = (p.mixer_struct(t) for _, p, t in self.parts(design))
+            s.out_scale, right.out_scale = self.sizes["left_scale"], self.sizes["right_scale"]
+            s.beside = C.addressof(right)
+            s.keep = [right]
+        else:
+            s = self.mixer_struct(design.attention)
+        s.ffn, s.act = self.ffn, self.act
+        s.weights_of = 0 if self.weights_of is None else self.weights_of + 1
         if self.experts:
-            e = self.experts
-            s.experts, s.top_k, s.router_scale, s.act_limit = e.count, e.top, e.scale, e.limit
+            e, r = self.experts, design.routing
+            s.experts, s.top_k, s.router_scale, s.act_limit, s.shared_ffn = e.count, e.top, e.scale, e.limit, e.shared
+            s.correction, s.scoring, s.weigh_input = int(r.correction), int(r.sigmoid), int(r.weigh_input)
+        return s
+
+    def mixer_struct(self, traits: AttentionTraits) -> LayerStruct:
+        s, m = LayerStruct(), self.sizes
+        s.mixer = MIXERS[self.mixer]
+        s.heads, s.vdim = m["heads"], m["vdim"]
         if self.mixer == "attention":
-            s.dim, s.kv_heads, s.scale, s.window = m["dim"], m["kv_heads"], m["scale"], self.window
+            s.dim, s.kv_heads, s.scale, s.window, s.keep_first = m["dim"], m["kv_heads"], m["scale"], self.window, self.kept
             s.rot_dim, s.rot_base = self.rotated, m["rot"]["base"] if self.rotated else 0.0
-            s.qk_norm, s.sink = int(design.qk_norm), int(design.sink)
+            scaling = (m.get("rot") or {}).get("scaling")
+            if scaling:
+                s.rot_factor, s.rot_low, s.rot_high, s.rot_original = (scaling[k] for k in ("factor", "low", "high", "original"))
+            s.qk_norm, s.sink, s.gate, s.rot_half = traits.qk_norm, int(traits.sink), int(traits.gate), int(traits.rot_half)
+        elif self.mixer == "lightning":
+            if len(m["decay"]) != m["heads"]:
+                raise ValueError("a decay per head")
+            s.dim = m["dim"]
+            s.keep = (C.c_double * m["heads"])(*m["decay"])
+            s.decay = C.addressof(s.keep)
         elif self.mixer == "latent_attention":
             s.dim, s.rot_dim, s.kv_rank, s.scale = m["dim"], m["rot_dim"], m["kv_rank"], m["scale"]
             s.rot_base = m["rot"]["base"] if m["rot_dim"] else 0.0
@@ -118,6 +190,8 @@ class LayeredConfig:
     design: Design = DESIGNS["Ralapel"]
     streams: int = 0                           # rows of the residual stream per token; 0 = a plain one
     embed_scale: float = 1.0
+    residual_mult: float = 1.0
+    logit_scale: float = 1.0
     extras: dict = field(default_factory=dict)
 
     @classmethod
@@ -128,24 +202,36 @@ class LayeredConfig:
         for i, e in enumerate(d["layers"]):
             if e["type"] not in design.mixers:
                 raise ValueError(f"layer {i}: unknown mixer {e['type']!r}")
-            mlp = e.get("mlp")
-            if mlp and not (mlp["kind"] == "dense" or (mlp["kind"] == "moe" and design.experts)):
+            mlp, of = e.get("mlp"), e.get("weights_of")
+            if mlp and not ((mlp["kind"] == "dense" and design.dense_act is not None) or (mlp["kind"] == "moe" and design.routing)):
                 raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
             if e["type"] == "latent_attention" and e["mixer"]["rot_dim"] and e["mixer"]["rot"]["dims"] != e["mixer"]["rot_dim"]:
                 raise ValueError(f"layer {i}: the rotated part must be rotated whole")
+            seen = set()
+            while of is not None and d["layers"][of].get("weights_of") is not None and of not in seen:
+                seen.add(of)
+                of = d["layers"][of]["weights_of"]
             if mlp and mlp["kind"] == "moe":
                 r, x = mlp["router"], mlp["expert"]
-                layers.append(LayerSpec(e["type"], e["mixer"], x["ff"], BOUNDED, Experts(r["experts"], r["top"], r["scale"], x["limit"])))
+                ex = Experts(r["experts"], r["top"], r.get("scale", 1.0), x.get("limit", 0.0), (mlp.get("shared") or {}).get("ff", 0))
+                layers.append(LayerSpec(e["type"], e["mixer"], x["ff"], design.routing.act, ex, of))
             else:
-                layers.append(LayerSpec(e["type"], e["mixer"], mlp["ff"] if mlp else 0, design.dense_act))
+                act = SILU if design.dense_act is None else design.dense_act
+                layers.append(LayerSpec(e["type"], e["mixer"], mlp["ff"] if mlp else 0, act, None, of))
         lp = d.get("loop")
         return cls(name, d["width"], d["vocab"], layers, (lp["start"], lp["stop"], lp["times"]) if lp else None, d["norm"]["eps"],
-                   design=design, streams=d.get("streams") or 0, embed_scale=(d.get("embedding") or {}).get("scale", 1.0))
+                   design=design, streams=d.get("streams") or 0, embed_scale=(d.get("embedding") or {}).get("scale", 1.0),
+                   residual_mult=d.get("residual_mult", 1.0), logit_scale=d.get("logit_scale", 1.0))
 
     @property
     def recurrent(self) -> bool:
         """Whether some layer's state cannot go back to an earlier position."""
-        return any(L.mixer in ("delta", "mamba2") for L in self.layers)
+        return any(p.mixer in ("delta", "mamba2", "lightning") for L in self.layers for _, p, _ in L.parts(self.design))
+
+    def owner(self, i: int) -> int:
+        """The layer whose parameters layer i uses."""
+        of = self.layers[i].weights_of
+        return i if of is None else of
 
     def layer_runs(self) -> list[int]:
         """Layers in the order they run."""
@@ -159,6 +245,8 @@ class LayeredConfig:
         """Tensor names and shapes of a checkpoint (weights [out, in])."""
         W, D = self.hidden_size, self.design
         s = {"embed": (self.vocab_size, W), "final.norm": (W,)}
+        if D.layer_norm:
+            s["final.norm.b"] = (W,)
         if D.embed_norm:
             s["embed.norm"] = (W,)
         if not D.tied_head:
@@ -166,52 +254,66 @@ class LayeredConfig:
         if self.loop and D.loop_input:
             s["loop.in"] = (W, 2 * W)
         for i, L in enumerate(self.layers):
-            p, m = f"l{i}.", L.sizes
-            H, dv = m["heads"], m["vdim"]
+            if L.weights_of is not None:
+                continue
+            p = f"l{i}."
             for q in (1, 2) if L.ffn else (1,):
-                s[p + f"norm{q}"] = (W,)
-                if D.post_norms:
-                    s[p + f"norm{q}b"] = (W,)
+                s.update({p + n: (W,) for n in D.norms(q)})
                 if self.streams:
                     s[p + f"hc{q}.in"] = s[p + f"hc{q}.out"] = (self.streams,)
                     s[p + f"hc{q}.mix"] = (self.streams, self.streams)
             if L.experts:
-                s[p + "mlp.router"], s[p + "mlp.correction"] = (L.experts.count, W), (L.experts.count,)
-                for e in range(L.experts.count):
-                    s[p + f"mlp.e{e}.gate"] = s[p + f"mlp.e{e}.up"] = (L.ffn, W)
-                    s[p + f"mlp.e{e}.down"] = (W, L.ffn)
+                s[p + "mlp.router"] = (L.experts.count, W)
+                if D.routing.correction:
+                    s[p + "mlp.correction"] = (L.experts.count,)
+                units = {f"mlp.e{e}.": L.ffn for e in range(L.experts.count)} | ({"mlp.shared.": L.experts.shared} if L.experts.shared else {})
+                for n, f in units.items():
+                    s[p + n + "gate"] = s[p + n + "up"] = (f, W)
+                    s[p + n + "down"] = (W, f)
             elif L.ffn:
                 s[p + "mlp.up"], s[p + "mlp.down"] = (L.ffn, W), (W, L.ffn)
                 if L.act != RELU2:
                     s[p + "mlp.gate"] = (L.ffn, W)
-            p += "mix."
-            s[p + "o"] = (W, H * dv)
-            if L.mixer == "attention":
-                G, d = m["kv_heads"], m["dim"]
-                s[p + "q"], s[p + "k"], s[p + "v"] = (H * d, W), (G * d, W), (G * dv, W)
-                if D.qk_norm:
-                    s[p + "q.norm"], s[p + "k.norm"] = (H * d,), (G * d,)
-                if D.sink:
-                    s[p + "sink"] = (H,)
-            elif L.mixer == "latent_attention":
-                d, r, R = m["dim"], m["rot_dim"], m["kv_rank"]
-                s[p + "q"], s[p + "dkv"], s[p + "dkv.norm"] = (H * (d + r), W), (R + r, W), (R,)
-                s[p + "uk"], s[p + "uv"] = (H * d, R), (H * dv, R)
-            elif L.mixer == "delta":
-                K, d, taps = m["kv_heads"], m["dim"], m["conv"]
-                for n, rows in (("q", K * d), ("k", K * d), ("v", H * dv)):
-                    s[p + n], s[p + n + ".conv"] = (rows, W), (rows, taps)
-                s[p + "b"] = s[p + "a"] = (H, W)
-                s[p + "g"] = (H * dv, W)
-                s[p + "A_log"] = s[p + "dt_bias"] = (H,)
-                s[p + "norm"] = (dv,)
-            else:
-                N, G, taps = m["state"], m["groups"], m["conv"]
-                ch = H * dv + 2 * G * N
-                s[p + "in"], s[p + "conv"], s[p + "conv.b"] = (H * dv + ch + H, W), (ch, taps), (ch,)
-                s[p + "A_log"] = s[p + "dt_bias"] = s[p + "D"] = (H,)
-                s[p + "norm"] = (H * dv,)
+            for side, part, traits in L.parts(D):
+                self._mixer_shapes(s, p + "mix." + side, part, traits)
         return s
+
+    def _mixer_shapes(self, s: dict, p: str, L: LayerSpec, traits: AttentionTraits):
+        W, m = self.hidden_size, L.sizes
+        H, dv = m["heads"], m["vdim"]
+        s[p + "o"] = (W, H * dv)
+        if L.mixer == "attention":
+            G, d = m["kv_heads"], m["dim"]
+            s[p + "q"], s[p + "k"], s[p + "v"] = (H * d, W), (G * d, W), (G * dv, W)
+            if traits.qk_norm == 1:
+                s[p + "q.norm"], s[p + "k.norm"] = (H * d,), (G * d,)
+            if traits.sink:
+                s[p + "sink"] = (H,)
+            if traits.gate:
+                s[p + "g"] = (H, W)
+        elif L.mixer == "lightning":
+            d = m["dim"]
+            s[p + "q"] = s[p + "k"] = (H * d, W)
+            s[p + "v"] = s[p + "g"] = (H * dv, W)
+            s[p + "norm"] = (H * dv,)
+        elif L.mixer == "latent_attention":
+            d, r, R = m["dim"], m["rot_dim"], m["kv_rank"]
+            s[p + "q"], s[p + "dkv"], s[p + "dkv.norm"] = (H * (d + r), W), (R + r, W), (R,)
+            s[p + "uk"], s[p + "uv"] = (H * d, R), (H * dv, R)
+        elif L.mixer == "delta":
+            K, d, taps = m["kv_heads"], m["dim"], m["conv"]
+            for n, rows in (("q", K * d), ("k", K * d), ("v", H * dv)):
+                s[p + n], s[p + n + ".conv"] = (rows, W), (rows, taps)
+            s[p + "b"] = s[p + "a"] = (H, W)
+            s[p + "g"] = (H * dv, W)
+            s[p + "A_log"] = s[p + "dt_bias"] = (H,)
+            s[p + "norm"] = (dv,)
+        else:
+            N, G, taps = m["state"], m["groups"], m["conv"]
+            ch = H * dv + 2 * G * N
+            s[p + "in"], s[p + "conv"], s[p + "conv.b"] = (H * dv + ch + H, W), (ch, taps), (ch,)
+            s[p + "A_log"] = s[p + "dt_bias"] = s[p + "D"] = (H,)
+            s[p + "norm"] = (H * dv,)
 
     def synthetic(self, name: str) -> tuple[float, float]:
         """(mean, std) a synthetic checkpoint draws a tensor with: gains 1, slow decays, wide taps,
@@ -224,6 +326,8 @@ class LayeredConfig:
         if name.endswith("conv"):
             return 0.0, 0.4
         if name.endswith("conv.b"):
+            return 0.0, 0.1
+        if name.endswith(".b") and not name.endswith(".mix.b"):
             return 0.0, 0.1
         if leaf in ("D", "norm", "norm1", "norm1b", "norm2", "norm2b"):
             plus_one = self.design.norm_plus_one and ".mix." not in name
@@ -258,6 +362,27 @@ def segedra_shape(name: str, width: int, heads: int, kv_heads: int, dim: int, wi
                          embed_scale=width ** 0.5)
 
 
+def regupel_shape(name: str, width: int, heads: int, kv_heads: int, dim: int, window: int, kept: int, experts: Experts, ff: int,
+                  vocab: int) -> LayeredConfig:
+    """A Regupel-shaped model at a real model's widths, for measurements: three of four layers carry windowed
+    attention beside lightning attention (half the heads, values as wide as keys), every fourth is
+    gated attention with a window four times as long; one of those uses another one's weights."""
+    def layer(i):
+        if i % 4 == 1:
+            m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** 0.5, "mask": {"size": 4 * window},
+                 "rot": {"base": 500000.0, "dims": dim // 2, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+            return LayerSpec("attention", m, ff, SILU, experts, weights_of=1 if i == 5 else None)
+        left = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "mask": {"size": window, "keep_first": kept}}
+        n = heads // 2
+        right = {"heads": n, "dim": dim, "vdim": dim, "decay": [1.0 - 2.0 ** -(1.0 + 9.0 * h / max(n - 1, 1)) for h in range(n)]}
+        return LayerSpec("parallel", {"left": left, "right": right, "left_scale": 0.7, "right_scale": 0.7}, ff, SILU, experts)
+    return LayeredConfig(name, width, vocab, [layer(i) for i in range(8)], None, 1e-6, design=DESIGNS["Regupel"], embed_scale=width ** 0.5,
+                         residual_mult=0.8, logit_scale=0.25)
+
+
+REGUPEL_W1024 = regupel_shape("regupel-w1024-shape", 1024, 16, 4, 64, 128, 16, Experts(32, 4, shared=512), 512, 32000)
+REGUPEL_W2048 = regupel_shape("regupel-w2048-shape", 2048, 32, 4, 128, 512, 64, Experts(128, 8, shared=768), 768, 151936)
+REGUPEL_W2880 = regupel_shape("regupel-w2880-shape", 2880, 64, 8, 64, 128, 128, Experts(32, 4, shared=2880), 2880, 201088)
 SEGEDRA_W1024 = segedra_shape("segedra-w1024-shape", 1024, 16, 4, 64, 128, Experts(32, 4, 1.0, 7.0), 512, 4096, 2, 32000)
 SEGEDRA_W2048 = segedra_shape("segedra-w2048-shape", 2048, 32, 4, 128, 512, Experts(128, 8, 2.5, 7.0), 768, 8192, 4, 151936)
 SEGEDRA_W2880 = segedra_shape("segedra-w2880-shape", 2880, 64, 8, 64, 128, Experts(32, 4, 1.0, 7.0), 2880, 11520, 4, 201088)

@@ -46,6 +46,7 @@ ARCHITECTURES = {
     "Gemma3ForCausalLM": _hf("gemma"),
     "Ralapel": LayeredConfig.from_json,
     "Segedra": LayeredConfig.from_json,
+    "Regupel": LayeredConfig.from_json,
 }
 
 

@@ -55,6 +55,9 @@ pub struct DecoderConfig {
     pub streams: i32,
     pub embed_norm: i32,
     pub loop_input: i32,
+    pub layer_norm: i32,
+    pub residual_mult: f32,
+    pub logit_scale: f32,
 }
 
 #[repr(C)]

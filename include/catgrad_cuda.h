@@ -294,7 +294,8 @@ typedef struct cg_decoder_config {
   int32_t qk_norm;          /* per-head RMSNorm on q and k (qwen3.rs:187-217) */
   int32_t act;              /* 0 silu, 1 tanh-gelu */
   int32_t norm_plus_one;    /* (1 + gamma) norms (gemma3.rs:60-68) */
-  int32_t post_norms;       /* post-attention and post-ffn norms (gemma3.rs:192-238) */
+  int32_t post_norms;       /* post-attention and post-ffn norms (gemma3.rs:192-238); layer by layer: 2 = these only, no
+                               norms before the sublayers */
   float embed_scale;        /* 0 = none, else multiply embeddings (gemma3.rs:257-260) */
   float attn_softcap;
   float final_softcap;
@@ -337,6 +338,9 @@ typedef struct cg_decoder_config {
                                residual stream) */
   int32_t embed_norm;       /* an RMS norm of the embedding */
   int32_t loop_input;       /* a loop's passes start from W [x; normed embedding] */
+  int32_t layer_norm;       /* the layers' and the final norm take the mean off and add a bias (with post_norms) */
+  float residual_mult;      /* factor on what a sublayer adds to the residual stream (0 = 1; with post_norms) */
+  float logit_scale;        /* factor on the logits (0 = 1; with post_norms) */
 } cg_decoder_config;
 
 int32_t cg_decoder_create(cg_ctx*, const cg_decoder_config* cfg, cg_decoder** out);
@@ -391,9 +395,11 @@ int32_t cg_decoder_generate(cg_decoder*, const uint32_t* prompt, int32_t batch, 
 
 /* --- decoders built layer by layer: layers with different sequence mixers, optionally run in a loop.
  * No counterpart in the reference, whose decoders are attention-only.  Every layer is
- *   x <- x + post1(mixer(norm1(x))),  x <- x + post2(ff(norm2(x)))
- * with RMS norms (the second line only where the layer has a feed-forward; post1, post2 are norms with
- * post_norms, else nothing) and a norm before the head.  With streams = s > 0 the residual stream is s
+ *   x <- x + m post1(mixer(norm1(x))),  x <- x + m post2(ff(norm2(x)))
+ * with m the residual_mult and RMS norms or, with layer_norm, layer norms with biases (the second line
+ * only where the layer has a feed-forward; post1, post2 are norms with post_norms, else nothing; with
+ * post_norms 2 norm1, norm2 are nothing) and a norm before the head.  A layer may have two mixers side by
+ * side, which read the same rows and whose scaled results are added.  With streams = s > 0 the residual stream is s
  * rows x_1 .. x_s, all equal to the embedding at first, and a sublayer f with coefficients in [s],
  * out [s], mix [s, s] takes u = sum_s in[s] x_s and leaves
  *   x_t <- sum_s mix[s, t] x_s + out[t] f(norm(u));
@@ -406,7 +412,9 @@ typedef enum cg_mixer {
   CG_MIX_LATENT = 1, /* latent attention: keys and values are linear maps of a cached low-rank row */
   CG_MIX_DELTA = 2,  /* gated delta rule behind short convolutions */
   CG_MIX_SSD = 3,    /* Mamba-2: scalar-decay state space with a gated group norm */
-  CG_MIX_ATTENTION = 4 /* grouped-query attention: optional norms, window and sink */
+  CG_MIX_ATTENTION = 4, /* grouped-query attention: optional norms, window, kept first tokens, sink and gate */
+  CG_MIX_LIGHTNING = 5 /* lightning attention: silu of queries, keys and values, a matrix state with a constant
+                          decay per head, an RMS norm over all heads and a sigmoid gate */
 } cg_mixer;
 typedef enum cg_act {
   CG_ACT_SILU = 0,    /* down(silu(gate h) * up h) */
@@ -418,9 +426,9 @@ typedef struct cg_layer_config {
   int32_t mixer;     /* cg_mixer */
   int32_t ffn;       /* width of the feed-forward (of one expert), 0 = none */
   int32_t act;       /* cg_act */
-  int32_t heads;     /* latent, attention: query heads; delta, ssd: value heads */
+  int32_t heads;     /* latent, attention: query heads; delta, ssd: value heads; lightning: heads */
   int32_t kv_heads;  /* delta: query/key heads, attention: key/value heads; a divisor of heads */
-  int32_t dim;       /* latent: unrotated query/key size per head; delta, attention: query/key size per head */
+  int32_t dim;       /* latent: unrotated query/key size per head; delta, attention, lightning: query/key size per head */
   int32_t rot_dim;   /* latent: rotated query/key size, the key part shared by all heads; attention: how many
                         components of a head are rotated, from the first */
   int32_t vdim;      /* value size per head */
@@ -430,30 +438,49 @@ typedef struct cg_layer_config {
   int32_t norm_groups; /* ssd: equal parts of the gated norm */
   int32_t conv;      /* delta, ssd: taps of the short convolutions */
   int32_t window;    /* attention: a token sees itself and the window - 1 tokens before it, 0 = all */
-  int32_t qk_norm;   /* attention: 1 = RMS norm over all query heads at once, and over all key heads, before rotation */
+  int32_t qk_norm;   /* attention: 1 = RMS norm over all query heads at once, and over all key heads, before rotation;
+                        2 = per head, without gains */
   int32_t sink;      /* attention: 1 = the softmax has one more term per head, exp(sink), without a value */
-  int32_t experts;   /* feed-forward: 0 = dense, else the number of experts, softmax-routed */
-  int32_t top_k;     /* experts per token: those with the largest probability + correction */
-  double rot_base;   /* latent, attention: base of the rotary frequencies; neighbouring components are paired */
+  int32_t experts;   /* feed-forward: 0 = dense, else the number of experts */
+  int32_t top_k;     /* experts per token: those with the largest probability (+ correction) */
+  int32_t correction; /* experts: 1 = a learned number per expert is added for the choice */
+  int32_t scoring;   /* experts: 0 = softmax of the router's logits, 1 = the sigmoid of each */
+  int32_t weigh_input; /* experts: 1 = the weights multiply the experts' inputs instead of their outputs */
+  int32_t shared_ffn; /* experts: width of one more that every token runs, unweighted (0 = none) */
+  int32_t keep_first; /* attention with a window: the first keep_first tokens of a sequence stay visible */
+  int32_t rot_half;  /* attention: 1 = component i is rotated with component i + rot_dim / 2, 0 = with its neighbour */
+  int32_t gate;      /* attention: 1 = a head's output is multiplied by the sigmoid of a projection, one number per head */
+  int32_t weights_of; /* 0 = the layer has its own parameters, else 1 + the layer whose parameters it uses (with a
+                        cache or state of its own); the other fields are then those of that layer */
+  double rot_base;   /* latent, attention: base of the rotary frequencies */
+  double rot_factor, rot_low, rot_high, rot_original; /* rot_factor > 0: with l = 2 pi / f, frequencies f stay where
+                        l < original / high, become f / factor where l > original / low, and blend in between */
   double scale;      /* latent, attention: factor on the scores */
   double router_scale; /* factor on the chosen experts' probabilities, which are not renormalised */
   double act_limit;  /* CG_ACT_BOUNDED */
+  double out_scale;  /* two mixers: factor on this one's result (0 = 1) */
+  const double* decay; /* lightning: [heads], the state's factor per token, in [0, 1] (read during the call) */
+  const struct cg_layer_config* beside; /* a second mixer, of which the mixer's fields count (read during the call) */
 } cg_layer_config;
 typedef struct cg_loop_config {
   int32_t start, stop, times; /* layers [start, stop) run `times` times in a row, each pass with its own cache or
                                  state; with loop_input, before a pass x <- W [x; x0], x0 the normed embedding */
 } cg_loop_config;
 /* cfg supplies hidden, vocab, rms_eps, max_seq (capacity per sequence), max_batch (sequences held at
- * once), embed_scale, norm_plus_one (layer and final norms), post_norms (excludes streams), tie_embeddings,
- * streams, embed_norm and loop_input (excludes streams).  loop may be NULL.  Parameters
+ * once), embed_scale, norm_plus_one (layer and final norms, without post_norms), post_norms (excludes
+ * streams), layer_norm, residual_mult, logit_scale, tie_embeddings, streams, embed_norm and loop_input
+ * (excludes streams).  loop may be NULL.  Parameters
  * (cg_decoder_set_param / _load_safetensors), weights [out, in]: embed, final.norm, with the options above
- * embed.norm, loop.in [hidden, 2 hidden] and head, and per layer l<i>.norm1, .norm2, with post_norms
- * .norm1b, .norm2b, with streams .hc1.{in,out,mix}, .hc2.{in,out,mix}, dense .mlp.{gate,up,down},
- * experts .mlp.{router,correction} and .mlp.e<j>.{gate,up,down}, .mix.o and
- *   attention  .mix.{q,k,v}, with qk_norm .mix.{q,k}.norm, with sink .mix.sink
+ * embed.norm, loop.in [hidden, 2 hidden] and head, and per layer l<i>.norm1, .norm2, with post_norms 1
+ * .norm1b, .norm2b (with post_norms 2 .norm1, .norm2 are the norms behind), with layer_norm also
+ * <norm>.b, with streams .hc1.{in,out,mix}, .hc2.{in,out,mix}, dense .mlp.{gate,up,down},
+ * experts .mlp.router, .mlp.correction, .mlp.e<j>.{gate,up,down}, .mlp.shared.{gate,up,down}, .mix.o and
+ *   attention  .mix.{q,k,v}, with qk_norm 1 .mix.{q,k}.norm, with sink .mix.sink, with gate .mix.g
  *   latent  .mix.{q,dkv,dkv.norm,uk,uv}
  *   delta   .mix.{q,k,v,b,a,g}, .mix.{q,k,v}.conv, .mix.{A_log,dt_bias,norm}
- *   ssd     .mix.{in,conv,conv.b,dt_bias,A_log,D,norm}.
+ *   ssd     .mix.{in,conv,conv.b,dt_bias,A_log,D,norm}
+ *   lightning  .mix.{q,k,v,g,norm};
+ * two mixers have theirs under .mix.left. and .mix.right.
  * The decoder then serves cg_decoder_prefill / append / decode / step_with / tokens / generate like
  * any other (rows = slots 0 .. B-1, equal lengths), and the calls below.  cg_decoder_truncate takes
  * 0 or the cached position only if the model has a recurrent layer: a state has no earlier versions
