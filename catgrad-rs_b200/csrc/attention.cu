@@ -151,8 +151,8 @@ __global__ void __launch_bounds__(BQ * 2, D <= 64 ? 2 : 1) k_attn_prefill(AttnAr
         const int64_t qp = qpos[e >> 1];
         float v = s[j][e] * scale;
         if (a.softcap > 0.f) v = a.softcap * tanh_sig(v / a.softcap);
-        const bool keep = kpos <= qp && kpos < kv_len && (a.window <= 0 || kpos > qp - a.window || kpos < keep);
-        v = keep ? v : -INFINITY;
+        const bool sees = kpos <= qp && kpos < kv_len && (a.window <= 0 || kpos > qp - a.window || kpos < keep);
+        v = sees ? v : -INFINITY;
         s[j][e] = v;
         mx[e >> 1] = fmaxf(mx[e >> 1], v);
       }
