@@ -121,6 +121,11 @@ LAYERED_WORKLOADS = {
     "segedra-w2048-b1": ("SEGEDRA_W2048", 1, 1024, 128),
     "segedra-w2048-long": ("SEGEDRA_W2048", 4, 4096, 128),
     "segedra-w2880": ("SEGEDRA_W2880", 8, 1024, 128),
+    "regupel-w1024": ("REGUPEL_W1024", 8, 512, 128),
+    "regupel-w2048": ("REGUPEL_W2048", 8, 1024, 128),
+    "regupel-w2048-b1": ("REGUPEL_W2048", 1, 1024, 128),
+    "regupel-w2048-long": ("REGUPEL_W2048", 4, 4096, 128),
+    "regupel-w2880": ("REGUPEL_W2880", 8, 1024, 128),
 }
 
 
@@ -138,17 +143,18 @@ def layered_step_bytes(cfg, batch: int, context: float) -> dict:
     for i in cfg.layer_runs():
         e = cfg.layers[i].experts
         mats += sum(2 * n[0] * n[1] for k, n in shapes.items()
-                    if k.startswith(f"l{i}.") and len(n) == 2 and not k.endswith("conv") and ".mlp.e" not in k)
+                    if k.startswith(f"l{cfg.owner(i)}.") and len(n) == 2 and not k.endswith("conv") and ".mlp.e" not in k)
         if e:
             mats += 6 * cfg.hidden_size * cfg.layers[i].ffn * experts_reached(e.count, e.top, batch)
-        m = cfg.layers[i].sizes
-        if cfg.layers[i].mixer == "attention":
-            seen = min(context, cfg.layers[i].window or context)
-            cache += batch * seen * m["kv_heads"] * (m["dim"] + m["vdim"]) * 2
-        elif cfg.layers[i].mixer == "latent_attention":
-            cache += batch * context * (m["kv_rank"] + m["rot_dim"]) * 2
-        else:
-            states += 2 * 4 * batch * m["heads"] * m["vdim"] * (m["dim"] if cfg.layers[i].mixer == "delta" else m["state"])
+        for _, part, _ in cfg.layers[i].parts(cfg.design):
+            m = part.sizes
+            if part.mixer == "attention":
+                seen = min(context, part.window + part.kept if part.window else context)
+                cache += batch * seen * m["kv_heads"] * (m["dim"] + m["vdim"]) * 2
+            elif part.mixer == "latent_attention":
+                cache += batch * context * (m["kv_rank"] + m["rot_dim"]) * 2
+            else:
+                states += 2 * 4 * batch * m["heads"] * m["vdim"] * (m["state"] if part.mixer == "mamba2" else m["dim"])
     if cfg.loop and "loop.in" in shapes:
         mats += cfg.loop[2] * 2 * shapes["loop.in"][0] * shapes["loop.in"][1]
     return {"weights": mats, "states": states, "cached_rows": cache}
@@ -165,8 +171,9 @@ def layered_workload(cg, C, args, local):
     heads = max(1, cfg.hidden_size // 128)
     last = cfg.layers[-1]
     if last.experts:
-        closest = cg.synth.ModelConfig("qwen3-moe-equal-size", cfg.hidden_size, last.ffn, len(cfg.layer_runs()), last.sizes["heads"],
-                                       last.sizes["kv_heads"], cfg.vocab_size, head_dim=last.sizes["dim"], dtype="bf16", arch="qwen3",
+        sizes = last.parts(cfg.design)[0][1].sizes
+        closest = cg.synth.ModelConfig("qwen3-moe-equal-size", cfg.hidden_size, last.ffn, len(cfg.layer_runs()), sizes["heads"],
+                                       sizes["kv_heads"], cfg.vocab_size, head_dim=sizes["dim"], dtype="bf16", arch="qwen3",
                                        num_local_experts=last.experts.count, num_experts_per_tok=last.experts.top, moe_intermediate_size=last.ffn)
     else:
         closest = cg.synth.ModelConfig("llama-equal-size", cfg.hidden_size, max(L.ffn for L in cfg.layers), len(cfg.layer_runs()), heads,
@@ -486,7 +493,7 @@ def main():
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--workload", default="llama1b", choices=sorted(WORKLOADS) + sorted(LAYERED_WORKLOADS),
                     help="llama1b is the configuration the metric is quoted on; the others are the remaining "
-                         "model shapes at their own batch / prompt / decode sizes; ralapel-* and segedra-* measure a model "
+                         "model shapes at their own batch / prompt / decode sizes; ralapel-*, segedra-* and regupel-* measure a model "
                          "built layer by layer beside an attention-only decoder of equal size (one GPU)")
     ap.add_argument("--batch", type=int, default=0)
     ap.add_argument("--prompt", type=int, default=0)

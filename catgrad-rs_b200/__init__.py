@@ -6,7 +6,8 @@ The directory name is not a Python identifier; import it with
 * `backend`  — `CudaBackend`, the mirror of `trait Backend` over the C ABI
 * `graphs`   — the op streams of catgrad's stdlib and catgrad-llm model graphs
 * `decoder`  — the fused, KV-cached greedy runner
-* `layered`  — configurations of models with different mixers per layer (the Ralapel and Segedra designs)
+* `layered`  — configurations of models with different mixers per layer (the Ralapel, Segedra
+  and Regupel designs)
 * `registry` — from a checkpoint folder to a decoder, by the architecture its config.json names
 * `synth`    — seeded synthetic checkpoints and prompts
 * `safetensors_io` — .safetensors checkpoint files: library-side reader, numpy writer

@@ -32,6 +32,8 @@
 // loops, meet at the closing cluster barrier, free TMEM and return.
 #include <algorithm>
 
+#include <type_traits>
+
 #include "act.cuh"
 #include "tc_common.cuh"
 
@@ -310,12 +312,18 @@ k_gemm_tcp2(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ C
                 if (m < m_end) ((float*)p.out)[(int64_t)m * p.ldo + n] = __uint_as_float(cur[j]);
               }
             } else {
+              // (the mode is chosen outside the loop: inside, every element would pay for all of them)
+              auto store = [&](auto mode) {
 #pragma unroll
-              for (int j = 0; j < 32; ++j) {
-                const int m = m0 + c0 + j;
-                const float a = __uint_as_float(cur[j]);
-                if (m < m_end) ((__nv_bfloat16*)p.out)[(int64_t)m * p.ldo + n] = __float2bfloat16_rn(bf16_out(p.out_mode, a));
-              }
+                for (int j = 0; j < 32; ++j) {
+                  const int m = m0 + c0 + j;
+                  if (m < m_end)
+                    ((__nv_bfloat16*)p.out)[(int64_t)m * p.ldo + n] = __float2bfloat16_rn(bf16_out(decltype(mode)::value, __uint_as_float(cur[j])));
+                }
+              };
+              if (p.out_mode == 5) store(std::integral_constant<int, 5>());
+              else if (p.out_mode == 4) store(std::integral_constant<int, 4>());
+              else store(std::integral_constant<int, 1>());
             }
           }
           if (c0 + 32 < col0 + P2_TOK / 2) asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");

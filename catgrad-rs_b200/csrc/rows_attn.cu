@@ -48,38 +48,54 @@ __device__ __forceinline__ void st4(__nv_bfloat16* p, float4 v) {
   *(uint2*)p = make_uint2(*(const uint32_t*)&lo, *(const uint32_t*)&hi);
 }
 
-// One block per token; Dk and Dv are multiples of 8, so four neighbours belong to one head.
-template <class T>
-__global__ void __launch_bounds__(256) k_rows_qkv(RowsAttnArgs a) {
+// One block per token; Dk and Dv are multiples of 8, so four neighbours belong to one head.  A thread holds
+// RQ vectors of the row at a time, all requested before the first is used.
+// NORM: 0 none, 1 over all heads at once, 2 per head where one warp holds a head's vectors side by side,
+// 3 per head of any size.
+constexpr int RQ = 8, RQ_THREADS = 256;
+template <class T, int NORM>
+__global__ void __launch_bounds__(RQ_THREADS) k_rows_qkv(RowsAttnArgs a) {
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
   asm volatile("griddepcontrol.wait;" ::: "memory");
   __shared__ float sh[32];
-  extern __shared__ float per_head[];  // [H + G] with head_norm
+  extern __shared__ float per_head[];  // [H + G], NORM 3
   const int64_t m = blockIdx.x;
   const int row = a.rows.tok_row[m];
   const int64_t pos = row_pos0(a.rows, row) + (m - a.rows.start[row]);
   const int64_t slot = a.rows.slot[row];
   const float* p = a.proj + m * a.ldp;
-  const int nq = a.H * a.Dk, nk = a.G * a.Dk, n_v = a.G * a.Dv;
-  float fq = 1.f, fk = 1.f;
-  if (a.q_gain) {
-    float sq = 0.f, sk = 0.f;
-    for (int i = 4 * threadIdx.x; i < nq + nk; i += 4 * blockDim.x) {
-      const float4 v = *(const float4*)(p + i);
-      const float s = v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
-      if (i < nq) sq += s;
-      else sk += s;
+  const int nq = a.H * a.Dk, nk = a.G * a.Dk, total = nq + nk + a.G * a.Dv;
+  const int lanes = a.Dk / 4;
+  float4 v[RQ];
+  auto load = [&](int base) {
+#pragma unroll
+    for (int u = 0; u < RQ; ++u) {
+      const int i = base + 4 * (threadIdx.x + u * RQ_THREADS);
+      v[u] = i < total ? *(const float4*)(p + i) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
+  };
+  load(0);
+  float fq = 1.f, fk = 1.f;
+  if (NORM == 1) {
+    float sq = 0.f, sk = 0.f;
+    auto add = [&](int i, float4 x) {
+      const float s = x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
+      if (i < nq) sq += s;
+      else if (i < nq + nk) sk += s;
+    };
+#pragma unroll
+    for (int u = 0; u < RQ; ++u) add(4 * (threadIdx.x + u * RQ_THREADS), v[u]);
+    for (int i = 4 * (threadIdx.x + RQ * RQ_THREADS); i < nq + nk; i += 4 * RQ_THREADS) add(i, *(const float4*)(p + i));
     fq = 1.f / sqrtf(block_sum(sq, sh) / (float)(a.H * a.d) + a.eps);
     fk = 1.f / sqrtf(block_sum(sk, sh) / (float)(a.G * a.d) + a.eps);
   }
-  if (a.head_norm) {
+  if (NORM == 3) {
     const int lane = threadIdx.x & 31;
-    for (int h = threadIdx.x >> 5; h < a.H + a.G; h += blockDim.x >> 5) {
+    for (int h = threadIdx.x >> 5; h < a.H + a.G; h += RQ_THREADS >> 5) {
       float ss = 0.f;
       for (int i = 4 * lane; i < a.Dk; i += 128) {
-        const float4 v = *(const float4*)(p + h * a.Dk + i);
-        ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+        const float4 x = *(const float4*)(p + h * a.Dk + i);
+        ss += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
       }
       ss = warp_sum(ss);
       if (lane == 0) per_head[h] = 1.f / sqrtf(ss / (float)a.d + a.eps);
@@ -89,28 +105,53 @@ __global__ void __launch_bounds__(256) k_rows_qkv(RowsAttnArgs a) {
   const int half = a.rot / 2;
   const float* ct = a.cos_t + pos * half;
   const float* sn = a.sin_t + pos * half;
-  for (int i = 4 * threadIdx.x; i < nq + nk + n_v; i += 4 * blockDim.x) {
-    float4 v = *(const float4*)(p + i);
-    if (i >= nq + nk) {
-      const int j = i - nq - nk, g = j / a.Dv;
-      st4((T*)a.v_cache + ((slot * a.G + g) * a.Tmax + pos) * a.Dv + (j - g * a.Dv), v);
-      continue;
+  T* const qo = (T*)a.q + m * nq;
+  T* const ko = (T*)a.k_cache + (slot * a.G * a.Tmax + pos) * a.Dk;
+  T* const vo = (T*)a.v_cache + (slot * a.G * a.Tmax + pos) * a.Dv;
+  // head of a column: a shift where the head size is a power of two
+  const int kshift = (a.Dk & (a.Dk - 1)) ? -1 : __ffs(a.Dk) - 1;
+  for (int base = 0; base < total; base += 4 * RQ * RQ_THREADS) {
+    if (base) load(base);
+#pragma unroll
+    for (int u = 0; u < RQ; ++u) {
+      const int i = base + 4 * (threadIdx.x + u * RQ_THREADS);
+      if (base + 4 * u * RQ_THREADS >= total) break;  // uniform over the block
+      float4 x = v[u];
+      if (NORM == 2) {
+        float ss = x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
+#pragma unroll
+        for (int o = 16; o; o >>= 1) {
+          const float t = __shfl_xor_sync(0xffffffffu, ss, o);
+          if (o < lanes) ss += t;
+        }
+        if (i < nq + nk) {
+          const float f = 1.f / sqrtf(ss / (float)a.d + a.eps);
+          x = make_float4(x.x * f, x.y * f, x.z * f, x.w * f);
+        }
+      }
+      if (i >= nq + nk) {
+        if (i < total) {
+          const int j = i - nq - nk, g = j / a.Dv;
+          st4(vo + g * a.Tmax * a.Dv + (j - g * a.Dv), x);
+        }
+      } else {
+        const bool is_q = i < nq;
+        const int j = is_q ? i : i - nq, h = kshift >= 0 ? j >> kshift : j / a.Dk, e = j - h * a.Dk;
+        if (NORM == 1) {
+          const float f = is_q ? fq : fk;
+          const float4 w = *(const float4*)((is_q ? a.q_gain : a.k_gain) + j);
+          x = make_float4(x.x * (f * w.x), x.y * (f * w.y), x.z * (f * w.z), x.w * (f * w.w));
+        } else if (NORM == 3) {
+          const float f = per_head[is_q ? h : a.H + h];
+          x = make_float4(x.x * f, x.y * f, x.z * f, x.w * f);
+        }
+        const int k = e >> 1;
+        if (k < half) x = make_float4(x.x * ct[k] - x.y * sn[k], x.y * ct[k] + x.x * sn[k], x.z, x.w);
+        if (k + 1 < half) x = make_float4(x.x, x.y, x.z * ct[k + 1] - x.w * sn[k + 1], x.w * ct[k + 1] + x.z * sn[k + 1]);
+        if (is_q) st4(qo + i, x);
+        else st4(ko + h * a.Tmax * a.Dk + e, x);
+      }
     }
-    const bool is_q = i < nq;
-    const int j = is_q ? i : i - nq, h = j / a.Dk, e = j - h * a.Dk;
-    if (a.q_gain) {
-      const float f = is_q ? fq : fk;
-      const float4 w = *(const float4*)((is_q ? a.q_gain : a.k_gain) + j);
-      v = make_float4(v.x * (f * w.x), v.y * (f * w.y), v.z * (f * w.z), v.w * (f * w.w));
-    } else if (a.head_norm) {
-      const float f = per_head[is_q ? h : a.H + h];
-      v = make_float4(v.x * f, v.y * f, v.z * f, v.w * f);
-    }
-    const int k = e >> 1;
-    if (k < half) v = make_float4(v.x * ct[k] - v.y * sn[k], v.y * ct[k] + v.x * sn[k], v.z, v.w);
-    if (k + 1 < half) v = make_float4(v.x, v.y, v.z * ct[k + 1] - v.w * sn[k + 1], v.w * ct[k + 1] + v.z * sn[k + 1]);
-    if (is_q) st4((T*)a.q + m * nq + i, v);
-    else st4((T*)a.k_cache + ((slot * a.G + h) * a.Tmax + pos) * a.Dk + e, v);
   }
 }
 
@@ -181,10 +222,16 @@ __global__ void __launch_bounds__(128) k_rows_attn(RowsAttnArgs a) {
 int k_launch_rows_qkv(cg_ctx* c, const RowsAttnArgs& a) {
   if (a.rows.M == 0) return CG_OK;
   if (a.Dk % 8 || a.Dv % 8 || a.ldp % 4) return fail(c, CG_ERR_INVALID, "attention: head sizes must be padded to multiples of 8");
-  const size_t smem = a.head_norm ? (size_t)(a.H + a.G) * 4 : 0;
+  const int lanes = a.Dk / 4;
+  const int norm = a.q_gain ? 1 : !a.head_norm ? 0 : lanes == 2 || lanes == 4 || lanes == 8 || lanes == 16 || lanes == 32 ? 2 : 3;
+  const size_t smem = norm == 3 ? (size_t)(a.H + a.G) * 4 : 0;
   if (smem > 40 * 1024) return fail(c, CG_ERR_UNSUPPORTED, "attention: too many heads");
-  if (a.bf16) CG_CUDA(c, launch_kernel(c, k_rows_qkv<__nv_bfloat16>, dim3((unsigned)a.rows.M), dim3(256), smem, 1, a));
-  else CG_CUDA(c, launch_kernel(c, k_rows_qkv<float>, dim3((unsigned)a.rows.M), dim3(256), smem, 1, a));
+  auto run = [&](auto t) {
+    using T = decltype(t);
+    auto kernel = norm == 0 ? k_rows_qkv<T, 0> : norm == 1 ? k_rows_qkv<T, 1> : norm == 2 ? k_rows_qkv<T, 2> : k_rows_qkv<T, 3>;
+    return launch_kernel(c, kernel, dim3((unsigned)a.rows.M), dim3(RQ_THREADS), smem, 1, a);
+  };
+  CG_CUDA(c, a.bf16 ? run(__nv_bfloat16()) : run(float()));
   CG_LAUNCHED(c);
   return CG_OK;
 }

@@ -43,6 +43,13 @@ def test_layered_workloads_count_looped_layers():
     layered = importlib.import_module("catgrad-rs_b200.layered")
     for name, (cfg_name, batch, prompt, decode) in bench.LAYERED_WORKLOADS.items():
         cfg = getattr(layered, cfg_name)
+        if not cfg.loop:
+            # a layer with another one's weights counts them again
+            own = dataclasses.replace(cfg, layers=[dataclasses.replace(L, weights_of=None) for L in cfg.layers])
+            assert any(L.weights_of is not None for L in cfg.layers)
+            assert bench.layered_step_bytes(own, batch, prompt) == bench.layered_step_bytes(cfg, batch, prompt)
+            assert all(v > 0 for v in bench.layered_step_bytes(cfg, batch, prompt).values())
+            continue
         once = bench.layered_step_bytes(dataclasses.replace(cfg, loop=None), batch, prompt)
         looped = bench.layered_step_bytes(cfg, batch, prompt)
         assert all(looped[k] > once[k] > 0 for k in once if k != "states" or cfg.recurrent)
