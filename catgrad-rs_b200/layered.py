@@ -369,7 +369,7 @@ def regupel_shape(name: str, width: int, heads: int, kv_heads: int, dim: int, wi
     gated attention with a window four times as long; one of those uses another one's weights."""
     def layer(i):
         if i % 4 == 1:
-            m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** 0.5, "mask": {"size": 4 * window},
+            m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "mask": {"size": 4 * window},
                  "rot": {"base": 500000.0, "dims": dim // 2, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
             return LayerSpec("attention", m, ff, SILU, experts, weights_of=1 if i == 5 else None)
         left = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "mask": {"size": window, "keep_first": kept}}
