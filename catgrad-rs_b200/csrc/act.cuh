@@ -23,8 +23,8 @@ __device__ __forceinline__ float gelu_fast(float x) {
 
 // What a feed-forward applies to its projections (cg_act, include/catgrad_cuda.h).  Two projections:
 // ACT_SILU and ACT_GELU gate the second one, ACT_BOUNDED is min(g, limit) sigmoid(1.702 g) (u + 1) with
-// u kept within +-limit.  One projection: ACT_RELU2 is the square of relu.
-enum Act : int { ACT_SILU = 0, ACT_GELU = 1, ACT_BOUNDED = 2, ACT_RELU2 = 3 };
+// u kept within +-limit.  One projection: ACT_RELU2 is the square of relu, ACT_GELU1 gelu.
+enum Act : int { ACT_SILU = 0, ACT_GELU = 1, ACT_BOUNDED = 2, ACT_RELU2 = 3, ACT_GELU1 = 4 };
 __device__ __forceinline__ float bounded_glu(float g, float u, float limit) {
   g = fminf(g, limit);
   u = fminf(fmaxf(u, -limit), limit);
@@ -38,7 +38,29 @@ __device__ __forceinline__ float relu2_f(float x) {
   return x * x;
 }
 
-// What a GEMM stores in bf16: output mode 1 the product itself, 4 the square of its relu, 5 its silu.
-__device__ __forceinline__ float bf16_out(int mode, float v) { return mode == 4 ? relu2_f(v) : mode == 5 ? silu_fast(v) : v; }
+// What a GEMM stores in bf16: output mode 1 the product itself, 4 the square of its relu, 5 its silu, 6 the
+// gelu of its sum with bias[n].
+__device__ __forceinline__ float bf16_out(int mode, float v, const float* bias, int64_t n) {
+  return mode == 4 ? relu2_f(v) : mode == 5 ? silu_fast(v) : mode == 6 ? gelu_fast(v + bias[n]) : v;
+}
+
+// ln(1 + e^x) with a relative error of about 1e-6: with e = e^-|x| and s = e / (2 + e),
+// ln(1 + e) = 2 artanh(s), whose power series in s <= 1 / 3 needs eight terms.
+__device__ __forceinline__ float softplus_f(float x) {
+  const float e = __expf(-fabsf(x)), s = __fdividef(e, 2.f + e), q = s * s;
+  float p = 1.f / 15.f;
+  p = fmaf(p, q, 1.f / 13.f);
+  p = fmaf(p, q, 1.f / 11.f);
+  p = fmaf(p, q, 1.f / 9.f);
+  p = fmaf(p, q, 1.f / 7.f);
+  p = fmaf(p, q, 1.f / 5.f);
+  p = fmaf(p, q, 1.f / 3.f);
+  p = fmaf(p, q, 1.f);
+  return fmaxf(x, 0.f) + 2.f * s * p;
+}
+// tanh-gelu on accurate exponentials
+__device__ __forceinline__ float gelu_exact(float x) {
+  return 0.5f * x * (1.f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
+}
 
 }  // namespace cg

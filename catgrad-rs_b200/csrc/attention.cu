@@ -12,6 +12,7 @@
 // shared-memory buffers, so the loads of tile i+1 overlap the math of tile i; query tiles are
 // scheduled longest first (under the causal mask the last tile of a row has the most keys).
 // (The one-token decode step has its own fused kernel.)
+#include "act.cuh"
 #include "kernels.h"
 #include "mma.cuh"
 
@@ -152,6 +153,7 @@ __global__ void __launch_bounds__(BQ * 2, D <= 64 ? 2 : 1) k_attn_prefill(AttnAr
         float v = s[j][e] * scale;
         if (a.softcap > 0.f) v = a.softcap * tanh_sig(v / a.softcap);
         const bool sees = kpos <= qp && kpos < kv_len && (a.window <= 0 || kpos > qp - a.window || kpos < keep);
+        if (a.bias && sees) v -= a.bias[h * a.ld_bias + (qp - kpos)];
         v = sees ? v : -INFINITY;
         s[j][e] = v;
         mx[e >> 1] = fmaxf(mx[e >> 1], v);
@@ -220,11 +222,17 @@ __global__ void __launch_bounds__(BQ * 2, D <= 64 ? 2 : 1) k_attn_prefill(AttnAr
     float inv = lrow[r] > 0.f ? 1.f / lrow[r] : 0.f;
     if (a.sink) inv = sink_scale(mrow[r], lrow[r], a.sink[h]);
     inv *= a.out_scale;
-    if (a.gate) inv *= 1.f / (1.f + expf(-a.gate[(tok0 + qi) * a.ld_gate + h]));
+    const float* gate = a.gate ? a.gate + (tok0 + qi) * a.ld_gate + (a.wide_gate ? (int64_t)h * D : h) : nullptr;
+    if (gate && !a.wide_gate) inv *= 1.f / (1.f + expf(-*gate));
     __nv_bfloat16* dst = a.out + (tok0 + qi) * (a.ld_out > 0 ? a.ld_out : (int64_t)a.nh * D) + (int64_t)h * D;
 #pragma unroll
     for (int j = 0; j < D / 8; ++j) {
-      __nv_bfloat162 v = __floats2bfloat162_rn(o[j][2 * r] * inv, o[j][2 * r + 1] * inv);
+      float f0 = inv, f1 = inv;
+      if (gate && a.wide_gate) {
+        f0 *= sigmoid_f(gate[j * 8 + cq]);
+        f1 *= sigmoid_f(gate[j * 8 + cq + 1]);
+      }
+      __nv_bfloat162 v = __floats2bfloat162_rn(o[j][2 * r] * f0, o[j][2 * r + 1] * f1);
       *(__nv_bfloat162*)(dst + j * 8 + cq) = v;
     }
   }

@@ -22,6 +22,7 @@
 // roles leave their loops, TMEM is freed and the kernel returns.
 #include <algorithm>
 
+#include "act.cuh"
 #include "kernels.h"
 #include "tc_common.cuh"
 
@@ -32,6 +33,7 @@ namespace {
 using namespace tc;
 
 constexpr int FA_BQ = 128;
+constexpr float LOG2E = 1.4426950408889634f;
 
 struct FaArgs {
   __nv_bfloat16* out;  // [B * S, nh D]
@@ -44,6 +46,9 @@ struct FaArgs {
   const float* sink;   // [nh] or null
   const float* gate;   // [tokens, ld_gate] or null: sigmoid(gate) multiplies a head's output, as out_scale does
   int64_t ld_gate, ld_out;
+  int wide_gate;       // a gate per value instead of one per head
+  const float* bias;   // BIAS: bias[h * ld_bias + distance] is taken off the scores
+  int64_t ld_bias;
   float out_scale;
   RowsDev rows;        // rows of unequal length (rows.rows > 0)
   int32_t* err;
@@ -85,7 +90,10 @@ __device__ __forceinline__ void tmem_ld32(uint32_t taddr, uint32_t* v) {
       : "memory");
 }
 
-template <int D, int FA_BK>
+// BIAS: a number per head and distance is taken off the scores, monotone in the distance, read from a table
+// (neighbouring rows read neighbouring entries).  A row's maximum is then an upper bound: the largest
+// product less the smallest number of the tile.
+template <int D, int FA_BK, bool BIAS>
 __global__ void __launch_bounds__(192, FA_BK == 64 ? 2 : 1)
 k_attn_fa(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
           const __grid_constant__ CUtensorMap map_v, FaArgs p) {
@@ -294,10 +302,17 @@ k_attn_fa(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUt
         }
         if (c + 1 < NCH) asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
       }
+      const float* bias_row = nullptr;  // of this row against the tile's first key
+      if (BIAS) {
+        bias_row = p.bias + h * p.ld_bias + (qpos - k0);
+        const int64_t nearest = lim64 < FA_BK ? lim64 : FA_BK - 1;  // (rows that see no key of the tile have none: lim64 < 0)
+        mx = lim64 < 0 ? -INFINITY : mx * p.scale_log2e - LOG2E * fminf(__ldg(bias_row), __ldg(bias_row - nearest));
+      }
       const float m_new = fmaxf(m, mx);
       const float m_safe = m_new == -INFINITY ? 0.f : m_new;
-      const float corr = fast_exp2((m - m_safe) * p.scale_log2e);  // 0 while m is -inf
-      const float mc = m_safe * p.scale_log2e;
+      const float m_unit = BIAS ? 1.f : p.scale_log2e;             // (with BIAS the maxima are scaled already)
+      const float corr = fast_exp2((m - m_safe) * m_unit);         // 0 while m is -inf
+      const float mc = m_safe * m_unit;
       // the previous tile's P must have been consumed before it is overwritten
       if (j >= 1) {
         ok = mbar_wait(b_p_empty, ((uint32_t)j & 1u) ^ 1u, cta_abort, p.err);
@@ -316,8 +331,13 @@ k_attn_fa(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUt
         uint32_t pk[16];
 #pragma unroll
         for (int i = 0; i < 32; i += 2) {
-          float e0 = fast_exp2(fmaf(__uint_as_float(cur[i]), p.scale_log2e, -mc));
-          float e1 = fast_exp2(fmaf(__uint_as_float(cur[i + 1]), p.scale_log2e, -mc));
+          float t0 = -mc, t1 = -mc;
+          if (BIAS) {
+            t0 = fmaf(__ldg(bias_row - (c * 32 + i)), -LOG2E, t0);
+            t1 = fmaf(__ldg(bias_row - (c * 32 + i + 1)), -LOG2E, t1);
+          }
+          float e0 = fast_exp2(fmaf(__uint_as_float(cur[i]), p.scale_log2e, t0));
+          float e1 = fast_exp2(fmaf(__uint_as_float(cur[i + 1]), p.scale_log2e, t1));
           if (diag) {
             e0 = vis & (1u << i) ? e0 : 0.f;
             e1 = vis & (2u << i) ? e1 : 0.f;
@@ -366,18 +386,23 @@ k_attn_fa(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUt
       float inv = l > 0.f ? 1.f / l : 0.f;
       if (p.sink) {
         // one more term of the denominator, without a value
-        const float mc = m * p.scale_log2e, sk = p.sink[h] * 1.4426950408889634f, top = fmaxf(mc, sk);
+        const float mc = BIAS ? m : m * p.scale_log2e, sk = p.sink[h] * LOG2E, top = fmaxf(mc, sk);
         const float f = fast_exp2(mc - top);
         inv = f / (l * f + fast_exp2(sk - top));
       }
       inv *= p.out_scale;
-      if (p.gate) inv *= 1.f / (1.f + expf(-p.gate[(tok0 + qi) * p.ld_gate + h]));
+      const float* gate = p.gate ? p.gate + (tok0 + qi) * p.ld_gate + (p.wide_gate ? h * D : h) : nullptr;
+      if (gate && !p.wide_gate) inv *= 1.f / (1.f + expf(-*gate));
       __nv_bfloat16* dst = p.out + (tok0 + qi) * p.ld_out + (int64_t)h * D;
 #pragma unroll
       for (int c0 = 0; c0 < D; c0 += 8) {
         uint32_t w[4];
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
+          if (gate && p.wide_gate) {
+            const float2 g = *(const float2*)(gate + c0 + 2 * i);
+            o[c0 + 2 * i] *= sigmoid_f(g.x); o[c0 + 2 * i + 1] *= sigmoid_f(g.y);
+          }
           const __nv_bfloat162 pr = __floats2bfloat162_rn(o[c0 + 2 * i] * inv, o[c0 + 2 * i + 1] * inv);
           w[i] = *(const uint32_t*)&pr;
         }
@@ -394,14 +419,14 @@ k_attn_fa(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUt
   }
 }
 
-template <int D, int FA_BK>
+template <int D, int FA_BK, bool BIAS>
 int launch_fa(cg_ctx* c, const AttnArgs& a) {
   constexpr size_t smem =
       (size_t)(D / 64) * (128 + 4 * FA_BK) * 128 + (size_t)(FA_BK / 64) * 128 * 128 + (FA_BK == 64 ? 0 : 1024) + 160;
   static PerDeviceFlag configured_on;
   bool& configured = configured_on.at(c->core->device);
   if (!configured) {
-    CG_CUDA(c, cudaFuncSetAttribute(k_attn_fa<D, FA_BK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    CG_CUDA(c, cudaFuncSetAttribute(k_attn_fa<D, FA_BK, BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     configured = true;
   }
   CUtensorMap mq, mk, mv;
@@ -419,12 +444,13 @@ int launch_fa(cg_ctx* c, const AttnArgs& a) {
   p.window = a.window > 0 ? a.window : 0;
   p.keep = p.window ? std::max<int64_t>(a.keep_first, 0) : 0;
   p.sink = a.sink;
+  p.wide_gate = a.wide_gate; p.bias = a.bias; p.ld_bias = a.ld_bias;
   p.gate = a.gate; p.ld_gate = a.ld_gate; p.out_scale = a.out_scale;
   p.ld_out = a.ld_out > 0 ? a.ld_out : (int64_t)a.nh * D;
   p.rows = a.rows;
   p.err = c->core->dev_err;
   dim3 grid((unsigned)((a.S + FA_BQ - 1) / FA_BQ), (unsigned)a.nh, (unsigned)(a.rows.rows ? a.rows.rows : a.B));
-  CG_CUDA(c, launch_kernel(c, k_attn_fa<D, FA_BK>, grid, dim3(192), smem, 1, mq, mk, mv, p));
+  CG_CUDA(c, launch_kernel(c, k_attn_fa<D, FA_BK, BIAS>, grid, dim3(192), smem, 1, mq, mk, mv, p));
   CG_LAUNCHED(c);
   return CG_OK;
 }
@@ -434,7 +460,8 @@ int launch_fa(cg_ctx* c, const AttnArgs& a) {
 bool attn_fa_supported(const AttnArgs& a) {
   return (a.d == 64 || a.d == 128) && a.softcap <= 0.f && !a.pos_dev && a.S >= 64 &&
          (a.rows.rows ? a.rows.M : a.B * a.S) < 2147483647ll && a.B * a.nkv * a.Tmax < 2147483647ll && ((uintptr_t)a.q % 16) == 0 &&
-         ((uintptr_t)a.k_cache % 16) == 0 && ((uintptr_t)a.v_cache % 16) == 0 && a.kv_ld % 8 == 0 && ((uintptr_t)a.out % 16) == 0 && a.ld_out % 8 == 0;
+         ((uintptr_t)a.k_cache % 16) == 0 && ((uintptr_t)a.v_cache % 16) == 0 && a.kv_ld % 8 == 0 && ((uintptr_t)a.out % 16) == 0 && a.ld_out % 8 == 0 &&
+         (!a.wide_gate || (((uintptr_t)a.gate % 8) == 0 && a.ld_gate % 2 == 0));
 }
 
 int k_launch_attn_fa(cg_ctx* c, const AttnArgs& a) {
@@ -442,8 +469,12 @@ int k_launch_attn_fa(cg_ctx* c, const AttnArgs& a) {
   // 64-key tiles: two CTAs per SM.  Head size 64 gains from it (8 x 1024 tokens, 64 heads: 380 -> 315 us,
   // with a window of 128 225 -> 165 us), head size 128 does not (242 -> 264 us).
   const bool k64 = c->opt_fa == 2 || a.d == 64;
-  if (a.d == 64) return k64 ? launch_fa<64, 64>(c, a) : launch_fa<64, 128>(c, a);
-  return k64 ? launch_fa<128, 64>(c, a) : launch_fa<128, 128>(c, a);
+  if (a.bias) {
+    if (a.d == 64) return launch_fa<64, 64, true>(c, a);
+    return k64 ? launch_fa<128, 64, true>(c, a) : launch_fa<128, 128, true>(c, a);
+  }
+  if (a.d == 64) return k64 ? launch_fa<64, 64, false>(c, a) : launch_fa<64, 128, false>(c, a);
+  return k64 ? launch_fa<128, 64, false>(c, a) : launch_fa<128, 128, false>(c, a);
 }
 
 }  // namespace cg

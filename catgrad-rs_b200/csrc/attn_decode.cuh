@@ -173,6 +173,7 @@ __device__ __forceinline__ void attn_dec_item(const AttnDecArgs& a, float scale,
     }
     // neighbouring components (2 j, 2 j + 1) of the first rot_dims turn together
     const int rh = a.rot_dims / 2;
+    const float temp = a.q_temp ? a.q_temp[pos] : 1.f;
     const float* ct = a.cos_t + pos * rh;
     const float* st = a.sin_t + pos * rh;
     for (int i = tid; i < 16 * half; i += 128) {
@@ -192,6 +193,7 @@ __device__ __forceinline__ void attn_dec_item(const AttnDecArgs& a, float scale,
           x1 = cs * t - sn * x2;
           x2 = cs * x2 + sn * t;
         }
+        x1 *= temp; x2 *= temp;
       }
       *(__nv_bfloat162*)(qt + h * LD + 2 * j) = __floats2bfloat162_rn(x1, x2);
     }
@@ -278,6 +280,9 @@ __device__ __forceinline__ void attn_dec_item(const AttnDecArgs& a, float scale,
   // A thread owns head r = lane / 4 (rows 8..15 of the MMA tile are padding) and, per 8-key
   // or 8-column tile, the two columns 2 * (lane % 4) + {0, 1}.
   const int hr = lane >> 2, cq = (lane & 3) * 2;
+  const float* bias = nullptr;
+  if constexpr (Env::kRows)
+    if (a.bias && hr < rep) bias = a.bias + (int64_t)(kvh * rep + hr) * a.ld_bias;
   float m = -INFINITY, l = 0.f;
   float o[NT][4];
 #pragma unroll
@@ -341,6 +346,11 @@ __device__ __forceinline__ void attn_dec_item(const AttnDecArgs& a, float scale,
         float v = s[j][e] * scale;
         if (a.softcap > 0.f) v = a.softcap * attn_tanh_sig(v / a.softcap);
         const bool keep = cbase + j * 8 + cq + e < limit;
+        if constexpr (Env::kRows)
+          if (bias && keep && !do_new) {   // (at the new token itself the distance is 0, and so is what is taken off)
+            const int64_t i = cbase + j * 8 + cq + e;
+            v -= bias[pos - (i < kf ? i : i - kf + lo)];
+          }
         v = keep ? v : -INFINITY;
         s[j][e] = v;
         mx = fmaxf(mx, v);
@@ -406,10 +416,10 @@ __device__ __forceinline__ void attn_dec_item(const AttnDecArgs& a, float scale,
   float* part_o = part_ml + 2 * MAX_REP;       // [MAX_REP][D]
   const int S = a.splits;
   // the merged output oo over the merged sum ll of exp(score - mm), which the sink joins, gated and scaled
-  auto finished = [&](int r, float mm, float ll, float oo) {
+  auto finished = [&](int r, int e, float mm, float ll, float oo) {
     if constexpr (Env::kRows) {
       oo *= a.out_scale;
-      if (a.gate) oo *= 1.f / (1.f + __expf(-__ldcg(a.gate + b * a.ld_gate + kvh * rep + r)));
+      if (a.gate) oo *= 1.f / (1.f + __expf(-__ldcg(a.gate + b * a.ld_gate + (a.wide_gate ? (kvh * rep + r) * D + e : kvh * rep + r))));
       if (a.sink) {
         const float sk = a.sink[kvh * rep + r], top = fmaxf(mm, sk);
         const float f = __expf(mm - top);
@@ -483,7 +493,7 @@ __device__ __forceinline__ void attn_dec_item(const AttnDecArgs& a, float scale,
         ll += ls[s] * f;
         oo += os[s] * f;
       }
-      a.out[b * ld_out + (kvh * rep + r) * (int64_t)D + (i - r * D)] = __float2bfloat16_rn(finished(r, mm, ll, oo));
+      a.out[b * ld_out + (kvh * rep + r) * (int64_t)D + (i - r * D)] = __float2bfloat16_rn(finished(r, i - r * D, mm, ll, oo));
     }
     return;
   }
@@ -492,7 +502,7 @@ __device__ __forceinline__ void attn_dec_item(const AttnDecArgs& a, float scale,
     for (int i = tid; i < rep * D; i += 128) {
       const int r = i / D, e = i - r * D;
       const float ll = part_ml[2 * r + 1];
-      a.out[b * ld_out + (kvh * rep + r) * (int64_t)D + e] = __float2bfloat16_rn(finished(r, part_ml[2 * r], ll, part_o[i]));
+      a.out[b * ld_out + (kvh * rep + r) * (int64_t)D + e] = __float2bfloat16_rn(finished(r, e, part_ml[2 * r], ll, part_o[i]));
     }
     env.sync_cta();  // the partials are read: the next item of a resident CTA may reuse the space
     return;
@@ -523,7 +533,7 @@ __device__ __forceinline__ void attn_dec_item(const AttnDecArgs& a, float scale,
       ll += ls[s] * f;
       oo += os[s] * f;
     }
-    a.out[b * ld_out + (kvh * rep + r) * (int64_t)D + (i - r * D)] = __float2bfloat16_rn(finished(r, mm, ll, oo));
+    a.out[b * ld_out + (kvh * rep + r) * (int64_t)D + (i - r * D)] = __float2bfloat16_rn(finished(r, i - r * D, mm, ll, oo));
   }
   // nobody leaves while a peer may still read its shared memory
   env.sync_group();

@@ -7,7 +7,8 @@
 //   attention          [kv heads, max_seq, head size] keys and values
 //   latent attention   [max_seq, Lw] cached rows (normed latent, rotated key part)
 //   delta, ssd         an f32 matrix per head and the last inputs of the convolutions
-//   lightning          an f32 matrix per head
+//   lightning, gla     an f32 matrix per head
+//   lru                an f32 value per channel and the last inputs of the convolution
 // (of two mixers side by side, both their parts).
 // Nothing is cleared when a slot is reused: a row whose first position is 0 starts from zeros.
 // Batches are rows of unequal length, packed token after token; every kernel finds a token's row,
@@ -54,8 +55,12 @@ struct MixedLayer {
   // experts, stacked
   cg_tensor *router = nullptr, *correction = nullptr, *we_gate = nullptr, *we_up = nullptr, *we_down = nullptr;
   int64_t Fd = 0;       // padded width of w_gu: the dense feed-forward or the shared expert, 0 = neither
+  cg_tensor *up_bias = nullptr, *down_bias = nullptr;
+  // sublayers side by side: norms of two mixers' results, weights of the depth average, the token's input
+  cg_tensor *out_gain = nullptr, *average = nullptr, *side_gate = nullptr, *side_proj = nullptr, *side_norm = nullptr;
+  int64_t ff_col = -1;  // >= 0: the feed-forward's units are columns of the mixer's output, w_down part of w_o
   // attention
-  cg_tensor *q_gain = nullptr, *k_gain = nullptr, *sink = nullptr;
+  cg_tensor *q_gain = nullptr, *k_gain = nullptr, *sink = nullptr, *q_temp = nullptr, *bias = nullptr;
   int Dk = 0, Dv = 0;   // columns a key and a value head take
   // latent attention
   cg_tensor *c_gain = nullptr, *uk = nullptr, *uv = nullptr, *w_kv = nullptr, *cos_t = nullptr, *sin_t = nullptr;
@@ -63,14 +68,19 @@ struct MixedLayer {
   int dkv_off = 0, Dq = 0;
   // recurrences
   cg_tensor *conv_w = nullptr, *conv_b = nullptr, *a_log = nullptr, *dt_bias = nullptr, *dskip = nullptr, *norm = nullptr,
-            *log_decay = nullptr;
+            *log_decay = nullptr, *coef = nullptr, *w_a2 = nullptr, *w_g2 = nullptr;
+  cg_tensor *ra = nullptr, *ri = nullptr, *ra_b = nullptr, *ri_b = nullptr, *xb = nullptr, *yb = nullptr;  // lru
+  int zs = 0, a1_off = 0, g1_off = 0, a_rank = 0, g_rank = 0, x_off = 0;
   bool chunked = false;  // prompts run on the tensor cores, 64 tokens at a time
   int H = 0, KH = 0, dk = 0, dv = 0, dvs = 0, C = 0, gate_off = 0, small_off = 0, q_off = 0, k_off = 0, v_off = 0, qs = 0, vs = 0;
 
-  bool recurrent() const { return k.mixer == CG_MIX_DELTA || k.mixer == CG_MIX_SSD || k.mixer == CG_MIX_LIGHTNING; }
+  bool lru() const { return k.mixer == CG_MIX_LRU; }
+  bool key_decay() const { return k.mixer == CG_MIX_CHANNEL_DELTA || k.mixer == CG_MIX_GLA; }
+  bool delta() const { return k.mixer == CG_MIX_DELTA || k.mixer == CG_MIX_CHANNEL_DELTA; }
+  bool recurrent() const { return delta() || lru() || k.mixer == CG_MIX_SSD || k.mixer == CG_MIX_LIGHTNING || k.mixer == CG_MIX_GLA; }
   float out_scale() const { return k.out_scale != 0. ? (float)k.out_scale : 1.f; }
   int64_t in_width() const { return Np + (beside ? beside->Np : 0); }
-  int64_t out_width() const { return Ko + (beside ? beside->Ko : 0); }
+  int64_t out_width() const { return Ko + (beside ? beside->Ko : 0) + (ff_col >= 0 ? Fd : 0); }
 };
 
 struct MixedRun {
@@ -88,6 +98,7 @@ struct MixedModel {
   bool loop = false;        // passes start from w_loop
   bool f32 = false;
   bool sandwich = false;    // norms behind the sublayers too (k_row_update); else streams (k_stream_update)
+  bool parallel = false;    // the sublayers of a layer run side by side (walk_parallel)
   bool recurrent = false;   // some layer has a state that cannot go back
   int streams = 1;
   float embed_scale = 1.f;
@@ -105,6 +116,9 @@ struct MixedModel {
   cg_tensor *x = nullptr, *xn = nullptr, *xcat = nullptr, *y = nullptr, *proj = nullptr, *cv = nullptr, *gl = nullptr, *co = nullptr,
             *ro = nullptr, *att = nullptr, *hact = nullptr, *gu = nullptr, *q = nullptr, *cpk = nullptr, *tok = nullptr, *xw = nullptr,
             *qkv = nullptr, *rn = nullptr, *tinv = nullptr, *kv = nullptr, *lat = nullptr;
+  cg_tensor *z = nullptr, *low_gate = nullptr, *u = nullptr, *lru_a = nullptr, *lru_b = nullptr, *y2 = nullptr, *depth = nullptr,
+            *side_z = nullptr, *side_h = nullptr, *side_embed = nullptr;
+  int64_t side_p = 0;   // padded width of a layer's token input
   // experts: (token, expert) pairs
   cg_tensor *m_logits = nullptr, *m_ids = nullptr, *m_wts = nullptr, *m_pos = nullptr, *m_tiles = nullptr, *m_xg = nullptr, *m_h = nullptr,
             *m_y = nullptr;
@@ -184,6 +198,24 @@ int coefficients(cg_decoder* D, const std::string& name, int64_t n, cg_tensor** 
   return k_launch_affine(D->c, (float*)(*out)->data(), n, 1.f, 1.f);
 }
 
+// a parameter's values on the host, and the other way round
+int download(cg_decoder* D, const std::string& name, int64_t n, std::vector<float>* out) {
+  Hold w;
+  CG_TRY(norm_weight(D, name, n, &w.t));
+  out->resize((size_t)n);
+  CG_CUDA(D->c, cudaMemcpyAsync(out->data(), w.t->data(), (size_t)n * 4, cudaMemcpyDeviceToHost, D->c->core->stream));
+  CG_CUDA(D->c, cudaStreamSynchronize(D->c->core->stream));
+  return CG_OK;
+}
+int upload(cg_decoder* D, const std::vector<float>& v, cg_tensor** out) {
+  CG_TRY(new2(D->c, ST_F32, 1, (int64_t)v.size(), out, false));
+  CG_CUDA(D->c, cudaMemcpyAsync((*out)->data(), v.data(), v.size() * 4, cudaMemcpyHostToDevice, D->c->core->stream));
+  CG_CUDA(D->c, cudaStreamSynchronize(D->c->core->stream));
+  return CG_OK;
+}
+// entries before and behind a head's distance biases, which kernels may read for keys and rows that do not exist
+constexpr int64_t BIAS_PAD = 256;
+
 int rope_tables(cg_decoder* D, const MixedLayer& L, cg_tensor** cos_t, cg_tensor** sin_t) {
   const int64_t half = std::max(L.k.rot_dim / 2, 1);
   CG_TRY(new2(D->c, ST_F32, D->cfg.max_seq, half, cos_t));
@@ -229,13 +261,30 @@ int finalize_attention(cg_decoder* D, MixedLayer& L, const std::string& mx) {
   L.Dk = Dp ? Dp : (int)up8(d);
   L.Dv = L.Do = Dp ? Dp : (int)up8(dv);
   L.gate_off = (int)((H + G) * L.Dk + G * L.Dv);
-  L.Np = up8(L.gate_off + (k.gate ? H : 0));
+  L.Np = up8(L.gate_off + (k.gate == 2 ? H * L.Dv : k.gate ? H : 0));
   L.Ko = H * L.Dv;
   CG_TRY(new2(c, st, L.Np, X.Wp, &L.w_in));
   CG_TRY(place_heads(D, mx + "q", k, H, d, L.Dk, L.w_in, 0));
   CG_TRY(place_heads(D, mx + "k", k, G, d, L.Dk, L.w_in, H * L.Dk));
   for (int64_t g = 0; g < G; ++g) CG_TRY(place(D, mx + "v", G * dv, W, g * dv, dv, 0, W, L.w_in, (H + G) * L.Dk + g * L.Dv, 0));
-  if (k.gate) CG_TRY(place_all(D, mx + "g", H, W, L.w_in, L.gate_off));
+  if (k.gate == 1) CG_TRY(place_all(D, mx + "g", H, W, L.w_in, L.gate_off));
+  if (k.gate == 2)
+    for (int64_t h = 0; h < H; ++h) CG_TRY(place(D, mx + "g", H * dv, W, h * dv, dv, 0, W, L.w_in, L.gate_off + h * L.Dv, 0));
+  if (k.q_temp_every > 0) {
+    std::vector<float> t((size_t)D->cfg.max_seq);
+    for (size_t p = 0; p < t.size(); ++p) t[p] = (float)(1.0 + k.q_temp_coef * std::log(std::floor((double)(p + 1) / k.q_temp_every) + 1.0));
+    CG_TRY(upload(D, t, &L.q_temp));
+  }
+  if (k.dist_bias) {
+    std::vector<float> r1, r2;
+    CG_TRY(download(D, mx + "r1", H, &r1));
+    CG_TRY(download(D, mx + "r2", H, &r2));
+    const int64_t T = D->cfg.max_seq, ld = T + 2 * BIAS_PAD;
+    std::vector<float> t((size_t)(H * ld), 0.f);
+    for (int64_t h = 0; h < H; ++h)
+      for (int64_t x = 0; x < T + BIAS_PAD; ++x) t[(size_t)(h * ld + BIAS_PAD + x)] = (float)((double)r1[h] * std::log1p((double)r2[h] * (double)x));
+    CG_TRY(upload(D, t, &L.bias));
+  }
   CG_TRY(new2(c, st, X.Wp, L.Ko, &L.w_o));
   for (int64_t h = 0; h < H; ++h) CG_TRY(place(D, mx + "o", W, H * dv, 0, W, h * dv, dv, L.w_o, 0, h * L.Dv));
   if (k.qk_norm == 1) {
@@ -260,7 +309,7 @@ int finalize_experts(cg_decoder* D, MixedLayer& L, const std::string& ff) {
   CG_TRY(new2(D->c, X.act_storage(), E, X.Wp, &L.router));
   CG_TRY(place_all(D, ff + "router", E, W, L.router, 0));
   if (L.k.correction) CG_TRY(norm_weight(D, ff + "correction", E, &L.correction));
-  CG_TRY(stack_experts(D, ff, "gate", E, F, W, L.Fp, X.Wp, &L.we_gate));
+  if (L.k.act != CG_ACT_RELU2) CG_TRY(stack_experts(D, ff, "gate", E, F, W, L.Fp, X.Wp, &L.we_gate));
   CG_TRY(stack_experts(D, ff, "up", E, F, W, L.Fp, X.Wp, &L.we_up));
   return stack_experts(D, ff, "down", E, W, F, X.Wp, L.Fp, &L.we_down);
 }
@@ -396,16 +445,135 @@ int finalize_recurrent(cg_decoder* D, MixedLayer& L, const std::string& mx) {
   return place_all(D, mx + "o", W, inner, L.w_o, 0);
 }
 
+// rows of the first factor of a low-rank projection, as many as its tensor has
+int low_rank_of(cg_decoder* D, const std::string& name, int* rank) {
+  cg_tensor* w = nullptr;
+  CG_TRY(get_param(D, name, &w));
+  if (w->rank != 2 || w->dims[0] < 1 || w->dims[0] > 4096) return fail(D->c, CG_ERR_SHAPE, "decoder: " + name + " has an unexpected shape");
+  *rank = (int)w->dims[0];
+  return CG_OK;
+}
+
+// Decays per key channel: z = W_a2 (W_a1 h), its heads zs columns apart, ln g = -coef softplus(sign (z + bias)).
+int finalize_key_decay(cg_decoder* D, MixedLayer& L, const std::string& mx) {
+  cg_ctx* c = D->c;
+  MixedModel& X = *D->mixed;
+  const cg_layer_config& k = L.k;
+  const bool delta = L.delta();
+  const int64_t W = D->H, H = k.heads, KH = delta ? k.kv_heads : H, d = k.dim, dv = k.vdim;
+  const int st = X.act_storage();
+  L.H = (int)H; L.KH = (int)KH;
+  L.dk = k.dim; L.dv = k.vdim;
+  L.dvs = (int)up8(dv);
+  L.zs = (int)up16(d);
+  // without convolutions the projection itself is the chunk kernels' operand: heads as far apart as they read them
+  L.qs = delta ? L.dk : L.zs;
+  L.vs = delta ? L.dv : L.dvs;
+  L.q_off = 0; L.k_off = (int)(KH * L.qs); L.v_off = 2 * L.k_off;
+  L.C = L.v_off + (int)(H * L.vs);
+  L.chunked = false;
+  int ra = 0, rg = 0;
+  CG_TRY(low_rank_of(D, mx + "a1", &ra));
+  if (delta) CG_TRY(low_rank_of(D, mx + "g1", &rg));
+  L.a_rank = (int)up8(ra); L.g_rank = (int)up8(rg);
+  L.gate_off = (int)up8(L.C);
+  L.a1_off = (int)up8(L.gate_off + (delta ? 0 : H * dv));
+  L.g1_off = L.a1_off + L.a_rank;
+  L.small_off = L.g1_off + L.g_rank;
+  L.Np = up8(L.small_off + (delta ? H : 0));
+  CG_TRY(new2(c, st, L.Np, X.Wp, &L.w_in));
+  for (int64_t h = 0; h < KH; ++h) {
+    CG_TRY(place(D, mx + "q", KH * d, W, h * d, d, 0, W, L.w_in, L.q_off + h * L.qs, 0));
+    CG_TRY(place(D, mx + "k", KH * d, W, h * d, d, 0, W, L.w_in, L.k_off + h * L.qs, 0));
+  }
+  for (int64_t h = 0; h < H; ++h) CG_TRY(place(D, mx + "v", H * dv, W, h * dv, dv, 0, W, L.w_in, L.v_off + h * L.vs, 0));
+  CG_TRY(place_all(D, mx + "a1", ra, W, L.w_in, L.a1_off));
+  CG_TRY(new2(c, st, H * L.zs, L.a_rank, &L.w_a2));
+  for (int64_t h = 0; h < H; ++h) CG_TRY(place(D, mx + "a2", H * d, ra, h * d, d, 0, ra, L.w_a2, h * L.zs, 0));
+  CG_TRY(head_gains(D, mx + (delta ? "dt_bias" : "a2.b"), H, d, L.zs, &L.dt_bias));
+  CG_TRY(gains(D, mx + "norm", dv, &L.norm, L.out_scale()));
+  std::vector<float> f((size_t)H, (float)(1.0 / k.tau));
+  if (delta) {
+    CG_TRY(download(D, mx + "A_log", H, &f));
+    for (float& x : f) x = (float)std::exp((double)x);
+    CG_TRY(place_all(D, mx + "b", H, W, L.w_in, L.small_off));
+    CG_TRY(place_all(D, mx + "g1", rg, W, L.w_in, L.g1_off));
+    CG_TRY(new2(c, st, H * dv, L.g_rank, &L.w_g2));
+    CG_TRY(place_all(D, mx + "g2", H * dv, rg, L.w_g2, 0));
+    CG_TRY(new2(c, ST_F32, L.C, k.conv, &L.conv_w, false));
+    CG_TRY(place_all(D, mx + "q.conv", KH * d, k.conv, L.conv_w, L.q_off));
+    CG_TRY(place_all(D, mx + "k.conv", KH * d, k.conv, L.conv_w, L.k_off));
+    CG_TRY(place_all(D, mx + "v.conv", H * dv, k.conv, L.conv_w, L.v_off));
+  } else {
+    CG_TRY(place_all(D, mx + "g", H * dv, W, L.w_in, L.gate_off));
+  }
+  CG_TRY(upload(D, f, &L.coef));
+  L.Do = L.dv;
+  L.Ko = up8(H * dv);
+  CG_TRY(new2(c, st, X.Wp, L.Ko, &L.w_o));
+  return place_all(D, mx + "o", W, H * dv, L.w_o, 0);
+}
+
+// [blocks, n, n] as [blocks n, n] in the activations' type
+int block_diagonal(cg_decoder* D, const std::string& name, int64_t blocks, int64_t n, cg_tensor** out) {
+  cg_ctx* c = D->c;
+  cg_tensor* w = nullptr;
+  CG_TRY(get_param(D, name, &w));
+  if (w->rank != 3 || w->dims[0] != blocks || w->dims[1] != n || w->dims[2] != n)
+    return fail(c, CG_ERR_SHAPE, "decoder: " + name + " has an unexpected shape");
+  Hold h;
+  const int st = D->mixed->act_storage();
+  if (st == ST_BF16) CG_TRY(cg_to_bf16(c, w, &h.t));
+  else CG_TRY(as_contiguous_f32(c, w, &h.t));
+  CG_TRY(new2(c, st, blocks * n, n, out, false));
+  CG_CUDA(c, cudaMemcpyAsync((*out)->data(), h.t->data(), (size_t)(blocks * n * n) * storage_bytes(st), cudaMemcpyDeviceToDevice, c->core->stream));
+  return CG_OK;
+}
+
+int finalize_lru(cg_decoder* D, MixedLayer& L, const std::string& mx) {
+  cg_ctx* c = D->c;
+  MixedModel& X = *D->mixed;
+  const int64_t W = D->H, B = L.k.heads, n = L.k.vdim, C = B * n;
+  const int st = X.act_storage();
+  L.C = (int)C;
+  L.H = (int)B; L.dv = L.dvs = (int)n;
+  L.x_off = (int)up8(C);
+  L.Np = up8(L.x_off + C);
+  L.Ko = up8(C);
+  L.Do = (int)n;
+  CG_TRY(new2(c, st, L.Np, X.Wp, &L.w_in));
+  CG_TRY(place_all(D, mx + "y", C, W, L.w_in, 0));
+  CG_TRY(place_all(D, mx + "x", C, W, L.w_in, L.x_off));
+  CG_TRY(gains(D, mx + "y.b", C, &L.yb));
+  CG_TRY(gains(D, mx + "x.b", C, &L.xb));
+  CG_TRY(f32_matrix(D, mx + "conv", C, L.k.conv, &L.conv_w));
+  CG_TRY(gains(D, mx + "conv.b", C, &L.conv_b));
+  CG_TRY(block_diagonal(D, mx + "ra", B, n, &L.ra));
+  CG_TRY(block_diagonal(D, mx + "ri", B, n, &L.ri));
+  CG_TRY(gains(D, mx + "ra.b", C, &L.ra_b));
+  CG_TRY(gains(D, mx + "ri.b", C, &L.ri_b));
+  std::vector<float> f;
+  CG_TRY(download(D, mx + "lam", C, &f));
+  for (float& x : f) x = (float)(-8.0 * (std::max((double)x, 0.0) + std::log1p(std::exp(-std::fabs((double)x)))));
+  CG_TRY(upload(D, f, &L.coef));
+  CG_TRY(new2(c, st, X.Wp, L.Ko, &L.w_o));
+  return place_all(D, mx + "o", W, C, L.w_o, 0);
+}
+
 int finalize_mixer(cg_decoder* D, MixedLayer& L, const std::string& mx) {
   switch (L.k.mixer) {
     case CG_MIX_ATTENTION: return finalize_attention(D, L, mx);
     case CG_MIX_LATENT: return finalize_latent(D, L, mx);
     case CG_MIX_LIGHTNING: return finalize_lightning(D, L, mx);
+    case CG_MIX_CHANNEL_DELTA:
+    case CG_MIX_GLA: return finalize_key_decay(D, L, mx);
+    case CG_MIX_LRU: return finalize_lru(D, L, mx);
     default: return finalize_recurrent(D, L, mx);
   }
 }
 
-// two mixers' projections become one matrix, and their output projections one whose rows span both
+// two mixers' projections become one matrix, and their output projections one whose rows span both (unless each
+// result has a norm of its own)
 int finalize_beside(cg_decoder* D, MixedLayer& L, const std::string& mx) {
   cg_ctx* c = D->c;
   MixedModel& X = *D->mixed;
@@ -416,20 +584,24 @@ int finalize_beside(cg_decoder* D, MixedLayer& L, const std::string& mx) {
   R.out_col = L.Ko;
   Hold in, out;
   CG_TRY(new2(c, X.act_storage(), L.in_width(), X.Wp, &in.t));
-  CG_TRY(new2(c, X.act_storage(), X.Wp, L.out_width(), &out.t));
+  if (!L.k.out_norm) CG_TRY(new2(c, X.act_storage(), X.Wp, L.out_width(), &out.t));
   const size_t es = storage_bytes(X.act_storage());
   for (MixedLayer* m : {&L, &R}) {
     CG_CUDA(c, cudaMemcpyAsync((char*)in.t->data() + (size_t)(m->in_row * X.Wp) * es, m->w_in->data(), (size_t)(m->Np * X.Wp) * es,
                                cudaMemcpyDeviceToDevice, c->core->stream));
-    CG_CUDA(c, cudaMemcpy2DAsync((char*)out.t->data() + (size_t)m->out_col * es, (size_t)L.out_width() * es, m->w_o->data(), (size_t)m->Ko * es,
+    if (!L.k.out_norm) CG_CUDA(c, cudaMemcpy2DAsync((char*)out.t->data() + (size_t)m->out_col * es, (size_t)L.out_width() * es, m->w_o->data(), (size_t)m->Ko * es,
                                  (size_t)m->Ko * es, (size_t)X.Wp, cudaMemcpyDeviceToDevice, c->core->stream));
     drop(m->w_in);
-    drop(m->w_o);
+    if (!L.k.out_norm) drop(m->w_o);
   }
   L.w_in = in.take();
-  L.w_o = out.take();
+  if (!L.k.out_norm) L.w_o = out.take();
   R.w_in = L.w_in;
   R.w_in->rc++;
+  if (L.k.out_norm) {
+    CG_TRY(gains(D, mx + "left.out", D->H, &L.out_gain, 0.5f));
+    CG_TRY(gains(D, mx + "right.out", D->H, &R.out_gain, 0.5f));
+  }
   return CG_OK;
 }
 
@@ -443,13 +615,20 @@ int ensure_mixed(cg_decoder* D, int64_t M) {
   cg_ctx* c = D->c;
   forget_graph(D);  // it holds the old buffers
   int64_t np = 0, cc = 0, hh = 0, inner = 0, ko = 0, fp = 0, qw = 0, lw = 0, qkv = 0, kh = 0, top = 0, experts = 0, fe = 0;
+  int64_t zw = 0, gw = 0, lru = 0;
   auto count_mixer = [&](const MixedLayer& L) {
     if (L.k.mixer == CG_MIX_ATTENTION) {
       qw = std::max<int64_t>(qw, (int64_t)L.k.heads * L.Dk);
     } else if (L.k.mixer == CG_MIX_LATENT) {
       qw = std::max<int64_t>(qw, (int64_t)L.k.heads * L.Dq);
       lw = std::max(lw, L.Lw);
+    } else if (L.lru()) {
+      lru = std::max<int64_t>(lru, L.C);
     } else {
+      if (L.key_decay()) {
+        zw = std::max<int64_t>(zw, (int64_t)L.H * L.zs);
+        if (L.w_g2) gw = std::max<int64_t>(gw, (int64_t)L.H * L.dv);
+      }
       cc = std::max<int64_t>(cc, up8(L.C));
       hh = std::max<int64_t>(hh, L.H);
       inner = std::max<int64_t>(inner, (int64_t)L.H * L.dvs);
@@ -477,6 +656,21 @@ int ensure_mixed(cg_decoder* D, int64_t M) {
   CG_TRY(new2(c, st, M, X.Wp, &X.xn));
   CG_TRY(new2(c, ST_F32, M, X.Wp, &X.y));
   if (X.loop) CG_TRY(new2(c, st, M, 2 * X.Wp, &X.xcat));
+  if (X.parallel) {
+    CG_TRY(new2(c, ST_F32, 2 * M, X.Wp, &X.y2));
+    if (D->cfg.depth_average) CG_TRY(new2(c, ST_F32, (int64_t)(X.layers.size() + 1) * M, X.Wp, &X.depth));
+    if (X.side_p) {
+      CG_TRY(new2(c, ST_F32, M, X.side_p, &X.side_z));
+      CG_TRY(new2(c, st, M, X.side_p, &X.side_h));
+    }
+  }
+  if (zw) CG_TRY(new2(c, ST_F32, M, zw, &X.z));
+  if (gw) CG_TRY(new2(c, ST_F32, M, gw, &X.low_gate));
+  if (lru) {
+    CG_TRY(new2(c, st, M, lru, &X.u));
+    CG_TRY(new2(c, ST_F32, M, lru, &X.lru_a));
+    CG_TRY(new2(c, ST_F32, M, lru, &X.lru_b));
+  }
   CG_TRY(new2(c, ST_F32, M, np, &X.proj));
   CG_TRY(new2(c, st, M, ko, &X.att));
   if (fp) {
@@ -526,9 +720,9 @@ int ensure_mixed(cg_decoder* D, int64_t M) {
 }
 
 // out[M, N] = x[M, K] w[row0 .. row0 + N, K]^T; out_mode (of the GEMMs) 0 f32 or, only in a bf16 context,
-// 1 bf16, 4 bf16 of the square of relu
+// 1 bf16, 4 bf16 of the square of relu, 6 bf16 of gelu(product + bias)
 int lin(cg_decoder* D, const void* x, int64_t ldx, int64_t M, const cg_tensor* w, int64_t row0, int64_t N, void* out, int64_t ldo,
-        int out_mode = 0) {
+        int out_mode = 0, const float* bias = nullptr) {
   cg_ctx* c = D->c;
   const int64_t K = w->dims[1];
   if (D->mixed->f32)
@@ -538,15 +732,21 @@ int lin(cg_decoder* D, const void* x, int64_t ldx, int64_t M, const cg_tensor* w
   if (gemm_dec_supported(M, K)) {
     DecGemm g;
     g.x = xb; g.ldx = ldx; g.w = wb; g.ldw = K; g.w_rows = N;
-    g.out = out; g.ldo = ldo; g.residual = nullptr; g.out_mode = out_mode;
+    g.out = out; g.ldo = ldo; g.residual = bias; g.out_mode = out_mode;
     g.push = nullptr; g.dual = 0; g.act = 0;
     g.M = M; g.N = N; g.K = K;
     return gemm_dec(c, g);
   }
   const int splits = gemm_tc_pick_splits(M, N, K);
   float* ws = (int64_t)splits * M * N <= D->splitk_floats ? (float*)D->splitk->data() : nullptr;
-  return gemm_tc(c, xb, ldx, wb, K, out, ldo, nullptr, M, N, K, out_mode, splits, ws);
+  return gemm_tc(c, xb, ldx, wb, K, out, ldo, bias, M, N, K, out_mode, splits, ws);
 }
+
+// Rows of a matrix some columns wide: where the first starts, and from one to the next.
+struct Rows {
+  void* p = nullptr;
+  int64_t ld = 0;
+};
 
 // hact = act(x gate^T) * (x up^T)
 int glu(cg_decoder* D, const MixedLayer& L, const void* x, int64_t M) {
@@ -570,10 +770,21 @@ int glu(cg_decoder* D, const MixedLayer& L, const void* x, int64_t M) {
   return gemm_tc_pair(c, xb, K, w, K, (__nv_bfloat16*)X.hact->data(), F, M, F, K, L.k.act);
 }
 
-// y = the dense feed-forward or the shared expert of the rows xn
+// units = gelu(up h + b) of the rows h = xn
+int gelu_units(cg_decoder* D, const MixedLayer& L, int64_t M, Rows units) {
+  MixedModel& X = *D->mixed;
+  const float* bias = (const float*)L.up_bias->data();
+  CG_TRY(lin(D, X.xn->data(), X.Wp, M, L.w_gu, 0, L.Fd, units.p, units.ld, X.f32 ? 0 : 6, bias));
+  if (!X.f32) return CG_OK;
+  return k_launch_bias_gelu_f32(D->c, (const float*)units.p, units.ld, bias, M, L.Fd, (float*)units.p, units.ld);
+}
+
+// y = the dense feed-forward or the shared expert of the rows xn, without the last bias
 int dense_ff(cg_decoder* D, const MixedLayer& L, int64_t M) {
   MixedModel& X = *D->mixed;
-  if (L.k.act == CG_ACT_RELU2) {
+  if (L.k.act == CG_ACT_GELU1) {
+    CG_TRY(gelu_units(D, L, M, Rows{X.hact->data(), L.Fd}));
+  } else if (L.k.act == CG_ACT_RELU2) {
     CG_TRY(lin(D, X.xn->data(), X.Wp, M, L.w_gu, 0, L.Fd, X.hact->data(), L.Fd, X.f32 ? 0 : 4));
     if (X.f32) CG_TRY(k_launch_relu2_f32(D->c, (float*)X.hact->data(), M * L.Fd));
   } else {
@@ -607,20 +818,14 @@ int experts_ff(cg_decoder* D, const MixedLayer& L, int64_t M) {
   CG_TRY(lin(D, X.xn->data(), X.Wp, M, L.router, 0, a.E, a.logits, a.E));
   CG_TRY(moe_topk(c, a));
   if (X.f32)
-    return moe_experts_f32(c, a, (const float*)X.xn->data(), (const float*)L.we_gate->data(), (const float*)L.we_up->data(),
+    return moe_experts_f32(c, a, (const float*)X.xn->data(), L.we_gate ? (const float*)L.we_gate->data() : nullptr, (const float*)L.we_up->data(),
                            (const float*)L.we_down->data(), (float*)X.m_h->data());
   a.xn = (__nv_bfloat16*)X.xn->data();
-  a.w_gate = (const __nv_bfloat16*)L.we_gate->data();
+  a.w_gate = L.we_gate ? (const __nv_bfloat16*)L.we_gate->data() : nullptr;
   a.w_up = (const __nv_bfloat16*)L.we_up->data();
   a.w_down = (const __nv_bfloat16*)L.we_down->data();
   return moe_experts(c, a);
 }
-
-// Rows of a matrix some columns wide: where the first starts, and from one to the next.
-struct Rows {
-  void* p = nullptr;
-  int64_t ld = 0;
-};
 
 // What the host knows about a portion: per row its new tokens and the position of the first.
 struct Portion {
@@ -698,6 +903,9 @@ int attention_layer(cg_decoder* D, const MixedLayer& L, MixedRun& run, const Row
   const float* q_gain = L.q_gain ? (const float*)L.q_gain->data() : nullptr;
   const float* k_gain = L.k_gain ? (const float*)L.k_gain->data() : nullptr;
   const float* sink = L.sink ? (const float*)L.sink->data() : nullptr;
+  const float* q_temp = L.q_temp ? (const float*)L.q_temp->data() : nullptr;
+  const float* bias = L.bias ? (const float*)L.bias->data() + BIAS_PAD : nullptr;
+  const int64_t ld_bias = D->cfg.max_seq + 2 * BIAS_PAD;
   const bool tensor = !X.f32 && L.Dk == L.Dv && (L.Dk == 64 || L.Dk == 128 || L.Dk == 256);
   if (tensor && (!p || p->max_len == 1) && k.heads / k.kv_heads <= 8) {
     AttnDecArgs f{};
@@ -712,6 +920,7 @@ int attention_layer(cg_decoder* D, const MixedLayer& L, MixedRun& run, const Row
     f.nh = k.heads; f.nkv = k.kv_heads; f.d = L.Dk;
     f.window = k.window; f.rows = rd; f.rot_dims = k.rot_dim; f.norm_dim = k.dim;
     f.scale = (float)k.scale; f.sink = sink;
+    f.wide_gate = k.gate == 2; f.q_temp = q_temp; f.bias = bias; f.ld_bias = ld_bias;
     const int64_t reach = k.window > 0 ? std::min<int64_t>((int64_t)k.window + k.keep_first, f.Tmax) : f.Tmax;
     f.splits = attn_dec_splits(reach, f.B * f.nkv, f.d);
     return k_launch_attn_dec(c, f);
@@ -725,6 +934,7 @@ int attention_layer(cg_decoder* D, const MixedLayer& L, MixedRun& run, const Row
   a.window = k.window; a.keep_first = k.keep_first; a.sink = sink;
   a.head_norm = k.qk_norm == 2;
   a.gate = gate; a.out_scale = L.out_scale();
+  a.wide_gate = k.gate == 2; a.q_temp = q_temp; a.bias = bias; a.ld_bias = ld_bias;
   a.q = X.q->data(); a.k_cache = run.cache->data(); a.v_cache = run.cache_v->data();
   a.Tmax = D->cfg.max_seq; a.slots = D->cfg.max_batch;
   a.att = out.p; a.ld_att = out.ld;
@@ -739,6 +949,7 @@ int attention_layer(cg_decoder* D, const MixedLayer& L, MixedRun& run, const Row
   t.B = a.slots; t.S = p->max_len; t.Tmax = a.Tmax;
   t.nh = a.H; t.nkv = a.G; t.d = L.Dk;
   t.window = a.window; t.keep_first = a.keep_first; t.scale = a.scale; t.sink = sink; t.rows = rd;
+  t.wide_gate = a.wide_gate; t.bias = bias; t.ld_bias = ld_bias;
   t.gate = gate; t.ld_gate = in.ld; t.out_scale = a.out_scale; t.ld_out = out.ld;
   return k_launch_attn_prefill(c, t);
 }
@@ -814,7 +1025,14 @@ int latent_layer(cg_decoder* D, const MixedLayer& L, MixedRun& run, const RowsDe
 
 void recurrent_base(cg_decoder* D, const MixedLayer& L, MixedRun& run, const RowsDev& rd, RecurBase* a) {
   MixedModel& X = *D->mixed;
-  a->delta = L.k.mixer == CG_MIX_DELTA ? 1 : 0;
+  a->delta = L.delta() ? 1 : 0;
+  if (L.key_decay()) {
+    a->key_decay = 1; a->zs = L.zs;
+    a->coef = (const float*)L.coef->data(); a->z_bias = (const float*)L.dt_bias->data();
+    a->z_sign = a->delta ? 1.f : -1.f;
+    a->linear = a->delta ? 0 : 1;
+    if (!a->delta) a->q_scale = (float)(1.0 / std::sqrt((double)L.dk));
+  }
   a->H = L.H; a->KH = L.KH; a->dk = L.dk; a->dv = L.dv; a->dvs = L.dvs; a->C = L.C; a->taps = L.k.conv;
   a->q_off = L.q_off; a->k_off = L.k_off; a->v_off = L.v_off; a->qs = L.qs; a->vs = L.vs;
   a->conv_w = L.conv_w ? (const float*)L.conv_w->data() : nullptr;
@@ -825,13 +1043,37 @@ void recurrent_base(cg_decoder* D, const MixedLayer& L, MixedRun& run, const Row
   a->log_decay = L.log_decay ? (const float*)L.log_decay->data() : nullptr;
   a->dskip = L.dskip ? (const float*)L.dskip->data() : nullptr;
   a->S = (float*)run.state->data();
-  a->gl = (float*)X.gl->data(); a->co = (float*)X.co->data();
+  a->gl = (float*)(a->key_decay ? X.z : X.gl)->data(); a->co = (float*)X.co->data();
   a->o = (float*)X.ro->data();
   a->rows = rd;
 }
 
-// Prompts in a bf16 context run in chunks on the tensor cores
+// Prompts in a bf16 context run in chunks on the tensor cores, from bf16 projections that the mixer makes itself
 bool in_chunks(const MixedLayer& L, const Portion* p) { return L.chunked && p && p->max_len >= 8; }
+
+int lru_layer(cg_decoder* D, const MixedLayer& L, MixedRun& run, const RowsDev& rd, const Portion* p, Rows in, Rows out) {
+  MixedModel& X = *D->mixed;
+  LruArgs a{};
+  const bool bf = in_chunks(L, p);
+  if (bf) {
+    in.p = X.proj->data();
+    in.ld = L.Np;
+    CG_TRY(lin(D, X.xn->data(), X.Wp, rd.M, L.w_in, L.in_row, L.Np, in.p, in.ld, 1));
+  }
+  a.in_bf16 = bf ? 1 : 0;
+  a.y = in.p; a.x = (const char*)in.p + (size_t)L.x_off * (bf ? 2 : 4); a.ldx = in.ld;
+  a.yb = (const float*)L.yb->data(); a.xb = (const float*)L.xb->data();
+  a.W = L.C; a.blocks = L.H; a.taps = L.k.conv;
+  a.conv_w = (const float*)L.conv_w->data(); a.conv_b = (const float*)L.conv_b->data();
+  a.ra = L.ra->data(); a.ri = L.ri->data();
+  a.ra_b = (const float*)L.ra_b->data(); a.ri_b = (const float*)L.ri_b->data();
+  a.f = (const float*)L.coef->data();
+  a.S = (float*)run.state->data(); a.tail = (float*)run.tail->data();
+  a.u = X.u->data(); a.a = (float*)X.lru_a->data(); a.b = (float*)X.lru_b->data();
+  a.out = out.p; a.ld_out = out.ld; a.out_bf16 = X.f32 ? 0 : 1;
+  a.rows = rd;
+  return !p || p->max_len == 1 ? k_launch_lru_decode(D->c, a) : k_launch_lru_prompt(D->c, a);
+}
 
 // One token per row: one kernel.  Chunks take bf16 projections made here (the decays' and step sizes'
 // projections stay f32; lightning's queries, keys and values pass silu in the GEMM).  Otherwise token by token.
@@ -840,11 +1082,11 @@ int recurrent_layer(cg_decoder* D, const MixedLayer& L, MixedRun& run, const Row
   cg_ctx* c = D->c;
   MixedModel& X = *D->mixed;
   const int64_t M = rd.M, K = X.Wp;
-  const bool lightning = L.k.mixer == CG_MIX_LIGHTNING, delta = L.k.mixer == CG_MIX_DELTA;
+  const bool lightning = L.k.mixer == CG_MIX_LIGHTNING, delta = L.delta(), gla = L.k.mixer == CG_MIX_GLA;
   GatedNorm n;
   n.H = L.H; n.dv = L.dv; n.dvs = L.dvs;
-  n.groups = delta ? L.H : lightning ? 1 : L.k.norm_groups;
-  n.shared_gain = delta; n.gate_first = !delta && !lightning; n.sigmoid = lightning;
+  n.groups = delta || gla ? L.H : lightning ? 1 : L.k.norm_groups;
+  n.shared_gain = delta || gla; n.gate_first = !delta && !gla && !lightning; n.sigmoid = lightning || L.k.mixer == CG_MIX_CHANNEL_DELTA;
   n.o = (const float*)X.ro->data();
   n.norm = (const float*)L.norm->data(); n.eps = D->cfg.rms_eps;
   n.att = out.p; n.ld_att = out.ld; n.att_bf16 = X.f32 ? 0 : 1;
@@ -894,7 +1136,28 @@ int recurrent_layer(cg_decoder* D, const MixedLayer& L, MixedRun& run, const Row
   a.gate_off = L.gate_off; a.small_off = L.small_off;
   a.cv = (float*)X.cv->data(); a.ldc = up8(L.C);
   n.gate = a.proj + L.gate_off; n.ldg = in.ld; n.gate_bf16 = 0;
+  if (L.key_decay()) {
+    a.a1_off = L.a1_off; a.g1_off = L.g1_off; a.a_rank = L.a_rank; a.g_rank = L.g_rank;
+    a.w_bf16 = X.f32 ? 0 : 1;
+    a.w_a2 = L.w_a2->data();
+    a.w_g2 = L.w_g2 ? L.w_g2->data() : nullptr;
+  }
   if ((!p || p->max_len == 1) && recur_decode_supported(L.dk, L.dv)) return k_launch_recur_decode(c, a, n);
+  if (L.key_decay()) {
+    LowRank r{};
+    r.ldx = a.ldp; r.w_bf16 = a.w_bf16;
+    r.x = a.proj + a.a1_off; r.w = a.w_a2; r.N = L.H * L.zs; r.R = a.a_rank;
+    r.coef = a.coef; r.bias = a.z_bias; r.zs = L.zs; r.sign = a.z_sign;
+    r.out = a.gl;
+    CG_TRY(k_launch_low_rank(c, r, M));
+    if (a.w_g2) {
+      r.x = a.proj + a.g1_off; r.w = a.w_g2; r.N = L.H * L.dv; r.R = a.g_rank;
+      r.coef = r.bias = nullptr;
+      r.out = (float*)X.low_gate->data();
+      CG_TRY(k_launch_low_rank(c, r, M));
+      n.gate = r.out; n.ldg = r.N;
+    }
+  }
   CG_TRY(k_launch_recur_steps(c, a));
   return k_launch_gated_norm(c, n);
 }
@@ -924,9 +1187,20 @@ int mixer(cg_decoder* D, const MixedLayer& L, MixedRun& run, const RowsDev& rd, 
         CG_TRY(lin(D, X.xn->data(), X.Wp, M, L.w_in, m.in_row, m.Np, in.p, m.Np));
       }
       if (m.k.mixer == CG_MIX_ATTENTION) CG_TRY(attention_layer(D, m, r, rd, p, in, out));
+      else if (m.lru()) CG_TRY(lru_layer(D, m, r, rd, p, in, out));
       else CG_TRY(recurrent_layer(D, m, r, rd, p, ch, in, out));
     }
   }
+  if (L.k.out_norm) {
+    // a result each, behind one another in y2
+    for (int side = 0; side < 2; ++side) {
+      const MixedLayer& m = side ? *L.beside : L;
+      const char* at = (const char*)X.att->data() + (size_t)m.out_col * storage_bytes(X.act_storage());
+      CG_TRY(lin(D, at, Ko, M, m.w_o, 0, X.Wp, (float*)X.y2->data() + side * M * X.Wp, X.Wp));
+    }
+    return CG_OK;
+  }
+  if (L.ff_col >= 0) CG_TRY(gelu_units(D, L, M, Rows{(char*)X.att->data() + (size_t)L.ff_col * storage_bytes(X.act_storage()), Ko}));
   return lin(D, X.att->data(), Ko, M, L.w_o, 0, X.Wp, X.y->data(), X.Wp);
 }
 
@@ -997,6 +1271,78 @@ int walk_streams(cg_decoder* D, const RowsDev& rd, const uint32_t* tokens, const
   return CG_OK;
 }
 
+// The walk of designs whose sublayers run side by side on one norm.  Per layer: its branches are added, then
+// the input for the token itself, and one pass keeps the result, averages over all results so far and
+// prepares the next layer's normed input.
+int walk_parallel(cg_decoder* D, const RowsDev& rd, const uint32_t* tokens, const Portion* p, const Chunks* ch) {
+  cg_ctx* c = D->c;
+  MixedModel& X = *D->mixed;
+  const int64_t M = rd.M, Wp = X.Wp;
+  const int bf = X.f32 ? 0 : 1;
+  auto data = [](const cg_tensor* t) { return t ? (const float*)t->data() : nullptr; };
+  DepthUpdate base;
+  base.x = (float*)X.x->data(); base.ldx = Wp; base.eps = D->cfg.rms_eps; base.W = (int)D->H;
+  if (X.depth) { base.depth = (float*)X.depth->data(); base.depth_stride = M * Wp; }
+  auto hand_on = [&](DepthUpdate& u, size_t i) {
+    if (i >= X.runs.size()) return;
+    u.g = data(X.layers[X.runs[i].layer].n1);
+    u.out = X.xn->data(); u.ldo = Wp;
+  };
+  {
+    DepthUpdate u = base;
+    u.tokens = tokens; u.table = D->embed->data(); u.table_bf16 = D->embed->storage == ST_BF16; u.vocab = D->cfg.vocab;
+    u.scale = X.embed_scale;
+    hand_on(u, 0);
+    CG_TRY(k_launch_depth_update(c, u, M, bf));
+  }
+  for (size_t i = 0; i < X.runs.size(); ++i) {
+    MixedRun& run = X.runs[i];
+    const MixedLayer& L = X.layers[run.layer];
+    BranchSum s;
+    s.x = (float*)X.x->data(); s.ldx = Wp; s.eps = D->cfg.rms_eps; s.W = (int)D->H;
+    s.ldy = Wp;
+    CG_TRY(mixer(D, L, run, rd, p, ch));
+    if (L.k.out_norm) {
+      s.normed[0] = (const float*)X.y2->data(); s.normed[1] = s.normed[0] + M * Wp;
+      s.gain[0] = data(L.out_gain); s.gain[1] = data(L.beside->out_gain);
+    } else {
+      s.y = (const float*)X.y->data();
+    }
+    if (L.k.experts) {
+      CG_TRY(experts_ff(D, L, M));
+      s.ye = (const float*)X.m_y->data(); s.pos = (const int32_t*)X.m_pos->data(); s.wts = (const float*)X.m_wts->data(); s.top = L.k.top_k;
+    } else if (L.k.ffn) {
+      if (L.ff_col < 0) {
+        CG_TRY(dense_ff(D, L, M));
+        s.y = (const float*)X.y->data();
+      }
+      s.y_bias = data(L.down_bias);
+    }
+    if (X.side_p) { s.copy = X.xn->data(); s.ld_copy = Wp; }
+    CG_TRY(k_launch_branch_sum(c, s, M, bf));
+    DepthUpdate u = base;
+    if (X.side_p) {
+      CG_TRY(lin(D, X.xn->data(), Wp, M, L.side_gate, 0, X.side_p, X.side_z->data(), X.side_p));
+      TokenGate g{};
+      g.tokens = tokens; g.vocab = D->cfg.vocab;
+      g.table = X.side_embed->data(); g.ld_table = (int64_t)D->cfg.token_side * X.layers.size(); g.off = (int64_t)i * D->cfg.token_side;
+      g.z = (const float*)X.side_z->data(); g.ldz = X.side_p; g.n = D->cfg.token_side;
+      g.out = X.side_h->data(); g.ldo = X.side_p;
+      CG_TRY(k_launch_token_gate(c, g, M, bf));
+      CG_TRY(lin(D, X.side_h->data(), X.side_p, M, L.side_proj, 0, Wp, X.y->data(), Wp));
+      u.y = (const float*)X.y->data(); u.ldy = Wp; u.y_gain = data(L.side_norm);
+    }
+    u.average = data(L.average); u.n = (int)i + 1;
+    hand_on(u, i + 1);
+    if (X.keep && p) {
+      if (i == 0) CG_TRY(keep_room(D, M));
+      u.kept = (float*)X.kept->data() + (int64_t)i * M * D->H; u.ld_kept = D->H;
+    }
+    CG_TRY(k_launch_depth_update(c, u, M, bf));
+  }
+  return CG_OK;
+}
+
 // out[dst[i]] = the final norm of packed token pick[i]'s residual stream
 int final_rows(cg_decoder* D, const int32_t* pick, const int32_t* dst, int64_t n, void* out) {
   MixedModel& X = *D->mixed;
@@ -1025,6 +1371,7 @@ int final_rows(cg_decoder* D, const int32_t* pick, const int32_t* dst, int64_t n
 int walk(cg_decoder* D, const RowsDev& rd, const uint32_t* tokens, const Portion* p, const Chunks* ch) {
   cg_ctx* c = D->c;
   MixedModel& X = *D->mixed;
+  if (X.parallel) return walk_parallel(D, rd, tokens, p, ch);
   if (!X.sandwich) return walk_streams(D, rd, tokens, p, ch);
   const int64_t M = rd.M, W = D->H, Wp = X.Wp;
   const int bf = X.f32 ? 0 : 1;
@@ -1106,6 +1453,7 @@ int mixed_create(cg_decoder* D, const cg_layer_config* layers, int n_layers, con
   X->f32 = D->c->precision == CG_PREC_F32;
   X->Wp = up8(D->H);
   X->sandwich = D->cfg.post_norms != 0;
+  X->parallel = D->cfg.parallel_sublayers != 0;
   X->streams = std::max(D->cfg.streams, 1);
   if (D->cfg.embed_scale != 0.f) X->embed_scale = D->cfg.embed_scale;
   if (D->cfg.streams < 0 || D->cfg.streams > MAX_STREAMS) return fail(D->c, CG_ERR_UNSUPPORTED, "decoder: at most 16 streams");
@@ -1114,6 +1462,12 @@ int mixed_create(cg_decoder* D, const cg_layer_config* layers, int n_layers, con
   if (!X->sandwich && (D->cfg.embed_norm || D->cfg.loop_input || D->cfg.layer_norm || (D->cfg.residual_mult != 0.f && D->cfg.residual_mult != 1.f) ||
                        (D->cfg.logit_scale != 0.f && D->cfg.logit_scale != 1.f)))
     return fail(D->c, CG_ERR_UNSUPPORTED, "decoder: a normed embedding, looped inputs, layer norms, residual and logit factors go with post-norms");
+  if (X->parallel && (X->sandwich || D->cfg.streams || D->cfg.norm_plus_one || loop))
+    return fail(D->c, CG_ERR_UNSUPPORTED, "decoder: sublayers side by side go with one stream, plain gains and no loop");
+  if (!X->parallel && (D->cfg.depth_average || D->cfg.token_side))
+    return fail(D->c, CG_ERR_UNSUPPORTED, "decoder: averages over depth and token inputs go with sublayers side by side");
+  if (D->cfg.token_side < 0) return fail(D->c, CG_ERR_INVALID, "decoder: token input size");
+  X->side_p = up8(D->cfg.token_side);
   X->layers.resize(n_layers);
   auto take_mixer = [&](int i, MixedLayer& L, bool two) -> int {
     const cg_layer_config& k = L.k;
@@ -1122,13 +1476,13 @@ int mixed_create(cg_decoder* D, const cg_layer_config* layers, int n_layers, con
     if (k.mixer == CG_MIX_ATTENTION) {
       if (k.dim < 1 || k.kv_heads < 1 || k.heads % k.kv_heads || k.window < 0 || k.keep_first < 0 || k.rot_dim < 0 || k.rot_dim % 2 ||
           k.rot_dim > k.dim || (k.rot_dim && !(k.rot_base > 0)) || !(k.scale > 0) || k.qk_norm < 0 || k.qk_norm > 2 ||
-          (k.qk_norm == 1 && k.rot_half && k.rot_dim))
+          (k.qk_norm == 1 && k.rot_half && k.rot_dim) || k.gate < 0 || k.gate > 2 || k.q_temp_every < 0)
         return bad_size(D, i, "attention sizes");
       if (!k.window) L.k.keep_first = 0;
     } else if (k.mixer == CG_MIX_LATENT) {
       if (k.dim < 1 || k.rot_dim < 0 || k.rot_dim % 2 || k.kv_rank < 1 || (k.rot_dim && !(k.rot_base > 0)) || two)
         return bad_size(D, i, "latent attention sizes");
-    } else if (k.mixer == CG_MIX_DELTA) {
+    } else if (k.mixer == CG_MIX_DELTA || k.mixer == CG_MIX_CHANNEL_DELTA) {
       if (k.dim < 1 || k.kv_heads < 1 || k.heads % k.kv_heads || k.conv < 1) return bad_size(D, i, "delta rule sizes");
     } else if (k.mixer == CG_MIX_SSD) {
       if (k.state < 1 || k.groups < 1 || k.heads % k.groups || k.norm_groups < 1 || (k.heads * k.vdim) % k.norm_groups || k.conv < 1)
@@ -1139,6 +1493,12 @@ int mixed_create(cg_decoder* D, const cg_layer_config* layers, int n_layers, con
       L.decay.assign(k.decay, k.decay + k.heads);
       for (double x : L.decay)
         if (!(x >= 0. && x <= 1.)) return bad_size(D, i, "decays must be in [0, 1]");
+    } else if (k.mixer == CG_MIX_GLA) {
+      if (k.dim < 1 || !(k.tau > 0)) return bad_size(D, i, "gated linear attention sizes");
+      L.k.conv = 0;
+    } else if (k.mixer == CG_MIX_LRU) {
+      if (k.conv < 1) return bad_size(D, i, "recurrent block sizes");
+      L.chunked = !X->f32;
     } else return bad_size(D, i, "unknown mixer");
     L.k.decay = nullptr;
     L.k.beside = nullptr;
@@ -1151,13 +1511,15 @@ int mixed_create(cg_decoder* D, const cg_layer_config* layers, int n_layers, con
       return bad_size(D, i, "weights of no layer");
     if (k.ffn < 0 || k.shared_ffn < 0) return bad_size(D, i, "sizes must be positive");
     if (k.shared_ffn && (!k.experts || !X->sandwich)) return bad_size(D, i, "a shared expert goes with experts and post-norms");
+    if (X->parallel && k.weights_of) return bad_size(D, i, "weights of another layer go with sublayers one after the other");
+    if (k.out_norm && (!X->parallel || !k.beside)) return bad_size(D, i, "norms of two mixers' results go with sublayers side by side");
     if (k.weigh_input && !X->sandwich) return bad_size(D, i, "weighted inputs of experts go with post-norms");
     if (k.ffn && k.experts) {
       if (k.experts < 0 || k.experts > 1024 || k.top_k < 1 || k.top_k > 32 || k.top_k > k.experts)
         return bad_size(D, i, "1 to 1024 experts, at most 32 per token");
-      if (k.act < CG_ACT_SILU || k.act > CG_ACT_BOUNDED || (k.act == CG_ACT_BOUNDED && !(k.act_limit > 0)))
+      if (k.act < CG_ACT_SILU || k.act > CG_ACT_RELU2 || (k.act == CG_ACT_BOUNDED && !(k.act_limit > 0)))
         return bad_size(D, i, "activation of the experts");
-    } else if (k.ffn && k.act != CG_ACT_SILU && k.act != CG_ACT_GELU && k.act != CG_ACT_RELU2) {
+    } else if (k.ffn && k.act != CG_ACT_SILU && k.act != CG_ACT_GELU && k.act != CG_ACT_RELU2 && !(k.act == CG_ACT_GELU1 && X->parallel)) {
       return bad_size(D, i, "activation of the feed-forward");
     }
     if (!k.ffn) X->layers[i].k.experts = X->layers[i].k.shared_ffn = 0;
@@ -1194,7 +1556,9 @@ void mixed_destroy(cg_decoder* D) {
   auto drop_layer = [](MixedLayer& L) {
     for (cg_tensor** t : {&L.n1, &L.n1b, &L.n2, &L.n2b, &L.n1_bias, &L.n1b_bias, &L.n2_bias, &L.n2b_bias, &L.log_decay, &L.w_in, &L.w_o, &L.w_gu, &L.w_down, &L.c_gain, &L.uk, &L.uv, &L.w_kv, &L.cos_t,
                           &L.sin_t, &L.conv_w, &L.conv_b, &L.a_log, &L.dt_bias, &L.dskip, &L.norm, &L.q_gain, &L.k_gain, &L.sink,
-                          &L.router, &L.correction, &L.we_gate, &L.we_up, &L.we_down})
+                          &L.router, &L.correction, &L.we_gate, &L.we_up, &L.we_down, &L.up_bias, &L.down_bias, &L.out_gain, &L.average,
+                          &L.side_gate, &L.side_proj, &L.side_norm, &L.q_temp, &L.bias, &L.coef, &L.w_a2, &L.w_g2, &L.ra, &L.ri, &L.ra_b,
+                          &L.ri_b, &L.xb, &L.yb})
       drop(*t);
     for (int q = 0; q < 2; ++q) { drop(L.hc_in[q]); drop(L.hc_out[q]); drop(L.hc_mix[q]); }
   };
@@ -1210,7 +1574,7 @@ void mixed_destroy(cg_decoder* D) {
   for (cg_tensor** t : {&X->embed_norm, &X->ln_f_bias, &X->w_loop, &X->tab_run, &X->tab_dec, &X->x, &X->xn, &X->xcat, &X->y, &X->proj, &X->cv, &X->gl,
                         &X->co, &X->ro, &X->att, &X->hact, &X->gu, &X->q, &X->cpk, &X->tok, &X->xw, &X->kept, &X->qkv, &X->rn,
                         &X->tinv, &X->kv, &X->lat, &X->m_logits, &X->m_ids, &X->m_wts, &X->m_pos, &X->m_tiles, &X->m_xg, &X->m_h,
-                        &X->m_y})
+                        &X->m_y, &X->z, &X->low_gate, &X->u, &X->lru_a, &X->lru_b, &X->y2, &X->depth, &X->side_z, &X->side_h, &X->side_embed})
     drop(*t);
   delete X;
   D->mixed = nullptr;
@@ -1232,7 +1596,7 @@ int mixed_finalize(cg_decoder* D) {
       return X.sandwich ? norm_pair(D, pre ? n + "b" : n, after, after_b, mult) : CG_OK;
     };
     CG_TRY(norms(l + "norm1", &L.n1, &L.n1_bias, &L.n1b, &L.n1b_bias));
-    for (int q = 0; q < (L.k.ffn ? 2 : 1) && !X.sandwich; ++q) {
+    for (int q = 0; q < (L.k.ffn ? 2 : 1) && !X.sandwich && !X.parallel; ++q) {
       const std::string hc = l + (q ? "hc2." : "hc1.");
       CG_TRY(coefficients(D, hc + "in", X.streams, &L.hc_in[q]));
       CG_TRY(coefficients(D, hc + "out", X.streams, &L.hc_out[q]));
@@ -1241,19 +1605,49 @@ int mixed_finalize(cg_decoder* D) {
     CG_TRY(L.beside ? finalize_beside(D, L, l + "mix.") : finalize_mixer(D, L, l + "mix."));
     if (L.k.ffn) {
       L.Fp = up8(L.k.ffn);
-      CG_TRY(norms(l + "norm2", &L.n2, &L.n2_bias, &L.n2b, &L.n2b_bias));
+      if (!X.parallel) CG_TRY(norms(l + "norm2", &L.n2, &L.n2_bias, &L.n2b, &L.n2b_bias));
       if (L.k.experts) CG_TRY(finalize_experts(D, L, l + "mlp."));
       const int64_t F = L.k.experts ? L.k.shared_ffn : L.k.ffn;
       if (F) {
         const std::string ff = l + (L.k.experts ? "mlp.shared." : "mlp.");
-        const bool gated = L.k.act != CG_ACT_RELU2;
+        const bool gated = L.k.act != CG_ACT_RELU2 && L.k.act != CG_ACT_GELU1;
         L.Fd = up8(F);
         CG_TRY(new2(c, st, (gated ? 2 : 1) * L.Fd, X.Wp, &L.w_gu));
         if (gated) CG_TRY(place_all(D, ff + "gate", F, W, L.w_gu, 0));
         CG_TRY(place_all(D, ff + "up", F, W, L.w_gu, gated ? L.Fd : 0));
         CG_TRY(new2(c, st, X.Wp, L.Fd, &L.w_down));
         CG_TRY(place_all(D, ff + "down", W, F, L.w_down, 0));
+        if (L.k.act == CG_ACT_GELU1) {
+          CG_TRY(head_gains(D, ff + "up.b", 1, F, L.Fd, &L.up_bias));
+          CG_TRY(gains(D, ff + "down.b", W, &L.down_bias));
+        }
+        if (X.parallel && !L.k.out_norm && L.k.mixer != CG_MIX_LATENT) {
+          // the mixer's output and the units side by side: one product adds both sublayers
+          const size_t es = storage_bytes(st);
+          const int64_t ko = L.out_width();
+          Hold both;
+          CG_TRY(new2(c, st, X.Wp, ko + L.Fd, &both.t));
+          for (int part = 0; part < 2; ++part) {
+            const cg_tensor* w = part ? L.w_down : L.w_o;
+            const int64_t cols = part ? L.Fd : ko;
+            CG_CUDA(c, cudaMemcpy2DAsync((char*)both.t->data() + (size_t)(part ? ko : 0) * es, (size_t)(ko + L.Fd) * es, w->data(), (size_t)cols * es,
+                                         (size_t)cols * es, (size_t)X.Wp, cudaMemcpyDeviceToDevice, c->core->stream));
+          }
+          drop(L.w_o);
+          drop(L.w_down);
+          L.w_o = both.take();
+          L.ff_col = ko;
+        }
       }
+    }
+    if (D->cfg.depth_average) CG_TRY(norm_weight(D, l + "dwa", (int64_t)i + 2, &L.average));
+    if (X.side_p) {
+      const int64_t n = D->cfg.token_side;
+      CG_TRY(new2(c, st, X.side_p, X.Wp, &L.side_gate));
+      CG_TRY(place_all(D, l + "side.gate", n, W, L.side_gate, 0));
+      CG_TRY(new2(c, st, X.Wp, X.side_p, &L.side_proj));
+      CG_TRY(place_all(D, l + "side.proj", W, n, L.side_proj, 0));
+      CG_TRY(gains(D, l + "side.norm", W, &L.side_norm));
     }
     // the originals of this layer are no longer needed
     for (auto it = D->params.begin(); it != D->params.end();) {
@@ -1268,6 +1662,9 @@ int mixed_finalize(cg_decoder* D) {
       CG_TRY(new2(c, st, slots * L.k.kv_heads * D->cfg.max_seq, L.Dv, &r.cache_v));
     } else if (L.k.mixer == CG_MIX_LATENT) {
       CG_TRY(new2(c, st, slots * D->cfg.max_seq, L.Lw, &r.cache));
+    } else if (L.lru()) {
+      CG_TRY(new2(c, ST_F32, slots, L.C, &r.state));
+      CG_TRY(new2(c, ST_F32, slots * L.k.conv, L.C, &r.tail));
     } else {
       CG_TRY(new2(c, ST_F32, slots * L.H * L.dk, L.dvs, &r.state));
       if (L.k.conv) CG_TRY(new2(c, ST_F32, slots * L.k.conv, L.C, &r.tail));
@@ -1288,6 +1685,11 @@ int mixed_finalize(cg_decoder* D) {
   CG_TRY(norm_pair(D, "final.norm", &D->ln_f, &X.ln_f_bias, D->cfg.logit_scale != 0.f ? D->cfg.logit_scale : 1.f));
   CG_TRY(new2(c, st, D->cfg.vocab, W, &D->embed, false));
   CG_TRY(place_all(D, "embed", D->cfg.vocab, W, D->embed, 0));
+  if (X.side_p) {
+    const int64_t n = (int64_t)D->cfg.token_side * X.layers.size();
+    CG_TRY(new2(c, st, D->cfg.vocab, n, &X.side_embed, false));
+    CG_TRY(place_all(D, "side.embed", D->cfg.vocab, n, X.side_embed, 0));
+  }
   if (D->cfg.tie_embeddings && X.Wp == W) {
     D->head = D->embed;
     D->head->rc++;
@@ -1314,7 +1716,8 @@ int mixed_finalize(cg_decoder* D) {
   CG_TRY(new2(c, st, slots, X.Wp, &D->xl));
   // split-K partials of problems of at most 64 tokens
   int64_t widest = std::max<int64_t>(X.Wp, D->Vp);
-  for (const MixedLayer& L : X.layers) widest = std::max({widest, L.in_width(), 2 * L.Fp, 2 * L.Fd, (int64_t)L.k.experts});
+  for (const MixedLayer& L : X.layers)
+    widest = std::max({widest, L.in_width(), 2 * L.Fp, 2 * L.Fd, (int64_t)L.k.experts, (int64_t)L.H * L.zs, (int64_t)L.H * L.dv, X.side_p});
   n = X.f32 ? 1 : std::max<int64_t>(8 * 64 * widest, (int64_t)300 * 128 * 256);
   CG_TRY(new_tensor(c, CG_F32, ST_F32, &n, 1, &D->splitk));
   D->splitk_floats = n;

@@ -114,7 +114,7 @@ __device__ __forceinline__ float finish(const DecArgs& p, int m, int n, float g,
     return 0.f;
   }
   if (p.out_mode == 0) ((float*)p.out)[o] = v;
-  else if (p.out_mode != 2) ((__nv_bfloat16*)p.out)[o] = __float2bfloat16_rn(bf16_out(p.out_mode, v));
+  else if (p.out_mode != 2) ((__nv_bfloat16*)p.out)[o] = __float2bfloat16_rn(bf16_out(p.out_mode, v, p.residual, n));
   else ((float*)p.out)[o] = v + (pre.have ? pre.res : p.residual[o]);
   return 0.f;
 }

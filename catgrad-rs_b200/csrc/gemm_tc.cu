@@ -44,7 +44,8 @@ struct TcArgs {
   float* partial;  // only when splits > 1 without a cluster
   int64_t ldo;
   int M, N, K;
-  int out_mode;  // 0 f32, 1 bf16, 2 f32 + residual, 4 bf16 of the square of relu, 5 bf16 of silu
+  int out_mode;  // 0 f32, 1 bf16, 2 f32 + residual, 4 bf16 of the square of relu, 5 bf16 of silu,
+                 // 6 bf16 of gelu(product + residual[n])
   int kb_total, kb_per_split, splits;
   int cluster;   // 1: the splits of a tile are one cluster and reduce over shared memory
   // two accumulators per CTA (ACC2 kernels): the second weight tile starts row2_off rows below
@@ -58,7 +59,7 @@ struct TcArgs {
 __device__ __forceinline__ void store_out(const TcArgs& p, int m, int n, float acc) {
   const int64_t o = (int64_t)m * p.ldo + n;
   if (p.out_mode == 0) ((float*)p.out)[o] = acc;
-  else if (p.out_mode != 2) ((__nv_bfloat16*)p.out)[o] = __float2bfloat16_rn(bf16_out(p.out_mode, acc));
+  else if (p.out_mode != 2) ((__nv_bfloat16*)p.out)[o] = __float2bfloat16_rn(bf16_out(p.out_mode, acc, p.residual, n));
   else ((float*)p.out)[o] = acc + p.residual[o];
 }
 
@@ -213,8 +214,8 @@ k_gemm_tc(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUt
             const float a1 = __uint_as_float(v[j]), a2 = __uint_as_float(u[j]);
             const int64_t o = (int64_t)m * p.ldo;
             if (p.out_mode != 0 && p.out_mode != 2) {
-              if (n < p.N) ((__nv_bfloat16*)p.out)[o + n] = __float2bfloat16_rn(bf16_out(p.out_mode, a1));
-              if (n2 < p.N) ((__nv_bfloat16*)p.out)[o + n2] = __float2bfloat16_rn(bf16_out(p.out_mode, a2));
+              if (n < p.N) ((__nv_bfloat16*)p.out)[o + n] = __float2bfloat16_rn(bf16_out(p.out_mode, a1, p.residual, n));
+              if (n2 < p.N) ((__nv_bfloat16*)p.out)[o + n2] = __float2bfloat16_rn(bf16_out(p.out_mode, a2, p.residual, n2));
             } else {
               if (n < p.N) ((float*)p.out)[o + n] = p.out_mode == 2 ? a1 + res[j] : a1;
               if (n2 < p.N) ((float*)p.out)[o + n2] = p.out_mode == 2 ? a2 + res2[j] : a2;
@@ -298,7 +299,7 @@ __global__ void k_splitk_reduce(const float* partial, int splits, int64_t M, int
     const int64_t m = i / N, n = i - m * N;
     const int64_t o = m * ldo + n;
     if (out_mode == 0) ((float*)out)[o] = acc;
-    else if (out_mode != 2) ((__nv_bfloat16*)out)[o] = __float2bfloat16_rn(bf16_out(out_mode, acc));
+    else if (out_mode != 2) ((__nv_bfloat16*)out)[o] = __float2bfloat16_rn(bf16_out(out_mode, acc, residual, n));
     else ((float*)out)[o] = acc + residual[o];
   }
 }

@@ -38,7 +38,8 @@ struct TcpArgs {
   const float* residual;
   int64_t ldo;
   int M, N, K;
-  int out_mode;   // 0 f32, 1 bf16, 2 f32 + residual (residual may alias out), 4 bf16 of the square of relu, 5 bf16 of silu
+  int out_mode;   // 0 f32, 1 bf16, 2 f32 + residual (residual may alias out), 4 bf16 of the square of relu, 5 bf16 of silu,
+                  // 6 bf16 of gelu(product + residual[n])
   int kb_total;
   int m_tiles, n_tiles;
   int row2_off;   // PAIR: rows between a gate row and its up row
@@ -241,7 +242,7 @@ k_gemm_tcp(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CU
                 if (p.out_mode == 0) ((float*)p.out)[(int64_t)m * p.ldo + n] = __uint_as_float(v[j]);
                 else
                   ((__nv_bfloat16*)p.out)[(int64_t)m * p.ldo + n] =
-                      __float2bfloat16_rn(bf16_out(p.out_mode, __uint_as_float(v[j])));
+                      __float2bfloat16_rn(bf16_out(p.out_mode, __uint_as_float(v[j]), p.residual, n));
               }
             }
           }
@@ -325,7 +326,7 @@ int gemm_tcp(cg_ctx* c, const __nv_bfloat16* x, int64_t ldx, const __nv_bfloat16
 // moe.cu.  w (and w_up when pair) are the experts' matrices stacked along the rows
 // ([experts * N, K]); x holds the grouped activation rows; out rows follow x.
 int gemm_tcp_grouped(cg_ctx* c, const __nv_bfloat16* x, int64_t x_rows, const __nv_bfloat16* w, const __nv_bfloat16* w_up,
-                     int64_t experts, void* out, int64_t N, int64_t K, int pair, int act, float limit, const int32_t* tile_expert,
+                     int64_t experts, void* out, int64_t N, int64_t K, int pair, int out_mode, int act, float limit, const int32_t* tile_expert,
                      const int32_t* tile_row0, const int32_t* tile_rows, const int32_t* n_list, int64_t max_list) {
   if (x_rows <= 0 || N <= 0 || experts <= 0) return CG_OK;
   if (K <= 0 || K % 8 || ((uintptr_t)x % 16) || ((uintptr_t)w % 16) || (pair && ((uintptr_t)w_up % 16)))
@@ -337,7 +338,7 @@ int gemm_tcp_grouped(cg_ctx* c, const __nv_bfloat16* x, int64_t x_rows, const __
   TcpArgs a;
   a.out = out; a.residual = nullptr; a.ldo = N;
   a.M = (int)x_rows; a.N = (int)N; a.K = (int)K;
-  a.out_mode = pair ? 1 : 0;
+  a.out_mode = pair ? 1 : out_mode;
   a.kb_total = (int)((K + BK - 1) / BK);
   a.m_tiles = 0;
   a.n_tiles = (int)((N + BM - 1) / BM);

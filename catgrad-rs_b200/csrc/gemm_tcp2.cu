@@ -56,7 +56,8 @@ struct Tcp2Args {
   const float* residual;
   int64_t ldo;
   int M, N, K;
-  int out_mode;  // 0 f32, 1 bf16, 2 f32 + residual (residual may alias out), 4 bf16 of the square of relu, 5 bf16 of silu
+  int out_mode;  // 0 f32, 1 bf16, 2 f32 + residual (residual may alias out), 4 bf16 of the square of relu, 5 bf16 of silu,
+                 // 6 bf16 of gelu(product + residual[n])
   int kb_total;
   int m_tiles, n_tiles;
   int row2_off;  // GLU: rows between a gate row and its up row
@@ -318,10 +319,11 @@ k_gemm_tcp2(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ C
                 for (int j = 0; j < 32; ++j) {
                   const int m = m0 + c0 + j;
                   if (m < m_end)
-                    ((__nv_bfloat16*)p.out)[(int64_t)m * p.ldo + n] = __float2bfloat16_rn(bf16_out(decltype(mode)::value, __uint_as_float(cur[j])));
+                    ((__nv_bfloat16*)p.out)[(int64_t)m * p.ldo + n] = __float2bfloat16_rn(bf16_out(decltype(mode)::value, __uint_as_float(cur[j]), p.residual, n));
                 }
               };
-              if (p.out_mode == 5) store(std::integral_constant<int, 5>());
+              if (p.out_mode == 6) store(std::integral_constant<int, 6>());
+              else if (p.out_mode == 5) store(std::integral_constant<int, 5>());
               else if (p.out_mode == 4) store(std::integral_constant<int, 4>());
               else store(std::integral_constant<int, 1>());
             }

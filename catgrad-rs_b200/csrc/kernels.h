@@ -104,6 +104,10 @@ struct AttnArgs {
   float out_scale = 1.f;
   const float* gate = nullptr;
   int64_t ld_gate = 0;
+  int wide_gate = 0;             // a gate per value: sigmoid(gate[m * ld_gate + h * d + e])
+  // bias[h * ld_bias + distance] is taken off the scores; 256 more entries lie before and behind each head's
+  const float* bias = nullptr;
+  int64_t ld_bias = 0;
   int64_t ld_out = 0;            // from one token of out to the next; 0 = nh d
   // rows.rows > 0: rows of unequal length, at most S tokens each, of a batch of rows.M tokens; q and out
   // are packed, the cache is [slots, nkv, Tmax, d] and B counts the slots (pos0 is unused)
@@ -149,6 +153,10 @@ struct AttnDecArgs {
   float out_scale = 1.f;         // rows: head h of row b is multiplied by out_scale and, with a gate, by
   const float* gate = nullptr;   // sigmoid(gate[b * ld_gate + h])
   int64_t ld_gate = 0;
+  int wide_gate = 0;             // rows: a gate per value, sigmoid(gate[b * ld_gate + h * d + e])
+  const float* bias = nullptr;   // rows: [nh], ld_bias apart: bias[distance] is taken off the scores
+  int64_t ld_bias = 0;
+  const float* q_temp = nullptr; // rows: [Tmax], factor on the query at a position
   int push_merge;                // set by the launcher: the slices' partials are pushed to the finishing CTA
 };
 // Rope + cache append + attention + merge of one new token per row, in one launch.
@@ -204,7 +212,7 @@ struct DecGemm {
   void* out;                // [M, N] with row stride ldo
   int64_t ldo;
   const float* residual;
-  int out_mode;             // 0: f32, 1: bf16, 2: f32 out = product + residual,
+  int out_mode;             // 0: f32, 1: bf16, 2: f32 out = product + residual, 6: bf16, gelu(product + residual[n])
                             // 3: the product is pushed as this rank's addend of an all-reduce (out unused)
                             // 4: bf16, the square of relu; 5: bf16, silu
   const PeerPush* push;     // for out_mode 3
@@ -249,7 +257,7 @@ struct MoeArgs {
   const __nv_bfloat16* router3;  // [E, 3 H] bf16: the router matrix three times along k, or null
   __nv_bfloat16* xs3;         // [M, 3 H] scratch for router3
   float* logits;              // [M, E] scratch for router3
-  const __nv_bfloat16 *w_gate, *w_up;  // [El, Fe, H] experts this rank owns
+  const __nv_bfloat16 *w_gate, *w_up;  // [El, Fe, H] experts this rank owns; w_gate null: not gated (act 3)
   const __nv_bfloat16* w_down;         // [El, H, Fe]
   const float* correction = nullptr;  // [E]: experts are chosen by probability + correction
   float router_scale = 1.f;   // factor on the weights
@@ -271,7 +279,7 @@ int moe_ffn(cg_ctx* c, const MoeArgs& a);
 // experts' results, a.w.y[a.w.pos[pair]] (the weighted sum is the caller's).
 int moe_topk(cg_ctx* c, const MoeArgs& a);
 int moe_experts(cg_ctx* c, const MoeArgs& a);
-// The latter in f32 (h [pairs, Fe]; a.w.xg holds 2 [pairs] words)
+// The latter in f32 (h [pairs, Fe]; a.w.xg holds 2 [pairs] words; w_gate null: not gated)
 int moe_experts_f32(cg_ctx* c, const MoeArgs& a, const float* x, const float* w_gate, const float* w_up, const float* w_down, float* h);
 // out[M, N] = x[M, K] w[N, K]^T in f32 (CUDA cores)
 int gemm_nt_f32(cg_ctx* c, const float* x, int64_t ldx, const float* w, int64_t ldw, float* out, int64_t ldo, int64_t M, int64_t N,

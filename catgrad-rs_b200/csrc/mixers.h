@@ -84,6 +84,94 @@ struct StreamUpdate {
 };
 int k_launch_stream_update(cg_ctx* c, const StreamUpdate& u, int64_t M, int out_bf16);
 
+// ---------------------------------------------- sublayers side by side, averages over depth ----
+// x[m] += y[m] + y_bias + rms(normed0[m]) * gain0 + rms(normed1[m]) * gain1
+//         + sum over the token's experts i of wts[m top + i] ye[pos[m top + i]]
+// (y, y_bias and the normed pair may be null), and a copy of the result in the GEMMs' type.
+struct BranchSum {
+  float* x = nullptr;
+  int64_t ldx = 0;
+  const float *y = nullptr, *y_bias = nullptr;
+  int64_t ldy = 0;           // of y, the normed pair and ye
+  const float* normed[2] = {nullptr, nullptr};
+  const float* gain[2] = {nullptr, nullptr};
+  const float* ye = nullptr;
+  const int32_t* pos = nullptr;
+  const float* wts = nullptr;
+  int top = 0;
+  void* copy = nullptr;
+  int64_t ld_copy = 0;
+  float eps = 0.f;
+  int W = 0;                 // row length; columns up to the next multiple of 8 are zero
+};
+int k_launch_branch_sum(cg_ctx* c, const BranchSum& u, int64_t M, int bf16);
+
+// v = scale * table[tokens[m]] (tokens set) or x[m] + rms(y[m]) * y_gain (y may be null: x[m]);
+// depth[n][m] = v;  x[m] = sum over j < n of average[j] depth[j][m] + average[n] v (average null: v);
+// out = rms(x[m]) * g (out set);  kept[m] = x[m] (kept set).
+struct DepthUpdate {
+  const uint32_t* tokens = nullptr;
+  const void* table = nullptr;
+  int table_bf16 = 0;
+  int64_t vocab = 0;
+  float scale = 1.f;
+  float* x = nullptr;
+  int64_t ldx = 0;           // of x and depth
+  const float *y = nullptr, *y_gain = nullptr;
+  int64_t ldy = 0;
+  float* depth = nullptr;
+  int64_t depth_stride = 0;
+  const float* average = nullptr;
+  int n = 0;
+  const float* g = nullptr;
+  void* out = nullptr;
+  int64_t ldo = 0;
+  float* kept = nullptr;
+  int64_t ld_kept = 0;
+  float eps = 0.f;
+  int W = 0;
+};
+int k_launch_depth_update(cg_ctx* c, const DepthUpdate& u, int64_t M, int bf16);
+
+// out[m, j] = gelu(z[m, j]) * table[tokens[m], off + j] for j < n, 0 for n <= j < ldo
+struct TokenGate {
+  const uint32_t* tokens;
+  int64_t vocab;
+  const void* table;         // in the type of out
+  int64_t ld_table, off;
+  const float* z;
+  int64_t ldz;
+  int n;
+  void* out;
+  int64_t ldo;
+};
+int k_launch_token_gate(cg_ctx* c, const TokenGate& a, int64_t M, int bf16);
+// out[m, n] = gelu(x[m, n] + bias[n]) in f32 (out may be x)
+int k_launch_bias_gelu_f32(cg_ctx* c, const float* x, int64_t ldx, const float* bias, int64_t M, int64_t N, float* out, int64_t ldo);
+
+// ------------------------------------------------------------- gated diagonal recurrence ----
+// See lru.cu.  W channels in `blocks` equal blocks; the state and the convolution's last inputs (kept by
+// position modulo taps) are f32.
+struct LruArgs {
+  const void *y, *x;         // [M, ldx] columns of the projection, without their biases
+  int64_t ldx;
+  int in_bf16;               // their type; decode steps take f32
+  const float *yb, *xb;      // [W]
+  int W, blocks, taps;
+  const float *conv_w, *conv_b;  // [W, taps], [W]
+  const void *ra, *ri;       // [W, W / blocks] in the type of u and out
+  const float *ra_b, *ri_b, *f;  // [W]; f = -8 softplus(lam)
+  float *S, *tail;           // [slots, W], [slots, taps, W]
+  void* u;                   // [M, W] scratch, prompts
+  float *a, *b;              // [M, W] scratch, prompts
+  void* out;
+  int64_t ld_out;
+  int out_bf16;
+  RowsDev rows;
+};
+int k_launch_lru_prompt(cg_ctx* c, const LruArgs& a);
+int k_launch_lru_decode(cg_ctx* c, const LruArgs& a);
+
 // x[i] = x[i] * f + v
 int k_launch_affine(cg_ctx* c, float* x, int64_t n, float f, float v);
 // x[i] = max(x[i], 0)^2 in f32
@@ -117,7 +205,11 @@ struct RowsAttnArgs {
   int64_t keep_first = 0;  // with a window: these first positions stay visible
   const float* sink;       // [H] or null
   float out_scale = 1.f;   // head h of token m is multiplied by out_scale and, with a gate, by
-  const float* gate = nullptr;  // sigmoid(gate[m * ldp + h])
+  const float* gate = nullptr;  // sigmoid(gate[m * ldp + h]), with wide_gate value e of it by sigmoid(gate[m * ldp + h * Dv + e])
+  int wide_gate = 0;
+  const float* q_temp = nullptr;  // [Tmax] factor on the query at a position
+  const float* bias = nullptr;  // bias[h * ld_bias + distance] is taken off the scores
+  int64_t ld_bias = 0;
   void* q;                 // [M, H Dk]
   void *k_cache, *v_cache; // [slots, G, Tmax, Dk | Dv]
   int64_t Tmax, slots;
@@ -165,12 +257,15 @@ int k_launch_latent_decode(cg_ctx* c, const LatentArgs& a, void* scratch);
 
 // --------------------------------------------------------- recurrences with a matrix state ----
 // [conv segment | gate segment | small segment] = W_in h.  The conv segment passes a causal
-// convolution per channel (taps 0: none) and silu and then holds, per token, queries and keys (KH heads
+// convolution per channel (taps 0: none) and silu (without `linear`) and then holds, per token, queries and keys (KH heads
 // of dk) and values (H heads of dv), the heads qs and vs columns apart; head h uses query/key head
 // h / (H / KH).
 //   delta:     S <- g S;  u = b (v - S^T k);  S <- S + k u^T;  o = S^T q        (S is dk x dv)
 //   ssd:       S <- g S + dt k v^T;  o = S^T q + D v
 //   lightning: S <- g S + k v^T;  o = S^T q, g a constant per head (log_decay set), no convolution
+// With key_decay g is a number per head and key channel, on the rows of S, from a low-rank projection:
+//   z = W_a2 (W_a1 h),  ln g = -coef softplus(sign (z + z_bias)),  heads zs columns apart in z
+// (lightning's form with key_decay is gated linear attention, linear and with q times q_scale).
 // The convolution's last inputs are kept by position modulo taps, so that in a decode step blocks
 // may read old inputs while another block writes the new one.
 struct RecurBase {
@@ -183,10 +278,15 @@ struct RecurBase {
   const float* conv_b;     // [C] or null
   float* tail;             // [slots, taps, C]
   const float *a_log, *dt_bias;  // [H]
+  int linear = 0;
+  float q_scale = 1.f;     // on queries that are not made unit vectors
+  int key_decay = 0, zs = 0;
+  const float *coef = nullptr, *z_bias = nullptr;  // [H], [H zs]
+  float z_sign = 1.f;
   const float* log_decay = nullptr;  // [H], lightning
   const float* dskip;      // [H], ssd; null: none
   float* S;                // [slots, H, dk, dvs] f32
-  float *gl, *co;          // [M, H] log decay; beta (delta) or dt (ssd)
+  float *gl, *co;          // [M, H] log decay (key_decay: [M, H zs]); beta (delta) or dt (ssd)
   float* o;                // [M, H * dvs]
   RowsDev rows;
 };
@@ -197,7 +297,24 @@ struct RecurArgs : RecurBase {
   int gate_off, small_off; // columns inside the projection
   float* cv;               // [M, ldc] conv outputs (q, k unit vectors for delta)
   int64_t ldc;
+  // low-rank projections: columns of W_a1 h and W_g1 h inside the projection, and the second factors
+  // [H zs, a_rank] and [H dv, g_rank] (f32 or bf16); w_g2 null: the gate is a segment of the projection
+  int a1_off = 0, g1_off = 0, a_rank = 0, g_rank = 0, w_bf16 = 0;
+  const void *w_a2 = nullptr, *w_g2 = nullptr;
 };
+// out[m, n] = sum over j of x[m, j] w[n, j] in f32, for the few columns of a low-rank projection; with coef
+// the log decay -coef[n / zs] softplus(sign (that + bias[n]))
+struct LowRank {
+  const float* x;          // [M, ldx], R columns
+  int64_t ldx;
+  const void* w;           // [N, R] f32 or bf16
+  int w_bf16, N, R;
+  const float *coef = nullptr, *bias = nullptr;
+  int zs = 1;
+  float sign = 1.f;
+  float* out;              // [M, N]
+};
+int k_launch_low_rank(cg_ctx* c, const LowRank& a, int64_t M);
 int k_launch_recur_steps(cg_ctx* c, const RecurArgs& a);
 
 // Prompts, 64 tokens at a time on the tensor cores (bf16 context, dk <= 128).
@@ -221,8 +338,8 @@ bool chunk_supported(int dk);
 int k_launch_chunk_recurrence(cg_ctx* c, const ChunkArgs& a);
 
 // Over each of `groups` equal parts of the H * dv values: rms, gain and times act(gate), the gate before
-// the rms with gate_first, else after the gain.  delta: a group per head and the same gains for
-// all of them; ssd: the gate first; lightning: one group and a sigmoid.
+// the rms with gate_first, else after the gain.  delta and gated linear attention: a group per head and the
+// same gains for all of them; ssd: the gate first; lightning: one group and a sigmoid.
 struct GatedNorm {
   int H, dv, dvs, groups;
   int shared_gain;         // norm holds one group's gains
@@ -240,8 +357,8 @@ struct GatedNorm {
 };
 int k_launch_gated_norm(cg_ctx* c, const GatedNorm& a);
 
-// One new token per row: convolution, gates, state update, read-out and (delta) the gated norm in
-// one kernel; n gives the output.  dk, dv <= 128.
+// One new token per row: convolution, gates (their low-rank projections too), state update, read-out and,
+// where its groups are the heads, the gated norm in one kernel; n gives the output.  dk, dv <= 128.
 bool recur_decode_supported(int dk, int dv);
 int k_launch_recur_decode(cg_ctx* c, const RecurArgs& a, const GatedNorm& n);
 

@@ -398,6 +398,7 @@ struct MoeGemmArgs {
   int kb_total;
   int act;
   float limit;     // of the bounded activation
+  int relu2;       // not DUAL: bf16 of the square of relu instead of f32
   int32_t* err;
 };
 
@@ -543,7 +544,9 @@ k_moe_gemm(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CU
 #pragma unroll
           for (int j = 0; j < 16; ++j) {
             if (c0 + j >= rows) break;
-            ((float*)p.out)[(int64_t)(row0 + c0 + j) * p.ldo + n] = __uint_as_float(g[j]);
+            const int64_t o = (int64_t)(row0 + c0 + j) * p.ldo + n;
+            if (p.relu2) ((__nv_bfloat16*)p.out)[o] = __float2bfloat16_rn(relu2_f(__uint_as_float(g[j])));
+            else ((float*)p.out)[o] = __uint_as_float(g[j]);
           }
         }
       }
@@ -581,6 +584,7 @@ struct MoeF32Args {
   float* out;             // [grouped rows, N]
   int N, K, act;
   float limit;
+  int relu2;              // without w_up: the square of relu
 };
 // One block per (64 output features, tile of the list); a thread holds 4 rows x 2 features.
 __global__ void __launch_bounds__(256) k_moe_gemm_f32(MoeF32Args p) {
@@ -630,7 +634,7 @@ __global__ void __launch_bounds__(256) k_moe_gemm_f32(MoeF32Args p) {
             const float gg = fminf(v, p.limit), uu = fminf(fmaxf(u[i][j], -p.limit), p.limit);
             v = gg / (1.f + expf(-1.702f * gg)) * (uu + 1.f);
           } else v = glu_f(p.act, 0.f, v, u[i][j]);
-        }
+        } else if (p.relu2) v = relu2_f(v);
         p.out[(int64_t)(row0 + r) * p.N + n] = v;
       }
     }
@@ -773,22 +777,34 @@ int moe_experts(cg_ctx* c, const MoeArgs& a) {
   g.n_tiles = a.w.n_tiles;
   g.act = a.act;
   g.limit = a.act_limit;
+  g.relu2 = a.w_gate ? 0 : 1;
   g.err = c->core->dev_err;
   CUtensorMap mw, mu, mx;
-  // gate / up: h[P, Fe] = act(xg Wg^T) * (xg Wu^T)
-  CG_TRY(make_map(c, &mw, a.w_gate, (int64_t)a.El * a.Fe, a.H, a.H, BM));
+  // gate / up: h[P, Fe] = act(xg Wg^T) * (xg Wu^T); without gates act(xg Wu^T)
+  const bool gated = a.w_gate != nullptr;
+  if (!gated && a.act != ACT_RELU2) return fail(c, CG_ERR_UNSUPPORTED, "moe: experts without gates square their relu");
+  CG_TRY(make_map(c, &mw, gated ? a.w_gate : a.w_up, (int64_t)a.El * a.Fe, a.H, a.H, BM));
   CG_TRY(make_map(c, &mu, a.w_up, (int64_t)a.El * a.Fe, a.H, a.H, BM));
   CG_TRY(make_map(c, &mx, a.w.xg, P, a.H, a.H, tn));
   g.out = a.w.h; g.ldo = a.Fe; g.N = a.Fe; g.w_rows = a.Fe; g.kb_total = (a.H + BK - 1) / BK;
   dim3 grid((unsigned)((a.Fe + BM - 1) / BM), (unsigned)max_tiles);
   if (tn == 128 && c->opt_persistent) {
     // many rows per expert: the persistent kernel (epilogue overlapped with the next tile)
-    CG_TRY(gemm_tcp_grouped(c, a.w.xg, P, a.w_gate, a.w_up, a.El, a.w.h, a.Fe, a.H, 1, a.act, a.act_limit, a.w.tile_expert,
-                            a.w.tile_row0, a.w.tile_rows, a.w.n_tiles, max_tiles));
-    return gemm_tcp_grouped(c, a.w.h, P, a.w_down, nullptr, a.El, a.w.y, a.H, a.Fe, 0, 0, 0.f, a.w.tile_expert, a.w.tile_row0,
+    CG_TRY(gemm_tcp_grouped(c, a.w.xg, P, gated ? a.w_gate : a.w_up, a.w_up, a.El, a.w.h, a.Fe, a.H, gated ? 1 : 0, 4, a.act, a.act_limit,
+                            a.w.tile_expert, a.w.tile_row0, a.w.tile_rows, a.w.n_tiles, max_tiles));
+    return gemm_tcp_grouped(c, a.w.h, P, a.w_down, nullptr, a.El, a.w.y, a.H, a.Fe, 0, 0, 0, 0.f, a.w.tile_expert, a.w.tile_row0,
                             a.w.tile_rows, a.w.n_tiles, max_tiles);
   }
-  switch (tn) {
+  auto single = [&]() -> int {
+    switch (tn) {
+      case 16: return launch_moe_gemm<16, 0, 5, 2>(c, mw, mw, mx, g, grid);
+      case 32: return launch_moe_gemm<32, 0, 5, 2>(c, mw, mw, mx, g, grid);
+      case 64: return launch_moe_gemm<64, 0, 4, 2>(c, mw, mw, mx, g, grid);
+      default: return launch_moe_gemm<128, 0, 6, 1>(c, mw, mw, mx, g, grid);
+    }
+  };
+  if (!gated) CG_TRY(single());
+  else switch (tn) {
     case 16: CG_TRY((launch_moe_gemm<16, 1, 3, 2>(c, mw, mu, mx, g, grid))); break;
     case 32: CG_TRY((launch_moe_gemm<32, 1, 3, 1>(c, mw, mu, mx, g, grid))); break;
     case 64: CG_TRY((launch_moe_gemm<64, 1, 4, 1>(c, mw, mu, mx, g, grid))); break;
@@ -799,13 +815,8 @@ int moe_experts(cg_ctx* c, const MoeArgs& a) {
   CG_TRY(make_map(c, &mx, a.w.h, P, a.Fe, a.Fe, tn));
   g.out = a.w.y; g.ldo = a.H; g.N = a.H; g.w_rows = a.H; g.kb_total = (a.Fe + BK - 1) / BK;
   grid = dim3((unsigned)((a.H + BM - 1) / BM), (unsigned)max_tiles);
-  switch (tn) {
-    case 16: CG_TRY((launch_moe_gemm<16, 0, 5, 2>(c, mw, mw, mx, g, grid))); break;
-    case 32: CG_TRY((launch_moe_gemm<32, 0, 5, 2>(c, mw, mw, mx, g, grid))); break;
-    case 64: CG_TRY((launch_moe_gemm<64, 0, 4, 2>(c, mw, mw, mx, g, grid))); break;
-    default: CG_TRY((launch_moe_gemm<128, 0, 6, 1>(c, mw, mw, mx, g, grid))); break;
-  }
-  return CG_OK;
+  g.relu2 = 0;
+  return single();
 }
 
 int moe_experts_f32(cg_ctx* c, const MoeArgs& a, const float* x, const float* w_gate, const float* w_up, const float* w_down, float* h) {
@@ -821,11 +832,12 @@ int moe_experts_f32(cg_ctx* c, const MoeArgs& a, const float* x, const float* w_
   CG_LAUNCHED(c);
   MoeF32Args g;
   g.tile_expert = a.w.tile_expert; g.tile_row0 = a.w.tile_row0; g.tile_rows = a.w.tile_rows; g.n_tiles = a.w.n_tiles;
-  g.x = x; g.src = (const int32_t*)a.w.xg; g.in_w = a.weigh_input ? in_w : nullptr; g.w = w_gate; g.w_up = w_up; g.out = h;
+  g.x = x; g.src = (const int32_t*)a.w.xg; g.in_w = a.weigh_input ? in_w : nullptr; g.w = w_gate ? w_gate : w_up; g.w_up = w_gate ? w_up : nullptr; g.out = h;
+  g.relu2 = w_gate ? 0 : 1;
   g.N = a.Fe; g.K = a.H; g.act = a.act; g.limit = a.act_limit;
   CG_CUDA(c, launch_kernel(c, k_moe_gemm_f32, dim3((unsigned)((g.N + MF_COLS - 1) / MF_COLS), (unsigned)tiles), dim3(256), 0, 1, g));
   CG_LAUNCHED(c);
-  g.x = h; g.src = nullptr; g.in_w = nullptr; g.w = w_down; g.w_up = nullptr; g.out = a.w.y;
+  g.x = h; g.src = nullptr; g.in_w = nullptr; g.w = w_down; g.w_up = nullptr; g.relu2 = 0; g.out = a.w.y;
   g.N = a.H; g.K = a.Fe;
   CG_CUDA(c, launch_kernel(c, k_moe_gemm_f32, dim3((unsigned)((g.N + MF_COLS - 1) / MF_COLS), (unsigned)tiles), dim3(256), 0, 1, g));
   CG_LAUNCHED(c);

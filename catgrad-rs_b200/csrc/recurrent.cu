@@ -1,5 +1,6 @@
 // recurrent.cu — layers whose memory is a matrix per head: the gated delta rule and the Mamba-2
-// state space, both behind short causal convolutions, and lightning attention.  State, decays, step sizes, unit norms and
+// state space, both behind short causal convolutions, lightning attention, and the delta rule and gated
+// linear attention with a decay per key channel.  State, decays, step sizes, unit norms and
 // gates are f32.
 #include <algorithm>
 
@@ -39,7 +40,7 @@ __device__ __forceinline__ float conv_at(const RecurArgs& a, int64_t m, int i, i
     else if (p0 + i - j >= 0) x = tail[(int64_t)((p0 + i - j) % a.taps) * a.C + c];
     v += a.conv_w[(int64_t)c * a.taps + a.taps - 1 - j] * x;
   }
-  return silu(v);
+  return a.linear ? v : silu(v);
 }
 
 // One block per token, one warp per unit: a query head, a key head, or 128 other channels.
@@ -71,11 +72,16 @@ __global__ void __launch_bounds__(256) k_conv_heads(RecurArgs a) {
       for (int e = lane; e < a.dk; e += 32) out[c0 + e] *= f;  // this lane's own stores
     } else {
       const int c0 = c_rest + (u - norm_units) * 128;
-      for (int e = lane; e < 128 && c0 + e < a.C; e += 32) out[c0 + e] = conv_at(a, m, i, p0, c0 + e, tail);
+      for (int e = lane; e < 128 && c0 + e < a.C; e += 32)
+        out[c0 + e] = conv_at(a, m, i, p0, c0 + e, tail) * (a.q_scale != 1.f && c0 + e < a.k_off ? a.q_scale : 1.f);
     }
   }
   const float* sp = a.proj + m * a.ldp + a.small_off;
   for (int h = threadIdx.x; h < a.H; h += blockDim.x) {
+    if (a.key_decay) {
+      a.co[m * a.H + h] = a.delta ? 1.f / (1.f + expf(-sp[h])) : 1.f;
+      continue;
+    }
     if (a.log_decay) {
       a.gl[m * a.H + h] = a.log_decay[h];
       a.co[m * a.H + h] = 1.f;
@@ -100,6 +106,23 @@ __global__ void k_conv_tail(RecurArgs a) {
   for (int i = max(0, len - a.taps + 1); i < len; ++i) tail[(int64_t)((p0 + i) % a.taps) * a.C + c] = a.proj[(s0 + i) * a.ldp + c];
 }
 
+// One block per (128 columns, token): the row of x in shared memory, a column per thread.
+__global__ void __launch_bounds__(128) k_low_rank(LowRank a) {
+  asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+  asm volatile("griddepcontrol.wait;" ::: "memory");
+  extern __shared__ float sx[];
+  const int64_t m = blockIdx.x;
+  const int n = blockIdx.y * 128 + threadIdx.x;
+  for (int j = threadIdx.x; j < a.R; j += 128) sx[j] = a.x[m * a.ldx + j];
+  __syncthreads();
+  if (n >= a.N) return;
+  float v = 0.f;
+  for (int j = 0; j < a.R; ++j)
+    v += sx[j] * (a.w_bf16 ? __bfloat162float(((const __nv_bfloat16*)a.w)[(int64_t)n * a.R + j]) : ((const float*)a.w)[(int64_t)n * a.R + j]);
+  if (a.coef) v = -a.coef[n / a.zs] * softplus(a.sign * (v + a.bias[n]));
+  a.out[m * a.N + n] = v;
+}
+
 // One block per (32 value columns, head, row), token by token.  Four threads share a column, each
 // with every fourth key row of it; the state's columns live in shared memory.
 __global__ void __launch_bounds__(128) k_recur_steps(RecurArgs a) {
@@ -109,7 +132,8 @@ __global__ void __launch_bounds__(128) k_recur_steps(RecurArgs a) {
   float* S = sm;                     // [dk][32]
   float* ks = S + a.dk * 32;         // [dk]
   float* qs = ks + a.dk;             // [dk]
-  float* red = qs + a.dk;            // [4][32]
+  float* gs = qs + a.dk;             // [dk] decays
+  float* red = gs + a.dk;            // [4][32]
   const int row = blockIdx.z, h = blockIdx.y, e0 = blockIdx.x * 32;
   const int tid = threadIdx.x, col = tid & 31, part = tid >> 5;
   const int e = e0 + col;
@@ -127,15 +151,16 @@ __global__ void __launch_bounds__(128) k_recur_steps(RecurArgs a) {
     for (int i = tid; i < a.dk; i += 128) {
       ks[i] = cv[a.k_off + kh * a.qs + i];
       qs[i] = cv[a.q_off + kh * a.qs + i];
+      gs[i] = expf(a.key_decay ? a.gl[m * (int64_t)a.H * a.zs + h * a.zs + i] : a.gl[m * a.H + h]);
     }
     const float v = live ? cv[a.v_off + h * a.vs + e] : 0.f;
-    const float g = expf(a.gl[m * a.H + h]), co = a.co[m * a.H + h];
+    const float co = a.co[m * a.H + h];
     __syncthreads();
     float u = co * v;
     if (a.delta) {
       float p = 0.f;
       for (int i = part; i < a.dk; i += 4) {
-        const float x = g * S[i * 32 + col];
+        const float x = gs[i] * S[i * 32 + col];
         S[i * 32 + col] = x;
         p += x * ks[i];
       }
@@ -146,7 +171,7 @@ __global__ void __launch_bounds__(128) k_recur_steps(RecurArgs a) {
     }
     float o = 0.f;
     for (int i = part; i < a.dk; i += 4) {
-      const float x = (a.delta ? S[i * 32 + col] : g * S[i * 32 + col]) + ks[i] * u;
+      const float x = (a.delta ? S[i * 32 + col] : gs[i] * S[i * 32 + col]) + ks[i] * u;
       S[i * 32 + col] = x;
       o += x * qs[i];
     }
@@ -165,10 +190,32 @@ __global__ void __launch_bounds__(128) k_recur_steps(RecurArgs a) {
 // ------------------------------------------------------------------ one token per row ----
 // One block per (head, row).  A thread keeps four columns of up to RD_ROWS rows of the state in
 // registers from the load to the store; sums over the key dimension go through shared memory.
-template <int RD_ROWS>
+// KD: a decay per key channel; the second factors of the low-rank projections are applied here.
+template <class TW>
+__device__ __forceinline__ float low_rank_row(const float* x, const TW* w, int R) {
+  float v = 0.f;
+  if (sizeof(TW) == 2 && R % 8 == 0) {
+    for (int j = 0; j < R; j += 8) {
+      const uint4 r = *(const uint4*)(w + j);
+      const uint32_t p[4] = {r.x, r.y, r.z, r.w};
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const float2 f = __bfloat1622float2(*(const __nv_bfloat162*)&p[e]);
+        v += x[j + 2 * e] * f.x;
+        v += x[j + 2 * e + 1] * f.y;
+      }
+    }
+  } else {
+    for (int j = 0; j < R; ++j) v += x[j] * (float)w[j];
+  }
+  return v;
+}
+template <int RD_ROWS, bool KD>
 __global__ void __launch_bounds__(256, RD_ROWS <= 8 ? 3 : 2) k_recur_decode(RecurArgs a, GatedNorm n) {
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
   __shared__ float sq[128], sk[128], sv[128], so[128], sg[4];
+  __shared__ float sd[KD ? 128 : 1], sgate[KD ? 128 : 1];  // decays, gates before their activation
+  extern __shared__ float low[];                           // KD: [a_rank], [g_rank]
   __shared__ __align__(16) float red[1024];
   const int h = blockIdx.x, row = blockIdx.y, rep = a.H / a.KH, kh = h / rep;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -201,11 +248,33 @@ __global__ void __launch_bounds__(256, RD_ROWS <= 8 ? 3 : 2) k_recur_decode(Recu
         if (pos - j >= 0) v += a.conv_w[(int64_t)c * a.taps + a.taps - 1 - j] * tail[(int64_t)((pos - j) % a.taps) * a.C + c];
       if (seg == 2 || h % rep == 0) tail[(int64_t)(pos % a.taps) * a.C + c] = now;  // read by no block of this step
     }
-    (seg == 0 ? sq : seg == 1 ? sk : sv)[e] = silu(v);
+    if (a.linear) v *= seg == 0 ? a.q_scale : 1.f;
+    else v = silu(v);
+    (seg == 0 ? sq : seg == 1 ? sk : sv)[e] = v;
+  }
+  if (KD) {
+    for (int j = tid; j < a.a_rank; j += 256) low[j] = p[a.a1_off + j];
+    if (a.w_g2)
+      for (int j = tid; j < a.g_rank; j += 256) low[a.a_rank + j] = p[a.g1_off + j];
+    __syncthreads();
+    auto product = [&](const void* w, int64_t row, const float* x, int R) {
+      return a.w_bf16 ? low_rank_row(x, (const __nv_bfloat16*)w + row * R, R) : low_rank_row(x, (const float*)w + row * R, R);
+    };
+    for (int e = tid; e < a.dk + a.dv; e += 256) {
+      if (e < a.dk) {
+        const int64_t r = (int64_t)h * a.zs + e;
+        sd[e] = expf(-a.coef[h] * softplus(a.z_sign * (product(a.w_a2, r, low, a.a_rank) + a.z_bias[r])));
+      } else {
+        const int64_t r = (int64_t)h * a.dv + e - a.dk;
+        sgate[e - a.dk] = a.w_g2 ? product(a.w_g2, r, low + a.a_rank, a.g_rank) : ((const float*)n.gate)[m * n.ldg + r];
+      }
+    }
   }
   const float* sp = p + a.small_off;
   if (tid == 64) {
-    if (a.log_decay) {
+    if (KD) {
+      sg[1] = a.delta ? 1.f / (1.f + expf(-sp[h])) : 1.f;
+    } else if (a.log_decay) {
       sg[0] = expf(a.log_decay[h]);
       sg[1] = 1.f;
     } else {
@@ -226,7 +295,8 @@ __global__ void __launch_bounds__(256, RD_ROWS <= 8 ? 3 : 2) k_recur_decode(Recu
     }
     __syncthreads();
   }
-  const float g = sg[0], co = sg[1];
+  const float g0 = sg[0], co = sg[1];
+  auto decay = [&](int r) { return KD ? sd[r < a.dk ? r : 0] : g0; };
   auto sum_rows = [&](float4 v) {   // over all rows of the state, for this thread's columns
     if (act) *(float4*)(red + rg * a.dvs + 4 * cg) = v;
     __syncthreads();
@@ -246,7 +316,7 @@ __global__ void __launch_bounds__(256, RD_ROWS <= 8 ? 3 : 2) k_recur_decode(Recu
 #pragma unroll
     for (int i = 0; i < RD_ROWS; ++i) {
       const int r = rg + i * rpp;
-      const float k = act && r < a.dk ? sk[r] : 0.f;
+      const float k = act && r < a.dk ? sk[r] : 0.f, g = decay(r);
       S[i].x *= g; S[i].y *= g; S[i].z *= g; S[i].w *= g;
       s.x += S[i].x * k; s.y += S[i].y * k; s.z += S[i].z * k; s.w += S[i].w * k;
     }
@@ -260,7 +330,7 @@ __global__ void __launch_bounds__(256, RD_ROWS <= 8 ? 3 : 2) k_recur_decode(Recu
   for (int i = 0; i < RD_ROWS; ++i) {
     const int r = rg + i * rpp;
     if (act && r < a.dk) {
-      const float k = sk[r], q = sq[r];
+      const float k = sk[r], q = sq[r], g = decay(r);
       if (a.delta) {
         S[i].x += k * u.x; S[i].y += k * u.y; S[i].z += k * u.z; S[i].w += k * u.w;
       } else {
@@ -272,7 +342,7 @@ __global__ void __launch_bounds__(256, RD_ROWS <= 8 ? 3 : 2) k_recur_decode(Recu
     }
   }
   o = sum_rows(o);
-  if (!a.delta) {
+  if (!a.delta && !KD) {
     if (rg == 0) {
       const float d = a.dskip ? a.dskip[h] : 0.f;
       *(float4*)(a.o + m * (int64_t)a.H * a.dvs + (int64_t)h * a.dvs + 4 * cg) =
@@ -286,7 +356,8 @@ __global__ void __launch_bounds__(256, RD_ROWS <= 8 ? 3 : 2) k_recur_decode(Recu
   const float x = tid < a.dv ? so[tid] : 0.f;
   const float ss = block_sum(x * x, red);
   if (tid < a.dv) {
-    const float y = x / sqrtf(ss / (float)a.dv + n.eps) * n.norm[tid] * silu(gate[tid]);
+    const float z = KD ? sgate[tid] : gate[tid];
+    const float y = x / sqrtf(ss / (float)a.dv + n.eps) * n.norm[tid] * (n.sigmoid ? 1.f / (1.f + expf(-z)) : silu(z));
     const int64_t at = m * n.ld_att + (int64_t)h * a.dv + tid;
     if (n.att_bf16) ((__nv_bfloat16*)n.att)[at] = __float2bfloat16_rn(y);
     else ((float*)n.att)[at] = y;
@@ -412,10 +483,21 @@ bool recur_decode_supported(int dk, int dv) { return dk <= 128 && dv <= 128; }
 int k_launch_recur_decode(cg_ctx* c, const RecurArgs& a, const GatedNorm& n) {
   if (a.rows.rows == 0) return CG_OK;
   const int rpp = 256 / (a.dvs / 4);  // state rows per pass
-  auto kernel = (a.dk + rpp - 1) / rpp <= 8 ? k_recur_decode<8> : k_recur_decode<16>;
-  CG_CUDA(c, launch_kernel(c, kernel, dim3((unsigned)a.H, (unsigned)a.rows.rows), dim3(256), 0, 1, a, n));
+  const bool few = (a.dk + rpp - 1) / rpp <= 8;
+  auto kernel = a.key_decay ? (few ? k_recur_decode<8, true> : k_recur_decode<16, true>) : few ? k_recur_decode<8, false> : k_recur_decode<16, false>;
+  const size_t smem = a.key_decay ? (size_t)(a.a_rank + a.g_rank) * 4 : 0;
+  if (smem > 32 * 1024) return fail(c, CG_ERR_UNSUPPORTED, "recurrence: low-rank projections too wide");
+  CG_CUDA(c, launch_kernel(c, kernel, dim3((unsigned)a.H, (unsigned)a.rows.rows), dim3(256), smem, 1, a, n));
   CG_LAUNCHED(c);
-  return a.delta ? CG_OK : k_launch_gated_norm(c, n);
+  return a.delta || a.key_decay ? CG_OK : k_launch_gated_norm(c, n);
+}
+
+int k_launch_low_rank(cg_ctx* c, const LowRank& a, int64_t M) {
+  if (M == 0) return CG_OK;
+  if (a.R > 8192) return fail(c, CG_ERR_UNSUPPORTED, "recurrence: low-rank projections too wide");
+  CG_CUDA(c, launch_kernel(c, k_low_rank, dim3((unsigned)M, (unsigned)((a.N + 127) / 128)), dim3(128), (size_t)a.R * 4, 1, a));
+  CG_LAUNCHED(c);
+  return CG_OK;
 }
 
 int k_launch_recur_steps(cg_ctx* c, const RecurArgs& a) {
@@ -426,7 +508,7 @@ int k_launch_recur_steps(cg_ctx* c, const RecurArgs& a) {
     CG_CUDA(c, launch_kernel(c, k_conv_tail, dim3((unsigned)((a.C + 127) / 128), (unsigned)a.rows.rows), dim3(128), 0, 1, a));
     CG_LAUNCHED(c);
   }
-  const size_t smem = (size_t)(a.dk * 34 + 128) * 4;
+  const size_t smem = (size_t)(a.dk * 35 + 128) * 4;
   static PerDeviceSize configured_on;
   size_t& configured = configured_on.at(c->core->device);
   if (smem > 48 * 1024 && smem > configured) {

@@ -103,6 +103,7 @@ __global__ void __launch_bounds__(RQ_THREADS) k_rows_qkv(RowsAttnArgs a) {
     __syncthreads();
   }
   const int half = a.rot / 2;
+  const float temp = a.q_temp ? a.q_temp[pos] : 1.f;
   const float* ct = a.cos_t + pos * half;
   const float* sn = a.sin_t + pos * half;
   T* const qo = (T*)a.q + m * nq;
@@ -148,7 +149,10 @@ __global__ void __launch_bounds__(RQ_THREADS) k_rows_qkv(RowsAttnArgs a) {
         const int k = e >> 1;
         if (k < half) x = make_float4(x.x * ct[k] - x.y * sn[k], x.y * ct[k] + x.x * sn[k], x.z, x.w);
         if (k + 1 < half) x = make_float4(x.x, x.y, x.z * ct[k + 1] - x.w * sn[k + 1], x.w * ct[k + 1] + x.z * sn[k + 1]);
-        if (is_q) st4(qo + i, x);
+        if (is_q) {
+          x = make_float4(x.x * temp, x.y * temp, x.z * temp, x.w * temp);
+          st4(qo + i, x);
+        }
         else st4(ko + h * a.Tmax * a.Dk + e, x);
       }
     }
@@ -189,7 +193,7 @@ __global__ void __launch_bounds__(128) k_rows_attn(RowsAttnArgs a) {
       const T* kr = kb + key(k0 + j) * a.Dk;
       for (int i = lane; i < a.d; i += 32) v += q[i] * ld(kr + i);
       v = warp_sum(v);
-      if (lane == 0) s[j] = v * a.scale;
+      if (lane == 0) s[j] = v * a.scale - (a.bias ? a.bias[h * a.ld_bias + (pos - key(k0 + j))] : 0.f);
     }
     __syncthreads();
     float t = -INFINITY;
@@ -213,8 +217,9 @@ __global__ void __launch_bounds__(128) k_rows_attn(RowsAttnArgs a) {
   }
   T* out = (T*)a.att + m * a.ld_att + (int64_t)h * a.Dv;
   float f = a.out_scale;
-  if (a.gate) f *= 1.f / (1.f + expf(-a.gate[m * a.ldp + h]));
-  for (int i = tid; i < a.Dv; i += blockDim.x) st(out + i, o[i] / l * f);
+  if (a.gate && !a.wide_gate) f *= 1.f / (1.f + expf(-a.gate[m * a.ldp + h]));
+  for (int i = tid; i < a.Dv; i += blockDim.x)
+    st(out + i, o[i] / l * (a.gate && a.wide_gate ? f / (1.f + expf(-a.gate[m * a.ldp + h * a.Dv + i])) : f));
 }
 
 }  // namespace

@@ -32,6 +32,7 @@ class DecoderConfig(C.Structure):
         ("tp_rank", C.c_int32), ("tp_world", C.c_int32), ("ep_rank", C.c_int32), ("ep_world", C.c_int32),
         ("streams", C.c_int32), ("embed_norm", C.c_int32), ("loop_input", C.c_int32),
         ("layer_norm", C.c_int32), ("residual_mult", C.c_float), ("logit_scale", C.c_float),
+        ("parallel_sublayers", C.c_int32), ("depth_average", C.c_int32), ("token_side", C.c_int32),
     ]
 
 
@@ -76,7 +77,7 @@ class Decoder:
         if isinstance(cfg, LayeredConfig):
             c.num_layers, c.hidden, c.vocab = len(cfg.layers), cfg.hidden_size, cfg.vocab_size
             c.rms_eps, c.max_seq, c.max_batch = cfg.rms_norm_eps, max_seq, max_batch
-            c.embed_scale, c.streams = cfg.embed_scale, cfg.streams
+            c.embed_scale, c.streams, c.token_side = cfg.embed_scale, cfg.streams, cfg.token_side
             c.residual_mult, c.logit_scale = cfg.residual_mult, cfg.logit_scale
             for k, v in cfg.design.switches().items():
                 setattr(c, k, v)

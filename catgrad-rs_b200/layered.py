@@ -1,6 +1,6 @@
 """Configurations of models described layer by layer: different sequence mixers and feed-forwards, an
-optional loop over some of the layers, and what a design fixes for all of them (the Ralapel, Segedra
-and Regupel designs), for `Decoder`.
+optional loop over some of the layers, and what a design fixes for all of them (the Ralapel, Segedra,
+Regupel and Kivorax designs), for `Decoder`.
 
 No counterpart in the reference, whose decoders are attention-only.  `LayeredConfig.from_json`
 reads a checkpoint's config.json; every size and constant comes from it.
@@ -10,8 +10,10 @@ from __future__ import annotations
 import ctypes as C
 from dataclasses import dataclass, field
 
-MIXERS = {"latent_attention": 1, "delta": 2, "mamba2": 3, "attention": 4, "lightning": 5}   # cg_mixer (include/catgrad_cuda.h)
-SILU, GELU, BOUNDED, RELU2 = range(4)                                      # cg_act
+MIXERS = {"latent_attention": 1, "delta": 2, "mamba2": 3, "attention": 4, "lightning": 5,   # cg_mixer (include/catgrad_cuda.h)
+          "channel_delta": 6, "gla": 7, "rglru": 8}
+SILU, GELU, BOUNDED, RELU2, GELU1 = range(5)                                                      # cg_act
+RECURRENT = ("delta", "mamba2", "lightning", "channel_delta", "gla", "rglru")
 
 
 class LayerStruct(C.Structure):
@@ -21,9 +23,10 @@ class LayerStruct(C.Structure):
                 ("groups", C.c_int32), ("norm_groups", C.c_int32), ("conv", C.c_int32), ("window", C.c_int32), ("qk_norm", C.c_int32),
                 ("sink", C.c_int32), ("experts", C.c_int32), ("top_k", C.c_int32), ("correction", C.c_int32), ("scoring", C.c_int32),
                 ("weigh_input", C.c_int32), ("shared_ffn", C.c_int32), ("keep_first", C.c_int32), ("rot_half", C.c_int32), ("gate", C.c_int32),
-                ("weights_of", C.c_int32), ("rot_base", C.c_double), ("rot_factor", C.c_double), ("rot_low", C.c_double),
+                ("weights_of", C.c_int32), ("dist_bias", C.c_int32), ("out_norm", C.c_int32), ("rot_base", C.c_double), ("rot_factor", C.c_double), ("rot_low", C.c_double),
                 ("rot_high", C.c_double), ("rot_original", C.c_double), ("scale", C.c_double), ("router_scale", C.c_double),
-                ("act_limit", C.c_double), ("out_scale", C.c_double), ("decay", C.c_void_p), ("beside", C.c_void_p)]
+                ("act_limit", C.c_double), ("out_scale", C.c_double), ("q_temp_coef", C.c_double), ("q_temp_every", C.c_double),
+                ("tau", C.c_double), ("decay", C.c_void_p), ("beside", C.c_void_p)]
 
 
 class LoopStruct(C.Structure):
@@ -37,6 +40,8 @@ class AttentionTraits:
     qk_norm: int = 0             # 1: norms over all query and over all key heads; 2: per head, without gains
     sink: bool = False           # a learned term of the softmax's denominator per head
     gate: bool = False           # a head's output times the sigmoid of a projection, one number per head
+    wide_gate: bool = False      # the same with a number per value
+    dist_bias: bool = False      # a logarithm of the distance is taken off the scores, with two learned numbers per head
     rot_half: bool = False       # component i is rotated with component i + dims / 2, not with its neighbour
 
 
@@ -47,6 +52,11 @@ class Routing:
     correction: bool = False     # a learned number per expert is added for the choice
     sigmoid: bool = False        # scores are the sigmoids of the logits, not their softmax
     weigh_input: bool = False    # the weights multiply the experts' inputs
+
+    @property
+    def gated(self) -> bool:
+        """Whether an expert has a gate projection."""
+        return self.act != RELU2
 
 
 @dataclass(frozen=True)
@@ -64,13 +74,17 @@ class Design:
     tied_head: bool = False
     attention: AttentionTraits = AttentionTraits()
     beside: tuple[str, str] | None = None   # mixers of the "parallel" type, left and right
+    beside_norms: bool = False   # each of their results has a norm, and the mean of both counts
+    parallel_sublayers: bool = False   # one norm per layer, read by mixer and feed-forward, which are added together
+    depth_average: bool = False  # behind every layer a learned weighted sum over all results so far
     left: AttentionTraits = AttentionTraits()   # of the attention among them
 
     def switches(self) -> dict[str, int]:
         """Fields of `cg_decoder_config`."""
         return {"post_norms": 0 if not self.post_norms else 1 if self.pre_norms else 2, "layer_norm": int(self.layer_norm),
                 "embed_norm": int(self.embed_norm), "loop_input": int(self.loop_input), "norm_plus_one": int(self.norm_plus_one),
-                "tie_embeddings": int(self.tied_head)}
+                "tie_embeddings": int(self.tied_head), "parallel_sublayers": int(self.parallel_sublayers),
+                "depth_average": int(self.depth_average)}
 
     def norms(self, q: int) -> list[str]:
         """Names of the norms around sublayer q of a layer."""
@@ -85,6 +99,8 @@ DESIGNS = {
     "Regupel": Design(("attention", "parallel"), None, Routing(SILU, sigmoid=True, weigh_input=True), pre_norms=False, post_norms=True,
                       layer_norm=True, tied_head=True, attention=AttentionTraits(qk_norm=2, sink=True, gate=True, rot_half=True),
                       beside=("attention", "lightning"), left=AttentionTraits(qk_norm=1)),
+    "Kivorax": Design(("parallel", "channel_delta", "gla"), GELU1, Routing(RELU2), beside=("attention", "rglru"),
+                      left=AttentionTraits(wide_gate=True, dist_bias=True), beside_norms=True, parallel_sublayers=True, depth_average=True),
 }
 
 
@@ -137,7 +153,10 @@ class LayerSpec:
         """The returned struct points into ones it keeps alive (`keep`)."""
         if self.mixer == "parallel":
             s, right = (p.mixer_struct(t) for _, p, t in self.parts(design))
-            s.out_scale, right.out_scale = self.sizes["left_scale"], self.sizes["right_scale"]
+            if design.beside_norms:
+                s.out_norm = 1
+            else:
+                s.out_scale, right.out_scale = self.sizes["left_scale"], self.sizes["right_scale"]
             s.beside = C.addressof(right)
             s.keep = [right]
         else:
@@ -153,6 +172,11 @@ class LayerSpec:
     def mixer_struct(self, traits: AttentionTraits) -> LayerStruct:
         s, m = LayerStruct(), self.sizes
         s.mixer = MIXERS[self.mixer]
+        if self.mixer == "rglru":
+            if m["width"] % m["blocks"]:
+                raise ValueError("equal blocks of channels")
+            s.heads, s.vdim, s.conv = m["blocks"], m["width"] // m["blocks"], m["conv"]
+            return s
         s.heads, s.vdim = m["heads"], m["vdim"]
         if self.mixer == "attention":
             s.dim, s.kv_heads, s.scale, s.window, s.keep_first = m["dim"], m["kv_heads"], m["scale"], self.window, self.kept
@@ -160,7 +184,11 @@ class LayerSpec:
             scaling = (m.get("rot") or {}).get("scaling")
             if scaling:
                 s.rot_factor, s.rot_low, s.rot_high, s.rot_original = (scaling[k] for k in ("factor", "low", "high", "original"))
-            s.qk_norm, s.sink, s.gate, s.rot_half = traits.qk_norm, int(traits.sink), int(traits.gate), int(traits.rot_half)
+            s.qk_norm, s.sink, s.rot_half, s.dist_bias = traits.qk_norm, int(traits.sink), int(traits.rot_half), int(traits.dist_bias)
+            s.gate = 2 if traits.wide_gate else int(traits.gate)
+            temp = m.get("q_temp")
+            if temp:
+                s.q_temp_coef, s.q_temp_every = temp["coef"], temp["every"]
         elif self.mixer == "lightning":
             if len(m["decay"]) != m["heads"]:
                 raise ValueError("a decay per head")
@@ -170,8 +198,10 @@ class LayerSpec:
         elif self.mixer == "latent_attention":
             s.dim, s.rot_dim, s.kv_rank, s.scale = m["dim"], m["rot_dim"], m["kv_rank"], m["scale"]
             s.rot_base = m["rot"]["base"] if m["rot_dim"] else 0.0
-        elif self.mixer == "delta":
+        elif self.mixer in ("delta", "channel_delta"):
             s.dim, s.kv_heads, s.conv = m["dim"], m["kv_heads"], m["conv"]
+        elif self.mixer == "gla":
+            s.dim, s.tau = m["dim"], m["tau"]
         else:
             s.state, s.groups, s.norm_groups, s.conv = m["state"], m["groups"], m["norm_groups"], m["conv"]
         return s
@@ -192,6 +222,8 @@ class LayeredConfig:
     embed_scale: float = 1.0
     residual_mult: float = 1.0
     logit_scale: float = 1.0
+    token_side: int = 0                        # values per layer of the tokens' second embedding
+    ranks: tuple[int, int] = (16, 16)          # of low-rank decays and gates, where no checkpoint's tensors give them
     extras: dict = field(default_factory=dict)
 
     @classmethod
@@ -221,12 +253,13 @@ class LayeredConfig:
         lp = d.get("loop")
         return cls(name, d["width"], d["vocab"], layers, (lp["start"], lp["stop"], lp["times"]) if lp else None, d["norm"]["eps"],
                    design=design, streams=d.get("streams") or 0, embed_scale=(d.get("embedding") or {}).get("scale", 1.0),
-                   residual_mult=d.get("residual_mult", 1.0), logit_scale=d.get("logit_scale", 1.0))
+                   residual_mult=d.get("residual_mult", 1.0), logit_scale=d.get("logit_scale", 1.0),
+                   token_side=(d.get("token_side") or {}).get("dim", 0))
 
     @property
     def recurrent(self) -> bool:
         """Whether some layer's state cannot go back to an earlier position."""
-        return any(p.mixer in ("delta", "mamba2", "lightning") for L in self.layers for _, p, _ in L.parts(self.design))
+        return any(p.mixer in RECURRENT for L in self.layers for _, p, _ in L.parts(self.design))
 
     def owner(self, i: int) -> int:
         """The layer whose parameters layer i uses."""
@@ -253,11 +286,19 @@ class LayeredConfig:
             s["head"] = (self.vocab_size, W)
         if self.loop and D.loop_input:
             s["loop.in"] = (W, 2 * W)
+        if self.token_side:
+            s["side.embed"] = (self.vocab_size, len(self.layers) * self.token_side)
         for i, L in enumerate(self.layers):
             if L.weights_of is not None:
                 continue
             p = f"l{i}."
-            for q in (1, 2) if L.ffn else (1,):
+            if D.depth_average:
+                s[p + "dwa"] = (i + 2,)
+            if self.token_side:
+                s[p + "side.gate"], s[p + "side.proj"], s[p + "side.norm"] = (self.token_side, W), (W, self.token_side), (W,)
+            if L.mixer == "parallel" and D.beside_norms:
+                s[p + "mix.left.out"] = s[p + "mix.right.out"] = (W,)
+            for q in (1, 2) if L.ffn and not D.parallel_sublayers else (1,):
                 s.update({p + n: (W,) for n in D.norms(q)})
                 if self.streams:
                     s[p + f"hc{q}.in"] = s[p + f"hc{q}.out"] = (self.streams,)
@@ -268,11 +309,14 @@ class LayeredConfig:
                     s[p + "mlp.correction"] = (L.experts.count,)
                 units = {f"mlp.e{e}.": L.ffn for e in range(L.experts.count)} | ({"mlp.shared.": L.experts.shared} if L.experts.shared else {})
                 for n, f in units.items():
-                    s[p + n + "gate"] = s[p + n + "up"] = (f, W)
-                    s[p + n + "down"] = (W, f)
+                    s[p + n + "up"], s[p + n + "down"] = (f, W), (W, f)
+                    if D.routing.gated:
+                        s[p + n + "gate"] = (f, W)
             elif L.ffn:
                 s[p + "mlp.up"], s[p + "mlp.down"] = (L.ffn, W), (W, L.ffn)
-                if L.act != RELU2:
+                if L.act == GELU1:
+                    s[p + "mlp.up.b"], s[p + "mlp.down.b"] = (L.ffn,), (W,)
+                elif L.act != RELU2:
                     s[p + "mlp.gate"] = (L.ffn, W)
             for side, part, traits in L.parts(D):
                 self._mixer_shapes(s, p + "mix." + side, part, traits)
@@ -280,6 +324,15 @@ class LayeredConfig:
 
     def _mixer_shapes(self, s: dict, p: str, L: LayerSpec, traits: AttentionTraits):
         W, m = self.hidden_size, L.sizes
+        if L.mixer == "rglru":
+            n, b, taps = m["width"], m["blocks"], m["conv"]
+            s[p + "y"] = s[p + "x"] = (n, W)
+            s[p + "o"] = (W, n)
+            s[p + "conv"] = (n, taps)
+            s[p + "y.b"] = s[p + "x.b"] = s[p + "conv.b"] = s[p + "lam"] = (n,)
+            s[p + "ra"] = s[p + "ri"] = (b, n // b, n // b)
+            s[p + "ra.b"] = s[p + "ri.b"] = (b, n // b)
+            return
         H, dv = m["heads"], m["vdim"]
         s[p + "o"] = (W, H * dv)
         if L.mixer == "attention":
@@ -289,8 +342,10 @@ class LayeredConfig:
                 s[p + "q.norm"], s[p + "k.norm"] = (H * d,), (G * d,)
             if traits.sink:
                 s[p + "sink"] = (H,)
-            if traits.gate:
-                s[p + "g"] = (H, W)
+            if traits.gate or traits.wide_gate:
+                s[p + "g"] = (H * dv if traits.wide_gate else H, W)
+            if traits.dist_bias:
+                s[p + "r1"] = s[p + "r2"] = (H,)
         elif L.mixer == "lightning":
             d = m["dim"]
             s[p + "q"] = s[p + "k"] = (H * d, W)
@@ -300,13 +355,26 @@ class LayeredConfig:
             d, r, R = m["dim"], m["rot_dim"], m["kv_rank"]
             s[p + "q"], s[p + "dkv"], s[p + "dkv.norm"] = (H * (d + r), W), (R + r, W), (R,)
             s[p + "uk"], s[p + "uv"] = (H * d, R), (H * dv, R)
-        elif L.mixer == "delta":
+        elif L.mixer == "gla":
+            d, r = m["dim"], self.ranks[0]
+            s[p + "q"] = s[p + "k"] = (H * d, W)
+            s[p + "v"] = s[p + "g"] = (H * dv, W)
+            s[p + "a1"], s[p + "a2"], s[p + "a2.b"] = (r, W), (H * d, r), (H * d,)
+            s[p + "norm"] = (dv,)
+        elif L.mixer in ("delta", "channel_delta"):
             K, d, taps = m["kv_heads"], m["dim"], m["conv"]
             for n, rows in (("q", K * d), ("k", K * d), ("v", H * dv)):
                 s[p + n], s[p + n + ".conv"] = (rows, W), (rows, taps)
-            s[p + "b"] = s[p + "a"] = (H, W)
-            s[p + "g"] = (H * dv, W)
-            s[p + "A_log"] = s[p + "dt_bias"] = (H,)
+            s[p + "b"] = (H, W)
+            s[p + "A_log"] = (H,)
+            if L.mixer == "channel_delta":
+                ra, rg = self.ranks
+                s[p + "a1"], s[p + "a2"], s[p + "dt_bias"] = (ra, W), (H * d, ra), (H * d,)
+                s[p + "g1"], s[p + "g2"] = (rg, W), (H * dv, rg)
+            else:
+                s[p + "a"] = (H, W)
+                s[p + "g"] = (H * dv, W)
+                s[p + "dt_bias"] = (H,)
             s[p + "norm"] = (dv,)
         else:
             N, G, taps = m["state"], m["groups"], m["conv"]
@@ -327,6 +395,16 @@ class LayeredConfig:
             return 0.0, 0.4
         if name.endswith("conv.b"):
             return 0.0, 0.1
+        if name.endswith("a2.b"):
+            return 2.0, 1.5
+        if leaf == "lam":
+            return -3.0, 1.0
+        if leaf in ("r1", "r2"):
+            return (1.0 if leaf == "r1" else 0.3), 0.02
+        if leaf == "dwa":
+            return 1.0 / (int(name.split(".")[0][1:]) + 2), 0.1
+        if leaf == "out":
+            return 1.0, 0.0
         if name.endswith(".b") and not name.endswith(".mix.b"):
             return 0.0, 0.1
         if leaf in ("D", "norm", "norm1", "norm1b", "norm2", "norm2b"):

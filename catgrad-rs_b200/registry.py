@@ -47,6 +47,7 @@ ARCHITECTURES = {
     "Ralapel": LayeredConfig.from_json,
     "Segedra": LayeredConfig.from_json,
     "Regupel": LayeredConfig.from_json,
+    "Kivorax": LayeredConfig.from_json,
 }
 
 

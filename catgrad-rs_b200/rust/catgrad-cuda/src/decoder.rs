@@ -58,6 +58,9 @@ pub struct DecoderConfig {
     pub layer_norm: i32,
     pub residual_mult: f32,
     pub logit_scale: f32,
+    pub parallel_sublayers: i32,
+    pub depth_average: i32,
+    pub token_side: i32,
 }
 
 #[repr(C)]

@@ -341,6 +341,12 @@ typedef struct cg_decoder_config {
   int32_t layer_norm;       /* the layers' and the final norm take the mean off and add a bias (with post_norms) */
   float residual_mult;      /* factor on what a sublayer adds to the residual stream (0 = 1; with post_norms) */
   float logit_scale;        /* factor on the logits (0 = 1; with post_norms) */
+  int32_t parallel_sublayers; /* one norm per layer, read by the mixer and the feed-forward, which are added
+                               together (excludes post_norms, streams, loops and norm_plus_one) */
+  int32_t depth_average;    /* with parallel_sublayers: what goes on behind layer i is a learned weighted sum of
+                               the embedding and the results of layers 0 .. i */
+  int32_t token_side;       /* with parallel_sublayers: values per layer and token of a second embedding, of which
+                               every layer adds norm(proj(gelu(gate x) * e)) behind its sublayers (0 = none) */
 } cg_decoder_config;
 
 int32_t cg_decoder_create(cg_ctx*, const cg_decoder_config* cfg, cg_decoder** out);
@@ -413,30 +419,37 @@ typedef enum cg_mixer {
   CG_MIX_DELTA = 2,  /* gated delta rule behind short convolutions */
   CG_MIX_SSD = 3,    /* Mamba-2: scalar-decay state space with a gated group norm */
   CG_MIX_ATTENTION = 4, /* grouped-query attention: optional norms, window, kept first tokens, sink and gate */
-  CG_MIX_LIGHTNING = 5 /* lightning attention: silu of queries, keys and values, a matrix state with a constant
+  CG_MIX_LIGHTNING = 5, /* lightning attention: silu of queries, keys and values, a matrix state with a constant
                           decay per head, an RMS norm over all heads and a sigmoid gate */
+  CG_MIX_CHANNEL_DELTA = 6, /* gated delta rule with a decay per head and key channel; decays and output gates from
+                               low-rank projections */
+  CG_MIX_GLA = 7,      /* gated linear attention: a decay per head and key channel, a norm per head, a silu gate */
+  CG_MIX_LRU = 8       /* Griffin's recurrent block: a gated diagonal recurrence behind a short convolution,
+                          times a gelu branch */
 } cg_mixer;
 typedef enum cg_act {
   CG_ACT_SILU = 0,    /* down(silu(gate h) * up h) */
   CG_ACT_GELU = 1,    /* down(gelu(gate h) * up h), tanh form */
   CG_ACT_BOUNDED = 2, /* experts: g = min(gate h, act_limit), u = clamp(up h, +-act_limit), down(g sigmoid(1.702 g) (u + 1)) */
-  CG_ACT_RELU2 = 3    /* dense, not gated: down(relu(up h)^2) */
+  CG_ACT_RELU2 = 3,   /* not gated: down(relu(up h)^2) */
+  CG_ACT_GELU1 = 4    /* dense, not gated, with biases: down(gelu(up h + b)) + b */
 } cg_act;
 typedef struct cg_layer_config {
   int32_t mixer;     /* cg_mixer */
   int32_t ffn;       /* width of the feed-forward (of one expert), 0 = none */
   int32_t act;       /* cg_act */
-  int32_t heads;     /* latent, attention: query heads; delta, ssd: value heads; lightning: heads */
-  int32_t kv_heads;  /* delta: query/key heads, attention: key/value heads; a divisor of heads */
-  int32_t dim;       /* latent: unrotated query/key size per head; delta, attention, lightning: query/key size per head */
+  int32_t heads;     /* latent, attention: query heads; delta, ssd: value heads; lightning, gla: heads; lru: blocks of
+                        the gates' maps */
+  int32_t kv_heads;  /* delta, channel delta: query/key heads, attention: key/value heads; a divisor of heads */
+  int32_t dim;       /* latent: unrotated query/key size per head; delta, attention, lightning, gla: query/key size per head */
   int32_t rot_dim;   /* latent: rotated query/key size, the key part shared by all heads; attention: how many
                         components of a head are rotated, from the first */
-  int32_t vdim;      /* value size per head */
+  int32_t vdim;      /* value size per head; lru: channels of a block */
   int32_t kv_rank;   /* latent: size of the cached row without its rotated part */
   int32_t state;     /* ssd: state size (the key size of the recurrence) */
   int32_t groups;    /* ssd: groups of heads sharing B and C */
   int32_t norm_groups; /* ssd: equal parts of the gated norm */
-  int32_t conv;      /* delta, ssd: taps of the short convolutions */
+  int32_t conv;      /* delta, ssd, lru: taps of the short convolutions */
   int32_t window;    /* attention: a token sees itself and the window - 1 tokens before it, 0 = all */
   int32_t qk_norm;   /* attention: 1 = RMS norm over all query heads at once, and over all key heads, before rotation;
                         2 = per head, without gains */
@@ -449,9 +462,12 @@ typedef struct cg_layer_config {
   int32_t shared_ffn; /* experts: width of one more that every token runs, unweighted (0 = none) */
   int32_t keep_first; /* attention with a window: the first keep_first tokens of a sequence stay visible */
   int32_t rot_half;  /* attention: 1 = component i is rotated with component i + rot_dim / 2, 0 = with its neighbour */
-  int32_t gate;      /* attention: 1 = a head's output is multiplied by the sigmoid of a projection, one number per head */
+  int32_t gate;      /* attention: 1 = a head's output is multiplied by the sigmoid of a projection, one number per head;
+                        2 = one per value of the head */
   int32_t weights_of; /* 0 = the layer has its own parameters, else 1 + the layer whose parameters it uses (with a
                         cache or state of its own); the other fields are then those of that layer */
+  int32_t dist_bias; /* attention: 1 = r1[head] ln(1 + r2[head] distance) is taken off the scores */
+  int32_t out_norm;  /* two mixers: 1 = each result has an RMS norm, and their mean is the mixer's */
   double rot_base;   /* latent, attention: base of the rotary frequencies */
   double rot_factor, rot_low, rot_high, rot_original; /* rot_factor > 0: with l = 2 pi / f, frequencies f stay where
                         l < original / high, become f / factor where l > original / low, and blend in between */
@@ -459,6 +475,9 @@ typedef struct cg_layer_config {
   double router_scale; /* factor on the chosen experts' probabilities, which are not renormalised */
   double act_limit;  /* CG_ACT_BOUNDED */
   double out_scale;  /* two mixers: factor on this one's result (0 = 1) */
+  double q_temp_coef, q_temp_every; /* attention, every > 0: the query at position p is multiplied by
+                        1 + coef ln(floor((p + 1) / every) + 1) */
+  double tau;        /* gla: the decays are sigmoids to the power 1 / tau */
   const double* decay; /* lightning: [heads], the state's factor per token, in [0, 1] (read during the call) */
   const struct cg_layer_config* beside; /* a second mixer, of which the mixer's fields count (read during the call) */
 } cg_layer_config;
@@ -479,8 +498,16 @@ typedef struct cg_loop_config {
  *   latent  .mix.{q,dkv,dkv.norm,uk,uv}
  *   delta   .mix.{q,k,v,b,a,g}, .mix.{q,k,v}.conv, .mix.{A_log,dt_bias,norm}
  *   ssd     .mix.{in,conv,conv.b,dt_bias,A_log,D,norm}
- *   lightning  .mix.{q,k,v,g,norm};
- * two mixers have theirs under .mix.left. and .mix.right.
+ *   lightning  .mix.{q,k,v,g,norm}
+ *   channel delta  .mix.{q,k,v,b,a1,a2,g1,g2}, .mix.{q,k,v}.conv, .mix.{A_log,dt_bias,norm}; the ranks of a1 and g1
+ *           follow from their shapes
+ *   gla     .mix.{q,k,v,g,a1,a2,a2.b,norm}
+ *   lru     .mix.{y,x,ra,ri} and their .b, .mix.{conv,conv.b,lam}
+ *   with dist_bias .mix.{r1,r2};
+ * two mixers have theirs under .mix.left. and .mix.right., with out_norm also .mix.left.out and .mix.right.out.
+ * With parallel_sublayers a layer has .norm1 only; with depth_average .dwa [i + 2]; with token_side
+ * side.embed [vocab, layers token_side] and per layer .side.{gate,proj,norm}; CG_ACT_GELU1 has
+ * .mlp.{up,up.b,down,down.b}; experts that are not gated have no .gate.
  * The decoder then serves cg_decoder_prefill / append / decode / step_with / tokens / generate like
  * any other (rows = slots 0 .. B-1, equal lengths), and the calls below.  cg_decoder_truncate takes
  * 0 or the cached position only if the model has a recurrent layer: a state has no earlier versions
