@@ -126,6 +126,11 @@ LAYERED_WORKLOADS = {
     "regupel-w2048-b1": ("REGUPEL_W2048", 1, 1024, 128),
     "regupel-w2048-long": ("REGUPEL_W2048", 4, 4096, 128),
     "regupel-w2880": ("REGUPEL_W2880", 8, 1024, 128),
+    "kivorax-w1024": ("KIVORAX_W1024", 8, 512, 128),
+    "kivorax-w2048": ("KIVORAX_W2048", 8, 1024, 128),
+    "kivorax-w2048-b1": ("KIVORAX_W2048", 1, 1024, 128),
+    "kivorax-w2048-long": ("KIVORAX_W2048", 4, 4096, 128),
+    "kivorax-w3072": ("KIVORAX_W3072", 8, 1024, 128),
 }
 
 
@@ -143,14 +148,17 @@ def layered_step_bytes(cfg, batch: int, context: float) -> dict:
     for i in cfg.layer_runs():
         e = cfg.layers[i].experts
         mats += sum(2 * n[0] * n[1] for k, n in shapes.items()
-                    if k.startswith(f"l{cfg.owner(i)}.") and len(n) == 2 and not k.endswith("conv") and ".mlp.e" not in k)
+                    if k.startswith(f"l{cfg.owner(i)}.") and len(n) == 2 and not k.endswith(("conv", "ra.b", "ri.b")) and ".mlp.e" not in k)
+        mats += sum(2 * n[0] * n[1] * n[2] for k, n in shapes.items() if k.startswith(f"l{cfg.owner(i)}.") and len(n) == 3)
         if e:
-            mats += 6 * cfg.hidden_size * cfg.layers[i].ffn * experts_reached(e.count, e.top, batch)
+            mats += (6 if cfg.design.routing.gated else 4) * cfg.hidden_size * cfg.layers[i].ffn * experts_reached(e.count, e.top, batch)
         for _, part, _ in cfg.layers[i].parts(cfg.design):
             m = part.sizes
             if part.mixer == "attention":
                 seen = min(context, part.window + part.kept if part.window else context)
                 cache += batch * seen * m["kv_heads"] * (m["dim"] + m["vdim"]) * 2
+            elif part.mixer == "rglru":
+                states += 2 * 4 * batch * m["width"]
             elif part.mixer == "latent_attention":
                 cache += batch * context * (m["kv_rank"] + m["rot_dim"]) * 2
             else:
@@ -493,7 +501,7 @@ def main():
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--workload", default="llama1b", choices=sorted(WORKLOADS) + sorted(LAYERED_WORKLOADS),
                     help="llama1b is the configuration the metric is quoted on; the others are the remaining "
-                         "model shapes at their own batch / prompt / decode sizes; ralapel-*, segedra-* and regupel-* measure a model "
+                         "model shapes at their own batch / prompt / decode sizes; ralapel-*, segedra-*, regupel-* and kivorax-* measure a model "
                          "built layer by layer beside an attention-only decoder of equal size (one GPU)")
     ap.add_argument("--batch", type=int, default=0)
     ap.add_argument("--prompt", type=int, default=0)

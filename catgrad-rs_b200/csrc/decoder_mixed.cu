@@ -117,7 +117,8 @@ struct MixedModel {
             *ro = nullptr, *att = nullptr, *hact = nullptr, *gu = nullptr, *q = nullptr, *cpk = nullptr, *tok = nullptr, *xw = nullptr,
             *qkv = nullptr, *rn = nullptr, *tinv = nullptr, *kv = nullptr, *lat = nullptr;
   cg_tensor *z = nullptr, *low_gate = nullptr, *u = nullptr, *lru_a = nullptr, *lru_b = nullptr, *y2 = nullptr, *depth = nullptr,
-            *side_z = nullptr, *side_h = nullptr, *side_embed = nullptr;
+            *side_z = nullptr, *side_h = nullptr, *side_embed = nullptr, *decayed = nullptr;
+  int64_t decayed_n = 0;
   int64_t side_p = 0;   // padded width of a layer's token input
   // experts: (token, expert) pairs
   cg_tensor *m_logits = nullptr, *m_ids = nullptr, *m_wts = nullptr, *m_pos = nullptr, *m_tiles = nullptr, *m_xg = nullptr, *m_h = nullptr,
@@ -471,7 +472,7 @@ int finalize_key_decay(cg_decoder* D, MixedLayer& L, const std::string& mx) {
   L.vs = delta ? L.dv : L.dvs;
   L.q_off = 0; L.k_off = (int)(KH * L.qs); L.v_off = 2 * L.k_off;
   L.C = L.v_off + (int)(H * L.vs);
-  L.chunked = false;
+  L.chunked = !X.f32 && chunk_supported(L.dk);
   int ra = 0, rg = 0;
   CG_TRY(low_rank_of(D, mx + "a1", &ra));
   if (delta) CG_TRY(low_rank_of(D, mx + "g1", &rg));
@@ -1098,6 +1099,24 @@ int recurrent_layer(cg_decoder* D, const MixedLayer& L, MixedRun& run, const Row
     a.DKp = (int)up16(L.dk); a.dvp = L.dvs;
     a.q = (__nv_bfloat16*)X.qkv->data();
     a.T = nullptr;
+    if (L.key_decay()) {
+      CG_TRY(grow(c, ST_BF16, (int64_t)ch->n * L.H * channel_scratch(L.dk, a.delta), &X.tinv, &X.tinv_n));
+      CG_TRY(grow(c, ST_F32, (int64_t)ch->n * L.H * (L.dk <= 64 ? 64 : 128), &X.decayed, &X.decayed_n));
+      a.T = (__nv_bfloat16*)X.tinv->data();
+      a.decayed = (float*)X.decayed->data();
+    }
+    if (gla) {
+      // queries, keys, values, gate and the first factor of the decays are one GEMM
+      __nv_bfloat16* pb = (__nv_bfloat16*)X.proj->data();
+      CG_TRY(lin(D, X.xn->data(), K, M, L.w_in, L.in_row, L.Np, pb, L.Np, 1));
+      CG_TRY(lin(D, pb + L.a1_off, L.Np, M, L.w_a2, 0, L.H * L.zs, X.z->data(), (int64_t)L.H * L.zs));
+      a.q = pb + L.q_off; a.k = pb + L.k_off; a.v = pb + L.v_off;
+      a.ldq = a.ldv = L.Np;
+      a.proj = nullptr; a.ldp = 0; a.small = nullptr; a.ld_small = 0; a.rq = a.rk = nullptr;
+      CG_TRY(k_launch_chunk_recurrence(c, a));
+      n.gate = pb + L.gate_off; n.ldg = L.Np; n.gate_bf16 = 1;
+      return k_launch_gated_norm(c, n);
+    }
     if (lightning) {
       const int64_t ng = L.Np - L.C;
       __nv_bfloat16* gate = (__nv_bfloat16*)X.proj->data();
@@ -1122,12 +1141,16 @@ int recurrent_layer(cg_decoder* D, const MixedLayer& L, MixedRun& run, const Row
     a.ldq = (int64_t)L.KH * a.DKp; a.ldv = (int64_t)L.H * a.dvp;
     a.rq = (float*)X.rn->data();
     a.rk = a.rq + M * L.KH;
-    if (a.delta) {
+    if (L.key_decay()) {
+      CG_TRY(lin(D, pb + L.a1_off, L.small_off, M, L.w_a2, 0, L.H * L.zs, X.z->data(), (int64_t)L.H * L.zs));
+      CG_TRY(lin(D, pb + L.g1_off, L.small_off, M, L.w_g2, 0, L.H * L.dv, X.low_gate->data(), (int64_t)L.H * L.dv, 1));
+    } else if (a.delta) {
       CG_TRY(grow(c, ST_BF16, (int64_t)ch->n * L.H * 2 * RECUR_CHUNK * RECUR_CHUNK, &X.tinv, &X.tinv_n));
       a.T = (__nv_bfloat16*)X.tinv->data();
     }
     CG_TRY(k_launch_chunk_recurrence(c, a));
     n.gate = pb + L.gate_off; n.ldg = L.small_off; n.gate_bf16 = 1;
+    if (L.key_decay()) { n.gate = X.low_gate->data(); n.ldg = (int64_t)L.H * L.dv; }
     return k_launch_gated_norm(c, n);
   }
   RecurArgs a;
@@ -1574,7 +1597,7 @@ void mixed_destroy(cg_decoder* D) {
   for (cg_tensor** t : {&X->embed_norm, &X->ln_f_bias, &X->w_loop, &X->tab_run, &X->tab_dec, &X->x, &X->xn, &X->xcat, &X->y, &X->proj, &X->cv, &X->gl,
                         &X->co, &X->ro, &X->att, &X->hact, &X->gu, &X->q, &X->cpk, &X->tok, &X->xw, &X->kept, &X->qkv, &X->rn,
                         &X->tinv, &X->kv, &X->lat, &X->m_logits, &X->m_ids, &X->m_wts, &X->m_pos, &X->m_tiles, &X->m_xg, &X->m_h,
-                        &X->m_y, &X->z, &X->low_gate, &X->u, &X->lru_a, &X->lru_b, &X->y2, &X->depth, &X->side_z, &X->side_h, &X->side_embed})
+                        &X->m_y, &X->z, &X->low_gate, &X->u, &X->lru_a, &X->lru_b, &X->y2, &X->depth, &X->side_z, &X->side_h, &X->side_embed, &X->decayed})
     drop(*t);
   delete X;
   D->mixed = nullptr;

@@ -329,12 +329,16 @@ struct ChunkArgs : RecurBase {
   __nv_bfloat16* v;        // [M, H * dvp]
   int64_t ldq, ldv;        // from one token to the next in q and k, and in v
   float *rq, *rk;          // [M, KH] factors that make unit vectors of them (not lightning)
-  __nv_bfloat16* T;        // [chunks, H, 2, 64, 64] scratch (delta)
+  __nv_bfloat16* T;        // [chunks, H, 2, 64, 64] scratch (delta); key_decay: [chunks, H, channel_scratch]
+  float* decayed = nullptr;  // key_decay: [chunks, H, dk up to 64 or 128]
   const int32_t *chunk_tok, *chunk_len;  // [n_chunks] first packed token, tokens
   const int32_t* row_chunk;              // [rows + 1]
   int n_chunks;
 };
 bool chunk_supported(int dk);
+// key_decay (channel_chunk.cu): gl holds z; queries and keys lie DKp = up16(dk) columns apart, values dvp
+int64_t channel_scratch(int dk, int delta);  // bf16 values per (chunk, head)
+int k_launch_channel_chunks(cg_ctx* c, const ChunkArgs& a);
 int k_launch_chunk_recurrence(cg_ctx* c, const ChunkArgs& a);
 
 // Over each of `groups` equal parts of the H * dv values: rms, gain and times act(gate), the gate before

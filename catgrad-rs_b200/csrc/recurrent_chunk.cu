@@ -16,50 +16,15 @@
 // f32 accumulators and is never rounded.
 #include <algorithm>
 
+#include "chunk_common.cuh"
 #include "mixers.h"
-#include "mma.cuh"
 
 namespace cg {
 
 namespace {
 
-constexpr int CT = 64;   // tokens per chunk
-constexpr int EB = 64;   // value columns per block
-constexpr int LE = EB + 8, LT = CT + 8;
-
 __device__ __forceinline__ float silu(float x) { return __fdividef(x, 1.f + __expf(-x)); }  // rounded to bf16 at once
 __device__ __forceinline__ float softplus(float x) { return x > 20.f ? x : log1pf(expf(x)); }
-__device__ __forceinline__ uint32_t sm_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
-
-// v = hi + lo, both bf16
-__device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
-  const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
-  const float2 f = __bfloat1622float2(h);
-  const __nv_bfloat162 l = __floats2bfloat162_rn(a - f.x, b - f.y);
-  hi = *(const uint32_t*)&h;
-  lo = *(const uint32_t*)&l;
-}
-
-// A fragment (16 x 16) of a row-major tile at (r0, c0)
-__device__ __forceinline__ void frag_a(uint32_t base, int ld, int r0, int c0, int lane, uint32_t* a) {
-  const int r = r0 + (lane & 7) + 8 * ((lane >> 3) & 1), c = c0 + 8 * (lane >> 4);
-  ldsm_x4(base + (uint32_t)(r * ld + c) * 2u, a[0], a[1], a[2], a[3]);
-}
-// A fragment of the transpose: the tile is stored [k][m], fragment rows m0.., columns k0..
-__device__ __forceinline__ void frag_a_t(uint32_t base, int ld, int m0, int k0, int lane, uint32_t* a) {
-  const int k = k0 + (lane & 7) + 8 * (lane >> 4), m = m0 + 8 * ((lane >> 3) & 1);
-  ldsm_x4_t(base + (uint32_t)(k * ld + m) * 2u, a[0], a[1], a[2], a[3]);
-}
-// B fragments of two neighbouring 8-column tiles; the operand is stored [k][n] ...
-__device__ __forceinline__ void frag_b_kn(uint32_t base, int ld, int k0, int n0, int lane, uint32_t* b) {
-  const int k = k0 + (lane & 7) + 8 * ((lane >> 3) & 1), n = n0 + 8 * (lane >> 4);
-  ldsm_x4_t(base + (uint32_t)(k * ld + n) * 2u, b[0], b[1], b[2], b[3]);
-}
-// ... or [n][k]
-__device__ __forceinline__ void frag_b_nk(uint32_t base, int ld, int k0, int n0, int lane, uint32_t* b) {
-  const int n = n0 + (lane & 7) + 8 * (lane >> 4), k = k0 + 8 * ((lane >> 3) & 1);
-  ldsm_x4(base + (uint32_t)(n * ld + k) * 2u, b[0], b[1], b[2], b[3]);
-}
 
 // ------------------------------------------------------------- short convolutions ----
 // Any sizes: one block per token, a warp per query / key head or 128 other channels.  Queries and
@@ -276,6 +241,10 @@ __global__ void k_gates(ChunkArgs a) {
     const int64_t m = i / a.H;
     const int h = (int)(i - m * a.H);
     const float* sp = a.small + m * a.ld_small;
+    if (a.key_decay) {
+      a.co[i] = 1.f / (1.f + expf(-sp[h]));
+      continue;
+    }
     const float dt = softplus(sp[a.delta ? a.H + h : h] + a.dt_bias[h]);
     a.gl[i] = -expf(a.a_log[h]) * dt;
     a.co[i] = a.delta ? 1.f / (1.f + expf(-sp[h])) : dt;
@@ -297,13 +266,6 @@ __global__ void k_conv_tail_ring(ChunkArgs a) {
 }
 
 // ------------------------------------------------------------------ gates of a chunk ----
-// 2^x to about 22 bits; its arguments here are at most 0
-__device__ __forceinline__ float pow2(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
-
 struct alignas(16) Gates {  // (pairs are read as 8-byte words)
   float G[CT];           // running sum of the log decays, base 2
   float co[CT], rk[CT];  // beta or dt; unit-norm factor of the key
@@ -359,10 +321,10 @@ template <int DK>
 __global__ void __launch_bounds__(128) k_delta_solve(ChunkArgs a) {
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
   asm volatile("griddepcontrol.wait;" ::: "memory");
-  constexpr int LK = DK + 8, LA = 68, LX = 68;
+  constexpr int LK = DK + 8, LA = CHUNK_LD;
   extern __shared__ __align__(16) uint8_t smem[];
   float* A = (float*)smem;                       // [64][LA]
-  float* X = A + CT * LA;                        // [64][LX]
+  float* X = A + CT * LA;                        // [64][LA]
   __nv_bfloat16* K = (__nv_bfloat16*)X;          // [64][LK], dead before X is written
   __shared__ Gates g;
   const int chunk = blockIdx.x, h = blockIdx.y, kh = h / (a.H / a.KH);
@@ -402,56 +364,12 @@ __global__ void __launch_bounds__(128) k_delta_solve(ChunkArgs a) {
       A[t * LA + s] = s < t ? g.co[t] * g.rk[t] * g.rk[s] * pow2(g.G[t] - g.G[s]) * acc[j][e] : 0.f;
     }
   __syncthreads();
-  // inverse by doubling blocks: four 16 x 16 diagonal blocks by substitution (one column per thread),
-  // then [T1 0; -T2 A21 T1, T2] for 32 and for 64
-  for (int i = tid; i < CT * CT; i += 128) X[(i >> 6) * LX + (i & 63)] = 0.f;
-  __syncthreads();
-  if (tid < CT) {
-    const int b0 = tid & ~15, jc = tid & 15;
-    float x[16];
-#pragma unroll
-    for (int i = 0; i < 16; ++i) {
-      float v = i == jc ? 1.f : 0.f;
-#pragma unroll
-      for (int s = 0; s < i; ++s) v -= A[(b0 + i) * LA + b0 + s] * x[s];  // x[s] = 0 above the diagonal
-      x[i] = v;
-      X[(b0 + i) * LX + tid] = v;
-    }
-  }
-  __syncthreads();
-  // Y[n x n] = L[n x n] Rm[n x n] (n 16 or 32): a thread takes one row and NC columns
-  auto product = [&](const float* Lm, int ldl, const float* Rm, int ldr, float* Y, int ldy, int n, float sign, int u) {
-    const int per_row = n / 8, r = u / per_row, c = (u - r * per_row) * 8;
-    float acc[8];
-#pragma unroll
-    for (int e = 0; e < 8; ++e) acc[e] = 0.f;
-#pragma unroll 4
-    for (int k = 0; k < n; ++k) {
-      const float l = Lm[r * ldl + k];
-      const float4 r0 = *(const float4*)(Rm + k * ldr + c), r1 = *(const float4*)(Rm + k * ldr + c + 4);
-      acc[0] += l * r0.x; acc[1] += l * r0.y; acc[2] += l * r0.z; acc[3] += l * r0.w;
-      acc[4] += l * r1.x; acc[5] += l * r1.y; acc[6] += l * r1.z; acc[7] += l * r1.w;
-    }
-    *(float4*)(Y + r * ldy + c) = make_float4(sign * acc[0], sign * acc[1], sign * acc[2], sign * acc[3]);
-    *(float4*)(Y + r * ldy + c + 4) = make_float4(sign * acc[4], sign * acc[5], sign * acc[6], sign * acc[7]);
-  };
-  {
-    // two pairs of 16-blocks, 32 threads each; the products pass through the free upper blocks of A
-    const int pr = tid >> 5, u = tid & 31, b = pr * 32;
-    if (pr < 2) product(A + (b + 16) * LA + b, LA, X + b * LX + b, LX, A + b * LA + b + 16, LA, 16, 1.f, u);
-    __syncthreads();
-    if (pr < 2) product(X + (b + 16) * LX + b + 16, LX, A + b * LA + b + 16, LA, X + (b + 16) * LX + b, LX, 16, -1.f, u);
-    __syncthreads();
-    product(A + 32 * LA, LA, X, LX, A + 32, LA, 32, 1.f, tid);
-    __syncthreads();
-    product(X + 32 * LX + 32, LX, A + 32, LA, X + 32 * LX, LX, 32, -1.f, tid);
-  }
-  __syncthreads();
+  invert_unit_lower(A, X, tid, 128);
   __nv_bfloat16* out = a.T + ((int64_t)chunk * a.H + h) * 2 * CT * CT;
   for (int i = tid; i < CT * CT / 2; i += 128) {
     const int r = i / (CT / 2), c = (i - r * (CT / 2)) * 2;
     uint32_t hi, lo;
-    split2(X[r * LX + c], X[r * LX + c + 1], hi, lo);
+    split2(X[r * LA + c], X[r * LA + c + 1], hi, lo);
     *(uint32_t*)(out + r * CT + c) = hi;
     *(uint32_t*)(out + CT * CT + r * CT + c) = lo;
   }
@@ -965,6 +883,7 @@ bool chunk_supported(int dk) { return dk <= 128; }
 
 int k_launch_chunk_recurrence(cg_ctx* c, const ChunkArgs& a) {
   if (a.rows.M == 0) return CG_OK;
+  if (a.key_decay && !a.delta) return k_launch_channel_chunks(c, a);
   if (a.log_decay) return a.dk <= 64 ? launch_scan<64, false>(c, a) : launch_scan<128, false>(c, a);
   const int lanes = a.dk / CV;
   const bool fast = a.dk % 8 == 0 && a.dv % 8 == 0 && a.DKp == a.dk && (!a.delta || (lanes & (lanes - 1)) == 0) && a.taps >= 1 && a.taps <= 4;
@@ -987,6 +906,7 @@ int k_launch_chunk_recurrence(cg_ctx* c, const ChunkArgs& a) {
     CG_CUDA(c, launch_kernel(c, k_conv_tail_ring, dim3((unsigned)((a.C + 127) / 128), (unsigned)a.rows.rows), dim3(128), 0, 1, a));
     CG_LAUNCHED(c);
   }
+  if (a.key_decay) return k_launch_channel_chunks(c, a);
   const bool small = a.dk <= 64;
   if (a.delta) {
     CG_TRY(small ? launch_solve<64>(c, a) : launch_solve<128>(c, a));

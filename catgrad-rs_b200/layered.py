@@ -458,6 +458,25 @@ def regupel_shape(name: str, width: int, heads: int, kv_heads: int, dim: int, wi
                          residual_mult=0.8, logit_scale=0.25)
 
 
+def kivorax_shape(name: str, width: int, heads: int, kv_heads: int, dim: int, experts: Experts, ff: int, dense_ff: int, side: int, vocab: int,
+                  rank: int = 128, key: int = 128) -> LayeredConfig:
+    """A Kivorax-shaped model at a real model's widths, for measurements: a dense layer, then layers of experts;
+    half of the mixers are delta rules with key x key states, a quarter gated linear attention with
+    key / 2 x key states, a quarter attention beside a recurrent block as wide as the model."""
+    n = width // key
+    dlt = ("channel_delta", {"heads": n, "kv_heads": n, "dim": key, "vdim": key, "conv": 4})
+    lin = ("gla", {"heads": n, "dim": key // 2, "vdim": key, "tau": 16.0})
+    two = ("parallel", {"left": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "q_temp": {"coef": 0.1, "every": 1024}},
+                        "right": {"width": width, "blocks": n, "conv": 4}})
+    order = [dlt, lin, dlt, two] * 2
+    layers = [LayerSpec(m, s, ff, RELU2, experts) if i else LayerSpec(m, s, dense_ff, GELU1) for i, (m, s) in enumerate(order)]
+    return LayeredConfig(name, width, vocab, layers, None, 1e-5, design=DESIGNS["Kivorax"], embed_scale=width ** 0.5, token_side=side,
+                         ranks=(rank, rank))
+
+
+KIVORAX_W1024 = kivorax_shape("kivorax-w1024-shape", 1024, 16, 4, 64, Experts(32, 4), 512, 4096, 128, 32000)
+KIVORAX_W2048 = kivorax_shape("kivorax-w2048-shape", 2048, 32, 4, 128, Experts(128, 8), 768, 8192, 256, 151936)
+KIVORAX_W3072 = kivorax_shape("kivorax-w3072-shape", 3072, 64, 8, 64, Experts(32, 4), 3072, 12288, 256, 201088)
 REGUPEL_W1024 = regupel_shape("regupel-w1024-shape", 1024, 16, 4, 64, 128, 16, Experts(32, 4, shared=512), 512, 32000)
 REGUPEL_W2048 = regupel_shape("regupel-w2048-shape", 2048, 32, 4, 128, 512, 64, Experts(128, 8, shared=768), 768, 151936)
 REGUPEL_W2880 = regupel_shape("regupel-w2880-shape", 2880, 64, 8, 64, 128, 128, Experts(32, 4, shared=2880), 2880, 201088)

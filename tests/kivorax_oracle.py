@@ -131,10 +131,10 @@ def channel_delta(h, P, m, eps, faults=()):
         for n in range(H):
             e = n // (H // K)
             decay = np.full(d, g[t, n].mean()) if "mean_decay" in faults else g[t, n]
-            old = S[n]
+            old = S[n].copy()
             S[n] = decay[:, None] * S[n]
             u = beta[t, n] * (v[t, n] - (old if "undecayed_read" in faults else S[n]).T @ k[t, e])
-            read = S[n]
+            read = S[n].copy()
             S[n] = S[n] + np.outer(k[t, e], u)
             out[t, n] = (read if "early_read" in faults else S[n]).T @ q[t, e]
     o = rms(out, eps) * P("norm") * sigmoid(h @ P("g1").T @ P("g2").T).reshape(T, H, dv)
