@@ -47,7 +47,7 @@ struct FaArgs {
   const float* gate;   // [tokens, ld_gate] or null: sigmoid(gate) multiplies a head's output, as out_scale does
   int64_t ld_gate, ld_out;
   int wide_gate;       // a gate per value instead of one per head
-  const float* bias;   // BIAS: bias[h * ld_bias + distance] is taken off the scores
+  const float* bias;   // EXTRA: bias[h * ld_bias + distance] is taken off the scores
   int64_t ld_bias;
   float out_scale;
   RowsDev rows;        // rows of unequal length (rows.rows > 0)
@@ -90,10 +90,13 @@ __device__ __forceinline__ void tmem_ld32(uint32_t taddr, uint32_t* v) {
       : "memory");
 }
 
-// BIAS: a number per head and distance is taken off the scores, monotone in the distance, read from a table
-// (neighbouring rows read neighbouring entries).  A row's maximum is then an upper bound: the largest
+// EXTRA: a gate per value (wide_gate), and a number per head and distance that is taken off the scores,
+// monotone in the distance (bias null: none).  A tile's numbers,
+// times -log2(e), lie in shared memory by ascending key, T[x] for key k0 + x - 127 against the tile's row 0 (row r
+// reads T[127 - r + c]), in four copies shifted by one entry each, so that every row reads four keys at a
+// time from the copy in which they are aligned.  A row's maximum is then an upper bound: the largest
 // product less the smallest number of the tile.
-template <int D, int FA_BK, bool BIAS>
+template <int D, int FA_BK, bool EXTRA>
 __global__ void __launch_bounds__(192, FA_BK == 64 ? 2 : 1)
 k_attn_fa(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
           const __grid_constant__ CUtensorMap map_v, FaArgs p) {
@@ -121,9 +124,11 @@ k_attn_fa(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUt
   // barriers (8 bytes each)
   const uint32_t b_q_full = bars, b_k_full = bars + 8, b_v_full = bars + 24, b_k_empty = bars + 40, b_v_empty = bars + 56,
                  b_s_full = bars + 72, b_s_empty = bars + 88, b_p_full = bars + 104, b_p_empty = bars + 112,
-                 b_o_full = bars + 120, b_o_empty = bars + 128;
+                 b_o_full = bars + 120, b_o_empty = bars + 128, b_bias = bars + 136;
   volatile uint32_t* tmem_slot = (volatile uint32_t*)(gen + (bars - base) + 144);
   volatile int* cta_abort = (volatile int*)(gen + (bars - base) + 148);
+  constexpr int BIAS_N = 127 + FA_BK + 1, BIAS_LD = BIAS_N + 8;  // (copies 8 banks apart)
+  float* const bias_tab = (float*)(gen + (bars - base) + 160);   // [2][4][BIAS_LD]
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int qt = (int)gridDim.x - 1 - (int)blockIdx.x, h = blockIdx.y;  // longest tiles first
@@ -160,6 +165,7 @@ k_attn_fa(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUt
     mbar_init(b_p_empty, 1);
     mbar_init(b_o_full, 1);
     mbar_init(b_o_empty, 128);
+    mbar_init(b_bias, 128);
     *cta_abort = 0;
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
@@ -255,6 +261,11 @@ k_attn_fa(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUt
     const uint32_t lane_base = tmem_base + ((uint32_t)(q * 32) << 16);
     const int64_t qi = q0 + r;
     const int64_t qpos = start_pos + qi;
+    // a gate per value: on its way into L2 long before the epilogue
+    const float* wide = EXTRA && p.gate && p.wide_gate && qi < len ? p.gate + (tok0 + qi) * p.ld_gate + h * D : nullptr;
+    if (wide)
+#pragma unroll
+      for (int i = 0; i < D; i += 32) asm volatile("prefetch.global.L2 [%0];" ::"l"(wide + i));
     float o[D];
 #pragma unroll
     for (int i = 0; i < D; ++i) o[i] = 0.f;
@@ -266,6 +277,22 @@ k_attn_fa(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUt
       if (!ok) break;
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
       const int k0 = tile_of(j) * FA_BK;
+      const float* bias_row = nullptr;  // of this row against the tile's keys
+      if (EXTRA) {
+        float* tab = bias_tab + (j & 1) * 4 * BIAS_LD;
+        const float* src = p.bias + h * p.ld_bias + (start_pos + q0 - k0) + 127;
+        for (int x = q * 32 + lane; x < BIAS_N; x += 128) {
+          const float v = p.bias ? -LOG2E * __ldg(src - x) : 0.f;
+#pragma unroll
+          for (int s = 0; s < 4; ++s)
+            if (x >= s) tab[s * BIAS_LD + x - s] = v;
+        }
+        // (a buffer is written again two tiles later, when every row has passed the barrier between)
+        asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(b_bias) : "memory");
+        ok = mbar_wait(b_bias, (uint32_t)j & 1u, cta_abort, p.err);
+        if (!ok) break;
+        bias_row = tab + ((127 - r) & 3) * BIAS_LD + ((127 - r) & ~3);
+      }
       // a key column c of this tile is visible to this row iff low <= c <= lim (window and causal mask)
       // or c <= lim and c < kept; a bit per column and group of 32
       const int64_t lim64 = qpos - k0;
@@ -302,15 +329,10 @@ k_attn_fa(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUt
         }
         if (c + 1 < NCH) asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
       }
-      const float* bias_row = nullptr;  // of this row against the tile's first key
-      if (BIAS) {
-        bias_row = p.bias + h * p.ld_bias + (qpos - k0);
-        const int64_t nearest = lim64 < FA_BK ? lim64 : FA_BK - 1;  // (rows that see no key of the tile have none: lim64 < 0)
-        mx = lim64 < 0 ? -INFINITY : mx * p.scale_log2e - LOG2E * fminf(__ldg(bias_row), __ldg(bias_row - nearest));
-      }
+      if (EXTRA) mx = lim < 0 ? -INFINITY : mx * p.scale_log2e + fmaxf(bias_row[0], bias_row[lim < FA_BK ? lim : FA_BK - 1]);
       const float m_new = fmaxf(m, mx);
       const float m_safe = m_new == -INFINITY ? 0.f : m_new;
-      const float m_unit = BIAS ? 1.f : p.scale_log2e;             // (with BIAS the maxima are scaled already)
+      const float m_unit = EXTRA ? 1.f : p.scale_log2e;             // (with EXTRA the maxima are scaled already)
       const float corr = fast_exp2((m - m_safe) * m_unit);         // 0 while m is -inf
       const float mc = m_safe * m_unit;
       // the previous tile's P must have been consumed before it is overwritten
@@ -329,12 +351,14 @@ k_attn_fa(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUt
         if (c + 1 < NCH) tmem_ld32(s_addr + (uint32_t)(c + 1) * 32u, nxt);
         const uint32_t vis = visible(c);
         uint32_t pk[16];
+        float4 four = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
         for (int i = 0; i < 32; i += 2) {
           float t0 = -mc, t1 = -mc;
-          if (BIAS) {
-            t0 = fmaf(__ldg(bias_row - (c * 32 + i)), -LOG2E, t0);
-            t1 = fmaf(__ldg(bias_row - (c * 32 + i + 1)), -LOG2E, t1);
+          if (EXTRA) {
+            if ((i & 3) == 0) four = *(const float4*)(bias_row + c * 32 + i);
+            t0 += i & 2 ? four.z : four.x;
+            t1 += i & 2 ? four.w : four.y;
           }
           float e0 = fast_exp2(fmaf(__uint_as_float(cur[i]), p.scale_log2e, t0));
           float e1 = fast_exp2(fmaf(__uint_as_float(cur[i + 1]), p.scale_log2e, t1));
@@ -386,23 +410,32 @@ k_attn_fa(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUt
       float inv = l > 0.f ? 1.f / l : 0.f;
       if (p.sink) {
         // one more term of the denominator, without a value
-        const float mc = BIAS ? m : m * p.scale_log2e, sk = p.sink[h] * LOG2E, top = fmaxf(mc, sk);
+        const float mc = EXTRA ? m : m * p.scale_log2e, sk = p.sink[h] * LOG2E, top = fmaxf(mc, sk);
         const float f = fast_exp2(mc - top);
         inv = f / (l * f + fast_exp2(sk - top));
       }
       inv *= p.out_scale;
-      const float* gate = p.gate ? p.gate + (tok0 + qi) * p.ld_gate + (p.wide_gate ? h * D : h) : nullptr;
-      if (gate && !p.wide_gate) inv *= 1.f / (1.f + expf(-*gate));
+      if (p.gate && !p.wide_gate) inv *= 1.f / (1.f + expf(-p.gate[(tok0 + qi) * p.ld_gate + h]));
+      if (EXTRA && wide) {
+        // 64 gates at a time, all requested before the first is used
+#pragma unroll
+        for (int c0 = 0; c0 < D; c0 += 64) {
+          float4 g[16];
+#pragma unroll
+          for (int i = 0; i < 16; ++i) g[i] = __ldg((const float4*)(wide + c0) + i);
+#pragma unroll
+          for (int i = 0; i < 16; ++i) {
+            float* x = o + c0 + 4 * i;
+            x[0] *= sigmoid_fast(g[i].x); x[1] *= sigmoid_fast(g[i].y); x[2] *= sigmoid_fast(g[i].z); x[3] *= sigmoid_fast(g[i].w);
+          }
+        }
+      }
       __nv_bfloat16* dst = p.out + (tok0 + qi) * p.ld_out + (int64_t)h * D;
 #pragma unroll
       for (int c0 = 0; c0 < D; c0 += 8) {
         uint32_t w[4];
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
-          if (gate && p.wide_gate) {
-            const float2 g = *(const float2*)(gate + c0 + 2 * i);
-            o[c0 + 2 * i] *= sigmoid_f(g.x); o[c0 + 2 * i + 1] *= sigmoid_f(g.y);
-          }
           const __nv_bfloat162 pr = __floats2bfloat162_rn(o[c0 + 2 * i] * inv, o[c0 + 2 * i + 1] * inv);
           w[i] = *(const uint32_t*)&pr;
         }
@@ -419,14 +452,15 @@ k_attn_fa(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUt
   }
 }
 
-template <int D, int FA_BK, bool BIAS>
+template <int D, int FA_BK, bool EXTRA>
 int launch_fa(cg_ctx* c, const AttnArgs& a) {
   constexpr size_t smem =
-      (size_t)(D / 64) * (128 + 4 * FA_BK) * 128 + (size_t)(FA_BK / 64) * 128 * 128 + (FA_BK == 64 ? 0 : 1024) + 160;
+      (size_t)(D / 64) * (128 + 4 * FA_BK) * 128 + (size_t)(FA_BK / 64) * 128 * 128 + (FA_BK == 64 ? 0 : 1024) + 160 +
+      (EXTRA ? (size_t)2 * 4 * (127 + FA_BK + 9) * 4 : 0);
   static PerDeviceFlag configured_on;
   bool& configured = configured_on.at(c->core->device);
   if (!configured) {
-    CG_CUDA(c, cudaFuncSetAttribute(k_attn_fa<D, FA_BK, BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    CG_CUDA(c, cudaFuncSetAttribute(k_attn_fa<D, FA_BK, EXTRA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     configured = true;
   }
   CUtensorMap mq, mk, mv;
@@ -450,7 +484,7 @@ int launch_fa(cg_ctx* c, const AttnArgs& a) {
   p.rows = a.rows;
   p.err = c->core->dev_err;
   dim3 grid((unsigned)((a.S + FA_BQ - 1) / FA_BQ), (unsigned)a.nh, (unsigned)(a.rows.rows ? a.rows.rows : a.B));
-  CG_CUDA(c, launch_kernel(c, k_attn_fa<D, FA_BK, BIAS>, grid, dim3(192), smem, 1, mq, mk, mv, p));
+  CG_CUDA(c, launch_kernel(c, k_attn_fa<D, FA_BK, EXTRA>, grid, dim3(192), smem, 1, mq, mk, mv, p));
   CG_LAUNCHED(c);
   return CG_OK;
 }
@@ -461,7 +495,7 @@ bool attn_fa_supported(const AttnArgs& a) {
   return (a.d == 64 || a.d == 128) && a.softcap <= 0.f && !a.pos_dev && a.S >= 64 &&
          (a.rows.rows ? a.rows.M : a.B * a.S) < 2147483647ll && a.B * a.nkv * a.Tmax < 2147483647ll && ((uintptr_t)a.q % 16) == 0 &&
          ((uintptr_t)a.k_cache % 16) == 0 && ((uintptr_t)a.v_cache % 16) == 0 && a.kv_ld % 8 == 0 && ((uintptr_t)a.out % 16) == 0 && a.ld_out % 8 == 0 &&
-         (!a.wide_gate || (((uintptr_t)a.gate % 8) == 0 && a.ld_gate % 2 == 0));
+         (!a.wide_gate || (((uintptr_t)a.gate % 16) == 0 && a.ld_gate % 4 == 0));
 }
 
 int k_launch_attn_fa(cg_ctx* c, const AttnArgs& a) {
@@ -469,7 +503,7 @@ int k_launch_attn_fa(cg_ctx* c, const AttnArgs& a) {
   // 64-key tiles: two CTAs per SM.  Head size 64 gains from it (8 x 1024 tokens, 64 heads: 380 -> 315 us,
   // with a window of 128 225 -> 165 us), head size 128 does not (242 -> 264 us).
   const bool k64 = c->opt_fa == 2 || a.d == 64;
-  if (a.bias) {
+  if (a.bias || (a.gate && a.wide_gate)) {
     if (a.d == 64) return launch_fa<64, 64, true>(c, a);
     return k64 ? launch_fa<128, 64, true>(c, a) : launch_fa<128, 128, true>(c, a);
   }

@@ -46,42 +46,35 @@ struct PrepSmem {
   static constexpr uint32_t QBYTES = 2 * QPART > CT * CHUNK_LD * 4 ? 2 * QPART : CT * CHUNK_LD * 4;
   static constexpr uint32_t A = Q + QBYTES;                      // [64][68] f32 | V [64][LE]
   static constexpr uint32_t P = A + CT * CHUNK_LD * 4;           // [64][68] f32 | T [2][64][LT]
-  static constexpr uint32_t ENDS = P + 2 * CT * LT * 2;          // [4][DK] f32
-  static constexpr uint32_t ROW = ENDS + 4 * DK * 4;             // beta, rq, rk [64] f32
+  static constexpr uint32_t ENDS = P + 2 * CT * LT * 2;          // [8][DK] f32
+  static constexpr uint32_t ROW = ENDS + 8 * DK * 4;             // beta, rq, rk [64] f32
   static constexpr uint32_t BYTES = ROW + 3 * CT * 4;
 };
 
 __device__ __forceinline__ float2 widen(uint32_t v) { return make_float2(__uint_as_float(v << 16), __uint_as_float(v & 0xffff0000u)); }
 
-// v[0] of lane l becomes the sum over all lanes of value l * N / 32 + (0 .. N / 32 - 1); N 32 or 16 (then two
-// neighbouring lanes get the same)
-template <int N>
+// v[0] of lane l becomes the sum over all lanes of value l / 2 of 16
 __device__ __forceinline__ void reduce_scatter(float* v, int lane) {
-  int n = N;
 #pragma unroll
-  for (int o = 16; o; o >>= 1) {
-    if (n > 1) {
-      n >>= 1;
-      const bool upper = lane & o;
+  for (int n = 8; n; n >>= 1) {
+    const bool upper = lane & (2 * n);
 #pragma unroll
-      for (int i = 0; i < N / 2; ++i)
-        if (i < n) {
-          const float send = upper ? v[i] : v[i + n], keep = upper ? v[i + n] : v[i];
-          v[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
-        }
-    } else {
-      v[0] += __shfl_xor_sync(0xffffffffu, v[0], o);
-    }
+    for (int i = 0; i < 8; ++i)
+      if (i < n) {
+        const float send = upper ? v[i] : v[i + n], keep = upper ? v[i + n] : v[i];
+        v[i] = keep + __shfl_xor_sync(0xffffffffu, send, 2 * n);
+      }
   }
+  v[0] += __shfl_xor_sync(0xffffffffu, v[0], 1);
 }
 
-// One block of 2 DK threads per (chunk, head).  A thread holds two neighbouring channels of 16 tokens: k and q
+// One block of 4 DK threads per (chunk, head).  A thread holds two neighbouring channels of 8 tokens: k and q
 // as they are, and the running sums L of the log decays inside those tokens.
 template <int DK, bool DELTA>
-__global__ void __launch_bounds__(2 * DK, DK == 128 ? 2 : 4) k_channel_prep(ChunkArgs a) {
+__global__ void __launch_bounds__(4 * DK, DK == 128 ? 2 : 4) k_channel_prep(ChunkArgs a) {
   using M = PrepSmem<DK>;
   using SC = Scratch<DK, DELTA>;
-  constexpr int NT = 2 * DK, NW = NT / 32, LK = M::LK;
+  constexpr int NT = 4 * DK, NW = NT / 32, LK = M::LK;
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
   asm volatile("griddepcontrol.wait;" ::: "memory");
   extern __shared__ __align__(16) uint8_t smem[];
@@ -94,17 +87,17 @@ __global__ void __launch_bounds__(2 * DK, DK == 128 ? 2 : 4) k_channel_prep(Chun
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int len = a.chunk_len[chunk];
   const int64_t m0 = a.chunk_tok[chunk];
-  const int c = 2 * (tid % (DK / 2)), qd = tid / (DK / 2), t0 = 16 * qd;
+  const int c = 2 * (tid % (DK / 2)), od = tid / (DK / 2), t0 = 8 * od;
 
-  uint32_t k[16], q[16];
-  float2 L[16];
+  uint32_t k[8], q[8];
+  float2 L[8];
   {
     const bool in_k = c < a.DKp, in_z = c < a.zs;
     const float coef = a.coef[h] * 1.4426950408889634f;
     float2 zb = make_float2(0.f, 0.f);
     if (in_z) zb = *(const float2*)(a.z_bias + h * a.zs + c);
 #pragma unroll
-    for (int i = 0; i < 16; ++i) {
+    for (int i = 0; i < 8; ++i) {
       const bool in = t0 + i < len;
       const int64_t m = m0 + (in ? t0 + i : 0);
       k[i] = in && in_k ? *(const uint32_t*)(a.k + m * a.ldq + (int64_t)kh * a.DKp + c) : 0;
@@ -113,14 +106,14 @@ __global__ void __launch_bounds__(2 * DK, DK == 128 ? 2 : 4) k_channel_prep(Chun
     }
     float2 sum = make_float2(0.f, 0.f);
 #pragma unroll
-    for (int i = 0; i < 16; ++i) {
+    for (int i = 0; i < 8; ++i) {
       if (t0 + i < len && in_z) {
         sum.x -= coef * softplus_f(a.z_sign * (L[i].x + zb.x));
         sum.y -= coef * softplus_f(a.z_sign * (L[i].y + zb.y));
       }
       L[i] = sum;
     }
-    *(float2*)(ends + qd * DK + c) = sum;
+    *(float2*)(ends + od * DK + c) = sum;
   }
   for (int t = tid; t < CT; t += NT) {
     const bool in = t < len;
@@ -130,49 +123,55 @@ __global__ void __launch_bounds__(2 * DK, DK == 128 ? 2 : 4) k_channel_prep(Chun
   }
   for (int i = tid; i < CT * CHUNK_LD; i += NT) sA[i] = sP[i] = 0.f;
   __syncthreads();
-  float2 end[4];  // the four quarters' sums
-#pragma unroll
-  for (int j = 0; j < 4; ++j) end[j] = *(const float2*)(ends + j * DK + c);
+  // the log decays of groups [from, to) of 8 tokens
+  auto between = [&](int from, int to) {
+    float2 v = make_float2(0.f, 0.f);
+    for (int j = from; j < to; ++j) {
+      const float2 e = *(const float2*)(ends + j * DK + c);
+      v.x += e.x; v.y += e.y;
+    }
+    return v;
+  };
 
   // pairs inside 8 tokens: rows T0 .. T1 - 1, of row t first t products of k and k, then t + 1 of q and k
-  auto inside = [&](auto blk_, auto t0_, auto t1_) {
-    constexpr int B8 = 8 * decltype(blk_)::value, T0 = decltype(t0_)::value, T1 = decltype(t1_)::value;
-    constexpr int N = T1 * T1 - T0 * T0, NP = N > 16 ? 32 : 16;
-    float v[NP];
+  auto inside = [&](auto t0_, auto t1_) {
+    constexpr int T0 = decltype(t0_)::value, T1 = decltype(t1_)::value;
+    constexpr int N = T1 * T1 - T0 * T0;
+    static_assert(N <= 16, "values of one reduction");
+    float v[16];
 #pragma unroll
-    for (int i = 0; i < NP; ++i) v[i] = 0.f;
+    for (int i = 0; i < 16; ++i) v[i] = 0.f;
 #pragma unroll
     for (int t = T0; t < T1; ++t) {
-      const float2 kt = widen(k[B8 + t]), qt = widen(q[B8 + t]);
+      const float2 kt = widen(k[t]), qt = widen(q[t]);
       float* row = v + (t * t - T0 * T0);
 #pragma unroll
       for (int s = 0; s <= t; ++s) {
-        float2 ks = widen(k[B8 + s]);
+        float2 ks = widen(k[s]);
         if (s < t) {
-          ks.x *= pow2(L[B8 + t].x - L[B8 + s].x);
-          ks.y *= pow2(L[B8 + t].y - L[B8 + s].y);
+          ks.x *= pow2(L[t].x - L[s].x);
+          ks.y *= pow2(L[t].y - L[s].y);
           if (DELTA) row[s] = kt.x * ks.x + kt.y * ks.y;
         }
         row[t + s] = qt.x * ks.x + qt.y * ks.y;
       }
     }
-    reduce_scatter<NP>(v, lane);
-    const int at = NP == 32 ? lane : lane >> 1;
-    if (at < N && (NP == 32 || !(lane & 1))) {
+    reduce_scatter(v, lane);
+    const int at = lane >> 1;
+    if (at < N && !(lane & 1)) {
       int t = T0;
       while ((t + 1) * (t + 1) - T0 * T0 <= at) ++t;
-      const int j = at - (t * t - T0 * T0), r = t0 + B8 + t;
+      const int j = at - (t * t - T0 * T0), r = t0 + t;
       // (at most two warps hold channels of the same tokens: their sum does not depend on their order)
-      if (j < t) atomicAdd(sA + r * CHUNK_LD + t0 + B8 + j, v[0]);
-      else atomicAdd(sP + r * CHUNK_LD + t0 + B8 + j - t, v[0]);
+      if (j < t) atomicAdd(sA + r * CHUNK_LD + t0 + j, v[0]);
+      else atomicAdd(sP + r * CHUNK_LD + t0 + j - t, v[0]);
     }
   };
-  inside(std::integral_constant<int, 0>(), std::integral_constant<int, 0>(), std::integral_constant<int, 5>());
-  inside(std::integral_constant<int, 0>(), std::integral_constant<int, 5>(), std::integral_constant<int, 7>());
-  inside(std::integral_constant<int, 0>(), std::integral_constant<int, 7>(), std::integral_constant<int, 8>());
-  inside(std::integral_constant<int, 1>(), std::integral_constant<int, 0>(), std::integral_constant<int, 5>());
-  inside(std::integral_constant<int, 1>(), std::integral_constant<int, 5>(), std::integral_constant<int, 7>());
-  inside(std::integral_constant<int, 1>(), std::integral_constant<int, 7>(), std::integral_constant<int, 8>());
+  inside(std::integral_constant<int, 0>(), std::integral_constant<int, 4>());
+  inside(std::integral_constant<int, 4>(), std::integral_constant<int, 5>());
+  inside(std::integral_constant<int, 5>(), std::integral_constant<int, 6>());
+  inside(std::integral_constant<int, 6>(), std::integral_constant<int, 7>());
+  inside(std::integral_constant<int, 7>(), std::integral_constant<int, 8>());
 
   auto put = [&](uint32_t at, uint32_t part, uint32_t v, float fx, float fy) {
     const float2 f = widen(v);
@@ -204,26 +203,17 @@ __global__ void __launch_bounds__(2 * DK, DK == 128 ? 2 : 4) k_channel_prep(Chun
   auto halving = [&](auto half_) {
     constexpr int HALF = decltype(half_)::value;
     __syncthreads();  // the buffers are read
+    constexpr int GROUPS = HALF / 8;
+    const bool upper = od & GROUPS;          // uniform over the warp
+    const int half0 = od & ~(GROUPS - 1);    // first group of this half
+    const float2 far = upper ? between(half0, od) : between(od + 1, half0 + GROUPS);
 #pragma unroll
-    for (int i = 0; i < 16; ++i) {
+    for (int i = 0; i < 8; ++i) {
       const int t = t0 + i;
-      const bool upper = HALF == 8 ? i >= 8 : (t & HALF) != 0;
-      float2 e;
-      if (HALF == 8) {
-        e = upper ? make_float2(L[i].x - L[7].x, L[i].y - L[7].y) : make_float2(L[7].x - L[i].x, L[7].y - L[i].y);
-      } else if (upper) {
-        e = L[i];
-        if (HALF == 32 && qd == 3) { e.x += end[2].x; e.y += end[2].y; }
-      } else {
-        e = make_float2(L[15].x - L[i].x, L[15].y - L[i].y);
-        if (HALF == 32 && qd == 0) { e.x += end[1].x; e.y += end[1].y; }
-      }
+      const float2 e = upper ? make_float2(far.x + L[i].x, far.y + L[i].y) : make_float2(far.x + (L[7].x - L[i].x), far.y + (L[7].y - L[i].y));
       const float fx = pow2(e.x), fy = pow2(e.y);
       if (DELTA || !upper) put(M::K + (uint32_t)(t * LK + c) * 2u, M::KPART, k[i], fx, fy);
-      if (upper) {
-        const int u = HALF == 32 ? t - 32 : HALF == 16 ? (qd >> 1) * 16 + i : qd * 8 + i - 8;
-        put(M::Q + (uint32_t)(u * LK + c) * 2u, M::QPART, q[i], fx, fy);
-      }
+      if (upper) put(M::Q + (uint32_t)(((t / (2 * HALF)) * HALF + (t & (HALF - 1))) * LK + c) * 2u, M::QPART, q[i], fx, fy);
     }
     __syncthreads();
     constexpr int UNITS = HALF == 16 ? 2 : 4;  // 16 x 16 (HALF 8: 8 x 8 inside) per operand
@@ -261,22 +251,18 @@ __global__ void __launch_bounds__(2 * DK, DK == 128 ? 2 : 4) k_channel_prep(Chun
   };
   {
     // to the chunk's start and to its end
-    float2 before = make_float2(0.f, 0.f), behind = make_float2(0.f, 0.f);
+    const float2 before = between(0, od), behind = between(od + 1, 8);
+    const float2 last = L[7];
 #pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      if (j < qd) { before.x += end[j].x; before.y += end[j].y; }
-      if (j > qd) { behind.x += end[j].x; behind.y += end[j].y; }
-    }
-#pragma unroll
-    for (int i = 0; i < 16; ++i) {
+    for (int i = 0; i < 8; ++i) {
       const int t = t0 + i;
       const float2 kf = widen(k[i]), qf = widen(q[i]);
       const float fx = pow2(before.x + L[i].x), fy = pow2(before.y + L[i].y);
       store(SC::QT, t, qf.x * (rq[t] * fx), qf.y * (rq[t] * fy));
-      store(SC::KD, t, kf.x * (rk[t] * pow2(behind.x + (L[15].x - L[i].x))), kf.y * (rk[t] * pow2(behind.y + (L[15].y - L[i].y))));
+      store(SC::KD, t, kf.x * (rk[t] * pow2(behind.x + (last.x - L[i].x))), kf.y * (rk[t] * pow2(behind.y + (last.y - L[i].y))));
       if (DELTA) L[i] = make_float2(rk[t] * fx, rk[t] * fy);  // from here on the factor of K~
     }
-    if (qd == 3) *(float2*)(a.decayed + ((int64_t)chunk * a.H + h) * DK + c) = make_float2(pow2(before.x + end[3].x), pow2(before.y + end[3].y));
+    if (od == 7) *(float2*)(a.decayed + ((int64_t)chunk * a.H + h) * DK + c) = make_float2(pow2(before.x + last.x), pow2(before.y + last.y));
   }
   __syncthreads();  // pair products are complete, K and Q read
   for (int i = tid; i < CT * CT / 2; i += NT) {
@@ -293,7 +279,7 @@ __global__ void __launch_bounds__(2 * DK, DK == 128 ? 2 : 4) k_channel_prep(Chun
   }
   if (!DELTA) return;
 #pragma unroll
-  for (int i = 0; i < 16; ++i) put(M::K + (uint32_t)((t0 + i) * LK + c) * 2u, M::KPART, k[i], L[i].x, L[i].y);
+  for (int i = 0; i < 8; ++i) put(M::K + (uint32_t)((t0 + i) * LK + c) * 2u, M::KPART, k[i], L[i].x, L[i].y);
   __syncthreads();
   float* X = (float*)(smem + M::Q);
   invert_unit_lower(sA, X, tid, NT);
@@ -587,7 +573,7 @@ int launch_channel(cg_ctx* c, const ChunkArgs& a) {
     CG_CUDA(c, cudaFuncSetAttribute(k_channel_scan<DK, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)walk));
     configured = true;
   }
-  CG_CUDA(c, launch_kernel(c, k_channel_prep<DK, DELTA>, dim3((unsigned)a.n_chunks, (unsigned)a.H), dim3(2 * DK), prep, 1, a));
+  CG_CUDA(c, launch_kernel(c, k_channel_prep<DK, DELTA>, dim3((unsigned)a.n_chunks, (unsigned)a.H), dim3(4 * DK), prep, 1, a));
   CG_LAUNCHED(c);
   dim3 grid((unsigned)((a.dv + EB - 1) / EB), (unsigned)a.H, (unsigned)a.rows.rows);
   CG_CUDA(c, launch_kernel(c, k_channel_scan<DK, DELTA>, grid, dim3(256), walk, 1, a));

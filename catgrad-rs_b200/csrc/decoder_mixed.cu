@@ -1052,7 +1052,7 @@ void recurrent_base(cg_decoder* D, const MixedLayer& L, MixedRun& run, const Row
 // Prompts in a bf16 context run in chunks on the tensor cores, from bf16 projections that the mixer makes itself
 bool in_chunks(const MixedLayer& L, const Portion* p) { return L.chunked && p && p->max_len >= 8; }
 
-int lru_layer(cg_decoder* D, const MixedLayer& L, MixedRun& run, const RowsDev& rd, const Portion* p, Rows in, Rows out) {
+int lru_layer(cg_decoder* D, const MixedLayer& L, MixedRun& run, const RowsDev& rd, const Portion* p, const Chunks* ch, Rows in, Rows out) {
   MixedModel& X = *D->mixed;
   LruArgs a{};
   const bool bf = in_chunks(L, p);
@@ -1073,6 +1073,7 @@ int lru_layer(cg_decoder* D, const MixedLayer& L, MixedRun& run, const RowsDev& 
   a.u = X.u->data(); a.a = (float*)X.lru_a->data(); a.b = (float*)X.lru_b->data();
   a.out = out.p; a.ld_out = out.ld; a.out_bf16 = X.f32 ? 0 : 1;
   a.rows = rd;
+  if (ch) { a.chunk_tok = ch->tok; a.chunk_len = ch->len; a.n_chunks = ch->n; }
   return !p || p->max_len == 1 ? k_launch_lru_decode(D->c, a) : k_launch_lru_prompt(D->c, a);
 }
 
@@ -1210,7 +1211,7 @@ int mixer(cg_decoder* D, const MixedLayer& L, MixedRun& run, const RowsDev& rd, 
         CG_TRY(lin(D, X.xn->data(), X.Wp, M, L.w_in, m.in_row, m.Np, in.p, m.Np));
       }
       if (m.k.mixer == CG_MIX_ATTENTION) CG_TRY(attention_layer(D, m, r, rd, p, in, out));
-      else if (m.lru()) CG_TRY(lru_layer(D, m, r, rd, p, in, out));
+      else if (m.lru()) CG_TRY(lru_layer(D, m, r, rd, p, ch, in, out));
       else CG_TRY(recurrent_layer(D, m, r, rd, p, ch, in, out));
     }
   }

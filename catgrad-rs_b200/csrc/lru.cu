@@ -31,6 +31,21 @@ __device__ __forceinline__ float2 gate_pair(float zr, float zi, float f, float u
   return make_float2(expf(la), sqrtf(-expm1f(2.f * la)) * sigmoid(zi) * u);
 }
 
+// The same for prompts in a bf16 context.  1 - a^2 = -(e^y - 1), y = 2 ln a, by its power series where
+// 1 - e^y would lose digits.
+__device__ __forceinline__ float2 gate_pair_fast(float zr, float zi, float f, float u) {
+  const float la = f * sigmoid_fast(zr), y = 2.f * la, a = __expf(la);
+  float p = fmaf(y, 1.f / 720.f, 1.f / 120.f);
+  p = fmaf(p, y, 1.f / 24.f);
+  p = fmaf(p, y, 1.f / 6.f);
+  p = fmaf(p, y, 0.5f);
+  p = fmaf(p, y, 1.f);
+  const float q = y > -0.25f ? -y * p : 1.f - a * a;
+  float s;
+  asm("sqrt.approx.ftz.f32 %0, %1;" : "=f"(s) : "f"(q));
+  return make_float2(a, s * sigmoid_fast(zi) * u);
+}
+
 // the convolution at channel c of token i of its row, whose first position is p0
 template <class TP>
 __device__ __forceinline__ float conv_at(const LruArgs& a, const TP* x, int64_t m, int i, int64_t p0, int c, const float* tail) {
@@ -62,6 +77,84 @@ __global__ void __launch_bounds__(128) k_lru_conv(LruArgs a) {
     const int row = a.rows.tok_row[m];
     const float* tail = a.tail + (int64_t)a.rows.slot[row] * a.taps * a.W;
     st((T*)a.u + m * a.W + c, conv_at(a, x, m, (int)(m - a.rows.start[row]), row_pos0(a.rows, row), c, tail));
+  }
+}
+
+// Channels in groups of 4 (bf16): a thread slides over 32 tokens of 4 channels, the next four tokens' inputs
+// requested while four are summed.
+constexpr int LV_TOK = 32;
+__device__ __forceinline__ void widen4(uint2 r, float* v) {
+  v[0] = __uint_as_float(r.x << 16); v[1] = __uint_as_float(r.x & 0xffff0000u);
+  v[2] = __uint_as_float(r.y << 16); v[3] = __uint_as_float(r.y & 0xffff0000u);
+}
+template <int TAPS>
+__global__ void __launch_bounds__(128) k_lru_conv_vec(LruArgs a) {
+  asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+  asm volatile("griddepcontrol.wait;" ::: "memory");
+  constexpr int G = 4, PER = RECUR_CHUNK / LV_TOK;
+  const int chunk = blockIdx.x / PER, t_lo = (blockIdx.x % PER) * LV_TOK;
+  const int n = min(LV_TOK, a.chunk_len[chunk] - t_lo), c = (blockIdx.y * 128 + threadIdx.x) * 4;
+  if (n <= 0 || c >= a.W) return;
+  const int64_t m0 = a.chunk_tok[chunk] + t_lo;
+  const int row = a.rows.tok_row[m0], i0 = (int)(m0 - a.rows.start[row]);
+  const int64_t p0 = row_pos0(a.rows, row);
+  const float* tail = a.tail + (int64_t)a.rows.slot[row] * a.taps * a.W + c;
+  const __nv_bfloat16* in = (const __nv_bfloat16*)a.x + m0 * a.ldx + c;
+  float w[TAPS][4], xb[4], cb[4];
+#pragma unroll
+  for (int e = 0; e < 4; ++e) {
+    xb[e] = a.xb[c + e];
+    cb[e] = a.conv_b[c + e];
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) w[j][e] = a.conv_w[(int64_t)(c + e) * TAPS + TAPS - 1 - j];
+  }
+  // x[TAPS - 1 + i]: the input of the group's token i; x[TAPS - 1 - j]: the one j tokens before the group
+  float x[TAPS - 1 + G][4];
+#pragma unroll
+  for (int j = 1; j < TAPS; ++j) {
+    float* v = x[TAPS - 1 - j];
+    v[0] = v[1] = v[2] = v[3] = 0.f;
+    if (j <= i0) {
+      widen4(*(const uint2*)(in - j * a.ldx), v);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) v[e] += xb[e];
+    } else if (p0 + i0 - j >= 0) {
+      const float* tp = tail + (int64_t)((p0 + i0 - j) % TAPS) * a.W;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) v[e] = tp[e];
+    }
+  }
+  uint2 raw[G];
+  auto fetch = [&](int t) {
+#pragma unroll
+    for (int i = 0; i < G; ++i) raw[i] = t + i < n ? *(const uint2*)(in + (int64_t)(t + i) * a.ldx) : make_uint2(0, 0);
+  };
+  fetch(0);
+  __nv_bfloat16* out = (__nv_bfloat16*)a.u + m0 * a.W + c;
+  for (int t = 0; t < n; t += G) {
+#pragma unroll
+    for (int i = 0; i < G; ++i) {
+      widen4(raw[i], x[TAPS - 1 + i]);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) x[TAPS - 1 + i][e] += xb[e];
+    }
+    fetch(t + G);
+#pragma unroll
+    for (int i = 0; i < G; ++i) {
+      float v[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        v[e] = cb[e];
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) v[e] = fmaf(w[j][e], x[TAPS - 1 + i - j][e], v[e]);
+      }
+      const __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
+      if (t + i < n) *(uint2*)(out + (int64_t)(t + i) * a.W) = make_uint2(*(const uint32_t*)&lo, *(const uint32_t*)&hi);
+    }
+#pragma unroll
+    for (int j = 0; j < TAPS - 1; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) x[j][e] = x[j + G][e];
   }
 }
 
@@ -193,8 +286,8 @@ __global__ void __launch_bounds__(256) k_lru_gates(LruArgs a) {
       const int64_t m = m0 + wm * 16 + (lane >> 2) + 8 * x;
       if (m >= a.rows.M) continue;
       const float2 uu = __bfloat1622float2(*(const __nv_bfloat162*)(u + m * a.W + c));
-      const float2 g0 = gate_pair(acc[0][j][2 * x] + br.x, acc[1][j][2 * x] + bi.x, f.x, uu.x);
-      const float2 g1 = gate_pair(acc[0][j][2 * x + 1] + br.y, acc[1][j][2 * x + 1] + bi.y, f.y, uu.y);
+      const float2 g0 = gate_pair_fast(acc[0][j][2 * x] + br.x, acc[1][j][2 * x] + bi.x, f.x, uu.x);
+      const float2 g1 = gate_pair_fast(acc[0][j][2 * x + 1] + br.y, acc[1][j][2 * x + 1] + bi.y, f.y, uu.y);
       *(float2*)(a.a + m * a.W + c) = make_float2(g0.x, g1.x);
       *(float2*)(a.b + m * a.W + c) = make_float2(g0.y, g1.y);
     }
@@ -264,62 +357,99 @@ __global__ void __launch_bounds__(32 * LS_SEG) k_lru_scan(LruArgs a) {
 
 // ----------------------------------------------------------------- one token per row ----
 // One block per (block of channels, 32 of its outputs, 8 rows): the convolution of the whole block of every
-// row in shared memory, a warp per 4 outputs, lanes over the inputs.
+// row in shared memory, a warp per 4 outputs of both gates, lanes over the inputs; the sums over the lanes
+// leave lane l with output l / 8 of row l % 8.  The first weights are requested before the wait.
 constexpr int LD_OUT = 32, LD_ROWS = 8;
 template <class T>
+__device__ __forceinline__ void load4(const T* p, bool in, float* v) {
+  if constexpr (sizeof(T) == 2) {
+    widen4(in ? *(const uint2*)p : make_uint2(0, 0), v);
+  } else {
+    const float4 f = in ? *(const float4*)p : make_float4(0.f, 0.f, 0.f, 0.f);
+    v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+  }
+}
+// VEC: blocks of a multiple of 4 channels
+template <class T, bool VEC>
 __global__ void __launch_bounds__(256) k_lru_decode(LruArgs a) {
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
-  extern __shared__ float su[];  // [LD_ROWS][n]
-  const int n = a.W / a.blocks, per = (n + LD_OUT - 1) / LD_OUT;
+  extern __shared__ __align__(16) float su[];  // [LD_ROWS][np], np = n rounded up to 128
+  const int n = a.W / a.blocks, np = (n + 127) / 128 * 128, per = (n + LD_OUT - 1) / LD_OUT;
   const int blk = blockIdx.x / per, e0 = (blockIdx.x - blk * per) * LD_OUT, r0 = blockIdx.y * LD_ROWS;
   const int rows = min(LD_ROWS, a.rows.rows - r0);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int o0 = e0 + warp * 4;                     // this warp's outputs inside the block
+  float w[2][4][4];                                 // [gate][output][input]
+  auto weights = [&](int k) {
+#pragma unroll
+    for (int o = 0; o < 4; ++o) {
+      const bool in = o0 + o < n && k < n;
+      const int64_t at = in ? (int64_t)(blk * n + o0 + o) * n + k : 0;
+#pragma unroll
+      for (int g = 0; g < 2; ++g) {
+        const T* p = (const T*)(g ? a.ri : a.ra) + at;
+        if constexpr (VEC) load4(p, in, w[g][o]);
+        else
+#pragma unroll
+          for (int e = 0; e < 4; ++e) w[g][o][e] = in && k + e < n ? ld(p + e) : 0.f;
+      }
+    }
+  };
+  weights(4 * lane);
   asm volatile("griddepcontrol.wait;" ::: "memory");
   const float* x = (const float*)a.x;
-  for (int i = tid; i < rows * n; i += 256) {
-    const int q = i / n, e = i - q * n, c = blk * n + e, row = r0 + q;
-    const int64_t pos = row_pos0(a.rows, row);
-    float* tail = a.tail + (int64_t)a.rows.slot[row] * a.taps * a.W;
-    const float now = x[(int64_t)row * a.ldx + c] + a.xb[c];
-    float v = a.conv_b[c] + a.conv_w[(int64_t)c * a.taps + a.taps - 1] * now;
-    for (int j = 1; j < a.taps; ++j)
-      if (pos - j >= 0) v += a.conv_w[(int64_t)c * a.taps + a.taps - 1 - j] * tail[(int64_t)((pos - j) % a.taps) * a.W + c];
-    if (e >= e0 && e < e0 + LD_OUT) tail[(int64_t)(pos % a.taps) * a.W + c] = now;  // read by no block of this step
-    su[i] = as(v, (const T*)nullptr);
+  for (int i = tid; i < LD_ROWS * np; i += 256) {
+    const int q = i / np, e = i - q * np, c = blk * n + e, row = r0 + q;
+    float v = 0.f;
+    if (q < rows && e < n) {
+      const int64_t pos = row_pos0(a.rows, row);
+      float* tail = a.tail + (int64_t)a.rows.slot[row] * a.taps * a.W;
+      const int ring = (int)((uint32_t)pos % (uint32_t)a.taps);
+      const float now = x[(int64_t)row * a.ldx + c] + a.xb[c];
+      v = a.conv_b[c] + a.conv_w[(int64_t)c * a.taps + a.taps - 1] * now;
+      for (int j = 1; j < a.taps; ++j)
+        if (pos >= j) v += a.conv_w[(int64_t)c * a.taps + a.taps - 1 - j] * tail[(int64_t)(ring >= j ? ring - j : ring - j + a.taps) * a.W + c];
+      if (e >= e0 && e < e0 + LD_OUT) tail[(int64_t)ring * a.W + c] = now;  // read by no block of this step
+      v = as(v, (const T*)nullptr);
+    }
+    su[i] = v;
   }
   __syncthreads();
-  for (int o = warp; o < LD_OUT && e0 + o < n; o += 8) {
-    const int c = blk * n + e0 + o;
-    float zr[LD_ROWS], zi[LD_ROWS];
+  if (o0 >= n) return;
+  float z[64];  // [output][row][gate]
 #pragma unroll
-    for (int q = 0; q < LD_ROWS; ++q) zr[q] = zi[q] = 0.f;
-    for (int k = lane; k < n; k += 32) {
-      const float wr = ld((const T*)a.ra + (int64_t)c * n + k), wi = ld((const T*)a.ri + (int64_t)c * n + k);
-#pragma unroll
-      for (int q = 0; q < LD_ROWS; ++q) {
-        const float v = q < rows ? su[q * n + k] : 0.f;
-        zr[q] += wr * v;
-        zi[q] += wi * v;
-      }
-    }
-    float r = 0.f, i = 0.f;   // of the row this lane finishes
+  for (int i = 0; i < 64; ++i) z[i] = 0.f;
+  for (int k0 = 0; k0 < n; k0 += 128) {
+    if (k0) weights(k0 + 4 * lane);
 #pragma unroll
     for (int q = 0; q < LD_ROWS; ++q) {
+      const float4 u = *(const float4*)(su + q * np + k0 + 4 * lane);
 #pragma unroll
-      for (int s = 16; s; s >>= 1) {
-        zr[q] += __shfl_xor_sync(0xffffffffu, zr[q], s);
-        zi[q] += __shfl_xor_sync(0xffffffffu, zi[q], s);
+      for (int o = 0; o < 4; ++o)
+#pragma unroll
+        for (int g = 0; g < 2; ++g)
+          z[(o * 8 + q) * 2 + g] += w[g][o][0] * u.x + w[g][o][1] * u.y + w[g][o][2] * u.z + w[g][o][3] * u.w;
+    }
+  }
+#pragma unroll
+  for (int step = 0; step < 5; ++step) {
+    const int off = 16 >> step, half = 32 >> step;  // values kept: half, the upper ones by lanes with this bit
+    const bool upper = lane & off;
+#pragma unroll
+    for (int i = 0; i < 32; ++i)
+      if (i < half) {
+        const float send = upper ? z[i] : z[i + half], keep = upper ? z[i + half] : z[i];
+        z[i] = keep + __shfl_xor_sync(0xffffffffu, send, off);
       }
-      if (lane == q) { r = zr[q]; i = zi[q]; }
-    }
-    if (lane < rows) {
-      const int row = r0 + lane;
-      float* Sg = a.S + (int64_t)a.rows.slot[row] * a.W + c;
-      const float2 g = gate_pair(r + a.ra_b[c], i + a.ri_b[c], a.f[c], su[lane * n + e0 + o]);
-      const float S = g.x * (row_pos0(a.rows, row) > 0 ? *Sg : 0.f) + g.y;
-      *Sg = S;
-      st((T*)a.out + (int64_t)row * a.ld_out + c, S * gelu_exact(((const float*)a.y)[(int64_t)row * a.ldx + c] + a.yb[c]));
-    }
+  }
+  const int e = o0 + (lane >> 3), q = lane & 7, c = blk * n + e;
+  if (e < n && q < rows) {
+    const int row = r0 + q;
+    float* Sg = a.S + (int64_t)a.rows.slot[row] * a.W + c;
+    const float2 g = gate_pair(z[0] + a.ra_b[c], z[1] + a.ri_b[c], a.f[c], su[q * np + e]);
+    const float S = g.x * (row_pos0(a.rows, row) > 0 ? *Sg : 0.f) + g.y;
+    *Sg = S;
+    st((T*)a.out + (int64_t)row * a.ld_out + c, S * gelu_exact(((const float*)a.y)[(int64_t)row * a.ldx + c] + a.yb[c]));
   }
 }
 
@@ -329,11 +459,13 @@ __global__ void __launch_bounds__(256) k_lru_decode(LruArgs a) {
 int k_launch_lru_decode(cg_ctx* c, const LruArgs& a) {
   if (a.rows.rows == 0) return CG_OK;
   const int n = a.W / a.blocks;
-  const size_t smem = (size_t)LD_ROWS * n * 4;
+  const size_t smem = (size_t)LD_ROWS * ((n + 127) / 128 * 128) * 4;
   if (smem > 200 * 1024) return fail(c, CG_ERR_UNSUPPORTED, "recurrence: gate blocks too wide");
-  auto kernel = a.out_bf16 ? k_lru_decode<__nv_bfloat16> : k_lru_decode<float>;
-  static PerDeviceSize configured_on[2];
-  size_t& configured = configured_on[a.out_bf16 ? 1 : 0].at(c->core->device);
+  const bool vec = n % 4 == 0;
+  auto kernel = a.out_bf16 ? (vec ? k_lru_decode<__nv_bfloat16, true> : k_lru_decode<__nv_bfloat16, false>)
+                           : (vec ? k_lru_decode<float, true> : k_lru_decode<float, false>);
+  static PerDeviceSize configured_on[4];
+  size_t& configured = configured_on[2 * (a.out_bf16 ? 1 : 0) + (vec ? 1 : 0)].at(c->core->device);
   if (smem > 48 * 1024 && smem > configured) {
     CG_CUDA(c, cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     configured = smem;
@@ -348,8 +480,14 @@ int k_launch_lru_prompt(cg_ctx* c, const LruArgs& a) {
   if (a.rows.M == 0) return CG_OK;
   const int n = a.W / a.blocks;
   const dim3 conv_grid((unsigned)((a.rows.M + LC_TOK - 1) / LC_TOK), (unsigned)((a.W + 127) / 128));
-  auto conv = !a.out_bf16 ? k_lru_conv<float, float> : a.in_bf16 ? k_lru_conv<__nv_bfloat16, __nv_bfloat16> : k_lru_conv<float, __nv_bfloat16>;
-  CG_CUDA(c, launch_kernel(c, conv, conv_grid, dim3(128), 0, 1, a));
+  if (a.in_bf16 && a.W % 4 == 0 && a.taps <= 4) {
+    const dim3 grid((unsigned)(a.n_chunks * (RECUR_CHUNK / LV_TOK)), (unsigned)((a.W + 511) / 512));
+    auto conv = a.taps == 1 ? k_lru_conv_vec<1> : a.taps == 2 ? k_lru_conv_vec<2> : a.taps == 3 ? k_lru_conv_vec<3> : k_lru_conv_vec<4>;
+    CG_CUDA(c, launch_kernel(c, conv, grid, dim3(128), 0, 1, a));
+  } else {
+    auto conv = !a.out_bf16 ? k_lru_conv<float, float> : a.in_bf16 ? k_lru_conv<__nv_bfloat16, __nv_bfloat16> : k_lru_conv<float, __nv_bfloat16>;
+    CG_CUDA(c, launch_kernel(c, conv, conv_grid, dim3(128), 0, 1, a));
+  }
   CG_LAUNCHED(c);
   if (a.taps > 1) {
     auto tail = a.in_bf16 ? k_lru_tail<__nv_bfloat16> : k_lru_tail<float>;

@@ -164,6 +164,8 @@ struct LruArgs {
   float *S, *tail;           // [slots, W], [slots, taps, W]
   void* u;                   // [M, W] scratch, prompts
   float *a, *b;              // [M, W] scratch, prompts
+  const int32_t *chunk_tok, *chunk_len;  // [n_chunks] first packed token, tokens (prompts)
+  int n_chunks;
   void* out;
   int64_t ld_out;
   int out_bf16;
@@ -301,6 +303,7 @@ struct RecurArgs : RecurBase {
   // [H zs, a_rank] and [H dv, g_rank] (f32 or bf16); w_g2 null: the gate is a segment of the projection
   int a1_off = 0, g1_off = 0, a_rank = 0, g_rank = 0, w_bf16 = 0;
   const void *w_a2 = nullptr, *w_g2 = nullptr;
+  int w_staged = 0;        // set by the launcher: a decode block keeps its rows of them in shared memory
 };
 // out[m, n] = sum over j of x[m, j] w[n, j] in f32, for the few columns of a low-rank projection; with coef
 // the log decay -coef[n / zs] softplus(sign (that + bias[n]))

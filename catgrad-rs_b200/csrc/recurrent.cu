@@ -6,6 +6,7 @@
 
 #include "act.cuh"
 #include "mixers.h"
+#include "mma.cuh"
 
 namespace cg {
 
@@ -190,32 +191,42 @@ __global__ void __launch_bounds__(128) k_recur_steps(RecurArgs a) {
 // ------------------------------------------------------------------ one token per row ----
 // One block per (head, row).  A thread keeps four columns of up to RD_ROWS rows of the state in
 // registers from the load to the store; sums over the key dimension go through shared memory.
-// KD: a decay per key channel; the second factors of the low-rank projections are applied here.
-template <class TW>
-__device__ __forceinline__ float low_rank_row(const float* x, const TW* w, int R) {
-  float v = 0.f;
-  if (sizeof(TW) == 2 && R % 8 == 0) {
-    for (int j = 0; j < R; j += 8) {
-      const uint4 r = *(const uint4*)(w + j);
-      const uint32_t p[4] = {r.x, r.y, r.z, r.w};
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const float2 f = __bfloat1622float2(*(const __nv_bfloat162*)&p[e]);
-        v += x[j + 2 * e] * f.x;
-        v += x[j + 2 * e + 1] * f.y;
-      }
-    }
-  } else {
-    for (int j = 0; j < R; ++j) v += x[j] * (float)w[j];
+// KD: a decay per key channel; the second factors of the low-rank projections are applied here, a row of them
+// per thread, from shared memory where they fit (rows R + 8 apart: no bank conflicts).
+__device__ __forceinline__ float low_rank_staged(const float* x, const __nv_bfloat16* w, int R) {
+  float v[2] = {0.f, 0.f};
+#pragma unroll 2
+  for (int j = 0; j < R; j += 8) {
+    const uint4 r = *(const uint4*)(w + j);
+    const float4 x0 = *(const float4*)(x + j), x1 = *(const float4*)(x + j + 4);
+    v[0] += x0.x * __uint_as_float(r.x << 16) + x0.y * __uint_as_float(r.x & 0xffff0000u);
+    v[1] += x0.z * __uint_as_float(r.y << 16) + x0.w * __uint_as_float(r.y & 0xffff0000u);
+    v[0] += x1.x * __uint_as_float(r.z << 16) + x1.y * __uint_as_float(r.z & 0xffff0000u);
+    v[1] += x1.z * __uint_as_float(r.w << 16) + x1.w * __uint_as_float(r.w & 0xffff0000u);
   }
-  return v;
+  return v[0] + v[1];
 }
 template <int RD_ROWS, bool KD>
 __global__ void __launch_bounds__(256, RD_ROWS <= 8 ? 3 : 2) k_recur_decode(RecurArgs a, GatedNorm n) {
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
   __shared__ float sq[128], sk[128], sv[128], so[128], sg[4];
   __shared__ float sd[KD ? 128 : 1], sgate[KD ? 128 : 1];  // decays, gates before their activation
-  extern __shared__ float low[];                           // KD: [a_rank], [g_rank]
+  // KD: [a_rank], [g_rank]; with w_staged then this head's rows of the second factors
+  extern __shared__ __align__(16) float low[];
+  __nv_bfloat16* const staged = (__nv_bfloat16*)(low + (a.a_rank + a.g_rank));  // (ranks are multiples of 8)
+  if (KD && a.w_staged) {
+    // weights: on their way while the projection still runs
+    const uint32_t to = (uint32_t)__cvta_generic_to_shared(staged);
+    const int na = a.dk * a.a_rank / 8, ng = a.w_g2 ? a.dv * a.g_rank / 8 : 0;
+    const __nv_bfloat16* wa = (const __nv_bfloat16*)a.w_a2 + (int64_t)blockIdx.x * a.zs * a.a_rank;
+    const __nv_bfloat16* wg = (const __nv_bfloat16*)a.w_g2 + (int64_t)blockIdx.x * a.dv * a.g_rank;
+    for (int i = threadIdx.x; i < na + ng; i += 256) {
+      const bool decay = i < na;
+      const int R8 = (decay ? a.a_rank : a.g_rank) / 8, x = decay ? i : i - na, r = x / R8;
+      cp_async16(to + (decay ? 0u : (uint32_t)(a.dk * (a.a_rank + 8)) * 2u) + (uint32_t)(r * (8 * R8 + 8) + (x - r * R8) * 8) * 2u,
+                 (decay ? wa : wg) + x * 8, 16);
+    }
+  }
   __shared__ __align__(16) float red[1024];
   const int h = blockIdx.x, row = blockIdx.y, rep = a.H / a.KH, kh = h / rep;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -235,6 +246,7 @@ __global__ void __launch_bounds__(256, RD_ROWS <= 8 ? 3 : 2) k_recur_decode(Recu
   // short convolutions of this head's channels
   const float* p = a.proj + m * a.ldp;
   float* tail = a.tail + (int64_t)slot * a.taps * a.C;
+  const int ring = a.taps ? (int)((uint32_t)pos % (uint32_t)a.taps) : 0;  // this position's place among the last inputs
   for (int x = tid; x < 2 * a.dk + a.dvs; x += 256) {
     const int seg = x < a.dk ? 0 : x < 2 * a.dk ? 1 : 2;
     const int e = seg == 0 ? x : seg == 1 ? x - a.dk : x - 2 * a.dk;
@@ -245,8 +257,8 @@ __global__ void __launch_bounds__(256, RD_ROWS <= 8 ? 3 : 2) k_recur_decode(Recu
     if (a.taps) {
       v = (a.conv_b ? a.conv_b[c] : 0.f) + a.conv_w[(int64_t)c * a.taps + a.taps - 1] * now;
       for (int j = 1; j < a.taps; ++j)
-        if (pos - j >= 0) v += a.conv_w[(int64_t)c * a.taps + a.taps - 1 - j] * tail[(int64_t)((pos - j) % a.taps) * a.C + c];
-      if (seg == 2 || h % rep == 0) tail[(int64_t)(pos % a.taps) * a.C + c] = now;  // read by no block of this step
+        if (pos >= j) v += a.conv_w[(int64_t)c * a.taps + a.taps - 1 - j] * tail[(int64_t)(ring >= j ? ring - j : ring - j + a.taps) * a.C + c];
+      if (seg == 2 || h % rep == 0) tail[(int64_t)ring * a.C + c] = now;  // read by no block of this step
     }
     if (a.linear) v *= seg == 0 ? a.q_scale : 1.f;
     else v = silu(v);
@@ -256,18 +268,26 @@ __global__ void __launch_bounds__(256, RD_ROWS <= 8 ? 3 : 2) k_recur_decode(Recu
     for (int j = tid; j < a.a_rank; j += 256) low[j] = p[a.a1_off + j];
     if (a.w_g2)
       for (int j = tid; j < a.g_rank; j += 256) low[a.a_rank + j] = p[a.g1_off + j];
+    cp_async_wait_all();
     __syncthreads();
-    auto product = [&](const void* w, int64_t row, const float* x, int R) {
-      return a.w_bf16 ? low_rank_row(x, (const __nv_bfloat16*)w + row * R, R) : low_rank_row(x, (const float*)w + row * R, R);
-    };
+#pragma unroll 1
     for (int e = tid; e < a.dk + a.dv; e += 256) {
-      if (e < a.dk) {
-        const int64_t r = (int64_t)h * a.zs + e;
-        sd[e] = expf(-a.coef[h] * softplus(a.z_sign * (product(a.w_a2, r, low, a.a_rank) + a.z_bias[r])));
+      const bool decay = e < a.dk;
+      const int64_t r = decay ? (int64_t)h * a.zs + e : (int64_t)h * a.dv + e - a.dk;
+      const int R = decay ? a.a_rank : a.g_rank;
+      const float* x = decay ? low : low + a.a_rank;
+      float v = 0.f;
+      if (!decay && !a.w_g2) {
+        v = ((const float*)n.gate)[m * n.ldg + r];
+      } else if (a.w_staged) {
+        v = low_rank_staged(x, staged + (decay ? e * (R + 8) : a.dk * (a.a_rank + 8) + (e - a.dk) * (R + 8)), R);
       } else {
-        const int64_t r = (int64_t)h * a.dv + e - a.dk;
-        sgate[e - a.dk] = a.w_g2 ? product(a.w_g2, r, low + a.a_rank, a.g_rank) : ((const float*)n.gate)[m * n.ldg + r];
+        const void* w = decay ? a.w_a2 : a.w_g2;
+#pragma unroll 1
+        for (int j = 0; j < R; ++j) v += x[j] * (a.w_bf16 ? __bfloat162float(((const __nv_bfloat16*)w)[r * R + j]) : ((const float*)w)[r * R + j]);
       }
+      if (decay) sd[e] = expf(-a.coef[h] * softplus(a.z_sign * (v + a.z_bias[r])));
+      else sgate[e - a.dk] = v;
     }
   }
   const float* sp = p + a.small_off;
@@ -478,6 +498,8 @@ int launch_gated_norm(cg_ctx* c, const GatedNorm& a) {
 
 }  // namespace
 
+constexpr size_t LOW_RANK_SMEM = 70 * 1024;  // of a decode block: three share an SM
+
 bool recur_decode_supported(int dk, int dv) { return dk <= 128 && dv <= 128; }
 
 int k_launch_recur_decode(cg_ctx* c, const RecurArgs& a, const GatedNorm& n) {
@@ -485,9 +507,21 @@ int k_launch_recur_decode(cg_ctx* c, const RecurArgs& a, const GatedNorm& n) {
   const int rpp = 256 / (a.dvs / 4);  // state rows per pass
   const bool few = (a.dk + rpp - 1) / rpp <= 8;
   auto kernel = a.key_decay ? (few ? k_recur_decode<8, true> : k_recur_decode<16, true>) : few ? k_recur_decode<8, false> : k_recur_decode<16, false>;
-  const size_t smem = a.key_decay ? (size_t)(a.a_rank + a.g_rank) * 4 : 0;
+  RecurArgs args = a;
+  size_t smem = a.key_decay ? (size_t)(a.a_rank + a.g_rank) * 4 : 0;
   if (smem > 32 * 1024) return fail(c, CG_ERR_UNSUPPORTED, "recurrence: low-rank projections too wide");
-  CG_CUDA(c, launch_kernel(c, kernel, dim3((unsigned)a.H, (unsigned)a.rows.rows), dim3(256), smem, 1, a, n));
+  if (a.key_decay && a.w_bf16) {
+    const size_t rows = ((size_t)a.dk * (a.a_rank + 8) + (a.w_g2 ? (size_t)a.dv * (a.g_rank + 8) : 0)) * 2;
+    args.w_staged = a.a_rank % 8 == 0 && a.g_rank % 8 == 0 && smem + rows <= LOW_RANK_SMEM;
+    if (args.w_staged) smem += rows;
+    static PerDeviceFlag configured_on[2];
+    bool& configured = configured_on[few ? 1 : 0].at(c->core->device);
+    if (!configured) {
+      CG_CUDA(c, cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)LOW_RANK_SMEM));
+      configured = true;
+    }
+  }
+  CG_CUDA(c, launch_kernel(c, kernel, dim3((unsigned)a.H, (unsigned)a.rows.rows), dim3(256), smem, 1, args, n));
   CG_LAUNCHED(c);
   return a.delta || a.key_decay ? CG_OK : k_launch_gated_norm(c, n);
 }
