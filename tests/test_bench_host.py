@@ -46,11 +46,17 @@ def test_layered_workloads_count_looped_layers():
         if not cfg.loop:
             # a layer with another one's weights counts them again
             own = dataclasses.replace(cfg, layers=[dataclasses.replace(L, weights_of=None) for L in cfg.layers])
-            assert any(L.weights_of is not None for L in cfg.layers)
+            assert any(L.weights_of is not None for L in cfg.layers) == (cfg.design is layered.DESIGNS["Regupel"])
             assert bench.layered_step_bytes(own, batch, prompt) == bench.layered_step_bytes(cfg, batch, prompt)
             assert all(v > 0 for v in bench.layered_step_bytes(cfg, batch, prompt).values())
             continue
         once = bench.layered_step_bytes(dataclasses.replace(cfg, loop=None), batch, prompt)
         looped = bench.layered_step_bytes(cfg, batch, prompt)
         assert all(looped[k] > once[k] > 0 for k in once if k != "states" or cfg.recurrent)
+    # experts without gates are two matrices each; block-diagonal gates count
+    cfg = layered.KIVORAX_W1024
+    plain = dataclasses.replace(cfg, layers=[dataclasses.replace(L, experts=None) if L.experts else L for L in cfg.layers])
+    a, b = (bench.layered_step_bytes(c, 8, 512)["weights"] for c in (cfg, plain))
+    more = sum(4 * 1024 * L.ffn * bench.experts_reached(32, 4, 8) + 2 * 32 * 1024 - 4 * 1024 * L.ffn for L in cfg.layers if L.experts)
+    assert abs(a - b - more) < 1
     assert abs(bench.experts_reached(64, 64, 3) - 64) < 1e-9 and abs(bench.experts_reached(64, 1, 1) - 1) < 1e-9

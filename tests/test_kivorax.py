@@ -9,6 +9,7 @@ the decoder's entry points.
 Errors are measured as in test_hybrid.py.  In a bf16 context a token whose choice of experts is a close
 call may choose otherwise, so such tokens are left out there.
 """
+import functools
 import importlib
 import json
 import os
@@ -447,14 +448,11 @@ def rounded(w):
     return cg.synth.bf16_round(np.asarray(w, np.float32))
 
 
-@gpu
-@pytest.mark.parametrize("prec", ["f32", "bf16"])
-@pytest.mark.parametrize("how", ["prompt", "decode", "portion", "short"])
-@pytest.mark.parametrize("dim,vdim,slope", [(24, 20, 1.0), (64, 64, 0.2), (64, 128, 1.5), (128, 128, 1.0), (96, 256, 0.7), (300, 40, 1.0)])
-def test_far_keys(backends, dim, vdim, slope, how, prec):
-    """The last token looks for one key, which stands out at every distance of interest: near, at the borders of
-    key tiles, at the start.  A nearer token with the same key and another value competes with it by the
-    distance alone."""
+@functools.lru_cache(maxsize=None)
+def far_keys(dim, vdim, slope):
+    """A model, its weights and (distance, tokens, the oracle's last logits): the last token looks for one key,
+    which stands out at every distance of interest: near, at the borders of key tiles, at the start.  A
+    nearer token with the same key and another value competes with it by the distance alone."""
     cfg = model([par(heads=2, kv_heads=1, dim=dim, vdim=vdim, scale=1.0, temp=(0.3, 100), width=8, blocks=2)], side=0)
     W, n, p, rng = weights(cfg, 11), 450, "l0.mix.left.", np.random.default_rng(5)
     asks, sought, rival = 103, 102, 101
@@ -463,7 +461,7 @@ def test_far_keys(backends, dim, vdim, slope, how, prec):
     W[p + "q"] = rounded(np.outer(np.concatenate([k, k]) * 14.0 / (k @ k), telling(cfg, W, {asks: 1, sought: 0, rival: 0})))
     W[p + "r1"], W[p + "r2"] = np.asarray([slope, 0.3 * slope], np.float32), np.asarray([0.3, 0.05], np.float32)
     W["l0.mix.right.out"] *= 0.1
-    dec = decoder(backends[prec], cfg, W)
+    cases = []
     for back in (1, 2, 31, 32, 63, 64, 65, 127, 128, 129, 300, 449):
         seq = np.random.default_rng(back).integers(0, len(QUIET), n)
         seq[n - 1], seq[n - 1 - back] = asks, sought
@@ -475,7 +473,27 @@ def test_far_keys(backends, dim, vdim, slope, how, prec):
         assert err(oracle.forward(cfg, W, swapped)[-1], want) > TOL["bf16"]
         if back > 64:
             assert err(oracle.forward(cfg, W, seq, faults=("no_distance",))[-1], want) > 300 * TOL["f32"]
-        assert close(play(dec, seq, how), want, prec), back
+        cases.append((back, seq, want))
+    return cfg, W, cases
+
+
+FAR = [(24, 20, 1.0), (64, 64, 0.2), (64, 128, 1.5), (128, 128, 1.0), (96, 256, 0.7), (300, 40, 1.0)]
+
+
+@pytest.mark.parametrize("sizes", FAR)
+def test_far_keys_decide(sizes):
+    far_keys(*sizes)
+
+
+@gpu
+@pytest.mark.parametrize("prec", ["f32", "bf16"])
+@pytest.mark.parametrize("sizes", FAR)
+def test_far_keys(backends, sizes, prec):
+    cfg, W, cases = far_keys(*sizes)
+    dec = decoder(backends[prec], cfg, W)
+    for back, seq, want in cases:
+        for how in ("prompt", "decode", "portion", "short"):
+            assert close(play(dec, seq, how), want, prec), (back, how)
     dec.close()
 
 
