@@ -58,9 +58,9 @@ __device__ __forceinline__ float softplus_f(float x) {
   p = fmaf(p, q, 1.f);
   return fmaxf(x, 0.f) + 2.f * s * p;
 }
-// tanh-gelu on accurate exponentials
+// tanh-gelu on accurate exponentials; (1 + tanh u) / 2 as a sigmoid keeps its digits where u is far below 0
 __device__ __forceinline__ float gelu_exact(float x) {
-  return 0.5f * x * (1.f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
+  return x / (1.f + expf(-1.5957691216057308f * (x + 0.044715f * x * x * x)));
 }
 
 }  // namespace cg

@@ -180,26 +180,29 @@ __global__ void k_depth_update(DepthUpdate u, int32_t* err) {
 
 __device__ __forceinline__ float gelu_as(float x, const float*) { return gelu_exact(x); }
 __device__ __forceinline__ float gelu_as(float x, const __nv_bfloat16*) { return gelu_fast(x); }
-__device__ __forceinline__ void st(float* p, float v) { *p = v; }
-__device__ __forceinline__ void st(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
-
-// out[m, j] = gelu(z[m, j]) * table[token, off + j], zero past n
+// out[m, j] = gelu(z[m, j]) * table[token, off + j], zero past n.  `per` threads per token, neighbouring columns per
+// thread.
+__device__ __forceinline__ void st2(float* p, float a, float b) { *(float2*)p = make_float2(a, b); }
+__device__ __forceinline__ void st2(__nv_bfloat16* p, float a, float b) { *(__nv_bfloat162*)p = __floats2bfloat162_rn(a, b); }
 template <class T>
-__global__ void k_token_gate(TokenGate a, int64_t M, int32_t* err) {
+__global__ void __launch_bounds__(256) k_token_gate(TokenGate a, int64_t M, int per, int32_t* err) {
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
   asm volatile("griddepcontrol.wait;" ::: "memory");
-  const int64_t total = M * a.ldo;
-  for (int64_t i = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; i < total; i += (int64_t)gridDim.x * blockDim.x) {
-    const int64_t m = i / a.ldo;
-    const int j = (int)(i - m * a.ldo);
-    float v = 0.f;
-    if (j < a.n) {
-      uint32_t tok = a.tokens[m];
-      if (tok >= a.vocab) { *err = DEV_INDEX; tok = 0; }
-      const float e = (float)((const T*)a.table)[(int64_t)tok * a.ld_table + a.off + j];
-      v = gelu_as(a.z[m * a.ldz + j], (const T*)nullptr) * e;
-    }
-    st((T*)a.out + i, v);
+  const int sub = threadIdx.x / per, t = threadIdx.x - sub * per;
+  const int64_t m = (int64_t)blockIdx.x * (blockDim.x / per) + sub;
+  if (m >= M) return;
+  uint32_t tok = a.tokens[m];
+  if (tok >= a.vocab) {
+    if (t == 0) *err = DEV_INDEX;
+    tok = 0;
+  }
+  const T* e = (const T*)a.table + (int64_t)tok * a.ld_table + a.off;
+  T* out = (T*)a.out + m * a.ldo;
+#pragma unroll 4
+  for (int j = 2 * t; j < a.ldo; j += 2 * per) {
+    const float2 z = *(const float2*)(a.z + m * a.ldz + j);
+    const float e0 = j < a.n ? (float)e[j] : 0.f, e1 = j + 1 < a.n ? (float)e[j + 1] : 0.f;
+    st2(out + j, gelu_as(z.x, (const T*)nullptr) * e0, gelu_as(z.y, (const T*)nullptr) * e1);
   }
 }
 
@@ -253,7 +256,9 @@ int k_launch_depth_update(cg_ctx* c, const DepthUpdate& u, int64_t M, int bf16) 
 int k_launch_token_gate(cg_ctx* c, const TokenGate& a, int64_t M, int bf16) {
   if (M == 0) return CG_OK;
   auto kernel = bf16 ? k_token_gate<__nv_bfloat16> : k_token_gate<float>;
-  CG_CUDA(c, launch_kernel(c, kernel, dim3(grid_for(M * a.ldo, 256)), dim3(256), 0, 1, a, M, c->core->dev_err));
+  if (a.ldo % 2 || a.ldz % 2) return fail(c, CG_ERR_INVALID, "decoder: token inputs must be padded to pairs");
+  const int per = M <= 296 ? 128 : 32, block = M <= 296 ? 128 : 256;
+  CG_CUDA(c, launch_kernel(c, kernel, dim3((unsigned)((M + block / per - 1) / (block / per))), dim3(block), 0, 1, a, M, per, c->core->dev_err));
   CG_LAUNCHED(c);
   return CG_OK;
 }
